@@ -36,6 +36,7 @@ class ModelLoadOptions:
     max_batch: int = 8
     max_seq_len: int = 4096
     kv_pages: Optional[int] = None
+    state_slots: Optional[int] = None    # recurrent-state slots of hybrid models (None: twice the decode batch)
     prefix_cache: bool = False           # later requests lease the published KV pages of an equal prompt prefix
     kv_host_tier_bytes: int = 0          # with prefix_cache: evicted published pages are kept in pinned host memory ...
     kv_disk_tier_dir: Optional[str] = None   # ... and spilled to files in this directory when the host tier is full
@@ -225,7 +226,7 @@ class LoadedModel:
         engine = Engine(model, max_batch=opt.max_batch, max_seq_len=opt.max_seq_len, num_pages=opt.kv_pages,
                         use_cuda_graph=opt.use_cuda_graph, prefix_cache=opt.prefix_cache,
                         kv_host_tier_bytes=opt.kv_host_tier_bytes, kv_disk_tier_dir=opt.kv_disk_tier_dir,
-                        kv_disk_tier_bytes=opt.kv_disk_tier_bytes)
+                        kv_disk_tier_bytes=opt.kv_disk_tier_bytes, state_slots=opt.state_slots)
         tokenizer = None
         try:
             from ..text.tokenizer import load_tokenizer

@@ -74,7 +74,15 @@ def host_sources() -> list[Path]:
     return sorted((CSRC / "host").glob("*.cpp"))
 
 
-def build_cuda(verbose: bool = False) -> Path:
+# Kernel sources a family needs when only it is to run (see ensure_family); every other use builds all of them.
+FAMILY_SOURCES = {
+    "nidozen": ("attention", "attention_tc", "gemm_persistent", "gemm_tcgen05", "gla", "launch_count", "mingru",
+                "residual_stream", "simt_fp32"),
+}
+
+
+def build_cuda(verbose: bool = False, sources: list[Path] | None = None, out: Path | None = None) -> Path:
+    """All CUDA sources into liberedu_cuda.so, or ``sources`` into ``out``."""
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found: cannot build liberedu_cuda.so")
@@ -82,7 +90,7 @@ def build_cuda(verbose: bool = False) -> Path:
     LIB.mkdir(exist_ok=True)
     jobs = []
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as pool:
-        for src in cuda_sources():
+        for src in sources or cuda_sources():
             obj = OBJ / (src.stem + ".o")
             cmd = [nvcc, *NVCC_FLAGS, "-c", str(src), "-o", str(obj)]
             jobs.append(pool.submit(_compile, cmd, src, obj, _digest(src, " ".join(NVCC_FLAGS)), verbose))
@@ -92,7 +100,7 @@ def build_cuda(verbose: bool = False) -> Path:
             objs.append(obj)
             if log:
                 print(log, file=sys.stderr)
-    out = LIB / "liberedu_cuda.so"
+    out = out or LIB / "liberedu_cuda.so"
     newest = max(o.stat().st_mtime for o in objs)
     if not out.exists() or out.stat().st_mtime < newest:
         cmd = [nvcc, "-shared", "-o", str(out), *map(str, objs)]
@@ -127,6 +135,22 @@ def build_host(verbose: bool = False) -> Path:
         if proc.returncode != 0:
             raise RuntimeError(f"link failed: {proc.stderr}")
     return out
+
+
+def ensure_family(family: str) -> Path:
+    """Bring the native code up to date for running one model family and return the CUDA library to load: the complete
+    library where it has been built before (sources that changed are recompiled), else a library of the kernels this family
+    uses. Safe against concurrent callers."""
+    import fcntl
+
+    OBJ.mkdir(exist_ok=True)
+    with open(OBJ / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        build_host()
+        if family not in FAMILY_SOURCES or (LIB / "liberedu_cuda.so").exists():
+            return build_cuda()
+        return build_cuda(sources=[CSRC / "kernels" / (n + ".cu") for n in FAMILY_SOURCES[family]],
+                          out=LIB / f"liberedu_{family}.so")
 
 
 def build_all(verbose: bool = False) -> None:

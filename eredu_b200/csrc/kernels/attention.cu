@@ -36,6 +36,8 @@ struct AttnParams {
   int t0, t_count;  // decode: token sub-range handled by this launch
   int splits;
   int window;  // 0 = full attention, else sliding window width
+  int chunk;   // decode: > 0 = a query sees the keys of its own chunk of positions only
+  int dk, dv;  // decode: stored key / value width of a head (multiples of 8; the tiles are padded to 64 or 128)
   float scale_log2;  // softmax scale * log2(e)
   // Decode with the projection output taken as is (qkv != null): the kernel applies the per-head q/k RMSNorm and RoPE
   // itself and appends the new K/V rows to their pages, so no separate RoPE / append launch precedes it.
@@ -143,6 +145,12 @@ __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1
 template <int D>
 __device__ __forceinline__ uint32_t swz(int r, int c) {
   return static_cast<uint32_t>(r * (D * 2) + (((c & ~7) | ((c ^ r) & 7)) << 4));
+}
+
+// First key position a query at `pos` can see.
+__device__ __forceinline__ int lowest_key(const AttnParams& p, int pos) {
+  if (p.window > 0) return pos - p.window + 1;
+  return p.chunk > 0 ? pos - pos % p.chunk : 0;
 }
 
 // ============================================================================ prefill
@@ -342,17 +350,20 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(AttnParams p) {
 // grid (splits, n_kv_heads, B). The MT*16 MMA rows hold (query token t, head-in-group g) pairs,
 // row = (t - t0) * group + g. Each of the 4 warps streams every 4th page through its own 3-stage
 // cp.async ring and keeps private (m, l, O); the warps are merged through shared memory at the end.
-template <int D, int MT>
+// Keys and values may differ in width: tiles are DK / DV wide (64 or 128), rows of the cache p.dk / p.dv (the rest of a
+// tile row is zero-filled, which adds nothing to scores or outputs).
+template <int DK, int DV, int MT>
 __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
-  constexpr int CH = D / 8;
-  constexpr int KS = D / 16;
+  constexpr int CHK = DK / 8, CHV = DV / 8;
+  constexpr int KS = DK / 16;
   constexpr int NSTAGE = 3;
   constexpr int ROWS = 16 * MT;
-  constexpr int PAGE_BYTES = kPage * D * 2;
+  constexpr int KPAGE_BYTES = kPage * DK * 2;
+  constexpr int STAGE_BYTES = kPage * (DK + DV) * 2;
   extern __shared__ __align__(128) uint8_t smem[];
-  uint8_t* q_s = smem;                   // [ROWS][D] bf16
-  uint8_t* newkv_s = smem + ROWS * D * 2;                    // [kMaxFusedNew][K row, V row] bf16 (fused path)
-  uint8_t* ring = newkv_s + kMaxFusedNew * 2 * D * 2;        // [4 warps][NSTAGE][K page, V page]
+  uint8_t* q_s = smem;                   // [ROWS][DK] bf16
+  uint8_t* newkv_s = smem + ROWS * DK * 2;                   // [kMaxFusedNew][K row, V row] bf16 (fused path)
+  uint8_t* ring = newkv_s + kMaxFusedNew * (DK + DV) * 2;    // [4 warps][NSTAGE][K page, V page]
 
   __shared__ int s_last;
   pdl_launch_early();
@@ -368,9 +379,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   pdl_launch_dependents();
   const int kv_len = p.seq_lens[b];
   const int npages = (kv_len + kPage - 1) / kPage;
-  int pps = (npages + p.splits - 1) / p.splits;
+  // pages before the first query's window / chunk hold nothing any query of this launch can see
+  const int first_pos = kv_len - p.q_per_seq + p.t0;
+  const int first_page = max(0, lowest_key(p, first_pos)) / kPage;
+  int pps = (npages - first_page + p.splits - 1) / p.splits;
   pps = (pps + 3) & ~3;
-  const int page0 = split * pps;
+  const int page0 = first_page + split * pps;
   const int page1 = min(npages, page0 + pps);
 
   const bool fused = p.qkv != nullptr;
@@ -381,41 +395,46 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   const int new_pos0 = kv_len - p.q_per_seq;
   const int first_new_page = appending ? new_pos0 / kPage : 0x7fffffff;
   if (!fused) {
-    for (int i = threadIdx.x; i < ROWS * CH; i += 128) {
-      const int r = i / CH, c = i % CH;
-      const bool ok = r < rows;
-      const int t = p.t0 + (ok ? r / group : 0), hg = ok ? r % group : 0;
+    for (int i = threadIdx.x; i < ROWS * CHK; i += 128) {
+      const int r = i / CHK, c = i % CHK;
+      const bool ok = r < rows && c * 8 < p.dk;
+      const int t = p.t0 + (r < rows ? r / group : 0), hg = r < rows ? r % group : 0;
       const __nv_bfloat16* src =
-          p.q + (static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + kvh * group + hg) * D + c * 8;
-      cp_async16(q_s + swz<D>(r, c), src, ok ? 16 : 0);
+          p.q + (static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + kvh * group + hg) * p.dk + (ok ? c * 8 : 0);
+      cp_async16(q_s + swz<DK>(r, c), src, ok ? 16 : 0);
     }
   }
   cp_async_commit();
 
-  uint8_t* my_ring = ring + warp * NSTAGE * 2 * PAGE_BYTES;
+  uint8_t* my_ring = ring + warp * NSTAGE * STAGE_BYTES;
   auto load_page = [&](int pg, int stage) {
     if (pg < page1) {
       const int phys = bt[pg];
-      const __nv_bfloat16* ksrc = p.k_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * D;
-      const __nv_bfloat16* vsrc = p.v_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * D;
-      uint8_t* kd = my_ring + stage * 2 * PAGE_BYTES;
-      uint8_t* vd = kd + PAGE_BYTES;
-      for (int i = lane; i < kPage * CH; i += 32) {
-        const int r = i / CH, c = i % CH;
-        cp_async16(kd + swz<D>(r, c), ksrc + r * D + c * 8, 16);
-        cp_async16(vd + swz<D>(r, c), vsrc + r * D + c * 8, 16);
+      const __nv_bfloat16* ksrc = p.k_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * p.dk;
+      const __nv_bfloat16* vsrc = p.v_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * p.dv;
+      uint8_t* kd = my_ring + stage * STAGE_BYTES;
+      uint8_t* vd = kd + KPAGE_BYTES;
+      for (int i = lane; i < kPage * CHK; i += 32) {
+        const int r = i / CHK, c = i % CHK;
+        const bool in = c * 8 < p.dk;
+        cp_async16(kd + swz<DK>(r, c), ksrc + r * p.dk + (in ? c * 8 : 0), in ? 16 : 0);
+      }
+      for (int i = lane; i < kPage * CHV; i += 32) {
+        const int r = i / CHV, c = i % CHV;
+        const bool in = c * 8 < p.dv;
+        cp_async16(vd + swz<DV>(r, c), vsrc + r * p.dv + (in ? c * 8 : 0), in ? 16 : 0);
       }
     }
   };
 
-  float o[MT][D / 8][4];
+  float o[MT][DV / 8][4];
   float m_run[MT][2], l_run[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
     m_run[mt][0] = m_run[mt][1] = -INFINITY;
     l_run[mt][0] = l_run[mt][1] = 0.f;
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
+    for (int i = 0; i < DV / 8; ++i) o[mt][i][0] = o[mt][i][1] = o[mt][i][2] = o[mt][i][3] = 0.f;
   }
 
   const int first = page0 + warp;
@@ -427,16 +446,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     // ---- q rows: norm + RoPE straight into the swizzled tile (rows beyond `rows` are zero)
     for (int r = warp; r < ROWS; r += 4) {
       auto put = [&](int i0, float a, int i1, float bb) {
-        *reinterpret_cast<__nv_bfloat16*>(q_s + swz<D>(r, i0 >> 3) + (i0 & 7) * 2) = __float2bfloat16(a);
-        *reinterpret_cast<__nv_bfloat16*>(q_s + swz<D>(r, i1 >> 3) + (i1 & 7) * 2) = __float2bfloat16(bb);
+        *reinterpret_cast<__nv_bfloat16*>(q_s + swz<DK>(r, i0 >> 3) + (i0 & 7) * 2) = __float2bfloat16(a);
+        *reinterpret_cast<__nv_bfloat16*>(q_s + swz<DK>(r, i1 >> 3) + (i1 & 7) * 2) = __float2bfloat16(bb);
       };
       if (r < rows) {
         const int t = p.t0 + r / group, hg = r % group;
         const size_t m = static_cast<size_t>(b) * p.q_per_seq + t;
-        rope_head_row<D>(p, p.qkv + m * p.ld_qkv + static_cast<size_t>(kvh * group + hg) * D, p.q_norm_w, p.positions[m],
+        rope_head_row<DK>(p, p.qkv + m * p.ld_qkv + static_cast<size_t>(kvh * group + hg) * DK, p.q_norm_w, p.positions[m],
                          lane, put);
       } else {
-        for (int i = lane; i < D / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
+        for (int i = lane; i < DK / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
       }
     }
     // ---- new K / V rows whose page lies in this CTA's range: norm + RoPE on K; both go to the cache (for later
@@ -447,23 +466,23 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         const size_t m = static_cast<size_t>(b) * p.q_per_seq + t;
         const long long slot = p.slots[m];
         if (pg < page0 || pg >= page1 || slot < 0) continue;  // warp-uniform
-        const size_t dst = ((static_cast<size_t>(slot >> 4) * p.n_kv_heads + kvh) * kPage + static_cast<size_t>(slot & 15)) * D;
+        const size_t dst = ((static_cast<size_t>(slot >> 4) * p.n_kv_heads + kvh) * kPage + static_cast<size_t>(slot & 15)) * DK;
         __nv_bfloat16* kd = const_cast<__nv_bfloat16*>(p.k_cache) + dst;
         __nv_bfloat16* vd = const_cast<__nv_bfloat16*>(p.v_cache) + dst;
-        __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(newkv_s) + static_cast<size_t>(t) * 2 * D;
-        const __nv_bfloat16* krow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + kvh) * D;
-        const __nv_bfloat16* vrow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + p.n_kv_heads + kvh) * D;
-        rope_head_row<D>(p, krow, p.k_norm_w, p.positions[m], lane, [&](int i0, float a, int i1, float bb) {
+        __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(newkv_s) + static_cast<size_t>(t) * 2 * DK;
+        const __nv_bfloat16* krow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + kvh) * DK;
+        const __nv_bfloat16* vrow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + p.n_kv_heads + kvh) * DK;
+        rope_head_row<DK>(p, krow, p.k_norm_w, p.positions[m], lane, [&](int i0, float a, int i1, float bb) {
           const __nv_bfloat16 ha = __float2bfloat16(a), hb = __float2bfloat16(bb);
           kd[i0] = ha;
           kd[i1] = hb;
           ks[i0] = ha;
           ks[i1] = hb;
         });
-        for (int i = lane; i < D / 2; i += 32) {
+        for (int i = lane; i < DK / 2; i += 32) {
           const uint32_t vv = reinterpret_cast<const uint32_t*>(vrow)[i];
           reinterpret_cast<uint32_t*>(vd)[i] = vv;
-          reinterpret_cast<uint32_t*>(ks + D)[i] = vv;
+          reinterpret_cast<uint32_t*>(ks + DK)[i] = vv;
         }
       }
     }
@@ -480,21 +499,21 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     __syncwarp();
     if (pg >= first_new_page) {
       // this page holds rows appended in this step: overwrite them in the landed copy (16-byte chunks, lanes 0-15 the
-      // K row, 16-31 the V row; D / 8 chunks per row)
-      uint8_t* kst = my_ring + (it % NSTAGE) * 2 * PAGE_BYTES;
+      // K row, 16-31 the V row; head size / 8 chunks per row)
+      uint8_t* kst = my_ring + (it % NSTAGE) * STAGE_BYTES;
       for (int t = 0; t < p.q_per_seq; ++t) {
         const int pos = new_pos0 + t;
         if (pos / kPage != pg || p.slots[static_cast<size_t>(b) * p.q_per_seq + t] < 0) continue;  // warp-uniform
-        const uint4* src = reinterpret_cast<const uint4*>(newkv_s + static_cast<size_t>(t) * 2 * D * 2);
-        for (int i = lane; i < 2 * CH; i += 32) {
-          const int which = i / CH, c = i % CH;
-          *reinterpret_cast<uint4*>(kst + which * PAGE_BYTES + swz<D>(pos & (kPage - 1), c)) = src[i];
+        const uint4* src = reinterpret_cast<const uint4*>(newkv_s + static_cast<size_t>(t) * (DK + DV) * 2);
+        for (int i = lane; i < CHK + CHV; i += 32) {
+          const int dst = i < CHK ? swz<DK>(pos & (kPage - 1), i) : KPAGE_BYTES + swz<DV>(pos & (kPage - 1), i - CHK);
+          *reinterpret_cast<uint4*>(kst + dst) = src[i];
         }
       }
       __syncwarp();
     }
-    const uint32_t k_base = smem_u32(my_ring + (it % NSTAGE) * 2 * PAGE_BYTES);
-    const uint32_t v_base = k_base + PAGE_BYTES;
+    const uint32_t k_base = smem_u32(my_ring + (it % NSTAGE) * STAGE_BYTES);
+    const uint32_t v_base = k_base + KPAGE_BYTES;
 
     float s[MT][2][4];
 #pragma unroll
@@ -504,11 +523,11 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
 #pragma unroll
     for (int ks = 0; ks < KS; ++ks) {
       uint32_t b0, b1, b2, b3;
-      ldsm_x4(k_base + swz<D>((lane & 7) + (lane >> 4) * 8, ks * 2 + ((lane >> 3) & 1)), b0, b1, b2, b3);
+      ldsm_x4(k_base + swz<DK>((lane & 7) + (lane >> 4) * 8, ks * 2 + ((lane >> 3) & 1)), b0, b1, b2, b3);
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
         uint32_t a0, a1, a2, a3;
-        ldsm_x4(q_base + swz<D>(mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4)), a0, a1, a2, a3);
+        ldsm_x4(q_base + swz<DK>(mt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, ks * 2 + (lane >> 4)), a0, a1, a2, a3);
         mma16816(s[mt][0], a0, a1, a2, a3, b0, b1);
         mma16816(s[mt][1], a0, a1, a2, a3, b2, b3);
       }
@@ -525,7 +544,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
           const int r = mt * 16 + g + (e >> 1) * 8;
           const int qp = kv_len - p.q_per_seq + p.t0 + r / group;
           bool ok = (r < rows) && (j <= qp) && (j < kv_len);
-          if (p.window > 0) ok = ok && (j > qp - p.window);
+          ok = ok && (j >= lowest_key(p, qp));
           const float v = ok ? s[mt][nt][e] * p.scale_log2 : -INFINITY;
           s[mt][nt][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -542,7 +561,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         l_run[mt][r] *= corr[r];
       }
 #pragma unroll
-      for (int i = 0; i < D / 8; ++i) {
+      for (int i = 0; i < DV / 8; ++i) {
         o[mt][i][0] *= corr[0];
         o[mt][i][1] *= corr[0];
         o[mt][i][2] *= corr[1];
@@ -558,9 +577,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         }
     }
 #pragma unroll
-    for (int dn = 0; dn < D / 8; dn += 2) {
+    for (int dn = 0; dn < DV / 8; dn += 2) {
       uint32_t b0, b1, b2, b3;
-      ldsm_x4_t(v_base + swz<D>((lane & 7) + ((lane >> 3) & 1) * 8, dn + (lane >> 4)), b0, b1, b2, b3);
+      ldsm_x4_t(v_base + swz<DV>((lane & 7) + ((lane >> 3) & 1) * 8, dn + (lane >> 4)), b0, b1, b2, b3);
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
         const uint32_t a0 = pack_bf16x2(s[mt][0][0], s[mt][0][1]);
@@ -576,12 +595,12 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   cp_async_wait<0>();
   __syncthreads();  // every warp is done with its ring: reuse it for the merge
 
-  // ---- merge the 4 warps: mo[w][row][D] fp32, mm/ml[w][row]; then this CTA's merged partial (cluster mode)
+  // ---- merge the 4 warps: mo[w][row][DV] fp32, mm/ml[w][row]; then this CTA's merged partial (cluster mode)
   float* mo = reinterpret_cast<float*>(ring);
-  float* mm = mo + 4 * ROWS * D;
+  float* mm = mo + 4 * ROWS * DV;
   float* ml = mm + 4 * ROWS;
-  float* part_s = ml + 4 * ROWS;   // [ROWS][D]
-  float* part_m = part_s + ROWS * D;
+  float* part_s = ml + 4 * ROWS;   // [ROWS][DV]
+  float* part_m = part_s + ROWS * DV;
   float* part_l = part_m + ROWS;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
@@ -596,15 +615,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         ml[warp * ROWS + row] = l;
       }
 #pragma unroll
-      for (int dn = 0; dn < D / 8; ++dn) {
+      for (int dn = 0; dn < DV / 8; ++dn) {
         float2 v = make_float2(o[mt][dn][2 * r], o[mt][dn][2 * r + 1]);
-        *reinterpret_cast<float2*>(&mo[(warp * ROWS + row) * D + dn * 8 + tig * 2]) = v;
+        *reinterpret_cast<float2*>(&mo[(warp * ROWS + row) * DV + dn * 8 + tig * 2]) = v;
       }
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < rows * D; i += 128) {
-    const int row = i / D, d = i % D;
+  for (int i = threadIdx.x; i < rows * DV; i += 128) {
+    const int row = i / DV, d = i % DV;
+    if (d >= p.dv) continue;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) M = fmaxf(M, mm[w * ROWS + row]);
@@ -614,7 +634,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     for (int w = 0; w < 4; ++w) {
       const float e = exp2f(mm[w * ROWS + row] - Ms);
       L += ml[w * ROWS + row] * e;
-      acc += mo[(w * ROWS + row) * D + d] * e;
+      acc += mo[(w * ROWS + row) * DV + d] * e;
     }
     const int t = p.t0 + row / group, hg = row % group;
     const int head = kvh * group + hg;
@@ -622,15 +642,15 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     if (p.splits == 1) {
       float Lf = L;
       if (p.sinks != nullptr) Lf += exp2f(p.sinks[head] * 1.4426950408889634f - Ms);
-      p.out[qrow * D + d] = __float2bfloat16(Lf > 0.f ? acc / Lf : 0.f);
+      p.out[qrow * p.dv + d] = __float2bfloat16(Lf > 0.f ? acc / Lf : 0.f);
     } else if (p.cluster_reduce) {
-      part_s[row * D + d] = acc;
+      part_s[row * DV + d] = acc;
       if (d == 0) {
         part_m[row] = M;
         part_l[row] = L;
       }
     } else {
-      p.part_o[(qrow * p.splits + split) * D + d] = acc;
+      p.part_o[(qrow * p.splits + split) * p.dv + d] = acc;
       if (d == 0) {
         p.part_ml[(qrow * p.splits + split) * 2 + 0] = M;
         p.part_ml[(qrow * p.splits + split) * 2 + 1] = L;
@@ -643,8 +663,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     cluster_arrive_release();
     cluster_wait_acquire();
     const uint32_t a_s = smem_u32(part_s), a_m = smem_u32(part_m), a_l = smem_u32(part_l);
-    for (int i = threadIdx.x + split * 128; i < rows * D; i += 128 * p.splits) {  // row-major: a warp stays in one row
-      const int row = i / D, d = i % D;
+    for (int i = threadIdx.x + split * 128; i < rows * DV; i += 128 * p.splits) {  // row-major: a warp stays in one row
+      const int row = i / DV, d = i % DV;
+      if (d >= p.dv) continue;
       float M = -INFINITY;
       float ms[kMaxClusterSplits], pv[kMaxClusterSplits], ls[kMaxClusterSplits];
 #pragma unroll
@@ -652,7 +673,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         if (sp < p.splits) {
           ms[sp] = ld_dsmem_f32(mapa_shared(a_m + row * 4, sp));
           ls[sp] = ld_dsmem_f32(mapa_shared(a_l + row * 4, sp));
-          pv[sp] = ld_dsmem_f32(mapa_shared(a_s + (row * D + d) * 4, sp));
+          pv[sp] = ld_dsmem_f32(mapa_shared(a_s + (row * DV + d) * 4, sp));
           M = fmaxf(M, ms[sp]);
         }
       }
@@ -669,7 +690,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
       const int t = p.t0 + row / group, hg = row % group;
       const int head = kvh * group + hg;
       if (p.sinks != nullptr) L += exp2f(p.sinks[head] * 1.4426950408889634f - Ms);
-      p.out[(static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + head) * D + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
+      p.out[(static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + head) * p.dv + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
     }
     cluster_arrive_release();  // done reading the peers' shared memory
     cluster_wait_acquire();    // and nobody reads this CTA's any more
@@ -686,7 +707,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     if (s_last) {
       __threadfence();
       // per (row, split) weights first (rows * splits <= 32 * 64 values, in the free merge area), then the
-      // D-wide accumulation with independent loads
+      // value-wide accumulation with independent loads
       float* wgt = mo;                       // [rows][splits]  exp2(m_s - M)
       float* linv = mo + ROWS * 64;          // [rows]          1 / L
       __syncthreads();
@@ -708,21 +729,22 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         linv[row] = L > 0.f ? 1.f / L : 0.f;
       }
       __syncthreads();
-      for (int i = threadIdx.x; i < rows * D; i += 128) {
-        const int row = i / D, d = i % D;
+      for (int i = threadIdx.x; i < rows * DV; i += 128) {
+        const int row = i / DV, d = i % DV;
+        if (d >= p.dv) continue;
         const int t = p.t0 + row / group, hg = row % group;
         const size_t qrow = static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + kvh * group + hg;
-        const float* po = p.part_o + qrow * p.splits * D + d;
+        const float* po = p.part_o + qrow * p.splits * p.dv + d;
         float acc = 0.f;
         int sp = 0;
         for (; sp + 4 <= p.splits; sp += 4) {
-          const float a0 = __ldcg(po + (sp + 0) * D), a1 = __ldcg(po + (sp + 1) * D);
-          const float a2 = __ldcg(po + (sp + 2) * D), a3 = __ldcg(po + (sp + 3) * D);
+          const float a0 = __ldcg(po + (sp + 0) * p.dv), a1 = __ldcg(po + (sp + 1) * p.dv);
+          const float a2 = __ldcg(po + (sp + 2) * p.dv), a3 = __ldcg(po + (sp + 3) * p.dv);
           acc += a0 * wgt[row * 64 + sp] + a1 * wgt[row * 64 + sp + 1] + a2 * wgt[row * 64 + sp + 2] +
                  a3 * wgt[row * 64 + sp + 3];
         }
-        for (; sp < p.splits; ++sp) acc += __ldcg(po + sp * D) * wgt[row * 64 + sp];
-        p.out[qrow * D + d] = __float2bfloat16(acc * linv[row]);
+        for (; sp < p.splits; ++sp) acc += __ldcg(po + sp * p.dv) * wgt[row * 64 + sp];
+        p.out[qrow * p.dv + d] = __float2bfloat16(acc * linv[row]);
       }
     }
   }
@@ -733,11 +755,11 @@ template <int D>
 static size_t prefill_smem() {
   return 64 * D * 2 + 4 * 64 * D * 2;
 }
-template <int D, int MT>
+template <int DK, int DV, int MT>
 static size_t decode_smem() {
-  const size_t ring = 4 * 3 * 2 * kPage * D * 2;
-  const size_t merge = (4 * 16 * MT * D + 2 * 4 * 16 * MT + 16 * MT * D + 2 * 16 * MT) * sizeof(float);
-  return 16 * MT * D * 2 + kMaxFusedNew * 2 * D * 2 + (ring > merge ? ring : merge);
+  const size_t ring = 4 * 3 * kPage * (DK + DV) * 2;
+  const size_t merge = (4 * 16 * MT * DV + 2 * 4 * 16 * MT + 16 * MT * DV + 2 * 16 * MT) * sizeof(float);
+  return 16 * MT * DK * 2 + kMaxFusedNew * (DK + DV) * 2 + (ring > merge ? ring : merge);
 }
 
 }  // namespace eredu
@@ -803,14 +825,14 @@ extern "C" int eredu_attn_prefill(const void* q, const void* k_cache, const void
   return static_cast<int>(e);
 }
 
-template <int D, int MT>
+template <int DK, int DV, int MT>
 static cudaError_t launch_decode(const AttnParams& p, dim3 grid, cudaStream_t stream) {
   static bool cfg[kMaxDevices] = {};
-  if (!configure_once(cfg, attn_decode_kernel<D, MT>, decode_smem<D, MT>())) return cudaErrorInvalidValue;
+  if (!configure_once(cfg, attn_decode_kernel<DK, DV, MT>, decode_smem<DK, DV, MT>())) return cudaErrorInvalidValue;
   cudaLaunchConfig_t lc = {};
   lc.gridDim = grid;
   lc.blockDim = dim3(128);
-  lc.dynamicSmemBytes = decode_smem<D, MT>();
+  lc.dynamicSmemBytes = decode_smem<DK, DV, MT>();
   lc.stream = stream;
   cudaLaunchAttribute attr[2];
   int nattr = 0;
@@ -828,20 +850,25 @@ static cudaError_t launch_decode(const AttnParams& p, dim3 grid, cudaStream_t st
   }
   lc.attrs = attr;
   lc.numAttrs = nattr;
-  const cudaError_t e = cudaLaunchKernelEx(&lc, attn_decode_kernel<D, MT>, p);
+  const cudaError_t e = cudaLaunchKernelEx(&lc, attn_decode_kernel<DK, DV, MT>, p);
   eredu_count_launches(1);
   return e;
 }
 
-// q: [batch * q_per_seq, n_q_heads, D]; every sequence contributes exactly q_per_seq query tokens whose
+// q: [batch * q_per_seq, n_q_heads, key_dim]; every sequence contributes exactly q_per_seq query tokens whose
 // positions are the last q_per_seq positions of its kv (causal among themselves). part_o / part_ml are
 // caller-provided fp32 scratch (see eredu_attn_decode_scratch_elems) and `counters` a zeroed int32
 // [batch * n_kv_heads] array (left zeroed again on return); all unused when splits == 1.
-static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_heads, int n_kv_heads, int head_dim,
+static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_heads, int n_kv_heads, int key_dim, int value_dim,
                              cudaStream_t stream, bool force_scratch = false) {
   if (n_kv_heads <= 0 || n_q_heads <= 0 || n_q_heads % n_kv_heads != 0) return -1;
   const int group = n_q_heads / n_kv_heads;
-  if (group > 32 || (head_dim != 128 && head_dim != 64)) return -1;
+  if (group > 32 || key_dim <= 0 || key_dim > 128 || key_dim % 8 != 0 || value_dim <= 0 || value_dim > 128 || value_dim % 8 != 0)
+    return -1;
+  // the fused form rotates and appends rows of one head size that fills its tile
+  if (p.qkv != nullptr && (key_dim != value_dim || (key_dim != 128 && key_dim != 64))) return -1;
+  p.dk = key_dim;
+  p.dv = value_dim;
   const int t_per = group > 16 ? 1 : (32 / group < q_per_seq ? 32 / group : q_per_seq);
   if (p.qkv != nullptr && q_per_seq > kMaxFusedNew) return -1;
   // Few splits: a cluster per (sequence, kv head) combines the partials in shared memory. More splits than a portable
@@ -854,8 +881,11 @@ static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_hea
     p.t_count = (q_per_seq - t0 < t_per) ? q_per_seq - t0 : t_per;
     const int rows = p.t_count * group;
     cudaError_t e;
-    if (head_dim == 128) e = rows <= 16 ? launch_decode<128, 1>(p, grid, stream) : launch_decode<128, 2>(p, grid, stream);
-    else e = rows <= 16 ? launch_decode<64, 1>(p, grid, stream) : launch_decode<64, 2>(p, grid, stream);
+    const bool one = rows <= 16;
+    if (key_dim > 64 && value_dim > 64) e = one ? launch_decode<128, 128, 1>(p, grid, stream) : launch_decode<128, 128, 2>(p, grid, stream);
+    else if (key_dim > 64) e = one ? launch_decode<128, 64, 1>(p, grid, stream) : launch_decode<128, 64, 2>(p, grid, stream);
+    else if (value_dim > 64) e = one ? launch_decode<64, 128, 1>(p, grid, stream) : launch_decode<64, 128, 2>(p, grid, stream);
+    else e = one ? launch_decode<64, 64, 1>(p, grid, stream) : launch_decode<64, 64, 2>(p, grid, stream);
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   return 0;
@@ -863,8 +893,8 @@ static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_hea
 
 static int attn_decode_impl(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                             const int* seq_lens, const float* sinks, float* part_o, float* part_ml, int* counters,
-                            int batch, int q_per_seq, int max_pages, int n_q_heads, int n_kv_heads, int head_dim,
-                            int splits, int window, float scale, cudaStream_t stream, bool force_scratch) {
+                            int batch, int q_per_seq, int max_pages, int n_q_heads, int n_kv_heads, int key_dim, int value_dim,
+                            int splits, int window, int chunk, float scale, cudaStream_t stream, bool force_scratch) {
   AttnParams p = {};
   p.q = static_cast<const __nv_bfloat16*>(q);
   p.k_cache = static_cast<const __nv_bfloat16*>(k_cache);
@@ -882,8 +912,9 @@ static int attn_decode_impl(const void* q, const void* k_cache, const void* v_ca
   p.q_per_seq = q_per_seq;
   p.splits = splits < 1 ? 1 : (splits > 64 ? 64 : splits);
   p.window = window;
+  p.chunk = chunk;
   p.scale_log2 = scale * 1.4426950408889634f;
-  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, head_dim, stream, force_scratch);
+  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, key_dim, value_dim, stream, force_scratch);
 }
 
 // Up to 8 splits combine inside a thread-block cluster and ignore the scratch arguments (they may be null); more
@@ -891,10 +922,10 @@ static int attn_decode_impl(const void* q, const void* k_cache, const void* v_ca
 extern "C" int eredu_attn_decode(const void* q, const void* k_cache, const void* v_cache, void* out,
                                  const int* block_table, const int* seq_lens, const float* sinks, float* part_o,
                                  float* part_ml, int* counters, int batch, int q_per_seq, int max_pages, int n_q_heads,
-                                 int n_kv_heads, int head_dim, int splits, int window, float scale,
+                                 int n_kv_heads, int key_dim, int value_dim, int splits, int window, int chunk, float scale,
                                  cudaStream_t stream) {
-  return attn_decode_impl(q, k_cache, v_cache, out, block_table, seq_lens, sinks, part_o, part_ml, counters, batch,
-                          q_per_seq, max_pages, n_q_heads, n_kv_heads, head_dim, splits, window, scale, stream, false);
+  return attn_decode_impl(q, k_cache, v_cache, out, block_table, seq_lens, sinks, part_o, part_ml, counters, batch, q_per_seq,
+                          max_pages, n_q_heads, n_kv_heads, key_dim, value_dim, splits, window, chunk, scale, stream, false);
 }
 
 // Decode attention that starts from the projection output: qkv [batch * q_per_seq, ld_qkv] = [q heads | k heads |
@@ -940,7 +971,7 @@ extern "C" int eredu_attn_decode_rope(const void* qkv, int ld_qkv, void* k_cache
   p.splits = splits < 1 ? 1 : (splits > 64 ? 64 : splits);
   p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
-  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, head_dim, stream);
+  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, head_dim, head_dim, stream);
 }
 
 // ---------------------------------------------------------------------------------------------- no-allocation variant
@@ -986,6 +1017,6 @@ extern "C" int eredu_attn_decode_static(const void* q, const void* k_cache, cons
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   // always the scratch form of the split reduction: that is the form whose scratch this entry point provides
-  return attn_decode_impl(q, k_cache, v_cache, out, block_table, seq_lens, sinks, part_o, part_ml, counters, batch,
-                          q_per_seq, max_pages, n_q_heads, n_kv_heads, head_dim, splits, window, scale, stream, true);
+  return attn_decode_impl(q, k_cache, v_cache, out, block_table, seq_lens, sinks, part_o, part_ml, counters, batch, q_per_seq,
+                          max_pages, n_q_heads, n_kv_heads, head_dim, head_dim, splits, window, 0, scale, stream, true);
 }

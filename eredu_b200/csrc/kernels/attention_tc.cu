@@ -19,7 +19,9 @@
 // prefixes work); key tiles beyond a query tile's last position are never loaded. CTAs with the most key tiles are
 // scheduled first.
 //
-// Head size 64 or 128, optional sliding window (key tiles before the window are skipped) and sink logits. Same
+// Key and value widths up to 128 (multiples of 8, not necessarily equal: a 64-wide half that reaches beyond the stored
+// width is filled with zeros by the TMA), optional sliding window or chunks of positions (key tiles before what a tile's
+// rows can see are skipped) and sink logits. Same
 // online-softmax recurrence and semantics as attn_prefill_kernel in attention.cu and as the reference's blockwise attention (eredu/src/backend/mlx/nn/attention.rs:346-436,
 // runtime/cache/kv.rs:2267-2436). Every wait is bounded; on expiry the status word is set and the CTA leaves through the
 // common exit (TMEM is freed there).
@@ -34,7 +36,7 @@
 namespace eredu {
 
 struct AttnTcParams {
-  __nv_bfloat16* out;          // [tokens, n_q, 128]
+  __nv_bfloat16* out;          // [tokens, n_q, dv]
   const int* block_table;      // [batch, max_pages]
   const int* seq_lens;         // kv length after this call, per sequence
   const int* cu_q;             // [batch + 1] query-row offsets
@@ -42,6 +44,8 @@ struct AttnTcParams {
   int max_pages;
   int n_q_heads, n_kv_heads;
   int window;                  // 0: none; else a query at position p sees keys in (p - window, p]
+  int chunk;                   // > 0 (window 0): a query sees the keys of its own chunk of positions
+  int dk, dv;                  // key / value width of a head (multiples of 8); the rest of a 64-wide half reads as zero
   float scale_log2;
   int* status;
 };
@@ -50,8 +54,8 @@ constexpr int kTcThreads = 320;
 constexpr int kTcTile = 128;            // query rows per tile and keys per tile
 constexpr int kTcRows = 2 * kTcTile;    // query rows per CTA
 constexpr int kTcHalf = 128 * 64 * 2;   // one [128 rows][64 bf16] swizzled half tile: 16 KB
-// shared memory: Q_a, Q_b (D / 64 halves each) | K ring (2 x D / 64 halves) | V ring (2 x D / 64 halves) | barriers
-constexpr int tc_smem(int d) { return 1024 + 3 * 2 * (d / 64) * kTcHalf + 256; }
+// shared memory: Q_a, Q_b (NK halves each) | K ring (2 x NK halves) | V ring (2 x NV halves) | barriers
+constexpr int tc_smem(int nk, int nv) { return 1024 + 2 * (2 * nk + nv) * kTcHalf + 256; }
 // A quarter of the exponentials as a polynomial on the FMA pipe (build option). Measured slower here (1153 against 1192
 // TFLOP/s at 32k tokens, 1112 against 1170 at 8k): the softmax warps are bound by instruction issue, not by the
 // special-function unit, so the extra FMA-pipe instructions cost more than the unit they relieve.
@@ -82,18 +86,25 @@ __device__ __forceinline__ void tma_load_4d(void* smem_dst, const CUtensorMap* m
       : "memory");
 }
 
-template <int D>
+// First key position a query at `pos` can see.
+__device__ __forceinline__ int tc_lowest_key(const AttnTcParams& p, int pos) {
+  if (p.window > 0) return max(0, pos - p.window + 1);
+  return p.chunk > 0 ? pos - pos % p.chunk : 0;
+}
+
+// NK / NV: 64-wide halves of the key and of the value width
+template <int NK, int NV>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                        const __grid_constant__ CUtensorMap tmV, const AttnTcParams p) {
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  constexpr int NH = D / 64;                                           // 64-wide halves of the head dimension
-  constexpr uint32_t kIdescPV = umma_idesc_bf16(128, D) | (1u << 16);  // B (= V) MN-major, N = head dimension
-  uint8_t* q_s = smem;                                                 // tile w at + w * NH halves
-  uint8_t* k_s = q_s + 2 * NH * kTcHalf;                               // stage s at + s * NH halves
-  uint8_t* v_s = k_s + 2 * NH * kTcHalf;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + 2 * NH * kTcHalf);
+  const uint32_t kIdescPV = umma_idesc_bf16(128, (p.dv + 15) & ~15) | (1u << 16);  // B (= V) MN-major, N = value width
+  const int k_steps = (p.dk + 15) >> 4, o_steps = (p.dv + 15) >> 4;
+  uint8_t* q_s = smem;                                                 // tile w at + w * NK halves
+  uint8_t* k_s = q_s + 2 * NK * kTcHalf;                               // stage s at + s * NK (K), s * NV (V) halves
+  uint8_t* v_s = k_s + 2 * NK * kTcHalf;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + 2 * NV * kTcHalf);
   uint64_t* q_full = bars;                  // 1
   uint64_t* k_full = bars + 1;              // [2]
   uint64_t* k_empty = bars + 3;             // [2]
@@ -120,9 +131,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int n_a = min(kv_len - 1, pos0 + kTcTile - 1) / kTcTile + 1;
   const int n_b = row0 + kTcTile < q_len ? min(kv_len - 1, pos0 + kTcRows - 1) / kTcTile + 1 : 0;
   const int n_tiles = max(n_a, n_b);
-  // sliding window: key tiles that lie wholly before the window of a tile's FIRST row are skipped
-  const int j0_a = p.window > 0 ? max(0, pos0 - p.window + 1) / kTcTile : 0;
-  const int j0_b = p.window > 0 ? max(0, pos0 + kTcTile - p.window + 1) / kTcTile : 0;
+  // window / chunk: key tiles that lie wholly before what a tile's FIRST row sees are skipped
+  const int j0_a = tc_lowest_key(p, pos0) / kTcTile;
+  const int j0_b = tc_lowest_key(p, pos0 + kTcTile) / kTcTile;
   const int j0 = n_b > 0 ? min(j0_a, j0_b) : j0_a;
 
   if (threadIdx.x == 0) {
@@ -157,10 +168,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
-      mbar_arrive_expect_tx(q_full, 2 * NH * kTcHalf);
+      mbar_arrive_expect_tx(q_full, 2 * NK * kTcHalf);
       for (int w = 0; w < 2; ++w)
-        for (int h = 0; h < NH; ++h)
-          tma_load_3d(q_s + (w * NH + h) * kTcHalf, &tmQ, h * 64, head, q0 + row0 + w * kTcTile, q_full);
+        for (int h = 0; h < NK; ++h)
+          tma_load_3d(q_s + (w * NK + h) * kTcHalf, &tmQ, h * 64, head, q0 + row0 + w * kTcTile, q_full);
       const int* pages = p.block_table + static_cast<size_t>(b) * p.max_pages;
       for (int jj = 0; j0 + jj < n_tiles && ok; ++jj) {
         const int j = j0 + jj;                                           // key tile; jj counts this CTA's iterations
@@ -174,16 +185,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         }
         if (jj >= 2) ok = mbar_wait(&k_empty[s], reuse_parity, p.status, kStatusSmemEmptyTimeout);
         if (!ok) break;
-        mbar_arrive_expect_tx(&k_full[s], NH * kTcHalf);
+        mbar_arrive_expect_tx(&k_full[s], NK * kTcHalf);
 #pragma unroll
         for (int pg = 0; pg < 8; ++pg)
-          for (int h = 0; h < NH; ++h) tma_load_4d(k_s + (s * NH + h) * kTcHalf + pg * 2048, &tmK, h * 64, 0, kv_head, page[pg], &k_full[s]);
+          for (int h = 0; h < NK; ++h) tma_load_4d(k_s + (s * NK + h) * kTcHalf + pg * 2048, &tmK, h * 64, 0, kv_head, page[pg], &k_full[s]);
         if (jj >= 2) ok = mbar_wait(&v_empty[s], reuse_parity, p.status, kStatusSmemEmptyTimeout);
         if (!ok) break;
-        mbar_arrive_expect_tx(&v_full[s], NH * kTcHalf);
+        mbar_arrive_expect_tx(&v_full[s], NV * kTcHalf);
 #pragma unroll
         for (int pg = 0; pg < 8; ++pg)
-          for (int h = 0; h < NH; ++h) tma_load_4d(v_s + (s * NH + h) * kTcHalf + pg * 2048, &tmV, h * 64, 0, kv_head, page[pg], &v_full[s]);
+          for (int h = 0; h < NV; ++h) tma_load_4d(v_s + (s * NV + h) * kTcHalf + pg * 2048, &tmV, h * 64, 0, kv_head, page[pg], &v_full[s]);
       }
     }
   } else if (warp == 1) {
@@ -193,18 +204,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       // jj: this CTA's iteration (selects the K / V stage); tile w is active on key tiles [first_w, n_w)
       const int first[2] = {j0_a, j0_b}, last[2] = {n_a, n_b};
       auto issue_s = [&](int w, int jj) {
-        const uint32_t qa = q_addr + w * NH * kTcHalf;
-        const uint32_t ka = smem_u32(k_s + (jj & 1) * NH * kTcHalf);
+        const uint32_t qa = q_addr + w * NK * kTcHalf;
+        const uint32_t ka = smem_u32(k_s + (jj & 1) * NK * kTcHalf);
         const uint32_t d = tmem + w * 128;
 #pragma unroll
-        for (int kk = 0; kk < D / 16; ++kk) {      // K = head dimension: four 16-steps per 64-wide half
+        for (int kk = 0; kk < NK * 4; ++kk) {      // K = key width: four 16-steps per 64-wide half
+          if (kk >= k_steps) break;
           const uint32_t off = (kk >> 2) * kTcHalf + (kk & 3) * 32;
           umma_f16(d, umma_desc_k_sw128(qa + off), umma_desc_k_sw128(ka + off), kIdescQK, kk > 0 ? 1u : 0u);
         }
         umma_commit(&s_full[w]);
       };
       auto issue_pv = [&](int w, int jj, bool fresh) {
-        const uint32_t va = smem_u32(v_s + (jj & 1) * NH * kTcHalf);
+        const uint32_t va = smem_u32(v_s + (jj & 1) * NV * kTcHalf);
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)             // K = keys: P from tensor memory (8 columns per step), V MN-major (2048 bytes per step)
           umma_f16_ts(tmem + 256 + w * 128, tmem + w * 128 + kk * 8, umma_desc_mn_sw128(va + kk * 2048, kTcHalf), kIdescPV,
@@ -262,7 +274,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
     const uint32_t s_addr = tmem + lane_addr + w * 128;
     const uint32_t o_addr = tmem + lane_addr + 256 + w * 128;
-    float m = 0.f, l = 0.f;
+    float m = -INFINITY, l = 0.f;                                        // -inf: this row has not seen a key yet
     for (int j = j0_w; j < n_w && ok; ++j) {
       const int it = j - j0_w;                                           // this tile's round: parity of its barriers
       ok = mbar_wait(&s_full[w], it & 1, p.status, kStatusAccumTimeout);
@@ -273,10 +285,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       for (int c = 0; c < 8; ++c) tmem_ld16(s_addr + c * 16, sc[c]);
       tmem_wait_ld();
       const int key0 = j * kTcTile;
-      const bool before = p.window > 0 && key0 <= tile_pos0 + kTcTile - 1 - p.window;     // some row's window starts inside or after this tile
+      const bool before = key0 < tc_lowest_key(p, tile_pos0 + kTcTile - 1);     // some row's visible keys start inside or after this tile
       if (key0 + kTcTile - 1 > tile_pos0 || key0 + kTcTile > kv_len || before) {   // some (row, key) of the tile is masked: -inf gives p = 0
         const int visible = min(qpos, kv_len - 1) - key0;                // keys hidden .. visible of this tile are seen by this row
-        const int hidden = p.window > 0 ? qpos - p.window + 1 - key0 : 0;
+        const int hidden = tc_lowest_key(p, qpos) - key0;
 #pragma unroll
         for (int c = 0; c < 8; ++c)
 #pragma unroll
@@ -290,16 +302,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         for (int i = 0; i < 16; i += 2) mx4[(i >> 1) & 3] = max3(mx4[(i >> 1) & 3], __uint_as_float(sc[c][i]), __uint_as_float(sc[c][i + 1]));
       const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       const float m_new = mx * p.scale_log2;                             // -inf for a fully masked row: every comparison below is false
-      if (it == 0) {
-        m = m_new == -INFINITY ? 0.f : m_new;
+      bool grow = false;
+      if (m == -INFINITY) {
+        m = m_new;                                                       // what the row added so far is zero
       } else {
-        const bool grow = m_new > m + kTcRescale;
+        grow = m_new > m + kTcRescale;
+      }
+      if (it > 0) {
         if (__any_sync(0xffffffffu, grow)) {                             // O_w(j - 1) is complete: s_full followed it on the tensor core
           const float alpha = grow ? ex2_approx(m - m_new) : 1.f;
           if (grow) m = m_new;
           l *= alpha;
 #pragma unroll 1
-          for (int c = 0; c < 8; ++c) {
+          for (int c = 0; c < o_steps; ++c) {
             uint32_t r[16];
             tmem_ld16(o_addr + c * 16, r);
             tmem_wait_ld();
@@ -310,7 +325,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         }
       }
       // p = exp2(s * scale - m), two values per FMA / add; sums in four chains
-      const uint64_t scale2 = pack_f32x2(p.scale_log2, p.scale_log2), shift2 = pack_f32x2(-m, -m);
+      const float shift = m == -INFINITY ? 0.f : -m;
+      const uint64_t scale2 = pack_f32x2(p.scale_log2, p.scale_log2), shift2 = pack_f32x2(shift, shift);
       uint64_t acc[4] = {0ull, 0ull, 0ull, 0ull};
 #pragma unroll
       for (int c2 = 0; c2 < 4; ++c2) {
@@ -341,9 +357,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       const bool store = tile_row0 + row < q_len;
       if (p.sinks != nullptr) l += ex2_approx(p.sinks[head] * 1.4426950408889634f - m);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      uint4* dst = reinterpret_cast<uint4*>(p.out + (static_cast<size_t>(q0 + tile_row0 + row) * p.n_q_heads + head) * D);
+      uint4* dst = reinterpret_cast<uint4*>(p.out + (static_cast<size_t>(q0 + tile_row0 + row) * p.n_q_heads + head) * p.dv);
 #pragma unroll 1
-      for (int c = 0; c < D / 16; ++c) {
+      for (int c = 0; c < o_steps; ++c) {
         uint32_t r[16];
         tmem_ld16(o_addr + c * 16, r);
         tmem_wait_ld();
@@ -358,7 +374,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           v1.z = pack_bf16x2(__uint_as_float(r[12]) * inv, __uint_as_float(r[13]) * inv);
           v1.w = pack_bf16x2(__uint_as_float(r[14]) * inv, __uint_as_float(r[15]) * inv);
           dst[c * 2] = v0;
-          dst[c * 2 + 1] = v1;
+          if (c * 16 + 8 < p.dv) dst[c * 2 + 1] = v1;
         }
       }
     }
@@ -374,29 +390,30 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 
 using namespace eredu;
 
-// Causal prefill attention over the paged cache, head size 64 or 128, optional sliding window and sink logits.
-// q: [tokens, n_q, D] bf16 (contiguous); k_cache / v_cache: [pages, n_kv, 16, D] bf16 (contiguous); sinks: fp32 [n_q] or
+// Causal prefill attention over the paged cache, key / value widths up to 128, optional window or chunks and sink logits.
+// q: [tokens, n_q, key_dim] bf16 (contiguous); k_cache / v_cache: [pages, n_kv, 16, width] bf16 (contiguous); sinks: fp32 [n_q] or
 // null. Same arguments as eredu_attn_prefill otherwise. Returns -2 for shapes it does not take.
-template <int D>
+template <int NK, int NV>
 static int launch_attn_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnTcParams& p, dim3 grid,
                           cudaStream_t stream) {
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(D)) != cudaSuccess) return -1;
+    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<NK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(NK, NV)) != cudaSuccess) return -1;
     configured[dev] = true;
   }
-  return static_cast<int>(launch_pdl(attn_prefill_tc_kernel<D>, grid, dim3(kTcThreads), tc_smem(D), stream, tmQ, tmK, tmV, p));
+  return static_cast<int>(launch_pdl(attn_prefill_tc_kernel<NK, NV>, grid, dim3(kTcThreads), tc_smem(NK, NV), stream, tmQ, tmK, tmV, p));
 }
 
 extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                                      const int* seq_lens, const int* cu_q, const float* sinks, int batch, int total_q, int max_q_len,
-                                     int max_pages, int num_pages, int n_q_heads, int n_kv_heads, int head_dim, int window, float scale,
-                                     int* status, cudaStream_t stream) {
-  if ((head_dim != 128 && head_dim != 64) || batch <= 0 || total_q <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || window < 0)
+                                     int max_pages, int num_pages, int n_q_heads, int n_kv_heads, int key_dim, int value_dim, int window,
+                                     int chunk, float scale, int* status, cudaStream_t stream) {
+  if (key_dim <= 0 || key_dim > 128 || key_dim % 8 != 0 || value_dim <= 0 || value_dim > 128 || value_dim % 8 != 0 || batch <= 0 ||
+      total_q <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || window < 0 || chunk < 0)
     return -2;
-  const uint64_t D = static_cast<uint64_t>(head_dim);
+  const uint64_t D = static_cast<uint64_t>(key_dim), V = static_cast<uint64_t>(value_dim);
   CUtensorMap tmQ, tmK, tmV;
   // q as [tokens][heads][D]: box = 128 tokens x 1 head x 64 values
   int r = make_tma_3d(&tmQ, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, static_cast<uint64_t>(n_q_heads),
@@ -405,8 +422,8 @@ extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const v
   r = make_tma_4d(&tmK, k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, D, 16, static_cast<uint64_t>(n_kv_heads),
                   static_cast<uint64_t>(num_pages), D * 2, 16 * D * 2, static_cast<uint64_t>(n_kv_heads) * 16 * D * 2, 64, 16, 1, 1);
   if (r != 0) return -200 + r;
-  r = make_tma_4d(&tmV, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, D, 16, static_cast<uint64_t>(n_kv_heads),
-                  static_cast<uint64_t>(num_pages), D * 2, 16 * D * 2, static_cast<uint64_t>(n_kv_heads) * 16 * D * 2, 64, 16, 1, 1);
+  r = make_tma_4d(&tmV, v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, V, 16, static_cast<uint64_t>(n_kv_heads),
+                  static_cast<uint64_t>(num_pages), V * 2, 16 * V * 2, static_cast<uint64_t>(n_kv_heads) * 16 * V * 2, 64, 16, 1, 1);
   if (r != 0) return -300 + r;
   AttnTcParams p = {};
   p.out = static_cast<__nv_bfloat16*>(out);
@@ -418,10 +435,15 @@ extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const v
   p.n_q_heads = n_q_heads;
   p.n_kv_heads = n_kv_heads;
   p.window = window;
+  p.chunk = chunk;
+  p.dk = key_dim;
+  p.dv = value_dim;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.status = status;
   dim3 grid(n_q_heads, (max_q_len + kTcRows - 1) / kTcRows, batch);
-  const int e = head_dim == 128 ? launch_attn_tc<128>(tmQ, tmK, tmV, p, grid, stream) : launch_attn_tc<64>(tmQ, tmK, tmV, p, grid, stream);
+  int e;
+  if (key_dim > 64) e = value_dim > 64 ? launch_attn_tc<2, 2>(tmQ, tmK, tmV, p, grid, stream) : launch_attn_tc<2, 1>(tmQ, tmK, tmV, p, grid, stream);
+  else e = value_dim > 64 ? launch_attn_tc<1, 2>(tmQ, tmK, tmV, p, grid, stream) : launch_attn_tc<1, 1>(tmQ, tmK, tmV, p, grid, stream);
   eredu_count_launches(1);
   return e;
 }

@@ -47,6 +47,7 @@ struct PGemmParams {
   float norm_eps;
   float norm_inv_dim;
   float* ssq_out;
+  int act;  // plain tiles: 2 = squared ReLU before the residual
   int n_tiles, m_tiles;
 };
 
@@ -251,6 +252,13 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
 #pragma unroll
             for (int j = 0; j < 8; ++j) v[j] = silu_f(v[j]) * u[j];
           }
+          if (!DUAL && p.act == 2) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+              v[j] = fmaxf(v[j], 0.f);
+              v[j] *= v[j];
+            }
+          }
           const uint32_t r[4] = {rv[i].x, rv[i].y, rv[i].z, rv[i].w};
           uint4 o;
           o.x = pack_bf16x2(v[0] + bf16_lo(r[0]), v[1] + bf16_hi(r[0]));
@@ -289,7 +297,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
 int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* residual, const void* bias, int M, int N,
                            int K, int ldx, int ldw, int ldy, int ldr, int w_rows, int dual, int dual_row_offset,
                            int sm_count, int* status, const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim,
-                           float* ssq_out, cudaStream_t stream) {
+                           float* ssq_out, int act, cudaStream_t stream) {
   if (N % 8 != 0 || ldy % 8 != 0 || (reinterpret_cast<uintptr_t>(Y) & 15) != 0) return kPersistentUnsupported;
   if (dual && (ssq_out != nullptr || N % 64 != 0 || dual_row_offset % 8 != 0)) return kPersistentUnsupported;
   if (residual != nullptr && (ldr % 8 != 0 || (reinterpret_cast<uintptr_t>(residual) & 15) != 0)) return kPersistentUnsupported;
@@ -314,6 +322,7 @@ int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* re
   p.norm_eps = norm_eps;
   p.norm_inv_dim = norm_dim > 0 ? 1.0f / static_cast<float>(norm_dim) : 0.f;
   p.ssq_out = ssq_out;
+  p.act = act;
   p.n_tiles = dual ? (N + 63) / 64 : (N + 127) / 128;
   p.m_tiles = (M + kTN - 1) / kTN;
   const int total = p.n_tiles * p.m_tiles;

@@ -11,6 +11,6 @@ constexpr int kPersistentUnsupported = -7777;
 int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* residual, const void* bias, int M, int N,
                            int K, int ldx, int ldw, int ldy, int ldr, int w_rows, int dual, int dual_row_offset,
                            int sm_count, int* status, const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim,
-                           float* ssq_out, cudaStream_t stream);
+                           float* ssq_out, int act, cudaStream_t stream);
 
 }  // namespace eredu

@@ -58,7 +58,7 @@ struct GemmParams {
   // Large token tiles: the epilogue goes through shared memory so that the output (and the residual) move as
   // 16-byte row chunks instead of one 2-byte element per thread. Needs 16-byte aligned rows (host-checked).
   int staged;
-  // Gated activation of DUAL tiles: 0 = silu(g) * u (SwiGLU); 1 = g * sigmoid(1.702 g) * (u + 1) (GPT-OSS). With
+  // Plain tiles: 2 = squared ReLU of the output (after bias, before the residual). Gated activation of DUAL tiles: 0 = silu(g) * u (SwiGLU); 1 = g * sigmoid(1.702 g) * (u + 1) (GPT-OSS). With
   // act_limit > 0 the gate is clamped from above and the linear branch to [-limit, limit] first
   // (eredu/src/backend/mlx/architectures/gpt_oss/model.rs:748-753; nn/moe.rs swiglu_limit).
   int act;
@@ -110,6 +110,14 @@ __device__ __forceinline__ float gated_act(const GemmParams& p, float g, float u
   return silu_f(g) * u;
 }
 
+__device__ __forceinline__ float plain_act(const GemmParams& p, float g) {
+  if (p.act == 2) {
+    g = fmaxf(g, 0.f);
+    g *= g;
+  }
+  return g;
+}
+
 // Applies row scale, bias, activation and residual, stores, and returns the value as stored (after rounding).
 __device__ __forceinline__ float residual_at(const GemmParams& p, int m, int n) {
   return __bfloat162float(static_cast<const __nv_bfloat16*>(p.residual)[static_cast<size_t>(m) * p.ldr + n]);
@@ -126,7 +134,7 @@ __device__ __forceinline__ float epilogue_store(const GemmParams& p, float g, fl
     g += __bfloat162float(b[n]);
     if (DUAL) u += __bfloat162float(b[p.N + n]);
   }
-  float v = (DUAL ? gated_act(p, g, u) : g) + rv;
+  float v = (DUAL ? gated_act(p, g, u) : plain_act(p, g)) + rv;
   if (p.out_fp32) {
     static_cast<float*>(p.y)[static_cast<size_t>(m) * p.ldy + n] = v;
     return v;
@@ -405,7 +413,7 @@ gemm_wt_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           for (int j = 0; j < 16; ++j) {
             const float sc = (p.ssq_in != nullptr) ? s_scale[c0 + j] : 1.f;
             const float gg = __uint_as_float(g[j]) * sc + bg;
-            red[(c0 + j) * 128 + row] = DUAL ? gated_act(p, gg, __uint_as_float(u[j]) * sc + bu) : gg;
+            red[(c0 + j) * 128 + row] = DUAL ? gated_act(p, gg, __uint_as_float(u[j]) * sc + bu) : plain_act(p, gg);
           }
         } else {
           float rr[16];
@@ -791,7 +799,8 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   if (tn == 256 && !out_fp32 && force_split <= 1 && persistent_enabled()) {
     // prefill-sized: persistent kernel with double-buffered accumulators
     const int pr = launch_gemm_persistent(X, W, Y, residual, bias, M, N, K, ldx, ldw, ldy, ldr, w_rows, dual, dual_row_offset,
-                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, stream);
+                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, (flags & 2) ? 2 : 0,
+                                         stream);
     if (pr != kPersistentUnsupported) return pr;
   }
   CUtensorMap tmW, tmX;
@@ -820,10 +829,10 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   p.work = nullptr;
   p.w_rows_per_expert = 0;
   p.staged = 0;
-  p.act = 0;
+  p.act = (flags & 2) && !dual ? 2 : 0;
   p.act_limit = 0.f;
   p.bias_expert_stride = 0;
-  // flag bit 0: W was produced by a preceding kernel of the stream (no early fetch at all). Otherwise the ring's
+  // flag bit 1: squared ReLU of the output (plain tiles). Flag bit 0: W was produced by a preceding kernel of the stream (no early fetch at all). Otherwise the ring's
   // first stages are fetched before the dependency wait (level 1), and for matrices that fit L2 many times over
   // the remaining tiles are prefetched into L2 as well (level 2). EREDU_GEMM_PREFETCH overrides the level.
   p.w_static = (flags & 1) ? 0 : prefetch_level(static_cast<long long>(w_rows) * K * 2);

@@ -1,0 +1,249 @@
+// Glue of decoders that keep their residual stream in fp32 and normalise a sublayer's OUTPUT before it is added:
+//   * rms_residual: x = residual + w * y / rms(y), in fp32, plus the copy of x in the compute dtype that the next
+//     projections read (one number or one vector as w; without a residual: a plain norm, as in front of the head)
+//   * embedding_stream: the first rows of the stream and their copy
+//   * qkv_prepare: RMSNorm over the WHOLE query and key projections, rotation of the leading dims of every head, RMSNorm of
+//     every value head, and the append to the paged cache, whose key and value widths may differ
+// All of them for bf16 and for fp32 activations.
+#include "../common/elem.cuh"
+#include "../common/launch.h"
+#include "../common/launch_count.h"
+#include "../common/ptx.cuh"
+
+namespace eredu {
+
+// One CTA per row; NV groups of four columns per thread stay in registers between the two passes. NV = 0: any width, the
+// row is read twice.
+template <typename TY, int NV>
+__global__ void __launch_bounds__(256) rms_residual_kernel(const TY* __restrict__ y, const float* __restrict__ w, int w_vec,
+                                                            const float* __restrict__ residual, float* __restrict__ x_out,
+                                                            __nv_bfloat16* __restrict__ act, int W, float eps) {
+  __shared__ float red[8];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t base = static_cast<size_t>(blockIdx.x) * W;
+  const float w0 = w[0];
+  if constexpr (NV > 0) {
+    float4 v[NV], rv[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      v[i] = rv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < W) {
+        v[i] = load4(y + base + c);
+        if (residual != nullptr) rv[i] = load4(residual + base + c);
+      }
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / static_cast<float>(W) + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= W) continue;
+      const float4 g = w_vec ? load4(w + c) : make_float4(w0, w0, w0, w0);
+      const float4 o = make_float4(rv[i].x + v[i].x * inv * g.x, rv[i].y + v[i].y * inv * g.y, rv[i].z + v[i].z * inv * g.z,
+                                   rv[i].w + v[i].w * inv * g.w);
+      if (x_out != nullptr) store4(x_out + base + c, o);
+      if (act != nullptr) store4(act + base + c, o);
+    }
+  } else {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float t = to_f32(y[base + c]);
+      ss += t * t;
+    }
+    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / static_cast<float>(W) + eps);
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float o = (residual != nullptr ? residual[base + c] : 0.f) + to_f32(y[base + c]) * inv * (w_vec ? w[c] : w0);
+      if (x_out != nullptr) x_out[base + c] = o;
+      if (act != nullptr) act[base + c] = __float2bfloat16(o);
+    }
+  }
+}
+
+template <typename TY>
+static cudaError_t launch_rms_residual(const TY* y, const float* w, int w_vec, const float* residual, float* x_out, __nv_bfloat16* act,
+                                       int M, int W, float eps, cudaStream_t stream) {
+  const int quads = W % 4 == 0 ? (W / 4 + 255) / 256 : 0;
+#define ER_RMS(NV_) launch_pdl(rms_residual_kernel<TY, NV_>, dim3(M), dim3(256), 0, stream, y, w, w_vec, residual, x_out, act, W, eps)
+  switch (quads) {
+    case 1: return ER_RMS(1);
+    case 2: return ER_RMS(2);
+    case 3:
+    case 4: return ER_RMS(4);
+    case 5:
+    case 6:
+    case 7:
+    case 8: return ER_RMS(8);
+    default: return ER_RMS(0);
+  }
+#undef ER_RMS
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table,
+                                                                float* __restrict__ x, T* __restrict__ act, int W, int rows) {
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int id = ids[blockIdx.x];
+  const bool ok = id >= 0 && id < rows;
+  const T* src = table + static_cast<size_t>(ok ? id : 0) * W;
+  const size_t base = static_cast<size_t>(blockIdx.x) * W;
+  for (int c = threadIdx.x; c < W; c += 256) {
+    const T v = ok ? src[c] : from_f32<T>(0.f);
+    x[base + c] = to_f32(v);
+    if (act != nullptr) act[base + c] = v;
+  }
+}
+
+struct QkvPrepParams {
+  const void* qkv;
+  void* q_out;      // [M, n_q, dk]
+  void* k_cache;    // [pages, n_kv, 16, dk]
+  void* v_cache;    // [pages, n_kv, 16, dv]
+  const int* positions;
+  const long long* slots;     // page * 16 + offset, < 0 = do not store
+  const float* inv_freq;      // [rot / 2]
+  const float* q_norm_w;      // [n_q dk] or null
+  const float* k_norm_w;      // [n_kv dk] or null
+  int ld, n_q, n_kv, dk, dv, rot;
+  int value_norm, append;
+  float eps;
+};
+
+constexpr int kMaxRotPairs = 256;
+
+// One CTA per token.
+template <typename T>
+__global__ void __launch_bounds__(256) qkv_prepare_kernel(QkvPrepParams p) {
+  __shared__ float red[8];
+  __shared__ float cs[kMaxRotPairs], sn[kMaxRotPairs];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int m = blockIdx.x;
+  const int half = p.rot >> 1;
+  const T* row = static_cast<const T*>(p.qkv) + static_cast<size_t>(m) * p.ld;
+  const int qn = p.n_q * p.dk, kn = p.n_kv * p.dk;
+  const long long slot = p.slots[m];
+  const bool store = p.append && slot >= 0;
+  const float pos = static_cast<float>(p.positions[m]);
+  for (int i = threadIdx.x; i < half; i += 256) sincosf(pos * p.inv_freq[i], &sn[i], &cs[i]);
+  float sq = 0.f, sk = 0.f;
+  if (p.q_norm_w != nullptr)
+    for (int c = threadIdx.x; c < qn; c += 256) {
+      const float v = to_f32(row[c]);
+      sq += v * v;
+    }
+  if (store && p.k_norm_w != nullptr)
+    for (int c = threadIdx.x; c < kn; c += 256) {
+      const float v = to_f32(row[qn + c]);
+      sk += v * v;
+    }
+  const float q_inv = p.q_norm_w != nullptr ? 1.f / sqrtf(block_sum_f32(sq, red) / static_cast<float>(qn) + p.eps) : 1.f;
+  const float k_inv = p.k_norm_w != nullptr && p.append ? 1.f / sqrtf(block_sum_f32(sk, red) / static_cast<float>(kn) + p.eps) : 1.f;
+  __syncthreads();  // cs / sn
+  const int per = p.dk - half;  // rotation pairs and pass-through elements of a head
+  auto head = [&](const T* src, const float* w, float inv, int h, int j, T* dst) {
+    const int c = h * p.dk + j;
+    float u = to_f32(src[c]) * inv * (w != nullptr ? w[c] : 1.f);
+    if (j < half) {
+      const float v = to_f32(src[c + half]) * inv * (w != nullptr ? w[c + half] : 1.f);
+      dst[j] = from_f32<T>(u * cs[j] - v * sn[j]);
+      dst[j + half] = from_f32<T>(v * cs[j] + u * sn[j]);
+    } else {
+      dst[j + half] = from_f32<T>(to_f32(src[c + half]) * inv * (w != nullptr ? w[c + half] : 1.f));
+    }
+  };
+  T* q = static_cast<T*>(p.q_out) + static_cast<size_t>(m) * qn;
+  for (int i = threadIdx.x; i < p.n_q * per; i += 256) {
+    const int h = i / per, j = i - h * per;
+    head(row, p.q_norm_w, q_inv, h, j, q + static_cast<size_t>(h) * p.dk);
+  }
+  if (!store) return;
+  const size_t page = static_cast<size_t>(slot >> 4);
+  const int off = static_cast<int>(slot & 15);
+  T* kc = static_cast<T*>(p.k_cache);
+  for (int i = threadIdx.x; i < p.n_kv * per; i += 256) {
+    const int h = i / per, j = i - h * per;
+    head(row + qn, p.k_norm_w, k_inv, h, j, kc + ((page * p.n_kv + h) * 16 + off) * p.dk);
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  T* vc = static_cast<T*>(p.v_cache);
+  for (int h = warp; h < p.n_kv; h += 8) {
+    const T* src = row + qn + kn + static_cast<size_t>(h) * p.dv;
+    T* dst = vc + ((page * p.n_kv + h) * 16 + off) * p.dv;
+    float inv = 1.f;
+    if (p.value_norm) {
+      float ss = 0.f;
+      for (int c = lane; c < p.dv; c += 32) {
+        const float v = to_f32(src[c]);
+        ss += v * v;
+      }
+      inv = 1.f / sqrtf(warp_sum_f32(ss) / static_cast<float>(p.dv) + p.eps);
+    }
+    for (int c = lane; c < p.dv; c += 32) dst[c] = from_f32<T>(to_f32(src[c]) * inv);
+  }
+}
+
+}  // namespace eredu
+
+using namespace eredu;
+
+// y [M, W] bf16 (y_fp32 = 0) or fp32; w fp32 [1] (w_vec = 0) or [W]; residual, x_out fp32 [M, W] or null; act bf16 [M, W] or null.
+extern "C" int eredu_rms_residual(const void* y, const float* w, const float* residual, float* x_out, void* act, int M, int W,
+                                  int y_fp32, int w_vec, float eps, cudaStream_t stream) {
+  if (M <= 0 || W <= 0) return 0;
+  __nv_bfloat16* a = static_cast<__nv_bfloat16*>(act);
+  const cudaError_t e = y_fp32 ? launch_rms_residual(static_cast<const float*>(y), w, w_vec, residual, x_out, a, M, W, eps, stream)
+                               : launch_rms_residual(static_cast<const __nv_bfloat16*>(y), w, w_vec, residual, x_out, a, M, W, eps, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// table [rows, W] bf16 or fp32; x fp32 [M, W]; act [M, W] in the table's dtype or null.
+extern "C" int eredu_embedding_stream(const int* ids, const void* table, float* x, void* act, int M, int W, int rows, int fp32,
+                                      cudaStream_t stream) {
+  if (M <= 0 || W <= 0) return 0;
+  cudaError_t e;
+  if (fp32) e = launch_pdl(embedding_stream_kernel<float>, dim3(M), dim3(256), 0, stream, ids, static_cast<const float*>(table), x,
+                           static_cast<float*>(act), W, rows);
+  else e = launch_pdl(embedding_stream_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, stream, ids,
+                      static_cast<const __nv_bfloat16*>(table), x, static_cast<__nv_bfloat16*>(act), W, rows);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+extern "C" int eredu_qkv_prepare(const void* qkv, void* q_out, void* k_cache, void* v_cache, const int* positions,
+                                 const long long* slots, const float* inv_freq, const float* q_norm_w, const float* k_norm_w, int M,
+                                 int ld, int n_q, int n_kv, int dk, int dv, int rot, int value_norm, int append, int fp32, float eps,
+                                 cudaStream_t stream) {
+  if (M <= 0) return 0;
+  if (rot < 0 || rot > dk || rot % 2 != 0 || rot / 2 > kMaxRotPairs) return -1;
+  QkvPrepParams p;
+  p.qkv = qkv;
+  p.q_out = q_out;
+  p.k_cache = k_cache;
+  p.v_cache = v_cache;
+  p.positions = positions;
+  p.slots = slots;
+  p.inv_freq = inv_freq;
+  p.q_norm_w = q_norm_w;
+  p.k_norm_w = k_norm_w;
+  p.ld = ld;
+  p.n_q = n_q;
+  p.n_kv = n_kv;
+  p.dk = dk;
+  p.dv = dv;
+  p.rot = rot;
+  p.value_norm = value_norm;
+  p.append = append;
+  p.eps = eps;
+  const cudaError_t e = fp32 ? launch_pdl(qkv_prepare_kernel<float>, dim3(M), dim3(256), 0, stream, p)
+                             : launch_pdl(qkv_prepare_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, stream, p);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}

@@ -1,0 +1,221 @@
+// CUDA-core kernels in true 32-bit arithmetic: the linear layer and paged attention of models that run in fp32, and of bf16
+// shapes the tensor-core kernels do not take (row pitches a TMA descriptor cannot express, head sizes beyond 128 or not a
+// multiple of 8).
+#include "../common/elem.cuh"
+#include "../common/launch.h"
+#include "../common/launch_count.h"
+#include "../common/ptx.cuh"
+
+namespace eredu {
+
+constexpr int kTile = 64, kTileK = 16;
+
+// Y[M, N] = act(X[M, K] W[N, K]^T + bias): 64 x 64 outputs per CTA, 4 x 4 per thread, K in steps of 16 through shared memory.
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, TO* __restrict__ y,
+                                                         const T* __restrict__ bias, int M, int N, int K, int ldx, int ldw, int ldy,
+                                                         int act) {
+  __shared__ float xs[kTileK][kTile + 4], ws[kTileK][kTile + 4];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int n0 = blockIdx.x * kTile, m0 = blockIdx.y * kTile;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kTileK) {
+    for (int i = threadIdx.x; i < kTile * kTileK; i += 256) {
+      const int r = i / kTileK, k = i % kTileK;
+      xs[k][r] = (m0 + r < M && k0 + k < K) ? to_f32(x[static_cast<size_t>(m0 + r) * ldx + k0 + k]) : 0.f;
+      ws[k][r] = (n0 + r < N && k0 + k < K) ? to_f32(w[static_cast<size_t>(n0 + r) * ldw + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kTileK; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[k][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) break;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) break;
+      float v = acc[i][j] + (bias != nullptr ? to_f32(bias[n]) : 0.f);
+      if (act == 1) {
+        v = fmaxf(v, 0.f);
+        v *= v;
+      }
+      y[static_cast<size_t>(m) * ldy + n] = from_f32<TO>(v);
+    }
+  }
+}
+
+struct AttnSimtParams {
+  const void* q;         // [total_q, n_q, dk]
+  const void* k_cache;   // [pages, n_kv, 16, dk]
+  const void* v_cache;   // [pages, n_kv, 16, dv]
+  void* out;             // [total_q, n_q, dv]
+  const int* block_table;
+  const int* seq_lens;
+  const int* cu_q;       // null: q_per_seq queries per sequence
+  const float* sinks;    // [n_q] or null
+  int q_per_seq, max_pages, n_q, n_kv, dk, dv, window, chunk;
+  float scale;
+};
+
+constexpr int kMaxValueRegs = 16;  // value widths up to 512
+
+// One CTA per (query token, head); its four warps take every fourth group of 32 keys, one key per lane for the scores and
+// one value column per lane for the sum, each with a running maximum of its own; merged at the end.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_simt_kernel(AttnSimtParams p) {
+  extern __shared__ float sm[];
+  float* qs = sm;                      // [dk]
+  float* merge = sm + p.dk;            // [4][dv + 2]
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = blockIdx.z, h = blockIdx.y, qi = blockIdx.x;
+  const int q0 = p.cu_q != nullptr ? p.cu_q[b] : b * p.q_per_seq;
+  const int q_len = p.cu_q != nullptr ? p.cu_q[b + 1] - q0 : p.q_per_seq;
+  if (qi >= q_len) return;
+  const int pos = p.seq_lens[b] - q_len + qi;
+  const int kvh = h / (p.n_q / p.n_kv);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int* bt = p.block_table + static_cast<size_t>(b) * p.max_pages;
+  const T* q = static_cast<const T*>(p.q) + (static_cast<size_t>(q0 + qi) * p.n_q + h) * p.dk;
+  for (int i = threadIdx.x; i < p.dk; i += 128) qs[i] = to_f32(q[i]) * p.scale;
+  __syncthreads();
+  int lo = 0;
+  if (p.window > 0) lo = max(0, pos - p.window + 1);
+  else if (p.chunk > 0) lo = pos - pos % p.chunk;
+  float acc[kMaxValueRegs];
+#pragma unroll
+  for (int c = 0; c < kMaxValueRegs; ++c) acc[c] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  for (int k0 = lo + warp * 32; k0 <= pos; k0 += 128) {
+    const int key = k0 + lane;
+    const bool ok = key <= pos;
+    size_t row = 0;
+    float s = -INFINITY;
+    if (ok) {
+      row = (static_cast<size_t>(bt[key >> 4]) * p.n_kv + kvh) * 16 + (key & 15);
+      const T* k = static_cast<const T*>(p.k_cache) + row * p.dk;
+      s = 0.f;
+      for (int i = 0; i < p.dk; ++i) s = fmaf(qs[i], to_f32(k[i]), s);
+    }
+    float mx = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float m_new = fmaxf(m, mx);
+    const float corr = expf(m - m_new);
+    const float pe = ok ? expf(s - m_new) : 0.f;
+    m = m_new;
+    l = l * corr + warp_sum_f32(pe);
+    const int n = min(32, pos - k0 + 1);
+#pragma unroll
+    for (int c = 0; c < kMaxValueRegs; ++c) acc[c] *= corr;
+    for (int j = 0; j < n; ++j) {
+      const float pj = __shfl_sync(0xffffffffu, pe, j);
+      const size_t rj = __shfl_sync(0xffffffffu, static_cast<unsigned long long>(row), j);
+      const T* v = static_cast<const T*>(p.v_cache) + rj * p.dv;
+#pragma unroll
+      for (int c = 0; c < kMaxValueRegs; ++c)
+        if (lane + 32 * c < p.dv) acc[c] = fmaf(pj, to_f32(v[lane + 32 * c]), acc[c]);
+    }
+  }
+  float* mine = merge + warp * (p.dv + 2);
+#pragma unroll
+  for (int c = 0; c < kMaxValueRegs; ++c)
+    if (lane + 32 * c < p.dv) mine[lane + 32 * c] = acc[c];
+  if (lane == 0) {
+    mine[p.dv] = m;
+    mine[p.dv + 1] = l;
+  }
+  __syncthreads();
+  float M = p.sinks != nullptr ? p.sinks[h] : -INFINITY;
+  for (int w = 0; w < 4; ++w) M = fmaxf(M, merge[w * (p.dv + 2) + p.dv]);
+  float L = p.sinks != nullptr ? expf(p.sinks[h] - M) : 0.f, e[4];
+  for (int w = 0; w < 4; ++w) {
+    e[w] = expf(merge[w * (p.dv + 2) + p.dv] - M);
+    L += merge[w * (p.dv + 2) + p.dv + 1] * e[w];
+  }
+  T* out = static_cast<T*>(p.out) + (static_cast<size_t>(q0 + qi) * p.n_q + h) * p.dv;
+  for (int d = threadIdx.x; d < p.dv; d += 128) {
+    float o = 0.f;
+    for (int w = 0; w < 4; ++w) o += merge[w * (p.dv + 2) + d] * e[w];
+    out[d] = from_f32<T>(o / L);
+  }
+}
+
+}  // namespace eredu
+
+using namespace eredu;
+
+// X [M, K], W [N, K], bias [N] (or null) fp32 (in_fp32 = 1) or bf16; Y [M, N] fp32 or bf16. act 1: squared ReLU.
+extern "C" int eredu_gemm_simt(const void* x, const void* w, void* y, const void* bias, int M, int N, int K, int ldx, int ldw, int ldy,
+                               int in_fp32, int out_fp32, int act, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  const dim3 grid((N + kTile - 1) / kTile, (M + kTile - 1) / kTile);
+  if (grid.y > 65535) return -1;
+  cudaError_t e;
+  using B = __nv_bfloat16;
+  if (in_fp32) {
+    auto X = static_cast<const float*>(x);
+    auto Wt = static_cast<const float*>(w);
+    auto b = static_cast<const float*>(bias);
+    if (!out_fp32) return -1;
+    e = launch_pdl(gemm_simt_kernel<float, float>, grid, dim3(256), 0, stream, X, Wt, static_cast<float*>(y), b, M, N, K, ldx, ldw, ldy, act);
+  } else {
+    auto X = static_cast<const B*>(x);
+    auto Wt = static_cast<const B*>(w);
+    auto b = static_cast<const B*>(bias);
+    e = out_fp32 ? launch_pdl(gemm_simt_kernel<B, float>, grid, dim3(256), 0, stream, X, Wt, static_cast<float*>(y), b, M, N, K, ldx, ldw, ldy, act)
+                 : launch_pdl(gemm_simt_kernel<B, B>, grid, dim3(256), 0, stream, X, Wt, static_cast<B*>(y), b, M, N, K, ldx, ldw, ldy, act);
+  }
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// Causal attention over the paged cache for any key width and value widths up to 512; arguments as the tensor-core kernels.
+extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                               const int* seq_lens, const int* cu_q, const float* sinks, int batch, int q_per_seq, int max_q_len,
+                               int max_pages, int n_q, int n_kv, int dk, int dv, int window, int chunk, int fp32, float scale,
+                               cudaStream_t stream) {
+  if (batch <= 0 || max_q_len <= 0) return 0;
+  if (n_kv <= 0 || n_q % n_kv != 0 || dk <= 0 || dv <= 0 || dv > 32 * kMaxValueRegs || window < 0 || chunk < 0) return -1;
+  AttnSimtParams p;
+  p.q = q;
+  p.k_cache = k_cache;
+  p.v_cache = v_cache;
+  p.out = out;
+  p.block_table = block_table;
+  p.seq_lens = seq_lens;
+  p.cu_q = cu_q;
+  p.sinks = sinks;
+  p.q_per_seq = q_per_seq;
+  p.max_pages = max_pages;
+  p.n_q = n_q;
+  p.n_kv = n_kv;
+  p.dk = dk;
+  p.dv = dv;
+  p.window = window;
+  p.chunk = chunk;
+  p.scale = scale;
+  const size_t smem = (dk + 4 * (dv + 2)) * sizeof(float);
+  if (smem > 48 * 1024) return -1;
+  const dim3 grid(max_q_len, n_q, batch);
+  const cudaError_t e = fp32 ? launch_pdl(attn_simt_kernel<float>, grid, dim3(128), smem, stream, p)
+                             : launch_pdl(attn_simt_kernel<__nv_bfloat16>, grid, dim3(128), smem, stream, p);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}

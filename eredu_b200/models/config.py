@@ -16,6 +16,33 @@ QWEN_HYBRID_TYPES = {"qwen3_next", "qwen3_5", "qwen3_5_moe", "qwen3_5_text", "qw
 
 
 @dataclass
+class MixerSpec:
+    """Geometry and constants of one layer of a family whose layers do not share them (``ModelConfig.mixers``)."""
+    kind: str                        # "attention" | "gla" (gated linear attention) | "mingru"
+    heads: int = 0                   # query heads (attention) or recurrent heads (gla)
+    kv_heads: int = 0
+    dim: int = 0                     # query / key size of a head
+    vdim: int = 0                    # value size of a head
+    width: int = 0                   # mingru: channels
+    scale: float = 1.0               # attention: score multiplier
+    chunk: int = 0                   # attention: keys are visible inside the query's own chunk of positions (0: all earlier)
+    rot_dims: int = 0                # rotated leading dimensions of a head (0: no rotation)
+    rot_base: float = 10000.0
+    kv_from: int | None = None       # attention: the earlier layer whose cached keys and values are read
+    tau: float = 1.0                 # gla: decay = sigmoid(z)^(1 / tau)
+    ff: int = 0                      # feed-forward width (0: the layer has none)
+
+    @property
+    def state_shape(self) -> tuple | None:
+        """fp32 recurrent state of one sequence (None: no recurrence)."""
+        if self.kind == "mingru":
+            return (self.width,)
+        if self.kind == "gla":
+            return (self.heads, self.dim, self.vdim)
+        return None
+
+
+@dataclass
 class ModelConfig:
     model_type: str = "llama"
     vocab_size: int = 32000
@@ -84,6 +111,7 @@ class ModelConfig:
     eos_token_id: Any = None
     bos_token_id: Any = None
     torch_dtype: str = "bfloat16"
+    mixers: list[MixerSpec] | None = None   # per-layer geometry of families whose layers differ in kind and size
     extra: dict = field(default_factory=dict)
 
     @property
@@ -105,6 +133,21 @@ class ModelConfig:
             n = max(self.num_key_value_heads, int(g.get("num_global_key_value_heads") or 0))
             return n, d, d
         return self.num_key_value_heads, self.head_dim, self.head_dim
+
+    def layer_kv_dims(self, layer: int) -> tuple:
+        """(heads, key width, value width) of one cached token of this layer."""
+        if self.mixers is not None:
+            m = self.mixers[layer]
+            return m.kv_heads, m.dim, m.vdim
+        return self.kv_cache_dims
+
+    def layer_kv_donor(self, layer: int) -> int | None:
+        """The earlier layer whose cached keys and values this layer reads instead of keeping its own."""
+        return self.mixers[layer].kv_from if self.mixers is not None else None
+
+    def layer_state_shape(self, layer: int) -> tuple | None:
+        """fp32 state one sequence keeps in this layer, for families that state it per layer."""
+        return self.mixers[layer].state_shape if self.mixers is not None else None
 
     @property
     def rotary_dim(self) -> int:
@@ -141,6 +184,8 @@ class ModelConfig:
 
     def layer_has_kv(self, layer: int) -> bool:
         """The layer appends K/V pages (softmax attention); every other operator keeps a fixed state or none."""
+        if self.mixers is not None:
+            return self.mixers[layer].kind == "attention" and self.mixers[layer].kv_from is None
         if self.layer_types is None:
             return True
         if self.model_type == "gemma4":      # the KV-sharing tail reads an earlier layer's pages
@@ -149,10 +194,14 @@ class ModelConfig:
         return self.layer_types[layer] in ("full_attention", "sliding_attention", "attention_only")
 
     def layer_has_recurrent_state(self, layer: int) -> bool:
+        if self.mixers is not None:
+            return self.layer_state_shape(layer) is not None
         return self.layer_types is not None and self.layer_types[layer] in ("linear_attention", "mamba", "kda")
 
     @property
     def is_hybrid(self) -> bool:
+        if self.mixers is not None:
+            return any(m.state_shape is not None for m in self.mixers)
         return self.layer_types is not None and any(t in ("conv", "linear_attention", "mamba", "kda") for t in self.layer_types)
 
     def layer_window(self, layer: int) -> int:
@@ -163,7 +212,11 @@ class ModelConfig:
         return self.sliding_window
 
     def to_hf_dict(self) -> dict:
-        d = {k: v for k, v in asdict(self).items() if k not in ("extra", "qk_norm", "rope_traditional",
+        if self.model_type == "nidozen":
+            from .nidozen import config_dict
+
+            return config_dict(self)
+        d = {k: v for k, v in asdict(self).items() if k not in ("extra", "mixers", "qk_norm", "rope_traditional",
                                                                 "norm_weight_offset", "embedding_scale",
                                                                 "router_scoring", "attention_sinks", "quantization",
                                                                 "routed_scaling_factor", "n_group", "topk_group")}
@@ -243,6 +296,10 @@ class ModelConfig:
     # -------------------------------------------------------------------------------------- HF
     @classmethod
     def from_hf_dict(cls, d: dict) -> "ModelConfig":
+        if d.get("architecture") == "Nidozen" or d.get("model_type") == "nidozen":
+            from .nidozen import config_from_dict
+
+            return config_from_dict(cls, d)
         mt = d.get("model_type", "llama")
         if "text_config" in d and isinstance(d["text_config"], dict):
             outer = d

@@ -61,6 +61,16 @@ class ForwardBatch:
     # block drafters that condition on intermediate activations: the outputs of these layers (all rows) land in ``layer_hidden``
     capture_layers: Optional[tuple] = None
     layer_hidden: Optional[dict] = None
+    # families with an fp32 residual stream: (stream, its copy in the compute dtype) as the last sublayer left them
+    stream: Optional[tuple] = None
+    max_kv_len: int = 0                # decode: the longest context the step (or every replay of its graph) can see
+    sm_count: int = 1
+
+    def layer_splits(self, n_kv: int, chunk: int = 0) -> int:
+        """Split-KV factor of one layer in a decode step, for families whose layers see contexts of their own length.
+        At most the splits one thread-block cluster combines, so no scratch is needed."""
+        seen = min(self.max_kv_len, chunk) if chunk else self.max_kv_len
+        return min(ops.decode_splits(self.seq_lens.shape[0] * self.q_per_seq, n_kv, seen, self.sm_count), ops.CLUSTER_SPLITS)
 
 
 @dataclass
@@ -230,6 +240,10 @@ class CausalLM:
             from .muse_glimmer import block_forward as muse_block
 
             return muse_block(self, li, lw, h, batch, kv), None
+        if lw.block_kind == "nidozen":
+            from .nidozen import block_forward as nidozen_block
+
+            return nidozen_block(self, li, lw, h, batch, kv), None
         if lw.block_kind:
             from .nemotron_h import block_forward
 
@@ -313,7 +327,11 @@ class CausalLM:
         """Runs this shard's layers. Returns (h, ssq) - ssq is None unless the next consumer folds its norm."""
         fused = bool(self.layers) and self.layers[0].fold_attn and batch.token_ids.shape[0] <= self.FUSED_NORM_MAX_TOKENS
         ssq = None
-        if self.par.owns_embedding() and batch.hidden_in is None:
+        if self.cfg.model_type == "nidozen" and batch.hidden_in is None:
+            from .nidozen import enter
+
+            h = enter(self, batch)
+        elif self.par.owns_embedding() and batch.hidden_in is None:
             if fused:
                 h, ssq = ops.embedding(batch.token_ids, self.embed, 0, self.cfg.embedding_scale, want_ssq=True)
             else:
@@ -366,7 +384,11 @@ class CausalLM:
             h = h.index_select(0, rows)
             ssq = ssq.index_select(0, rows) if ssq is not None else None
         h = h.contiguous()
-        if self.head_folded:
+        if self.cfg.model_type == "nidozen":
+            from .nidozen import final_norm
+
+            h, ssq = final_norm(self, h), None
+        elif self.head_folded:
             if ssq is None or h.shape[0] > self.FUSED_NORM_MAX_TOKENS:
                 h, _ = ops.rmsnorm(h, self._ones(h.shape[1]), self.cfg.rms_norm_eps)
                 ssq = None
@@ -505,6 +527,10 @@ def build_from_tensors(cfg: ModelConfig, get: Callable[[str], torch.Tensor], has
     model = CausalLM(cfg, device, dtype, parallel)
     par = model.par
     tp, r = par.tp_size, par.tp_rank
+    if cfg.model_type == "nidozen":
+        from .nidozen import canonical_access
+
+        get, has = canonical_access(get, has)
 
     def up(t, dt=None):
         return t.to(device=model.device, dtype=dt or dtype).contiguous()
@@ -527,6 +553,14 @@ def build_from_tensors(cfg: ModelConfig, get: Callable[[str], torch.Tensor], has
         from .gemma4 import build as build_gemma4
 
         build_gemma4(model, cfg, get, has, up)
+        return model
+    if cfg.model_type == "nidozen":
+        from .nidozen import build as build_nidozen
+
+        if quantizer is not None or on_layer is not None:
+            raise NotImplementedError("Nidozen weights are dense and resident: no quantisation or host residency")
+        model.final_norm = model.final_norm.reshape(1)
+        build_nidozen(model, cfg, get, has, up)
         return model
     if cfg.model_type == "muse_glimmer":
         from .muse_glimmer import build as build_muse
@@ -673,6 +707,13 @@ def random_state(cfg: ModelConfig, seed: int = 0, std: float = 0.02, dtype=torch
     import zlib
 
     out: dict[str, torch.Tensor] = {}
+    if cfg.model_type == "nidozen":
+        from .nidozen import random_tensor, tensor_shapes
+
+        for name, shape in tensor_shapes(cfg).items():
+            g = torch.Generator(device="cpu").manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
+            out[name] = random_tensor(name, shape, g, std).to(dtype=dtype, device=device)
+        return out
 
     def mat(name, *shape):
         g = torch.Generator(device="cpu")
@@ -772,6 +813,16 @@ def build_random(cfg: ModelConfig, device, dtype, seed: int = 0, parallel=None, 
     import zlib
 
     dev = torch.device(device)
+    if cfg.model_type == "nidozen":
+        from .nidozen import random_tensor, tensor_shapes
+
+        shapes = tensor_shapes(cfg)
+
+        def draw(name: str) -> torch.Tensor:
+            g = torch.Generator(device=dev).manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
+            return random_tensor(name, shapes[name], g, std, dev).to(dtype)
+
+        return build_from_tensors(cfg, draw, shapes.__contains__, device, dtype, parallel)
 
     def get(name: str) -> torch.Tensor:
         shape = _shape_of(cfg, name)

@@ -27,8 +27,10 @@ def _sm_count(device) -> int:
 
 
 # ------------------------------------------------------------------------------------------ linear
-def linear_ref(x, w, bias=None, residual=None, out_dtype=None):
+def linear_ref(x, w, bias=None, residual=None, out_dtype=None, activation=None):
     y = F.linear(x.float(), w.float(), None if bias is None else bias.float())
+    if activation == "relu2":
+        y = torch.relu(y).square()
     if residual is not None:
         y = y + residual.float()
     return y.to(out_dtype or x.dtype)
@@ -52,19 +54,27 @@ def _norm_args(x, row_ssq, norm_eps, want_ssq, n_out):
 
 
 def linear(x, w, bias=None, residual=None, out_dtype=None, out=None, force_split=0, row_ssq=None, norm_eps=0.0,
-           want_ssq=False, dynamic_weight=False):
+           want_ssq=False, dynamic_weight=False, activation=None):
     """y = x @ w.T (+ bias) (+ residual). x: [M, K], w: [N, K].
 
     ``row_ssq`` ([M, parts] fp32 partial sums of squares of x's rows): the output rows are scaled by
     ``rsqrt(sum(row_ssq) / K + norm_eps)`` - an RMSNorm whose weight vector was folded into ``w``.
     ``want_ssq``: also return per-128-column-tile sums of squares of the stored output ([M, ceil(N/128)]).
     ``dynamic_weight``: ``w`` was written by a kernel enqueued just before this call (e.g. a dequantised scratch
-    matrix); the kernel then does not fetch weight tiles ahead of its stream dependency."""
+    matrix); the kernel then does not fetch weight tiles ahead of its stream dependency.
+    ``activation``: None or "relu2" (the square of ReLU), applied in the epilogue before the residual.
+    fp32 operands are multiplied in true 32-bit; bf16 operands whose rows a TMA descriptor cannot describe (a row pitch or
+    start that is not a multiple of 16 bytes) take the same CUDA-core kernel."""
+    if activation not in (None, "relu2"):
+        raise ValueError(f"unknown activation {activation!r}")
     if not x.is_cuda:
         if row_ssq is not None:
             x = x.float() * torch.rsqrt(row_ssq.sum(-1, keepdim=True) / x.shape[1] + norm_eps)
-        y = linear_ref(x, w, bias, residual, out_dtype or w.dtype)
+        y = linear_ref(x, w, bias, residual, out_dtype or w.dtype, activation)
         return (y, y.float().pow(2).sum(-1, keepdim=True)) if want_ssq else y
+    if x.dtype == torch.float32 or not (_tma_rows(x) and _tma_rows(w)):
+        assert residual is None and row_ssq is None and not want_ssq, "the CUDA-core linear has no norm or residual fusion"
+        return _linear_simt(x, w, bias, out_dtype or x.dtype, activation, out)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16, "CUDA linear is bf16"
     M, K = x.shape
     N = w.shape[0]
@@ -80,9 +90,33 @@ def linear(x, w, bias=None, residual=None, out_dtype=None, out=None, force_split
         ptr(x), ptr(w), ptr(out), ptr(residual), ptr(bias), M, N, K, x.stride(0), w.stride(0), out.stride(0),
         residual.stride(0) if residual is not None else 0, w.shape[0], 0, 0, 1 if out_dtype == torch.float32 else 0,
         force_split, _sm_count(x.device), ptr(status_word(x.device)), ptr(ssq_in), parts, eps, dim, ptr(ssq_out),
-        1 if dynamic_weight else 0, stream_ptr(x.device))
+        (1 if dynamic_weight else 0) | (2 if activation == "relu2" else 0), stream_ptr(x.device))
     check(code, "eredu_gemm_bf16")
     return (out, ssq_out) if want_ssq else out
+
+
+def _tma_rows(t) -> bool:
+    return t.stride(1) == 1 and (t.stride(0) * t.element_size()) % 16 == 0 and t.data_ptr() % 16 == 0
+
+
+native.register("eredu_gemm_simt", native.I, [native.P] * 4 + [native.I] * 9 + [native.P])
+
+
+def _linear_simt(x, w, bias, out_dtype, activation, out=None):
+    """fp32-accumulating GEMM on the CUDA cores: fp32 operands, or bf16 operands of any pitch."""
+    assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16) and x.stride(1) == 1 and w.stride(1) == 1
+    assert bias is None or (bias.dtype == x.dtype and bias.is_contiguous())
+    M, K = x.shape
+    N = w.shape[0]
+    if out is None:
+        out = torch.empty((M, N), dtype=out_dtype, device=x.device)
+    if M == 0:
+        return out
+    code = lib().eredu_gemm_simt(ptr(x), ptr(w), ptr(out), ptr(bias), M, N, K, x.stride(0), w.stride(0), out.stride(0),
+                                 1 if x.dtype == torch.float32 else 0, 1 if out.dtype == torch.float32 else 0,
+                                 1 if activation == "relu2" else 0, stream_ptr(x.device))
+    check(code, "eredu_gemm_simt")
+    return out
 
 
 def gated_linear(x, w_gate_up, inter, bias=None, out=None, force_split=0, row_ssq=None, norm_eps=0.0):
@@ -129,7 +163,106 @@ def rmsnorm(x, weight, eps, residual=None, weight_offset=0.0):
     return y, h
 
 
+native.register("eredu_rms_residual", native.I, [native.P] * 5 + [native.I] * 4 + [native.F, native.P])
+native.register("eredu_embedding_stream", native.I, [native.P] * 4 + [native.I] * 4 + [native.P])
+native.register("eredu_qkv_prepare", native.I, [native.P] * 9 + [native.I] * 10 + [native.F, native.P])
+
+
+def rms_residual_ref(y, weight, eps, residual=None, act_dtype=None):
+    n = y.float()
+    n = n * torch.rsqrt(n.square().mean(-1, keepdim=True) + eps) * weight.float()
+    if residual is not None:
+        n = residual + n
+    return n, n.to(act_dtype or y.dtype)
+
+
+def rms_residual(y, weight, eps, residual=None, act_dtype=None):
+    """Norm on a sublayer's output: ``x = residual + weight * y / rms(y)`` in fp32, and its copy in ``act_dtype``.
+    ``weight``: fp32, one number for all coordinates ([1]) or one per coordinate. Without a residual only the copy of the
+    normalised rows is made (the first result is then None, or the copy itself when it is fp32). Returns (x, copy)."""
+    act_dtype = act_dtype or y.dtype
+    if not y.is_cuda:
+        return rms_residual_ref(y, weight, eps, residual, act_dtype)
+    assert y.is_contiguous() and weight.dtype == torch.float32 and weight.numel() in (1, y.shape[1])
+    assert residual is None or (residual.dtype == torch.float32 and residual.is_contiguous())
+    M, W = y.shape
+    act = torch.empty((M, W), dtype=act_dtype, device=y.device)
+    fp32_act = act_dtype == torch.float32
+    x = act if fp32_act else (torch.empty((M, W), dtype=torch.float32, device=y.device) if residual is not None else None)
+    code = lib().eredu_rms_residual(ptr(y), ptr(weight), ptr(residual), ptr(x), None if fp32_act else ptr(act), M, W,
+                                    1 if y.dtype == torch.float32 else 0, 0 if weight.numel() == 1 else 1, eps,
+                                    stream_ptr(y.device))
+    check(code, "eredu_rms_residual")
+    return x, act
+
+
+def embedding_stream(ids, table):
+    """Rows of ``table`` as the start of an fp32 residual stream: (fp32 rows, rows in the table's dtype)."""
+    if not table.is_cuda:
+        act = table[ids.long()]
+        return act.float(), act
+    assert ids.dtype == torch.int32 and table.is_contiguous()
+    M, W = ids.shape[0], table.shape[1]
+    x = torch.empty((M, W), dtype=torch.float32, device=table.device)
+    fp32 = table.dtype == torch.float32
+    act = x if fp32 else torch.empty((M, W), dtype=table.dtype, device=table.device)
+    code = lib().eredu_embedding_stream(ptr(ids), ptr(table), ptr(x), None if fp32 else ptr(act), M, W, table.shape[0],
+                                        1 if fp32 else 0, stream_ptr(table.device))
+    check(code, "eredu_embedding_stream")
+    return x, act
+
+
 # ------------------------------------------------------------------------------------------ rope + kv append
+def qkv_prepare_ref(qkv, positions, slots, inv_freq, k_cache, v_cache, n_q, n_kv, dk, dv, q_norm_w=None, k_norm_w=None,
+                    norm_eps=1e-6, value_norm=False, append=True):
+    M = qkv.shape[0]
+    rot = 2 * inv_freq.shape[0]
+    ang = positions.float()[:, None] * inv_freq.float()[None, :]
+    cos, sin = ang.cos()[:, None, :], ang.sin()[:, None, :]
+
+    def rms(t):
+        return t * torch.rsqrt(t.square().mean(-1, keepdim=True) + norm_eps)
+
+    def project(t, w, heads):
+        if w is not None:
+            t = rms(t) * w.float()
+        t = t.view(M, heads, dk)
+        u, v = t[..., :rot // 2], t[..., rot // 2:rot]
+        return torch.cat((u * cos - v * sin, v * cos + u * sin, t[..., rot:]), -1)
+
+    x = qkv.float()
+    if append:
+        k = project(x[:, n_q * dk:(n_q + n_kv) * dk], k_norm_w, n_kv)
+        v = x[:, (n_q + n_kv) * dk:(n_q + n_kv) * dk + n_kv * dv].reshape(M, n_kv, dv)
+        v = rms(v) if value_norm else v
+        ok = slots >= 0
+        page, off = slots[ok] // PAGE, slots[ok] % PAGE
+        k_cache[page, :, off] = k[ok].to(k_cache.dtype)
+        v_cache[page, :, off] = v[ok].to(v_cache.dtype)
+    return project(x[:, :n_q * dk], q_norm_w, n_q).to(qkv.dtype).contiguous()
+
+
+def qkv_prepare(qkv, positions, slots, inv_freq, k_cache, v_cache, n_q, n_kv, dk, dv, q_norm_w=None, k_norm_w=None,
+                norm_eps=1e-6, value_norm=False, append=True):
+    """``qkv`` [M, n_q dk (+ n_kv dk + n_kv dv)]: RMSNorm over the WHOLE query and the whole key projection (weights of that
+    size; None: no norm), rotation of the first ``2 len(inv_freq)`` dims of every head (pairs i, i + half), optional
+    weight-free RMSNorm of every value head, keys and values scattered into their pages. ``append=False``: the rows hold
+    queries only (the layer reads another layer's pages). Returns q [M, n_q, dk] in qkv's dtype."""
+    if not qkv.is_cuda:
+        return qkv_prepare_ref(qkv, positions, slots, inv_freq, k_cache, v_cache, n_q, n_kv, dk, dv, q_norm_w, k_norm_w,
+                               norm_eps, value_norm, append)
+    assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and inv_freq.dtype == torch.float32
+    assert qkv.stride(1) == 1 and k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == qkv.dtype
+    M = qkv.shape[0]
+    q = torch.empty((M, n_q, dk), dtype=qkv.dtype, device=qkv.device)
+    code = lib().eredu_qkv_prepare(ptr(qkv), ptr(q), ptr(k_cache), ptr(v_cache), ptr(positions), ptr(slots), ptr(inv_freq),
+                                   ptr(q_norm_w), ptr(k_norm_w), M, qkv.stride(0), n_q, n_kv, dk, dv, 2 * inv_freq.shape[0],
+                                   1 if value_norm else 0, 1 if append else 0, 1 if qkv.dtype == torch.float32 else 0,
+                                   norm_eps, stream_ptr(qkv.device))
+    check(code, "eredu_qkv_prepare")
+    return q
+
+
 def rope_kv_ref(qkv, positions, slots, inv_freq, k_cache, v_cache, n_q, n_kv, head_dim, rot=None, interleaved=False,
                 attn_factor=1.0, q_norm_w=None, k_norm_w=None, norm_eps=1e-6, norm_w_off=0.0, mrope_section=None):
     """``positions`` [M], or [3, M] (temporal, height, width axes of multimodal prompts) with ``mrope_section``: frequency
@@ -207,14 +340,15 @@ def _gather_kv(cache, block_table_row, kv_len):
     return pages.permute(1, 0, 2, 3).reshape(cache.shape[1], n_pages * PAGE, cache.shape[3])[:, :kv_len]
 
 
-def attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, window=0, sinks=None, bidir=None):
+def attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, window=0, sinks=None, bidir=None, chunk=0):
     """q: [total_q, n_q, D]; the last q_lens[b] positions of sequence b are its queries (causal).
+    ``chunk``: a query sees the keys of its own chunk of positions [c * chunk, (c + 1) * chunk) only.
     ``bidir``: per sequence None or an int tensor [kv_len] of group ids (negative: none); positions of one group see each
     other in both directions, whatever the causal order and the window say (soft tokens of one image)."""
     total, n_q, D = q.shape
     n_kv = k_cache.shape[1]
     group = n_q // n_kv
-    out = torch.empty_like(q)
+    out = torch.empty((total, n_q, v_cache.shape[3]), dtype=q.dtype, device=q.device)
     start = 0
     for b, (kv_len, ql) in enumerate(zip(seq_lens.tolist(), q_lens)):
         k = _gather_kv(k_cache, block_table[b], kv_len).float()  # [n_kv, T, D]
@@ -228,6 +362,8 @@ def attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, win
         mask = kpos <= qpos
         if window > 0:
             mask = mask & (kpos > qpos - window)
+        if chunk > 0:
+            mask = mask & (kpos // chunk == qpos // chunk)
         if bidir is not None and bidir[b] is not None:
             grp = bidir[b].to(q.device)
             mask = mask | ((grp[kv_len - ql:kv_len, None] == grp[None, :kv_len]) & (grp[kv_len - ql:kv_len, None] >= 0))
@@ -245,23 +381,54 @@ def attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, win
 TC_PREFILL = _environ.get("EREDU_TC_PREFILL", "1") != "0"      # head size 64 / 128: the tcgen05 kernel (else the mma.sync one)
 
 
+native.register("eredu_attn_simt", native.I, [native.P] * 8 + [native.I] * 11 + [native.F, native.P])
+
+
+def _attention_simt(q, k_cache, v_cache, block_table, seq_lens, cu_q, q_per_seq, max_q_len, scale, window, chunk, sinks):
+    """Paged attention on the CUDA cores: fp32 caches, and head sizes the tensor-core kernels are not built for."""
+    assert q.is_contiguous() and k_cache.is_contiguous() and v_cache.is_contiguous() and q.dtype == k_cache.dtype == v_cache.dtype
+    out = torch.empty((q.shape[0], q.shape[1], v_cache.shape[3]), dtype=q.dtype, device=q.device)
+    if q.shape[0] == 0:
+        return out
+    code = lib().eredu_attn_simt(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), ptr(block_table), ptr(seq_lens), ptr(cu_q),
+                                 ptr(sinks), seq_lens.shape[0], q_per_seq, max_q_len, block_table.stride(0), q.shape[1],
+                                 k_cache.shape[1], q.shape[2], v_cache.shape[3], int(window), int(chunk),
+                                 1 if q.dtype == torch.float32 else 0, scale, stream_ptr(q.device))
+    check(code, "eredu_attn_simt")
+    return out
+
+
+def _tensor_core_dims(q, k_cache, v_cache) -> bool:
+    """Head sizes (multiples of 8 up to 128, keys and values may differ) and dtype of the tensor-core attention kernels."""
+    dk, dv = q.shape[2], v_cache.shape[3]
+    return (q.dtype == torch.bfloat16 and dk % 8 == 0 and dv % 8 == 0 and 0 < dk <= 128 and 0 < dv <= 128
+            and k_cache.is_contiguous() and v_cache.is_contiguous())
+
+
 def attention_prefill(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, scale, window=0, sinks=None,
-                      out=None):
-    if not q.is_cuda or q.shape[2] not in KERNEL_HEAD_DIMS:
+                      out=None, chunk=0):
+    """``window`` > 0: a query at position p sees keys in (p - window, p]; ``chunk`` > 0: the keys of its own chunk of
+    positions. Key and value widths are those of the caches. Returns [total_q, n_q, value width]."""
+    if q.is_cuda and (chunk > 0 or q.dtype == torch.float32 or v_cache.shape[3] != q.shape[2]):
+        if not _tensor_core_dims(q, k_cache, v_cache):
+            return _attention_simt(q, k_cache, v_cache, block_table, seq_lens, cu_q, 0, max_q_len, scale, window, chunk, sinks)
+    elif not q.is_cuda or q.shape[2] not in KERNEL_HEAD_DIMS:
         q_lens = (cu_q[1:] - cu_q[:-1]).tolist()
-        return attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, window, sinks)
+        return attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, window, sinks, chunk=chunk)
     assert q.dtype == torch.bfloat16 and q.is_contiguous()
     assert block_table.dtype == torch.int32 and seq_lens.dtype == torch.int32 and cu_q.dtype == torch.int32
+    dk, dv = q.shape[2], v_cache.shape[3]
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty((q.shape[0], q.shape[1], dv), dtype=q.dtype, device=q.device)
     B = seq_lens.shape[0]
-    if (TC_PREFILL and q.shape[2] in (64, 128) and k_cache.is_contiguous() and v_cache.is_contiguous()
-            and k_cache.shape[2] == 16 and k_cache.shape[3] == q.shape[2] and v_cache.shape == k_cache.shape and out.is_contiguous()
+    only_tc = chunk > 0 or dk != dv
+    if ((TC_PREFILL or only_tc) and (only_tc or dk in (64, 128)) and k_cache.is_contiguous() and v_cache.is_contiguous()
+            and k_cache.shape[2] == 16 and k_cache.shape[3] == dk and v_cache.shape[:3] == k_cache.shape[:3] and out.is_contiguous()
             and (sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous()))):
         # tcgen05 kernel (csrc/kernels/attention_tc.cu): QK^T and PV on the 5th-generation tensor cores, pages by TMA
         code = lib().eredu_attn_prefill_tc(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), ptr(block_table), ptr(seq_lens),
                                            ptr(cu_q), ptr(sinks), B, q.shape[0], max_q_len, block_table.stride(0),
-                                           k_cache.shape[0], q.shape[1], k_cache.shape[1], q.shape[2], int(window), scale,
+                                           k_cache.shape[0], q.shape[1], k_cache.shape[1], dk, dv, int(window), int(chunk), scale,
                                            ptr(status_word(q.device)), stream_ptr(q.device))
         check(code, "eredu_attn_prefill_tc")
         return out
@@ -296,17 +463,21 @@ def decode_splits(batch, n_kv, max_kv_len, sm_count=148):
 
 
 def attention_decode(q, k_cache, v_cache, block_table, seq_lens, q_per_seq, scale, splits=1, window=0, sinks=None,
-                     scratch=None, out=None):
-    """q: [B * q_per_seq, n_q, D]. ``scratch`` = (part_o, part_ml, counters) from :func:`decode_scratch` when
+                     scratch=None, out=None, chunk=0):
+    """q: [B * q_per_seq, n_q, D]; ``window`` / ``chunk`` as in :func:`attention_prefill`. ``scratch`` = (part_o, part_ml, counters) from :func:`decode_scratch` when
     splits > 1 (fp32 partials and zeroed int32 arrival tickets)."""
-    if not q.is_cuda or q.shape[2] not in KERNEL_HEAD_DIMS:
+    if q.is_cuda and (chunk > 0 or q.dtype == torch.float32 or v_cache.shape[3] != q.shape[2]):
+        if not _tensor_core_dims(q, k_cache, v_cache) or q.shape[1] // k_cache.shape[1] > 32:
+            return _attention_simt(q, k_cache, v_cache, block_table, seq_lens, None, q_per_seq, q_per_seq, scale, window, chunk,
+                                   sinks)
+    elif not q.is_cuda or q.shape[2] not in KERNEL_HEAD_DIMS:
         return attention_ref(q, k_cache, v_cache, block_table, seq_lens, [q_per_seq] * seq_lens.shape[0], scale,
-                             window, sinks)
+                             window, sinks, chunk=chunk)
     assert q.dtype == torch.bfloat16 and q.is_contiguous()
     B = seq_lens.shape[0]
-    n_q, D = q.shape[1], q.shape[2]
+    n_q, D = q.shape[1], v_cache.shape[3]
     if out is None:
-        out = torch.empty_like(q)
+        out = torch.empty((q.shape[0], n_q, D), dtype=q.dtype, device=q.device)
     part_o = part_ml = counters = None
     if splits > CLUSTER_SPLITS:
         if scratch is None:
@@ -316,7 +487,7 @@ def attention_decode(q, k_cache, v_cache, block_table, seq_lens, q_per_seq, scal
         assert counters.numel() >= B * k_cache.shape[1] and counters.dtype == torch.int32
     code = lib().eredu_attn_decode(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), ptr(block_table), ptr(seq_lens),
                                    ptr(sinks), ptr(part_o), ptr(part_ml), ptr(counters), B, q_per_seq, block_table.stride(0), n_q,
-                                   k_cache.shape[1], D, splits, window, scale, stream_ptr(q.device))
+                                   k_cache.shape[1], q.shape[2], D, splits, window, chunk, scale, stream_ptr(q.device))
     check(code, "eredu_attn_decode")
     return out
 

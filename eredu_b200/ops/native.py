@@ -21,10 +21,10 @@ _SIGNATURES = {
     "eredu_gemm_pick_split": (I, [I, I, I, I]),
     "eredu_gemm_bf16": (I, [P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, P, P, I, F, I, P, I, P]),
     "eredu_attn_prefill": (I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, P]),
-    "eredu_attn_decode": (I, [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P]),
+    "eredu_attn_decode": (I, [P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, P]),
     "eredu_peer_send": (I, [P, I, I, P, L, P, I, P, P]),
     "eredu_peer_recv": (I, [P, I, I, P, L, P, I, P, P]),
-    "eredu_attn_prefill_tc": (I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, F, P, P]),
+    "eredu_attn_prefill_tc": (I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P]),
     "eredu_attn_decode_scratch_elems": (None, [I, I, I, I, I, POINTER(L), POINTER(L)]),
     "eredu_attn_decode_rope": (I, [P, I, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, F, F, P]),
     "eredu_rmsnorm": (I, [P, P, P, P, P, I, I, F, F, P]),
@@ -38,6 +38,14 @@ _SIGNATURES = {
     "eredu_sample": (I, [P, P, I, P, P, I, P, P, I, I, P]),
     "eredu_spec_verify": (I, [P, P, P, P, P, I, I, I, P]),
 }
+
+
+def use_library(path) -> None:
+    """Load this build of the library instead of the complete one (``build.ensure_family``); before the first ``lib()``."""
+    global _LIB_PATH
+    if _lib is not None and Path(path) != _LIB_PATH:
+        raise RuntimeError("the CUDA library is loaded already")
+    _LIB_PATH = Path(path)
 
 
 def available() -> bool:

@@ -14,10 +14,12 @@ from typing import Optional
 import torch
 
 from . import native
-from .native import I, P, check, lib, ptr, stream_ptr
+from .native import F, I, P, check, lib, ptr, stream_ptr
 
 native.register("eredu_gated_delta_scan", I, [P, P, P, P, P, P, P, I, I, I, I, I, I, P])
 native.register("eredu_mamba2_scan", I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, P])
+native.register("eredu_mingru_scan", I, [P] * 7 + [I] * 7 + [P])
+native.register("eredu_gla_scan", I, [P] * 10 + [I] * 10 + [F, F, P])
 
 
 # From this many tokens per call the chunk-parallel Mamba-2 form takes over from the token-by-token kernel (measured on a
@@ -235,3 +237,101 @@ def mamba2_scan(x, B, C, dt, A, D, state: Optional[torch.Tensor] = None):
                                    P_, N, stream_ptr(x.device))
     check(code, "eredu_mamba2_scan")
     return S, out
+
+
+# ---------------------------------------------------------------------------------------------- ragged recurrences
+# The operators below take the rows of a whole batch - portions of prompts of any length beside single decoded tokens -
+# and find each sequence's fp32 state on the device: state[page_to_slot[first page of the sequence]]. ``batch`` gives the
+# rows of every sequence (``cu_q`` or ``q_per_seq`` each), the block table and the cache slots; a sequence whose first row has
+# no cache slot (an idle row of a captured decode batch) leaves its state alone.
+def _sequences(batch):
+    B = batch.block_table.shape[0]
+    return batch.cu_q.tolist() if batch.is_prefill else [i * batch.q_per_seq for i in range(B + 1)]
+
+
+def mingru_scan_ref(proj, state, width, batch, page_to_slot):
+    out = torch.zeros((proj.shape[0], width), dtype=proj.dtype, device=proj.device)
+    z, u, g = (proj[:, i * width:(i + 1) * width].float() for i in range(3))
+    z, cand = torch.sigmoid(z), torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    bounds = _sequences(batch)
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(batch.slots[r0]) < 0:
+            continue
+        slot = int(page_to_slot[int(batch.block_table[b, 0])])
+        S = state[slot].clone()
+        for t in range(r0, r1):
+            S = (1 - z[t]) * S + z[t] * cand[t]
+            out[t] = (S * torch.nn.functional.silu(g[t])).to(out.dtype)
+        state[slot] = S
+    return out
+
+
+def mingru_scan(proj, state, width, batch, page_to_slot):
+    """minGRU: ``proj`` [M, 3 width] = [z | u | gate]; ``S <- (1 - sigmoid(z)) S + sigmoid(z) c(u)`` with ``c(u) = u + 1/2``
+    for u >= 0 and ``sigmoid(u)`` below, output ``S * silu(gate)`` [M, width]. ``state`` fp32 [slots, width], in place."""
+    if not proj.is_cuda:
+        return mingru_scan_ref(proj, state, width, batch, page_to_slot)
+    assert proj.stride(1) == 1 and state.is_contiguous() and state.dtype == torch.float32
+    out = torch.empty((proj.shape[0], width), dtype=proj.dtype, device=proj.device)
+    if proj.shape[0] == 0:
+        return out
+    code = lib().eredu_mingru_scan(ptr(proj), ptr(state), ptr(out), ptr(batch.block_table), ptr(page_to_slot),
+                                   ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), width, proj.stride(0),
+                                   batch.block_table.shape[0], batch.q_per_seq, batch.max_q_len if batch.is_prefill else
+                                   batch.q_per_seq, batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0,
+                                   stream_ptr(proj.device))
+    check(code, "eredu_mingru_scan")
+    return out
+
+
+def gla_scan_ref(q, k, v, log_decay, state):
+    """q, k, log_decay [T, H, D], v [T, H, V], state [H, D, V] (all fp32): ``S <- diag(exp(log_decay)) S + k v^T``,
+    ``o = S^T q``. Returns (o [T, H, V], state)."""
+    S, out = state.clone(), []
+    decay = torch.exp(log_decay)
+    for t in range(q.shape[0]):
+        S = S * decay[t][:, :, None] + k[t][:, :, None] * v[t][:, None, :]
+        out.append(torch.einsum("hdv,hd->hv", S, q[t]))
+    return torch.stack(out), S
+
+
+def gla_attention_ref(proj, a2, a2_b, norm_w, state, heads, dk, dv, tau, eps, batch, page_to_slot):
+    M, qk, vw = proj.shape[0], heads * dk, heads * dv
+    x = proj.float()
+    q, k = x[:, :qk].view(M, heads, dk) * dk ** -0.5, x[:, qk:2 * qk].view(M, heads, dk)
+    v, g = x[:, 2 * qk:2 * qk + vw].view(M, heads, dv), x[:, 2 * qk + vw:2 * qk + 2 * vw]
+    z = x[:, 2 * qk + 2 * vw:] @ a2.t() + a2_b
+    logd = (torch.nn.functional.logsigmoid(z) / tau).view(M, heads, dk)
+    out = torch.zeros((M, vw), dtype=proj.dtype, device=proj.device)
+    bounds = _sequences(batch)
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(batch.slots[r0]) < 0:
+            continue
+        slot = int(page_to_slot[int(batch.block_table[b, 0])])
+        o, state[slot] = gla_scan_ref(q[r0:r1], k[r0:r1], v[r0:r1], logd[r0:r1], state[slot])
+        o = o * torch.rsqrt(o.square().mean(-1, keepdim=True) + eps) * norm_w
+        out[r0:r1] = (o.reshape(r1 - r0, vw) * torch.nn.functional.silu(g[r0:r1])).to(out.dtype)
+    return out
+
+
+def gla_attention(proj, a2, a2_b, norm_w, state, heads, dk, dv, tau, eps, batch, page_to_slot):
+    """Gated linear attention over ``proj`` [M, 2 H dk + 2 H dv + r] = [q | k | v | gate | low-rank decay input]:
+    per head ``S <- diag(alpha) S + k v^T``, ``o = S^T q / sqrt(dk)`` with ``alpha = sigmoid(a2 low + a2_b)^(1 / tau)`` per key
+    channel; each head's o is RMS-normed (weight ``norm_w`` [dv]) and multiplied by ``silu(gate)``. ``a2`` fp32 [H dk, r];
+    ``state`` fp32 [slots, H, dk, dv], in place. Returns [M, H dv]."""
+    if not proj.is_cuda:
+        return gla_attention_ref(proj, a2, a2_b, norm_w, state, heads, dk, dv, tau, eps, batch, page_to_slot)
+    M = proj.shape[0]
+    assert proj.stride(1) == 1 and state.is_contiguous() and state.dtype == torch.float32 and a2.is_contiguous()
+    out = torch.empty((M, heads * dv), dtype=proj.dtype, device=proj.device)
+    if M == 0:
+        return out
+    code = lib().eredu_gla_scan(ptr(proj), ptr(a2), ptr(a2_b), ptr(norm_w), ptr(state), ptr(out), ptr(batch.block_table),
+                                ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv,
+                                a2.shape[1], proj.stride(0), batch.block_table.shape[0], batch.q_per_seq,
+                                batch.max_q_len if batch.is_prefill else batch.q_per_seq, batch.block_table.stride(0),
+                                1 if proj.dtype == torch.float32 else 0, tau, eps, stream_ptr(proj.device))
+    check(code, "eredu_gla_scan")
+    return out

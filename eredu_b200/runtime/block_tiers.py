@@ -26,6 +26,7 @@ import torch
 class BlockTierStore:
     def __init__(self, kv, host_bytes: int, disk_dir=None, disk_bytes: int = 0, copy_stream=None):
         self.kv = kv
+        kv.require_uniform("a lower tier for published pages")
         L, _, nkv, page, D = kv.k.shape
         self.k_elems = L * nkv * page * D
         self.v_elems = L * kv.v.shape[2] * kv.v.shape[3] * kv.v.shape[4]

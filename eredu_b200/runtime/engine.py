@@ -49,7 +49,8 @@ class Sequence:
 class Engine:
     def __init__(self, model: CausalLM, max_batch: int = 32, max_seq_len: int = 4096, num_pages: Optional[int] = None,
                  use_cuda_graph: Optional[bool] = None, prefill_chunk: int = 8192, hist_cap: int = 1024,
-                 prefix_cache: bool = False, kv_host_tier_bytes: int = 0, kv_disk_tier_dir=None, kv_disk_tier_bytes: int = 0):
+                 prefix_cache: bool = False, kv_host_tier_bytes: int = 0, kv_disk_tier_dir=None, kv_disk_tier_bytes: int = 0,
+                 state_slots: Optional[int] = None):
         self.model = model
         self.cfg = model.cfg
         self.device = model.device
@@ -62,25 +63,34 @@ class Engine:
         conv_layers = [li for li in local if self.cfg.layer_is_conv(li)]
         kv_layers = [li for li in local if self.cfg.layer_has_kv(li)]
         _, key_dim, value_dim = self.cfg.kv_cache_dims
+        layer_dims = donors = None
+        if self.cfg.mixers is not None:
+            layer_dims = {li: self.cfg.layer_kv_dims(li) for li in kv_layers}
+            donors = {li: self.cfg.layer_kv_donor(li) for li in local if self.cfg.layer_kv_donor(li) is not None}
         self.kv = PagedKVCache(model.num_local_layers(), model.n_kv_local, key_dim, num_pages, model.dtype,
                                self.device, first_layer=model.first_layer, value_dim=value_dim,
                                attention_layers=kv_layers,
                                conv_layers=conv_layers,
                                conv_channels=self.cfg.hidden_size // model.par.tp_size if conv_layers else 0,
-                               conv_hist=self.cfg.conv_l_cache - 1)
+                               conv_hist=self.cfg.conv_l_cache - 1, layer_dims=layer_dims, donors=donors)
+        # recurrent-state slots: by default twice the decode batch, so that prompts can be prefilled while a batch decodes
+        slots = max(2 * max_batch, 8) if state_slots is None else state_slots
+        shapes = {li: self.cfg.layer_state_shape(li) for li in local if self.cfg.layer_state_shape(li) is not None}
+        if shapes:
+            self.kv.enable_layer_states(shapes, slots)
         mamba_layers = [li for li in local if self.cfg.layer_is_mamba(li)]
         if mamba_layers:
             from ..models.nemotron_h import mamba_dims
 
             heads, _, _, conv_dim = mamba_dims(self.cfg, model.par.tp_size)
-            self.kv.enable_linear_attention_state(mamba_layers, slots=max(2 * max_batch, 8),
+            self.kv.enable_linear_attention_state(mamba_layers, slots=slots,
                                                   conv_hist=self.cfg.mamba_conv_kernel - 1, conv_channels=conv_dim, heads=heads,
                                                   dk=self.cfg.mamba_head_dim, dv=self.cfg.ssm_state_size)
         kda_layers = [li for li in local if self.cfg.layer_is_kda(li)]
         if kda_layers:
             c = self.cfg
             kh = c.linear_num_value_heads // model.par.tp_size
-            self.kv.enable_linear_attention_state(kda_layers, slots=max(2 * max_batch, 8), conv_hist=c.linear_conv_kernel_dim - 1,
+            self.kv.enable_linear_attention_state(kda_layers, slots=slots, conv_hist=c.linear_conv_kernel_dim - 1,
                                                   conv_channels=3 * kh * c.linear_value_head_dim,
                                                   heads=kh, dk=c.linear_value_head_dim,
                                                   dv=c.linear_value_head_dim)
@@ -89,7 +99,7 @@ class Engine:
             c = self.cfg
             tp = model.par.tp_size
             self.kv.enable_linear_attention_state(
-                la_layers, slots=max(2 * max_batch, 8), conv_hist=c.linear_conv_kernel_dim - 1,
+                la_layers, slots=slots, conv_hist=c.linear_conv_kernel_dim - 1,
                 conv_channels=(2 * c.linear_num_key_heads * c.linear_key_head_dim
                                + c.linear_num_value_heads * c.linear_value_head_dim) // tp,
                 heads=c.linear_num_value_heads // tp, dk=c.linear_key_head_dim, dv=c.linear_value_head_dim)
@@ -161,6 +171,28 @@ class Engine:
                 seq.pages = []
                 raise
         return seq
+
+    def open_sequence(self, sampling=None, eos_ids=()) -> Sequence:
+        """A sequence without a reservation: it gets pages as its tokens arrive (:meth:`forward_tokens`)."""
+        seq = Sequence(self._next_id, [], sampling or SamplingParams(), 0, tuple(eos_ids))
+        self._next_id += 1
+        return seq
+
+    def _reserve(self, seq: Sequence, total: int) -> None:
+        """Pages (and, with the first one, a recurrent-state slot) for ``total`` tokens."""
+        if total > self.max_seq_len:
+            raise ValueError(f"{total} tokens exceed max_seq_len {self.max_seq_len}")
+        need = PagedKVCache.pages_for(total) - len(seq.pages)
+        if need <= 0:
+            return
+        fresh = self.kv.alloc(need)
+        if not seq.pages and self.kv.page_to_slot is not None:
+            try:
+                self.kv.bind_state(fresh[0])
+            except RuntimeError:
+                self.kv.allocator.release(fresh)
+                raise
+        seq.pages = seq.pages + fresh
 
     def _lease_prefix_through_tiers(self, tokens, need: int) -> list:
         """The longest prefix of ``tokens`` (whole pages) that is published on the device or held in a lower tier: device
@@ -282,32 +314,15 @@ class Engine:
         return torch.cat(outs)
 
     def _prefill_group(self, seqs):
-        toks, pos, slots, cu, lens = [], [], [], [0], []
-        max_q = 0
+        entries = []
         for s in seqs:
             new = s.prompt[s.kv_len:]
             if getattr(self, "_limits", None) is not None:
                 new = new[:self._limits[s.seq_id]]
-            n = len(new)
-            p = np.arange(s.kv_len, s.kv_len + n)
-            pages = np.asarray(s.pages, dtype=np.int64)
-            toks.extend(new)
-            pos.append(p)
-            slots.append(pages[p // PAGE] * PAGE + (p % PAGE))
-            cu.append(cu[-1] + n)
-            lens.append(s.kv_len + n)
-            max_q = max(max_q, n)
-        batch = ForwardBatch(
-            token_ids=self._t(np.asarray(toks, dtype=np.int32), torch.int32),
-            positions=self._t(np.concatenate(pos).astype(np.int32), torch.int32),
-            slots=self._t(np.concatenate(slots), torch.int64),
-            block_table=self._block_table(seqs),
-            seq_lens=self._t(np.asarray(lens, dtype=np.int32), torch.int32),
-            is_prefill=True,
-            cu_q=self._t(np.asarray(cu, dtype=np.int32), torch.int32),
-            max_q_len=max_q,
-            logit_rows=self._t(np.asarray(cu[1:], dtype=np.int64) - 1, torch.int64),
-        )
+            entries.append((s, new))
+        counts = [len(new) for _, new in entries]
+        lens, max_q = [s.kv_len + n for s, n in zip(seqs, counts)], max(counts)
+        batch = self._ragged_batch(entries, np.cumsum(counts) - 1)
         with nvtx.annotate(f"prefill[{len(seqs)}x{max_q}]"):
             logits = self.model.forward(batch, self.kv)
         for s, n in zip(seqs, lens):
@@ -360,6 +375,7 @@ class Engine:
             "all_greedy": all(s.sampling.greedy for s in seqs),
             "scratch": ops.decode_scratch(B, 1, self.model.n_q_local, self.cfg.head_dim, splits, dev)
             if (self.cuda and splits > 1) else None,
+            "max_len": max_len,
             "graph": None,
             "host_tokens": torch.zeros(B, dtype=torch.int32).pin_memory() if self.cuda else None,
             "host_in": torch.zeros(B, dtype=torch.int32).pin_memory() if self.cuda else None,
@@ -369,6 +385,43 @@ class Engine:
             s.slot = i
 
     # ------------------------------------------------------------------------------------------ host-driven steps
+    def _ragged_batch(self, entries, logit_rows, decode_form: bool = False) -> ForwardBatch:
+        """One batch from (sequence, next tokens) pairs: portions of prompts of any length beside single decoded tokens.
+        ``decode_form``: a batch in which every sequence brings one token is laid out for the decode kernels. Pages for the
+        new tokens are already reserved."""
+        seqs = [s for s, _ in entries]
+        counts = [len(t) for _, t in entries]
+        pos = [np.arange(s.kv_len, s.kv_len + n) for s, n in zip(seqs, counts)]
+        pages = [np.asarray(s.pages, dtype=np.int64) for s in seqs]
+        lens = np.asarray([s.kv_len + n for s, n in zip(seqs, counts)], dtype=np.int32)
+        common = dict(
+            token_ids=self._t(np.concatenate([np.asarray(t, dtype=np.int32) for _, t in entries]), torch.int32),
+            positions=self._t(np.concatenate(pos).astype(np.int32), torch.int32),
+            slots=self._t(np.concatenate([pg[p // PAGE] * PAGE + p % PAGE for pg, p in zip(pages, pos)]), torch.int64),
+            block_table=self._block_table(seqs), seq_lens=self._t(lens, torch.int32), sm_count=self.sm_count,
+            logit_rows=self._t(np.asarray(logit_rows, dtype=np.int64), torch.int64))
+        if decode_form and max(counts) == 1:
+            longest = int(lens.max())
+            splits = ops.decode_splits(len(seqs), self.model.n_kv_local, longest, self.sm_count) if self.cuda else 1
+            return ForwardBatch(**common, is_prefill=False, q_per_seq=1, max_kv_len=longest, splits=splits)
+        cu = np.concatenate(([0], np.cumsum(counts))).astype(np.int32)
+        return ForwardBatch(**common, is_prefill=True, cu_q=self._t(cu, torch.int32), max_q_len=max(counts))
+
+    @torch.no_grad()
+    def forward_tokens(self, entries) -> torch.Tensor:
+        """Feed ``entries`` = [(sequence, next tokens, wanted places among them)] as one batch, continuing from what the cache
+        and the recurrent states hold, and return the logits of the wanted places in order ([wanted, vocab], fp32)."""
+        for s, tokens, _ in entries:
+            self._reserve(s, s.kv_len + len(tokens))
+        rows, base = [], 0
+        for _, tokens, want in entries:
+            rows.extend(base + int(w) for w in want)
+            base += len(tokens)
+        logits = self.model.forward(self._ragged_batch([(s, t) for s, t, _ in entries], rows, decode_form=True), self.kv)
+        for s, tokens, _ in entries:
+            s.kv_len += len(tokens)
+        return logits
+
     @torch.no_grad()
     def feed_logits(self, seq: Sequence, tokens: list[int], multimodal=None) -> torch.Tensor:
         """Append ``tokens`` to the sequence's cache and return the logits after the last one ([V], on the model's
@@ -440,7 +493,7 @@ class Engine:
             "splits": splits, "all_greedy": True,
             "scratch": ops.decode_scratch(B, 1, self.model.n_q_local, self.cfg.head_dim, splits, dev)
             if (self.cuda and splits > 1) else None,
-            "graph": None, "graphs": {},
+            "graph": None, "graphs": {}, "max_len": max_len,
             "host_tokens": torch.zeros(B, dtype=torch.int32).pin_memory() if self.cuda else None,
             "host_in": torch.zeros(B, dtype=torch.int32).pin_memory() if self.cuda else None,
         }
@@ -505,6 +558,15 @@ class Engine:
             st["active"].copy_(self._t(act, torch.int32))
         else:
             st["active"] = torch.as_tensor(act)
+        # a row that is held back has no cache slot in this step (recurrent layers then keep its state) and gets the slot of
+        # its position back when it steps again
+        pos = st["positions"].long()
+        page = st["block_table"].long().gather(1, (pos // PAGE).clamp_max(self.max_pages - 1)[:, None]).squeeze(1)
+        slots = torch.where(st["active"] > 0, page * PAGE + pos % PAGE, torch.full_like(page, -1))
+        if self.cuda:
+            st["slots"].copy_(slots)
+        else:
+            st["slots"] = slots
 
     def _refresh_mode(self, st) -> None:
         greedy = all(s is None or s.sampling.greedy for s in st["seqs"])
@@ -515,7 +577,7 @@ class Engine:
     def _decode_body(self, st):
         batch = ForwardBatch(token_ids=st["token_ids"], positions=st["positions"], slots=st["slots"],
                              block_table=st["block_table"], seq_lens=st["seq_lens"], is_prefill=False, q_per_seq=1,
-                             splits=st["splits"], scratch=st["scratch"])
+                             splits=st["splits"], scratch=st["scratch"], max_kv_len=st["max_len"], sm_count=self.sm_count)
         logits = self.model.forward(batch, self.kv)
         if logits is not None:
             ops.sample(logits, st["rows"], history=st["history"], out=st["sampled"], all_greedy=st["all_greedy"])
@@ -538,6 +600,8 @@ class Engine:
     def _host_driven(self) -> bool:
         """True when a forward pass needs the host between kernels (layerwise host residency, expert cache)."""
         m = self.model
+        if self.cfg.mixers is not None:
+            return getattr(m, "observer", None) is not None    # every operator of these families has a kernel for every size
         if self.cfg.head_dim not in (64, 128) or self.cfg.is_mla or self.cfg.model_type == "gemma4":
             return True    # no attention kernel for this head size: the tensor-operation path reads lengths on the host
         if getattr(m, "residency", None) is not None or getattr(getattr(m, "inner", m), "observer", None) is not None:

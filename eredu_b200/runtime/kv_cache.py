@@ -40,8 +40,11 @@ class PageAllocator:
 class PagedKVCache:
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, num_pages: int, dtype, device,
                  first_layer: int = 0, attention_layers=None, conv_layers=None, conv_channels: int = 0, conv_hist: int = 0,
-                 value_dim: Optional[int] = None):
-        """``attention_layers`` / ``conv_layers``: global indices of the layers that keep K/V pages respectively a
+                 value_dim: Optional[int] = None, layer_dims: Optional[dict] = None, donors: Optional[dict] = None):
+        """``layer_dims``: layer -> (kv heads, key width, value width) for families whose layers differ; layers of one
+        geometry share a pool tensor, so a page id is valid in every layer. ``donors``: layer -> the earlier layer whose
+        keys and values it reads (it keeps none of its own).
+        ``attention_layers`` / ``conv_layers``: global indices of the layers that keep K/V pages respectively a
         short-convolution state (hybrid models); by default every one of the ``n_layers`` layers keeps K/V.
         The convolution state pool [layer, page, conv_hist, channels] is indexed by a sequence's first page."""
         self.n_kv_heads, self.head_dim = n_kv_heads, head_dim
@@ -49,12 +52,24 @@ class PagedKVCache:
         self.first_layer = first_layer
         if attention_layers is None:
             attention_layers = list(range(first_layer, first_layer + n_layers))
-        self._kv_index = {li: i for i, li in enumerate(attention_layers)}
         self.n_layers = len(attention_layers)
-        self.k = torch.zeros((self.n_layers, num_pages, n_kv_heads, PAGE, head_dim), dtype=dtype, device=device)
-        # latent-attention models cache one row per token in ``k`` and nothing in ``v`` (value_dim 1 keeps the plumbing)
-        self.v = torch.zeros_like(self.k) if value_dim in (None, head_dim) else \
-            torch.zeros((self.n_layers, num_pages, n_kv_heads, PAGE, value_dim), dtype=dtype, device=device)
+        default = (n_kv_heads, head_dim, head_dim if value_dim is None else value_dim)
+        groups: dict = {}
+        for li in attention_layers:
+            groups.setdefault(tuple((layer_dims or {}).get(li, default)), []).append(li)
+        if not groups:
+            groups[default] = []
+        self.pools, self._kv_index = [], {}
+        for g, ((heads, dk, dv), members) in enumerate(groups.items()):
+            k = torch.zeros((len(members), num_pages, heads, PAGE, dk), dtype=dtype, device=device)
+            # latent-attention models cache one row per token in ``k`` and nothing in ``v`` (value_dim 1 keeps the plumbing)
+            v = torch.zeros_like(k) if dv == dk else torch.zeros((len(members), num_pages, heads, PAGE, dv), dtype=dtype,
+                                                                 device=device)
+            self.pools.append((k, v))
+            self._kv_index.update({li: (g, i) for i, li in enumerate(members)})
+        for li, donor in (donors or {}).items():
+            self._kv_index[li] = self._kv_index[donor]
+        self.k, self.v = self.pools[0]
         self._conv_index = {li: i for i, li in enumerate(conv_layers or [])}
         self.conv_state = None
         if self._conv_index:
@@ -70,7 +85,9 @@ class PagedKVCache:
         # `page_to_slot` (indexed by a sequence's first page, read on the device) finds it.
         self.la_conv_state = self.la_rec_state = self.page_to_slot = None
         self._la_index: dict = {}
+        self.layer_state: dict = {}          # layer -> fp32 [slots, *shape] of families whose layers keep states of their own shape
         self._free_state_slots: list[int] = []
+        self._slot_of_page: dict = {}
 
     def alloc(self, n: int) -> list:
         """Pages from the allocator. When lower tiers are attached (``block_tiers``), published pages that this
@@ -87,9 +104,18 @@ class PagedKVCache:
         n = len(self._la_index)
         self.la_conv_state = torch.zeros((n, slots, conv_hist, conv_channels), dtype=dt, device=dev)
         self.la_rec_state = torch.zeros((n, slots, heads, dk, dv), dtype=torch.float32, device=dev)
-        self.page_to_slot = torch.zeros(self.num_pages, dtype=torch.int32, device=dev)
+        self._make_slots(slots)
+
+    def enable_layer_states(self, shapes: dict, slots: int):
+        """fp32 recurrent states given per layer (``shapes``: layer -> shape of one sequence's state)."""
+        dev = self.k.device
+        self.layer_state = {li: torch.zeros((slots, *shape), dtype=torch.float32, device=dev) for li, shape in shapes.items()}
+        self._make_slots(slots)
+
+    def _make_slots(self, slots: int):
+        self.page_to_slot = torch.zeros(self.num_pages, dtype=torch.int32, device=self.k.device)
         self._free_state_slots = list(range(slots - 1, -1, -1))
-        self._slot_of_page: dict = {}
+        self._slot_of_page = {}
 
     def bind_state(self, first_page: int) -> int:
         """Give the sequence that starts at ``first_page`` a zeroed state slot."""
@@ -100,9 +126,14 @@ class PagedKVCache:
         slot = self._free_state_slots.pop()
         self._slot_of_page[int(first_page)] = slot
         self.page_to_slot[int(first_page)] = slot
-        self.la_conv_state[:, slot].zero_()
-        self.la_rec_state[:, slot].zero_()
+        for t in self._slot_views(slot):
+            t.zero_()
         return slot
+
+    def _slot_views(self, slot: int) -> list:
+        """The recurrent state of one slot in every tensor that is indexed by slots."""
+        views = [t[:, slot] for t in (self.la_conv_state, self.la_rec_state) if t is not None]
+        return views + [t[slot] for t in self.layer_state.values()]
 
     def unbind_state(self, first_page: int) -> None:
         if self.page_to_slot is None:
@@ -137,7 +168,7 @@ class PagedKVCache:
         """Every fixed-size state tensor a forward pass mutates in place (empty for attention-only models). A step that
         is run twice on the same inputs - a warm-up before graph capture - must put these back in between: unlike a
         K/V append, advancing a recurrent state is not idempotent."""
-        return [t for t in (self.conv_state, self.la_conv_state, self.la_rec_state) if t is not None]
+        return [t for t in (self.conv_state, self.la_conv_state, self.la_rec_state, *self.layer_state.values()) if t is not None]
 
     def snapshot_state(self, first_page: int):
         """Copies of this sequence's recurrent states (None for attention-only models)."""
@@ -147,7 +178,7 @@ class PagedKVCache:
         la = None
         if self.page_to_slot is not None:
             slot = self._slot_of_page[int(first_page)]
-            la = (self.la_conv_state[:, slot].clone(), self.la_rec_state[:, slot].clone())
+            la = tuple(t.clone() for t in self._slot_views(slot))
         return conv, la
 
     def restore_state(self, first_page: int, snap) -> None:
@@ -158,16 +189,22 @@ class PagedKVCache:
             self.conv_state[:, int(first_page)].copy_(conv)
         if la is not None:
             slot = self._slot_of_page[int(first_page)]
-            self.la_conv_state[:, slot].copy_(la[0])
-            self.la_rec_state[:, slot].copy_(la[1])
+            for t, saved in zip(self._slot_views(slot), la):
+                t.copy_(saved)
 
     def linear_attention_state(self, li: int):
         i = self._la_index[li]
         return self.la_conv_state[i], self.la_rec_state[i]
 
     def layer(self, li: int):
-        i = self._kv_index[li]
-        return self.k[i], self.v[i]
+        g, i = self._kv_index[li]
+        k, v = self.pools[g]
+        return k[i], v[i]
+
+    def require_uniform(self, what: str) -> None:
+        """Raised by the features that move pages of one geometry (lower tiers, parking)."""
+        if len(self.pools) > 1:
+            raise NotImplementedError(f"{what} needs one key / value geometry for all layers; this model has {len(self.pools)}")
 
     def conv_layer(self, li: int):
         return self.conv_state[self._conv_index[li]]
@@ -176,7 +213,8 @@ class PagedKVCache:
         extra = self.conv_state.numel() * self.conv_state.element_size() if self.conv_state is not None else 0
         if self.la_rec_state is not None:
             extra += self.la_rec_state.numel() * 4 + self.la_conv_state.numel() * self.la_conv_state.element_size()
-        return (self.k.numel() + self.v.numel()) * self.k.element_size() + extra
+        extra += sum(t.numel() * 4 for t in self.layer_state.values())
+        return sum((k.numel() + v.numel()) * k.element_size() for k, v in self.pools) + extra
 
     @staticmethod
     def pages_for(tokens: int) -> int:

@@ -54,6 +54,7 @@ class KVHostTier:
     def __init__(self, engine, options: Optional[PagedCacheOptions] = None):
         self.engine = engine
         self.kv = engine.kv
+        self.kv.require_uniform("parking sequences in a host tier")
         self.opt = options or PagedCacheOptions()
         if self.opt.block_size_tokens != PAGE:
             raise ValueError(f"the device pool uses {PAGE}-token pages")

@@ -13,6 +13,7 @@ tensor ranks for sparse models, and only then falls back to load-time 4-bit weig
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Optional
@@ -21,7 +22,7 @@ from ..models.config import DENSE_TYPES, MOE_TYPES, ModelConfig
 
 EXECUTION_PLAN_SCHEMA_VERSION = 2
 DEFAULT_MAX_MAPPED_SHARDS = 4
-SUPPORTED_TYPES = DENSE_TYPES | {"qwen3_moe", "mixtral", "gpt_oss", "lfm2_moe", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "nemotron_h", "deepseek_v3", "deepseek_v4", "inkling_mm_model", "muse_glimmer", "kimi_linear", "gemma4"}
+SUPPORTED_TYPES = DENSE_TYPES | {"qwen3_moe", "mixtral", "gpt_oss", "lfm2_moe", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "nemotron_h", "deepseek_v3", "deepseek_v4", "inkling_mm_model", "muse_glimmer", "kimi_linear", "gemma4", "nidozen"}
 
 
 # ---------------------------------------------------------------------------------------------- inspection
@@ -79,6 +80,10 @@ def required_tensors(cfg: ModelConfig) -> list[tuple]:
     if cfg.model_type == "inkling_mm_model":
         return [("model.embed_tokens.weight", "model.llm.embed.weight"), ("model.norm.weight", "model.llm.norm.weight"),
                 ("model.layers.0.self_attn.r_proj.weight", "model.llm.layers.0.attn.wr_du.weight")]
+    if cfg.model_type == "nidozen":
+        from ..models.nidozen import tensor_shapes
+
+        return [(n,) for n in tensor_shapes(cfg)]
     p = "model.layers.0."
     kind = cfg.layer_types[0] if cfg.layer_types else "full_attention"
     if cfg.model_type == "nemotron_h":
@@ -151,7 +156,7 @@ def inspect_artifact(path) -> ModelInspectionReport:
         for alternatives in required_tensors(cfg):
             if not any(sp in keys for name in alternatives for sp in spellings(name)):
                 issues.append(InspectionIssue("missing_tensor", "error", f"required tensor {alternatives[0]} is absent"))
-        if cfg.model_type not in SPEECH_TYPES and not cfg.tie_word_embeddings and "lm_head.weight" not in keys:
+        if cfg.model_type not in SPEECH_TYPES and cfg.mixers is None and not cfg.tie_word_embeddings and "lm_head.weight" not in keys:
             issues.append(InspectionIssue("missing_tensor", "error", "untied model without lm_head.weight"))
     elif path.is_file():
         try:
@@ -188,7 +193,7 @@ def inspect_artifact(path) -> ModelInspectionReport:
         sev = "error"
         issues.append(InspectionIssue("unsupported_architecture", sev, f"model type {cfg.model_type!r} has no adapter here"
                                       + (" (recognised sparse family)" if cfg.model_type in MOE_TYPES else "")))
-    if cfg.head_dim not in (64, 128):
+    if cfg.mixers is None and cfg.head_dim not in (64, 128):
         issues.append(InspectionIssue("head_dim", "warning", f"head_dim {cfg.head_dim}: attention kernels cover 64 and 128; "
                                       "other sizes run the reference path"))
     if not rep.has_tokenizer:
@@ -259,6 +264,15 @@ def _family_profile(cfg: ModelConfig, weight_bytes, b: int):
     capability.rs): bytes that grow with the whole context, bytes kept only inside the window, fixed state."""
     L = cfg.num_hidden_layers
     H = cfg.hidden_size
+    if cfg.mixers is not None:
+        # per-layer geometry: pages of the layers that keep keys and values, fp32 states of the recurrent ones
+        kv = [cfg.layer_kv_dims(li) for li in range(L) if cfg.layer_has_kv(li)]
+        state = sum(math.prod(cfg.layer_state_shape(li)) * 4 for li in range(L) if cfg.layer_state_shape(li) is not None)
+        from ..models.nidozen import tensor_shapes
+
+        wb = weight_bytes if weight_bytes is not None else sum(math.prod(s) for s in tensor_shapes(cfg).values()) * 2
+        return ModelResourceProfile(int(wb), int(sum(n * (dk + dv) for n, dk, dv in kv) * b), max(1, len(kv)),
+                                    state_bytes_per_sequence=int(state))
     if cfg.model_type == "gemma4":
         from ..models.gemma4 import geometry
 

@@ -215,6 +215,8 @@ def architecture_fingerprint(cfg) -> str:
             "layer_types", "conv_l_cache", "linear_conv_kernel_dim", "linear_num_key_heads", "linear_num_value_heads",
             "linear_key_head_dim", "linear_value_head_dim", "mamba_num_heads", "mamba_head_dim", "ssm_state_size",
             "mamba_conv_kernel", "kv_lora_rank", "qk_rope_head_dim")
+    if getattr(cfg, "mixers", None) is not None:
+        keys += ("mixers",)          # families whose layers each have a geometry of their own
     blob = json.dumps({k: getattr(cfg, k, None) for k in keys}, sort_keys=True, default=str)
     return hashlib.sha256(blob.encode()).hexdigest()
 
@@ -229,11 +231,14 @@ def model_identity(engine, checkpoint_fingerprint: str) -> dict:
     for li in range(first, first + n_local):
         if cfg.layer_has_kv(li):
             layout.append({"kind": "key_value", "attention": ({"sliding": int(window)} if window else "full"),
-                           "num_key_value_heads": int(model.n_kv_local), "head_dim": int(cfg.head_dim)})
+                           "num_key_value_heads": int(model.n_kv_local if cfg.mixers is None else cfg.layer_kv_dims(li)[0]),
+                           "head_dim": int(cfg.head_dim if cfg.mixers is None else cfg.layer_kv_dims(li)[1])})
+        elif cfg.layer_kv_donor(li) is not None:
+            layout.append({"kind": "stateless"})
         elif cfg.layer_is_conv(li):
             layout.append({"kind": "recurrent", "fixed_state": ["convolution"]})
         elif cfg.layer_has_recurrent_state(li):
-            layout.append({"kind": "recurrent", "fixed_state": ["convolution", "recurrent"]})
+            layout.append({"kind": "recurrent", "fixed_state": ["recurrent"] if cfg.mixers is not None else ["convolution", "recurrent"]})
         else:
             layout.append({"kind": "stateless"})
     return dict(model_family=cfg.model_type.split("_")[0], effective_model_type=cfg.model_type,
@@ -301,6 +306,8 @@ def save_prompt_cache(engine, seq, directory, checkpoint_fingerprint: str, prefi
             for li, i in engine.kv._la_index.items():
                 per_layer_states.setdefault(li, {})["convolution"] = la[0][i]
                 per_layer_states[li]["recurrent"] = la[1][i]
+            for li, t in zip(engine.kv.layer_state, la[len(la) - len(engine.kv.layer_state):]):
+                per_layer_states.setdefault(li, {})["recurrent"] = t
         for li in sorted(per_layer_states):
             for role, t in sorted(per_layer_states[li].items()):
                 t = t.contiguous().cpu()
@@ -419,6 +426,8 @@ def load_prompt_cache(engine, directory, tokens, checkpoint_fingerprint: str, sa
                 li = e["layer"]
                 if li in engine.kv._conv_index:
                     dst = engine.kv.conv_state[engine.kv._conv_index[li], int(first_page)]
+                elif li in engine.kv.layer_state:
+                    dst = engine.kv.layer_state[li][slot]
                 elif e["role"] == "convolution":
                     dst = engine.kv.la_conv_state[engine.kv._la_index[li], slot]
                 else:
