@@ -76,7 +76,7 @@ def host_sources() -> list[Path]:
 
 # Kernel sources a family needs when only it is to run (see ensure_family); every other use builds all of them.
 FAMILY_SOURCES = {
-    "nidozen": ("attention", "attention_tc", "gemm_persistent", "gemm_tcgen05", "gla", "launch_count", "mingru",
+    "nidozen": ("attention", "attention_tc", "gemm_persistent", "gemm_tcgen05", "gla", "gla_chunk", "launch_count", "mingru",
                 "residual_stream", "simt_fp32"),
 }
 

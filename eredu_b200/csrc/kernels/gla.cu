@@ -101,6 +101,8 @@ __global__ void __launch_bounds__(256) gla_step_kernel(GlaParams<T> p) {
   }
 }
 
+constexpr int kGlaChunkMinRows = 16;  // from this portion length on the chunk-parallel form takes over
+
 template <typename T>
 static cudaError_t launch_gla_step(const GlaParams<T>& p, cudaStream_t stream) {
   const int vec = p.dv % 4 == 0 ? 4 : 1;
@@ -116,8 +118,21 @@ static cudaError_t launch_gla_step(const GlaParams<T>& p, cudaStream_t stream) {
 
 using namespace eredu;
 
+// fp32 elements of scratch a bf16 call over `rows` rows of `batch` sequences can use (0: the token-by-token kernel serves it).
+extern "C" long long eredu_gla_scratch_elems(int heads, int dk, int dv, int rank, int ld, int rows, int batch, int max_rows) {
+  GlaParams<__nv_bfloat16> p = {};
+  p.H = heads;
+  p.dk = dk;
+  p.dv = dv;
+  p.rank = rank;
+  p.ld = ld;
+  if (max_rows < kGlaChunkMinRows || !gla_chunk_supported(p)) return 0;
+  return gla_chunk_count(rows, batch) * heads * dk * (static_cast<long long>(dv) + 1);
+}
+
+// scratch: fp32 [eredu_gla_scratch_elems(...)] of a bf16 call over `rows` rows, or null (token by token).
 extern "C" int eredu_gla_scan(const void* proj, const float* a2, const float* a2_b, const float* norm_w, float* state, void* out,
-                              const int* block_table, const int* page_to_slot, const int* cu_q, const long long* slots, int heads,
+                              float* scratch, int rows, const int* block_table, const int* page_to_slot, const int* cu_q, const long long* slots, int heads,
                               int dk, int dv, int rank, int ld, int batch, int q_per_seq, int max_rows, int max_pages, int fp32,
                               float tau, float eps, cudaStream_t stream) {
   if (batch <= 0 || max_rows <= 0) return 0;
@@ -131,7 +146,13 @@ extern "C" int eredu_gla_scan(const void* proj, const float* a2, const float* a2
   } else {
     GlaParams<__nv_bfloat16> p = {static_cast<const __nv_bfloat16*>(proj), a2, a2_b, norm_w, state, static_cast<__nv_bfloat16*>(out),
                                   heads, dk, dv, rank, ld, 1.f / tau, eps, r};
-    e = launch_gla_step(p, stream);
+    if (scratch != nullptr && max_rows >= kGlaChunkMinRows && gla_chunk_supported(p)) {
+      float* decay = scratch + gla_chunk_count(rows, batch) * heads * dk * dv;
+      e = launch_gla_chunks(p, max_rows, scratch, decay, stream);
+      eredu_count_launches(2);
+    } else {
+      e = launch_gla_step(p, stream);
+    }
   }
   eredu_count_launches(1);
   return static_cast<int>(e);

@@ -145,9 +145,11 @@ def build(model, cfg, get, has, up) -> None:
     f32 = lambda n: up(get(n), torch.float32)                                          # noqa: E731
     opt = lambda n: get(n) if has(n) else None                                         # noqa: E731
 
-    def fused(names):
-        """Rows of several projections of the same input as one matrix, with their biases (zero where there is none)."""
+    def fused(names, pad: int = 1):
+        """Rows of several projections of the same input as one matrix, with their biases (zero where there is none);
+        ``pad``: zero rows bring the last projection to a multiple of this."""
         mats, biases = [get(n) for n in names], [opt(n + ".b") for n in names]
+        mats[-1] = torch.nn.functional.pad(mats[-1], (0, 0, 0, -mats[-1].shape[0] % pad))
         bias = None
         if any(b is not None for b in biases):
             bias = up(torch.cat([b if b is not None else torch.zeros(m.shape[0], dtype=m.dtype, device=m.device) for m, b in zip(mats, biases)]))
@@ -166,8 +168,12 @@ def build(model, cfg, get, has, up) -> None:
             inv = base_inv_freq(s.rot_base, s.rot_dims) if s.rot_dims else torch.zeros(0)
             lw.extra = {"inv_freq": inv.to(device=model.device, dtype=torch.float32)}
         elif s.kind == "gla":
-            lw.wqkv, lw.bqkv = fused([p + n for n in ("q", "k", "v", "g", "a1")])
-            lw.extra = {"a2": f32(p + "a2"), "a2_b": f32(p + "a2.b"), "o_norm": f32(p + "norm")}
+            # the rank of the decay projection is padded to a multiple of 8 with zeros: rows of the fused projection are then
+            # a whole number of 16-byte pieces
+            lw.wqkv, lw.bqkv = fused([p + n for n in ("q", "k", "v", "g", "a1")], pad=8)
+            a2 = f32(p + "a2")
+            lw.extra = {"a2": torch.nn.functional.pad(a2, (0, -a2.shape[1] % 8)).contiguous(), "a2_b": f32(p + "a2.b"),
+                        "o_norm": f32(p + "norm")}
         else:
             lw.wqkv, lw.bqkv = fused([p + n for n in "zxg"])
         if s.ff:

@@ -19,7 +19,8 @@ from .native import F, I, P, check, lib, ptr, stream_ptr
 native.register("eredu_gated_delta_scan", I, [P, P, P, P, P, P, P, I, I, I, I, I, I, P])
 native.register("eredu_mamba2_scan", I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, P])
 native.register("eredu_mingru_scan", I, [P] * 7 + [I] * 7 + [P])
-native.register("eredu_gla_scan", I, [P] * 10 + [I] * 10 + [F, F, P])
+native.register("eredu_gla_scan", I, [P] * 7 + [I] + [P] * 4 + [I] * 10 + [F, F, P])
+native.register("eredu_gla_scratch_elems", native.L, [I] * 8)
 
 
 # From this many tokens per call the chunk-parallel Mamba-2 form takes over from the token-by-token kernel (measured on a
@@ -328,10 +329,17 @@ def gla_attention(proj, a2, a2_b, norm_w, state, heads, dk, dv, tau, eps, batch,
     out = torch.empty((M, heads * dv), dtype=proj.dtype, device=proj.device)
     if M == 0:
         return out
-    code = lib().eredu_gla_scan(ptr(proj), ptr(a2), ptr(a2_b), ptr(norm_w), ptr(state), ptr(out), ptr(batch.block_table),
-                                ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv,
-                                a2.shape[1], proj.stride(0), batch.block_table.shape[0], batch.q_per_seq,
-                                batch.max_q_len if batch.is_prefill else batch.q_per_seq, batch.block_table.stride(0),
-                                1 if proj.dtype == torch.float32 else 0, tau, eps, stream_ptr(proj.device))
+    batch_size = batch.block_table.shape[0]
+    rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
+    scratch = None
+    if proj.dtype == torch.bfloat16 and proj.data_ptr() % 16 == 0:
+        elems = int(lib().eredu_gla_scratch_elems(heads, dk, dv, a2.shape[1], proj.stride(0), M, batch_size, rows))
+        if elems:
+            scratch = torch.empty(elems, dtype=torch.float32, device=proj.device)
+    code = lib().eredu_gla_scan(ptr(proj), ptr(a2), ptr(a2_b), ptr(norm_w), ptr(state), ptr(out), ptr(scratch), M,
+                                ptr(batch.block_table), ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None,
+                                ptr(batch.slots), heads, dk, dv, a2.shape[1], proj.stride(0), batch_size, batch.q_per_seq, rows,
+                                batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, tau, eps,
+                                stream_ptr(proj.device))
     check(code, "eredu_gla_scan")
     return out

@@ -127,3 +127,88 @@ def greedy(cfg, w, prompt, n, dtype=torch.float64):
     for _ in range(n):
         ids.append(int(forward(cfg, w, ids, dtype)[-1].argmax()))
     return ids[len(prompt):]
+
+
+# ---------------------------------------------------------------------------------------------- models for the tests
+def attn(heads, kv, dim, vdim, chunk, rot, base=10000.0, scale=0.25, ff=0, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "mask": {"size": chunk}, "rot": {"dims": rot, "base": base},
+         "scale": scale}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def gla_layer(heads, dim, vdim, tau, ff=0):
+    return {"type": "gla", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def mingru_layer(width, ff=0):
+    return {"type": "mingru", "mixer": {"width": width}, "mlp": {"kind": "dense", "ff": ff} if ff else None}
+
+
+def config(width, vocab, layers, eps=1e-5):
+    return {"architecture": "Nidozen", "width": width, "vocab": vocab, "norm": {"eps": eps}, "layers": layers}
+
+
+def weights(cfg, seed=0, rank=8, gain=1.0):
+    """bf16-valued random weights that keep every path of the model loud: unit-variance projections, norms around one,
+    decays from almost none to strong."""
+    g = torch.Generator().manual_seed(seed)
+    W, w = cfg["width"], {}
+
+    def mat(name, rows, cols, s=1.0):
+        w[name] = torch.randn(rows, cols, generator=g) * (s * gain / math.sqrt(cols))
+
+    def vec(name, n, s=0.5, mean=0.0):
+        w[name] = torch.randn(n, generator=g) * s + mean
+
+    def number(name):
+        w[name] = torch.rand((), generator=g) + 0.5
+
+    w["embed"] = torch.randn(cfg["vocab"], W, generator=g)
+    mat("head", cfg["vocab"], W)
+    number("final.norm")
+    for i, layer in enumerate(cfg["layers"]):
+        m, p = layer["mixer"], f"l{i}.mix."
+        number(f"l{i}.norm1")
+        if layer["type"] == "mingru":
+            for n in "zxg":
+                mat(p + n, m["width"], W)
+            vec(p + "z.b", m["width"], 1.0, -1.5)        # slow and fast channels
+            vec(p + "x.b", m["width"])
+            mat(p + "o", W, m["width"])
+        elif layer["type"] == "gla":
+            qk, v = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+            for n, rows in (("q", qk), ("k", qk), ("v", v), ("g", v)):
+                mat(p + n, rows, W)
+            mat(p + "a1", rank, W)
+            mat(p + "a2", qk, rank)
+            vec(p + "a2.b", qk, 2.0, 2.0)
+            vec(p + "norm", m["vdim"], 0.3, 1.0)
+            mat(p + "o", W, v)
+        else:
+            q, k, v = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"]
+            mat(p + "q", q, W)
+            vec(p + "q.b", q)
+            vec(p + "q.norm", q, 0.3, 1.0)
+            if m.get("kv_from") is None:
+                mat(p + "k", k, W)
+                vec(p + "k.b", k)
+                vec(p + "k.norm", k, 0.3, 1.0)
+                mat(p + "v", v, W)
+                vec(p + "v.b", v)
+            mat(p + "o", W, m["heads"] * m["vdim"])
+            vec(p + "o.b", W)
+        if layer["mlp"]:
+            number(f"l{i}.norm2")
+            mat(f"l{i}.mlp.up", layer["mlp"]["ff"], W)
+            mat(f"l{i}.mlp.down", W, layer["mlp"]["ff"])
+    return {k: v.to(torch.bfloat16) for k, v in w.items()}
+
+
+def error(got, want):
+    """Largest over the rows: root mean square difference of the logits (mean removed), relative to the logits' own."""
+    got, want = got.double().cpu(), want.double()
+    d = got - want
+    d, c = d - d.mean(-1, keepdim=True), want - want.mean(-1, keepdim=True)
+    return float((d.square().mean(-1).sqrt() / c.square().mean().sqrt()).max())
