@@ -218,12 +218,10 @@ def kernel_numbers(size: str, T: int = 8192, B: int = 32, context: int = 2048) -
             x, kc, vc = rnd(M, Q), pool(), pool()
             return lambda: ops.rope_kv(x, kv.positions, kv.slots, inv, kc, vc, H, G, D, rot=D // 2, q_norm_w=hw, k_norm_w=hw)
 
-        add(f"{phase} qkv_prepare", "rope_kv (per-head norms)", M * Q * 4, 0, prep, like_prep)
+        if phase == "prefill":           # decode steps prepare inside the attention kernel
+            add(f"{phase} qkv_prepare", "rope_kv (per-head norms)", M * Q * 4, 0, prep, like_prep)
         # ---- attention
         n = T if phase == "prefill" else context
-        seen = min(n, CHUNK)
-        full = torch.full((1,), 0)
-        del full
         if phase == "prefill":
             pairs, like_pairs = n // CHUNK * CHUNK * CHUNK / 2, n * n / 2
 
@@ -239,14 +237,24 @@ def kernel_numbers(size: str, T: int = 8192, B: int = 32, context: int = 2048) -
             lo = (context - 1) % CHUNK + 1
             sp = kv.layer_splits(G, CHUNK)
 
-            def attn(i, chunk=CHUNK, splits=sp):
-                q, kc, vc = rnd(B, H, D), rnd(n_pages, G, 16, D), rnd(n_pages, G, 16, D)
-                return lambda: ops.attention_decode(q, kc, vc, kv.block_table, kv.seq_lens, 1, D ** -0.5, splits=splits, chunk=chunk)
+            def attn(i):
+                x, kc, vc = rnd(B, Q), rnd(n_pages, G, 16, D), rnd(n_pages, G, 16, D)
+                return lambda: ops.attention_decode_rope(x, kc, vc, kv.block_table, kv.seq_lens, 1, D ** -0.5, kv.positions, kv.slots, inv, H, G, D,
+                                                         q_norm_w=qw, k_norm_w=kw, norm_eps=1e-5, splits=sp, chunk=CHUNK, value_dim=D,
+                                                         norm_whole=True, value_norm=True)
 
-            add("decode attention, chunks", "full attention", B * lo * G * D * 4, 0, attn,
-                lambda i: attn(i, 0, ops.decode_splits(B, G, context)), B * context * G * D * 4, 0)
-            del seen
-    return rows + recurrent_numbers(size, add_rows=rows, add=add, T=T, B=B)
+            def like_attn(i, window=0):
+                x, kc, vc = rnd(B, Q), rnd(n_pages, G, 16, D), rnd(n_pages, G, 16, D)
+                sl = ops.decode_splits(B, G, window or context)
+                return lambda: ops.attention_decode_rope(x, kc, vc, kv.block_table, kv.seq_lens, 1, D ** -0.5, kv.positions, kv.slots, inv, H, G, D,
+                                                         rot=D // 2, q_norm_w=hw, k_norm_w=hw, norm_eps=1e-5, splits=sl, window=window)
+
+            add("decode attention from the projection, chunks", "the same, full context, per-head norms", B * lo * G * D * 4, 0, attn, like_attn,
+                B * context * G * D * 4, 0)
+            add("decode attention from the projection, chunks", "the same, window of a chunk, per-head norms", B * lo * G * D * 4, 0, attn,
+                lambda i: like_attn(i, CHUNK), B * CHUNK * G * D * 4, 0)
+    recurrent_numbers(size, add, T, B)
+    return rows
 
 
 def window_attention(T, n_pages, H, G, D, kv):
@@ -257,7 +265,7 @@ def window_attention(T, n_pages, H, G, D, kv):
     return make
 
 
-def recurrent_numbers(size, add_rows, add, T, B) -> list:
+def recurrent_numbers(size, add, T, B) -> None:
     """Recurrences beside the Mamba-2 scan (the operator the closest model runs) and the gated-delta kernel."""
     _, _, _, _, _, R, dk, dv = SIZES[size]
     qk, vw, rank = R * dk, R * dv, 16
@@ -300,8 +308,13 @@ def recurrent_numbers(size, add_rows, add, T, B) -> list:
             x, s = rnd(M, 3 * vw), torch.zeros(n, vw, device=DEV)
             return lambda: ops.mingru_scan(x, s, vw, bt, p2s)
 
+        def conv(i):
+            x, s = rnd(M, vw), torch.zeros(n, 3, vw, device=DEV, dtype=BF)
+            w, slot = torch.ones(vw, 4, device=DEV), torch.arange(n, device=DEV, dtype=torch.int32).view(-1, 1).contiguous()
+            return lambda: ops.short_conv(x, w, None, s, slot, bt.cu_q, bt.q_per_seq, bt.positions, bt.slots, M // n, mode=1)
+
         add(f"{phase} mingru", "mamba2_scan", M * vw * 8 + n * vw * 8, 0, mingru, mamba, mio, flops)
-    return []
+        add(f"{phase} mingru", "short_conv", M * vw * 8 + n * vw * 8, 0, mingru, conv, M * vw * 4 + n * vw * 12, 0)
 
 
 def run(sizes, steps: int, models: bool = True, kernels: bool = True) -> dict:

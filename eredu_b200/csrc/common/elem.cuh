@@ -33,6 +33,9 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f32(float x) { return x / (1.f + expf(-x)); }
+// The same from the approximate exponential and reciprocal (a few units in the last place), for bf16 results or inputs.
+__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+__device__ __forceinline__ float silu_fast(float x) { return x * sigmoid_fast(x); }
 // log(sigmoid(x)) without overflow for either sign
 __device__ __forceinline__ float log_sigmoid_f32(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 

@@ -50,6 +50,9 @@ struct AttnParams {
   const float* k_norm_w;      // optional [D]
   int ld_qkv, rot, interleaved;
   float attn_factor, norm_eps, norm_w_off;
+  int norm_whole;   // the norms run over the whole q and the whole k projection (weights of that size) instead of per head
+  int value_norm;   // weight-free RMSNorm of every new value head
+  int append;       // 0: qkv rows hold queries only, the keys and values of the step are in the pages already
   // splits > 1: 1 = the `splits` CTAs of a (sequence, kv head) form a thread-block cluster and combine their partial
   // results through distributed shared memory (no global scratch, no arrival tickets); 0 = scratch + last-arriver.
   int cluster_reduce;
@@ -66,9 +69,10 @@ __device__ __forceinline__ float ld_dsmem_f32(uint32_t cluster_addr) {
 // One head row of the projection output: optional RMSNorm over D (result rounded to bf16 like a module boundary),
 // rotation of the first `rot` dims by the token's position. Executed by one warp; lane l owns the pairs l, l + 32, ...
 // `store(i0, a, i1, b)` receives the finished element pairs.
+// `whole_inv` > 0: the projection's own 1 / rms, instead of the head's. Heads may be narrower than D (p.dk).
 template <int D, typename Store>
-__device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bfloat16* src, const float* nw, int pos,
-                                              int lane, Store store) {
+__device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bfloat16* src, const float* nw, float whole_inv,
+                                              int pos, int lane, Store store) {
   constexpr int PER = D / 64;  // pairs per lane
   const int rh = p.rot >> 1;
   float a[PER], b[PER];
@@ -84,16 +88,25 @@ __device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bf
       i0[j] = p.rot + 2 * (i - rh);
       i1[j] = i0[j] + 1;
     }
-    a[j] = __bfloat162float(src[i0[j]]);
-    b[j] = __bfloat162float(src[i1[j]]);
+    const bool in = 2 * i < p.dk;
+    a[j] = in ? __bfloat162float(src[i0[j]]) : 0.f;
+    b[j] = in ? __bfloat162float(src[i1[j]]) : 0.f;
     ss += a[j] * a[j] + b[j] * b[j];
   }
-  if (nw != nullptr) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float inv = rsqrtf(ss / static_cast<float>(D) + p.norm_eps);
+  if (nw != nullptr && p.norm_whole) {
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
+      if (2 * (lane + 32 * j) >= p.dk) continue;
+      a[j] *= whole_inv * nw[i0[j]];
+      b[j] *= whole_inv * nw[i1[j]];
+    }
+  } else if (nw != nullptr) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = rsqrtf(ss / static_cast<float>(p.dk) + p.norm_eps);
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+      if (2 * (lane + 32 * j) >= p.dk) continue;
       a[j] = __bfloat162float(__float2bfloat16(a[j] * inv * (nw[i0[j]] + p.norm_w_off)));
       b[j] = __bfloat162float(__float2bfloat16(b[j] * inv * (nw[i1[j]] + p.norm_w_off)));
     }
@@ -111,8 +124,16 @@ __device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bf
       a[j] = ra;
       b[j] = rb;
     }
-    store(i0[j], a[j], i1[j], b[j]);
+    if (2 * i < p.dk) store(i0[j], a[j], i1[j], b[j]);
   }
+}
+
+__device__ __forceinline__ float sum_squares8(uint4 v) {
+  const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+  float s = 0.f;
+#pragma unroll
+  for (int j = 0; j < 4; ++j) s += bf16_lo(u[j]) * bf16_lo(u[j]) + bf16_hi(u[j]) * bf16_hi(u[j]);
+  return s;
 }
 
 // Byte offset of 16-byte chunk `c` of row `r` in a [rows][D] bf16 tile with XOR swizzle.
@@ -340,6 +361,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   uint8_t* ring = newkv_s + kMaxFusedNew * (DK + DV) * 2;    // [4 warps][NSTAGE][K page, V page]
 
   __shared__ int s_last;
+  __shared__ float s_part[2][4], s_inv[2][kMaxFusedNew];   // fused path with norms over whole projections
   pdl_launch_early();
   trace_mark(kTraceAttnDecode, kTraceStart);
   const int split = blockIdx.x, kvh = blockIdx.y, b = blockIdx.z;
@@ -365,7 +387,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   // The launch that handles the first query tokens also appends the new K / V rows. A page fetched from the cache may
   // then still hold the old bytes of a new row, so the rows are patched into the shared-memory copy of their page
   // (from `newkv_s`) after it has landed: no fence and no ordering between the append and the page fetches is needed.
-  const bool appending = fused && p.t0 == 0;
+  const bool appending = fused && p.append && p.t0 == 0;
   const int new_pos0 = kv_len - p.q_per_seq;
   const int first_new_page = appending ? new_pos0 / kPage : 0x7fffffff;
   if (!fused) {
@@ -417,6 +439,32 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   load_page(first + 4, 1);
   cp_async_commit();
   if (fused) {
+    if (p.norm_whole) {
+      // ---- 1 / rms of the whole q (and k) projection of every new token: each CTA sums the row for itself
+      for (int t = 0; t < p.q_per_seq; ++t) {
+        const uint4* row = reinterpret_cast<const uint4*>(p.qkv + (static_cast<size_t>(b) * p.q_per_seq + t) * p.ld_qkv);
+        const int nq = p.n_q_heads * p.dk / 8, nk = appending ? p.n_kv_heads * p.dk / 8 : 0;
+        float sq = 0.f, sk = 0.f;
+        for (int i = threadIdx.x; i < nq; i += 128) sq += sum_squares8(row[i]);
+        for (int i = threadIdx.x; i < nk; i += 128) sk += sum_squares8(row[nq + i]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+          sq += __shfl_xor_sync(0xffffffffu, sq, o);
+          sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        }
+        if (lane == 0) {
+          s_part[0][warp] = sq;
+          s_part[1][warp] = sk;
+        }
+        __syncthreads();
+        if (threadIdx.x < 2) {
+          const float* r = s_part[threadIdx.x];
+          const float n = static_cast<float>((threadIdx.x == 0 ? p.n_q_heads : p.n_kv_heads) * p.dk);
+          s_inv[threadIdx.x][t] = rsqrtf((r[0] + r[1] + r[2] + r[3]) / n + p.norm_eps);
+        }
+        __syncthreads();
+      }
+    }
     // ---- q rows: norm + RoPE straight into the swizzled tile (rows beyond `rows` are zero)
     for (int r = warp; r < ROWS; r += 4) {
       auto put = [&](int i0, float a, int i1, float bb) {
@@ -426,8 +474,11 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
       if (r < rows) {
         const int t = p.t0 + r / group, hg = r % group;
         const size_t m = static_cast<size_t>(b) * p.q_per_seq + t;
-        rope_head_row<DK>(p, p.qkv + m * p.ld_qkv + static_cast<size_t>(kvh * group + hg) * DK, p.q_norm_w, p.positions[m],
-                         lane, put);
+        const int head = kvh * group + hg;
+        const float* nw = p.q_norm_w == nullptr ? nullptr : p.q_norm_w + (p.norm_whole ? head * p.dk : 0);
+        rope_head_row<DK>(p, p.qkv + m * p.ld_qkv + static_cast<size_t>(head) * p.dk, nw, p.norm_whole ? s_inv[0][t] : 0.f,
+                          p.positions[m], lane, put);
+        for (int i = p.dk / 2 + lane; i < DK / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
       } else {
         for (int i = lane; i < DK / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
       }
@@ -440,22 +491,37 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         const size_t m = static_cast<size_t>(b) * p.q_per_seq + t;
         const long long slot = p.slots[m];
         if (pg < page0 || pg >= page1 || slot < 0) continue;  // warp-uniform
-        const size_t dst = ((static_cast<size_t>(slot >> 4) * p.n_kv_heads + kvh) * kPage + static_cast<size_t>(slot & 15)) * DK;
-        __nv_bfloat16* kd = const_cast<__nv_bfloat16*>(p.k_cache) + dst;
-        __nv_bfloat16* vd = const_cast<__nv_bfloat16*>(p.v_cache) + dst;
-        __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(newkv_s) + static_cast<size_t>(t) * 2 * DK;
-        const __nv_bfloat16* krow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + kvh) * DK;
-        const __nv_bfloat16* vrow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + p.n_kv_heads + kvh) * DK;
-        rope_head_row<DK>(p, krow, p.k_norm_w, p.positions[m], lane, [&](int i0, float a, int i1, float bb) {
+        const size_t cell = (static_cast<size_t>(slot >> 4) * p.n_kv_heads + kvh) * kPage + static_cast<size_t>(slot & 15);
+        __nv_bfloat16* kd = const_cast<__nv_bfloat16*>(p.k_cache) + cell * p.dk;
+        __nv_bfloat16* vd = const_cast<__nv_bfloat16*>(p.v_cache) + cell * p.dv;
+        __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(newkv_s) + static_cast<size_t>(t) * (DK + DV);
+        const __nv_bfloat16* krow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + kvh) * p.dk;
+        const __nv_bfloat16* vrow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + p.n_kv_heads) * p.dk +
+                                    static_cast<size_t>(kvh) * p.dv;
+        const float* nw = p.k_norm_w == nullptr ? nullptr : p.k_norm_w + (p.norm_whole ? kvh * p.dk : 0);
+        rope_head_row<DK>(p, krow, nw, p.norm_whole ? s_inv[1][t] : 0.f, p.positions[m], lane, [&](int i0, float a, int i1, float bb) {
           const __nv_bfloat16 ha = __float2bfloat16(a), hb = __float2bfloat16(bb);
           kd[i0] = ha;
           kd[i1] = hb;
           ks[i0] = ha;
           ks[i1] = hb;
         });
-        for (int i = lane; i < DK / 2; i += 32) {
-          const uint32_t vv = reinterpret_cast<const uint32_t*>(vrow)[i];
-          reinterpret_cast<uint32_t*>(vd)[i] = vv;
+        for (int i = p.dk / 2 + lane; i < DK / 2; i += 32) reinterpret_cast<uint32_t*>(ks)[i] = 0u;
+        float v_inv = 1.f;
+        if (p.value_norm) {
+          float ss = 0.f;
+          for (int i = lane; i < p.dv / 2; i += 32) {
+            const uint32_t vv = reinterpret_cast<const uint32_t*>(vrow)[i];
+            ss += bf16_lo(vv) * bf16_lo(vv) + bf16_hi(vv) * bf16_hi(vv);
+          }
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+          v_inv = rsqrtf(ss / static_cast<float>(p.dv) + p.norm_eps);
+        }
+        for (int i = lane; i < DV / 2; i += 32) {
+          uint32_t vv = 2 * i < p.dv ? reinterpret_cast<const uint32_t*>(vrow)[i] : 0u;
+          if (p.value_norm) vv = pack_bf16x2(bf16_lo(vv) * v_inv, bf16_hi(vv) * v_inv);
+          if (2 * i < p.dv) reinterpret_cast<uint32_t*>(vd)[i] = vv;
           reinterpret_cast<uint32_t*>(ks + DK)[i] = vv;
         }
       }
@@ -839,8 +905,6 @@ static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_hea
   const int group = n_q_heads / n_kv_heads;
   if (group > 32 || key_dim <= 0 || key_dim > 128 || key_dim % 8 != 0 || value_dim <= 0 || value_dim > 128 || value_dim % 8 != 0)
     return -1;
-  // the fused form rotates and appends rows of one head size that fills its tile
-  if (p.qkv != nullptr && (key_dim != value_dim || (key_dim != 128 && key_dim != 64))) return -1;
   p.dk = key_dim;
   p.dv = value_dim;
   const int t_per = group > 16 ? 1 : (32 / group < q_per_seq ? 32 / group : q_per_seq);
@@ -911,11 +975,13 @@ extern "C" int eredu_attn_decode_rope(const void* qkv, int ld_qkv, void* k_cache
                                       const int* block_table, const int* seq_lens, const float* sinks, float* part_o,
                                       float* part_ml, int* counters, const int* positions, const long long* slots,
                                       const float* inv_freq, const float* q_norm_w, const float* k_norm_w, int batch,
-                                      int q_per_seq, int max_pages, int n_q_heads, int n_kv_heads, int head_dim, int rot,
-                                      int interleaved, int splits, int window, float scale, float attn_factor,
-                                      float norm_eps, float norm_w_off, cudaStream_t stream) {
-  if (qkv == nullptr || positions == nullptr || slots == nullptr || inv_freq == nullptr) return -1;
-  if (rot <= 0 || rot > head_dim || rot % 2 != 0 || ld_qkv % 2 != 0) return -1;
+                                      int q_per_seq, int max_pages, int n_q_heads, int n_kv_heads, int key_dim, int value_dim,
+                                      int rot, int interleaved, int splits, int window, int chunk, int norm_whole,
+                                      int value_norm, int append, float scale, float attn_factor, float norm_eps,
+                                      float norm_w_off, cudaStream_t stream) {
+  if (qkv == nullptr || positions == nullptr || slots == nullptr || (inv_freq == nullptr && rot > 0)) return -1;
+  if (rot < 0 || rot > key_dim || rot % 2 != 0 || ld_qkv % 2 != 0) return -1;
+  if (norm_whole && (ld_qkv % 8 != 0 || (reinterpret_cast<uintptr_t>(qkv) & 15) != 0)) return -1;
   AttnParams p = {};
   p.qkv = static_cast<const __nv_bfloat16*>(qkv);
   p.ld_qkv = ld_qkv;
@@ -938,6 +1004,10 @@ extern "C" int eredu_attn_decode_rope(const void* qkv, int ld_qkv, void* k_cache
   p.attn_factor = attn_factor;
   p.norm_eps = norm_eps;
   p.norm_w_off = norm_w_off;
+  p.norm_whole = norm_whole;
+  p.value_norm = value_norm;
+  p.append = append;
+  p.chunk = chunk;
   p.max_pages = max_pages;
   p.n_q_heads = n_q_heads;
   p.n_kv_heads = n_kv_heads;
@@ -945,7 +1015,7 @@ extern "C" int eredu_attn_decode_rope(const void* qkv, int ld_qkv, void* k_cache
   p.splits = splits < 1 ? 1 : (splits > 64 ? 64 : splits);
   p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
-  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, head_dim, head_dim, stream);
+  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, key_dim, value_dim, stream);
 }
 
 // ---------------------------------------------------------------------------------------------- no-allocation variant

@@ -26,9 +26,18 @@ __global__ void __launch_bounds__(256) gla_step_kernel(GlaParams<T> p) {
   float* as = ks + dk;          // [dk] decay
   float* lows = as + dk;        // [rank]
   float* os = lows + p.rank;    // [row groups][dv]
+  const int h = blockIdx.x;
+  if (p.seqs.cu_q == nullptr && (dv & 3) == 0) {
+    // Decode: the state is not touched by the projection in front of this launch, so it starts towards L2 before the wait
+    // (a row that turns out idle wastes a fetch of slot 0).
+    const int slot = p.seqs.page_to_slot[p.seqs.block_table[static_cast<size_t>(blockIdx.y) * p.seqs.max_pages]];
+    const char* base = reinterpret_cast<const char*>(p.state + (static_cast<size_t>(slot) * p.H + h) * dk * dv);
+    const size_t bytes = static_cast<size_t>(dk) * dv * sizeof(float);
+    for (size_t o = threadIdx.x * 1024; o < bytes; o += 256 * 1024)
+      bulk_prefetch_l2(base + o, static_cast<uint32_t>(bytes - o < 1024 ? bytes - o : 1024));
+  }
   pdl_wait();
   pdl_launch_dependents();
-  const int h = blockIdx.x;
   const RaggedSeq s = ragged_seq(p.seqs, blockIdx.y);
   if (s.rows <= 0) return;  // uniform
   const int qk = p.H * dk, vw = p.H * dv;
@@ -48,7 +57,15 @@ __global__ void __launch_bounds__(256) gla_step_kernel(GlaParams<T> p) {
       ks[i] = to_f32(row[qk + h * dk + i]);
       const float* a2 = p.a2 + static_cast<size_t>(h * dk + i) * p.rank;
       float z = p.a2_b[h * dk + i];
-      for (int j = 0; j < p.rank; ++j) z = fmaf(a2[j], lows[j], z);
+      if ((p.rank & 3) == 0) {
+#pragma unroll 4
+        for (int j = 0; j < p.rank; j += 4) {
+          const float4 w = load4(a2 + j);
+          z = fmaf(w.x, lows[j], fmaf(w.y, lows[j + 1], fmaf(w.z, lows[j + 2], fmaf(w.w, lows[j + 3], z))));
+        }
+      } else {
+        for (int j = 0; j < p.rank; ++j) z = fmaf(a2[j], lows[j], z);
+      }
       as[i] = expf(log_sigmoid_f32(z) * p.inv_tau);
     }
     __syncthreads();
@@ -60,7 +77,7 @@ __global__ void __launch_bounds__(256) gla_step_kernel(GlaParams<T> p) {
           v[e] = to_f32(row[2 * qk + h * dv + c * VEC + e]);
           o[e] = 0.f;
         }
-#pragma unroll 4
+#pragma unroll 8
         for (int r = grp; r < dk; r += groups) {
           float* cell = st + static_cast<size_t>(r) * dv + c * VEC;
           float x[VEC];

@@ -33,15 +33,16 @@ constexpr int kAStride = kChunk + 8;
 // Shared memory of one chunk: rows of a padded width so that ldmatrix and fragment loads are free of bank conflicts.
 struct ChunkSmem {
   bf16 *q, *k, *v, *ah, *al;   // q, k [64][ks]; v [64][vs]; scores hi / lo [64][kAStride]
-  float *bl, *R, *a2, *low;    // bl [64][ks]: log2 decay since the start of the token's block; R [5][dkp]: at block starts, end
-  int ks, vs, dkp;
+  float *bl, *R;               // bl [64][ks]: log2 decay since the start of the token's block; R [5][dkp]: at block starts, end
+  bf16 *low, *a2h, *a2l;       // inputs of the decays: low [64][rs], the expansion hi / lo [dkp][rs]
+  int ks, vs, dkp, rs;
 };
 
 __host__ __device__ inline int chunk_dkp(int dk) { return (dk + 15) & ~15; }
 __host__ __device__ inline size_t chunk_scores_bytes(int dk, int rank) {
   const size_t scores = 2 * kChunk * kAStride * sizeof(bf16);
-  const size_t inputs = (static_cast<size_t>(chunk_dkp(dk)) * (rank + 1) + static_cast<size_t>(kChunk) * rank) * sizeof(float);
-  return (scores > inputs ? scores : inputs) + 15 & ~static_cast<size_t>(15);
+  const size_t inputs = (2 * static_cast<size_t>(chunk_dkp(dk)) + kChunk) * (chunk_dkp(rank) + 8) * sizeof(bf16);
+  return ((scores > inputs ? scores : inputs) + 15) & ~static_cast<size_t>(15);
 }
 __host__ __device__ inline size_t chunk_smem_bytes(int dk, int dv, int rank) {
   const size_t ks = chunk_dkp(dk) + 8;
@@ -61,8 +62,10 @@ __device__ __forceinline__ ChunkSmem chunk_smem(uint8_t* base, int dk, int dv, i
   s.R = s.bl + kChunk * s.ks;
   s.ah = reinterpret_cast<bf16*>(s.R + 5 * s.dkp);
   s.al = s.ah + kChunk * kAStride;
-  s.a2 = reinterpret_cast<float*>(s.ah);   // dead before the scores are written
-  s.low = s.a2 + s.dkp * (rank + 1);
+  s.rs = chunk_dkp(rank) + 8;
+  s.low = s.ah;                            // dead before the scores are written
+  s.a2h = s.low + kChunk * s.rs;
+  s.a2l = s.a2h + s.dkp * s.rs;
   return s;
 }
 
@@ -70,6 +73,16 @@ __device__ __forceinline__ ChunkSmem chunk_smem(uint8_t* base, int dk, int dv, i
 __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(a, b);
   lo = pack_bf16x2(a - bf16_lo(hi), b - bf16_hi(hi));
+}
+
+// log2(sigmoid(x)) = min(x, 0) log2(e) - log2(1 + t), t = e^-|x|. The logarithm of 1 + t keeps its relative accuracy for small t
+// by the correction t / ((1 + t) - 1) (Goldberg, "What every computer scientist should know about floating-point arithmetic").
+__device__ __forceinline__ float log2_sigmoid(float x) {
+  const float y = x * 1.4426950408889634f;
+  const float t = ex2_approx(-fabsf(y));
+  const float u = 1.f + t;
+  const float l = u == 1.f ? t * 1.4426950408889634f : __log2f(u) * __fdividef(t, u - 1.f);
+  return fminf(y, 0.f) - l;
 }
 
 // Rows of the chunk and its decays. Tokens behind the portion: zero rows without decay.
@@ -92,30 +105,53 @@ __device__ __forceinline__ void load_chunk(const GlaParams<bf16>& p, const Chunk
     *reinterpret_cast<uint4*>(s.v + t * s.vs + c * 8) =
         t < n ? *reinterpret_cast<const uint4*>(rows + static_cast<size_t>(t) * p.ld + 2 * qk + h * p.dv + c * 8) : zero;
   }
-  for (int i = threadIdx.x; i < kChunk * p.rank; i += kThreads) {
-    const int t = i / p.rank, j = i % p.rank;
-    s.low[i] = t < n ? to_f32(rows[static_cast<size_t>(t) * p.ld + 2 * qk + 2 * vw + j]) : 0.f;
+  const int rp = s.rs - 8;                                        // rank, padded to whole steps of the products
+  for (int i = threadIdx.x; i < kChunk * rp; i += kThreads) {
+    const int t = i / rp, j = i % rp;
+    s.low[t * s.rs + j] = t < n && j < p.rank ? rows[static_cast<size_t>(t) * p.ld + 2 * qk + 2 * vw + j] : __float2bfloat16(0.f);
   }
-  for (int i = threadIdx.x; i < p.dk * p.rank; i += kThreads) {
-    const int c = i / p.rank, j = i % p.rank;
-    s.a2[c * (p.rank + 1) + j] = p.a2[static_cast<size_t>(h) * p.dk * p.rank + i];
+  for (int i = threadIdx.x; i < s.dkp * rp; i += kThreads) {
+    const int c = i / rp, j = i % rp;
+    const float w = c < p.dk && j < p.rank ? p.a2[(static_cast<size_t>(h) * p.dk + c) * p.rank + j] : 0.f;
+    const bf16 hi = __float2bfloat16(w);
+    s.a2h[c * s.rs + j] = hi;
+    s.a2l[c * s.rs + j] = __float2bfloat16(w - to_f32(hi));
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < kBlks * s.dkp; i += kThreads) {   // one (block, channel) per thread and round
-    const int blk = i / s.dkp, c = i % s.dkp;
-    const float bias = c < p.dk ? p.a2_b[h * p.dk + c] : 0.f;
-    const float* w = s.a2 + c * (p.rank + 1);
-    float acc = 0.f;
-#pragma unroll 4
-    for (int j = 0; j < kBlk; ++j) {
-      const int t = blk * kBlk + j;
-      if (c < p.dk && t < n) {
-        float z = bias;
-        for (int r = 0; r < p.rank; ++r) z = fmaf(w[r], s.low[t * p.rank + r], z);
-        acc += log_sigmoid_f32(z) * (p.inv_tau * 1.4426950408889634f);
-      }
-      s.bl[t * s.ks + c] = acc;
+  // z = low a2^T + bias on the tensor cores, one tile = one block of 16 tokens x 8 channels; the decays are summed along the
+  // tokens of the tile with shuffles (lane group g holds the rows g and g + 8)
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = lane >> 2, tig = lane & 3;
+  const int tiles = s.dkp / 8;
+  for (int i = warp; i < kBlks * tiles; i += 8) {
+    const int blk = i / tiles, c0 = (i % tiles) * 8;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int ks = 0; ks < rp; ks += 16) {
+      const bf16* lo = s.low + (blk * kBlk + g) * s.rs + ks + tig * 2;
+      const uint32_t a0 = *reinterpret_cast<const uint32_t*>(lo), a1 = *reinterpret_cast<const uint32_t*>(lo + 8 * s.rs);
+      const uint32_t a2 = *reinterpret_cast<const uint32_t*>(lo + 8), a3 = *reinterpret_cast<const uint32_t*>(lo + 8 * s.rs + 8);
+      const int off = (c0 + g) * s.rs + ks + tig * 2;
+      mma16816(acc, a0, a1, a2, a3, *reinterpret_cast<const uint32_t*>(s.a2h + off), *reinterpret_cast<const uint32_t*>(s.a2h + off + 8));
+      mma16816(acc, a0, a1, a2, a3, *reinterpret_cast<const uint32_t*>(s.a2l + off), *reinterpret_cast<const uint32_t*>(s.a2l + off + 8));
     }
+    const int c = c0 + tig * 2;
+    float d[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int ch = c + (e & 1), t = blk * kBlk + g + (e >> 1) * 8;
+      d[e] = ch < p.dk && t < n ? log2_sigmoid(acc[e] + p.a2_b[h * p.dk + ch]) * p.inv_tau : 0.f;
+    }
+#pragma unroll
+    for (int o = 4; o < 32; o <<= 1)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float up = __shfl_up_sync(0xffffffffu, d[e], o);
+        if (lane >= o) d[e] += up;
+      }
+    d[2] += __shfl_sync(0xffffffffu, d[0], 28 + tig);
+    d[3] += __shfl_sync(0xffffffffu, d[1], 28 + tig);
+    *reinterpret_cast<float2*>(s.bl + (blk * kBlk + g) * s.ks + c) = make_float2(d[0], d[1]);
+    *reinterpret_cast<float2*>(s.bl + (blk * kBlk + g + 8) * s.ks + c) = make_float2(d[2], d[3]);
   }
   __syncthreads();
   for (int c = threadIdx.x; c < s.dkp; c += kThreads) {
@@ -133,7 +169,7 @@ __device__ __forceinline__ int chunk_id(const RaggedSeq& s, int b, int c) { retu
 
 // ---------------------------------------------------------------- 1. contributions of the chunks
 template <int NT>
-__global__ void __launch_bounds__(kThreads) gla_chunk_state_kernel(GlaParams<bf16> p, float* __restrict__ ws, float* __restrict__ decay) {
+__global__ void __launch_bounds__(kThreads, NT <= 2 ? 2 : 1) gla_chunk_state_kernel(GlaParams<bf16> p, float* __restrict__ ws, float* __restrict__ decay) {
   extern __shared__ __align__(16) uint8_t smem[];
   pdl_launch_early();
   pdl_wait();
@@ -306,7 +342,7 @@ __device__ __forceinline__ void score_block(const ChunkSmem& s, int I, int J, fl
 }
 
 template <int NT>
-__global__ void __launch_bounds__(kThreads) gla_chunk_out_kernel(GlaParams<bf16> p, const float* __restrict__ ws) {
+__global__ void __launch_bounds__(kThreads, NT <= 2 ? 2 : 1) gla_chunk_out_kernel(GlaParams<bf16> p, const float* __restrict__ ws) {
   extern __shared__ __align__(16) uint8_t smem[];
   __shared__ float ssq[8][kChunk];
   pdl_launch_early();
@@ -317,6 +353,9 @@ __global__ void __launch_bounds__(kThreads) gla_chunk_out_kernel(GlaParams<bf16>
   const int t0 = blockIdx.x * kChunk;
   if (!seq.live || t0 >= seq.rows) return;  // uniform
   const ChunkSmem s = chunk_smem(smem, p.dk, p.dv, p.rank);
+  const float* S = ws + (static_cast<size_t>(chunk_id(seq, b, blockIdx.x)) * p.H + h) * p.dk * p.dv;
+  if (threadIdx.x < 32)                                           // on its way to L2 while the scores are formed
+    for (int r = threadIdx.x; r < p.dk; r += 32) bulk_prefetch_l2(S + static_cast<size_t>(r) * p.dv, p.dv * 4);
   load_chunk<true>(p, s, seq, h, t0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
@@ -345,8 +384,7 @@ __global__ void __launch_bounds__(kThreads) gla_chunk_out_kernel(GlaParams<bf16>
 #pragma unroll
     for (int m = 0; m < 4; ++m) acc[j][m][0] = acc[j][m][1] = acc[j][m][2] = acc[j][m][3] = 0.f;
   // ---- entering state: [64 x dk] x [dk x dv]; its fragments come straight from global memory, once per CTA
-  const float* S = ws + (static_cast<size_t>(chunk_id(seq, b, blockIdx.x)) * p.H + h) * p.dk * p.dv;
-#pragma unroll 2
+#pragma unroll 4
   for (int ks = 0; ks < s.dkp / 16; ++ks) {
     uint32_t bh[NT][2], bo[NT][2];
 #pragma unroll
@@ -409,8 +447,21 @@ __global__ void __launch_bounds__(kThreads) gla_chunk_out_kernel(GlaParams<bf16>
       ss += __shfl_xor_sync(0xffffffffu, ss, 2);
       if (tig == 0) ssq[warp][m * 16 + g + r * 8] = ss;
     }
-  __syncthreads();
   const int qk = p.H * p.dk, vw = p.H * p.dv;
+  uint32_t gate[4][2][NT];
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int t = t0 + m * 16 + g + r * 8;
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+        gate[m][r][j] = t < seq.rows && warp + 8 * j < nt
+                            ? *reinterpret_cast<const uint32_t*>(p.proj + static_cast<size_t>(seq.row0 + t) * p.ld + 2 * qk + vw + h * p.dv +
+                                                                 (warp + 8 * j) * 8 + tig * 2)
+                            : 0u;
+    }
+  __syncthreads();
 #pragma unroll
   for (int m = 0; m < 4; ++m)
 #pragma unroll
@@ -426,10 +477,10 @@ __global__ void __launch_bounds__(kThreads) gla_chunk_out_kernel(GlaParams<bf16>
       for (int j = 0; j < NT; ++j) {
         if (warp + 8 * j >= nt) continue;
         const int n = (warp + 8 * j) * 8 + tig * 2;
-        const uint32_t gate = *reinterpret_cast<const uint32_t*>(p.proj + row * p.ld + 2 * qk + vw + h * p.dv + n);
+        const uint32_t gt = gate[m][r][j];
         const float2 w = *reinterpret_cast<const float2*>(p.norm_w + n);
         *reinterpret_cast<uint32_t*>(p.out + row * vw + h * p.dv + n) =
-            pack_bf16x2(acc[j][m][2 * r] * inv * w.x * silu_f32(bf16_lo(gate)), acc[j][m][2 * r + 1] * inv * w.y * silu_f32(bf16_hi(gate)));
+            pack_bf16x2(acc[j][m][2 * r] * inv * w.x * silu_fast(bf16_lo(gt)), acc[j][m][2 * r + 1] * inv * w.y * silu_fast(bf16_hi(gt)));
       }
     }
 }

@@ -218,14 +218,17 @@ def final_norm(model, x):
 def _attention(model, li, lw, s, act, batch, kv):
     qkv = ops.linear(act, lw.wqkv, bias=lw.bqkv)
     k_cache, v_cache = kv.layer(li)
-    q = ops.qkv_prepare(qkv, batch.positions, batch.slots, lw.extra["inv_freq"], k_cache, v_cache, s.heads, s.kv_heads, s.dim,
-                        s.vdim, lw.q_norm, lw.k_norm, model.cfg.rms_norm_eps, value_norm=True, append=s.kv_from is None)
+    eps, inv_freq, own = model.cfg.rms_norm_eps, lw.extra["inv_freq"], s.kv_from is None
     if batch.is_prefill:
+        q = ops.qkv_prepare(qkv, batch.positions, batch.slots, inv_freq, k_cache, v_cache, s.heads, s.kv_heads, s.dim, s.vdim,
+                            lw.q_norm, lw.k_norm, eps, value_norm=True, append=own)
         attn = ops.attention_prefill(q, k_cache, v_cache, batch.block_table, batch.seq_lens, batch.cu_q, batch.max_q_len,
                                      s.scale, chunk=s.chunk)
     else:
-        attn = ops.attention_decode(q, k_cache, v_cache, batch.block_table, batch.seq_lens, batch.q_per_seq, s.scale,
-                                    splits=batch.layer_splits(s.kv_heads, s.chunk), chunk=s.chunk)
+        attn = ops.attention_decode_rope(qkv, k_cache, v_cache, batch.block_table, batch.seq_lens, batch.q_per_seq, s.scale,
+                                         batch.positions, batch.slots, inv_freq, s.heads, s.kv_heads, s.dim, q_norm_w=lw.q_norm,
+                                         k_norm_w=lw.k_norm, norm_eps=eps, splits=batch.layer_splits(s.kv_heads, s.chunk),
+                                         chunk=s.chunk, value_dim=s.vdim, norm_whole=True, value_norm=True, append=own)
     return ops.linear(attn.view(attn.shape[0], -1), lw.wo, bias=lw.bo)
 
 

@@ -494,18 +494,33 @@ def attention_decode(q, k_cache, v_cache, block_table, seq_lens, q_per_seq, scal
 
 def attention_decode_rope(qkv, k_cache, v_cache, block_table, seq_lens, q_per_seq, scale, positions, slots, inv_freq,
                           n_q, n_kv, head_dim, rot=None, interleaved=False, attn_factor=1.0, q_norm_w=None, k_norm_w=None,
-                          norm_eps=1e-6, norm_w_off=0.0, splits=1, window=0, sinks=None, scratch=None):
+                          norm_eps=1e-6, norm_w_off=0.0, splits=1, window=0, sinks=None, scratch=None, chunk=0, value_dim=None,
+                          norm_whole=False, value_norm=False, append=True):
     """Decode attention straight from the qkv projection output [B * q_per_seq, >= (n_q + 2 n_kv) * D]: per-head
     q/k norm, RoPE and the KV append run inside the attention kernel (one launch instead of two). CPU tensors and
-    head sizes without a kernel compose the two reference operators."""
-    if not qkv.is_cuda or head_dim not in KERNEL_HEAD_DIMS or positions.dim() != 1 or q_per_seq > FUSED_ROPE_MAX_NEW:
+    head sizes without a kernel compose the two reference operators.
+    ``norm_whole`` / ``value_norm`` / ``append``: the preparation of :func:`qkv_prepare` (norms over whole projections, value
+    heads of width ``value_dim``, rows that hold queries only) instead of that of :func:`rope_kv`."""
+    value_dim = value_dim or head_dim
+    if norm_whole or value_norm or not append or value_dim != head_dim or chunk:
+        whole = (qkv.is_cuda and qkv.dtype == torch.bfloat16 and _tma_rows(qkv) and head_dim % 8 == 0 and value_dim % 8 == 0
+                 and max(head_dim, value_dim) <= 128 and n_q // n_kv <= 32 and q_per_seq <= FUSED_ROPE_MAX_NEW
+                 and splits <= CLUSTER_SPLITS and norm_whole and not interleaved)
+        if not whole:
+            assert norm_whole and not interleaved and norm_w_off == 0.0 and attn_factor == 1.0
+            q = qkv_prepare(qkv, positions, slots, inv_freq, k_cache, v_cache, n_q, n_kv, head_dim, value_dim, q_norm_w, k_norm_w,
+                            norm_eps, value_norm, append)
+            return attention_decode(q, k_cache, v_cache, block_table, seq_lens, q_per_seq, scale, splits, window, sinks, scratch,
+                                    chunk=chunk)
+        rot = 2 * inv_freq.shape[0]
+    elif not qkv.is_cuda or head_dim not in KERNEL_HEAD_DIMS or positions.dim() != 1 or q_per_seq > FUSED_ROPE_MAX_NEW:
         q = rope_kv(qkv, positions, slots, inv_freq, k_cache, v_cache, n_q, n_kv, head_dim, rot, interleaved, attn_factor,
                     q_norm_w, k_norm_w, norm_eps, norm_w_off)
         return attention_decode(q, k_cache, v_cache, block_table, seq_lens, q_per_seq, scale, splits, window, sinks, scratch)
     assert qkv.dtype == torch.bfloat16 and qkv.stride(1) == 1
     assert positions.dtype == torch.int32 and slots.dtype == torch.int64 and inv_freq.dtype == torch.float32
     B = seq_lens.shape[0]
-    out = torch.empty((qkv.shape[0], n_q, head_dim), dtype=qkv.dtype, device=qkv.device)
+    out = torch.empty((qkv.shape[0], n_q, value_dim), dtype=qkv.dtype, device=qkv.device)
     part_o = part_ml = counters = None
     if splits > CLUSTER_SPLITS:
         if scratch is None:
@@ -515,8 +530,10 @@ def attention_decode_rope(qkv, k_cache, v_cache, block_table, seq_lens, q_per_se
     code = lib().eredu_attn_decode_rope(ptr(qkv), qkv.stride(0), ptr(k_cache), ptr(v_cache), ptr(out), ptr(block_table),
                                         ptr(seq_lens), ptr(sinks), ptr(part_o), ptr(part_ml), ptr(counters), ptr(positions),
                                         ptr(slots), ptr(inv_freq), ptr(q_norm_w), ptr(k_norm_w), B, q_per_seq,
-                                        block_table.stride(0), n_q, n_kv, head_dim, rot or head_dim, 1 if interleaved else 0,
-                                        splits, window, scale, attn_factor, norm_eps, norm_w_off, stream_ptr(qkv.device))
+                                        block_table.stride(0), n_q, n_kv, head_dim, value_dim,
+                                        head_dim if rot is None else rot, 1 if interleaved else 0, splits, window, chunk,
+                                        int(norm_whole), int(value_norm), int(append), scale, attn_factor, norm_eps,
+                                        norm_w_off, stream_ptr(qkv.device))
     check(code, "eredu_attn_decode_rope")
     return out
 

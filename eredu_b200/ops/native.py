@@ -26,7 +26,7 @@ _SIGNATURES = {
     "eredu_peer_recv": (I, [P, I, I, P, L, P, I, P, P]),
     "eredu_attn_prefill_tc": (I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, P, P]),
     "eredu_attn_decode_scratch_elems": (None, [I, I, I, I, I, POINTER(L), POINTER(L)]),
-    "eredu_attn_decode_rope": (I, [P, I, P, P, P, P, P, P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, F, F, F, F, P]),
+    "eredu_attn_decode_rope": (I, [P, I] + [P] * 14 + [I] * 15 + [F, F, F, F, P]),
     "eredu_rmsnorm": (I, [P, P, P, P, P, I, I, F, F, P]),
     "eredu_rope_kv": (I, [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, F, F, P]),
     "eredu_embedding": (I, [P, P, P, I, I, I, I, F, P, P]),

@@ -18,7 +18,8 @@ from .native import F, I, P, check, lib, ptr, stream_ptr
 
 native.register("eredu_gated_delta_scan", I, [P, P, P, P, P, P, P, I, I, I, I, I, I, P])
 native.register("eredu_mamba2_scan", I, [P, P, P, P, P, P, P, P, I, I, I, I, I, I, P])
-native.register("eredu_mingru_scan", I, [P] * 7 + [I] * 7 + [P])
+native.register("eredu_mingru_scan", I, [P] * 8 + [I] * 7 + [P])
+native.register("eredu_mingru_scratch_elems", native.L, [I] * 4)
 native.register("eredu_gla_scan", I, [P] * 7 + [I] + [P] * 4 + [I] * 10 + [F, F, P])
 native.register("eredu_gla_scratch_elems", native.L, [I] * 8)
 
@@ -277,11 +278,14 @@ def mingru_scan(proj, state, width, batch, page_to_slot):
     out = torch.empty((proj.shape[0], width), dtype=proj.dtype, device=proj.device)
     if proj.shape[0] == 0:
         return out
-    code = lib().eredu_mingru_scan(ptr(proj), ptr(state), ptr(out), ptr(batch.block_table), ptr(page_to_slot),
+    batch_size = batch.block_table.shape[0]
+    rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
+    elems = int(lib().eredu_mingru_scratch_elems(width, proj.shape[0], batch_size, rows))
+    scratch = torch.empty(elems, dtype=torch.float32, device=proj.device) if elems else None
+    code = lib().eredu_mingru_scan(ptr(proj), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table), ptr(page_to_slot),
                                    ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), width, proj.stride(0),
-                                   batch.block_table.shape[0], batch.q_per_seq, batch.max_q_len if batch.is_prefill else
-                                   batch.q_per_seq, batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0,
-                                   stream_ptr(proj.device))
+                                   batch_size, batch.q_per_seq, rows, batch.block_table.stride(0),
+                                   1 if proj.dtype == torch.float32 else 0, stream_ptr(proj.device))
     check(code, "eredu_mingru_scan")
     return out
 

@@ -202,6 +202,35 @@ def test_chunked_attention_sees_its_chunk_and_nothing_else(dev, dt, H, G, dk, dv
         assert float((got.double().cpu() - want[at]).abs().max()) <= limit * float(want.abs().max()), splits
 
 
+@both
+@pytest.mark.parametrize("nq,nkv,dk,dv,rot,chunk", [(6, 2, 40, 24, 8, 20), (2, 2, 128, 64, 128, 0), (8, 1, 64, 128, 32, 64), (4, 2, 128, 128, 0, 33)])
+@pytest.mark.parametrize("new,append", [(1, True), (3, True), (1, False)])
+def test_decode_step_from_the_projection(dev, dt, nq, nkv, dk, dv, rot, chunk, new, append):
+    """Preparation, append and attention in one operator: sequences at page and chunk edges, an idle row."""
+    lens = [1 + new, 16, 17, 33, 64, 65, 66, 130, 40]
+    B, P, eps = len(lens), 9, 1e-4
+    lens_t = torch.tensor(lens)
+    bt = (torch.arange(B * P).view(B, P) * 5 % (B * P)) + 1
+    pos = torch.cat([torch.arange(n - new, n) for n in lens])
+    slots = torch.cat([bt[b][torch.arange(n - new, n) // 16] * 16 + torch.arange(n - new, n) % 16 for b, n in enumerate(lens)])
+    slots[-new:] = -1                                                  # idle: its result is not looked at, its pages stay
+    x = rand(B * new, nq * dk + (nkv * (dk + dv) if append else 0), seed=1)
+    qw, kw = rand(nq * dk, seed=2) * 0.3 + 1, rand(nkv * dk, seed=3) * 0.3 + 1
+    inv = torch.tensor([100.0 ** (-2.0 * i / max(rot, 1)) for i in range(rot // 2)], dtype=torch.float32)
+    k0, v0 = rand(B * P + 1, nkv, 16, dk, seed=4), rand(B * P + 1, nkv, 16, dv, seed=5)
+    kr, vr = k0.float(), v0.float()
+    q = ops.qkv_prepare_ref(x.float(), pos, slots, inv, kr, vr, nq, nkv, dk, dv, qw.float(), kw.float(), eps, True, append)
+    want = ops.attention_ref(q, kr, vr, bt, lens_t, [new] * B, 0.2, chunk=chunk)
+    for splits in (1, 4, 8):
+        kc, vc = k0.to(dev, dt), v0.to(dev, dt)
+        got = ops.attention_decode_rope(x.to(dev, dt), kc, vc, bt.int().to(dev), lens_t.int().to(dev), new, 0.2, pos.int().to(dev), slots.to(dev),
+                                        inv.to(dev), nq, nkv, dk, q_norm_w=qw.float().to(dev), k_norm_w=kw.float().to(dev), norm_eps=eps, splits=splits,
+                                        chunk=chunk, value_dim=dv, norm_whole=True, value_norm=True, append=append)
+        close(got[:-new], want[:-new], dt, scale=float(want.abs().max()) * (3 if dt == torch.bfloat16 else 1))
+        close(kc, kr, dt)
+        close(vc, vr, dt)
+
+
 def ragged(rows, starts, pages, dev):
     """ForwardBatch of portions: sequence i brings rows[i] tokens from position starts[i]; its first page is pages[i]."""
     cu = torch.tensor([0] + rows).cumsum(0)
