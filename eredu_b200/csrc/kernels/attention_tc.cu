@@ -92,6 +92,18 @@ __device__ __forceinline__ int tc_lowest_key(const AttnTcParams& p, int pos) {
   return p.chunk > 0 ? pos - pos % p.chunk : 0;
 }
 
+// Order in which query tiles are taken, longest first: the last positions of a causal prompt, the last tiles of every chunk.
+__device__ __forceinline__ int tc_query_tile(const AttnTcParams& p, int tiles, int y) {
+  const int per = p.chunk / kTcRows;                                    // query tiles of a chunk
+  if (per < 2) return tiles - 1 - y;
+  for (int r = min(per, tiles) - 1; r > 0; --r) {
+    const int n = (tiles - r + per - 1) / per;
+    if (y < n) return r + y * per;
+    y -= n;
+  }
+  return y * per;
+}
+
 // NK / NV: 64-wide halves of the key and of the value width
 template <int NK, int NV>
 __global__ void __launch_bounds__(kTcThreads, 1)
@@ -120,7 +132,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // heads vary fastest: the first wave holds the longest query tiles of every head (longest-first balances the causal
   // triangle), and neighbouring CTAs are query heads of one key / value head reading the same pages
-  const int b = blockIdx.z, head = blockIdx.x, qt = gridDim.y - 1 - blockIdx.y;
+  const int b = blockIdx.z, head = blockIdx.x, qt = tc_query_tile(p, gridDim.y, blockIdx.y);
   const int q0 = p.cu_q[b], q_len = p.cu_q[b + 1] - q0;
   const int kv_len = p.seq_lens[b];
   const int row0 = qt * kTcRows;

@@ -91,40 +91,47 @@ __device__ __forceinline__ void load_chunk(const GlaParams<bf16>& p, const Chunk
   const int qk = p.H * p.dk, vw = p.H * p.dv;
   const int n = min(kChunk, seq.rows - t0);
   const bf16* rows = p.proj + static_cast<size_t>(seq.row0 + t0) * p.ld;
-  const uint4 zero = make_uint4(0, 0, 0, 0);
   const int kc = s.dkp / 8, kreal = p.dk / 8, vc = p.dv / 8;
-  for (int i = threadIdx.x; i < kChunk * kc; i += kThreads) {
-    const int t = i / kc, c = i % kc;
-    const bool ok = t < n && c < kreal;
-    const bf16* src = rows + static_cast<size_t>(t) * p.ld + h * p.dk + c * 8;
-    if (WITH_Q) *reinterpret_cast<uint4*>(s.q + t * s.ks + c * 8) = ok ? *reinterpret_cast<const uint4*>(src) : zero;
-    *reinterpret_cast<uint4*>(s.k + t * s.ks + c * 8) = ok ? *reinterpret_cast<const uint4*>(src + qk) : zero;
-  }
-  for (int i = threadIdx.x; i < kChunk * vc; i += kThreads) {
-    const int t = i / vc, c = i % vc;
-    *reinterpret_cast<uint4*>(s.v + t * s.vs + c * 8) =
-        t < n ? *reinterpret_cast<const uint4*>(rows + static_cast<size_t>(t) * p.ld + 2 * qk + h * p.dv + c * 8) : zero;
-  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rp = s.rs - 8;                                        // rank, padded to whole steps of the products
-  for (int i = threadIdx.x; i < kChunk * rp; i += kThreads) {
-    const int t = i / rp, j = i % rp;
-    s.low[t * s.rs + j] = t < n && j < p.rank ? rows[static_cast<size_t>(t) * p.ld + 2 * qk + 2 * vw + j] : __float2bfloat16(0.f);
+  // a warp takes every eighth row; half-warps take two rows at a time where a row has at most 16 pieces. Everything is in
+  // flight at once.
+  const int kper = kc <= 16 ? 2 : 1, kl = kc <= 16 ? lane & 15 : lane;
+  for (int t = warp * kper + (kc <= 16 ? lane >> 4 : 0); t < kChunk; t += 8 * kper)
+    for (int c = kl; c < kc; c += 32) {
+      const int bytes = t < n && c < kreal ? 16 : 0;
+      const bf16* src = bytes ? rows + static_cast<size_t>(t) * p.ld + h * p.dk + c * 8 : rows;
+      if (WITH_Q) cp_async16(s.q + t * s.ks + c * 8, src, bytes);
+      cp_async16(s.k + t * s.ks + c * 8, bytes ? src + qk : rows, bytes);
+    }
+  const int vper = vc <= 16 ? 2 : 1, vl = vc <= 16 ? lane & 15 : lane;
+  for (int t = warp * vper + (vc <= 16 ? lane >> 4 : 0); t < kChunk; t += 8 * vper)
+    for (int c = vl; c < vc; c += 32)
+      cp_async16(s.v + t * s.vs + c * 8, t < n ? rows + static_cast<size_t>(t) * p.ld + 2 * qk + h * p.dv + c * 8 : rows, t < n ? 16 : 0);
+  const int pieces = rp / 8;
+  for (int i = threadIdx.x; i < kChunk * pieces; i += kThreads) {
+    const int t = i / pieces, c = i % pieces;
+    const int bytes = t < n && c * 8 < p.rank ? 16 : 0;
+    cp_async16(s.low + t * s.rs + c * 8, bytes ? rows + static_cast<size_t>(t) * p.ld + 2 * qk + 2 * vw + c * 8 : rows, bytes);
   }
-  for (int i = threadIdx.x; i < s.dkp * rp; i += kThreads) {
-    const int c = i / rp, j = i % rp;
-    const float w = c < p.dk && j < p.rank ? p.a2[(static_cast<size_t>(h) * p.dk + c) * p.rank + j] : 0.f;
-    const bf16 hi = __float2bfloat16(w);
-    s.a2h[c * s.rs + j] = hi;
-    s.a2l[c * s.rs + j] = __float2bfloat16(w - to_f32(hi));
+  cp_async_commit();
+  const int quads = rp / 4;
+  for (int i = threadIdx.x; i < s.dkp * quads; i += kThreads) {
+    const int c = i / quads, j = (i % quads) * 4;
+    const float4 w = c < p.dk && j < p.rank ? load4(p.a2 + (static_cast<size_t>(h) * p.dk + c) * p.rank + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    uint2 hi, lo;
+    split2(w.x, w.y, hi.x, lo.x);
+    split2(w.z, w.w, hi.y, lo.y);
+    *reinterpret_cast<uint2*>(s.a2h + c * s.rs + j) = hi;
+    *reinterpret_cast<uint2*>(s.a2l + c * s.rs + j) = lo;
   }
+  cp_async_wait<0>();
   __syncthreads();
   // z = low a2^T + bias on the tensor cores, one tile = one block of 16 tokens x 8 channels; the decays are summed along the
   // tokens of the tile with shuffles (lane group g holds the rows g and g + 8)
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
-  const int tiles = s.dkp / 8;
-  for (int i = warp; i < kBlks * tiles; i += 8) {
-    const int blk = i / tiles, c0 = (i % tiles) * 8;
+  for (int i = warp; i < kBlks * (s.dkp / 8); i += 8) {
+    const int blk = i & (kBlks - 1), c0 = (i / kBlks) * 8;
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     for (int ks = 0; ks < rp; ks += 16) {
       const bf16* lo = s.low + (blk * kBlk + g) * s.rs + ks + tig * 2;
@@ -181,20 +188,23 @@ __global__ void __launch_bounds__(kThreads, NT <= 2 ? 2 : 1) gla_chunk_state_ker
   load_chunk<false>(p, s, seq, h, blockIdx.x * kChunk);
   const size_t cell = static_cast<size_t>(chunk_id(seq, b, blockIdx.x)) * p.H + h;
   // k e^{b_end - b_s}: hi over the keys, lo in the place of the queries
-  for (int i = threadIdx.x; i < kChunk * (s.dkp / 2); i += kThreads) {
-    const int t = i / (s.dkp / 2), c = (i % (s.dkp / 2)) * 2;
-    const uint32_t kk = *reinterpret_cast<const uint32_t*>(s.k + t * s.ks + c);
-    const float* r0 = s.R + (t / kBlk) * s.dkp + c;
-    const float* r1 = s.R + kBlks * s.dkp + c;
-    const float2 bl = *reinterpret_cast<const float2*>(s.bl + t * s.ks + c);
-    uint32_t hi, lo;
-    split2(bf16_lo(kk) * ex2_approx(r1[0] - r0[0] - bl.x), bf16_hi(kk) * ex2_approx(r1[1] - r0[1] - bl.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(s.k + t * s.ks + c) = hi;
-    *reinterpret_cast<uint32_t*>(s.q + t * s.ks + c) = lo;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int c = lane * 2; c < s.dkp; c += 64) {
+    const float2 end = *reinterpret_cast<const float2*>(s.R + kBlks * s.dkp + c);
+#pragma unroll
+    for (int i = 0; i < kChunk / 8; ++i) {                         // this warp's rows: two of every block
+      const int t = warp + 8 * i;
+      const uint32_t kk = *reinterpret_cast<const uint32_t*>(s.k + t * s.ks + c);
+      const float2 r0 = *reinterpret_cast<const float2*>(s.R + (i >> 1) * s.dkp + c);
+      const float2 bl = *reinterpret_cast<const float2*>(s.bl + t * s.ks + c);
+      uint32_t hi, lo;
+      split2(bf16_lo(kk) * ex2_approx(end.x - r0.x - bl.x), bf16_hi(kk) * ex2_approx(end.y - r0.y - bl.y), hi, lo);
+      *reinterpret_cast<uint32_t*>(s.k + t * s.ks + c) = hi;
+      *reinterpret_cast<uint32_t*>(s.q + t * s.ks + c) = lo;
+    }
   }
   for (int c = threadIdx.x; c < p.dk; c += kThreads) decay[cell * p.dk + c] = ex2_approx(s.R[kBlks * s.dkp + c]);
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, tig = lane & 3;
   const int nt = p.dv / 8;
   uint32_t vf[NT][8];
@@ -366,15 +376,18 @@ __global__ void __launch_bounds__(kThreads, NT <= 2 ? 2 : 1) gla_chunk_out_kerne
   }
   __syncthreads();
   // q e^{b_t} / sqrt(dk): hi in the place of the keys, lo over the queries
-  for (int i = threadIdx.x; i < kChunk * (s.dkp / 2); i += kThreads) {
-    const int t = i / (s.dkp / 2), c = (i % (s.dkp / 2)) * 2;
-    const uint32_t q = *reinterpret_cast<const uint32_t*>(s.q + t * s.ks + c);
-    const float2 bl = *reinterpret_cast<const float2*>(s.bl + t * s.ks + c);
-    const float* r = s.R + (t / kBlk) * s.dkp + c;
-    uint32_t hi, lo;
-    split2(bf16_lo(q) * q_scale * ex2_approx(r[0] + bl.x), bf16_hi(q) * q_scale * ex2_approx(r[1] + bl.y), hi, lo);
-    *reinterpret_cast<uint32_t*>(s.k + t * s.ks + c) = hi;
-    *reinterpret_cast<uint32_t*>(s.q + t * s.ks + c) = lo;
+  for (int c = lane * 2; c < s.dkp; c += 64) {
+#pragma unroll
+    for (int i = 0; i < kChunk / 8; ++i) {
+      const int t = warp + 8 * i;
+      const uint32_t q = *reinterpret_cast<const uint32_t*>(s.q + t * s.ks + c);
+      const float2 bl = *reinterpret_cast<const float2*>(s.bl + t * s.ks + c);
+      const float2 r = *reinterpret_cast<const float2*>(s.R + (i >> 1) * s.dkp + c);
+      uint32_t hi, lo;
+      split2(bf16_lo(q) * q_scale * ex2_approx(r.x + bl.x), bf16_hi(q) * q_scale * ex2_approx(r.y + bl.y), hi, lo);
+      *reinterpret_cast<uint32_t*>(s.k + t * s.ks + c) = hi;
+      *reinterpret_cast<uint32_t*>(s.q + t * s.ks + c) = lo;
+    }
   }
   __syncthreads();
   const int nt = p.dv / 8;
@@ -486,7 +499,7 @@ __global__ void __launch_bounds__(kThreads, NT <= 2 ? 2 : 1) gla_chunk_out_kerne
 }
 
 bool gla_chunk_supported(const GlaParams<bf16>& p) {
-  return p.dk % 8 == 0 && p.dk <= kMaxDk && p.dv % 8 == 0 && p.dv <= kMaxDv && p.rank <= kMaxRank && p.ld % 8 == 0 &&
+  return p.dk % 8 == 0 && p.dk <= kMaxDk && p.dv % 8 == 0 && p.dv <= kMaxDv && p.rank <= kMaxRank && p.rank % 8 == 0 && p.ld % 8 == 0 &&
          (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0;
 }
 
