@@ -70,10 +70,11 @@ __device__ __forceinline__ float ld_dsmem_f32(uint32_t cluster_addr) {
 // rotation of the first `rot` dims by the token's position. Executed by one warp; lane l owns the pairs l, l + 32, ...
 // `store(i0, a, i1, b)` receives the finished element pairs.
 // `whole_inv` > 0: the projection's own 1 / rms, instead of the head's. Heads may be narrower than D (p.dk).
-template <int D, typename Store>
+template <int D, bool EXT, typename Store>
 __device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bfloat16* src, const float* nw, float whole_inv,
                                               int pos, int lane, Store store) {
   constexpr int PER = D / 64;  // pairs per lane
+  const int dk = EXT ? p.dk : D;
   const int rh = p.rot >> 1;
   float a[PER], b[PER];
   int i0[PER], i1[PER];
@@ -88,25 +89,25 @@ __device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bf
       i0[j] = p.rot + 2 * (i - rh);
       i1[j] = i0[j] + 1;
     }
-    const bool in = 2 * i < p.dk;
+    const bool in = 2 * i < dk;
     a[j] = in ? __bfloat162float(src[i0[j]]) : 0.f;
     b[j] = in ? __bfloat162float(src[i1[j]]) : 0.f;
     ss += a[j] * a[j] + b[j] * b[j];
   }
-  if (nw != nullptr && p.norm_whole) {
+  if (nw != nullptr && (EXT && p.norm_whole)) {
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
-      if (2 * (lane + 32 * j) >= p.dk) continue;
+      if (2 * (lane + 32 * j) >= dk) continue;
       a[j] *= whole_inv * nw[i0[j]];
       b[j] *= whole_inv * nw[i1[j]];
     }
   } else if (nw != nullptr) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const float inv = rsqrtf(ss / static_cast<float>(p.dk) + p.norm_eps);
+    const float inv = rsqrtf(ss / static_cast<float>(dk) + p.norm_eps);
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
-      if (2 * (lane + 32 * j) >= p.dk) continue;
+      if (2 * (lane + 32 * j) >= dk) continue;
       a[j] = __bfloat162float(__float2bfloat16(a[j] * inv * (nw[i0[j]] + p.norm_w_off)));
       b[j] = __bfloat162float(__float2bfloat16(b[j] * inv * (nw[i1[j]] + p.norm_w_off)));
     }
@@ -124,7 +125,7 @@ __device__ __forceinline__ void rope_head_row(const AttnParams& p, const __nv_bf
       a[j] = ra;
       b[j] = rb;
     }
-    if (2 * i < p.dk) store(i0[j], a[j], i1[j], b[j]);
+    if (2 * i < dk) store(i0[j], a[j], i1[j], b[j]);
   }
 }
 
@@ -143,9 +144,10 @@ __device__ __forceinline__ uint32_t swz(int r, int c) {
 }
 
 // First key position a query at `pos` can see.
+template <bool CHUNKS>
 __device__ __forceinline__ int lowest_key(const AttnParams& p, int pos) {
   if (p.window > 0) return pos - p.window + 1;
-  return p.chunk > 0 ? pos - pos % p.chunk : 0;
+  return CHUNKS && p.chunk > 0 ? pos - pos % p.chunk : 0;
 }
 
 // ============================================================================ prefill
@@ -345,10 +347,13 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(AttnParams p) {
 // grid (splits, n_kv_heads, B). The MT*16 MMA rows hold (query token t, head-in-group g) pairs,
 // row = (t - t0) * group + g. Each of the 4 warps streams every 4th page through its own 3-stage
 // cp.async ring and keeps private (m, l, O); the warps are merged through shared memory at the end.
-// Keys and values may differ in width: tiles are DK / DV wide (64 or 128), rows of the cache p.dk / p.dv (the rest of a
-// tile row is zero-filled, which adds nothing to scores or outputs).
-template <int DK, int DV, int MT>
-__global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
+// Keys and values may differ in width: tiles are DK / DV wide (64 or 128), rows of the cache dk / dv (the rest of a
+// tile row is zero-filled, which adds nothing to scores or outputs). EXT = false is the common case with everything beyond
+// it folded away: one head size that fills the tile, no chunks, the preparation of rope_kv.
+template <int DK, int DV, int MT, bool EXT>
+__global__ void __launch_bounds__(128, MT == 1 ? (DK + DV <= 128 ? 5 : 4) : 1) attn_decode_kernel(AttnParams p) {
+  const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
+  const bool norm_whole = EXT && p.norm_whole, value_norm = EXT && p.value_norm;
   constexpr int CHK = DK / 8, CHV = DV / 8;
   constexpr int KS = DK / 16;
   constexpr int NSTAGE = 3;
@@ -377,7 +382,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   const int npages = (kv_len + kPage - 1) / kPage;
   // pages before the first query's window / chunk hold nothing any query of this launch can see
   const int first_pos = kv_len - p.q_per_seq + p.t0;
-  const int first_page = max(0, lowest_key(p, first_pos)) / kPage;
+  const int first_page = max(0, lowest_key<EXT>(p, first_pos)) / kPage;
   int pps = (npages - first_page + p.splits - 1) / p.splits;
   pps = (pps + 3) & ~3;
   const int page0 = first_page + split * pps;
@@ -387,16 +392,16 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   // The launch that handles the first query tokens also appends the new K / V rows. A page fetched from the cache may
   // then still hold the old bytes of a new row, so the rows are patched into the shared-memory copy of their page
   // (from `newkv_s`) after it has landed: no fence and no ordering between the append and the page fetches is needed.
-  const bool appending = fused && p.append && p.t0 == 0;
+  const bool appending = fused && (!EXT || p.append) && p.t0 == 0;
   const int new_pos0 = kv_len - p.q_per_seq;
   const int first_new_page = appending ? new_pos0 / kPage : 0x7fffffff;
   if (!fused) {
     for (int i = threadIdx.x; i < ROWS * CHK; i += 128) {
       const int r = i / CHK, c = i % CHK;
-      const bool ok = r < rows && c * 8 < p.dk;
+      const bool ok = r < rows && c * 8 < dk;
       const int t = p.t0 + (r < rows ? r / group : 0), hg = r < rows ? r % group : 0;
       const __nv_bfloat16* src =
-          p.q + (static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + kvh * group + hg) * p.dk + (ok ? c * 8 : 0);
+          p.q + (static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + kvh * group + hg) * dk + (ok ? c * 8 : 0);
       cp_async16(q_s + swz<DK>(r, c), src, ok ? 16 : 0);
     }
   }
@@ -406,19 +411,19 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   auto load_page = [&](int pg, int stage) {
     if (pg < page1) {
       const int phys = bt[pg];
-      const __nv_bfloat16* ksrc = p.k_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * p.dk;
-      const __nv_bfloat16* vsrc = p.v_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * p.dv;
+      const __nv_bfloat16* ksrc = p.k_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * dk;
+      const __nv_bfloat16* vsrc = p.v_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * dv;
       uint8_t* kd = my_ring + stage * STAGE_BYTES;
       uint8_t* vd = kd + KPAGE_BYTES;
       for (int i = lane; i < kPage * CHK; i += 32) {
         const int r = i / CHK, c = i % CHK;
-        const bool in = c * 8 < p.dk;
-        cp_async16(kd + swz<DK>(r, c), ksrc + r * p.dk + (in ? c * 8 : 0), in ? 16 : 0);
+        const bool in = c * 8 < dk;
+        cp_async16(kd + swz<DK>(r, c), ksrc + r * dk + (in ? c * 8 : 0), in ? 16 : 0);
       }
       for (int i = lane; i < kPage * CHV; i += 32) {
         const int r = i / CHV, c = i % CHV;
-        const bool in = c * 8 < p.dv;
-        cp_async16(vd + swz<DV>(r, c), vsrc + r * p.dv + (in ? c * 8 : 0), in ? 16 : 0);
+        const bool in = c * 8 < dv;
+        cp_async16(vd + swz<DV>(r, c), vsrc + r * dv + (in ? c * 8 : 0), in ? 16 : 0);
       }
     }
   };
@@ -439,11 +444,11 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   load_page(first + 4, 1);
   cp_async_commit();
   if (fused) {
-    if (p.norm_whole) {
+    if (norm_whole) {
       // ---- 1 / rms of the whole q (and k) projection of every new token: each CTA sums the row for itself
       for (int t = 0; t < p.q_per_seq; ++t) {
         const uint4* row = reinterpret_cast<const uint4*>(p.qkv + (static_cast<size_t>(b) * p.q_per_seq + t) * p.ld_qkv);
-        const int nq = p.n_q_heads * p.dk / 8, nk = appending ? p.n_kv_heads * p.dk / 8 : 0;
+        const int nq = p.n_q_heads * dk / 8, nk = appending ? p.n_kv_heads * dk / 8 : 0;
         float sq = 0.f, sk = 0.f;
         for (int i = threadIdx.x; i < nq; i += 128) sq += sum_squares8(row[i]);
         for (int i = threadIdx.x; i < nk; i += 128) sk += sum_squares8(row[nq + i]);
@@ -459,7 +464,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         __syncthreads();
         if (threadIdx.x < 2) {
           const float* r = s_part[threadIdx.x];
-          const float n = static_cast<float>((threadIdx.x == 0 ? p.n_q_heads : p.n_kv_heads) * p.dk);
+          const float n = static_cast<float>((threadIdx.x == 0 ? p.n_q_heads : p.n_kv_heads) * dk);
           s_inv[threadIdx.x][t] = rsqrtf((r[0] + r[1] + r[2] + r[3]) / n + p.norm_eps);
         }
         __syncthreads();
@@ -475,10 +480,10 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         const int t = p.t0 + r / group, hg = r % group;
         const size_t m = static_cast<size_t>(b) * p.q_per_seq + t;
         const int head = kvh * group + hg;
-        const float* nw = p.q_norm_w == nullptr ? nullptr : p.q_norm_w + (p.norm_whole ? head * p.dk : 0);
-        rope_head_row<DK>(p, p.qkv + m * p.ld_qkv + static_cast<size_t>(head) * p.dk, nw, p.norm_whole ? s_inv[0][t] : 0.f,
+        const float* nw = p.q_norm_w == nullptr ? nullptr : p.q_norm_w + (norm_whole ? head * dk : 0);
+        rope_head_row<DK, EXT>(p, p.qkv + m * p.ld_qkv + static_cast<size_t>(head) * dk, nw, norm_whole ? s_inv[0][t] : 0.f,
                           p.positions[m], lane, put);
-        for (int i = p.dk / 2 + lane; i < DK / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
+        for (int i = dk / 2 + lane; i < DK / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
       } else {
         for (int i = lane; i < DK / 2; i += 32) put(2 * i, 0.f, 2 * i + 1, 0.f);
       }
@@ -492,36 +497,36 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         const long long slot = p.slots[m];
         if (pg < page0 || pg >= page1 || slot < 0) continue;  // warp-uniform
         const size_t cell = (static_cast<size_t>(slot >> 4) * p.n_kv_heads + kvh) * kPage + static_cast<size_t>(slot & 15);
-        __nv_bfloat16* kd = const_cast<__nv_bfloat16*>(p.k_cache) + cell * p.dk;
-        __nv_bfloat16* vd = const_cast<__nv_bfloat16*>(p.v_cache) + cell * p.dv;
+        __nv_bfloat16* kd = const_cast<__nv_bfloat16*>(p.k_cache) + cell * dk;
+        __nv_bfloat16* vd = const_cast<__nv_bfloat16*>(p.v_cache) + cell * dv;
         __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(newkv_s) + static_cast<size_t>(t) * (DK + DV);
-        const __nv_bfloat16* krow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + kvh) * p.dk;
-        const __nv_bfloat16* vrow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + p.n_kv_heads) * p.dk +
-                                    static_cast<size_t>(kvh) * p.dv;
-        const float* nw = p.k_norm_w == nullptr ? nullptr : p.k_norm_w + (p.norm_whole ? kvh * p.dk : 0);
-        rope_head_row<DK>(p, krow, nw, p.norm_whole ? s_inv[1][t] : 0.f, p.positions[m], lane, [&](int i0, float a, int i1, float bb) {
+        const __nv_bfloat16* krow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + kvh) * dk;
+        const __nv_bfloat16* vrow = p.qkv + m * p.ld_qkv + static_cast<size_t>(p.n_q_heads + p.n_kv_heads) * dk +
+                                    static_cast<size_t>(kvh) * dv;
+        const float* nw = p.k_norm_w == nullptr ? nullptr : p.k_norm_w + (norm_whole ? kvh * dk : 0);
+        rope_head_row<DK, EXT>(p, krow, nw, norm_whole ? s_inv[1][t] : 0.f, p.positions[m], lane, [&](int i0, float a, int i1, float bb) {
           const __nv_bfloat16 ha = __float2bfloat16(a), hb = __float2bfloat16(bb);
           kd[i0] = ha;
           kd[i1] = hb;
           ks[i0] = ha;
           ks[i1] = hb;
         });
-        for (int i = p.dk / 2 + lane; i < DK / 2; i += 32) reinterpret_cast<uint32_t*>(ks)[i] = 0u;
+        for (int i = dk / 2 + lane; i < DK / 2; i += 32) reinterpret_cast<uint32_t*>(ks)[i] = 0u;
         float v_inv = 1.f;
-        if (p.value_norm) {
+        if (value_norm) {
           float ss = 0.f;
-          for (int i = lane; i < p.dv / 2; i += 32) {
+          for (int i = lane; i < dv / 2; i += 32) {
             const uint32_t vv = reinterpret_cast<const uint32_t*>(vrow)[i];
             ss += bf16_lo(vv) * bf16_lo(vv) + bf16_hi(vv) * bf16_hi(vv);
           }
 #pragma unroll
           for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-          v_inv = rsqrtf(ss / static_cast<float>(p.dv) + p.norm_eps);
+          v_inv = rsqrtf(ss / static_cast<float>(dv) + p.norm_eps);
         }
         for (int i = lane; i < DV / 2; i += 32) {
-          uint32_t vv = 2 * i < p.dv ? reinterpret_cast<const uint32_t*>(vrow)[i] : 0u;
-          if (p.value_norm) vv = pack_bf16x2(bf16_lo(vv) * v_inv, bf16_hi(vv) * v_inv);
-          if (2 * i < p.dv) reinterpret_cast<uint32_t*>(vd)[i] = vv;
+          uint32_t vv = 2 * i < dv ? reinterpret_cast<const uint32_t*>(vrow)[i] : 0u;
+          if (value_norm) vv = pack_bf16x2(bf16_lo(vv) * v_inv, bf16_hi(vv) * v_inv);
+          if (2 * i < dv) reinterpret_cast<uint32_t*>(vd)[i] = vv;
           reinterpret_cast<uint32_t*>(ks + DK)[i] = vv;
         }
       }
@@ -584,7 +589,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
           const int r = mt * 16 + g + (e >> 1) * 8;
           const int qp = kv_len - p.q_per_seq + p.t0 + r / group;
           bool ok = (r < rows) && (j <= qp) && (j < kv_len);
-          ok = ok && (j >= lowest_key(p, qp));
+          ok = ok && (j >= lowest_key<EXT>(p, qp));
           const float v = ok ? s[mt][nt][e] * p.scale_log2 : -INFINITY;
           s[mt][nt][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -664,7 +669,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
   __syncthreads();
   for (int i = threadIdx.x; i < rows * DV; i += 128) {
     const int row = i / DV, d = i % DV;
-    if (d >= p.dv) continue;
+    if (d >= dv) continue;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) M = fmaxf(M, mm[w * ROWS + row]);
@@ -682,7 +687,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     if (p.splits == 1) {
       float Lf = L;
       if (p.sinks != nullptr) Lf += exp2f(p.sinks[head] * 1.4426950408889634f - Ms);
-      p.out[qrow * p.dv + d] = __float2bfloat16(Lf > 0.f ? acc / Lf : 0.f);
+      p.out[qrow * dv + d] = __float2bfloat16(Lf > 0.f ? acc / Lf : 0.f);
     } else if (p.cluster_reduce) {
       part_s[row * DV + d] = acc;
       if (d == 0) {
@@ -690,7 +695,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
         part_l[row] = L;
       }
     } else {
-      p.part_o[(qrow * p.splits + split) * p.dv + d] = acc;
+      p.part_o[(qrow * p.splits + split) * dv + d] = acc;
       if (d == 0) {
         p.part_ml[(qrow * p.splits + split) * 2 + 0] = M;
         p.part_ml[(qrow * p.splits + split) * 2 + 1] = L;
@@ -705,7 +710,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
     const uint32_t a_s = smem_u32(part_s), a_m = smem_u32(part_m), a_l = smem_u32(part_l);
     for (int i = threadIdx.x + split * 128; i < rows * DV; i += 128 * p.splits) {  // row-major: a warp stays in one row
       const int row = i / DV, d = i % DV;
-      if (d >= p.dv) continue;
+      if (d >= dv) continue;
       float M = -INFINITY;
       float ms[kMaxClusterSplits], pv[kMaxClusterSplits], ls[kMaxClusterSplits];
 #pragma unroll
@@ -730,7 +735,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
       const int t = p.t0 + row / group, hg = row % group;
       const int head = kvh * group + hg;
       if (p.sinks != nullptr) L += exp2f(p.sinks[head] * 1.4426950408889634f - Ms);
-      p.out[(static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + head) * p.dv + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
+      p.out[(static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + head) * dv + d] = __float2bfloat16(L > 0.f ? acc / L : 0.f);
     }
     cluster_arrive_release();  // done reading the peers' shared memory
     cluster_wait_acquire();    // and nobody reads this CTA's any more
@@ -771,20 +776,20 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(AttnParams p) {
       __syncthreads();
       for (int i = threadIdx.x; i < rows * DV; i += 128) {
         const int row = i / DV, d = i % DV;
-        if (d >= p.dv) continue;
+        if (d >= dv) continue;
         const int t = p.t0 + row / group, hg = row % group;
         const size_t qrow = static_cast<size_t>(b * p.q_per_seq + t) * p.n_q_heads + kvh * group + hg;
-        const float* po = p.part_o + qrow * p.splits * p.dv + d;
+        const float* po = p.part_o + qrow * p.splits * dv + d;
         float acc = 0.f;
         int sp = 0;
         for (; sp + 4 <= p.splits; sp += 4) {
-          const float a0 = __ldcg(po + (sp + 0) * p.dv), a1 = __ldcg(po + (sp + 1) * p.dv);
-          const float a2 = __ldcg(po + (sp + 2) * p.dv), a3 = __ldcg(po + (sp + 3) * p.dv);
+          const float a0 = __ldcg(po + (sp + 0) * dv), a1 = __ldcg(po + (sp + 1) * dv);
+          const float a2 = __ldcg(po + (sp + 2) * dv), a3 = __ldcg(po + (sp + 3) * dv);
           acc += a0 * wgt[row * 64 + sp] + a1 * wgt[row * 64 + sp + 1] + a2 * wgt[row * 64 + sp + 2] +
                  a3 * wgt[row * 64 + sp + 3];
         }
-        for (; sp < p.splits; ++sp) acc += __ldcg(po + sp * p.dv) * wgt[row * 64 + sp];
-        p.out[qrow * p.dv + d] = __float2bfloat16(acc * linv[row]);
+        for (; sp < p.splits; ++sp) acc += __ldcg(po + sp * dv) * wgt[row * 64 + sp];
+        p.out[qrow * dv + d] = __float2bfloat16(acc * linv[row]);
       }
     }
   }
@@ -865,10 +870,10 @@ extern "C" int eredu_attn_prefill(const void* q, const void* k_cache, const void
   return static_cast<int>(e);
 }
 
-template <int DK, int DV, int MT>
+template <int DK, int DV, int MT, bool EXT>
 static cudaError_t launch_decode(const AttnParams& p, dim3 grid, cudaStream_t stream) {
   static bool cfg[kMaxDevices] = {};
-  if (!configure_once(cfg, attn_decode_kernel<DK, DV, MT>, decode_smem<DK, DV, MT>())) return cudaErrorInvalidValue;
+  if (!configure_once(cfg, attn_decode_kernel<DK, DV, MT, EXT>, decode_smem<DK, DV, MT>())) return cudaErrorInvalidValue;
   cudaLaunchConfig_t lc = {};
   lc.gridDim = grid;
   lc.blockDim = dim3(128);
@@ -890,7 +895,7 @@ static cudaError_t launch_decode(const AttnParams& p, dim3 grid, cudaStream_t st
   }
   lc.attrs = attr;
   lc.numAttrs = nattr;
-  const cudaError_t e = cudaLaunchKernelEx(&lc, attn_decode_kernel<DK, DV, MT>, p);
+  const cudaError_t e = cudaLaunchKernelEx(&lc, attn_decode_kernel<DK, DV, MT, EXT>, p);
   eredu_count_launches(1);
   return e;
 }
@@ -920,10 +925,17 @@ static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_hea
     const int rows = p.t_count * group;
     cudaError_t e;
     const bool one = rows <= 16;
-    if (key_dim > 64 && value_dim > 64) e = one ? launch_decode<128, 128, 1>(p, grid, stream) : launch_decode<128, 128, 2>(p, grid, stream);
-    else if (key_dim > 64) e = one ? launch_decode<128, 64, 1>(p, grid, stream) : launch_decode<128, 64, 2>(p, grid, stream);
-    else if (value_dim > 64) e = one ? launch_decode<64, 128, 1>(p, grid, stream) : launch_decode<64, 128, 2>(p, grid, stream);
-    else e = one ? launch_decode<64, 64, 1>(p, grid, stream) : launch_decode<64, 64, 2>(p, grid, stream);
+    const bool plain = key_dim == value_dim && (key_dim == 64 || key_dim == 128) && p.chunk == 0 && !p.norm_whole && !p.value_norm &&
+                       (p.qkv == nullptr || p.append);
+#define ER_DECODE(DK_, DV_, EXT_) \
+  e = one ? launch_decode<DK_, DV_, 1, EXT_>(p, grid, stream) : launch_decode<DK_, DV_, 2, EXT_>(p, grid, stream)
+    if (plain && key_dim == 128) ER_DECODE(128, 128, false);
+    else if (plain) ER_DECODE(64, 64, false);
+    else if (key_dim > 64 && value_dim > 64) ER_DECODE(128, 128, true);
+    else if (key_dim > 64) ER_DECODE(128, 64, true);
+    else if (value_dim > 64) ER_DECODE(64, 128, true);
+    else ER_DECODE(64, 64, true);
+#undef ER_DECODE
     if (e != cudaSuccess) return static_cast<int>(e);
   }
   return 0;
