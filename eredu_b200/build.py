@@ -78,6 +78,8 @@ def host_sources() -> list[Path]:
 FAMILY_SOURCES = {
     "nidozen": ("attention", "attention_tc", "gemm_persistent", "gemm_tcgen05", "gla", "gla_chunk", "launch_count", "mingru",
                 "residual_stream", "simt_fp32"),
+    "lenitar": ("attention_tc", "gemm_persistent", "gemm_tcgen05", "latent", "latent_attention", "launch_count", "mlstm", "mlstm_chunk",
+                "moe", "residual_stream", "simt_fp32"),
 }
 
 

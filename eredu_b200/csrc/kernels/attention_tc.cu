@@ -27,6 +27,7 @@
 // common exit (TMEM is freed there).
 #include <cuda_bf16.h>
 
+#include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
 #include "../common/ptx.cuh"
@@ -48,6 +49,12 @@ struct AttnTcParams {
   int dk, dv;                  // key / value width of a head (multiples of 8); the rest of a 64-wide half reads as zero
   float scale_log2;
   int* status;
+  // ROWS form: table {first query row, queries, first context row, context rows} per sequence instead of the four arrays above; keys
+  // of dk = dim + rot, of which the last rot are the shared part
+  const int4* table;
+  const __nv_bfloat16* gate;   // optional [tokens, ldg]: column head * dv + i
+  long long ldg;
+  int rot;
 };
 
 constexpr int kTcThreads = 320;
@@ -55,7 +62,9 @@ constexpr int kTcTile = 128;            // query rows per tile and keys per tile
 constexpr int kTcRows = 2 * kTcTile;    // query rows per CTA
 constexpr int kTcHalf = 128 * 64 * 2;   // one [128 rows][64 bf16] swizzled half tile: 16 KB
 // shared memory: Q_a, Q_b (NK halves each) | K ring (2 x NK halves) | V ring (2 x NV halves) | barriers
-constexpr int tc_smem(int nk, int nv) { return 1024 + 2 * (2 * nk + nv) * kTcHalf + 256; }
+// Three key halves and two value halves leave room for one V stage only.
+constexpr int tc_v_stages(int nk, int nv) { return nk + nv > 4 ? 1 : 2; }
+constexpr int tc_smem(int nk, int nv) { return 1024 + (4 * nk + tc_v_stages(nk, nv) * nv) * kTcHalf + 256; }
 // A quarter of the exponentials as a polynomial on the FMA pipe (build option). Measured slower here (1153 against 1192
 // TFLOP/s at 32k tokens, 1112 against 1170 at 8k): the softmax warps are bound by instruction issue, not by the
 // special-function unit, so the extra FMA-pipe instructions cost more than the unit they relieve.
@@ -105,10 +114,11 @@ __device__ __forceinline__ int tc_query_tile(const AttnTcParams& p, int tiles, i
 }
 
 // NK / NV: 64-wide halves of the key and of the value width
-template <int NK, int NV>
+template <int NK, int NV, bool ROWS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                       const __grid_constant__ CUtensorMap tmV, const AttnTcParams p) {
+                       const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR, const AttnTcParams p) {
+  constexpr int VST = tc_v_stages(NK, NV);
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const uint32_t kIdescPV = umma_idesc_bf16(128, (p.dv + 15) & ~15) | (1u << 16);  // B (= V) MN-major, N = value width
@@ -116,7 +126,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   uint8_t* q_s = smem;                                                 // tile w at + w * NK halves
   uint8_t* k_s = q_s + 2 * NK * kTcHalf;                               // stage s at + s * NK (K), s * NV (V) halves
   uint8_t* v_s = k_s + 2 * NK * kTcHalf;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + 2 * NV * kTcHalf);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + VST * NV * kTcHalf);
   uint64_t* q_full = bars;                  // 1
   uint64_t* k_full = bars + 1;              // [2]
   uint64_t* k_empty = bars + 3;             // [2]
@@ -133,8 +143,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   // heads vary fastest: the first wave holds the longest query tiles of every head (longest-first balances the causal
   // triangle), and neighbouring CTAs are query heads of one key / value head reading the same pages
   const int b = blockIdx.z, head = blockIdx.x, qt = tc_query_tile(p, gridDim.y, blockIdx.y);
-  const int q0 = p.cu_q[b], q_len = p.cu_q[b + 1] - q0;
-  const int kv_len = p.seq_lens[b];
+  const int4 seq = ROWS ? p.table[b] : make_int4(p.cu_q[b], p.cu_q[b + 1] - p.cu_q[b], 0, p.seq_lens[b]);
+  const int q0 = seq.x, q_len = seq.y, kv_len = seq.w;
   const int row0 = qt * kTcRows;
   if (row0 >= q_len) return;                                            // uniform: before any barrier or allocation
   const int kv_head = head / (p.n_q_heads / p.n_kv_heads);
@@ -163,6 +173,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
+    if (ROWS) tma_prefetch_desc(&tmR);
   }
   if (warp == 0) {
     tmem_alloc(tmem_slot, 512);
@@ -183,30 +194,40 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       mbar_arrive_expect_tx(q_full, 2 * NK * kTcHalf);
       for (int w = 0; w < 2; ++w)
         for (int h = 0; h < NK; ++h)
-          tma_load_3d(q_s + (w * NK + h) * kTcHalf, &tmQ, h * 64, head, q0 + row0 + w * kTcTile, q_full);
+          // ROWS: the last half starts where the shared part does; a box that reaches beyond the per-head part meets zeros on the key side
+          tma_load_3d(q_s + (w * NK + h) * kTcHalf, &tmQ, ROWS && h == NK - 1 ? p.dk - p.rot : h * 64, head, q0 + row0 + w * kTcTile, q_full);
       const int* pages = p.block_table + static_cast<size_t>(b) * p.max_pages;
       for (int jj = 0; j0 + jj < n_tiles && ok; ++jj) {
         const int j = j0 + jj;                                           // key tile; jj counts this CTA's iterations
         const int s = jj & 1;
         const uint32_t reuse_parity = ((jj >> 1) - 1) & 1;
+        const int sv = VST == 2 ? s : 0;
         int page[8];
+        if (!ROWS) {
 #pragma unroll
-        for (int pg = 0; pg < 8; ++pg) {
-          const int page_index = j * 8 + pg;
-          page[pg] = page_index < p.max_pages ? pages[page_index] : 0;            // beyond the table: the reserved page (masked)
+          for (int pg = 0; pg < 8; ++pg) {
+            const int page_index = j * 8 + pg;
+            page[pg] = page_index < p.max_pages ? pages[page_index] : 0;            // beyond the table: the reserved page (masked)
+          }
         }
         if (jj >= 2) ok = mbar_wait(&k_empty[s], reuse_parity, p.status, kStatusSmemEmptyTimeout);
         if (!ok) break;
         mbar_arrive_expect_tx(&k_full[s], NK * kTcHalf);
+        if (ROWS) {
+          for (int h = 0; h + 1 < NK; ++h) tma_load_3d(k_s + (s * NK + h) * kTcHalf, &tmK, h * 64, head, seq.z + j * kTcTile, &k_full[s]);
+          tma_load_2d(k_s + (s * NK + NK - 1) * kTcHalf, &tmR, 0, seq.z + j * kTcTile, &k_full[s]);
+        }
 #pragma unroll
-        for (int pg = 0; pg < 8; ++pg)
+        for (int pg = 0; pg < (ROWS ? 0 : 8); ++pg)
           for (int h = 0; h < NK; ++h) tma_load_4d(k_s + (s * NK + h) * kTcHalf + pg * 2048, &tmK, h * 64, 0, kv_head, page[pg], &k_full[s]);
-        if (jj >= 2) ok = mbar_wait(&v_empty[s], reuse_parity, p.status, kStatusSmemEmptyTimeout);
+        if (jj >= VST) ok = mbar_wait(&v_empty[sv], VST == 2 ? reuse_parity : (jj - 1) & 1, p.status, kStatusSmemEmptyTimeout);
         if (!ok) break;
-        mbar_arrive_expect_tx(&v_full[s], NV * kTcHalf);
+        mbar_arrive_expect_tx(&v_full[sv], NV * kTcHalf);
+        if (ROWS)
+          for (int h = 0; h < NV; ++h) tma_load_3d(v_s + (sv * NV + h) * kTcHalf, &tmV, h * 64, head, seq.z + j * kTcTile, &v_full[sv]);
 #pragma unroll
-        for (int pg = 0; pg < 8; ++pg)
-          for (int h = 0; h < NV; ++h) tma_load_4d(v_s + (s * NV + h) * kTcHalf + pg * 2048, &tmV, h * 64, 0, kv_head, page[pg], &v_full[s]);
+        for (int pg = 0; pg < (ROWS ? 0 : 8); ++pg)
+          for (int h = 0; h < NV; ++h) tma_load_4d(v_s + (sv * NV + h) * kTcHalf + pg * 2048, &tmV, h * 64, 0, kv_head, page[pg], &v_full[sv]);
       }
     }
   } else if (warp == 1) {
@@ -221,14 +242,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const uint32_t d = tmem + w * 128;
 #pragma unroll
         for (int kk = 0; kk < NK * 4; ++kk) {      // K = key width: four 16-steps per 64-wide half
-          if (kk >= k_steps) break;
+          if (ROWS ? (kk & 3) * 16 >= (kk >> 2 == NK - 1 ? p.rot : p.dk - p.rot - (kk >> 2) * 64) : kk >= k_steps) continue;
           const uint32_t off = (kk >> 2) * kTcHalf + (kk & 3) * 32;
           umma_f16(d, umma_desc_k_sw128(qa + off), umma_desc_k_sw128(ka + off), kIdescQK, kk > 0 ? 1u : 0u);
         }
         umma_commit(&s_full[w]);
       };
       auto issue_pv = [&](int w, int jj, bool fresh) {
-        const uint32_t va = smem_u32(v_s + (jj & 1) * NV * kTcHalf);
+        const uint32_t va = smem_u32(v_s + (VST == 2 ? jj & 1 : 0) * NV * kTcHalf);
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk)             // K = keys: P from tensor memory (8 columns per step), V MN-major (2048 bytes per step)
           umma_f16_ts(tmem + 256 + w * 128, tmem + w * 128 + kk * 8, umma_desc_mn_sw128(va + kk * 2048, kTcHalf), kIdescPV,
@@ -248,7 +269,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         const int j = j0 + jj;
         const bool next = j + 1 < n_tiles;
         bool k_ready = false;
-        ok = mbar_wait(&v_full[jj & 1], (jj >> 1) & 1, p.status, kStatusTmaFullTimeout);
+        ok = mbar_wait(&v_full[VST == 2 ? jj & 1 : 0], (VST == 2 ? jj >> 1 : jj) & 1, p.status, kStatusTmaFullTimeout);
         for (int w = 0; w < 2 && ok; ++w) {
           if (active(w, j)) {
             ok = mbar_wait(&p_full[w], done[w] & 1, p.status, kStatusAccumTimeout);   // P_w(j) is in tensor memory, O_w is rescaled
@@ -257,7 +278,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             issue_pv(w, jj, done[w] == 0);
             ++done[w];
           }
-          if (w == 1) umma_commit(&v_empty[jj & 1]);
+          if (w == 1) umma_commit(&v_empty[VST == 2 ? jj & 1 : 0]);
           if (active(w, j + 1)) {
             if (!k_ready) {
               ok = mbar_wait(&k_full[(jj + 1) & 1], ((jj + 1) >> 1) & 1, p.status, kStatusTmaFullTimeout);
@@ -376,6 +397,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         tmem_ld16(o_addr + c * 16, r);
         tmem_wait_ld();
         if (store) {
+          if (ROWS && p.gate != nullptr) {
+            const uint4* gp = reinterpret_cast<const uint4*>(p.gate + static_cast<size_t>(q0 + tile_row0 + row) * p.ldg + head * p.dv + c * 16);
+            const uint4 g0 = gp[0], g1 = c * 16 + 8 < p.dv ? gp[1] : make_uint4(0u, 0u, 0u, 0u);
+            const uint32_t gw[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+              r[2 * i] = __float_as_uint(__uint_as_float(r[2 * i]) * sigmoid_fast(bf16_lo(gw[i])));
+              r[2 * i + 1] = __float_as_uint(__uint_as_float(r[2 * i + 1]) * sigmoid_fast(bf16_hi(gw[i])));
+            }
+          }
           uint4 v0, v1;
           v0.x = pack_bf16x2(__uint_as_float(r[0]) * inv, __uint_as_float(r[1]) * inv);
           v0.y = pack_bf16x2(__uint_as_float(r[2]) * inv, __uint_as_float(r[3]) * inv);
@@ -405,17 +436,17 @@ using namespace eredu;
 // Causal prefill attention over the paged cache, key / value widths up to 128, optional window or chunks and sink logits.
 // q: [tokens, n_q, key_dim] bf16 (contiguous); k_cache / v_cache: [pages, n_kv, 16, width] bf16 (contiguous); sinks: fp32 [n_q] or
 // null. Same arguments as eredu_attn_prefill otherwise. Returns -2 for shapes it does not take.
-template <int NK, int NV>
-static int launch_attn_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnTcParams& p, dim3 grid,
-                          cudaStream_t stream) {
+template <int NK, int NV, bool ROWS = false>
+static int launch_attn_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmR,
+                          const AttnTcParams& p, dim3 grid, cudaStream_t stream) {
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<NK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(NK, NV)) != cudaSuccess) return -1;
+    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<NK, NV, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(NK, NV)) != cudaSuccess) return -1;
     configured[dev] = true;
   }
-  return static_cast<int>(launch_pdl(attn_prefill_tc_kernel<NK, NV>, grid, dim3(kTcThreads), tc_smem(NK, NV), stream, tmQ, tmK, tmV, p));
+  return static_cast<int>(launch_pdl(attn_prefill_tc_kernel<NK, NV, ROWS>, grid, dim3(kTcThreads), tc_smem(NK, NV), stream, tmQ, tmK, tmV, tmR, p));
 }
 
 extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
@@ -454,8 +485,58 @@ extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const v
   p.status = status;
   dim3 grid(n_q_heads, (max_q_len + kTcRows - 1) / kTcRows, batch);
   int e;
-  if (key_dim > 64) e = value_dim > 64 ? launch_attn_tc<2, 2>(tmQ, tmK, tmV, p, grid, stream) : launch_attn_tc<2, 1>(tmQ, tmK, tmV, p, grid, stream);
-  else e = value_dim > 64 ? launch_attn_tc<1, 2>(tmQ, tmK, tmV, p, grid, stream) : launch_attn_tc<1, 1>(tmQ, tmK, tmV, p, grid, stream);
+  if (key_dim > 64) e = value_dim > 64 ? launch_attn_tc<2, 2>(tmQ, tmK, tmV, tmK, p, grid, stream) : launch_attn_tc<2, 1>(tmQ, tmK, tmV, tmK, p, grid, stream);
+  else e = value_dim > 64 ? launch_attn_tc<1, 2>(tmQ, tmK, tmV, tmK, p, grid, stream) : launch_attn_tc<1, 1>(tmQ, tmK, tmV, tmK, p, grid, stream);
+  eredu_count_launches(1);
+  return e;
+}
+
+// The ROWS form. q [total_q rows of ldq elements], head h at column h * (dim + rot): [per-head part (dim) | shared part (rot)]; k [rows of
+// ldkv], head h at h * dim; v [rows of ldkv], head h at h * value_dim; kr [rows of ldkr]: the shared key part; table [n_seq] int4
+// {first query row, queries, first context row, context rows}: the queries are the last positions of their context rows. gate
+// [total_q rows of ldg] or null, column h * value_dim + i. out [total_q, heads, value_dim]. dim, value_dim <= 128, rot <= 64, all
+// multiples of 8, pitches and pointers 16-byte aligned.
+extern "C" int eredu_attn_prefill_rows(const void* q, const void* k, const void* v, const void* kr, const void* gate, const float* sinks,
+                                       void* out, const int* table, int n_seq, int total_q, int rows, int max_q, int heads, int dim,
+                                       int rot, int value_dim, int window, long long ldq, long long ldkv, long long ldkr, long long ldg,
+                                       float scale, int* status, cudaStream_t stream) {
+  if (n_seq <= 0 || max_q <= 0 || rows <= 0) return 0;
+  if (dim <= 0 || dim > 128 || dim % 8 != 0 || rot <= 0 || rot > 64 || rot % 8 != 0 || value_dim <= 0 || value_dim > 128 ||
+      value_dim % 8 != 0 || heads <= 0 || window < 0 || n_seq > 65535)
+    return -2;
+  const uint64_t D = static_cast<uint64_t>(dim), R = static_cast<uint64_t>(rot), V = static_cast<uint64_t>(value_dim);
+  const uint64_t H = static_cast<uint64_t>(heads);
+  CUtensorMap tmQ, tmK, tmV, tmR;
+  int r = make_tma_3d(&tmQ, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D + R, H, static_cast<uint64_t>(total_q), (D + R) * 2, ldq * 2, 64, 1, 128);
+  if (r != 0) return -100 + r;
+  r = make_tma_3d(&tmK, k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, H, static_cast<uint64_t>(rows), D * 2, ldkv * 2, 64, 1, 128);
+  if (r != 0) return -200 + r;
+  r = make_tma_3d(&tmV, v, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, V, H, static_cast<uint64_t>(rows), V * 2, ldkv * 2, 64, 1, 128);
+  if (r != 0) return -300 + r;
+  r = make_tma_2d(&tmR, kr, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, static_cast<uint64_t>(rows), R, static_cast<uint64_t>(ldkr), 128, 64);
+  if (r != 0) return -400 + r;
+  AttnTcParams p = {};
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.sinks = sinks;
+  p.n_q_heads = heads;
+  p.n_kv_heads = heads;
+  p.window = window;
+  p.dk = dim + rot;
+  p.dv = value_dim;
+  p.rot = rot;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.status = status;
+  p.table = reinterpret_cast<const int4*>(table);
+  p.gate = static_cast<const __nv_bfloat16*>(gate);
+  p.ldg = ldg;
+  const dim3 grid(heads, (max_q + kTcRows - 1) / kTcRows, n_seq);
+  if (grid.y > 65535) return -2;
+  int e;
+#define ER_ROWS(NK_) \
+  e = value_dim > 64 ? launch_attn_tc<NK_, 2, true>(tmQ, tmK, tmV, tmR, p, grid, stream) : launch_attn_tc<NK_, 1, true>(tmQ, tmK, tmV, tmR, p, grid, stream)
+  if (dim > 64) ER_ROWS(3);
+  else ER_ROWS(2);
+#undef ER_ROWS
   eredu_count_launches(1);
   return e;
 }

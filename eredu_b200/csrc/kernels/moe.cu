@@ -21,11 +21,11 @@ enum { SCORE_SOFTMAX = 0, SCORE_SIGMOID = 1, SCORE_SQRT_SOFTPLUS = 2, SCORE_TOPK
 // One warp routes one token, up to 512 experts (16 per lane).
 __device__ __forceinline__ void route_token(const float* __restrict__ logits, const float* __restrict__ sel_bias,
                                             int* __restrict__ ids, float* __restrict__ weights, int t, int lane, int E, int k,
-                                            int scoring, int renorm, float scale) {
+                                            int scoring, int renorm, float scale, int ld, int n_group, int keep_groups) {
   constexpr int PER = 16;
   float score[PER];   // value reported as the route weight
   float select[PER];  // value used for selection (score + bias)
-  const float* row = logits + static_cast<size_t>(t) * E;
+  const float* row = logits + static_cast<size_t>(t) * ld;
   float mx = -INFINITY;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
@@ -61,6 +61,47 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
   for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
     select[j] = (e < E) ? score[j] + (sel_bias != nullptr ? sel_bias[e] : 0.f) : -INFINITY;
+  }
+  if (n_group > 1) {
+    // group-limited selection: experts form equal groups of neighbours, a group's score is the sum of its two largest, and only the
+    // best keep_groups groups stay eligible. Lane g keeps the score of group g.
+    const int per = E / n_group;
+    float group_score = -INFINITY;
+    for (int gr = 0; gr < n_group; ++gr) {
+      float t1 = -INFINITY, t2 = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < PER; ++j) {
+        const int e = lane + 32 * j;
+        if (e >= gr * per && e < (gr + 1) * per) {
+          t2 = fmaxf(t2, fminf(t1, select[j]));
+          t1 = fmaxf(t1, select[j]);
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float o1 = __shfl_xor_sync(0xffffffffu, t1, o), o2 = __shfl_xor_sync(0xffffffffu, t2, o);
+        t2 = fmaxf(fmaxf(t2, o2), fminf(t1, o1));
+        t1 = fmaxf(t1, o1);
+      }
+      if (lane == gr) group_score = per > 1 ? t1 + t2 : t1;
+    }
+    uint32_t kept = 0u;
+    for (int i = 0; i < keep_groups; ++i) {
+      float best = lane < n_group && !((kept >> lane) & 1u) ? group_score : -INFINITY;
+      int best_g = best == -INFINITY ? 0x7fffffff : lane;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
+        if (ob > best || (ob == best && og < best_g)) { best = ob; best_g = og; }
+      }
+      if (best_g < 32) kept |= 1u << best_g;
+    }
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+      const int e = lane + 32 * j;
+      if (e < E && !((kept >> (e / per)) & 1u)) select[j] = -INFINITY;
+    }
   }
   float wsum = 0.f;
   float my_w = 0.f;  // lane i keeps the weight of slot i
@@ -111,15 +152,15 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
   }
 }
 
-__global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ sel_bias,
+__global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ sel_bias,
                                                          int* __restrict__ ids, float* __restrict__ weights, int T, int E,
-                                                         int k, int scoring, int renorm, float scale) {
+                                                         int k, int scoring, int renorm, float scale, int n_group, int keep_groups) {
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= T) return;
-  route_token(logits, sel_bias, ids, weights, t, threadIdx.x & 31, E, k, scoring, renorm, scale);
+  route_token(logits, sel_bias, ids, weights, t, threadIdx.x & 31, E, k, scoring, renorm, scale, ld, n_group, keep_groups);
 }
 
 // Single CTA. routes = T*k. Experts [e0, e1) are local. Outputs:
@@ -195,15 +236,15 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
 // three dependent launches. 32 warps route the tokens, the block plans the local experts' segments in shared
 // memory, then copies the token rows into expert order.
 __global__ void __launch_bounds__(1024) moe_route_plan_gather_kernel(
-    const float* __restrict__ logits, const float* __restrict__ sel_bias, int* __restrict__ ids, float* __restrict__ weights,
-    int T, int E, int k, int scoring, int renorm, float scale, int e0, int e1, int tile, int* __restrict__ seg,
+    const float* __restrict__ logits, int ld, const float* __restrict__ sel_bias, int* __restrict__ ids, float* __restrict__ weights,
+    int T, int E, int k, int scoring, int renorm, float scale, int n_group, int keep_groups, int e0, int e1, int tile, int* __restrict__ seg,
     int* __restrict__ route_pos, int* __restrict__ row_token, int4* __restrict__ work, int n_work_cap, int* __restrict__ counts,
     const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ xp, int H) {
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int t = warp; t < T; t += 32) route_token(logits, sel_bias, ids, weights, t, lane, E, k, scoring, renorm, scale);
+  for (int t = warp; t < T; t += 32) route_token(logits, sel_bias, ids, weights, t, lane, E, k, scoring, renorm, scale, ld, n_group, keep_groups);
   __syncthreads();  // ids written by this block are visible to it
   plan_block(ids, T * k, k, e0, e1, tile, seg, route_pos, row_token, work, n_work_cap, counts);
   __syncthreads();
@@ -614,12 +655,14 @@ __global__ void __launch_bounds__(128) moe_a2a_combine_kernel(PeerComm c, A2AVie
 
 using namespace eredu;
 
-extern "C" int eredu_moe_route(const float* logits, const float* sel_bias, int* ids, float* weights, int T, int E, int k,
-                               int scoring, int renorm, float scale, cudaStream_t stream) {
+// logits [T, ld], of which E entries per row. n_group > 1: group-limited selection (E in n_group <= 32 equal groups, the best
+// keep_groups stay eligible).
+extern "C" int eredu_moe_route(const float* logits, int ld, const float* sel_bias, int* ids, float* weights, int T, int E, int k,
+                               int scoring, int renorm, float scale, int n_group, int keep_groups, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (E > 512 || k > 32 || k > E) return -1;
-  launch_pdl(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, sel_bias, ids, weights, T, E, k, scoring,
-             renorm, scale);
+  if (E > 512 || k > 32 || k > E || n_group < 1 || n_group > 32 || E % n_group != 0 || keep_groups < 1 || keep_groups > n_group) return -1;
+  launch_pdl(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, sel_bias, ids, weights, T, E, k, scoring,
+             renorm, scale, n_group, keep_groups);
   eredu_count_launches(1);
   return static_cast<int>(cudaGetLastError());
 }
@@ -671,14 +714,15 @@ extern "C" int eredu_moe_combine_ar(const void* y, const int* route_pos, const f
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int eredu_moe_route_plan_gather(const float* logits, const float* sel_bias, int* ids, float* weights, int T, int E,
-                                           int k, int scoring, int renorm, float scale, int e0, int e1, int tile, int* seg,
+extern "C" int eredu_moe_route_plan_gather(const float* logits, int ld, const float* sel_bias, int* ids, float* weights, int T, int E,
+                                           int k, int scoring, int renorm, float scale, int n_group, int keep_groups, int e0, int e1, int tile, int* seg,
                                            int* route_pos, int* row_token, int* work, int n_work_cap, int* counts,
                                            const void* x, void* xp, int H, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E > 512 || k > 32 || k > E || e1 - e0 > 512 || e1 <= e0 || H % 8 != 0 || T > 64) return -1;
-  launch_pdl(moe_route_plan_gather_kernel, dim3(1), dim3(1024), 0, stream, logits, sel_bias, ids, weights, T, E, k, scoring,
-             renorm, scale, e0, e1, tile, seg, route_pos, row_token, reinterpret_cast<int4*>(work), n_work_cap, counts,
+  if (n_group < 1 || n_group > 32 || E % n_group != 0 || keep_groups < 1 || keep_groups > n_group) return -1;
+  launch_pdl(moe_route_plan_gather_kernel, dim3(1), dim3(1024), 0, stream, logits, ld, sel_bias, ids, weights, T, E, k, scoring,
+             renorm, scale, n_group, keep_groups, e0, e1, tile, seg, route_pos, row_token, reinterpret_cast<int4*>(work), n_work_cap, counts,
              static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(xp), H);
   eredu_count_launches(1);
   return static_cast<int>(cudaGetLastError());

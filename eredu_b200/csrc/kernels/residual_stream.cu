@@ -1,5 +1,6 @@
-// Glue of decoders that keep their residual stream in fp32 and normalise a sublayer's OUTPUT before it is added:
-//   * rms_residual: x = residual + w * y / rms(y), in fp32, plus the copy of x in the compute dtype that the next
+// Glue of decoders that keep their residual stream in fp32:
+//   * residual_norm: x' = x + y + the weighted expert rows of the token, and LayerNorm or RMSNorm of x' for the next layer
+//   * rms_residual (a norm on a sublayer's OUTPUT): x = residual + w * y / rms(y), in fp32, plus the copy of x in the compute dtype that the next
 //     projections read (one number or one vector as w; without a residual: a plain norm, as in front of the head)
 //   * embedding_stream: the first rows of the stream and their copy
 //   * qkv_prepare: RMSNorm over the WHOLE query and key projections, rotation of the leading dims of every head, RMSNorm of
@@ -82,9 +83,142 @@ static cudaError_t launch_rms_residual(const TY* y, const float* w, int w_vec, c
 #undef ER_RMS
 }
 
+struct ResidualNormParams {
+  const float* x;           // [M, W]
+  const void* y;            // [M, W] a sublayer's output, or null
+  const void* rows;         // expert outputs, or null
+  const int* route_pos;     // [M * k] row of a route, negative: none
+  const float* route_w;     // [M * k]
+  const float* weight;      // [W], or null: no norm
+  const float* bias;        // [W] or null
+  float* x_out;             // [M, W]; null when nothing is added
+  void* act;                // [M, W]
+  int W, k, center;
+  float eps;
+};
+
+constexpr int kMaxRoutes = 32;
+
+// One CTA per row. NV groups of four columns per thread stay in registers; NV = 0: any width, the sum is read back.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) residual_norm_kernel(ResidualNormParams p) {
+  __shared__ float red[8];
+  __shared__ int pos[kMaxRoutes];
+  __shared__ float rw[kMaxRoutes];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int W = p.W;
+  const size_t base = static_cast<size_t>(blockIdx.x) * W;
+  const T* y = static_cast<const T*>(p.y);
+  const T* rows = static_cast<const T*>(p.rows);
+  T* act = static_cast<T*>(p.act);
+  const float n = static_cast<float>(W);
+  if (p.k > 0) {
+    if (threadIdx.x < p.k) {
+      pos[threadIdx.x] = p.route_pos[static_cast<size_t>(blockIdx.x) * p.k + threadIdx.x];
+      rw[threadIdx.x] = p.route_w[static_cast<size_t>(blockIdx.x) * p.k + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  if constexpr (NV > 0) {
+    float4 v[NV];
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < W) {
+        v[i] = load4(p.x + base + c);
+        if (y != nullptr) {
+          const float4 a = load4(y + base + c);
+          v[i] = make_float4(v[i].x + a.x, v[i].y + a.y, v[i].z + a.z, v[i].w + a.w);
+        }
+      }
+    }
+#pragma unroll 4
+    for (int s = 0; s < p.k; ++s) {
+      if (pos[s] < 0) continue;
+      const T* r = rows + static_cast<size_t>(pos[s]) * W;
+      const float w = rw[s];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * 256) * 4;
+        if (c >= W) continue;
+        const float4 a = load4(r + c);
+        v[i] = make_float4(fmaf(w, a.x, v[i].x), fmaf(w, a.y, v[i].y), fmaf(w, a.z, v[i].z), fmaf(w, a.w, v[i].w));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c < W && p.x_out != nullptr) store4(p.x_out + base + c, v[i]);
+      sum += v[i].x + v[i].y + v[i].z + v[i].w;
+    }
+    if (p.weight == nullptr) return;
+    const float mean = p.center ? block_sum_f32(sum, red) / n : 0.f;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      if ((threadIdx.x + i * 256) * 4 >= W) continue;
+      v[i] = make_float4(v[i].x - mean, v[i].y - mean, v[i].z - mean, v[i].w - mean);
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= W) continue;
+      const float4 g = load4(p.weight + c);
+      const float4 b = p.bias != nullptr ? load4(p.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      store4(act + base + c, make_float4(fmaf(v[i].x * inv, g.x, b.x), fmaf(v[i].y * inv, g.y, b.y), fmaf(v[i].z * inv, g.z, b.z),
+                                         fmaf(v[i].w * inv, g.w, b.w)));
+    }
+  } else {
+    const float* src = p.x_out != nullptr ? p.x_out : p.x;      // a thread reads back only what it wrote itself
+    float sum = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) {
+      float v = p.x[base + c];
+      if (y != nullptr) v += to_f32(y[base + c]);
+      for (int s = 0; s < p.k; ++s)
+        if (pos[s] >= 0) v = fmaf(rw[s], to_f32(rows[static_cast<size_t>(pos[s]) * W + c]), v);
+      if (p.x_out != nullptr) p.x_out[base + c] = v;
+      sum += v;
+    }
+    if (p.weight == nullptr) return;
+    const float mean = p.center ? block_sum_f32(sum, red) / n : 0.f;
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float d = src[base + c] - mean;
+      ss += d * d;
+    }
+    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    for (int c = threadIdx.x; c < W; c += 256)
+      act[base + c] = from_f32<T>(fmaf((src[base + c] - mean) * inv, p.weight[c], p.bias != nullptr ? p.bias[c] : 0.f));
+  }
+}
+
+template <typename T>
+static cudaError_t launch_residual_norm(const ResidualNormParams& p, int M, bool quads_ok, cudaStream_t stream) {
+  const int quads = quads_ok ? (p.W / 4 + 255) / 256 : 0;
+#define ER_RN(NV_) launch_pdl(residual_norm_kernel<T, NV_>, dim3(M), dim3(256), 0, stream, p)
+  switch (quads) {
+    case 1: return ER_RN(1);
+    case 2: return ER_RN(2);
+    case 3:
+    case 4: return ER_RN(4);
+    case 5:
+    case 6:
+    case 7:
+    case 8: return ER_RN(8);
+    default: return ER_RN(0);
+  }
+#undef ER_RN
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table,
-                                                                float* __restrict__ x, T* __restrict__ act, int W, int rows) {
+                                                                float* __restrict__ x, T* __restrict__ act, int W, int rows, float scale) {
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
@@ -93,9 +227,9 @@ __global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __rest
   const T* src = table + static_cast<size_t>(ok ? id : 0) * W;
   const size_t base = static_cast<size_t>(blockIdx.x) * W;
   for (int c = threadIdx.x; c < W; c += 256) {
-    const T v = ok ? src[c] : from_f32<T>(0.f);
-    x[base + c] = to_f32(v);
-    if (act != nullptr) act[base + c] = v;
+    const float v = ok ? to_f32(src[c]) * scale : 0.f;
+    x[base + c] = v;
+    if (act != nullptr) act[base + c] = from_f32<T>(v);
   }
 }
 
@@ -204,15 +338,29 @@ extern "C" int eredu_rms_residual(const void* y, const float* w, const float* re
   return static_cast<int>(e);
 }
 
-// table [rows, W] bf16 or fp32; x fp32 [M, W]; act [M, W] in the table's dtype or null.
+// x, x_out, weight, bias fp32; y, rows, act bf16 (fp32 = 0) or fp32; k <= 32 routes per row; quads: rows are whole 16-byte pieces.
+extern "C" int eredu_residual_norm(const float* x, const void* y, const void* rows, const int* route_pos, const float* route_w,
+                                   const float* weight, const float* bias, float* x_out, void* act, int M, int W, int k, int fp32, int center,
+                                   int quads, float eps, cudaStream_t stream) {
+  if (M <= 0 || W <= 0) return 0;
+  if (k < 0 || k > kMaxRoutes || (k > 0 && (rows == nullptr || route_pos == nullptr || route_w == nullptr)) ||
+      (weight != nullptr && act == nullptr) || (x_out == nullptr && (y != nullptr || k > 0)))
+    return -1;
+  const ResidualNormParams p = {x, y, rows, route_pos, route_w, weight, bias, x_out, act, W, k, center, eps};
+  const cudaError_t e = fp32 ? launch_residual_norm<float>(p, M, quads != 0, stream) : launch_residual_norm<__nv_bfloat16>(p, M, quads != 0, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// table [rows, W] bf16 or fp32, times scale; x fp32 [M, W]; act [M, W] in the table's dtype or null.
 extern "C" int eredu_embedding_stream(const int* ids, const void* table, float* x, void* act, int M, int W, int rows, int fp32,
-                                      cudaStream_t stream) {
+                                      float scale, cudaStream_t stream) {
   if (M <= 0 || W <= 0) return 0;
   cudaError_t e;
   if (fp32) e = launch_pdl(embedding_stream_kernel<float>, dim3(M), dim3(256), 0, stream, ids, static_cast<const float*>(table), x,
-                           static_cast<float*>(act), W, rows);
+                           static_cast<float*>(act), W, rows, scale);
   else e = launch_pdl(embedding_stream_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, stream, ids,
-                      static_cast<const __nv_bfloat16*>(table), x, static_cast<__nv_bfloat16*>(act), W, rows);
+                      static_cast<const __nv_bfloat16*>(table), x, static_cast<__nv_bfloat16*>(act), W, rows, scale);
   eredu_count_launches(1);
   return static_cast<int>(e);
 }

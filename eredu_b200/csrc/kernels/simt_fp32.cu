@@ -59,20 +59,78 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ x,
   }
 }
 
+// Expert GEMMs over the work items of a routing plan ({expert, first row, rows, -}): Y[row] = X[index ? index[row] : row] W_e^T, or
+// with DUAL silu(X Wg^T) * (X Wu^T), Wg / Wu the first / following N rows of the expert's matrix. A CTA takes 64 rows at most.
+template <typename T, bool DUAL>
+__global__ void __launch_bounds__(256) gemm_simt_grouped_kernel(const T* __restrict__ x, const T* __restrict__ w, T* __restrict__ y,
+                                                                 const int4* __restrict__ work, const int* __restrict__ index, int N,
+                                                                 int K, int ldx, int ldy, int w_rows) {
+  __shared__ float xs[kTileK][kTile + 4], ws[DUAL ? 2 : 1][kTileK][kTile + 4];
+  __shared__ int src[kTile];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int4 item = work[blockIdx.y];
+  const int rows = min(item.z, kTile);
+  if (rows <= 0) return;
+  const int n0 = blockIdx.x * kTile;
+  const T* we = w + static_cast<size_t>(item.x) * w_rows * K;
+  if (threadIdx.x < kTile) src[threadIdx.x] = threadIdx.x < rows ? (index != nullptr ? index[item.y + threadIdx.x] : item.y + threadIdx.x) : 0;
+  __syncthreads();
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  float acc[DUAL ? 2 : 1][4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kTileK) {
+    for (int i = threadIdx.x; i < kTile * kTileK; i += 256) {
+      const int r = i / kTileK, k = i % kTileK;
+      const bool kin = k0 + k < K, nin = kin && n0 + r < N;
+      xs[k][r] = r < rows && kin ? to_f32(x[static_cast<size_t>(src[r]) * ldx + k0 + k]) : 0.f;
+      ws[0][k][r] = nin ? to_f32(we[static_cast<size_t>(n0 + r) * K + k0 + k]) : 0.f;
+      if constexpr (DUAL) ws[1][k][r] = nin ? to_f32(we[static_cast<size_t>(N + n0 + r) * K + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kTileK; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[k][ty * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+      for (int d = 0; d < (DUAL ? 2 : 1); ++d) {
+        const float4 b = *reinterpret_cast<const float4*>(&ws[d][k][tx * 4]);
+        const float bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[d][i][j] = fmaf(av[i], bv[j], acc[d][i][j]);
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = ty * 4 + i;
+    if (r >= rows) break;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= N) break;
+      y[static_cast<size_t>(item.y + r) * ldy + n] = from_f32<T>(DUAL ? silu_f32(acc[0][i][j]) * acc[DUAL ? 1 : 0][i][j] : acc[0][i][j]);
+    }
+  }
+}
+
 struct AttnSimtParams {
   const void* q;         // [total_q, n_q, dk]
   const void* k_cache;   // [pages, n_kv, 16, dk]
-  const void* v_cache;   // [pages, n_kv, 16, dv]
+  const void* v_cache;   // [pages, n_kv, 16, ldv], of which the first dv entries of a row are the value
   void* out;             // [total_q, n_q, dv]
   const int* block_table;
   const int* seq_lens;
   const int* cu_q;       // null: q_per_seq queries per sequence
   const float* sinks;    // [n_q] or null
-  int q_per_seq, max_pages, n_q, n_kv, dk, dv, window, chunk;
+  int q_per_seq, max_pages, n_q, n_kv, dk, dv, ldv, window, chunk;
   float scale;
 };
 
-constexpr int kMaxValueRegs = 16;  // value widths up to 512
+constexpr int kMaxValueRegs = 32;  // value widths up to 1024
 
 // One CTA per (query token, head); its four warps take every fourth group of 32 keys, one key per lane for the scores and
 // one value column per lane for the sum, each with a running maximum of its own; merged at the end.
@@ -127,7 +185,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(AttnSimtParams p) {
     for (int j = 0; j < n; ++j) {
       const float pj = __shfl_sync(0xffffffffu, pe, j);
       const size_t rj = __shfl_sync(0xffffffffu, static_cast<unsigned long long>(row), j);
-      const T* v = static_cast<const T*>(p.v_cache) + rj * p.dv;
+      const T* v = static_cast<const T*>(p.v_cache) + rj * p.ldv;
 #pragma unroll
       for (int c = 0; c < kMaxValueRegs; ++c)
         if (lane + 32 * c < p.dv) acc[c] = fmaf(pj, to_f32(v[lane + 32 * c]), acc[c]);
@@ -186,13 +244,14 @@ extern "C" int eredu_gemm_simt(const void* x, const void* w, void* y, const void
   return static_cast<int>(e);
 }
 
-// Causal attention over the paged cache for any key width and value widths up to 512; arguments as the tensor-core kernels.
+// Causal attention over the paged cache for any key width and value widths up to 1024; arguments as the tensor-core kernels. Rows of
+// v_cache are ldv >= dv wide: the values may be the head of a wider row (latent attention passes the same rows as keys and values).
 extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                                const int* seq_lens, const int* cu_q, const float* sinks, int batch, int q_per_seq, int max_q_len,
-                               int max_pages, int n_q, int n_kv, int dk, int dv, int window, int chunk, int fp32, float scale,
+                               int max_pages, int n_q, int n_kv, int dk, int dv, int ldv, int window, int chunk, int fp32, float scale,
                                cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || dk <= 0 || dv <= 0 || dv > 32 * kMaxValueRegs || window < 0 || chunk < 0) return -1;
+  if (n_kv <= 0 || n_q % n_kv != 0 || dk <= 0 || dv <= 0 || dv > 32 * kMaxValueRegs || ldv < dv || window < 0 || chunk < 0) return -1;
   AttnSimtParams p;
   p.q = q;
   p.k_cache = k_cache;
@@ -208,6 +267,7 @@ extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v
   p.n_kv = n_kv;
   p.dk = dk;
   p.dv = dv;
+  p.ldv = ldv;
   p.window = window;
   p.chunk = chunk;
   p.scale = scale;
@@ -216,6 +276,27 @@ extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v
   const dim3 grid(max_q_len, n_q, batch);
   const cudaError_t e = fp32 ? launch_pdl(attn_simt_kernel<float>, grid, dim3(128), smem, stream, p)
                              : launch_pdl(attn_simt_kernel<__nv_bfloat16>, grid, dim3(128), smem, stream, p);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// work [n_work] int4 items of at most 64 rows; w [experts, w_rows, K] (dual: gate rows, then up rows); index: source row of every row of
+// X (null: the row itself). X, W and Y fp32 or bf16 alike.
+extern "C" int eredu_gemm_simt_grouped(const void* x, const void* w, void* y, const int* work, int n_work, const int* index, int N, int K,
+                                       int ldx, int ldy, int w_rows, int dual, int fp32, cudaStream_t stream) {
+  if (n_work <= 0 || N <= 0 || K <= 0) return 0;
+  if (n_work > 65535) return -1;
+  const dim3 grid((N + kTile - 1) / kTile, n_work);
+  const int4* items = reinterpret_cast<const int4*>(work);
+  cudaError_t e;
+#define ER_GROUPED_SIMT(T_, D_)                                                                                                \
+  e = launch_pdl(gemm_simt_grouped_kernel<T_, D_>, grid, dim3(256), 0, stream, static_cast<const T_*>(x), static_cast<const T_*>(w), \
+                 static_cast<T_*>(y), items, index, N, K, ldx, ldy, w_rows)
+  if (fp32 && dual) ER_GROUPED_SIMT(float, true);
+  else if (fp32) ER_GROUPED_SIMT(float, false);
+  else if (dual) ER_GROUPED_SIMT(__nv_bfloat16, true);
+  else ER_GROUPED_SIMT(__nv_bfloat16, false);
+#undef ER_GROUPED_SIMT
   eredu_count_launches(1);
   return static_cast<int>(e);
 }

@@ -5,6 +5,7 @@ Defaults and field fall-backs follow the reference's Llama/Qwen config readers
 """
 from __future__ import annotations
 
+import importlib
 import json
 from dataclasses import dataclass, field, asdict
 from pathlib import Path
@@ -14,12 +15,37 @@ DENSE_TYPES = {"llama", "mistral", "qwen2", "qwen3", "phi3", "lfm2"}
 MOE_TYPES = {"qwen3_moe", "mixtral", "gpt_oss", "deepseek_v3", "lfm2_moe", "nemotron_h", "qwen3_next", "qwen3_5_moe", "qwen3_5_moe_text"}
 QWEN_HYBRID_TYPES = {"qwen3_next", "qwen3_5", "qwen3_5_moe", "qwen3_5_text", "qwen3_5_moe_text"}
 
+# Families whose layers each name their mixer and its sizes (``ModelConfig.mixers``). ``models/<model type>.py`` reads the
+# configuration and the tensors, and runs a block.
+MIXER_FAMILIES = ("nidozen", "lenitar")
+
+
+def mixer_family(model_type: str):
+    """Module of a family with per-layer mixers, None for every other model type."""
+    if model_type not in MIXER_FAMILIES:
+        return None
+    return importlib.import_module(f"{__package__}.{model_type}")
+
+
+@dataclass
+class RoutedSpec:
+    """Sparse feed-forward of one layer (the field names the expert block and its router read)."""
+    num_experts: int
+    num_experts_per_tok: int
+    moe_intermediate_size: int
+    n_group: int = 1                 # experts in equal groups of neighbours, of which the topk_group best stay eligible
+    topk_group: int = 1
+    router_scoring: str = "sigmoid"
+    norm_topk_prob: bool = False
+    routed_scaling_factor: float = 1.0
+    swiglu_limit: float = 0.0
+
 
 @dataclass
 class MixerSpec:
     """Geometry and constants of one layer of a family whose layers do not share them (``ModelConfig.mixers``)."""
-    kind: str                        # "attention" | "gla" (gated linear attention) | "mingru"
-    heads: int = 0                   # query heads (attention) or recurrent heads (gla)
+    kind: str                        # "attention" | "latent_attention" | "gla" (gated linear attention) | "mingru" | "mlstm"
+    heads: int = 0                   # query heads (attention) or recurrent heads (gla, mlstm)
     kv_heads: int = 0
     dim: int = 0                     # query / key size of a head
     vdim: int = 0                    # value size of a head
@@ -31,6 +57,18 @@ class MixerSpec:
     kv_from: int | None = None       # attention: the earlier layer whose cached keys and values are read
     tau: float = 1.0                 # gla: decay = sigmoid(z)^(1 / tau)
     ff: int = 0                      # feed-forward width (0: the layer has none)
+    window: int = 0                  # attention: keys at most window - 1 positions back are visible (0: all earlier)
+    q_rank: int = 0                  # latent attention: width of the query latent
+    kv_rank: int = 0                 # latent attention: width of the cached latent (``rot_dims`` more hold the rotated key part)
+    gate_cap: float = 0.0            # mlstm: soft cap of the gates' pre-activations
+    moe: RoutedSpec | None = None    # sparse feed-forward
+
+    @property
+    def kv_dims(self) -> tuple:
+        """(heads, key width, value width) of one cached token."""
+        if self.kind == "latent_attention":
+            return 1, self.kv_rank + self.rot_dims, 0
+        return self.kv_heads, self.dim, self.vdim
 
     @property
     def state_shape(self) -> tuple | None:
@@ -39,6 +77,9 @@ class MixerSpec:
             return (self.width,)
         if self.kind == "gla":
             return (self.heads, self.dim, self.vdim)
+        if self.kind == "mlstm":
+            # matrix memories, then normaliser vectors, then running maxima, padded to whole 16-byte pieces
+            return (-(-self.heads * (self.dim * self.vdim + self.dim + 1) // 4) * 4,)
         return None
 
 
@@ -137,8 +178,7 @@ class ModelConfig:
     def layer_kv_dims(self, layer: int) -> tuple:
         """(heads, key width, value width) of one cached token of this layer."""
         if self.mixers is not None:
-            m = self.mixers[layer]
-            return m.kv_heads, m.dim, m.vdim
+            return self.mixers[layer].kv_dims
         return self.kv_cache_dims
 
     def layer_kv_donor(self, layer: int) -> int | None:
@@ -185,7 +225,8 @@ class ModelConfig:
     def layer_has_kv(self, layer: int) -> bool:
         """The layer appends K/V pages (softmax attention); every other operator keeps a fixed state or none."""
         if self.mixers is not None:
-            return self.mixers[layer].kind == "attention" and self.mixers[layer].kv_from is None
+            m = self.mixers[layer]
+            return m.kind in ("attention", "latent_attention") and m.kv_from is None
         if self.layer_types is None:
             return True
         if self.model_type == "gemma4":      # the KV-sharing tail reads an earlier layer's pages
@@ -212,10 +253,8 @@ class ModelConfig:
         return self.sliding_window
 
     def to_hf_dict(self) -> dict:
-        if self.model_type == "nidozen":
-            from .nidozen import config_dict
-
-            return config_dict(self)
+        if mixer_family(self.model_type) is not None:
+            return mixer_family(self.model_type).config_dict(self)
         d = {k: v for k, v in asdict(self).items() if k not in ("extra", "mixers", "qk_norm", "rope_traditional",
                                                                 "norm_weight_offset", "embedding_scale",
                                                                 "router_scoring", "attention_sinks", "quantization",
@@ -296,10 +335,9 @@ class ModelConfig:
     # -------------------------------------------------------------------------------------- HF
     @classmethod
     def from_hf_dict(cls, d: dict) -> "ModelConfig":
-        if d.get("architecture") == "Nidozen" or d.get("model_type") == "nidozen":
-            from .nidozen import config_from_dict
-
-            return config_from_dict(cls, d)
+        family = mixer_family(str(d.get("model_type") or d.get("architecture", "")).lower())
+        if family is not None:
+            return family.config_from_dict(cls, d)
         mt = d.get("model_type", "llama")
         if "text_config" in d and isinstance(d["text_config"], dict):
             outer = d

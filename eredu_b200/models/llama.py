@@ -23,7 +23,7 @@ import torch
 
 from .. import ops
 from ..utils import nvtx
-from .config import ModelConfig
+from .config import ModelConfig, mixer_family
 from .rope import rope_tables
 
 
@@ -63,8 +63,17 @@ class ForwardBatch:
     layer_hidden: Optional[dict] = None
     # families with an fp32 residual stream: (stream, its copy in the compute dtype) as the last sublayer left them
     stream: Optional[tuple] = None
+    # prefill: (first new position, new tokens) of every sequence, known on the host (operators that size scratch by context)
+    portions: Optional[list] = None
     max_kv_len: int = 0                # decode: the longest context the step (or every replay of its graph) can see
     sm_count: int = 1
+
+    def host_portions(self) -> list:
+        """``portions``, read back from the device where whoever made the batch did not state them."""
+        if self.portions is None:
+            cu = self.cu_q.tolist()
+            self.portions = [(n - (b - a), b - a) for n, a, b in zip(self.seq_lens.tolist(), cu, cu[1:])]
+        return self.portions
 
     def layer_splits(self, n_kv: int, chunk: int = 0) -> int:
         """Split-KV factor of one layer in a decode step, for families whose layers see contexts of their own length.
@@ -143,6 +152,7 @@ class CausalLM:
         from ..parallel.context import ParallelContext
 
         self.cfg = cfg
+        self.family = mixer_family(cfg.model_type)   # module of a family whose layers each name their mixer
         self.device = torch.device(device)
         self.dtype = dtype
         self.par = parallel or ParallelContext.single()
@@ -240,10 +250,8 @@ class CausalLM:
             from .muse_glimmer import block_forward as muse_block
 
             return muse_block(self, li, lw, h, batch, kv), None
-        if lw.block_kind == "nidozen":
-            from .nidozen import block_forward as nidozen_block
-
-            return nidozen_block(self, li, lw, h, batch, kv), None
+        if self.family is not None:
+            return self.family.block_forward(self, li, lw, h, batch, kv), None
         if lw.block_kind:
             from .nemotron_h import block_forward
 
@@ -327,10 +335,8 @@ class CausalLM:
         """Runs this shard's layers. Returns (h, ssq) - ssq is None unless the next consumer folds its norm."""
         fused = bool(self.layers) and self.layers[0].fold_attn and batch.token_ids.shape[0] <= self.FUSED_NORM_MAX_TOKENS
         ssq = None
-        if self.cfg.model_type == "nidozen" and batch.hidden_in is None:
-            from .nidozen import enter
-
-            h = enter(self, batch)
+        if self.family is not None and batch.hidden_in is None:
+            h = self.family.enter(self, batch)
         elif self.par.owns_embedding() and batch.hidden_in is None:
             if fused:
                 h, ssq = ops.embedding(batch.token_ids, self.embed, 0, self.cfg.embedding_scale, want_ssq=True)
@@ -384,10 +390,8 @@ class CausalLM:
             h = h.index_select(0, rows)
             ssq = ssq.index_select(0, rows) if ssq is not None else None
         h = h.contiguous()
-        if self.cfg.model_type == "nidozen":
-            from .nidozen import final_norm
-
-            h, ssq = final_norm(self, h), None
+        if self.family is not None:
+            h, ssq = self.family.final_norm(self, h), None
         elif self.head_folded:
             if ssq is None or h.shape[0] > self.FUSED_NORM_MAX_TOKENS:
                 h, _ = ops.rmsnorm(h, self._ones(h.shape[1]), self.cfg.rms_norm_eps)
@@ -527,10 +531,8 @@ def build_from_tensors(cfg: ModelConfig, get: Callable[[str], torch.Tensor], has
     model = CausalLM(cfg, device, dtype, parallel)
     par = model.par
     tp, r = par.tp_size, par.tp_rank
-    if cfg.model_type == "nidozen":
-        from .nidozen import canonical_access
-
-        get, has = canonical_access(get, has)
+    if model.family is not None:
+        get, has = model.family.canonical_access(get, has)
 
     def up(t, dt=None):
         return t.to(device=model.device, dtype=dt or dtype).contiguous()
@@ -554,13 +556,12 @@ def build_from_tensors(cfg: ModelConfig, get: Callable[[str], torch.Tensor], has
 
         build_gemma4(model, cfg, get, has, up)
         return model
-    if cfg.model_type == "nidozen":
-        from .nidozen import build as build_nidozen
-
+    if model.family is not None:
         if quantizer is not None or on_layer is not None:
-            raise NotImplementedError("Nidozen weights are dense and resident: no quantisation or host residency")
-        model.final_norm = model.final_norm.reshape(1)
-        build_nidozen(model, cfg, get, has, up)
+            raise NotImplementedError(f"{cfg.model_type} weights are dense and resident: no quantisation or host residency")
+        if par.tp_size > 1 or par.pp_size > 1 or par.ep_size > 1:
+            raise NotImplementedError(f"{cfg.model_type} runs on one device: the parallel forms are not built for it")
+        model.family.build(model, cfg, get, has, up)
         return model
     if cfg.model_type == "muse_glimmer":
         from .muse_glimmer import build as build_muse
@@ -707,12 +708,11 @@ def random_state(cfg: ModelConfig, seed: int = 0, std: float = 0.02, dtype=torch
     import zlib
 
     out: dict[str, torch.Tensor] = {}
-    if cfg.model_type == "nidozen":
-        from .nidozen import random_tensor, tensor_shapes
-
-        for name, shape in tensor_shapes(cfg).items():
+    family = mixer_family(cfg.model_type)
+    if family is not None:
+        for name, shape in family.tensor_shapes(cfg).items():
             g = torch.Generator(device="cpu").manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
-            out[name] = random_tensor(name, shape, g, std).to(dtype=dtype, device=device)
+            out[name] = family.random_tensor(name, shape, g, std).to(dtype=dtype, device=device)
         return out
 
     def mat(name, *shape):
@@ -813,14 +813,13 @@ def build_random(cfg: ModelConfig, device, dtype, seed: int = 0, parallel=None, 
     import zlib
 
     dev = torch.device(device)
-    if cfg.model_type == "nidozen":
-        from .nidozen import random_tensor, tensor_shapes
-
-        shapes = tensor_shapes(cfg)
+    family = mixer_family(cfg.model_type)
+    if family is not None:
+        shapes = family.tensor_shapes(cfg)
 
         def draw(name: str) -> torch.Tensor:
             g = torch.Generator(device=dev).manual_seed((seed * 1000003 + zlib.crc32(name.encode())) & 0x7FFFFFFFFFFF)
-            return random_tensor(name, shapes[name], g, std, dev).to(dtype)
+            return family.random_tensor(name, shapes[name], g, std, dev).to(dtype)
 
         return build_from_tensors(cfg, draw, shapes.__contains__, device, dtype, parallel)
 

@@ -79,6 +79,21 @@ class MoEBlock:
         return moe_ops.route(logits.contiguous(), cfg.num_experts_per_tok, cfg.router_scoring, cfg.norm_topk_prob,
                              cfg.routed_scaling_factor, self.router_bias, cfg.n_group, cfg.topk_group)
 
+    def routed_rows(self, x, logits):
+        """Outputs of the routed experts, uncombined (:class:`ops.moe.RoutedRows`), for families that add them to the stream
+        together with the other sublayer. ``logits`` [T, E] fp32: rows of the router projection. Single rank, no shared expert."""
+        self.stats["calls"] += 1
+        c = self.cfg
+        args = (c.num_experts_per_tok, c.router_scoring, c.norm_topk_prob, c.routed_scaling_factor, self.router_bias)
+        plan = xp = None
+        if (x.is_cuda and x.dtype == torch.bfloat16 and x.shape[0] <= 64 and x.shape[1] % 8 == 0 and self.w_down.shape[2] % 8 == 0
+                and moe_ops.kernel_routes(logits.shape[1], c.num_experts_per_tok, c.n_group)):
+            ids, w, plan, xp = moe_ops.route_plan_gather(logits, x, *args, self.e0, self.w_gate_up.shape[0], c.n_group, c.topk_group)
+        else:
+            ids, w = moe_ops.route(logits, *args, c.n_group, c.topk_group)
+        rows, pos = moe_ops.expert_rows(x, ids, self.w_gate_up, self.w_down, self.e0, c.swiglu_limit, self.act, plan, xp)
+        return moe_ops.RoutedRows(rows, pos, w)
+
     def observed_call(self, x, residual, observer):
         """Unfused pass that materialises what an activation observer is shown (routing ids, scores, weights, routed /
         shared / combined outputs); numerically the same block."""
@@ -125,14 +140,13 @@ class MoEBlock:
                                     act=self.act)
             return self.ep_ops.all_reduce(partial, residual=residual)
         plan = xp = None
-        if x.is_cuda and x.shape[0] <= 64 and self.cfg.n_group <= 1:
+        if x.is_cuda and x.shape[0] <= 64 and moe_ops.kernel_routes(self.n_experts, self.cfg.num_experts_per_tok, self.cfg.n_group):
             # decode-sized: routing, expert plan and row gather in one kernel
             cfg = self.cfg
             logits = self.router_logits(x)
             ids, w, plan, xp = moe_ops.route_plan_gather(logits.contiguous(), x, cfg.num_experts_per_tok, cfg.router_scoring,
                                                          cfg.norm_topk_prob, cfg.routed_scaling_factor, self.router_bias,
-                                                         self.e0,
-                                                         self.w_gate_up.shape[0])
+                                                         self.e0, self.w_gate_up.shape[0], cfg.n_group, cfg.topk_group)
         else:
             ids, w = self.route(x)
         extra = self._shared_out(x)

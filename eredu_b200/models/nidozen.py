@@ -140,8 +140,7 @@ def build(model, cfg, get, has, up) -> None:
     """Fill ``model.layers`` (called by the generic loader after the embedding, final norm and head)."""
     from .llama import LayerWeights
 
-    if model.par.tp_size > 1 or model.par.pp_size > 1:
-        raise NotImplementedError("Nidozen runs on one device: tensor and pipeline parallelism are not built for it")
+    model.final_norm = model.final_norm.reshape(1)
     f32 = lambda n: up(get(n), torch.float32)                                          # noqa: E731
     opt = lambda n: get(n) if has(n) else None                                         # noqa: E731
 

@@ -164,7 +164,7 @@ def rmsnorm(x, weight, eps, residual=None, weight_offset=0.0):
 
 
 native.register("eredu_rms_residual", native.I, [native.P] * 5 + [native.I] * 4 + [native.F, native.P])
-native.register("eredu_embedding_stream", native.I, [native.P] * 4 + [native.I] * 4 + [native.P])
+native.register("eredu_embedding_stream", native.I, [native.P] * 4 + [native.I] * 4 + [native.F, native.P])
 native.register("eredu_qkv_prepare", native.I, [native.P] * 9 + [native.I] * 10 + [native.F, native.P])
 
 
@@ -196,20 +196,67 @@ def rms_residual(y, weight, eps, residual=None, act_dtype=None):
     return x, act
 
 
-def embedding_stream(ids, table):
-    """Rows of ``table`` as the start of an fp32 residual stream: (fp32 rows, rows in the table's dtype)."""
+def embedding_stream(ids, table, scale=1.0, want_act=True):
+    """Rows of ``table`` times ``scale`` as the start of an fp32 residual stream: (fp32 rows, rows in the table's dtype or None)."""
     if not table.is_cuda:
-        act = table[ids.long()]
-        return act.float(), act
+        x = table[ids.long()].float() * scale
+        return x, (x.to(table.dtype) if want_act else None)
     assert ids.dtype == torch.int32 and table.is_contiguous()
     M, W = ids.shape[0], table.shape[1]
     x = torch.empty((M, W), dtype=torch.float32, device=table.device)
     fp32 = table.dtype == torch.float32
-    act = x if fp32 else torch.empty((M, W), dtype=table.dtype, device=table.device)
+    act = x if fp32 else (torch.empty((M, W), dtype=table.dtype, device=table.device) if want_act else None)
     code = lib().eredu_embedding_stream(ptr(ids), ptr(table), ptr(x), None if fp32 else ptr(act), M, W, table.shape[0],
-                                        1 if fp32 else 0, stream_ptr(table.device))
+                                        1 if fp32 else 0, scale, stream_ptr(table.device))
     check(code, "eredu_embedding_stream")
     return x, act
+
+
+native.register("eredu_residual_norm", native.I, [native.P] * 9 + [native.I] * 6 + [native.F, native.P])
+
+
+def residual_norm_ref(x, y=None, routed=None, weight=None, bias=None, eps=1e-5, act_dtype=None, center=True):
+    out = x.float()
+    if y is not None:
+        out = out + y.float()
+    if routed is not None:
+        out = out + routed.summed()
+    if weight is None:
+        return out, None
+    n = out - out.mean(-1, keepdim=True) if center else out
+    n = n * torch.rsqrt(n.square().mean(-1, keepdim=True) + eps) * weight.float()
+    return out, (n if bias is None else n + bias.float()).to(act_dtype or x.dtype)
+
+
+def residual_norm(x, y=None, routed=None, weight=None, bias=None, eps=1e-5, act_dtype=None, center=True):
+    """What a layer's sublayers add to the fp32 stream and the norm of the sum in front of the next layer, in one launch:
+    ``x' = x + y + sum_k w_k rows_k`` with a sublayer's output ``y`` and the expert rows of ``routed`` (:class:`ops.moe.RoutedRows`)
+    in the compute dtype, both optional; ``act = weight * (x' - mean) / sqrt(var + eps) + bias`` in ``act_dtype`` (``center=False``:
+    RMSNorm; ``bias`` optional; no ``weight``: no norm). Returns (x', act); x' is x itself when nothing is added."""
+    if not x.is_cuda:
+        return residual_norm_ref(x, y, routed, weight, bias, eps, act_dtype, center)
+    M, W = x.shape
+    act_dtype = act_dtype or torch.bfloat16
+    assert x.dtype == torch.float32 and x.is_contiguous() and act_dtype in (torch.bfloat16, torch.float32)
+    assert y is None or (y.dtype == act_dtype and y.is_contiguous() and y.shape == x.shape)
+    assert weight is None or (weight.dtype == torch.float32 and weight.numel() == W)
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == W)
+    rows = pos = w = None
+    k = 0
+    if routed is not None:
+        rows, pos, w = routed.rows, routed.route_pos, routed.weights
+        k = w.shape[1]
+        assert rows.dtype == act_dtype and rows.is_contiguous() and rows.shape[1] == W and w.shape[0] == M and w.dtype == torch.float32
+    adds = y is not None or routed is not None
+    out = torch.empty_like(x) if adds else x
+    act = torch.empty((M, W), dtype=act_dtype, device=x.device) if weight is not None else None
+    if M == 0 or (not adds and weight is None):
+        return out, act
+    code = lib().eredu_residual_norm(ptr(x), ptr(y), ptr(rows), ptr(pos), ptr(w), ptr(weight), ptr(bias), ptr(out) if adds else None,
+                                     ptr(act), M, W, k, 1 if act_dtype == torch.float32 else 0, 1 if center else 0,
+                                     1 if W % 4 == 0 else 0, eps, stream_ptr(x.device))
+    check(code, "eredu_residual_norm")
+    return out, act
 
 
 # ------------------------------------------------------------------------------------------ rope + kv append
@@ -381,7 +428,7 @@ def attention_ref(q, k_cache, v_cache, block_table, seq_lens, q_lens, scale, win
 TC_PREFILL = _environ.get("EREDU_TC_PREFILL", "1") != "0"      # head size 64 / 128: the tcgen05 kernel (else the mma.sync one)
 
 
-native.register("eredu_attn_simt", native.I, [native.P] * 8 + [native.I] * 11 + [native.F, native.P])
+native.register("eredu_attn_simt", native.I, [native.P] * 8 + [native.I] * 12 + [native.F, native.P])
 
 
 def _attention_simt(q, k_cache, v_cache, block_table, seq_lens, cu_q, q_per_seq, max_q_len, scale, window, chunk, sinks):
@@ -392,7 +439,7 @@ def _attention_simt(q, k_cache, v_cache, block_table, seq_lens, cu_q, q_per_seq,
         return out
     code = lib().eredu_attn_simt(ptr(q), ptr(k_cache), ptr(v_cache), ptr(out), ptr(block_table), ptr(seq_lens), ptr(cu_q),
                                  ptr(sinks), seq_lens.shape[0], q_per_seq, max_q_len, block_table.stride(0), q.shape[1],
-                                 k_cache.shape[1], q.shape[2], v_cache.shape[3], int(window), int(chunk),
+                                 k_cache.shape[1], q.shape[2], v_cache.shape[3], v_cache.shape[3], int(window), int(chunk),
                                  1 if q.dtype == torch.float32 else 0, scale, stream_ptr(q.device))
     check(code, "eredu_attn_simt")
     return out

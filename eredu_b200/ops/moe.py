@@ -9,14 +9,15 @@ import torch
 import torch.nn.functional as F
 
 from . import native
-from .core import _sm_count, linear
+from .core import _sm_count, linear, residual_norm
 from .native import I, P, check, lib, ptr, status_word, stream_ptr
 
-native.register("eredu_moe_route", I, [P, P, P, P, I, I, I, I, I, native.F, P])
+native.register("eredu_moe_route", I, [P, I, P, P, P, I, I, I, I, I, native.F, I, I, P])
 native.register("eredu_moe_plan", I, [P, I, I, I, I, I, P, P, P, P, I, P, P])
 native.register("eredu_moe_gather", I, [P, P, P, P, I, I, P])
 native.register("eredu_moe_combine", I, [P, P, P, P, P, P, I, I, I, P])
-native.register("eredu_moe_route_plan_gather", I, [P, P, P, P, I, I, I, I, I, native.F, I, I, I, P, P, P, P, I, P, P, P, I, P])
+native.register("eredu_moe_route_plan_gather", I, [P, I, P, P, P, I, I, I, I, I, native.F, I, I, I, I, I, P, P, P, P, I, P, P, P, I, P])
+native.register("eredu_gemm_simt_grouped", I, [P, P, P, P, I, P, I, I, I, I, I, I, I, P])
 native.register("eredu_moe_combine_ar", I, [P, P, P, P, P, P, I, I, I, P, P, P])
 native.register("eredu_gemm_bf16_grouped", I, [P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, I, I, P, P, I, I, native.F, P])
 
@@ -63,18 +64,23 @@ def route_ref(logits, k, scoring="softmax", renorm=True, scale=1.0, sel_bias=Non
     return ids.to(torch.int32), (w * scale).float()
 
 
+def kernel_routes(experts: int, k: int, n_group: int = 1) -> bool:
+    """Router sizes the kernel takes: a warp holds a token's experts in registers and a group's score per lane."""
+    return experts <= 512 and k <= 32 and n_group <= 32
+
+
 def route(logits, k, scoring="softmax", renorm=True, scale=1.0, sel_bias=None, n_group=1, topk_group=1, norm_eps=0.0,
           routing_indices=None):
-    """Router logits [T, E] fp32 -> (ids [T, k] int32, weights [T, k] fp32). Group-limited selection, a renormalisation
-    epsilon and table-driven (hash) routing run as tensor operations; the plain forms use the routing kernel."""
-    if not logits.is_cuda or n_group > 1 or topk_group > 1 or norm_eps != 0.0 or routing_indices is not None:
+    """Router logits [T, E] fp32 (rows may be part of wider ones) -> (ids [T, k] int32, weights [T, k] fp32). A
+    renormalisation epsilon and table-driven (hash) routing run as tensor operations; the other forms use the routing kernel."""
+    if not logits.is_cuda or norm_eps != 0.0 or routing_indices is not None or not kernel_routes(logits.shape[1], k, n_group):
         return route_ref(logits, k, scoring, renorm, scale, sel_bias, n_group, topk_group, norm_eps, routing_indices)
     T, E = logits.shape
-    assert logits.dtype == torch.float32 and logits.is_contiguous()
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and 0 < topk_group <= n_group and E % n_group == 0
     ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
     w = torch.empty((T, k), dtype=torch.float32, device=logits.device)
-    code = lib().eredu_moe_route(ptr(logits), ptr(sel_bias), ptr(ids), ptr(w), T, E, k, SCORING[scoring],
-                                 1 if renorm else 0, scale, stream_ptr(logits.device))
+    code = lib().eredu_moe_route(ptr(logits), logits.stride(0), ptr(sel_bias), ptr(ids), ptr(w), T, E, k, SCORING[scoring],
+                                 1 if renorm else 0, scale, n_group, topk_group, stream_ptr(logits.device))
     check(code, "eredu_moe_route")
     return ids, w
 
@@ -152,9 +158,10 @@ def pick_tile(expected_rows_per_expert: float) -> int:
     return 128
 
 
-def route_plan_gather(logits, x, k, scoring, renorm, scale, sel_bias, e0, n_local):
+def route_plan_gather(logits, x, k, scoring, renorm, scale, sel_bias, e0, n_local, n_group=1, topk_group=1):
     """Decode-sized steps (<= 64 tokens): routing, the local experts' plan and the row gather in one kernel.
     Returns (ids, weights, plan, xp) for :func:`experts_forward`."""
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
     T, E = logits.shape
     H = x.shape[1]
     routes = T * k
@@ -166,8 +173,8 @@ def route_plan_gather(logits, x, k, scoring, renorm, scale, sel_bias, e0, n_loca
     xp = torch.empty((routes, H), dtype=x.dtype, device=dev)
     # one CTA copies the rows itself only when there are few of them (expected local routes <= 64)
     inline_gather = routes * n_local <= 64 * E
-    code = lib().eredu_moe_route_plan_gather(ptr(logits), ptr(sel_bias), ptr(ids), ptr(w), T, E, k, SCORING[scoring],
-                                             1 if renorm else 0, scale, e0, e0 + n_local, tile, ptr(plan.seg),
+    code = lib().eredu_moe_route_plan_gather(ptr(logits), logits.stride(0), ptr(sel_bias), ptr(ids), ptr(w), T, E, k, SCORING[scoring],
+                                             1 if renorm else 0, scale, n_group, topk_group, e0, e0 + n_local, tile, ptr(plan.seg),
                                              ptr(plan.route_pos), ptr(plan.row_token), ptr(plan.work), plan.n_work,
                                              ptr(plan.counts), ptr(x), ptr(xp) if inline_gather else None, H, stream_ptr(dev))
     check(code, "eredu_moe_route_plan_gather")
@@ -175,6 +182,60 @@ def route_plan_gather(logits, x, k, scoring, renorm, scale, sel_bias, e0, n_loca
         check(lib().eredu_moe_gather(ptr(x), ptr(plan.row_token), ptr(plan.counts), ptr(xp), routes, H, stream_ptr(dev)),
               "eredu_moe_gather")
     return ids, w, plan, xp
+
+
+class RoutedRows:
+    """Outputs of the routed experts before they are combined: ``rows`` in some order, ``route_pos`` [T * k] the row of every
+    (token, slot) route (negative: none), ``weights`` [T, k]."""
+
+    def __init__(self, rows, route_pos, weights):
+        self.rows, self.route_pos, self.weights = rows, route_pos, weights
+
+    def summed(self):
+        """fp32 [T, H]: the weighted sum over each token's routes (reference; kernels fold it into what follows)."""
+        T, k = self.weights.shape
+        pos = self.route_pos.view(T, k).long()
+        y = self.rows[pos.clamp_min(0)].float() * (self.weights * (pos >= 0))[..., None]
+        return y.sum(1)
+
+
+def expert_rows_ref(x, ids, w_gate_up, w_down, e0=0, limit=0.0, act="swiglu"):
+    """[T * k, H]: the output of every route's expert, routes in order."""
+    T, k = ids.shape
+    rows = torch.zeros((T * k, x.shape[1]), dtype=x.dtype, device=x.device)
+    one = torch.ones((T, 1), dtype=torch.float32, device=x.device)
+    for slot in range(k):
+        rows[slot::k] = experts_ref(x, ids[:, slot:slot + 1], one, w_gate_up, w_down, e0, limit, act=act).to(x.dtype)
+    return rows
+
+
+def expert_rows(x, ids, w_gate_up, w_down, e0=0, limit=0.0, act="swiglu", plan=None, xp=None):
+    """Outputs of the local experts for every route, uncombined: (rows, route_pos). bf16 rows that a TMA descriptor can describe
+    run the grouped tcgen05 GEMMs; fp32 and every other width run grouped GEMMs on the CUDA cores, which read the token rows
+    through the plan (``limit`` 0, SwiGLU)."""
+    if not x.is_cuda:
+        return expert_rows_ref(x, ids, w_gate_up, w_down, e0, limit, act), torch.arange(ids.numel(), dtype=torch.int32)
+    E_local, two_i, H = w_gate_up.shape
+    inter = two_i // 2
+    if x.dtype == torch.bfloat16 and H % 8 == 0 and inter % 8 == 0:
+        if plan is None:
+            routes = ids.numel()
+            plan = ExpertPlan(ids, ids.shape[1], e0, e0 + E_local, pick_tile(routes / max(1, E_local)), routes)
+            xp = torch.empty((routes, H), dtype=x.dtype, device=x.device)
+            check(lib().eredu_moe_gather(ptr(x), ptr(plan.row_token), ptr(plan.counts), ptr(xp), routes, H, stream_ptr(x.device)),
+                  "eredu_moe_gather")
+        return experts_forward(x, ids, None, w_gate_up, w_down, e0, limit=limit, plan=plan, xp=xp, act=act, rows_only=True,
+                               rows_cap=plan.rows_cap), plan.route_pos
+    assert act == "swiglu" and limit == 0.0 and x.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous()
+    routes, fp32 = ids.numel(), 1 if x.dtype == torch.float32 else 0
+    plan = ExpertPlan(ids, ids.shape[1], e0, e0 + E_local, 64, routes)
+    mid = torch.empty((routes, inter), dtype=x.dtype, device=x.device)
+    y = torch.empty((routes, H), dtype=x.dtype, device=x.device)
+    for src, w, dst, index, n, kk, per, dual in ((x, w_gate_up, mid, plan.row_token, inter, H, two_i, 1), (mid, w_down, y, None, H, inter, H, 0)):
+        code = lib().eredu_gemm_simt_grouped(ptr(src), ptr(w), ptr(dst), ptr(plan.work), plan.n_work, ptr(index), n, kk, kk, n, per, dual,
+                                             fp32, stream_ptr(x.device))
+        check(code, "eredu_gemm_simt_grouped")
+    return y, plan.route_pos
 
 
 def experts_forward(x, ids, weights, w_gate_up, w_down, e0=0, residual=None, extra=None, limit=0.0, rows_cap=None,
@@ -194,6 +255,11 @@ def experts_forward(x, ids, weights, w_gate_up, w_down, e0=0, residual=None, ext
     T, H = x.shape
     k = ids.shape[1] if ids is not None else 1
     E_local, two_i, _ = w_gate_up.shape
+    if x.dtype == torch.float32:         # the CUDA-core experts; the tensor-core path below is bf16
+        rows, pos = expert_rows(x, ids, w_gate_up, w_down, e0, limit, act)
+        assert comm is None and gu_bias is None and down_bias is None and not rows_only
+        out = torch.zeros_like(x) if residual is None else residual.contiguous()
+        return residual_norm(out, extra, RoutedRows(rows, pos, weights), act_dtype=x.dtype)[0]
     ungated = act in UNGATED
     inter = two_i if ungated else two_i // 2
     routes = T * k

@@ -347,3 +347,89 @@ def gla_attention(proj, a2, a2_b, norm_w, state, heads, dk, dv, tau, eps, batch,
                                 stream_ptr(proj.device))
     check(code, "eredu_gla_scan")
     return out
+
+
+native.register("eredu_mlstm", I, [P] * 10 + [I] * 13 + [F, F, P])
+native.register("eredu_mlstm_scratch_bytes", native.L, [I] * 7)
+
+
+def mlstm_state_views(state, heads, dk, dv):
+    """One sequence's state [>= H (dk dv + dk + 1)] as (memory [H, dk, dv], normaliser [H, dk], running maximum [H])."""
+    a, b = heads * dk * dv, heads * dk
+    return state[:a].view(heads, dk, dv), state[a:a + b].view(heads, dk), state[a + b:a + b + heads]
+
+
+def mlstm_scan_ref(q, k, v, i, f, state):
+    """q, k [T, H, dk], v [T, H, dv], log gates i, f [T, H] (fp32); state (S, n, m). Returns (o [T, H, dv], state)."""
+    S, n, m = (t.clone() for t in state)
+    out = []
+    for t in range(q.shape[0]):
+        new = torch.maximum(f[t] + m, i[t])
+        keep, take = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
+        kt = k[t] * take[:, None]
+        S = S * keep[:, None, None] + kt[:, :, None] * v[t][:, None, :]
+        n = n * keep[:, None] + kt
+        m = new
+        size = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + MLSTM_EPS
+        out.append(torch.einsum("hdv,hd->hv", S, q[t]) / size[:, None])
+    return torch.stack(out), (S, n, m)
+
+
+MLSTM_EPS = 1e-6        # added to the normaliser
+
+
+def mlstm_ref(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_slot):
+    M, qk, vw = proj.shape[0], heads * dk, heads * dv
+    x = proj.float()
+    q, k = x[:, :qk].view(M, heads, dk) * dk ** -0.5, x[:, qk:2 * qk].view(M, heads, dk)
+    v, g = x[:, 2 * qk:2 * qk + vw].view(M, heads, dv), x[:, 2 * qk + vw:2 * qk + 2 * vw]
+    z = cap * torch.tanh(gates.float() / cap)
+    i, f = z[:, :heads], torch.nn.functional.logsigmoid(z[:, heads:2 * heads])
+    out = torch.zeros((M, vw), dtype=proj.dtype, device=proj.device)
+    bounds = _sequences(batch)
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(batch.slots[r0]) < 0:
+            continue
+        views = mlstm_state_views(state[int(page_to_slot[int(batch.block_table[b, 0])])], heads, dk, dv)
+        o, new = mlstm_scan_ref(q[r0:r1], k[r0:r1], v[r0:r1], i[r0:r1], f[r0:r1], views)
+        for old, t in zip(views, new):
+            old.copy_(t)
+        o = (o * torch.rsqrt(o.square().mean(-1, keepdim=True) + eps)).reshape(r1 - r0, vw) * norm_w
+        out[r0:r1] = (o * torch.sigmoid(g[r0:r1])).to(out.dtype)
+    return out
+
+
+def mlstm(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_slot):
+    """Matrix memory with exponential gates (mLSTM) over ``proj`` [M, >= 2 H dk + 2 H dv] = [q | k | v | output gate] and ``gates``
+    fp32 [M, >= 2 H] = [input | forget] pre-activations, soft-capped by ``cap``. Per head, with ``i`` the capped input gate, ``f`` the
+    log-sigmoid of the capped forget gate and a running maximum m: ``m' = max(f + m, i)``, ``S' = e^(f + m - m') S + e^(i - m') k v^T``,
+    ``n'`` likewise with k alone, ``o = S'^T q / (max(|n'.q|, e^-m') + 1e-6)``, q scaled by dk^-1/2. Each head's o is RMS-normed, times
+    ``norm_w`` [H dv] and the sigmoid of the output gate. ``state`` fp32 [slots, >= H (dk dv + dk + 1)]: S, n, m of all heads
+    (:func:`mlstm_state_views`), zero for a new sequence, updated in place. Returns [M, H dv]."""
+    if not proj.is_cuda:
+        return mlstm_ref(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_slot)
+    M = proj.shape[0]
+    assert proj.stride(1) == 1 and gates.stride(1) == 1 and gates.dtype == torch.float32 and norm_w.dtype == torch.float32
+    assert state.is_contiguous() and state.dtype == torch.float32 and state.shape[1] >= heads * (dk * dv + dk + 1)
+    out = torch.empty((M, heads * dv), dtype=proj.dtype, device=proj.device)
+    if M == 0:
+        return out
+    batch_size = batch.block_table.shape[0]
+    rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
+    scratch = None
+    if proj.dtype == torch.bfloat16 and proj.data_ptr() % 16 == 0 and proj.stride(0) % 8 == 0:
+        size = int(lib().eredu_mlstm_scratch_bytes(heads, dk, dv, M, batch_size, rows, state.shape[1]))
+        if size:
+            scratch = torch.empty(size, dtype=torch.uint8, device=proj.device)
+    code = lib().eredu_mlstm(ptr(proj), ptr(gates), ptr(norm_w), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table),
+                             ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv,
+                             proj.stride(0), gates.stride(0), state.shape[1], M, batch_size, batch.q_per_seq, rows,
+                             batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, native_sms(proj.device), cap, eps,
+                             stream_ptr(proj.device))
+    check(code, "eredu_mlstm")
+    return out
+
+
+def native_sms(device) -> int:
+    return torch.cuda.get_device_properties(device).multi_processor_count

@@ -405,7 +405,8 @@ class Engine:
             splits = ops.decode_splits(len(seqs), self.model.n_kv_local, longest, self.sm_count) if self.cuda else 1
             return ForwardBatch(**common, is_prefill=False, q_per_seq=1, max_kv_len=longest, splits=splits)
         cu = np.concatenate(([0], np.cumsum(counts))).astype(np.int32)
-        return ForwardBatch(**common, is_prefill=True, cu_q=self._t(cu, torch.int32), max_q_len=max(counts))
+        return ForwardBatch(**common, is_prefill=True, cu_q=self._t(cu, torch.int32), max_q_len=max(counts),
+                            portions=[(s.kv_len, n) for s, n in zip(seqs, counts)])
 
     @torch.no_grad()
     def forward_tokens(self, entries) -> torch.Tensor:
@@ -456,7 +457,7 @@ class Engine:
             positions=self._t(p.astype(np.int32), torch.int32),
             slots=self._t(pages[p // PAGE] * PAGE + (p % PAGE), torch.int64),
             block_table=self._block_table([seq]), seq_lens=self._t(np.asarray([seq.kv_len + n], dtype=np.int32), torch.int32),
-            is_prefill=True, cu_q=self._t(np.asarray([0, n], dtype=np.int32), torch.int32), max_q_len=n,
+            is_prefill=True, cu_q=self._t(np.asarray([0, n], dtype=np.int32), torch.int32), max_q_len=n, portions=[(seq.kv_len, n)],
             logit_rows=self._t(np.asarray([n - 1], dtype=np.int64), torch.int64))
         logits = self.model.forward(batch, self.kv)
         seq.kv_len += n

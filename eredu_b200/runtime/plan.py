@@ -18,11 +18,11 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Optional
 
-from ..models.config import DENSE_TYPES, MOE_TYPES, ModelConfig
+from ..models.config import DENSE_TYPES, MIXER_FAMILIES, MOE_TYPES, ModelConfig, mixer_family
 
 EXECUTION_PLAN_SCHEMA_VERSION = 2
 DEFAULT_MAX_MAPPED_SHARDS = 4
-SUPPORTED_TYPES = DENSE_TYPES | {"qwen3_moe", "mixtral", "gpt_oss", "lfm2_moe", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "nemotron_h", "deepseek_v3", "deepseek_v4", "inkling_mm_model", "muse_glimmer", "kimi_linear", "gemma4", "nidozen"}
+SUPPORTED_TYPES = DENSE_TYPES | {"qwen3_moe", "mixtral", "gpt_oss", "lfm2_moe", "qwen3_next", "qwen3_5", "qwen3_5_text", "qwen3_5_moe", "qwen3_5_moe_text", "nemotron_h", "deepseek_v3", "deepseek_v4", "inkling_mm_model", "muse_glimmer", "kimi_linear", "gemma4"} | set(MIXER_FAMILIES)
 
 
 # ---------------------------------------------------------------------------------------------- inspection
@@ -80,10 +80,8 @@ def required_tensors(cfg: ModelConfig) -> list[tuple]:
     if cfg.model_type == "inkling_mm_model":
         return [("model.embed_tokens.weight", "model.llm.embed.weight"), ("model.norm.weight", "model.llm.norm.weight"),
                 ("model.layers.0.self_attn.r_proj.weight", "model.llm.layers.0.attn.wr_du.weight")]
-    if cfg.model_type == "nidozen":
-        from ..models.nidozen import tensor_shapes
-
-        return [(n,) for n in tensor_shapes(cfg)]
+    if mixer_family(cfg.model_type) is not None:
+        return [(n,) for n in mixer_family(cfg.model_type).tensor_shapes(cfg)]
     p = "model.layers.0."
     kind = cfg.layer_types[0] if cfg.layer_types else "full_attention"
     if cfg.model_type == "nemotron_h":
@@ -268,11 +266,11 @@ def _family_profile(cfg: ModelConfig, weight_bytes, b: int):
         # per-layer geometry: pages of the layers that keep keys and values, fp32 states of the recurrent ones
         kv = [cfg.layer_kv_dims(li) for li in range(L) if cfg.layer_has_kv(li)]
         state = sum(math.prod(cfg.layer_state_shape(li)) * 4 for li in range(L) if cfg.layer_state_shape(li) is not None)
-        from ..models.nidozen import tensor_shapes
-
-        wb = weight_bytes if weight_bytes is not None else sum(math.prod(s) for s in tensor_shapes(cfg).values()) * 2
+        total = sum(math.prod(s) for s in mixer_family(cfg.model_type).tensor_shapes(cfg).values()) * 2
+        wb = weight_bytes if weight_bytes is not None else total
+        experts = sum(3 * H * m.moe.num_experts * m.moe.moe_intermediate_size * 2 for m in cfg.mixers if m.moe is not None)
         return ModelResourceProfile(int(wb), int(sum(n * (dk + dv) for n, dk, dv in kv) * b), max(1, len(kv)),
-                                    state_bytes_per_sequence=int(state))
+                                    expert_bytes=int(wb * (experts / total)), state_bytes_per_sequence=int(state))
     if cfg.model_type == "gemma4":
         from ..models.gemma4 import geometry
 

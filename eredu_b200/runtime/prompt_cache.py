@@ -323,8 +323,8 @@ def save_prompt_cache(engine, seq, directory, checkpoint_fingerprint: str, prefi
             continue
         k_pool, v_pool = engine.kv.layer(li)
         # [pages, n_kv, PAGE, D] -> [n_kv, pages * PAGE, D]
-        k = k_pool[pages].permute(1, 0, 2, 3).reshape(k_pool.shape[1], -1, k_pool.shape[3])[:, :n]
-        v = v_pool[pages].permute(1, 0, 2, 3).reshape(v_pool.shape[1], -1, v_pool.shape[3])[:, :n]
+        k = k_pool[pages].permute(1, 0, 2, 3).reshape(k_pool.shape[1], pages.shape[0] * PAGE, k_pool.shape[3])[:, :n]
+        v = v_pool[pages].permute(1, 0, 2, 3).reshape(v_pool.shape[1], pages.shape[0] * PAGE, v_pool.shape[3])[:, :n]
         shard = f"layer-{li:04d}.safetensors"
         items = []
         for start in range(0, n, block_tokens):
