@@ -82,8 +82,8 @@ def timed(fn, reps: int) -> float:
     return e0.elapsed_time(e1) / reps
 
 
-def model_numbers(cfg: ModelConfig, steps: int, prefills=(2048, 8192), batches=(1, 32), context: int = 2048) -> dict:
-    model = random_model(cfg)
+def model_numbers(cfg: ModelConfig, steps: int, prefills=(2048, 8192), batches=(1, 32), context: int = 2048, build=random_model) -> dict:
+    model = build(cfg)
     eng = Engine(model, max_batch=max(batches), max_seq_len=max(max(prefills), context + steps + 64) + 16,
                  num_pages=max(batches) * ((context + steps + 64) // 16 + 2) + max(prefills) // 16 + 8, prefill_chunk=16384)
     g = torch.Generator().manual_seed(0)
