@@ -180,13 +180,13 @@ def kernel_numbers(size: str, T: int = 8192, Bn: int = 32, context: int = 2048, 
             return lambda: ops.latent_prepare(x[:, H * V:], Q, R, P, qn, kn, 1e-5, bt.positions, bt.slots, inv, c)
 
         hq, hk, hd = 16, 4, 128
-        hw, hinv = torch.ones(hd, device=DEV), torch.rand(hd // 2, device=DEV)
+        hw, gw, hinv = torch.ones(hq * hd, device=DEV), torch.ones(hk * hd, device=DEV), torch.rand(hd // 2, device=DEV)
 
         def like_prep(i):
             x, kc, vc = rnd(M, (hq + 2 * hk) * hd), rnd(pages, hk, 16, hd), rnd(pages, hk, 16, hd)
-            return lambda: ops.rope_kv(x, bt.positions, bt.slots, hinv, kc, vc, hq, hk, hd, q_norm_w=hw, k_norm_w=hw)
+            return lambda: ops.qkv_prepare(x, bt.positions, bt.slots, hinv, kc, vc, hq, hk, hd, hd, hw, gw, 1e-5)
 
-        add(f"{phase} latent_prepare", M * (Q + R + P) * 4, 0, prep, "rope_kv (per-head norms)", like_prep, M * (hq + 2 * hk) * hd * 4)
+        add(f"{phase} latent_prepare", M * (Q + R + P) * 4, 0, prep, "qkv_prepare (norms over whole projections)", like_prep, M * (hq + 2 * hk) * hd * 4)
 
         uk, uv, up = rnd(H, R, D, s=0.05), rnd(H, V, R, s=0.05), rnd(H * (D + V), R, s=0.05)
         sinks = torch.zeros(H, device=DEV)
@@ -228,11 +228,11 @@ def kernel_numbers(size: str, T: int = 8192, Bn: int = 32, context: int = 2048, 
 
             def attn(i):
                 qa, c, o = rnd(Bn, H, R + P), pool(), torch.empty(Bn, H, R, device=DEV, dtype=BF)
-                tile = 64 if H > 32 else (32 if H > 16 else 16)
-                sp = latent_ops.latent_splits(Bn, -(-H // tile), seen, 64 if tile == 16 else 32, 148)
+                tile, per_sm = latent_ops.latent_tile(H, R, P)
+                sp = latent_ops.latent_splits(Bn, -(-H // tile), seen, per_sm * 148)
                 return lambda: native.lib().eredu_latent_attn(qa.data_ptr(), c.data_ptr(), o.data_ptr(), bt.block_table.data_ptr(), bt.seq_lens.data_ptr(),
                                                               None, sinks.data_ptr(), Bn, 1, 1, bt.block_table.stride(0), H, R, P, tile, sp, WINDOW,
-                                                              (D + P) ** -0.5, native.stream_ptr(DEV))
+                                                              (D + P) ** -0.5, native.status_word(DEV).data_ptr(), native.stream_ptr(DEV))
 
             def like_attn(i):
                 q, kc, vc = rnd(Bn, 4 * hk, hd), rnd(pages, hk, 16, hd), rnd(pages, hk, 16, hd)

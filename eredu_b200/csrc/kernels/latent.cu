@@ -15,45 +15,112 @@ namespace eredu {
 
 using bf16 = __nv_bfloat16;
 
-// One CTA per token. proj row = [query latent (q_rank) | latent (rank) | key part (rot)].
-template <typename T>
+// Sums of two values over the block in one pass; `red` holds two floats per warp.
+__device__ __forceinline__ float2 block_sum2(float a, float b, float2* red) {
+  a = warp_sum_f32(a);
+  b = warp_sum_f32(b);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) {
+    t.x += red[w].x;
+    t.y += red[w].y;
+  }
+  return t;
+}
+
+// One CTA per token. proj row = [query latent (q_rank) | latent (rank) | key part (rot)]. NV > 0: rows and weights in groups of four,
+// both latents fit NV groups per thread and stay in registers; NV = 0: any width and alignment.
+template <typename T, int NV>
 __global__ void __launch_bounds__(256) latent_prepare_kernel(const T* __restrict__ proj, T* __restrict__ cq, T* __restrict__ cache,
                                                               const int* __restrict__ positions, const long long* __restrict__ slots,
                                                               const float* __restrict__ inv_freq, const float* __restrict__ q_norm_w,
                                                               const float* __restrict__ kv_norm_w, int ld, int q_rank, int rank, int rot,
                                                               float eps) {
-  __shared__ float red[8];
+  __shared__ float2 red[8];
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int m = blockIdx.x;
   const T* row = proj + static_cast<size_t>(m) * ld;
   const long long slot = slots[m];
-  float sq = 0.f, sk = 0.f;
-  for (int c = threadIdx.x; c < q_rank; c += 256) {
-    const float v = to_f32(row[c]);
-    sq += v * v;
-  }
-  for (int c = threadIdx.x; c < rank; c += 256) {
-    const float v = to_f32(row[q_rank + c]);
-    sk += v * v;
-  }
-  const float q_inv = 1.f / sqrtf(block_sum_f32(sq, red) / static_cast<float>(q_rank) + eps);
-  const float k_inv = 1.f / sqrtf(block_sum_f32(sk, red) / static_cast<float>(rank) + eps);
-  T* q = cq + static_cast<size_t>(m) * q_rank;
-  for (int c = threadIdx.x; c < q_rank; c += 256) q[c] = from_f32<T>(to_f32(row[c]) * q_inv * q_norm_w[c]);
-  if (slot < 0) return;
-  T* dst = cache + static_cast<size_t>(slot) * (rank + rot);
-  for (int c = threadIdx.x; c < rank; c += 256) dst[c] = from_f32<T>(to_f32(row[q_rank + c]) * k_inv * kv_norm_w[c]);
   const int half = rot >> 1;
-  const float pos = static_cast<float>(positions[m]);
-  for (int i = threadIdx.x; i < half; i += 256) {
-    float sn, cs;
-    sincosf(pos * inv_freq[i], &sn, &cs);
-    const float u = to_f32(row[q_rank + rank + i]), v = to_f32(row[q_rank + rank + half + i]);
-    dst[rank + i] = from_f32<T>(u * cs - v * sn);
-    dst[rank + half + i] = from_f32<T>(v * cs + u * sn);
+  float rot_u = 0.f, rot_v = 0.f, sn = 0.f, cs = 0.f;
+  if (static_cast<int>(threadIdx.x) < half) {                        // ahead of the norms, which do not touch this part
+    rot_u = to_f32(row[q_rank + rank + threadIdx.x]);
+    rot_v = to_f32(row[q_rank + rank + half + threadIdx.x]);
+    sincosf(static_cast<float>(positions[m]) * inv_freq[threadIdx.x], &sn, &cs);
   }
+  T* q = cq + static_cast<size_t>(m) * q_rank;
+  T* dst = cache + (slot >= 0 ? static_cast<size_t>(slot) * (rank + rot) : 0);
+  float sq = 0.f, sk = 0.f;
+  if constexpr (NV > 0) {
+    const int total = q_rank + rank;
+    float4 v[NV], w[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      v[i] = w[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < total) {
+        v[i] = load4(row + c);
+        w[i] = c < q_rank ? load4(q_norm_w + c) : load4(kv_norm_w + c - q_rank);
+        const float s = v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        if (c < q_rank) sq += s;
+        else sk += s;
+      }
+    }
+    const float2 t = block_sum2(sq, sk, red);
+    const float q_inv = 1.f / sqrtf(t.x / static_cast<float>(q_rank) + eps), k_inv = 1.f / sqrtf(t.y / static_cast<float>(rank) + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= total || (c >= q_rank && slot < 0)) continue;
+      const float inv = c < q_rank ? q_inv : k_inv;
+      store4(c < q_rank ? q + c : dst + c - q_rank, make_float4(v[i].x * inv * w[i].x, v[i].y * inv * w[i].y, v[i].z * inv * w[i].z, v[i].w * inv * w[i].w));
+    }
+  } else {
+    for (int c = threadIdx.x; c < q_rank; c += 256) {
+      const float v = to_f32(row[c]);
+      sq += v * v;
+    }
+    for (int c = threadIdx.x; c < rank; c += 256) {
+      const float v = to_f32(row[q_rank + c]);
+      sk += v * v;
+    }
+    const float2 t = block_sum2(sq, sk, red);
+    const float q_inv = 1.f / sqrtf(t.x / static_cast<float>(q_rank) + eps), k_inv = 1.f / sqrtf(t.y / static_cast<float>(rank) + eps);
+    for (int c = threadIdx.x; c < q_rank; c += 256) q[c] = from_f32<T>(to_f32(row[c]) * q_inv * q_norm_w[c]);
+    if (slot >= 0)
+      for (int c = threadIdx.x; c < rank; c += 256) dst[c] = from_f32<T>(to_f32(row[q_rank + c]) * k_inv * kv_norm_w[c]);
+  }
+  if (slot < 0) return;
+  for (int i = threadIdx.x; i < half; i += 256) {
+    if (i >= 256) {
+      rot_u = to_f32(row[q_rank + rank + i]);
+      rot_v = to_f32(row[q_rank + rank + half + i]);
+      sincosf(static_cast<float>(positions[m]) * inv_freq[i], &sn, &cs);
+    }
+    dst[rank + i] = from_f32<T>(rot_u * cs - rot_v * sn);
+    dst[rank + half + i] = from_f32<T>(rot_v * cs + rot_u * sn);
+  }
+}
+
+template <typename T>
+static cudaError_t launch_latent_prepare(const T* proj, T* cq, T* cache, const int* positions, const long long* slots, const float* inv_freq,
+                                         const float* q_norm_w, const float* kv_norm_w, int M, int ld, int q_rank, int rank, int rot,
+                                         float eps, cudaStream_t stream) {
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(cq) | reinterpret_cast<uintptr_t>(cache) |
+                         reinterpret_cast<uintptr_t>(q_norm_w) | reinterpret_cast<uintptr_t>(kv_norm_w);
+  const bool quads = (q_rank | rank | rot | ld) % 4 == 0 && (bits & 15) == 0;
+  const int need = quads ? ((q_rank + rank) / 4 + 255) / 256 : 0;
+#define ER_LP(NV_)                                                                                                                    \
+  launch_pdl(latent_prepare_kernel<T, NV_>, dim3(M), dim3(256), 0, stream, proj, cq, cache, positions, slots, inv_freq, q_norm_w, kv_norm_w, ld, \
+             q_rank, rank, rot, eps)
+  if (need == 1) return ER_LP(1);
+  if (need == 2) return ER_LP(2);
+  if (need == 3 || need == 4) return ER_LP(4);
+  return ER_LP(0);
+#undef ER_LP
 }
 
 // x [M, heads, width]: entries [off, off + rot) of every head are turned (pairs i, i + rot / 2) by the row's position.
@@ -288,13 +355,11 @@ extern "C" int eredu_latent_prepare(const void* proj, void* cq, void* cache, con
                                     int rank, int rot, int fp32, float eps, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (q_rank <= 0 || rank <= 0 || rot < 0 || rot % 2 != 0) return -1;
-  cudaError_t e;
-  if (fp32)
-    e = launch_pdl(latent_prepare_kernel<float>, dim3(M), dim3(256), 0, stream, static_cast<const float*>(proj), static_cast<float*>(cq),
-                   static_cast<float*>(cache), positions, slots, inv_freq, q_norm_w, kv_norm_w, ld, q_rank, rank, rot, eps);
-  else
-    e = launch_pdl(latent_prepare_kernel<bf16>, dim3(M), dim3(256), 0, stream, static_cast<const bf16*>(proj), static_cast<bf16*>(cq),
-                   static_cast<bf16*>(cache), positions, slots, inv_freq, q_norm_w, kv_norm_w, ld, q_rank, rank, rot, eps);
+  const cudaError_t e =
+      fp32 ? launch_latent_prepare(static_cast<const float*>(proj), static_cast<float*>(cq), static_cast<float*>(cache), positions, slots, inv_freq,
+                                   q_norm_w, kv_norm_w, M, ld, q_rank, rank, rot, eps, stream)
+           : launch_latent_prepare(static_cast<const bf16*>(proj), static_cast<bf16*>(cq), static_cast<bf16*>(cache), positions, slots, inv_freq,
+                                   q_norm_w, kv_norm_w, M, ld, q_rank, rank, rot, eps, stream);
   eredu_count_launches(1);
   return static_cast<int>(e);
 }

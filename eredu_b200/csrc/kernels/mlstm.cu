@@ -181,8 +181,11 @@ static cudaError_t launch_mlstm_step(const MlstmParams<T>& p, int slices, cudaSt
 template <typename T>
 static cudaError_t launch_mlstm_any(const MlstmParams<T>& p, int sms, cudaStream_t stream) {
   if (p.dv % 4 != 0 || p.stride % 4 != 0) return launch_mlstm_step<T, 1>(p, 1, stream);
-  int slices = 1;               // enough CTAs for the machine, at least 32 columns each
-  while (slices < 8 && p.H * p.seqs.B * slices < sms && p.dv % (slices * 8) == 0 && p.dv / (slices * 2) >= 32) slices *= 2;
+  // enough CTAs for the machine, at least 32 columns each; beyond one per SM, slices that balance the last wave
+  int slices = 1;
+  auto fits = [&](int columns) { return slices < 8 && p.dv % (slices * 8) == 0 && p.dv / (slices * 2) >= columns; };
+  while (fits(32) && p.H * p.seqs.B * slices < sms) slices *= 2;
+  while (fits(256) && p.H * p.seqs.B * slices < 8 * sms) slices *= 2;
   return launch_mlstm_step<T, 4>(p, slices, stream);
 }
 

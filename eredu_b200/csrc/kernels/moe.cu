@@ -18,14 +18,31 @@ namespace eredu {
 
 enum { SCORE_SOFTMAX = 0, SCORE_SIGMOID = 1, SCORE_SQRT_SOFTPLUS = 2, SCORE_TOPK_SOFTMAX = 3 };
 
-// One warp routes one token, up to 512 experts (16 per lane).
-__device__ __forceinline__ void route_token(const float* __restrict__ logits, const float* __restrict__ sel_bias,
-                                            int* __restrict__ ids, float* __restrict__ weights, int t, int lane, int E, int k,
-                                            int scoring, int renorm, float scale, int ld, int n_group, int keep_groups) {
-  constexpr int PER = 16;
-  float score[PER];   // value reported as the route weight
-  float select[PER];  // value used for selection (score + bias)
-  const float* row = logits + static_cast<size_t>(t) * ld;
+// Order-preserving map of a float to an unsigned key (larger float, larger key); 0 is below every float.
+__device__ __forceinline__ uint32_t order_key(float f) {
+  const uint32_t u = __float_as_uint(f);
+  return u ^ ((u >> 31) != 0u ? 0xffffffffu : 0x80000000u);
+}
+__device__ __forceinline__ float key_value(uint32_t k) { return __uint_as_float((k >> 31) != 0u ? k ^ 0x80000000u : ~k); }
+
+struct RouteParams {
+  const float* logits;     // [T, ld], E entries per row
+  const float* sel_bias;   // selection-only bias [E] or null
+  int* ids;                // [T, k]
+  float* weights;          // [T, k]
+  int ld, E, k, scoring, renorm, n_group, keep_groups;
+  float scale;
+};
+
+// One warp routes one token, up to 32 * PER experts (PER per lane; expert e belongs to lane e % 32). Ties go to the lowest expert.
+// `ids_out`: where the k chosen experts go (also to p.ids).
+template <int PER>
+__device__ __forceinline__ void route_token(const RouteParams& p, int t, int lane, int* ids_out) {
+  constexpr uint32_t kAll = 0xffffffffu;
+  float score[PER];     // value reported as the route weight
+  uint32_t key[PER];    // order of selection: 0 no expert, 1 retired or not eligible
+  const int E = p.E, k = p.k;
+  const float* row = p.logits + static_cast<size_t>(t) * p.ld;
   float mx = -INFINITY;
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
@@ -33,9 +50,9 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
     score[j] = e < E ? row[e] : -INFINITY;
     mx = fmaxf(mx, score[j]);
   }
+  if (p.scoring == SCORE_SOFTMAX) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-  if (scoring == SCORE_SOFTMAX) {
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(kAll, mx, o));
     float sum = 0.f;
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
@@ -43,14 +60,14 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
       sum += score[j];
     }
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(kAll, sum, o);
     const float inv = 1.f / sum;
 #pragma unroll
     for (int j = 0; j < PER; ++j) score[j] *= inv;
-  } else if (scoring == SCORE_SIGMOID) {
+  } else if (p.scoring == SCORE_SIGMOID) {
 #pragma unroll
     for (int j = 0; j < PER; ++j) score[j] = (lane + 32 * j < E) ? 1.f / (1.f + __expf(-score[j])) : -INFINITY;
-  } else if (scoring == SCORE_SQRT_SOFTPLUS) {
+  } else if (p.scoring == SCORE_SQRT_SOFTPLUS) {
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
       const float x = score[j];
@@ -60,107 +77,88 @@ __device__ __forceinline__ void route_token(const float* __restrict__ logits, co
 #pragma unroll
   for (int j = 0; j < PER; ++j) {
     const int e = lane + 32 * j;
-    select[j] = (e < E) ? score[j] + (sel_bias != nullptr ? sel_bias[e] : 0.f) : -INFINITY;
+    key[j] = e < E ? order_key(score[j] + (p.sel_bias != nullptr ? p.sel_bias[e] : 0.f)) : 0u;
   }
-  if (n_group > 1) {
+  if (p.n_group > 1) {
     // group-limited selection: experts form equal groups of neighbours, a group's score is the sum of its two largest, and only the
     // best keep_groups groups stay eligible. Lane g keeps the score of group g.
-    const int per = E / n_group;
-    float group_score = -INFINITY;
-    for (int gr = 0; gr < n_group; ++gr) {
-      float t1 = -INFINITY, t2 = -INFINITY;
+    const int per = E / p.n_group;
+    uint32_t group_key = 0u;
+    for (int gr = 0; gr < p.n_group; ++gr) {
+      uint32_t k1 = 0u, k2 = 0u;   // this lane's two largest of the group
 #pragma unroll
       for (int j = 0; j < PER; ++j) {
         const int e = lane + 32 * j;
         if (e >= gr * per && e < (gr + 1) * per) {
-          t2 = fmaxf(t2, fminf(t1, select[j]));
-          t1 = fmaxf(t1, select[j]);
+          k2 = max(k2, min(k1, key[j]));
+          k1 = max(k1, key[j]);
         }
       }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float o1 = __shfl_xor_sync(0xffffffffu, t1, o), o2 = __shfl_xor_sync(0xffffffffu, t2, o);
-        t2 = fmaxf(fmaxf(t2, o2), fminf(t1, o1));
-        t1 = fmaxf(t1, o1);
-      }
-      if (lane == gr) group_score = per > 1 ? t1 + t2 : t1;
+      const uint32_t top = __reduce_max_sync(kAll, k1);
+      // the largest leaves one lane: its next takes part in the second round
+      const uint32_t holders = __ballot_sync(kAll, k1 == top);
+      const uint32_t second = __reduce_max_sync(kAll, lane == __ffs(holders) - 1 ? k2 : k1);
+      if (lane == gr) group_key = order_key(per > 1 ? key_value(top) + key_value(second) : key_value(top));
     }
     uint32_t kept = 0u;
-    for (int i = 0; i < keep_groups; ++i) {
-      float best = lane < n_group && !((kept >> lane) & 1u) ? group_score : -INFINITY;
-      int best_g = best == -INFINITY ? 0x7fffffff : lane;
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-        const int og = __shfl_xor_sync(0xffffffffu, best_g, o);
-        if (ob > best || (ob == best && og < best_g)) { best = ob; best_g = og; }
-      }
-      if (best_g < 32) kept |= 1u << best_g;
+    for (int i = 0; i < p.keep_groups; ++i) {
+      const uint32_t mine = lane < p.n_group && !((kept >> lane) & 1u) ? group_key : 0u;
+      const uint32_t best = __reduce_max_sync(kAll, mine);
+      kept |= 1u << (__ffs(__ballot_sync(kAll, mine == best)) - 1);
     }
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
       const int e = lane + 32 * j;
-      if (e < E && !((kept >> (e / per)) & 1u)) select[j] = -INFINITY;
+      if (e < E && !((kept >> (e / per)) & 1u)) key[j] = 1u;
     }
   }
   float wsum = 0.f;
   float my_w = 0.f;  // lane i keeps the weight of slot i
   int my_id = 0;
-  for (int slot = 0; slot < k; ++slot) {
-    float best = -INFINITY;
-    int best_e = 0x7fffffff;
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      const int e = lane + 32 * j;
-      if (select[j] > best || (select[j] == best && e < best_e)) { best = select[j]; best_e = e; }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-      if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
-    }
-    // owner lane reports the score and retires the expert
+  for (int slot = 0; slot < k; ++slot) {  // k <= 32
+    uint32_t best = 0u;
+    int best_e = lane;
     float w = 0.f;
-    if ((best_e & 31) == lane) {
 #pragma unroll
-      for (int j = 0; j < PER; ++j) {
-        if (lane + 32 * j == best_e) { w = score[j]; select[j] = -INFINITY; }
-      }
-    }
-    w = __shfl_sync(0xffffffffu, w, best_e & 31);
-    if (lane == (slot & 31)) { my_w = w; my_id = best_e; }
+    for (int j = 0; j < PER; ++j)
+      if (key[j] > best) { best = key[j]; best_e = lane + 32 * j; w = score[j]; }
+    const uint32_t top = __reduce_max_sync(kAll, best);
+    const int e = static_cast<int>(__reduce_min_sync(kAll, best == top ? static_cast<uint32_t>(best_e) : 0x7fffffffu));
+    w = __shfl_sync(kAll, w, e & 31);
+#pragma unroll
+    for (int j = 0; j < PER; ++j)
+      if (lane + 32 * j == e) key[j] = 1u;
+    if (lane == slot) { my_w = w; my_id = e; }
     wsum += w;
-    if (slot >= 31) break;  // k <= 32
   }
-  if (scoring == SCORE_TOPK_SOFTMAX) {
+  if (p.scoring == SCORE_TOPK_SOFTMAX) {
     // softmax over the selected logits only
     float m2 = lane < k ? my_w : -INFINITY;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) m2 = fmaxf(m2, __shfl_xor_sync(0xffffffffu, m2, o));
+    for (int o = 16; o > 0; o >>= 1) m2 = fmaxf(m2, __shfl_xor_sync(kAll, m2, o));
     float ex = lane < k ? __expf(my_w - m2) : 0.f;
     float s2 = ex;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) s2 += __shfl_xor_sync(0xffffffffu, s2, o);
+    for (int o = 16; o > 0; o >>= 1) s2 += __shfl_xor_sync(kAll, s2, o);
     my_w = ex / s2;
-  } else if (renorm) {
+  } else if (p.renorm) {
     my_w = my_w / fmaxf(wsum, 1e-20f);
   }
   if (lane < k) {
-    ids[static_cast<size_t>(t) * k + lane] = my_id;
-    weights[static_cast<size_t>(t) * k + lane] = my_w * scale;
+    p.ids[static_cast<size_t>(t) * k + lane] = my_id;
+    p.weights[static_cast<size_t>(t) * k + lane] = my_w * p.scale;
+    if (ids_out != nullptr) ids_out[lane] = my_id;
   }
 }
 
-__global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ sel_bias,
-                                                         int* __restrict__ ids, float* __restrict__ weights, int T, int E,
-                                                         int k, int scoring, int renorm, float scale, int n_group, int keep_groups) {
+template <int PER>
+__global__ void __launch_bounds__(128) moe_route_kernel(RouteParams p, int T) {
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= T) return;
-  route_token(logits, sel_bias, ids, weights, t, threadIdx.x & 31, E, k, scoring, renorm, scale, ld, n_group, keep_groups);
+  route_token<PER>(p, t, threadIdx.x & 31, nullptr);
 }
 
 // Single CTA. routes = T*k. Experts [e0, e1) are local. Outputs:
@@ -179,23 +177,48 @@ __device__ __forceinline__ void plan_block(const int* __restrict__ ids, int rout
   const int n_local = e1 - e0;
   for (int i = threadIdx.x; i < n_local; i += blockDim.x) cnt[i] = 0;
   __syncthreads();
-  for (int r = threadIdx.x; r < routes; r += blockDim.x) {
-    const int e = ids[r] - e0;
-    if (e >= 0 && e < n_local) atomicAdd(&cnt[e], 1);
+  constexpr int kBatch = 8;   // routes a thread has in flight
+  for (int r0 = threadIdx.x; r0 < routes; r0 += kBatch * blockDim.x) {
+    int e[kBatch];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int r = r0 + i * blockDim.x;
+      e[i] = r < routes ? ids[r] - e0 : -1;
+    }
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i)
+      if (e[i] >= 0 && e[i] < n_local) atomicAdd(&cnt[e[i]], 1);
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (threadIdx.x < 32) {   // rows and work items in front of every expert: a lane sums a run of experts, the warp scans the runs
+    const int run = (n_local + 31) >> 5, first = threadIdx.x * run, last = min(n_local, first + run);
     int acc = 0, items = 0;
-    for (int e = 0; e < n_local; ++e) {
-      start[e] = acc;
-      item0[e] = items;
+    for (int e = first; e < last; ++e) {
       acc += cnt[e];
       items += (cnt[e] + tile - 1) / tile;
     }
-    start[n_local] = acc;
-    item0[n_local] = items;
-    counts[0] = acc;
-    counts[1] = items;
+    int acc_in = acc, items_in = items;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int a = __shfl_up_sync(0xffffffffu, acc_in, o), w = __shfl_up_sync(0xffffffffu, items_in, o);
+      if (static_cast<int>(threadIdx.x) >= o) {
+        acc_in += a;
+        items_in += w;
+      }
+    }
+    int at = acc_in - acc, item = items_in - items;
+    for (int e = first; e < last; ++e) {
+      start[e] = at;
+      item0[e] = item;
+      at += cnt[e];
+      item += (cnt[e] + tile - 1) / tile;
+    }
+    if (threadIdx.x == 31) {
+      start[n_local] = acc_in;
+      item0[n_local] = items_in;
+      counts[0] = acc_in;
+      counts[1] = items_in;
+    }
   }
   __syncthreads();
   for (int i = threadIdx.x; i <= n_local; i += blockDim.x) {
@@ -211,14 +234,22 @@ __device__ __forceinline__ void plan_block(const int* __restrict__ ids, int rout
       if (idx < n_work_cap) work[idx] = make_int4(e, start[e] + j * tile, min(tile, cnt[e] - j * tile), 0);
     }
   }
-  for (int r = threadIdx.x; r < routes; r += blockDim.x) {
-    const int e = ids[r] - e0;
-    int pos = -1;
-    if (e >= 0 && e < n_local) {
-      pos = start[e] + atomicAdd(&cursor[e], 1);
-      row_token[pos] = r / k;
+  for (int r0 = threadIdx.x; r0 < routes; r0 += kBatch * blockDim.x) {
+    int e[kBatch], pos[kBatch];
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int r = r0 + i * blockDim.x;
+      e[i] = r < routes ? ids[r] - e0 : -1;
     }
-    route_pos[r] = pos;
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) pos[i] = e[i] >= 0 && e[i] < n_local ? start[e[i]] + atomicAdd(&cursor[e[i]], 1) : -1;
+#pragma unroll
+    for (int i = 0; i < kBatch; ++i) {
+      const int r = r0 + i * blockDim.x;
+      if (r >= routes) continue;
+      if (pos[i] >= 0) row_token[pos[i]] = r / k;
+      route_pos[r] = pos[i];
+    }
   }
 }
 
@@ -235,18 +266,18 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
 // Decode-sized steps (T <= 64 tokens): routing, planning and the row gather in ONE single-CTA kernel instead of
 // three dependent launches. 32 warps route the tokens, the block plans the local experts' segments in shared
 // memory, then copies the token rows into expert order.
+template <int PER>
 __global__ void __launch_bounds__(1024) moe_route_plan_gather_kernel(
-    const float* __restrict__ logits, int ld, const float* __restrict__ sel_bias, int* __restrict__ ids, float* __restrict__ weights,
-    int T, int E, int k, int scoring, int renorm, float scale, int n_group, int keep_groups, int e0, int e1, int tile, int* __restrict__ seg,
-    int* __restrict__ route_pos, int* __restrict__ row_token, int4* __restrict__ work, int n_work_cap, int* __restrict__ counts,
-    const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ xp, int H) {
+    RouteParams p, int T, int e0, int e1, int tile, int* __restrict__ seg, int* __restrict__ route_pos, int* __restrict__ row_token,
+    int4* __restrict__ work, int n_work_cap, int* __restrict__ counts, const __nv_bfloat16* __restrict__ x, __nv_bfloat16* __restrict__ xp, int H) {
+  __shared__ int s_ids[64 * 32];
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int t = warp; t < T; t += 32) route_token(logits, sel_bias, ids, weights, t, lane, E, k, scoring, renorm, scale, ld, n_group, keep_groups);
-  __syncthreads();  // ids written by this block are visible to it
-  plan_block(ids, T * k, k, e0, e1, tile, seg, route_pos, row_token, work, n_work_cap, counts);
+  for (int t = warp; t < T; t += 32) route_token<PER>(p, t, lane, s_ids + t * p.k);
+  __syncthreads();
+  plan_block(s_ids, T * p.k, p.k, e0, e1, tile, seg, route_pos, row_token, work, n_work_cap, counts);
   __syncthreads();
   const int n_rows = xp != nullptr ? counts[0] : 0;  // large steps gather with the many-CTA kernel instead
   for (int pos = warp; pos < n_rows; pos += 32) {
@@ -661,8 +692,13 @@ extern "C" int eredu_moe_route(const float* logits, int ld, const float* sel_bia
                                int scoring, int renorm, float scale, int n_group, int keep_groups, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E > 512 || k > 32 || k > E || n_group < 1 || n_group > 32 || E % n_group != 0 || keep_groups < 1 || keep_groups > n_group) return -1;
-  launch_pdl(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, stream, logits, ld, sel_bias, ids, weights, T, E, k, scoring,
-             renorm, scale, n_group, keep_groups);
+  const RouteParams p = {logits, sel_bias, ids, weights, ld, E, k, scoring, renorm, n_group, keep_groups, scale};
+  const dim3 grid((T + 3) / 4);
+  if (E <= 32) launch_pdl(moe_route_kernel<1>, grid, dim3(128), 0, stream, p, T);
+  else if (E <= 64) launch_pdl(moe_route_kernel<2>, grid, dim3(128), 0, stream, p, T);
+  else if (E <= 128) launch_pdl(moe_route_kernel<4>, grid, dim3(128), 0, stream, p, T);
+  else if (E <= 256) launch_pdl(moe_route_kernel<8>, grid, dim3(128), 0, stream, p, T);
+  else launch_pdl(moe_route_kernel<16>, grid, dim3(128), 0, stream, p, T);
   eredu_count_launches(1);
   return static_cast<int>(cudaGetLastError());
 }
@@ -721,9 +757,16 @@ extern "C" int eredu_moe_route_plan_gather(const float* logits, int ld, const fl
   if (T <= 0) return 0;
   if (E > 512 || k > 32 || k > E || e1 - e0 > 512 || e1 <= e0 || H % 8 != 0 || T > 64) return -1;
   if (n_group < 1 || n_group > 32 || E % n_group != 0 || keep_groups < 1 || keep_groups > n_group) return -1;
-  launch_pdl(moe_route_plan_gather_kernel, dim3(1), dim3(1024), 0, stream, logits, ld, sel_bias, ids, weights, T, E, k, scoring,
-             renorm, scale, n_group, keep_groups, e0, e1, tile, seg, route_pos, row_token, reinterpret_cast<int4*>(work), n_work_cap, counts,
-             static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(xp), H);
+  const RouteParams p = {logits, sel_bias, ids, weights, ld, E, k, scoring, renorm, n_group, keep_groups, scale};
+#define ER_RPG(PER_)                                                                                                            \
+  launch_pdl(moe_route_plan_gather_kernel<PER_>, dim3(1), dim3(1024), 0, stream, p, T, e0, e1, tile, seg, route_pos, row_token, \
+             reinterpret_cast<int4*>(work), n_work_cap, counts, static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(xp), H)
+  if (E <= 32) ER_RPG(1);
+  else if (E <= 64) ER_RPG(2);
+  else if (E <= 128) ER_RPG(4);
+  else if (E <= 256) ER_RPG(8);
+  else ER_RPG(16);
+#undef ER_RPG
   eredu_count_launches(1);
   return static_cast<int>(cudaGetLastError());
 }

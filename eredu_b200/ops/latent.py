@@ -24,10 +24,10 @@ native.register("eredu_latent_prepare", I, [P] * 8 + [I] * 6 + [F, P])
 native.register("eredu_rotate_heads", I, [P] * 3 + [I] * 6 + [P])
 native.register("eredu_gather_rows", I, [P] * 3 + [I] * 3 + [P])
 native.register("eredu_head_linear", I, [P] * 8 + [I] * 4 + [L] * 5 + [I] * 3 + [P])
-native.register("eredu_latent_attn", I, [P] * 7 + [I] * 10 + [F, P])
+native.register("eredu_latent_attn", I, [P] * 7 + [I] * 10 + [F, P, P])
 native.register("eredu_attn_prefill_rows", I, [P] * 8 + [I] * 9 + [L] * 4 + [F, P, P])
 
-MAX_RANK = 512            # latent width of the tensor-core form of absorbed attention
+MAX_RANK, MAX_ROW = 512, 640   # widest latent and cached row of the tensor-core form of absorbed attention
 MAX_SIMT_RANK = 1024      # of its CUDA-core form
 
 
@@ -177,10 +177,17 @@ def _plan(batch, heads_cost, window, dims_ok, device):
     return plans[key]
 
 
-def latent_splits(batch: int, row_tiles: int, seen: int, keys_per_step: int, sm_count: int) -> int:
-    """Split-KV factor of the absorbed form: about one CTA per SM, at least four steps per split, one cluster at most."""
-    steps = max(1, -(-seen // keys_per_step))
-    return max(1, min(CLUSTER_SPLITS, sm_count // max(1, batch * row_tiles), steps // 4 or 1))
+def latent_tile(rows: int, rank: int, rot: int) -> tuple:
+    """(rows of a CTA, CTAs an SM holds) of the absorbed form for sequences of ``rows`` (token, head) pairs."""
+    tile = 64 if rows > 32 else (32 if rows > 16 else 16)
+    return tile, 2 if tile < 64 and rank <= 256 and rank + rot <= 320 else 1
+
+
+def latent_splits(batch: int, row_tiles: int, seen: int, ctas: int) -> int:
+    """Split-KV factor of the absorbed form: about as many CTAs as fit at once (``ctas``), at least two steps of 64 keys per split,
+    one cluster at most."""
+    steps = max(1, -(-seen // 32))
+    return max(1, min(CLUSTER_SPLITS, ctas // max(1, batch * row_tiles), steps // 4 or 1))
 
 
 def _absorbed(q, cache, uk, uv, gate, sinks, inv_freq, positions, heads, dim, rot, scale, window, block_table, seq_lens, cu, q_per_seq,
@@ -192,13 +199,13 @@ def _absorbed(q, cache, uk, uv, gate, sinks, inv_freq, positions, heads, dim, ro
     head_linear(q.view(-1, heads, dim + rot), uk, q_abs, in_rows=rows, rot=rot, positions=positions, inv_freq=inv_freq)
     lat = torch.empty((M, heads, rank), dtype=q.dtype, device=dev)
     B = seq_lens.shape[0]
-    tc = q.dtype == torch.bfloat16 and rank % 8 == 0 and rot % 8 == 0 and rank <= MAX_RANK
+    tc = q.dtype == torch.bfloat16 and rank % 8 == 0 and rot % 8 == 0 and rank <= MAX_RANK and rank + rot <= MAX_ROW
     if tc:
-        tile = 64 if heads * max_n > 32 else (32 if heads * max_n > 16 else 16)
-        tiles = -(-heads * max_n // tile)
-        splits = latent_splits(B, tiles, seen, 64 if tile == 16 else 32, _sm_count(dev))
+        tile, per_sm = latent_tile(heads * max_n, rank, rot)
+        splits = latent_splits(B, -(-heads * max_n // tile), seen, per_sm * _sm_count(dev))
         code = lib().eredu_latent_attn(ptr(q_abs), ptr(cache), ptr(lat), ptr(block_table), ptr(seq_lens), ptr(cu), ptr(sinks), B, q_per_seq,
-                                       max_n, block_table.stride(0), heads, rank, rot, tile, splits, window, scale, stream_ptr(dev))
+                                       max_n, block_table.stride(0), heads, rank, rot, tile, splits, window, scale, ptr(status_word(dev)),
+                                       stream_ptr(dev))
         check(code, "eredu_latent_attn")
     else:
         assert rank <= MAX_SIMT_RANK
