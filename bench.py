@@ -256,9 +256,9 @@ def main() -> int:
                     help="collectives of the tensor / expert ranks: kernels over NVLink peer memory, or torch.distributed (NCCL)")
     ap.add_argument("--router-skew", type=float, default=0.0,
                     help="sparse models: this fraction of the tokens is biased onto 8 hot experts (0 = as routed)")
-    ap.add_argument("--design", default=None, choices=["nidozen"],
+    ap.add_argument("--design", default=None, choices=["nidozen", "lenitar"],
                     help="instead of the headline workload: prefill and decode throughput of this design at a few sizes beside the "
-                         "closest model at equal size, and its kernels against their rooflines (benchmarks/bench_nidozen.py)")
+                         "closest model at equal size, and its kernels against their rooflines (benchmarks/bench_<design>.py)")
     ap.add_argument("--no-baseline", action="store_true", help="skip the in-process baseline arm that fills vs_baseline")
     args = ap.parse_args()
     if args.config == 3:
@@ -277,18 +277,20 @@ def main() -> int:
         return run_torch_baseline(args)
 
     if args.design:
-        from benchmarks import bench_nidozen
+        import importlib
+
+        bench = importlib.import_module(f"benchmarks.bench_{args.design}")
 
         if args.gpus != 1:
             print("--design runs on one GPU", file=sys.stderr)
             return 2
         sampler = ClockSampler(0)
         sampler.start()
-        result = bench_nidozen.run(list(bench_nidozen.SIZES), args.steps)
-        large = result["models"]["large"]["nidozen"]
-        print(json.dumps({"metric": "nidozen_decode_tokens_per_s", "value": large["decode_tokens_per_s"][32], "unit": "tokens/s", "n_gpus": 1,
+        result = bench.run(list(bench.SIZES), args.steps)
+        large = result["models"]["large"][args.design]
+        print(json.dumps({"metric": f"{args.design}_decode_tokens_per_s", "value": large["decode_tokens_per_s"][32], "unit": "tokens/s", "n_gpus": 1,
                           "steps": args.steps, "higher_is_better": True, "dtype": "bf16", "data": "synthetic (random weights and prompts)",
-                          "config": {"sizes": bench_nidozen.SIZES, "seq_len": 2048, "global_batch": 32}, "clocks": sampler.stop(), **result}))
+                          "config": {"sizes": bench.SIZES, "seq_len": 2048, "global_batch": 32}, "clocks": sampler.stop(), **result}))
         return 0
 
     import numpy as np

@@ -8,6 +8,8 @@
 //     the MMA warp already accumulates tile i+1;
 //   * a 4-stage TMA ring (48 KB per stage) runs ahead across tile boundaries;
 //   * the epilogue transposes through a 16 KB staging buffer so that Y leaves the SM as 16-byte row chunks;
+//   * grouped (MoE) form: the tiles come from a work table {expert, first row, rows, -} built on the device, an item of at most 256 rows
+//     each; a short item shortens the MMA instead of multiplying rows nobody stores;
 //   * SwiGLU ("dual") tiles load 64 gate rows and 64 up rows into ONE 128-row operand tile, so gate and up use the
 //     same single 128x256 MMA stream as a plain GEMM; silu(gate) * up is formed when the staged rows are combined.
 //
@@ -49,12 +51,37 @@ struct PGemmParams {
   float* ssq_out;
   int act;  // plain tiles: 2 = squared ReLU before the residual
   int n_tiles, m_tiles;
+  // grouped form: m_tiles work items, used ones first (the rest have no rows); the expert's weights start at row expert * w_rows_per_expert
+  const int4* work;
+  int w_rows_per_expert;
 };
+
+struct PTile {
+  int tile_n, w_row0, m_base, m_cnt;
+};
+
+// Tile t of the list; false behind the last one.
+template <bool GROUPED, int ROWS>
+__device__ __forceinline__ bool tile_at(const PGemmParams& p, int t, PTile& o) {
+  const int tile_m = t / p.n_tiles;
+  o.tile_n = t % p.n_tiles;
+  o.w_row0 = o.tile_n * ROWS;
+  if (GROUPED) {
+    const int4 item = p.work[tile_m];
+    o.w_row0 += item.x * p.w_rows_per_expert;
+    o.m_base = item.y;
+    o.m_cnt = min(item.z, kTN);
+    return item.z > 0;
+  }
+  o.m_base = tile_m * kTN;
+  o.m_cnt = min(kTN, p.M - o.m_base);
+  return true;
+}
 
 __device__ __forceinline__ void epi_bar() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
 
-template <bool DUAL>
+template <bool DUAL, bool GROUPED>
 __global__ void __launch_bounds__(192, 1)
 gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, PGemmParams p) {
   pdl_launch_early();
@@ -112,8 +139,9 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
       int it = 0, issued = 0;
       bool ok = true;
       for (int t = blockIdx.x; t < total && ok; t += gridDim.x) {
-        const int tile_m = t / p.n_tiles, tile_n = t % p.n_tiles;
-        const int w_row0 = tile_n * kRowsPerTile, m_base = tile_m * kTN;
+        PTile tl;
+        if (!tile_at<GROUPED, kRowsPerTile>(p, t, tl)) break;
+        const int w_row0 = tl.w_row0, m_base = tl.m_base;
         for (int kb = 0; kb < kblocks; ++kb, ++it) {
           const int s = it % kStages;
           const uint32_t ph = (it / kStages) & 1;
@@ -138,10 +166,15 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
   } else if (warp == 1) {
     // ------------------------------------------------------------ MMA issuer
     if (lane == 0) {
-      constexpr uint32_t idesc = umma_idesc_bf16(128, kTN);
+      uint32_t idesc = umma_idesc_bf16(128, kTN);
       int it = 0, lt = 0;
       bool ok = true;
       for (int t = blockIdx.x; t < total && ok; t += gridDim.x, ++lt) {
+        if (GROUPED) {
+          PTile tl;
+          if (!tile_at<GROUPED, kRowsPerTile>(p, t, tl)) break;
+          idesc = umma_idesc_bf16(128, (tl.m_cnt + 15) & ~15);
+        }
         const int buf = lt & 1;
         const uint32_t bph = (lt >> 1) & 1;
         ok = mbar_wait(&tempty_bar[buf], bph ^ 1, p.status, kStatusAccumTimeout);
@@ -174,9 +207,9 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
     __nv_bfloat16* yout = static_cast<__nv_bfloat16*>(p.y);
     int lt = 0;
     for (int t = blockIdx.x; t < total; t += gridDim.x, ++lt) {
-      const int tile_m = t / p.n_tiles, tile_n = t % p.n_tiles;
-      const int m_base = tile_m * kTN;
-      const int m_cnt = min(kTN, p.M - m_base);
+      PTile tl;
+      if (!tile_at<GROUPED, kRowsPerTile>(p, t, tl)) break;
+      const int tile_n = tl.tile_n, m_base = tl.m_base, m_cnt = tl.m_cnt;
       const int buf = lt & 1;
       const uint32_t bph = (lt >> 1) & 1;
       if (p.ssq_in != nullptr) {
@@ -340,7 +373,44 @@ int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* re
     }
     return launch_pdl(kern, dim3(grid), dim3(192), kSmemBytes, stream, tmW, tmX, p);
   };
-  const cudaError_t e = dual ? launch(gemm_persistent_kernel<true>) : launch(gemm_persistent_kernel<false>);
+  const cudaError_t e = dual ? launch(gemm_persistent_kernel<true, false>) : launch(gemm_persistent_kernel<false, false>);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+int launch_gemm_persistent_grouped(const void* X, const void* W, void* Y, const int* work, int n_work, int rows_cap, int N, int K, int ldx,
+                                   int ldw, int ldy, int w_rows_total, int w_rows_per_expert, int dual, int sm_count, int* status,
+                                   cudaStream_t stream) {
+  if (N % 8 != 0 || ldy % 8 != 0 || (reinterpret_cast<uintptr_t>(Y) & 15) != 0 || (dual && N % 64 != 0)) return kPersistentUnsupported;
+  CUtensorMap tmW, tmX;
+  int r = make_tma_2d(&tmW, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, w_rows_total, K, ldw, dual ? 64 : 128, 64);
+  if (r != 0) return -100 + r;
+  r = make_tma_2d(&tmX, X, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows_cap, K, ldx, kTN, 64);
+  if (r != 0) return -200 + r;
+  PGemmParams p = {};
+  p.y = Y;
+  p.M = rows_cap;
+  p.N = N;
+  p.K = K;
+  p.ldy = ldy;
+  p.dual_row_offset = N;
+  p.status = status;
+  p.n_tiles = dual ? N / 64 : (N + 127) / 128;
+  p.m_tiles = n_work;
+  p.work = reinterpret_cast<const int4*>(work);
+  p.w_rows_per_expert = w_rows_per_expert;
+  const int sms = sm_count > 0 ? sm_count : 148;
+  const int total = p.n_tiles * n_work;
+  static bool configured[2] = {};
+  if (!configured[dual ? 1 : 0]) {
+    const cudaError_t e = dual ? cudaFuncSetAttribute(gemm_persistent_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes)
+                               : cudaFuncSetAttribute(gemm_persistent_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemBytes);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured[dual ? 1 : 0] = true;
+  }
+  const dim3 grid(total < sms ? total : sms);
+  const cudaError_t e = dual ? launch_pdl(gemm_persistent_kernel<true, true>, grid, dim3(192), kSmemBytes, stream, tmW, tmX, p)
+                             : launch_pdl(gemm_persistent_kernel<false, true>, grid, dim3(192), kSmemBytes, stream, tmW, tmX, p);
   eredu_count_launches(1);
   return static_cast<int>(e);
 }

@@ -13,4 +13,9 @@ int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* re
                            int sm_count, int* status, const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim,
                            float* ssq_out, int act, cudaStream_t stream);
 
+// Expert GEMMs over a work table whose items have at most 256 rows (eredu_gemm_bf16_grouped with tile 256): no bias, SwiGLU when dual.
+int launch_gemm_persistent_grouped(const void* X, const void* W, void* Y, const int* work, int n_work, int rows_cap, int N, int K, int ldx,
+                                   int ldw, int ldy, int w_rows_total, int w_rows_per_expert, int dual, int sm_count, int* status,
+                                   cudaStream_t stream);
+
 }  // namespace eredu

@@ -795,7 +795,9 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
                                const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim, float* ssq_out,
                                int flags, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
-  const int tn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
+  int tn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
+  // a narrow output over many tokens (a router) fills the machine with small token tiles instead
+  if (tn == 256 && out_fp32 && ((N + 127) / 128) * ((M + 255) / 256) * 2 <= sm_count) tn = 64;
   if (tn == 256 && !out_fp32 && force_split <= 1 && persistent_enabled()) {
     // prefill-sized: persistent kernel with double-buffered accumulators
     const int pr = launch_gemm_persistent(X, W, Y, residual, bias, M, N, K, ldx, ldw, ldy, ldr, w_rows, dual, dual_row_offset,
@@ -954,6 +956,11 @@ extern "C" int eredu_gemm_bf16_grouped(const void* X, const void* W, void* Y, co
                                        const void* bias, int bias_expert_stride, int act, float act_limit,
                                        cudaStream_t stream) {
   if (n_work <= 0 || N <= 0 || K <= 0) return 0;
+  if (tile == 256) {
+    if (bias != nullptr || act != 0 || act_limit > 0.f) return -1;
+    return launch_gemm_persistent_grouped(X, W, Y, work, n_work, rows_cap, N, K, ldx, ldw, ldy, w_rows_total, w_rows_per_expert, dual, sm_count,
+                                          status, stream);
+  }
   CUtensorMap tmW, tmX;
   int r = make_tma_2d(&tmW, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, w_rows_total, K, ldw, 128, 64);
   if (r != 0) return -100 + r;

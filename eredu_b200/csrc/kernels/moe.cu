@@ -170,28 +170,52 @@ __global__ void __launch_bounds__(128) moe_route_kernel(RouteParams p, int T) {
 __device__ __forceinline__ void plan_block(const int* __restrict__ ids, int routes, int k, int e0, int e1, int tile,
                                            int* __restrict__ seg, int* __restrict__ route_pos, int* __restrict__ row_token,
                                            int4* __restrict__ work, int n_work_cap, int* __restrict__ counts) {
+  // Every warp takes a run of routes: it counts them per expert, and once the runs in front are known, ranks its own again in the same
+  // order - rows of an expert keep the order of the routes, and warps do not contend for counters.
   __shared__ int cnt[512];
   __shared__ int start[513];
-  __shared__ int cursor[512];
   __shared__ int item0[513];
+  __shared__ unsigned short hist[32][512];   // per warp and expert: routes counted, then the rows in front of the warp's own
   const int n_local = e1 - e0;
-  for (int i = threadIdx.x; i < n_local; i += blockDim.x) cnt[i] = 0;
-  __syncthreads();
-  constexpr int kBatch = 8;   // routes a thread has in flight
-  for (int r0 = threadIdx.x; r0 < routes; r0 += kBatch * blockDim.x) {
-    int e[kBatch];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int run = ((routes + warps - 1) / warps + 31) & ~31, r_first = warp * run, r_last = min(routes, r_first + run);
+  for (int i = lane; i < n_local; i += 32) hist[warp][i] = 0;
+  __syncwarp();
+  constexpr int kBatch = 4;                  // groups of 32 routes in flight
+  auto each_route = [&](auto visit) {
+    for (int r0 = r_first; r0 < r_last; r0 += 32 * kBatch) {
+      int e[kBatch];
 #pragma unroll
-    for (int i = 0; i < kBatch; ++i) {
-      const int r = r0 + i * blockDim.x;
-      e[i] = r < routes ? ids[r] - e0 : -1;
+      for (int i = 0; i < kBatch; ++i) {
+        const int r = r0 + i * 32 + lane;
+        e[i] = r < r_last ? ids[r] - e0 : -1;
+        if (e[i] < 0 || e[i] >= n_local) e[i] = -1;
+      }
+#pragma unroll
+      for (int i = 0; i < kBatch; ++i) {
+        const unsigned peers = __match_any_sync(0xffffffffu, e[i]);
+        const int before = __popc(peers & ((1u << lane) - 1u));
+        visit(r0 + i * 32 + lane, e[i], before, __popc(peers));
+        __syncwarp();
+      }
     }
-#pragma unroll
-    for (int i = 0; i < kBatch; ++i)
-      if (e[i] >= 0 && e[i] < n_local) atomicAdd(&cnt[e[i]], 1);
+  };
+  each_route([&](int, int e, int before, int n) {
+    if (e >= 0 && before == 0) hist[warp][e] = static_cast<unsigned short>(hist[warp][e] + n);
+  });
+  __syncthreads();
+  for (int e = threadIdx.x; e < n_local; e += blockDim.x) {
+    int acc = 0;
+    for (int w = 0; w < warps; ++w) {
+      const int n = hist[w][e];
+      hist[w][e] = static_cast<unsigned short>(acc);
+      acc += n;
+    }
+    cnt[e] = acc;
   }
   __syncthreads();
   if (threadIdx.x < 32) {   // rows and work items in front of every expert: a lane sums a run of experts, the warp scans the runs
-    const int run = (n_local + 31) >> 5, first = threadIdx.x * run, last = min(n_local, first + run);
+    const int per = (n_local + 31) >> 5, first = threadIdx.x * per, last = min(n_local, first + per);
     int acc = 0, items = 0;
     for (int e = first; e < last; ++e) {
       acc += cnt[e];
@@ -221,10 +245,7 @@ __device__ __forceinline__ void plan_block(const int* __restrict__ ids, int rout
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i <= n_local; i += blockDim.x) {
-    seg[i] = start[i];
-    if (i < n_local) cursor[i] = 0;
-  }
+  for (int i = threadIdx.x; i <= n_local; i += blockDim.x) seg[i] = start[i];
   for (int i = threadIdx.x; i < n_work_cap; i += blockDim.x) work[i] = make_int4(0, 0, 0, 0);
   __syncthreads();
   for (int e = threadIdx.x; e < n_local; e += blockDim.x) {
@@ -234,23 +255,16 @@ __device__ __forceinline__ void plan_block(const int* __restrict__ ids, int rout
       if (idx < n_work_cap) work[idx] = make_int4(e, start[e] + j * tile, min(tile, cnt[e] - j * tile), 0);
     }
   }
-  for (int r0 = threadIdx.x; r0 < routes; r0 += kBatch * blockDim.x) {
-    int e[kBatch], pos[kBatch];
-#pragma unroll
-    for (int i = 0; i < kBatch; ++i) {
-      const int r = r0 + i * blockDim.x;
-      e[i] = r < routes ? ids[r] - e0 : -1;
-    }
-#pragma unroll
-    for (int i = 0; i < kBatch; ++i) pos[i] = e[i] >= 0 && e[i] < n_local ? start[e[i]] + atomicAdd(&cursor[e[i]], 1) : -1;
-#pragma unroll
-    for (int i = 0; i < kBatch; ++i) {
-      const int r = r0 + i * blockDim.x;
-      if (r >= routes) continue;
-      if (pos[i] >= 0) row_token[pos[i]] = r / k;
-      route_pos[r] = pos[i];
-    }
-  }
+  each_route([&](int r, int e, int before, int n) {
+    int base = 0;
+    if (e >= 0) base = hist[warp][e];
+    __syncwarp();
+    if (e >= 0 && before == 0) hist[warp][e] = static_cast<unsigned short>(base + n);
+    if (r >= r_last) return;
+    const int pos = e >= 0 ? start[e] + base + before : -1;
+    if (pos >= 0) row_token[pos] = r / k;
+    route_pos[r] = pos;
+  });
 }
 
 __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ ids, int routes, int k, int e0, int e1,
@@ -705,7 +719,7 @@ extern "C" int eredu_moe_route(const float* logits, int ld, const float* sel_bia
 
 extern "C" int eredu_moe_plan(const int* ids, int routes, int k, int e0, int e1, int tile, int* seg, int* route_pos,
                               int* row_token, int* work, int n_work_cap, int* counts, cudaStream_t stream) {
-  if (e1 - e0 > 512 || e1 <= e0) return -1;
+  if (e1 - e0 > 512 || e1 <= e0 || routes > 65535 * 32) return -1;   // counters of 16 bits per warp
   launch_pdl(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, ids, routes, k, e0, e1, tile, seg, route_pos, row_token,
              reinterpret_cast<int4*>(work), n_work_cap, counts);
   eredu_count_launches(1);

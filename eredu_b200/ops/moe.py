@@ -158,6 +158,13 @@ def pick_tile(expected_rows_per_expert: float) -> int:
     return 128
 
 
+def expert_tile(routes: int, e_local: int, inter: int, hidden: int, plain: bool) -> int:
+    """Rows of a work item: as many as an expert is expected to get, up to 128, or the 256 of the persistent form where it applies
+    (prompt-sized steps, SwiGLU without bias or limit)."""
+    per = routes / max(1, e_local)
+    return 256 if plain and per > 128 and inter % 64 == 0 and hidden % 8 == 0 else pick_tile(per)
+
+
 def route_plan_gather(logits, x, k, scoring, renorm, scale, sel_bias, e0, n_local, n_group=1, topk_group=1):
     """Decode-sized steps (<= 64 tokens): routing, the local experts' plan and the row gather in one kernel.
     Returns (ids, weights, plan, xp) for :func:`experts_forward`."""
@@ -220,7 +227,7 @@ def expert_rows(x, ids, w_gate_up, w_down, e0=0, limit=0.0, act="swiglu", plan=N
     if x.dtype == torch.bfloat16 and H % 8 == 0 and inter % 8 == 0:
         if plan is None:
             routes = ids.numel()
-            plan = ExpertPlan(ids, ids.shape[1], e0, e0 + E_local, pick_tile(routes / max(1, E_local)), routes)
+            plan = ExpertPlan(ids, ids.shape[1], e0, e0 + E_local, expert_tile(routes, E_local, inter, H, act == "swiglu" and limit == 0.0), routes)
             xp = torch.empty((routes, H), dtype=x.dtype, device=x.device)
             check(lib().eredu_moe_gather(ptr(x), ptr(plan.row_token), ptr(plan.counts), ptr(xp), routes, H, stream_ptr(x.device)),
                   "eredu_moe_gather")
@@ -266,7 +273,7 @@ def experts_forward(x, ids, weights, w_gate_up, w_down, e0=0, residual=None, ext
     rows_cap = rows_cap or routes
     dev = x.device
     if plan is None:
-        tile = pick_tile(routes / max(1, E_local))
+        tile = expert_tile(routes, E_local, inter, H, act == "swiglu" and limit == 0.0 and gu_bias is None and down_bias is None)
         plan = ExpertPlan(ids, k, e0, e0 + E_local, tile, rows_cap)
         xp = torch.empty((rows_cap, H), dtype=x.dtype, device=dev)
         check(lib().eredu_moe_gather(ptr(x), ptr(plan.row_token), ptr(plan.counts), ptr(xp), rows_cap, H, stream_ptr(dev)),
