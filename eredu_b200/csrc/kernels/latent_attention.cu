@@ -119,8 +119,10 @@ __global__ void __launch_bounds__(256, RG < 4 && TIER < 4 ? 2 : 1) latent_attn_k
     *reinterpret_cast<uint4*>(ring + r * S + c * 8) = make_uint4(0u, 0u, 0u, 0u);
   }
   __syncthreads();
-  pdl_wait();
-  pdl_launch_dependents();
+  // Only the queries come from the kernel in front of this one: lengths, page tables and cached rows are older, so the rows start on their
+  // way before the wait. (A kernel starts once all CTAs in front have passed their own wait, that is, once everything before those is
+  // complete; not so when dependents are released early.)
+  if (EREDU_PDL_EARLY) pdl_wait();
   const int b = blockIdx.z, split = blockIdx.x;
   const int q0 = p.cu_q != nullptr ? p.cu_q[b] : b * p.q_per_seq;
   const int q_len = p.cu_q != nullptr ? p.cu_q[b + 1] - q0 : p.q_per_seq;
@@ -166,6 +168,8 @@ __global__ void __launch_bounds__(256, RG < 4 && TIER < 4 ? 2 : 1) latent_attn_k
   find_page(0);
 #pragma unroll
   for (int s = 0; s < kAhead; ++s) load_step(s);
+  pdl_wait();
+  pdl_launch_dependents();
   for (int i = threadIdx.x; i < T::kRows * chunks; i += 256) {
     const int r = i / chunks, c = i - r * chunks;
     const bool ok = row0 + r < rows && c < real;

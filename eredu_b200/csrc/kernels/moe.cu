@@ -84,21 +84,38 @@ __device__ __forceinline__ void route_token(const RouteParams& p, int t, int lan
     // best keep_groups groups stay eligible. Lane g keeps the score of group g.
     const int per = E / p.n_group;
     uint32_t group_key = 0u;
-    for (int gr = 0; gr < p.n_group; ++gr) {
-      uint32_t k1 = 0u, k2 = 0u;   // this lane's two largest of the group
+    if (per <= 32 && (per & (per - 1)) == 0) {
+      // a group is a run of neighbouring lanes at one j: all groups at once, two largest by exchanges inside the runs
 #pragma unroll
       for (int j = 0; j < PER; ++j) {
-        const int e = lane + 32 * j;
-        if (e >= gr * per && e < (gr + 1) * per) {
-          k2 = max(k2, min(k1, key[j]));
-          k1 = max(k1, key[j]);
+        uint32_t k1 = key[j], k2 = 0u;
+        for (int o = 1; o < per; o <<= 1) {
+          const uint32_t o1 = __shfl_xor_sync(kAll, k1, o), o2 = __shfl_xor_sync(kAll, k2, o);
+          k2 = max(max(k2, o2), min(k1, o1));
+          k1 = max(k1, o1);
         }
+        // lane g takes the sum of its group, whose experts start at g * per
+        const uint32_t first = __shfl_sync(kAll, k1, (lane * per) & 31), next = __shfl_sync(kAll, k2, (lane * per) & 31);
+        if (lane < p.n_group && (lane * per) >> 5 == j)
+          group_key = order_key(per > 1 ? key_value(first) + key_value(next) : key_value(first));
       }
-      const uint32_t top = __reduce_max_sync(kAll, k1);
-      // the largest leaves one lane: its next takes part in the second round
-      const uint32_t holders = __ballot_sync(kAll, k1 == top);
-      const uint32_t second = __reduce_max_sync(kAll, lane == __ffs(holders) - 1 ? k2 : k1);
-      if (lane == gr) group_key = order_key(per > 1 ? key_value(top) + key_value(second) : key_value(top));
+    } else {
+      for (int gr = 0; gr < p.n_group; ++gr) {
+        uint32_t k1 = 0u, k2 = 0u;   // this lane's two largest of the group
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+          const int e = lane + 32 * j;
+          if (e >= gr * per && e < (gr + 1) * per) {
+            k2 = max(k2, min(k1, key[j]));
+            k1 = max(k1, key[j]);
+          }
+        }
+        const uint32_t top = __reduce_max_sync(kAll, k1);
+        // the largest leaves one lane: its next takes part in the second round
+        const uint32_t holders = __ballot_sync(kAll, k1 == top);
+        const uint32_t second = __reduce_max_sync(kAll, lane == __ffs(holders) - 1 ? k2 : k1);
+        if (lane == gr) group_key = order_key(per > 1 ? key_value(top) + key_value(second) : key_value(top));
+      }
     }
     uint32_t kept = 0u;
     for (int i = 0; i < p.keep_groups; ++i) {
