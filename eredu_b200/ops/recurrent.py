@@ -14,6 +14,7 @@ from typing import Optional
 import torch
 
 from . import native
+from .core import _sm_count
 from .native import F, I, P, check, lib, ptr, stream_ptr
 
 native.register("eredu_gated_delta_scan", I, [P, P, P, P, P, P, P, I, I, I, I, I, I, P])
@@ -425,11 +426,7 @@ def mlstm(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_sl
     code = lib().eredu_mlstm(ptr(proj), ptr(gates), ptr(norm_w), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table),
                              ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv,
                              proj.stride(0), gates.stride(0), state.shape[1], M, batch_size, batch.q_per_seq, rows,
-                             batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, native_sms(proj.device), cap, eps,
+                             batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, _sm_count(proj.device), cap, eps,
                              stream_ptr(proj.device))
     check(code, "eredu_mlstm")
     return out
-
-
-def native_sms(device) -> int:
-    return torch.cuda.get_device_properties(device).multi_processor_count

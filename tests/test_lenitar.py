@@ -121,7 +121,7 @@ def test_stream_and_norm_of_the_sum(dev, dt, width):
 
 
 @both
-@pytest.mark.parametrize("E,top,groups,keep", [(12, 3, 2, 1), (12, 3, 3, 2), (8, 2, 1, 1), (8, 3, 8, 3), (64, 6, 8, 4), (256, 8, 8, 4), (30, 4, 3, 3), (512, 32, 32, 4)])
+@pytest.mark.parametrize("E,top,groups,keep", [(10, 3, 2, 1), (12, 3, 3, 2), (8, 2, 1, 1), (8, 3, 8, 3), (64, 6, 8, 4), (256, 8, 8, 4), (30, 4, 3, 3), (512, 32, 32, 4)])
 def test_routing_by_groups(dev, dt, E, top, groups, keep):
     T = 70
     z = rand(T, E, seed=1) * 2
@@ -147,14 +147,14 @@ def test_routing_by_groups(dev, dt, E, top, groups, keep):
 
 
 @both
-@pytest.mark.parametrize("T,W,ff,E,top", [(1, 64, 24, 4, 2), (40, 96, 40, 6, 3), (200, 64, 96, 5, 2), (130, 70, 51, 3, 1), (33, 40, 13, 7, 7)])
+@pytest.mark.parametrize("T,W,ff,E,top", [(1, 64, 24, 4, 2), (40, 96, 40, 6, 3), (200, 64, 96, 5, 2), (130, 70, 51, 3, 1), (33, 40, 13, 7, 7), (700, 64, 64, 3, 2), (450, 72, 128, 2, 1)])
 def test_experts_of_every_route(dev, dt, T, W, ff, E, top):
     x, gu, dn = rand(T, W, seed=1), rand(E, 2 * ff, W, seed=2) / 8, rand(E, W, ff, seed=3) / 8
     gu, dn = gu.to(torch.bfloat16).double(), dn.to(torch.bfloat16).double()
     ids = torch.stack([torch.randperm(E, generator=torch.Generator().manual_seed(t))[:top] for t in range(T)]).int()
     rows, pos = moe_ops.expert_rows(x.to(dev, dt), ids.to(dev), gu.to(dev, dt), dn.to(dev, dt))
     got = rows[pos.long()].double().cpu().view(T, top, W)
-    for t in range(T):
+    for t in range(0, T, 1 + T // 150):
         for s in range(top):
             e = int(ids[t, s])
             w = {"gate": gu[e, :ff], "up": gu[e, ff:], "down": dn[e]}
@@ -234,7 +234,7 @@ def decode_batch(lens, tables, dev, most):
                         seq_lens=torch.tensor(lens, dtype=torch.int32, device=dev), is_prefill=False, q_per_seq=1, max_kv_len=most)
 
 
-ATTENTION = [(4, 32, 32, 80, 96, 72), (3, 16, 8, 24, 40, 37), (2, 128, 64, 128, 256, 100), (5, 64, 64, 64, 128, 16), (1, 72, 16, 40, 512, 128),
+ATTENTION = [(4, 40, 24, 88, 112, 78), (3, 16, 8, 24, 40, 37), (2, 128, 64, 128, 256, 100), (5, 64, 64, 64, 128, 16), (1, 72, 16, 40, 512, 128),
              (20, 24, 16, 32, 64, 200), (2, 100, 24, 8, 48, 1), (3, 20, 6, 12, 33, 9), (1, 9, 4, 11, 18, 2), (40, 16, 8, 16, 384, 0)]
 
 
@@ -344,7 +344,7 @@ PORTIONS = [[300], [1] * 12 + [40, 2, 2, 100, 64, 65, 15], [64, 128, 16, 8, 9, 7
 @both
 @pytest.mark.parametrize("portions", PORTIONS)
 @pytest.mark.parametrize("H,D,V,cap,kind", [(3, 24, 40, 9.0, "plain"), (2, 64, 128, 15.0, "keep"), (1, 128, 256, 15.0, "loud"), (2, 16, 64, 15.0, "swing"),
-                                            (1, 256, 392, 12.0, "plain"), (2, 48, 48, 15.0, "loud"), (1, 20, 30, 2.0, "swing"), (3, 7, 5, 15.0, "keep")])
+                                            (1, 256, 392, 12.0, "plain"), (2, 40, 56, 15.0, "loud"), (1, 20, 30, 2.0, "swing"), (3, 7, 5, 15.0, "keep")])
 def test_matrix_memory(dev, dt, H, D, V, cap, kind, portions):
     T = 300
     x, z, nw = mlstm_inputs(T, H, D, V, 7, kind)
