@@ -17,7 +17,7 @@ QWEN_HYBRID_TYPES = {"qwen3_next", "qwen3_5", "qwen3_5_moe", "qwen3_5_text", "qw
 
 # Families whose layers each name their mixer and its sizes (``ModelConfig.mixers``). ``models/<model type>.py`` reads the
 # configuration and the tensors, and runs a block.
-MIXER_FAMILIES = ("nidozen", "lenitar")
+MIXER_FAMILIES = ("nidozen", "lenitar", "kasuvik")
 
 
 def mixer_family(model_type: str):
@@ -44,12 +44,14 @@ class RoutedSpec:
 @dataclass
 class MixerSpec:
     """Geometry and constants of one layer of a family whose layers do not share them (``ModelConfig.mixers``)."""
-    kind: str                        # "attention" | "latent_attention" | "gla" (gated linear attention) | "mingru" | "mlstm"
-    heads: int = 0                   # query heads (attention) or recurrent heads (gla, mlstm)
+    # "attention" | "latent_attention" | "gla" (gated linear attention) | "mingru" | "mlstm" | "mamba" | "general_delta" |
+    # "parallel" (an attention and a recurrent mixer side by side: ``left``, ``right``)
+    kind: str
+    heads: int = 0                   # query heads (attention) or recurrent heads (gla, mlstm, general_delta)
     kv_heads: int = 0
     dim: int = 0                     # query / key size of a head
     vdim: int = 0                    # value size of a head
-    width: int = 0                   # mingru: channels
+    width: int = 0                   # mingru, mamba: channels
     scale: float = 1.0               # attention: score multiplier
     chunk: int = 0                   # attention: keys are visible inside the query's own chunk of positions (0: all earlier)
     rot_dims: int = 0                # rotated leading dimensions of a head (0: no rotation)
@@ -62,17 +64,57 @@ class MixerSpec:
     kv_rank: int = 0                 # latent attention: width of the cached latent (``rot_dims`` more hold the rotated key part)
     gate_cap: float = 0.0            # mlstm: soft cap of the gates' pre-activations
     moe: RoutedSpec | None = None    # sparse feed-forward
+    pool: int = 0                    # attention: tokens of a block whose mean key and value stay visible behind the window (0: none)
+    conv: int = 0                    # taps of the causal convolution over q, k and v (attention) or the channels (mamba); 0, 1: no history
+    state: int = 0                   # mamba: states of a channel
+    dt_rank: int = 0                 # mamba: width of the step size's input
+    left: "MixerSpec | None" = None  # parallel: the attention
+    right: "MixerSpec | None" = None  # parallel: the recurrent mixer
+
+    @property
+    def has_kv(self) -> bool:
+        """The mixer appends keys and values of its own to the paged cache."""
+        if self.kind == "parallel":
+            return self.left.has_kv
+        return self.kind in ("attention", "latent_attention") and self.kv_from is None
+
+    @property
+    def kv_pool(self) -> int:
+        """Tokens of a pooled block of the cached keys and values (0: none are pooled)."""
+        return self.left.kv_pool if self.kind == "parallel" else self.pool
 
     @property
     def kv_dims(self) -> tuple:
         """(heads, key width, value width) of one cached token."""
+        if self.kind == "parallel":
+            return self.left.kv_dims
         if self.kind == "latent_attention":
             return 1, self.kv_rank + self.rot_dims, 0
         return self.kv_heads, self.dim, self.vdim
 
     @property
+    def conv_channels(self) -> int:
+        """Channels whose last inputs a causal convolution keeps."""
+        return self.width if self.kind == "mamba" else self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+
+    @property
+    def conv_elems(self) -> int:
+        """fp32 elements of the convolution's history, rounded up to whole 16-byte pieces."""
+        return -(-max(0, self.conv - 1) * self.conv_channels // 4) * 4
+
+    @property
     def state_shape(self) -> tuple | None:
         """fp32 recurrent state of one sequence (None: no recurrence)."""
+        if self.kind == "general_delta":
+            return (self.heads, self.dim, self.vdim)
+        if self.kind == "mamba":
+            # the states of all channels, then the convolution's history [taps - 1, channels]
+            return (-(-self.width * self.state // 4) * 4 + self.conv_elems,)
+        if self.kind == "attention" and self.conv > 1:
+            return (self.conv_elems,)
+        if self.kind == "parallel":
+            # both, the recurrent one first
+            return (self.right.state_shape[0] + (self.left.state_shape or (0,))[0],)
         if self.kind == "mingru":
             return (self.width,)
         if self.kind == "gla":
@@ -185,6 +227,10 @@ class ModelConfig:
         """The earlier layer whose cached keys and values this layer reads instead of keeping its own."""
         return self.mixers[layer].kv_from if self.mixers is not None else None
 
+    def layer_kv_pool(self, layer: int) -> int:
+        """Tokens of a pooled block of this layer's cached keys and values (0: none are pooled)."""
+        return self.mixers[layer].kv_pool if self.mixers is not None else 0
+
     def layer_state_shape(self, layer: int) -> tuple | None:
         """fp32 state one sequence keeps in this layer, for families that state it per layer."""
         return self.mixers[layer].state_shape if self.mixers is not None else None
@@ -225,8 +271,7 @@ class ModelConfig:
     def layer_has_kv(self, layer: int) -> bool:
         """The layer appends K/V pages (softmax attention); every other operator keeps a fixed state or none."""
         if self.mixers is not None:
-            m = self.mixers[layer]
-            return m.kind in ("attention", "latent_attention") and m.kv_from is None
+            return self.mixers[layer].has_kv
         if self.layer_types is None:
             return True
         if self.model_type == "gemma4":      # the KV-sharing tail reads an earlier layer's pages

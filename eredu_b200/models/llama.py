@@ -65,6 +65,7 @@ class ForwardBatch:
     stream: Optional[tuple] = None
     # prefill: (first new position, new tokens) of every sequence, known on the host (operators that size scratch by context)
     portions: Optional[list] = None
+    pool_rows: dict = field(default_factory=dict)   # prefill: where pooled blocks of each size lie as dense rows (ops.pooling)
     max_kv_len: int = 0                # decode: the longest context the step (or every replay of its graph) can see
     sm_count: int = 1
 

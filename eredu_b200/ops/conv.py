@@ -1,4 +1,5 @@
-"""Gated causal short convolution with recurrent state (the operator of LFM2's "conv" layers).
+"""Causal short convolutions with recurrent state: the gated operator of LFM2's "conv" layers, and the convolutions of projections
+in front of attention and selective scans (:func:`conv_project`).
 
 ``proj = in_proj(x) = [B | C | X]``; ``bx = B * X``; ``y[t] = sum_j w[:, j] * bx[t - (L-1) + j]`` (depthwise, causal);
 ``out = C * (y + bias)`` (eredu/src/backend/mlx/architectures/lfm2/model.rs:899-914; the rolling cache of the last
@@ -8,12 +9,15 @@ decode graph needs no host-side indices.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
 
 from . import native
 from .native import I, P, check, lib, ptr, stream_ptr
+from .pooling import PAGE, pool_block_ref
+from .recurrent import _sequences
 
 native.register("eredu_short_conv", I, [P, I, P, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, P])
 
@@ -70,3 +74,127 @@ def short_conv(proj: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor]
                                   B, max_q_len, mode, x_off, stream_ptr(proj.device))
     check(code, "eredu_short_conv")
     return out
+
+
+native.register("eredu_conv_project", I, [P] * 19 + [I] * 20 + [P])
+
+
+@dataclass
+class ConvHeads:
+    """Leading channels [q heads | k heads | v heads] of a projection: convolved, q and k rotated, q scaled per head, keys and
+    values appended to the paged cache (and the means of the blocks of ``pool`` tokens they complete)."""
+    taps: torch.Tensor                    # fp32 [taps, n_q dk + n_kv (dk + dv)]
+    n_q: int
+    n_kv: int
+    dk: int
+    dv: int
+    inv_freq: torch.Tensor                # fp32 [rotated dims / 2]; neighbouring dims (2 i, 2 i + 1) form a pair
+    k_cache: torch.Tensor
+    v_cache: torch.Tensor
+    q_scale: Optional[torch.Tensor] = None   # fp32 [n_q]
+    pool: int = 0
+    pooled: Optional[tuple] = None        # mean keys and values of the layer
+    hist: int = 0                         # where the history starts in a sequence's state
+
+    @property
+    def channels(self) -> int:
+        return self.taps.shape[1]
+
+
+@dataclass
+class ConvChannels:
+    """``width`` channels of a projection from column ``start``: convolved, bias, SiLU."""
+    taps: torch.Tensor                    # fp32 [taps, width]
+    bias: Optional[torch.Tensor]          # fp32 [width]
+    start: int
+    hist: int = 0
+
+    @property
+    def width(self) -> int:
+        return self.taps.shape[1]
+
+
+def _conv_rows(u, taps, hist):
+    """u [n, C] fp32, taps [L, C], hist [L - 1, C] -> (y [n, C], the new history)."""
+    full = torch.cat((hist, u))
+    return sum(taps[j] * full[j:j + u.shape[0]] for j in range(taps.shape[0])), full[full.shape[0] - hist.shape[0]:]
+
+
+def conv_project_ref(proj, state, batch, page_to_slot, heads=None, channels=None):
+    M = proj.shape[0]
+    bounds = _sequences(batch)
+    q = torch.zeros((M, heads.n_q, heads.dk), dtype=proj.dtype, device=proj.device) if heads is not None else None
+    out = torch.zeros((M, channels.width), dtype=proj.dtype, device=proj.device) if channels is not None else None
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(batch.slots[r0]) < 0:
+            continue
+        st = state[int(page_to_slot[int(batch.block_table[b, 0])])].view(-1)
+        for sec, start in ((heads, 0), (channels, channels.start if channels is not None else 0)):
+            if sec is None:
+                continue
+            L, C = sec.taps.shape
+            hist = st[sec.hist:sec.hist + (L - 1) * C].view(L - 1, C)
+            y, new = _conv_rows(proj[r0:r1, start:start + C].float(), sec.taps.float(), hist.clone())
+            hist.copy_(new)
+            if sec is channels:
+                y = y if sec.bias is None else y + sec.bias.float()
+                out[r0:r1] = torch.nn.functional.silu(y).to(out.dtype)
+                continue
+            n, kw = sec.n_q * sec.dk, sec.n_kv * sec.dk
+            rot = 2 * sec.inv_freq.shape[0]
+            ang = batch.positions[r0:r1].float()[:, None] * sec.inv_freq.float()[None, :]
+            cos, sin = ang.cos()[:, None, :], ang.sin()[:, None, :]
+
+            def rotate(t):
+                u, v = t[..., 0:rot:2], t[..., 1:rot:2]
+                return torch.cat((torch.stack((u * cos - v * sin, v * cos + u * sin), -1).flatten(-2), t[..., rot:]), -1)
+
+            qq = rotate(y[:, :n].view(-1, sec.n_q, sec.dk))
+            if sec.q_scale is not None:
+                qq = qq * sec.q_scale.float()[None, :, None]
+            q[r0:r1] = qq.to(q.dtype)
+            k, v = rotate(y[:, n:n + kw].view(-1, sec.n_kv, sec.dk)), y[:, n + kw:].view(-1, sec.n_kv, sec.dv)
+            slots = batch.slots[r0:r1].long()
+            sec.k_cache[slots // PAGE, :, slots % PAGE] = k.to(sec.k_cache.dtype)
+            sec.v_cache[slots // PAGE, :, slots % PAGE] = v.to(sec.v_cache.dtype)
+            if sec.pool:
+                end = int(batch.seq_lens[b])
+                for blk in range((end - (r1 - r0)) // sec.pool, end // sec.pool):
+                    pool_block_ref(sec.k_cache, sec.v_cache, sec.pooled, batch.block_table[b], blk, sec.pool)
+    return q, out
+
+
+def conv_project(proj, state, batch, page_to_slot, heads: Optional[ConvHeads] = None, channels: Optional[ConvChannels] = None):
+    """Causal depthwise convolutions ``y_t = sum_j taps[j] u_(t - L + 1 + j)`` over ranges of a projection's columns, one launch for
+    both kinds of range: ``heads`` -> queries [M, n_q, dk], keys and values into their pages; ``channels`` -> silu(y + bias) [M, width].
+    The last L - 1 inputs of a sequence live in ``state`` (fp32 [slots, ...]) from element ``hist`` on, [L - 1, channels]; zeros for a
+    new sequence. Portions may have any length. Returns (queries or None, channels or None)."""
+    if not proj.is_cuda:
+        return conv_project_ref(proj, state, batch, page_to_slot, heads, channels)
+    assert proj.stride(1) == 1 and state.is_contiguous() and state.dtype == torch.float32
+    M, fp32 = proj.shape[0], proj.dtype == torch.float32
+    q = out = None
+    a, c = heads, channels
+    if a is not None:
+        assert a.k_cache.is_contiguous() and a.v_cache.is_contiguous() and a.k_cache.dtype == proj.dtype and a.taps.is_contiguous()
+        q = torch.empty((M, a.n_q, a.dk), dtype=proj.dtype, device=proj.device)
+    if c is not None:
+        assert c.taps.is_contiguous()
+        out = torch.empty((M, c.width), dtype=proj.dtype, device=proj.device)
+    if M == 0:
+        return q, out
+    n = batch.block_table.shape[0]
+    rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
+    pk, pv = a.pooled if a is not None and a.pool else (None, None)
+    code = lib().eredu_conv_project(
+        ptr(proj), ptr(state), ptr(q), ptr(out), ptr(a.taps) if a else None, ptr(c.taps) if c else None, ptr(c.bias) if c else None,
+        ptr(a.k_cache) if a else None, ptr(a.v_cache) if a else None, ptr(pk), ptr(pv), ptr(a.inv_freq) if a else None,
+        ptr(a.q_scale) if a else None, ptr(batch.positions), ptr(batch.block_table), ptr(page_to_slot),
+        ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), ptr(batch.seq_lens), proj.stride(0), state[0].numel(),
+        a.taps.shape[0] if a else 0, c.taps.shape[0] if c else 0, a.n_q if a else 0, a.n_kv if a else 0, a.dk if a else 0, a.dv if a else 0,
+        2 * a.inv_freq.shape[0] if a else 0, a.pool if a else 0, pk.shape[2] if pk is not None else 0, a.hist if a else 0,
+        c.width if c else 0, c.start if c else 0, c.hist if c else 0, n, batch.q_per_seq, rows, batch.block_table.stride(0), M,
+        1 if fp32 else 0, stream_ptr(proj.device))
+    check(code, "eredu_conv_project")
+    return q, out

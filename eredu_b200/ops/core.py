@@ -36,10 +36,11 @@ def linear_ref(x, w, bias=None, residual=None, out_dtype=None, activation=None):
     return y.to(out_dtype or x.dtype)
 
 
-def gated_linear_ref(x, w_gate_up, inter, bias=None, out_dtype=None):
-    """silu(x Wg^T) * (x Wu^T) with Wg = w[:inter], Wu = w[inter:2*inter]."""
+def gated_linear_ref(x, w_gate_up, inter, bias=None, out_dtype=None, activation="silu"):
+    """act(x Wg^T) * (x Wu^T) with Wg = w[:inter], Wu = w[inter:2*inter]."""
     y = F.linear(x.float(), w_gate_up.float(), None if bias is None else bias.float())
-    return (F.silu(y[..., :inter]) * y[..., inter:]).to(out_dtype or x.dtype)
+    act = torch.relu if activation == "relu" else F.silu
+    return (act(y[..., :inter]) * y[..., inter:]).to(out_dtype or x.dtype)
 
 
 def _norm_args(x, row_ssq, norm_eps, want_ssq, n_out):
@@ -107,24 +108,31 @@ def _linear_simt(x, w, bias, out_dtype, activation, out=None):
     assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16) and x.stride(1) == 1 and w.stride(1) == 1
     assert bias is None or (bias.dtype == x.dtype and bias.is_contiguous())
     M, K = x.shape
-    N = w.shape[0]
+    act = {None: 0, "relu2": 1, "gated_silu": 2, "gated_relu": 3}[activation]
+    N = w.shape[0] // 2 if act >= 2 else w.shape[0]
     if out is None:
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
     if M == 0:
         return out
     code = lib().eredu_gemm_simt(ptr(x), ptr(w), ptr(out), ptr(bias), M, N, K, x.stride(0), w.stride(0), out.stride(0),
                                  1 if x.dtype == torch.float32 else 0, 1 if out.dtype == torch.float32 else 0,
-                                 1 if activation == "relu2" else 0, stream_ptr(x.device))
+                                 act, stream_ptr(x.device))
     check(code, "eredu_gemm_simt")
     return out
 
 
-def gated_linear(x, w_gate_up, inter, bias=None, out=None, force_split=0, row_ssq=None, norm_eps=0.0):
-    """Fused SwiGLU up-projection: one GEMM kernel, activation applied in the epilogue (``row_ssq``: see linear)."""
+def gated_linear(x, w_gate_up, inter, bias=None, out=None, force_split=0, row_ssq=None, norm_eps=0.0, activation="silu"):
+    """Fused gated up-projection (SwiGLU; ``activation`` "relu": ReLU of the gate): one GEMM kernel, activation applied in the
+    epilogue (``row_ssq``: see linear). fp32 operands, and bf16 rows a TMA descriptor cannot describe, take the CUDA-core kernel."""
+    if activation not in ("silu", "relu"):
+        raise ValueError(f"unknown activation {activation!r}")
     if not x.is_cuda:
         if row_ssq is not None:
             x = x.float() * torch.rsqrt(row_ssq.sum(-1, keepdim=True) / x.shape[1] + norm_eps)
-        return gated_linear_ref(x, w_gate_up, inter, bias, w_gate_up.dtype)
+        return gated_linear_ref(x, w_gate_up, inter, bias, w_gate_up.dtype, activation)
+    if x.dtype == torch.float32 or not (_tma_rows(x) and _tma_rows(w_gate_up)):
+        assert row_ssq is None, "the CUDA-core linear has no norm fusion"
+        return _linear_simt(x, w_gate_up, bias, x.dtype, "gated_" + activation, out)
     assert x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16
     M, K = x.shape
     if out is None:
@@ -135,7 +143,7 @@ def gated_linear(x, w_gate_up, inter, bias=None, out=None, force_split=0, row_ss
     code = lib().eredu_gemm_bf16(
         ptr(x), ptr(w_gate_up), ptr(out), None, ptr(bias), M, inter, K, x.stride(0), w_gate_up.stride(0),
         out.stride(0), 0, w_gate_up.shape[0], 1, inter, 0, force_split, _sm_count(x.device),
-        ptr(status_word(x.device)), ptr(ssq_in), parts, eps, dim, None, 0, stream_ptr(x.device))
+        ptr(status_word(x.device)), ptr(ssq_in), parts, eps, dim, None, 4 if activation == "relu" else 0, stream_ptr(x.device))
     check(code, "eredu_gemm_bf16(dual)")
     return out
 
@@ -256,6 +264,44 @@ def residual_norm(x, y=None, routed=None, weight=None, bias=None, eps=1e-5, act_
                                      ptr(act), M, W, k, 1 if act_dtype == torch.float32 else 0, 1 if center else 0,
                                      1 if W % 4 == 0 else 0, eps, stream_ptr(x.device))
     check(code, "eredu_residual_norm")
+    return out, act
+
+
+native.register("eredu_branch_norm", native.I, [native.P] * 9 + [native.I] * 4 + [native.F, native.F, native.P])
+
+
+def branch_norm_ref(x, branches, weight, next_weight=None, eps=1e-5, act_dtype=None, branch_weights=None, gain=1.0):
+    def rms(t, w):
+        t = t.float()
+        return t * torch.rsqrt(t.square().mean(-1, keepdim=True) + eps) * w.float()
+
+    y = sum(b.float() if branch_weights is None else rms(b, w) for b, w in zip(branches, branch_weights or branches)) * gain
+    out = x + rms(y, weight)
+    return out, None if next_weight is None else rms(out, next_weight).to(act_dtype or x.dtype)
+
+
+def branch_norm(x, branches, weight, next_weight=None, eps=1e-5, act_dtype=None, branch_weights=None, gain=1.0):
+    """A norm behind a sublayer, the residual sum and the norm in front of the next one, in one launch:
+    ``x' = x + rms(gain * sum_j y_j) * weight``, ``act = rms(x') * next_weight`` in ``act_dtype`` (None without a next weight). One or
+    two ``branches`` y_j in the compute dtype; with ``branch_weights`` each is RMS-normed with its own weight before the sum. x fp32.
+    Returns (x', act)."""
+    if not x.is_cuda:
+        return branch_norm_ref(x, branches, weight, next_weight, eps, act_dtype, branch_weights, gain)
+    M, W = x.shape
+    act_dtype = act_dtype or torch.bfloat16
+    assert x.dtype == torch.float32 and x.is_contiguous() and 1 <= len(branches) <= 2
+    assert all(y.is_contiguous() and y.dtype == act_dtype and y.shape == x.shape for y in branches)
+    ws = list(branch_weights) if branch_weights is not None else [None] * len(branches)
+    assert len(ws) == len(branches) and all(w is None or (w.dtype == torch.float32 and w.numel() == W) for w in (*ws, weight, next_weight))
+    out = torch.empty_like(x)
+    act = torch.empty((M, W), dtype=act_dtype, device=x.device) if next_weight is not None else None
+    if M == 0:
+        return out, act
+    second = len(branches) == 2
+    code = lib().eredu_branch_norm(ptr(x), ptr(branches[0]), ptr(branches[1]) if second else None, ptr(ws[0]), ptr(ws[1]) if second else None,
+                                   ptr(weight), ptr(next_weight), ptr(out), ptr(act), M, W, 1 if act_dtype == torch.float32 else 0,
+                                   1 if W % 4 == 0 else 0, gain, eps, stream_ptr(x.device))
+    check(code, "eredu_branch_norm")
     return out, act
 
 

@@ -430,3 +430,129 @@ def mlstm(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_sl
                              stream_ptr(proj.device))
     check(code, "eredu_mlstm")
     return out
+
+
+native.register("eredu_selective_scan", I, [P] * 15 + [I] * 13 + [P])
+native.register("eredu_selective_scan_scratch_elems", native.L, [I] * 5)
+
+# From this many rows a step size is worth a GEMM of its own in front of the scan (below, the scan multiplies it out).
+SCAN_STEP_GEMM_MIN_ROWS = 64
+
+
+def selective_scan_ref(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_to_slot):
+    c, n = A.shape
+    p = params.float()
+    dt = torch.nn.functional.softplus(p[:, :dt_rank] @ dt_w.float()[:, :dt_rank].t() + dt_b.float())
+    Bm, Cm = p[:, dt_rank:dt_rank + n], p[:, dt_rank + n:dt_rank + 2 * n]
+    xf = x.float()
+    out = torch.zeros((x.shape[0], c), dtype=x.dtype, device=x.device)
+    bounds = _sequences(batch)
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(batch.slots[r0]) < 0:
+            continue
+        cell = state[int(page_to_slot[int(batch.block_table[b, 0])])].view(-1)[:c * n].view(c, n)
+        S = cell.clone()
+        for t in range(r0, r1):
+            S = torch.exp(dt[t][:, None] * A) * S + (dt[t] * xf[t])[:, None] * Bm[t][None, :]
+            y = (S * Cm[t][None, :]).sum(-1) + D * xf[t]
+            out[t] = (y * torch.nn.functional.silu(z[t].float())).to(out.dtype)
+        cell.copy_(S)
+    return out
+
+
+def selective_scan(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_to_slot):
+    """Selective scan (Mamba) over the rows of a ragged batch: per channel c and state n ``S <- exp(dt_c A[c, n]) S + dt_c x_c B_n``,
+    ``y_c = sum_n S[c, n] C_n + D_c x_c``, output ``y silu(z)`` [M, channels].
+    x, z [M, channels]; ``params`` [M, >= dt_rank + 2 n] = [step size input | B | C], ``dt = softplus(dt_w input + dt_b)``; dt_w [channels,
+    dt_rank] in the compute dtype, dt_b, A (negative) [channels, n], D fp32; ``state`` fp32 [slots, >= channels n], in place."""
+    if not x.is_cuda:
+        return selective_scan_ref(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_to_slot)
+    from .core import linear
+
+    c, n = A.shape
+    M = x.shape[0]
+    assert x.is_contiguous() and z.stride(1) == 1 and params.stride(1) == 1 and dt_w.is_contiguous() and dt_w.shape == (c, dt_rank)
+    assert A.is_contiguous() and state.is_contiguous() and all(t.dtype == torch.float32 for t in (A, D, dt_b, state))
+    out = torch.empty((M, c), dtype=x.dtype, device=x.device)
+    if M == 0:
+        return out
+    B = batch.block_table.shape[0]
+    rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
+    dt = linear(params[:, :dt_rank], dt_w, out_dtype=torch.float32) if M >= SCAN_STEP_GEMM_MIN_ROWS else None
+    elems = int(lib().eredu_selective_scan_scratch_elems(c, n, M, B, rows)) if dt is not None else 0
+    scratch = torch.empty(elems, dtype=torch.float32, device=x.device) if elems else None
+    code = lib().eredu_selective_scan(
+        ptr(x), ptr(z), ptr(params), ptr(dt), ptr(dt_w), ptr(dt_b), ptr(A), ptr(D), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table),
+        ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), c, n, dt_rank, z.stride(0), params.stride(0),
+        state[0].numel(), M, B, batch.q_per_seq, rows, batch.block_table.stride(0), 1 if x.dtype == torch.float32 else 0,
+        _sm_count(x.device), stream_ptr(x.device))
+    check(code, "eredu_selective_scan")
+    return out
+
+
+native.register("eredu_general_delta", I, [P] * 12 + [I] * 12 + [F, F, P])
+native.register("eredu_general_delta_scratch_bytes", native.L, [I] * 6)
+
+DELTA_UNIT_EPS = 1e-6        # added to the squared length of a key before it is made a unit vector
+
+
+def general_delta_scan_ref(r, k, v, decay, rate, state):
+    """r, k, decay, rate [T, H, dk], v [T, H, dv], state [H, dk, dv] (fp32). Returns (o [T, H, dv], state)."""
+    u = k / torch.sqrt(k.square().sum(-1, keepdim=True) + DELTA_UNIT_EPS)
+    S, out = state.clone(), []
+    for t in range(r.shape[0]):
+        recalled = torch.einsum("hd,hdv->hv", u[t], S)
+        S = decay[t][:, :, None] * S - (rate[t] * u[t])[:, :, None] * recalled[:, None, :] + k[t][:, :, None] * v[t][:, None, :]
+        out.append(torch.einsum("hd,hdv->hv", r[t], S))
+    return torch.stack(out), S
+
+
+def general_delta_ref(proj, w2, w0, rate_b, norm_w, state, heads, dk, dv, log_decay, eps, batch, page_to_slot):
+    M, qk, vw = proj.shape[0], heads * dk, heads * dv
+    x = proj.float()
+    r, k, v, g, a, low = torch.split(x[:, :3 * qk + 2 * vw + w2.shape[1]], [qk, qk, vw, vw, qk, w2.shape[1]], 1)
+    decay = torch.exp(-log_decay * torch.sigmoid(torch.tanh(low) @ w2.t() + w0)).view(M, heads, dk)
+    rate = torch.sigmoid(a + rate_b).view(M, heads, dk)
+    r, k, v = r.view(M, heads, dk), k.view(M, heads, dk), v.view(M, heads, dv)
+    out = torch.zeros((M, vw), dtype=proj.dtype, device=proj.device)
+    bounds = _sequences(batch)
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(batch.slots[r0]) < 0:
+            continue
+        slot = int(page_to_slot[int(batch.block_table[b, 0])])
+        o, state[slot] = general_delta_scan_ref(r[r0:r1], k[r0:r1], v[r0:r1], decay[r0:r1], rate[r0:r1], state[slot])
+        o = (o * torch.rsqrt(o.square().mean(-1, keepdim=True) + eps)).reshape(r1 - r0, vw) * norm_w
+        out[r0:r1] = (o * torch.sigmoid(g[r0:r1])).to(out.dtype)
+    return out
+
+
+def general_delta(proj, w2, w0, rate_b, norm_w, state, heads, dk, dv, log_decay, eps, batch, page_to_slot):
+    """Generalised delta rule over ``proj`` [M, >= 3 H dk + 2 H dv + rank] = [r | k | v | output gate | removal rate | decay input]. Per
+    head, with the unit key u = k / |k|: ``S <- diag(w) S - (a u) (u^T S) + k v^T`` (both terms read the old state), ``o = S^T r``; decay
+    ``w = exp(-log_decay sigmoid(w2 tanh(input) + w0))`` and removal rate ``a = sigmoid(rate + rate_b)`` per head and key channel. Each
+    head's o is RMS-normed, times ``norm_w`` [H dv] and the sigmoid of the output gate. w2 fp32 [H dk, rank]; ``state`` fp32
+    [slots, H, dk, dv], in place. Returns [M, H dv]."""
+    if not proj.is_cuda:
+        return general_delta_ref(proj, w2, w0, rate_b, norm_w, state, heads, dk, dv, log_decay, eps, batch, page_to_slot)
+    M, rank = proj.shape[0], w2.shape[1]
+    assert proj.stride(1) == 1 and state.is_contiguous() and w2.is_contiguous()
+    assert all(t.dtype == torch.float32 for t in (w2, w0, rate_b, norm_w, state))
+    out = torch.empty((M, heads * dv), dtype=proj.dtype, device=proj.device)
+    if M == 0:
+        return out
+    B = batch.block_table.shape[0]
+    rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
+    scratch = None
+    if proj.dtype == torch.bfloat16 and proj.data_ptr() % 16 == 0 and proj.stride(0) % 8 == 0 and rank % 8 == 0:
+        size = int(lib().eredu_general_delta_scratch_bytes(heads, dk, dv, M, B, rows))
+        if size:
+            scratch = torch.empty(size, dtype=torch.uint8, device=proj.device)
+    code = lib().eredu_general_delta(
+        ptr(proj), ptr(w2), ptr(w0), ptr(rate_b), ptr(norm_w), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table), ptr(page_to_slot),
+        ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv, rank, proj.stride(0), M, B, batch.q_per_seq, rows,
+        batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, _sm_count(proj.device), log_decay, eps,
+        stream_ptr(proj.device))
+    check(code, "eredu_general_delta")
+    return out

@@ -63,16 +63,18 @@ class Engine:
         conv_layers = [li for li in local if self.cfg.layer_is_conv(li)]
         kv_layers = [li for li in local if self.cfg.layer_has_kv(li)]
         _, key_dim, value_dim = self.cfg.kv_cache_dims
-        layer_dims = donors = None
+        layer_dims = donors = layer_pools = None
         if self.cfg.mixers is not None:
             layer_dims = {li: self.cfg.layer_kv_dims(li) for li in kv_layers}
             donors = {li: self.cfg.layer_kv_donor(li) for li in local if self.cfg.layer_kv_donor(li) is not None}
+            layer_pools = {li: self.cfg.layer_kv_pool(li) for li in kv_layers if self.cfg.layer_kv_pool(li)}
         self.kv = PagedKVCache(model.num_local_layers(), model.n_kv_local, key_dim, num_pages, model.dtype,
                                self.device, first_layer=model.first_layer, value_dim=value_dim,
                                attention_layers=kv_layers,
                                conv_layers=conv_layers,
                                conv_channels=self.cfg.hidden_size // model.par.tp_size if conv_layers else 0,
-                               conv_hist=self.cfg.conv_l_cache - 1, layer_dims=layer_dims, donors=donors)
+                               conv_hist=self.cfg.conv_l_cache - 1, layer_dims=layer_dims, donors=donors,
+                               layer_pools=layer_pools)
         # recurrent-state slots: by default twice the decode batch, so that prompts can be prefilled while a batch decodes
         slots = max(2 * max_batch, 8) if state_slots is None else state_slots
         shapes = {li: self.cfg.layer_state_shape(li) for li in local if self.cfg.layer_state_shape(li) is not None}

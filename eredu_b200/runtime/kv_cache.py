@@ -40,10 +40,12 @@ class PageAllocator:
 class PagedKVCache:
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, num_pages: int, dtype, device,
                  first_layer: int = 0, attention_layers=None, conv_layers=None, conv_channels: int = 0, conv_hist: int = 0,
-                 value_dim: Optional[int] = None, layer_dims: Optional[dict] = None, donors: Optional[dict] = None):
+                 value_dim: Optional[int] = None, layer_dims: Optional[dict] = None, donors: Optional[dict] = None,
+                 layer_pools: Optional[dict] = None):
         """``layer_dims``: layer -> (kv heads, key width, value width) for families whose layers differ; layers of one
         geometry share a pool tensor, so a page id is valid in every layer. ``donors``: layer -> the earlier layer whose
-        keys and values it reads (it keeps none of its own).
+        keys and values it reads (it keeps none of its own). ``layer_pools``: layer -> tokens of a block whose mean key and
+        value are kept as well; a page holds the means of the blocks that end in it, so they come and go with the page.
         ``attention_layers`` / ``conv_layers``: global indices of the layers that keep K/V pages respectively a
         short-convolution state (hybrid models); by default every one of the ``n_layers`` layers keeps K/V.
         The convolution state pool [layer, page, conv_hist, channels] is indexed by a sequence's first page."""
@@ -69,6 +71,11 @@ class PagedKVCache:
             self._kv_index.update({li: (g, i) for i, li in enumerate(members)})
         for li, donor in (donors or {}).items():
             self._kv_index[li] = self._kv_index[donor]
+        self.pooled: dict = {}               # layer -> mean keys and values [pages, heads, blocks ending in a page, width]
+        for li, block in (layer_pools or {}).items():
+            k, v = self.layer(li)
+            rows = -(-PAGE // block)
+            self.pooled[li] = tuple(torch.zeros((*t.shape[:2], rows, t.shape[3]), dtype=dtype, device=device) for t in (k, v))
         self.k, self.v = self.pools[0]
         self._conv_index = {li: i for i, li in enumerate(conv_layers or [])}
         self.conv_state = None
@@ -205,6 +212,8 @@ class PagedKVCache:
         """Raised by the features that move pages of one geometry (lower tiers, parking)."""
         if len(self.pools) > 1:
             raise NotImplementedError(f"{what} needs one key / value geometry for all layers; this model has {len(self.pools)}")
+        if self.pooled:
+            raise NotImplementedError(f"{what} does not move pooled keys and values")
 
     def conv_layer(self, li: int):
         return self.conv_state[self._conv_index[li]]
@@ -214,7 +223,8 @@ class PagedKVCache:
         if self.la_rec_state is not None:
             extra += self.la_rec_state.numel() * 4 + self.la_conv_state.numel() * self.la_conv_state.element_size()
         extra += sum(t.numel() * 4 for t in self.layer_state.values())
-        return sum((k.numel() + v.numel()) * k.element_size() for k, v in self.pools) + extra
+        pools = (*self.pools, *self.pooled.values())
+        return sum((k.numel() + v.numel()) * k.element_size() for k, v in pools) + extra
 
     @staticmethod
     def pages_for(tokens: int) -> int:

@@ -263,13 +263,17 @@ def _family_profile(cfg: ModelConfig, weight_bytes, b: int):
     L = cfg.num_hidden_layers
     H = cfg.hidden_size
     if cfg.mixers is not None:
+        from .kv_cache import PAGE
+
         # per-layer geometry: pages of the layers that keep keys and values, fp32 states of the recurrent ones
-        kv = [cfg.layer_kv_dims(li) for li in range(L) if cfg.layer_has_kv(li)]
+        kv = [(li, cfg.layer_kv_dims(li)) for li in range(L) if cfg.layer_has_kv(li)]
         state = sum(math.prod(cfg.layer_state_shape(li)) * 4 for li in range(L) if cfg.layer_state_shape(li) is not None)
         total = sum(math.prod(s) for s in mixer_family(cfg.model_type).tensor_shapes(cfg).values()) * 2
         wb = weight_bytes if weight_bytes is not None else total
         experts = sum(3 * H * m.moe.num_experts * m.moe.moe_intermediate_size * 2 for m in cfg.mixers if m.moe is not None)
-        return ModelResourceProfile(int(wb), int(sum(n * (dk + dv) for n, dk, dv in kv) * b), max(1, len(kv)),
+        # a page also holds the mean key and value of every pooled block that ends in it
+        per_page = sum(n * (dk + dv) * (PAGE + (-(-PAGE // cfg.layer_kv_pool(li)) if cfg.layer_kv_pool(li) else 0)) for li, (n, dk, dv) in kv)
+        return ModelResourceProfile(int(wb), -(-per_page * b // PAGE), max(1, len(kv)),
                                     expert_bytes=int(wb * (experts / total)), state_bytes_per_sequence=int(state))
     if cfg.model_type == "gemma4":
         from ..models.gemma4 import geometry

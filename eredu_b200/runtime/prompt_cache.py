@@ -26,6 +26,7 @@ from typing import Optional
 import numpy as np
 import torch
 
+from .. import ops
 from .kv_cache import PAGE
 
 PROMPT_CACHE_SCHEMA_VERSION = 7
@@ -435,6 +436,8 @@ def load_prompt_cache(engine, directory, tokens, checkpoint_fingerprint: str, sa
                 if tuple(dst.shape) != tuple(t.shape):
                     raise Incompatible(f"fixed-state tensor {e['array']} has shape {tuple(t.shape)}, the model keeps {tuple(dst.shape)}")
                 dst.copy_(t.to(dst.dtype))
+        for li in engine.kv.pooled:
+            ops.pool_cached_blocks(engine.kv, li, engine.cfg.layer_kv_pool(li), seq.pages, usable)
         seq.kv_len = usable
     except Exception:
         engine.release(seq)
