@@ -80,6 +80,8 @@ FAMILY_SOURCES = {
                 "residual_stream", "simt_fp32"),
     "lenitar": ("attention_tc", "gemm_persistent", "gemm_tcgen05", "latent", "latent_attention", "launch_count", "mlstm", "mlstm_chunk",
                 "moe", "residual_stream", "simt_fp32"),
+    "kasuvik": ("attention", "attention_tc", "conv_project", "gemm_persistent", "gemm_tcgen05", "general_delta", "general_delta_chunk",
+                "launch_count", "residual_stream", "selective_scan", "simt_fp32"),
 }
 
 

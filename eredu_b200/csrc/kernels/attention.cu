@@ -12,6 +12,7 @@
 #include "../common/launch.h"
 #include "../common/launch_count.h"
 #include "../common/mma.cuh"
+#include "../common/pooled.cuh"
 #include "../common/ptx.cuh"
 #include "../common/trace.cuh"
 
@@ -56,6 +57,11 @@ struct AttnParams {
   // splits > 1: 1 = the `splits` CTAs of a (sequence, kv head) form a thread-block cluster and combine their partial
   // results through distributed shared memory (no global scratch, no arrival tickets); 0 = scratch + last-arriver.
   int cluster_reduce;
+  // decode with window > 0 over blocks as well: mean keys and values of blocks of `pool` tokens, [pages, n_kv_heads, pool_rows, width] at
+  // the page of a block's last token; a query sees those that end before its window
+  const __nv_bfloat16* pk;
+  const __nv_bfloat16* pv;
+  int pool, pool_rows;
 };
 constexpr int kMaxFusedNew = 8;       // new tokens per sequence the fused (RoPE + append) decode path handles
 constexpr int kMaxClusterSplits = 8;  // portable cluster size
@@ -349,8 +355,9 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(AttnParams p) {
 // cp.async ring and keeps private (m, l, O); the warps are merged through shared memory at the end.
 // Keys and values may differ in width: tiles are DK / DV wide (64 or 128), rows of the cache dk / dv (the rest of a
 // tile row is zero-filled, which adds nothing to scores or outputs). EXT = false is the common case with everything beyond
-// it folded away: one head size that fills the tile, no chunks, the preparation of rope_kv.
-template <int DK, int DV, int MT, bool EXT>
+// it folded away: one head size that fills the tile, no chunks, the preparation of rope_kv. POOL: sixteen pooled blocks at a time are
+// walked like a page, in front of the pages of the window.
+template <int DK, int DV, int MT, bool EXT, bool POOL>
 __global__ void __launch_bounds__(128, MT == 1 ? (DK + DV <= 128 ? 5 : 4) : 1) attn_decode_kernel(AttnParams p) {
   const int dk = EXT ? p.dk : DK, dv = EXT ? p.dv : DV;
   const bool norm_whole = EXT && p.norm_whole, value_norm = EXT && p.value_norm;
@@ -383,9 +390,12 @@ __global__ void __launch_bounds__(128, MT == 1 ? (DK + DV <= 128 ? 5 : 4) : 1) a
   // pages before the first query's window / chunk hold nothing any query of this launch can see
   const int first_pos = kv_len - p.q_per_seq + p.t0;
   const int first_page = max(0, lowest_key<EXT>(p, first_pos)) / kPage;
-  int pps = (npages - first_page + p.splits - 1) / p.splits;
+  // POOL: entries in front of first_page stand for sixteen blocks each (-1 the last sixteen, and so on back)
+  const int blocks = POOL ? pooled_seen(first_pos + p.t_count - 1, p.window, p.pool) : 0;
+  const int base_page = first_page - (POOL ? (blocks + kPage - 1) / kPage : 0);
+  int pps = (npages - base_page + p.splits - 1) / p.splits;
   pps = (pps + 3) & ~3;
-  const int page0 = first_page + split * pps;
+  const int page0 = base_page + split * pps;
   const int page1 = min(npages, page0 + pps);
 
   const bool fused = p.qkv != nullptr;
@@ -409,6 +419,22 @@ __global__ void __launch_bounds__(128, MT == 1 ? (DK + DV <= 128 ? 5 : 4) : 1) a
 
   uint8_t* my_ring = ring + warp * NSTAGE * STAGE_BYTES;
   auto load_page = [&](int pg, int stage) {
+    if (POOL && pg < first_page) {
+      if (pg >= page1) return;
+      const int b0 = (pg - base_page) * kPage;
+      uint8_t* kd = my_ring + stage * STAGE_BYTES;
+      uint8_t* vd = kd + KPAGE_BYTES;
+      for (int i = lane; i < kPage * (CHK + CHV); i += 32) {
+        const bool is_v = i >= kPage * CHK;
+        const int e = is_v ? i - kPage * CHK : i, r = is_v ? e / CHV : e / CHK, c = is_v ? e % CHV : e % CHK, d = is_v ? dv : dk;
+        const bool in = c * 8 < d && b0 + r < blocks;
+        const PooledRow at = pooled_row(in ? b0 + r : 0, p.pool);
+        const size_t row = (static_cast<size_t>(bt[at.page]) * p.n_kv_heads + kvh) * p.pool_rows + at.row;
+        const __nv_bfloat16* src = (is_v ? p.pv : p.pk) + row * d + (in ? c * 8 : 0);
+        cp_async16(is_v ? vd + swz<DV>(r, c) : kd + swz<DK>(r, c), src, in ? 16 : 0);
+      }
+      return;
+    }
     if (pg < page1) {
       const int phys = bt[pg];
       const __nv_bfloat16* ksrc = p.k_cache + (static_cast<size_t>(phys) * p.n_kv_heads + kvh) * kPage * dk;
@@ -590,6 +616,7 @@ __global__ void __launch_bounds__(128, MT == 1 ? (DK + DV <= 128 ? 5 : 4) : 1) a
           const int qp = kv_len - p.q_per_seq + p.t0 + r / group;
           bool ok = (r < rows) && (j <= qp) && (j < kv_len);
           ok = ok && (j >= lowest_key<EXT>(p, qp));
+          if (POOL && pg < first_page) ok = (r < rows) && (j - kv0 + (pg - base_page) * kPage < pooled_seen(qp, p.window, p.pool));
           const float v = ok ? s[mt][nt][e] * p.scale_log2 : -INFINITY;
           s[mt][nt][e] = v;
           mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -870,10 +897,10 @@ extern "C" int eredu_attn_prefill(const void* q, const void* k_cache, const void
   return static_cast<int>(e);
 }
 
-template <int DK, int DV, int MT, bool EXT>
+template <int DK, int DV, int MT, bool EXT, bool POOL = false>
 static cudaError_t launch_decode(const AttnParams& p, dim3 grid, cudaStream_t stream) {
   static bool cfg[kMaxDevices] = {};
-  if (!configure_once(cfg, attn_decode_kernel<DK, DV, MT, EXT>, decode_smem<DK, DV, MT>())) return cudaErrorInvalidValue;
+  if (!configure_once(cfg, attn_decode_kernel<DK, DV, MT, EXT, POOL>, decode_smem<DK, DV, MT>())) return cudaErrorInvalidValue;
   cudaLaunchConfig_t lc = {};
   lc.gridDim = grid;
   lc.blockDim = dim3(128);
@@ -895,7 +922,7 @@ static cudaError_t launch_decode(const AttnParams& p, dim3 grid, cudaStream_t st
   }
   lc.attrs = attr;
   lc.numAttrs = nattr;
-  const cudaError_t e = cudaLaunchKernelEx(&lc, attn_decode_kernel<DK, DV, MT, EXT>, p);
+  const cudaError_t e = cudaLaunchKernelEx(&lc, attn_decode_kernel<DK, DV, MT, EXT, POOL>, p);
   eredu_count_launches(1);
   return e;
 }
@@ -929,7 +956,15 @@ static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_hea
                        (p.qkv == nullptr || p.append);
 #define ER_DECODE(DK_, DV_, EXT_) \
   e = one ? launch_decode<DK_, DV_, 1, EXT_>(p, grid, stream) : launch_decode<DK_, DV_, 2, EXT_>(p, grid, stream)
-    if (plain && key_dim == 128) ER_DECODE(128, 128, false);
+    if (p.pool > 0) {
+#define ER_POOLED(DK_, DV_) \
+  e = one ? launch_decode<DK_, DV_, 1, true, true>(p, grid, stream) : launch_decode<DK_, DV_, 2, true, true>(p, grid, stream)
+      if (key_dim > 64 && value_dim > 64) ER_POOLED(128, 128);
+      else if (key_dim > 64) ER_POOLED(128, 64);
+      else if (value_dim > 64) ER_POOLED(64, 128);
+      else ER_POOLED(64, 64);
+#undef ER_POOLED
+    } else if (plain && key_dim == 128) ER_DECODE(128, 128, false);
     else if (plain) ER_DECODE(64, 64, false);
     else if (key_dim > 64 && value_dim > 64) ER_DECODE(128, 128, true);
     else if (key_dim > 64) ER_DECODE(128, 64, true);
@@ -976,6 +1011,34 @@ extern "C" int eredu_attn_decode(const void* q, const void* k_cache, const void*
                                  cudaStream_t stream) {
   return attn_decode_impl(q, k_cache, v_cache, out, block_table, seq_lens, sinks, part_o, part_ml, counters, batch, q_per_seq,
                           max_pages, n_q_heads, n_kv_heads, key_dim, value_dim, splits, window, chunk, scale, stream, false);
+}
+
+// Decode attention over the `window` newest tokens and the means of the blocks of `pool` tokens that end before them. pk / pv:
+// [pages, n_kv_heads, pool_rows, width], see pooled.cuh. At most 8 splits.
+extern "C" int eredu_attn_decode_pooled(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, void* out,
+                                        const int* block_table, const int* seq_lens, int batch, int q_per_seq, int max_pages, int n_q_heads,
+                                        int n_kv_heads, int key_dim, int value_dim, int splits, int window, int pool, int pool_rows,
+                                        float scale, cudaStream_t stream) {
+  if (window <= 0 || pool <= 0 || pool_rows < (kPage + pool - 1) / pool || splits > kMaxClusterSplits) return -1;
+  AttnParams p = {};
+  p.q = static_cast<const __nv_bfloat16*>(q);
+  p.k_cache = static_cast<const __nv_bfloat16*>(k_cache);
+  p.v_cache = static_cast<const __nv_bfloat16*>(v_cache);
+  p.pk = static_cast<const __nv_bfloat16*>(pk);
+  p.pv = static_cast<const __nv_bfloat16*>(pv);
+  p.out = static_cast<__nv_bfloat16*>(out);
+  p.block_table = block_table;
+  p.seq_lens = seq_lens;
+  p.max_pages = max_pages;
+  p.n_q_heads = n_q_heads;
+  p.n_kv_heads = n_kv_heads;
+  p.q_per_seq = q_per_seq;
+  p.splits = splits < 1 ? 1 : splits;
+  p.window = window;
+  p.pool = pool;
+  p.pool_rows = pool_rows;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  return launch_decode_all(p, batch, q_per_seq, n_q_heads, n_kv_heads, key_dim, value_dim, stream);
 }
 
 // Decode attention that starts from the projection output: qkv [batch * q_per_seq, ld_qkv] = [q heads | k heads |

@@ -30,6 +30,7 @@
 #include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
+#include "../common/pooled.cuh"
 #include "../common/ptx.cuh"
 #include "../common/tma_host.h"
 #include "../common/trace.cuh"
@@ -55,6 +56,9 @@ struct AttnTcParams {
   const __nv_bfloat16* gate;   // optional [tokens, ldg]: column head * dv + i
   long long ldg;
   int rot;
+  // POOL form (window > 0): all whole blocks of `pool` tokens of a sequence as dense rows from pool_first[b] on
+  const int* pool_first;
+  int pool;
 };
 
 constexpr int kTcThreads = 320;
@@ -113,11 +117,13 @@ __device__ __forceinline__ int tc_query_tile(const AttnTcParams& p, int tiles, i
   return y * per;
 }
 
-// NK / NV: 64-wide halves of the key and of the value width
-template <int NK, int NV, bool ROWS>
+// NK / NV: 64-wide halves of the key and of the value width. POOL: key tiles of 128 mean keys come in front of the tiles of the window; tile
+// index u walks the pooled tiles 0 .. pooled - 1, then the token tiles from j0 on.
+template <int NK, int NV, bool ROWS, bool POOL>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                       const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR, const AttnTcParams p) {
+                       const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR,
+                       const __grid_constant__ CUtensorMap tmS, const AttnTcParams p) {
   constexpr int VST = tc_v_stages(NK, NV);
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -157,6 +163,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   const int j0_a = tc_lowest_key(p, pos0) / kTcTile;
   const int j0_b = tc_lowest_key(p, pos0 + kTcTile) / kTcTile;
   const int j0 = n_b > 0 ? min(j0_a, j0_b) : j0_a;
+  // pooled tiles some row of query tile a, b sees (the last row sees most)
+  const int np_a = POOL ? (pooled_seen(min(kv_len - 1, pos0 + kTcTile - 1), p.window, p.pool) + kTcTile - 1) / kTcTile : 0;
+  const int np_b = POOL && n_b > 0 ? (pooled_seen(min(kv_len - 1, pos0 + kTcRows - 1), p.window, p.pool) + kTcTile - 1) / kTcTile : 0;
+  const int pooled = max(np_a, np_b);
+  const int total = pooled + n_tiles - j0;                              // tiles this CTA walks
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -173,7 +184,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     tma_prefetch_desc(&tmQ);
     tma_prefetch_desc(&tmK);
     tma_prefetch_desc(&tmV);
-    if (ROWS) tma_prefetch_desc(&tmR);
+    if (ROWS || POOL) tma_prefetch_desc(&tmR);
+    if (POOL) tma_prefetch_desc(&tmS);
   }
   if (warp == 0) {
     tmem_alloc(tmem_slot, 512);
@@ -197,13 +209,15 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           // ROWS: the last half starts where the shared part does; a box that reaches beyond the per-head part meets zeros on the key side
           tma_load_3d(q_s + (w * NK + h) * kTcHalf, &tmQ, ROWS && h == NK - 1 ? p.dk - p.rot : h * 64, head, q0 + row0 + w * kTcTile, q_full);
       const int* pages = p.block_table + static_cast<size_t>(b) * p.max_pages;
-      for (int jj = 0; j0 + jj < n_tiles && ok; ++jj) {
-        const int j = j0 + jj;                                           // key tile; jj counts this CTA's iterations
+      const int pool_row = POOL ? p.pool_first[b] : 0;
+      for (int jj = 0; jj < total && ok; ++jj) {
+        const bool means = POOL && jj < pooled;
+        const int j = means ? jj : j0 + jj - pooled;                     // key tile; jj counts this CTA's iterations
         const int s = jj & 1;
         const uint32_t reuse_parity = ((jj >> 1) - 1) & 1;
         const int sv = VST == 2 ? s : 0;
         int page[8];
-        if (!ROWS) {
+        if (!ROWS && !means) {
 #pragma unroll
           for (int pg = 0; pg < 8; ++pg) {
             const int page_index = j * 8 + pg;
@@ -217,17 +231,25 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           for (int h = 0; h + 1 < NK; ++h) tma_load_3d(k_s + (s * NK + h) * kTcHalf, &tmK, h * 64, head, seq.z + j * kTcTile, &k_full[s]);
           tma_load_2d(k_s + (s * NK + NK - 1) * kTcHalf, &tmR, 0, seq.z + j * kTcTile, &k_full[s]);
         }
+        if (means) {
+          for (int h = 0; h < NK; ++h) tma_load_3d(k_s + (s * NK + h) * kTcHalf, &tmR, h * 64, kv_head, pool_row + j * kTcTile, &k_full[s]);
+        } else {
 #pragma unroll
-        for (int pg = 0; pg < (ROWS ? 0 : 8); ++pg)
-          for (int h = 0; h < NK; ++h) tma_load_4d(k_s + (s * NK + h) * kTcHalf + pg * 2048, &tmK, h * 64, 0, kv_head, page[pg], &k_full[s]);
+          for (int pg = 0; pg < (ROWS ? 0 : 8); ++pg)
+            for (int h = 0; h < NK; ++h) tma_load_4d(k_s + (s * NK + h) * kTcHalf + pg * 2048, &tmK, h * 64, 0, kv_head, page[pg], &k_full[s]);
+        }
         if (jj >= VST) ok = mbar_wait(&v_empty[sv], VST == 2 ? reuse_parity : (jj - 1) & 1, p.status, kStatusSmemEmptyTimeout);
         if (!ok) break;
         mbar_arrive_expect_tx(&v_full[sv], NV * kTcHalf);
         if (ROWS)
           for (int h = 0; h < NV; ++h) tma_load_3d(v_s + (sv * NV + h) * kTcHalf, &tmV, h * 64, head, seq.z + j * kTcTile, &v_full[sv]);
+        if (means) {
+          for (int h = 0; h < NV; ++h) tma_load_3d(v_s + (sv * NV + h) * kTcHalf, &tmS, h * 64, kv_head, pool_row + j * kTcTile, &v_full[sv]);
+        } else {
 #pragma unroll
-        for (int pg = 0; pg < (ROWS ? 0 : 8); ++pg)
-          for (int h = 0; h < NV; ++h) tma_load_4d(v_s + (sv * NV + h) * kTcHalf + pg * 2048, &tmV, h * 64, 0, kv_head, page[pg], &v_full[sv]);
+          for (int pg = 0; pg < (ROWS ? 0 : 8); ++pg)
+            for (int h = 0; h < NV; ++h) tma_load_4d(v_s + (sv * NV + h) * kTcHalf + pg * 2048, &tmV, h * 64, 0, kv_head, page[pg], &v_full[sv]);
+        }
       }
     }
   } else if (warp == 1) {
@@ -255,23 +277,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           umma_f16_ts(tmem + 256 + w * 128, tmem + w * 128 + kk * 8, umma_desc_mn_sw128(va + kk * 2048, kTcHalf), kIdescPV,
                       (!fresh || kk > 0) ? 1u : 0u);
       };
-      auto active = [&](int w, int j) { return j >= first[w] && j < last[w]; };
+      const int seen[2] = {np_a, np_b};
+      // u counts this CTA's iterations; a query tile's last one is a token tile
+      auto active = [&](int w, int u) { return POOL && u < pooled ? u < seen[w] : u >= pooled + first[w] - j0 && u < pooled + last[w] - j0; };
       ok = mbar_wait(q_full, 0, p.status, kStatusTmaFullTimeout);
       if (ok) ok = mbar_wait(&k_full[0], 0, p.status, kStatusTmaFullTimeout);
       if (ok) {
         tc_fence_after_sync();
-        if (active(0, j0)) issue_s(0, 0);
-        if (active(1, j0)) issue_s(1, 0);
+        if (active(0, 0)) issue_s(0, 0);
+        if (active(1, 0)) issue_s(1, 0);
         umma_commit(&k_empty[0]);
       }
       int done[2] = {0, 0};                        // softmax rounds completed per tile: parity of p_full
-      for (int jj = 0; j0 + jj < n_tiles && ok; ++jj) {
-        const int j = j0 + jj;
-        const bool next = j + 1 < n_tiles;
+      for (int jj = 0; jj < total && ok; ++jj) {
+        const bool next = jj + 1 < total;
         bool k_ready = false;
         ok = mbar_wait(&v_full[VST == 2 ? jj & 1 : 0], (VST == 2 ? jj >> 1 : jj) & 1, p.status, kStatusTmaFullTimeout);
         for (int w = 0; w < 2 && ok; ++w) {
-          if (active(w, j)) {
+          if (active(w, jj)) {
             ok = mbar_wait(&p_full[w], done[w] & 1, p.status, kStatusAccumTimeout);   // P_w(j) is in tensor memory, O_w is rescaled
             if (!ok) break;
             tc_fence_after_sync();
@@ -279,7 +302,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             ++done[w];
           }
           if (w == 1) umma_commit(&v_empty[VST == 2 ? jj & 1 : 0]);
-          if (active(w, j + 1)) {
+          if (active(w, jj + 1)) {
             if (!k_ready) {
               ok = mbar_wait(&k_full[(jj + 1) & 1], ((jj + 1) >> 1) & 1, p.status, kStatusTmaFullTimeout);
               if (!ok) break;
@@ -287,7 +310,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
               k_ready = true;
             }
             issue_s(w, jj + 1);
-          } else if (j + 1 == last[w]) {
+          } else if (jj + 1 == pooled + last[w] - j0) {
             umma_commit(&o_final[w]);
           }
         }
@@ -308,8 +331,10 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const uint32_t s_addr = tmem + lane_addr + w * 128;
     const uint32_t o_addr = tmem + lane_addr + 256 + w * 128;
     float m = -INFINITY, l = 0.f;                                        // -inf: this row has not seen a key yet
-    for (int j = j0_w; j < n_w && ok; ++j) {
-      const int it = j - j0_w;                                           // this tile's round: parity of its barriers
+    const int np_w = w == 0 ? np_a : np_b;
+    for (int it = 0; it < np_w + n_w - j0_w && ok; ++it) {               // this tile's round: parity of its barriers
+      const bool means = POOL && it < np_w;
+      const int j = means ? it : j0_w + it - np_w;
       ok = mbar_wait(&s_full[w], it & 1, p.status, kStatusAccumTimeout);
       if (!ok) break;
       tc_fence_after_sync();
@@ -319,7 +344,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       tmem_wait_ld();
       const int key0 = j * kTcTile;
       const bool before = key0 < tc_lowest_key(p, tile_pos0 + kTcTile - 1);     // some row's visible keys start inside or after this tile
-      if (key0 + kTcTile - 1 > tile_pos0 || key0 + kTcTile > kv_len || before) {   // some (row, key) of the tile is masked: -inf gives p = 0
+      if (means) {
+        const int blocks = pooled_seen(qpos, p.window, p.pool) - key0;   // of this tile's
+        if (key0 + kTcTile > pooled_seen(tile_pos0, p.window, p.pool)) {
+#pragma unroll
+          for (int c = 0; c < 8; ++c)
+#pragma unroll
+            for (int i = 0; i < 16; ++i)
+              if (c * 16 + i >= blocks) sc[c][i] = 0xFF800000u;
+        }
+      } else if (key0 + kTcTile - 1 > tile_pos0 || key0 + kTcTile > kv_len || before) {   // some (row, key) of the tile is masked: -inf gives p = 0
         const int visible = min(qpos, kv_len - 1) - key0;                // keys hidden .. visible of this tile are seen by this row
         const int hidden = tc_lowest_key(p, qpos) - key0;
 #pragma unroll
@@ -436,23 +470,23 @@ using namespace eredu;
 // Causal prefill attention over the paged cache, key / value widths up to 128, optional window or chunks and sink logits.
 // q: [tokens, n_q, key_dim] bf16 (contiguous); k_cache / v_cache: [pages, n_kv, 16, width] bf16 (contiguous); sinks: fp32 [n_q] or
 // null. Same arguments as eredu_attn_prefill otherwise. Returns -2 for shapes it does not take.
-template <int NK, int NV, bool ROWS = false>
-static int launch_attn_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmR,
+template <int NK, int NV, bool ROWS = false, bool POOL = false>
+static int launch_attn_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmR, const CUtensorMap& tmS,
                           const AttnTcParams& p, dim3 grid, cudaStream_t stream) {
   static bool configured[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<NK, NV, ROWS>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(NK, NV)) != cudaSuccess) return -1;
+    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<NK, NV, ROWS, POOL>, cudaFuncAttributeMaxDynamicSharedMemorySize, tc_smem(NK, NV)) != cudaSuccess) return -1;
     configured[dev] = true;
   }
-  return static_cast<int>(launch_pdl(attn_prefill_tc_kernel<NK, NV, ROWS>, grid, dim3(kTcThreads), tc_smem(NK, NV), stream, tmQ, tmK, tmV, tmR, p));
+  return static_cast<int>(launch_pdl(attn_prefill_tc_kernel<NK, NV, ROWS, POOL>, grid, dim3(kTcThreads), tc_smem(NK, NV), stream, tmQ, tmK, tmV, tmR, tmS, p));
 }
 
-extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
-                                     const int* seq_lens, const int* cu_q, const float* sinks, int batch, int total_q, int max_q_len,
-                                     int max_pages, int num_pages, int n_q_heads, int n_kv_heads, int key_dim, int value_dim, int window,
-                                     int chunk, float scale, int* status, cudaStream_t stream) {
+static int attn_prefill_tc_impl(const void* q, const void* k_cache, const void* v_cache, const void* k_rows, const void* v_rows, void* out,
+                                const int* block_table, const int* seq_lens, const int* cu_q, const int* pool_first, const float* sinks, int batch,
+                                int total_q, int max_q_len, int max_pages, int num_pages, int rows, int n_q_heads, int n_kv_heads, int key_dim,
+                                int value_dim, int window, int chunk, int pool, float scale, int* status, cudaStream_t stream) {
   if (key_dim <= 0 || key_dim > 128 || key_dim % 8 != 0 || value_dim <= 0 || value_dim > 128 || value_dim % 8 != 0 || batch <= 0 ||
       total_q <= 0 || n_kv_heads <= 0 || n_q_heads % n_kv_heads != 0 || window < 0 || chunk < 0)
     return -2;
@@ -485,10 +519,50 @@ extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const v
   p.status = status;
   dim3 grid(n_q_heads, (max_q_len + kTcRows - 1) / kTcRows, batch);
   int e;
-  if (key_dim > 64) e = value_dim > 64 ? launch_attn_tc<2, 2>(tmQ, tmK, tmV, tmK, p, grid, stream) : launch_attn_tc<2, 1>(tmQ, tmK, tmV, tmK, p, grid, stream);
-  else e = value_dim > 64 ? launch_attn_tc<1, 2>(tmQ, tmK, tmV, tmK, p, grid, stream) : launch_attn_tc<1, 1>(tmQ, tmK, tmV, tmK, p, grid, stream);
+  if (pool > 0) {
+    // no whole block anywhere yet: the maps of the caches stand in, and no tile of means is walked
+    CUtensorMap tmR = tmK, tmS = tmV;
+    const uint64_t G = static_cast<uint64_t>(n_kv_heads), n = static_cast<uint64_t>(rows);
+    if (rows > 0) {
+      r = make_tma_3d(&tmR, k_rows, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, D, G, n, D * 2, G * D * 2, 64, 1, 128);
+      if (r != 0) return -400 + r;
+      r = make_tma_3d(&tmS, v_rows, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, V, G, n, V * 2, G * V * 2, 64, 1, 128);
+      if (r != 0) return -500 + r;
+    }
+    p.pool = pool;
+    p.pool_first = pool_first;
+#define ER_POOLED(NK_, NV_) e = launch_attn_tc<NK_, NV_, false, true>(tmQ, tmK, tmV, tmR, tmS, p, grid, stream)
+    if (key_dim > 64 && value_dim > 64) ER_POOLED(2, 2);
+    else if (key_dim > 64) ER_POOLED(2, 1);
+    else if (value_dim > 64) ER_POOLED(1, 2);
+    else ER_POOLED(1, 1);
+#undef ER_POOLED
+    eredu_count_launches(1);
+    return e;
+  }
+  if (key_dim > 64) e = value_dim > 64 ? launch_attn_tc<2, 2>(tmQ, tmK, tmV, tmK, tmV, p, grid, stream) : launch_attn_tc<2, 1>(tmQ, tmK, tmV, tmK, tmV, p, grid, stream);
+  else e = value_dim > 64 ? launch_attn_tc<1, 2>(tmQ, tmK, tmV, tmK, tmV, p, grid, stream) : launch_attn_tc<1, 1>(tmQ, tmK, tmV, tmK, tmV, p, grid, stream);
   eredu_count_launches(1);
   return e;
+}
+
+extern "C" int eredu_attn_prefill_tc(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                                     const int* seq_lens, const int* cu_q, const float* sinks, int batch, int total_q, int max_q_len,
+                                     int max_pages, int num_pages, int n_q_heads, int n_kv_heads, int key_dim, int value_dim, int window,
+                                     int chunk, float scale, int* status, cudaStream_t stream) {
+  return attn_prefill_tc_impl(q, k_cache, v_cache, nullptr, nullptr, out, block_table, seq_lens, cu_q, nullptr, sinks, batch, total_q, max_q_len,
+                              max_pages, num_pages, 0, n_q_heads, n_kv_heads, key_dim, value_dim, window, chunk, 0, scale, status, stream);
+}
+
+// The POOL form: over the `window` newest tokens and the means of the blocks of `pool` tokens that end before them. k_rows / v_rows [rows,
+// n_kv, width] bf16: all whole blocks of sequence b from row pool_first[b] on (null when rows = 0: no sequence has one).
+extern "C" int eredu_attn_prefill_tc_pooled(const void* q, const void* k_cache, const void* v_cache, const void* k_rows, const void* v_rows, void* out,
+                                            const int* block_table, const int* seq_lens, const int* cu_q, const int* pool_first, int batch,
+                                            int total_q, int max_q_len, int max_pages, int num_pages, int rows, int n_q_heads, int n_kv_heads,
+                                            int key_dim, int value_dim, int window, int pool, float scale, int* status, cudaStream_t stream) {
+  if (window <= 0 || pool <= 0 || rows < 0 || pool_first == nullptr || (rows > 0 && (k_rows == nullptr || v_rows == nullptr))) return -2;
+  return attn_prefill_tc_impl(q, k_cache, v_cache, k_rows, v_rows, out, block_table, seq_lens, cu_q, pool_first, nullptr, batch, total_q, max_q_len,
+                              max_pages, num_pages, rows, n_q_heads, n_kv_heads, key_dim, value_dim, window, 0, pool, scale, status, stream);
 }
 
 // The ROWS form. q [total_q rows of ldq elements], head h at column h * (dim + rot): [per-head part (dim) | shared part (rot)]; k [rows of
@@ -533,7 +607,7 @@ extern "C" int eredu_attn_prefill_rows(const void* q, const void* k, const void*
   if (grid.y > 65535) return -2;
   int e;
 #define ER_ROWS(NK_) \
-  e = value_dim > 64 ? launch_attn_tc<NK_, 2, true>(tmQ, tmK, tmV, tmR, p, grid, stream) : launch_attn_tc<NK_, 1, true>(tmQ, tmK, tmV, tmR, p, grid, stream)
+  e = value_dim > 64 ? launch_attn_tc<NK_, 2, true>(tmQ, tmK, tmV, tmR, tmV, p, grid, stream) : launch_attn_tc<NK_, 1, true>(tmQ, tmK, tmV, tmR, tmV, p, grid, stream)
   if (dim > 64) ER_ROWS(3);
   else ER_ROWS(2);
 #undef ER_ROWS

@@ -49,7 +49,7 @@ struct PGemmParams {
   float norm_eps;
   float norm_inv_dim;
   float* ssq_out;
-  int act;  // plain tiles: 2 = squared ReLU before the residual
+  int act;  // plain tiles: 2 = squared ReLU before the residual; dual tiles: 0 = silu(g) * u, 3 = relu(g) * u
   int n_tiles, m_tiles;
   // grouped form: m_tiles work items, used ones first (the rest have no rows); the expert's weights start at row expert * w_rows_per_expert
   const int4* work;
@@ -283,7 +283,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
             const float4 u1 = *reinterpret_cast<const float4*>(st + c * 128 + 64 + n0 + 4);
             const float u[8] = {u0.x, u0.y, u0.z, u0.w, u1.x, u1.y, u1.z, u1.w};
 #pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = silu_f(v[j]) * u[j];
+            for (int j = 0; j < 8; ++j) v[j] = (p.act == 3 ? fmaxf(v[j], 0.f) : silu_f(v[j])) * u[j];
           }
           if (!DUAL && p.act == 2) {
 #pragma unroll

@@ -58,7 +58,7 @@ struct GemmParams {
   // Large token tiles: the epilogue goes through shared memory so that the output (and the residual) move as
   // 16-byte row chunks instead of one 2-byte element per thread. Needs 16-byte aligned rows (host-checked).
   int staged;
-  // Plain tiles: 2 = squared ReLU of the output (after bias, before the residual). Gated activation of DUAL tiles: 0 = silu(g) * u (SwiGLU); 1 = g * sigmoid(1.702 g) * (u + 1) (GPT-OSS). With
+  // Plain tiles: 2 = squared ReLU of the output (after bias, before the residual). Gated activation of DUAL tiles: 0 = silu(g) * u (SwiGLU); 1 = g * sigmoid(1.702 g) * (u + 1) (GPT-OSS); 3 = relu(g) * u. With
   // act_limit > 0 the gate is clamped from above and the linear branch to [-limit, limit] first
   // (eredu/src/backend/mlx/architectures/gpt_oss/model.rs:748-753; nn/moe.rs swiglu_limit).
   int act;
@@ -107,6 +107,7 @@ __device__ __forceinline__ float gated_act(const GemmParams& p, float g, float u
     u = fminf(fmaxf(u, -p.act_limit), p.act_limit);
   }
   if (p.act == 1) return g / (1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+  if (p.act == 3) return fmaxf(g, 0.f) * u;
   return silu_f(g) * u;
 }
 
@@ -801,7 +802,7 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   if (tn == 256 && !out_fp32 && force_split <= 1 && persistent_enabled()) {
     // prefill-sized: persistent kernel with double-buffered accumulators
     const int pr = launch_gemm_persistent(X, W, Y, residual, bias, M, N, K, ldx, ldw, ldy, ldr, w_rows, dual, dual_row_offset,
-                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, (flags & 2) ? 2 : 0,
+                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : 0,
                                          stream);
     if (pr != kPersistentUnsupported) return pr;
   }
@@ -831,10 +832,10 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   p.work = nullptr;
   p.w_rows_per_expert = 0;
   p.staged = 0;
-  p.act = (flags & 2) && !dual ? 2 : 0;
+  p.act = dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : 0;
   p.act_limit = 0.f;
   p.bias_expert_stride = 0;
-  // flag bit 1: squared ReLU of the output (plain tiles). Flag bit 0: W was produced by a preceding kernel of the stream (no early fetch at all). Otherwise the ring's
+  // flag bit 1: squared ReLU of the output (plain tiles). Flag bit 2: ReLU instead of SiLU of the gate (dual tiles). Flag bit 0: W was produced by a preceding kernel of the stream (no early fetch at all). Otherwise the ring's
   // first stages are fetched before the dependency wait (level 1), and for matrices that fit L2 many times over
   // the remaining tiles are prefetched into L2 as well (level 2). EREDU_GEMM_PREFETCH overrides the level.
   p.w_static = (flags & 1) ? 0 : prefetch_level(static_cast<long long>(w_rows) * K * 2);

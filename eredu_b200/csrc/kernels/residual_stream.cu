@@ -2,6 +2,8 @@
 //   * residual_norm: x' = x + y + the weighted expert rows of the token, and LayerNorm or RMSNorm of x' for the next layer
 //   * rms_residual (a norm on a sublayer's OUTPUT): x = residual + w * y / rms(y), in fp32, plus the copy of x in the compute dtype that the next
 //     projections read (one number or one vector as w; without a residual: a plain norm, as in front of the head)
+//   * branch_norm (norms in front of and behind a sublayer): x' = x + w rms(gain (y0 + y1)), the branches normed by themselves first
+//     where they have weights, and the norm of x' in front of the next sublayer
 //   * embedding_stream: the first rows of the stream and their copy
 //   * qkv_prepare: RMSNorm over the WHOLE query and key projections, rotation of the leading dims of every head, RMSNorm of
 //     every value head, and the append to the paged cache, whose key and value widths may differ
@@ -216,6 +218,163 @@ static cudaError_t launch_residual_norm(const ResidualNormParams& p, int M, bool
 #undef ER_RN
 }
 
+struct BranchNormParams {
+  const float* x;           // [M, W]
+  const void* y0;           // [M, W]
+  const void* y1;           // [M, W] or null
+  const float* w0;          // [W] norms of the branches, or null
+  const float* w1;
+  const float* weight;      // [W] norm of their sum
+  const float* next;        // [W] or null: no activations
+  float* x_out;
+  void* act;
+  int W;
+  float gain, eps;
+};
+
+// Sums of two values over the block.
+__device__ __forceinline__ float2 block_sum2_f32(float a, float b, float2* red) {
+  a = warp_sum_f32(a);
+  b = warp_sum_f32(b);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) t.x += red[w].x, t.y += red[w].y;
+  __syncthreads();
+  return t;
+}
+
+// x' = x + rms(gain (y0 + y1)) weight (each branch RMS-normed by itself first where it has a weight), act = rms(x') next. One CTA per row;
+// NV groups of four columns per thread stay in registers; NV = 0: any width, rows are read again.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
+  __shared__ float2 red2[8];
+  __shared__ float red[8];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int W = p.W;
+  const size_t base = static_cast<size_t>(blockIdx.x) * W;
+  const T* y0 = static_cast<const T*>(p.y0) + base;
+  const T* y1 = p.y1 != nullptr ? static_cast<const T*>(p.y1) + base : nullptr;
+  T* act = static_cast<T*>(p.act);
+  const float n = static_cast<float>(W);
+  float i0 = 1.f, i1 = 1.f;
+  if constexpr (NV > 0) {
+    float4 v[NV], x[NV];
+    {
+      float4 u[NV];
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * 256) * 4;
+        v[i] = u[i] = x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < W) {
+          v[i] = load4(y0 + c);
+          if (y1 != nullptr) u[i] = load4(y1 + c);
+          x[i] = load4(p.x + base + c);
+        }
+        s0 += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        s1 += u[i].x * u[i].x + u[i].y * u[i].y + u[i].z * u[i].z + u[i].w * u[i].w;
+      }
+      if (p.w0 != nullptr) {
+        const float2 t = block_sum2_f32(s0, s1, red2);
+        i0 = 1.f / sqrtf(t.x / n + p.eps);
+        i1 = 1.f / sqrtf(t.y / n + p.eps);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * 256) * 4;
+        if (c >= W) continue;
+        float4 a = make_float4(i0, i0, i0, i0), b = make_float4(i1, i1, i1, i1);
+        if (p.w0 != nullptr) {
+          const float4 g = load4(p.w0 + c);
+          a = make_float4(a.x * g.x, a.y * g.y, a.z * g.z, a.w * g.w);
+        }
+        if (p.w1 != nullptr) {
+          const float4 g = load4(p.w1 + c);
+          b = make_float4(b.x * g.x, b.y * g.y, b.z * g.z, b.w * g.w);
+        }
+        v[i] = make_float4(p.gain * fmaf(v[i].x, a.x, u[i].x * b.x), p.gain * fmaf(v[i].y, a.y, u[i].y * b.y), p.gain * fmaf(v[i].z, a.z, u[i].z * b.z),
+                           p.gain * fmaf(v[i].w, a.w, u[i].w * b.w));
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= W) continue;
+      const float4 g = load4(p.weight + c);
+      x[i] = make_float4(fmaf(v[i].x * inv, g.x, x[i].x), fmaf(v[i].y * inv, g.y, x[i].y), fmaf(v[i].z * inv, g.z, x[i].z), fmaf(v[i].w * inv, g.w, x[i].w));
+      store4(p.x_out + base + c, x[i]);
+      ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+    }
+    if (p.next == nullptr) return;
+    const float out = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= W) continue;
+      const float4 g = load4(p.next + c);
+      store4(act + base + c, make_float4(x[i].x * out * g.x, x[i].y * out * g.y, x[i].z * out * g.z, x[i].w * out * g.w));
+    }
+  } else {
+    if (p.w0 != nullptr) {
+      float s0 = 0.f, s1 = 0.f;
+      for (int c = threadIdx.x; c < W; c += 256) {
+        const float a = to_f32(y0[c]), b = y1 != nullptr ? to_f32(y1[c]) : 0.f;
+        s0 += a * a;
+        s1 += b * b;
+      }
+      const float2 t = block_sum2_f32(s0, s1, red2);
+      i0 = 1.f / sqrtf(t.x / n + p.eps);
+      i1 = 1.f / sqrtf(t.y / n + p.eps);
+    }
+    auto mixed = [&](int c) {
+      const float a = to_f32(y0[c]) * i0 * (p.w0 != nullptr ? p.w0[c] : 1.f);
+      const float b = y1 != nullptr ? to_f32(y1[c]) * i1 * (p.w1 != nullptr ? p.w1[c] : 1.f) : 0.f;
+      return p.gain * (a + b);
+    };
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float m = mixed(c);
+      ss += m * m;
+    }
+    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float o = fmaf(mixed(c) * inv, p.weight[c], p.x[base + c]);
+      p.x_out[base + c] = o;
+      ss += o * o;
+    }
+    if (p.next == nullptr) return;
+    const float out = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    for (int c = threadIdx.x; c < W; c += 256) act[base + c] = from_f32<T>(p.x_out[base + c] * out * p.next[c]);
+  }
+}
+
+template <typename T>
+static cudaError_t launch_branch_norm(const BranchNormParams& p, int M, bool quads_ok, cudaStream_t stream) {
+  const int quads = quads_ok ? (p.W / 4 + 255) / 256 : 0;
+#define ER_BN(NV_) launch_pdl(branch_norm_kernel<T, NV_>, dim3(M), dim3(256), 0, stream, p)
+  switch (quads) {
+    case 1: return ER_BN(1);
+    case 2: return ER_BN(2);
+    case 3:
+    case 4: return ER_BN(4);
+    case 5:
+    case 6:
+    case 7:
+    case 8: return ER_BN(8);
+    default: return ER_BN(0);
+  }
+#undef ER_BN
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table,
                                                                 float* __restrict__ x, T* __restrict__ act, int W, int rows, float scale) {
@@ -348,6 +507,18 @@ extern "C" int eredu_residual_norm(const float* x, const void* y, const void* ro
     return -1;
   const ResidualNormParams p = {x, y, rows, route_pos, route_w, weight, bias, x_out, act, W, k, center, eps};
   const cudaError_t e = fp32 ? launch_residual_norm<float>(p, M, quads != 0, stream) : launch_residual_norm<__nv_bfloat16>(p, M, quads != 0, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// x, x_out, weights fp32; y0, y1 (or null), act bf16 (fp32 = 0) or fp32; w0, w1: norms of the branches, both or neither null.
+extern "C" int eredu_branch_norm(const float* x, const void* y0, const void* y1, const float* w0, const float* w1, const float* weight,
+                                 const float* next, float* x_out, void* act, int M, int W, int fp32, int quads, float gain, float eps,
+                                 cudaStream_t stream) {
+  if (M <= 0 || W <= 0) return 0;
+  if ((next != nullptr && act == nullptr) || (y1 != nullptr && (w0 == nullptr) != (w1 == nullptr))) return -1;
+  const BranchNormParams p = {x, y0, y1, w0, w1, weight, next, x_out, act, W, gain, eps};
+  const cudaError_t e = fp32 ? launch_branch_norm<float>(p, M, quads != 0, stream) : launch_branch_norm<__nv_bfloat16>(p, M, quads != 0, stream);
   eredu_count_launches(1);
   return static_cast<int>(e);
 }

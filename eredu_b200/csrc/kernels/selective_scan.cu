@@ -1,0 +1,252 @@
+// Selective scan (Mamba): a diagonal recurrence per channel and state whose step size, input and output vectors depend on the token.
+//   dt = softplus(W_dt low + b),  S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,  y_c = sum_n S[c, n] C_n + D_c x_c,  out = y silu(z)
+// params [M, rank + 2 n] = [low | B | C]; S fp32, the first c * n elements of a sequence's state. Step sizes, decays and S are fp32.
+//
+// A few neighbouring lanes share a channel, each with NS states in registers; a CTA takes the channels of 128 threads and stages B, C,
+// step sizes and inputs of some tokens at a time in shared memory. Because a step is affine in S and its factors over a tile
+// multiply to exp(A sum dt), long portions are cut into tiles that run in parallel: one launch leaves what every tile adds to a zero
+// state and its summed step size, a second one chains the tiles in front of its own and replays it.
+#include "../common/elem.cuh"
+#include "../common/launch.h"
+#include "../common/launch_count.h"
+#include "../common/ptx.cuh"
+#include "../common/ragged.cuh"
+
+namespace eredu {
+
+template <typename T>
+struct ScanParams {
+  const T* x;              // [M, C]
+  const T* z;              // [M, ldz]
+  const T* params;         // [M, ldp]
+  const float* dt;         // [M, C] W_dt low, or null: formed here
+  const T* dt_w;           // [C, rank]
+  const float* dt_b;       // [C]
+  const float* A;          // [C, N]
+  const float* D;          // [C]
+  float* state;
+  T* out;                  // [M, C]
+  float* maps;             // [B, tiles, C, N] what a tile adds, then [B, tiles, C] summed step sizes
+  int C, N, rank, ldz, ldp, state_elems;
+  int lanes, stage, tiles, tile_len;   // lanes of a channel; tokens staged at a time; tiles of the longest portion and their length
+  RaggedBatch seqs;
+};
+
+constexpr int kScanThreads = 128;
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+template <typename T>
+__device__ __forceinline__ float scan_decay(float dt, float a) {   // a: A, times log2(e) for bf16 activations
+  return sizeof(T) == 4 ? expf(dt * a) : ex2_approx(dt * a);
+}
+
+// MAPS: only the map of the tile, from a zero state. N4: states are whole groups of four.
+template <typename T, int NS, bool MAPS>
+__global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(ScanParams<T> p) {
+  extern __shared__ float sm[];
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = blockIdx.z, tile = blockIdx.y;
+  const RaggedSeq s = ragged_seq(p.seqs, b);
+  const int t_begin = tile * p.tile_len, t_end = min(s.rows, t_begin + p.tile_len);
+  if (t_begin >= t_end) return;                                            // uniform
+  if (MAPS && t_end >= s.rows) return;                                     // nothing follows the last tile
+  const int lanes = p.lanes, per = kScanThreads / lanes;                   // channels of the CTA
+  const int c0 = blockIdx.x * per, nc = min(per, p.C - c0);
+  const int width = lanes * NS;                                            // states of a channel, filled up with silent ones
+  float* bs = sm;                                                          // [stage][width]
+  float* cs = bs + p.stage * width;                                        // [stage][width]
+  float* ds = cs + p.stage * width;                                        // [stage][per] step size
+  float* xs = ds + p.stage * per;                                          // [stage][per] input
+  float* ys = xs + p.stage * per;                                          // [stage][per]
+  const int ch = threadIdx.x / lanes, part = threadIdx.x % lanes, n0 = part * NS;
+  const bool in = ch < nc;
+  const int c = c0 + (in ? ch : 0);
+  float a[NS], S[NS];
+  const size_t cell = static_cast<size_t>(c) * p.N + n0;
+#pragma unroll
+  for (int i = 0; i < NS; ++i) {
+    a[i] = n0 + i < p.N ? p.A[cell + i] * (sizeof(T) == 4 ? 1.f : kLog2e) : 0.f;
+    S[i] = 0.f;
+  }
+  float* st = p.state + static_cast<size_t>(s.slot) * p.state_elems + cell;
+  float* maps = p.maps + static_cast<size_t>(b) * p.tiles * p.C * p.N;
+  float* sums = p.maps + static_cast<size_t>(p.seqs.B) * p.tiles * p.C * p.N + static_cast<size_t>(b) * p.tiles * p.C;
+  if (!MAPS) {
+    if (s.live)
+#pragma unroll
+      for (int i = 0; i < NS; ++i) S[i] = n0 + i < p.N ? st[i] : 0.f;
+    for (int j = 0; j < tile; ++j) {                                       // the tiles in front
+      const float dt = sums[static_cast<size_t>(j) * p.C + c];
+#pragma unroll
+      for (int i = 0; i < NS; ++i)
+        if (n0 + i < p.N) S[i] = fmaf(scan_decay<T>(dt, a[i]), S[i], maps[static_cast<size_t>(j) * p.C * p.N + cell + i]);
+    }
+  }
+  float total = 0.f;
+  const float d_skip = MAPS ? 0.f : p.D[c];
+  for (int t0 = t_begin; t0 < t_end; t0 += p.stage) {
+    const int n = min(p.stage, t_end - t0);
+    const size_t m0 = static_cast<size_t>(s.row0 + t0);
+    __syncthreads();                                                       // the previous tokens are done with
+    for (int i = threadIdx.x; i < n * width; i += kScanThreads) {
+      const int t = i / width, k = i - t * width;
+      const T* row = p.params + (m0 + t) * p.ldp + p.rank;
+      bs[i] = k < p.N ? to_f32(row[k]) : 0.f;
+      if (!MAPS) cs[i] = k < p.N ? to_f32(row[p.N + k]) : 0.f;
+    }
+    if (p.dt != nullptr) {
+      for (int i = threadIdx.x; i < n * per; i += kScanThreads) {
+        const int t = i / per, k = i - t * per;
+        if (k >= nc) continue;
+        ds[i] = softplus_f32(p.dt[(m0 + t) * p.C + c0 + k] + p.dt_b[c0 + k]);
+        xs[i] = to_f32(p.x[(m0 + t) * p.C + c0 + k]);
+      }
+    } else {                                                               // the lanes of a channel share its row of W_dt
+      const T* w = p.dt_w + static_cast<size_t>(c) * p.rank;
+      for (int t = 0; t < n; ++t) {
+        const T* low = p.params + (m0 + t) * p.ldp;
+        float v = 0.f;
+        if constexpr (sizeof(T) == 2) {
+          if ((p.rank & 7) == 0 && (p.ldp & 7) == 0) {                     // 16-byte pieces
+            for (int j = part * 8; j < p.rank; j += lanes * 8) {
+              const float4 w0 = load4(w + j), w1 = load4(w + j + 4), l0 = load4(low + j), l1 = load4(low + j + 4);
+              v = fmaf(w0.x, l0.x, fmaf(w0.y, l0.y, fmaf(w0.z, l0.z, fmaf(w0.w, l0.w, v))));
+              v = fmaf(w1.x, l1.x, fmaf(w1.y, l1.y, fmaf(w1.z, l1.z, fmaf(w1.w, l1.w, v))));
+            }
+          } else {
+            for (int j = part; j < p.rank; j += lanes) v = fmaf(to_f32(w[j]), to_f32(low[j]), v);
+          }
+        } else {
+          for (int j = part; j < p.rank; j += lanes) v = fmaf(to_f32(w[j]), to_f32(low[j]), v);
+        }
+        for (int o = lanes >> 1; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        if (in && part == 0) {
+          ds[t * per + ch] = softplus_f32(v + p.dt_b[c]);
+          xs[t * per + ch] = to_f32(p.x[(m0 + t) * p.C + c]);
+        }
+      }
+    }
+    __syncthreads();
+    for (int t = 0; t < n; ++t) {
+      const float dt = in ? ds[t * per + ch] : 0.f, xv = in ? xs[t * per + ch] : 0.f;
+      const float dx = dt * xv;
+      float y = 0.f;
+#pragma unroll
+      for (int i = 0; i < NS; ++i) {
+        S[i] = fmaf(scan_decay<T>(dt, a[i]), S[i], dx * bs[t * width + n0 + i]);
+        if (!MAPS) y = fmaf(S[i], cs[t * width + n0 + i], y);
+      }
+      if (MAPS) {
+        total += dt;
+      } else {
+        for (int o = lanes >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+        if (in && part == 0) ys[t * per + ch] = fmaf(d_skip, xv, y);
+      }
+    }
+    if (!MAPS) {
+      __syncthreads();
+      for (int i = threadIdx.x; i < n * per; i += kScanThreads) {
+        const int t = i / per, k = i - t * per;
+        if (k >= nc) continue;
+        const float g = to_f32(p.z[(m0 + t) * p.ldz + c0 + k]);
+        p.out[(m0 + t) * p.C + c0 + k] = from_f32<T>(ys[i] * (sizeof(T) == 4 ? silu_f32(g) : silu_fast(g)));
+      }
+    }
+  }
+  if (!in) return;
+  if (MAPS) {
+    float* map = maps + static_cast<size_t>(tile) * p.C * p.N + cell;
+#pragma unroll
+    for (int i = 0; i < NS; ++i)
+      if (n0 + i < p.N) map[i] = S[i];
+    if (part == 0) sums[static_cast<size_t>(tile) * p.C + c] = total;
+  } else if (s.live && t_end >= s.rows) {
+#pragma unroll
+    for (int i = 0; i < NS; ++i)
+      if (n0 + i < p.N) st[i] = S[i];
+  }
+}
+
+struct ScanShape {
+  int ns, lanes, stage, tiles, tile_len, channels;
+};
+
+static size_t scan_smem(const ScanShape& s) {
+  return (static_cast<size_t>(2) * s.stage * s.lanes * s.ns + 3 * static_cast<size_t>(s.stage) * s.channels) * sizeof(float);
+}
+
+constexpr int kScanMinTile = 64;     // tokens of a tile at least
+
+static ScanShape scan_shape(int C, int N, int batch, int max_rows, int sm_count, bool tiled) {
+  ScanShape s;
+  s.ns = N <= 128 ? 4 : N <= 256 ? 8 : 16;
+  s.lanes = 1;
+  while (s.lanes * s.ns < N) s.lanes *= 2;
+  s.channels = kScanThreads / s.lanes;
+  s.stage = s.lanes * s.ns <= 64 ? 32 : 8;
+  while (scan_smem(s) > 48 * 1024) s.stage /= 2;
+  if (s.stage > max_rows) s.stage = max_rows;
+  // enough CTAs to fill the machine, in tiles of equal length
+  const long long ctas = static_cast<long long>((C + s.channels - 1) / s.channels) * batch;
+  const long long want = tiled ? (8LL * (sm_count > 0 ? sm_count : 148) + ctas - 1) / ctas : 1;
+  const int most = max_rows / kScanMinTile;
+  s.tiles = static_cast<int>(want < most ? want : most);
+  if (s.tiles < 1) s.tiles = 1;
+  s.tile_len = (max_rows + s.tiles - 1) / s.tiles;
+  s.tile_len = (s.tile_len + 31) & ~31;
+  s.tiles = (max_rows + s.tile_len - 1) / s.tile_len;
+  return s;
+}
+
+template <typename T, int NS>
+static cudaError_t launch_scan(const ScanParams<T>& p, const ScanShape& s, cudaStream_t stream) {
+  const size_t smem = scan_smem(s);
+  const dim3 grid((p.C + s.channels - 1) / s.channels, s.tiles, p.seqs.B);
+  if (grid.y > 65535 || grid.z > 65535) return cudaErrorInvalidValue;
+  if (s.tiles > 1) {
+    const cudaError_t e = launch_pdl(selective_scan_kernel<T, NS, true>, grid, dim3(kScanThreads), smem, stream, p);
+    if (e != cudaSuccess) return e;
+    eredu_count_launches(1);
+  }
+  return launch_pdl(selective_scan_kernel<T, NS, false>, grid, dim3(kScanThreads), smem, stream, p);
+}
+
+template <typename T>
+static cudaError_t run_scan(const void* x, const void* z, const void* params, const float* dt, const void* dt_w, const float* dt_b, const float* A,
+                            const float* D, float* state, void* out, float* scratch, const ScanShape& s, int C, int N, int rank, int ldz, int ldp,
+                            int state_elems, const RaggedBatch& r, cudaStream_t stream) {
+  const ScanParams<T> p = {static_cast<const T*>(x), static_cast<const T*>(z), static_cast<const T*>(params), dt, static_cast<const T*>(dt_w), dt_b, A, D,
+                           state, static_cast<T*>(out), scratch, C, N, rank, ldz, ldp, state_elems, s.lanes, s.stage, s.tiles, s.tile_len, r};
+  return s.ns == 4 ? launch_scan<T, 4>(p, s, stream) : s.ns == 8 ? launch_scan<T, 8>(p, s, stream) : launch_scan<T, 16>(p, s, stream);
+}
+
+}  // namespace eredu
+
+using namespace eredu;
+
+// fp32 elements of scratch that let a call over `rows` rows of `batch` sequences run its tiles in parallel (0: one tile each).
+extern "C" long long eredu_selective_scan_scratch_elems(int channels, int states, int batch, int max_rows, int sm_count) {
+  const ScanShape s = scan_shape(channels, states, batch, max_rows, sm_count, true);
+  return s.tiles > 1 ? static_cast<long long>(batch) * s.tiles * channels * (states + 1LL) : 0;
+}
+
+// dt: fp32 [M, channels] = dt_w low, or null (formed in the kernel); scratch: fp32 [eredu_selective_scan_scratch_elems(...)] or null.
+// At most 512 states a channel.
+extern "C" int eredu_selective_scan(const void* x, const void* z, const void* params, const float* dt, const void* dt_w, const float* dt_b,
+                                    const float* A, const float* D, float* state, void* out, float* scratch, const int* block_table,
+                                    const int* page_to_slot, const int* cu_q, const long long* slots, int channels, int states, int rank, int ldz,
+                                    int ldp, int state_elems, int batch, int q_per_seq, int max_rows, int max_pages, int fp32, int sm_count,
+                                    cudaStream_t stream) {
+  if (batch <= 0 || max_rows <= 0) return 0;
+  if (channels <= 0 || states <= 0 || states > 512 || rank <= 0) return -1;
+  const RaggedBatch r = {block_table, page_to_slot, cu_q, slots, batch, q_per_seq, max_pages};
+  const ScanShape s = scan_shape(channels, states, batch, max_rows, sm_count, scratch != nullptr);
+  const cudaError_t e = fp32 ? run_scan<float>(x, z, params, dt, dt_w, dt_b, A, D, state, out, scratch, s, channels, states, rank, ldz, ldp, state_elems, r, stream)
+                             : run_scan<__nv_bfloat16>(x, z, params, dt, dt_w, dt_b, A, D, state, out, scratch, s, channels, states, rank, ldz, ldp,
+                                                       state_elems, r, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}

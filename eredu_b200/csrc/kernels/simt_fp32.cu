@@ -4,6 +4,7 @@
 #include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
+#include "../common/pooled.cuh"
 #include "../common/ptx.cuh"
 
 namespace eredu {
@@ -11,33 +12,41 @@ namespace eredu {
 constexpr int kTile = 64, kTileK = 16;
 
 // Y[M, N] = act(X[M, K] W[N, K]^T + bias): 64 x 64 outputs per CTA, 4 x 4 per thread, K in steps of 16 through shared memory.
-template <typename T, typename TO>
+// GATED: W holds N gate rows, then N up rows, Y = act(gate) * up.
+template <typename T, typename TO, bool GATED>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, TO* __restrict__ y,
                                                          const T* __restrict__ bias, int M, int N, int K, int ldx, int ldw, int ldy,
                                                          int act) {
-  __shared__ float xs[kTileK][kTile + 4], ws[kTileK][kTile + 4];
+  constexpr int PARTS = GATED ? 2 : 1;
+  __shared__ float xs[kTileK][kTile + 4], ws[PARTS][kTileK][kTile + 4];
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int n0 = blockIdx.x * kTile, m0 = blockIdx.y * kTile;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
-  float acc[4][4] = {};
+  float acc[PARTS][4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kTileK) {
     for (int i = threadIdx.x; i < kTile * kTileK; i += 256) {
       const int r = i / kTileK, k = i % kTileK;
       xs[k][r] = (m0 + r < M && k0 + k < K) ? to_f32(x[static_cast<size_t>(m0 + r) * ldx + k0 + k]) : 0.f;
-      ws[k][r] = (n0 + r < N && k0 + k < K) ? to_f32(w[static_cast<size_t>(n0 + r) * ldw + k0 + k]) : 0.f;
+#pragma unroll
+      for (int d = 0; d < PARTS; ++d)
+        ws[d][k][r] = (n0 + r < N && k0 + k < K) ? to_f32(w[static_cast<size_t>(d * N + n0 + r) * ldw + k0 + k]) : 0.f;
     }
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < kTileK; ++k) {
       const float4 a = *reinterpret_cast<const float4*>(&xs[k][ty * 4]);
-      const float4 b = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
-      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+      const float av[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
-      for (int i = 0; i < 4; ++i)
+      for (int d = 0; d < PARTS; ++d) {
+        const float4 b = *reinterpret_cast<const float4*>(&ws[d][k][tx * 4]);
+        const float bv[4] = {b.x, b.y, b.z, b.w};
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[d][i][j] = fmaf(av[i], bv[j], acc[d][i][j]);
+      }
     }
     __syncthreads();
   }
@@ -49,8 +58,11 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ x,
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
       if (n >= N) break;
-      float v = acc[i][j] + (bias != nullptr ? to_f32(bias[n]) : 0.f);
-      if (act == 1) {
+      float v = acc[0][i][j] + (bias != nullptr ? to_f32(bias[n]) : 0.f);
+      if (GATED) {
+        v = act == 3 ? fmaxf(v, 0.f) : silu_f32(v);
+        v *= acc[PARTS - 1][i][j] + (bias != nullptr ? to_f32(bias[N + n]) : 0.f);
+      } else if (act == 1) {
         v = fmaxf(v, 0.f);
         v *= v;
       }
@@ -128,6 +140,10 @@ struct AttnSimtParams {
   const float* sinks;    // [n_q] or null
   int q_per_seq, max_pages, n_q, n_kv, dk, dv, ldv, window, chunk;
   float scale;
+  // pool > 0: the mean key and value of every block of `pool` tokens that ends before the window is seen as well
+  const void* pk;        // [pages, n_kv, pool_rows, dk], page of the block's last token
+  const void* pv;        // [pages, n_kv, pool_rows, dv]
+  int pool, pool_rows;
 };
 
 constexpr int kMaxValueRegs = 32;  // value widths up to 1024
@@ -160,14 +176,11 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(AttnSimtParams p) {
 #pragma unroll
   for (int c = 0; c < kMaxValueRegs; ++c) acc[c] = 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int k0 = lo + warp * 32; k0 <= pos; k0 += 128) {
-    const int key = k0 + lane;
-    const bool ok = key <= pos;
-    size_t row = 0;
+  // one group of up to 32 keys: `row` names the lane's row of `keys` and `values` where it has one
+  auto group = [&](const T* keys, const T* values, size_t row, bool ok, int n) {
     float s = -INFINITY;
     if (ok) {
-      row = (static_cast<size_t>(bt[key >> 4]) * p.n_kv + kvh) * 16 + (key & 15);
-      const T* k = static_cast<const T*>(p.k_cache) + row * p.dk;
+      const T* k = keys + row * p.dk;
       s = 0.f;
       for (int i = 0; i < p.dk; ++i) s = fmaf(qs[i], to_f32(k[i]), s);
     }
@@ -179,17 +192,32 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(AttnSimtParams p) {
     const float pe = ok ? expf(s - m_new) : 0.f;
     m = m_new;
     l = l * corr + warp_sum_f32(pe);
-    const int n = min(32, pos - k0 + 1);
 #pragma unroll
     for (int c = 0; c < kMaxValueRegs; ++c) acc[c] *= corr;
     for (int j = 0; j < n; ++j) {
       const float pj = __shfl_sync(0xffffffffu, pe, j);
       const size_t rj = __shfl_sync(0xffffffffu, static_cast<unsigned long long>(row), j);
-      const T* v = static_cast<const T*>(p.v_cache) + rj * p.ldv;
+      const T* v = values + rj * p.ldv;
 #pragma unroll
       for (int c = 0; c < kMaxValueRegs; ++c)
         if (lane + 32 * c < p.dv) acc[c] = fmaf(pj, to_f32(v[lane + 32 * c]), acc[c]);
     }
+  };
+  if (p.pool > 0) {
+    const int blocks = pooled_seen(pos, p.window, p.pool);
+    for (int b0 = warp * 32; b0 < blocks; b0 += 128) {
+      const int blk = b0 + lane;
+      const bool ok = blk < blocks;
+      const PooledRow r = pooled_row(ok ? blk : 0, p.pool);
+      const size_t row = (static_cast<size_t>(bt[r.page]) * p.n_kv + kvh) * p.pool_rows + r.row;
+      group(static_cast<const T*>(p.pk), static_cast<const T*>(p.pv), row, ok, min(32, blocks - b0));
+    }
+  }
+  for (int k0 = lo + warp * 32; k0 <= pos; k0 += 128) {
+    const int key = k0 + lane;
+    const bool ok = key <= pos;
+    const size_t row = ok ? (static_cast<size_t>(bt[key >> 4]) * p.n_kv + kvh) * 16 + (key & 15) : 0;
+    group(static_cast<const T*>(p.k_cache), static_cast<const T*>(p.v_cache), row, ok, min(32, pos - k0 + 1));
   }
   float* mine = merge + warp * (p.dv + 2);
 #pragma unroll
@@ -219,36 +247,31 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(AttnSimtParams p) {
 
 using namespace eredu;
 
-// X [M, K], W [N, K], bias [N] (or null) fp32 (in_fp32 = 1) or bf16; Y [M, N] fp32 or bf16. act 1: squared ReLU.
+// X [M, K], W [N, K], bias [N] (or null) fp32 (in_fp32 = 1) or bf16; Y [M, N] fp32 or bf16. act 1: squared ReLU; act 2, 3: W is [2 N, K],
+// Y = silu(gate) * up or relu(gate) * up (bias [2 N]).
 extern "C" int eredu_gemm_simt(const void* x, const void* w, void* y, const void* bias, int M, int N, int K, int ldx, int ldw, int ldy,
                                int in_fp32, int out_fp32, int act, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const dim3 grid((N + kTile - 1) / kTile, (M + kTile - 1) / kTile);
-  if (grid.y > 65535) return -1;
+  if (grid.y > 65535 || (in_fp32 && !out_fp32)) return -1;
   cudaError_t e;
   using B = __nv_bfloat16;
-  if (in_fp32) {
-    auto X = static_cast<const float*>(x);
-    auto Wt = static_cast<const float*>(w);
-    auto b = static_cast<const float*>(bias);
-    if (!out_fp32) return -1;
-    e = launch_pdl(gemm_simt_kernel<float, float>, grid, dim3(256), 0, stream, X, Wt, static_cast<float*>(y), b, M, N, K, ldx, ldw, ldy, act);
-  } else {
-    auto X = static_cast<const B*>(x);
-    auto Wt = static_cast<const B*>(w);
-    auto b = static_cast<const B*>(bias);
-    e = out_fp32 ? launch_pdl(gemm_simt_kernel<B, float>, grid, dim3(256), 0, stream, X, Wt, static_cast<float*>(y), b, M, N, K, ldx, ldw, ldy, act)
-                 : launch_pdl(gemm_simt_kernel<B, B>, grid, dim3(256), 0, stream, X, Wt, static_cast<B*>(y), b, M, N, K, ldx, ldw, ldy, act);
-  }
+#define ER_SIMT(T_, TO_, G_)                                                                                                     \
+  launch_pdl(gemm_simt_kernel<T_, TO_, G_>, grid, dim3(256), 0, stream, static_cast<const T_*>(x), static_cast<const T_*>(w),      \
+             static_cast<TO_*>(y), static_cast<const T_*>(bias), M, N, K, ldx, ldw, ldy, act)
+  if (in_fp32) e = act >= 2 ? ER_SIMT(float, float, true) : ER_SIMT(float, float, false);
+  else if (out_fp32) e = act >= 2 ? ER_SIMT(B, float, true) : ER_SIMT(B, float, false);
+  else e = act >= 2 ? ER_SIMT(B, B, true) : ER_SIMT(B, B, false);
+#undef ER_SIMT
   eredu_count_launches(1);
   return static_cast<int>(e);
 }
 
 // Causal attention over the paged cache for any key width and value widths up to 1024; arguments as the tensor-core kernels. Rows of
 // v_cache are ldv >= dv wide: the values may be the head of a wider row (latent attention passes the same rows as keys and values).
-extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+static int attn_simt_impl(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, void* out, const int* block_table,
                                const int* seq_lens, const int* cu_q, const float* sinks, int batch, int q_per_seq, int max_q_len,
-                               int max_pages, int n_q, int n_kv, int dk, int dv, int ldv, int window, int chunk, int fp32, float scale,
+                               int max_pages, int n_q, int n_kv, int dk, int dv, int ldv, int window, int chunk, int pool, int pool_rows, int fp32, float scale,
                                cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
   if (n_kv <= 0 || n_q % n_kv != 0 || dk <= 0 || dv <= 0 || dv > 32 * kMaxValueRegs || ldv < dv || window < 0 || chunk < 0) return -1;
@@ -271,13 +294,35 @@ extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v
   p.window = window;
   p.chunk = chunk;
   p.scale = scale;
-  const size_t smem = (dk + 4 * (dv + 2)) * sizeof(float);
+  p.pk = pk;
+  p.pv = pv;
+  p.pool = pool;
+  p.pool_rows = pool_rows;
+  const size_t smem = (dk + 4 * static_cast<size_t>(dv + 2)) * sizeof(float);
   if (smem > 48 * 1024) return -1;
   const dim3 grid(max_q_len, n_q, batch);
   const cudaError_t e = fp32 ? launch_pdl(attn_simt_kernel<float>, grid, dim3(128), smem, stream, p)
                              : launch_pdl(attn_simt_kernel<__nv_bfloat16>, grid, dim3(128), smem, stream, p);
   eredu_count_launches(1);
   return static_cast<int>(e);
+}
+
+extern "C" int eredu_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                               const int* seq_lens, const int* cu_q, const float* sinks, int batch, int q_per_seq, int max_q_len,
+                               int max_pages, int n_q, int n_kv, int dk, int dv, int ldv, int window, int chunk, int fp32, float scale,
+                               cudaStream_t stream) {
+  return attn_simt_impl(q, k_cache, v_cache, nullptr, nullptr, out, block_table, seq_lens, cu_q, sinks, batch, q_per_seq, max_q_len, max_pages,
+                        n_q, n_kv, dk, dv, ldv, window, chunk, 0, 0, fp32, scale, stream);
+}
+
+// The same over a sliding window and the means of the blocks of `pool` tokens behind it (pk, pv as eredu_pool_blocks leaves them).
+extern "C" int eredu_attn_simt_pooled(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, void* out,
+                                      const int* block_table, const int* seq_lens, const int* cu_q, int batch, int q_per_seq, int max_q_len,
+                                      int max_pages, int n_q, int n_kv, int dk, int dv, int window, int pool, int pool_rows, int fp32,
+                                      float scale, cudaStream_t stream) {
+  if (window <= 0 || pool <= 0 || pool_rows <= 0 || pk == nullptr || pv == nullptr) return -1;
+  return attn_simt_impl(q, k_cache, v_cache, pk, pv, out, block_table, seq_lens, cu_q, nullptr, batch, q_per_seq, max_q_len, max_pages, n_q,
+                        n_kv, dk, dv, dv, window, 0, pool, pool_rows, fp32, scale, stream);
 }
 
 // work [n_work] int4 items of at most 64 rows; w [experts, w_rows, K] (dual: gate rows, then up rows); index: source row of every row of

@@ -194,7 +194,7 @@ def conv_project(proj, state, batch, page_to_slot, heads: Optional[ConvHeads] = 
         ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), ptr(batch.seq_lens), proj.stride(0), state[0].numel(),
         a.taps.shape[0] if a else 0, c.taps.shape[0] if c else 0, a.n_q if a else 0, a.n_kv if a else 0, a.dk if a else 0, a.dv if a else 0,
         2 * a.inv_freq.shape[0] if a else 0, a.pool if a else 0, pk.shape[2] if pk is not None else 0, a.hist if a else 0,
-        c.width if c else 0, c.start if c else 0, c.hist if c else 0, n, batch.q_per_seq, rows, batch.block_table.stride(0), M,
+        c.width if c else 0, c.start if c else 0, c.hist if c else 0, n, batch.q_per_seq, rows, batch.block_table.stride(0),
         1 if fp32 else 0, stream_ptr(proj.device))
     check(code, "eredu_conv_project")
     return q, out

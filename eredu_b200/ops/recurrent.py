@@ -432,7 +432,7 @@ def mlstm(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_sl
     return out
 
 
-native.register("eredu_selective_scan", I, [P] * 15 + [I] * 13 + [P])
+native.register("eredu_selective_scan", I, [P] * 15 + [I] * 12 + [P])
 native.register("eredu_selective_scan_scratch_elems", native.L, [I] * 5)
 
 # From this many rows a step size is worth a GEMM of its own in front of the scan (below, the scan multiplies it out).
@@ -480,12 +480,12 @@ def selective_scan(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_t
     B = batch.block_table.shape[0]
     rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
     dt = linear(params[:, :dt_rank], dt_w, out_dtype=torch.float32) if M >= SCAN_STEP_GEMM_MIN_ROWS else None
-    elems = int(lib().eredu_selective_scan_scratch_elems(c, n, M, B, rows)) if dt is not None else 0
+    elems = int(lib().eredu_selective_scan_scratch_elems(c, n, B, rows, _sm_count(x.device))) if dt is not None else 0
     scratch = torch.empty(elems, dtype=torch.float32, device=x.device) if elems else None
     code = lib().eredu_selective_scan(
         ptr(x), ptr(z), ptr(params), ptr(dt), ptr(dt_w), ptr(dt_b), ptr(A), ptr(D), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table),
         ptr(page_to_slot), ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), c, n, dt_rank, z.stride(0), params.stride(0),
-        state[0].numel(), M, B, batch.q_per_seq, rows, batch.block_table.stride(0), 1 if x.dtype == torch.float32 else 0,
+        state[0].numel(), B, batch.q_per_seq, rows, batch.block_table.stride(0), 1 if x.dtype == torch.float32 else 0,
         _sm_count(x.device), stream_ptr(x.device))
     check(code, "eredu_selective_scan")
     return out

@@ -234,6 +234,8 @@ def model_identity(engine, checkpoint_fingerprint: str) -> dict:
             layout.append({"kind": "key_value", "attention": ({"sliding": int(window)} if window else "full"),
                            "num_key_value_heads": int(model.n_kv_local if cfg.mixers is None else cfg.layer_kv_dims(li)[0]),
                            "head_dim": int(cfg.head_dim if cfg.mixers is None else cfg.layer_kv_dims(li)[1])})
+            if cfg.mixers is not None and cfg.layer_state_shape(li) is not None:
+                layout[-1]["fixed_state"] = ["recurrent"]         # the layer keeps both
         elif cfg.layer_kv_donor(li) is not None:
             layout.append({"kind": "stateless"})
         elif cfg.layer_is_conv(li):
