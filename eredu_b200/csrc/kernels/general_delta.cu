@@ -13,7 +13,7 @@ namespace eredu {
 
 // What one token gives a head, in shared memory.
 struct DeltaToken {
-  float *r, *k, *w, *u, *au;   // [dk]
+  float *r, *k, *w, *u, *au;   // [dk]; w: decay - 1, so that rounding factors just below one does not add up over the tokens
   float *low;                  // [rank] tanh
 };
 
@@ -46,7 +46,7 @@ __device__ __forceinline__ float2 delta_token(const DeltaParams<T>& p, const Del
     }
     const float r = to_f32(row[c]), k = d.k[i], u = k * inv;
     const float au = sigmoid_f32(to_f32(row[2 * qk + 2 * vw + c]) + p.rate_b[c]) * u;
-    d.w[i] = expf(-p.log_decay * sigmoid_f32(z));
+    d.w[i] = expm1f(-p.log_decay * sigmoid_f32(z));
     d.r[i] = r;
     d.u[i] = u;
     d.au[i] = au;
@@ -127,7 +127,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaParams<T> p) {
       for (int i = 0; i < NR; ++i) {
         const int r = grp + i * groups;
         if (r >= dk) continue;
-        const float u = d.u[r], rw = d.r[r] * d.w[r];
+        const float u = d.u[r], rw = fmaf(d.r[r], d.w[r], d.r[r]);
         rec = make_float4(fmaf(u, S[i].x, rec.x), fmaf(u, S[i].y, rec.y), fmaf(u, S[i].z, rec.z), fmaf(u, S[i].w, rec.w));
         o = make_float4(fmaf(rw, S[i].x, o.x), fmaf(rw, S[i].y, o.y), fmaf(rw, S[i].z, o.z), fmaf(rw, S[i].w, o.w));
       }
@@ -157,8 +157,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaParams<T> p) {
         const int r = grp + i * groups;
         if (r >= dk) continue;
         const float w = d.w[r], au = d.au[r], k = d.k[r];
-        S[i] = make_float4(fmaf(w, S[i].x, fmaf(-au, rec.x, k * v.x)), fmaf(w, S[i].y, fmaf(-au, rec.y, k * v.y)),
-                           fmaf(w, S[i].z, fmaf(-au, rec.z, k * v.z)), fmaf(w, S[i].w, fmaf(-au, rec.w, k * v.w)));
+        S[i] = make_float4(S[i].x + fmaf(w, S[i].x, fmaf(-au, rec.x, k * v.x)), S[i].y + fmaf(w, S[i].y, fmaf(-au, rec.y, k * v.y)),
+                           S[i].z + fmaf(w, S[i].z, fmaf(-au, rec.z, k * v.z)), S[i].w + fmaf(w, S[i].w, fmaf(-au, rec.w, k * v.w)));
       }
     }
     __syncthreads();
@@ -205,7 +205,8 @@ __global__ void __launch_bounds__(256) delta_any_kernel(DeltaParams<T> p) {
         for (int i = 0; i < dk; ++i) rec = fmaf(d.u[i], st[static_cast<size_t>(i) * dv + j], rec);
       for (int i = 0; i < dk; ++i) {
         float* cell = st + static_cast<size_t>(i) * dv + j;
-        const float x = fmaf(d.w[i], s.live ? *cell : 0.f, fmaf(-d.au[i], rec, d.k[i] * v));
+        const float old = s.live ? *cell : 0.f;
+        const float x = old + fmaf(d.w[i], old, fmaf(-d.au[i], rec, d.k[i] * v));
         if (s.live) *cell = x;
         o = fmaf(d.r[i], x, o);
       }

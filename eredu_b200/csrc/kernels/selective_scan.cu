@@ -36,9 +36,12 @@ constexpr int kScanThreads = 128;
 constexpr float kLog2e = 1.4426950408889634f;
 
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// exp(dt A) S + add. With fp32 activations a slow decay is applied as S + (exp(dt A) - 1) S: rounding a factor just below one would
+// add up over the tokens that a state remembers. a: A, times log2(e) for bf16 activations.
 template <typename T>
-__device__ __forceinline__ float scan_decay(float dt, float a) {   // a: A, times log2(e) for bf16 activations
-  return sizeof(T) == 4 ? expf(dt * a) : ex2_approx(dt * a);
+__device__ __forceinline__ float scan_step(float dt, float a, float S, float add) {
+  if constexpr (sizeof(T) == 4) return S + fmaf(expm1f(dt * a), S, add);
+  return fmaf(ex2_approx(dt * a), S, add);
 }
 
 // MAPS: only the map of the tile, from a zero state. N4: states are whole groups of four.
@@ -82,7 +85,7 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(ScanParams
       const float dt = sums[static_cast<size_t>(j) * p.C + c];
 #pragma unroll
       for (int i = 0; i < NS; ++i)
-        if (n0 + i < p.N) S[i] = fmaf(scan_decay<T>(dt, a[i]), S[i], maps[static_cast<size_t>(j) * p.C * p.N + cell + i]);
+        if (n0 + i < p.N) S[i] = scan_step<T>(dt, a[i], S[i], maps[static_cast<size_t>(j) * p.C * p.N + cell + i]);
     }
   }
   float total = 0.f;
@@ -136,7 +139,7 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(ScanParams
       float y = 0.f;
 #pragma unroll
       for (int i = 0; i < NS; ++i) {
-        S[i] = fmaf(scan_decay<T>(dt, a[i]), S[i], dx * bs[t * width + n0 + i]);
+        S[i] = scan_step<T>(dt, a[i], S[i], dx * bs[t * width + n0 + i]);
         if (!MAPS) y = fmaf(S[i], cs[t * width + n0 + i], y);
       }
       if (MAPS) {
