@@ -248,8 +248,8 @@ extern "C" long long eredu_general_delta_scratch_bytes(int heads, int dk, int dv
 // scratch: [eredu_general_delta_scratch_bytes(...)] of a bf16 call whose rows are whole 16-byte pieces, or null (token by token).
 extern "C" int eredu_general_delta(const void* proj, const float* w2, const float* w0, const float* rate_b, const float* norm_w, float* state, void* out,
                                    void* scratch, const int* block_table, const int* page_to_slot, const int* cu_q, const long long* slots,
-                                   int heads, int dk, int dv, int rank, int ld, int rows, int batch, int q_per_seq, int max_rows, int max_pages,
-                                   int fp32, int sm_count, float log_decay, float eps, cudaStream_t stream) {
+                                   int heads, int dk, int dv, int rank, int ld, int batch, int q_per_seq, int max_rows, int max_pages,
+                                   int fp32, float log_decay, float eps, cudaStream_t stream) {
   if (batch <= 0 || max_rows <= 0) return 0;
   if (heads <= 0 || dk <= 0 || dv <= 0 || rank <= 0 || log_decay <= 0.f) return -1;
   const RaggedBatch r = {block_table, page_to_slot, cu_q, slots, batch, q_per_seq, max_pages};
@@ -261,7 +261,7 @@ extern "C" int eredu_general_delta(const void* proj, const float* w2, const floa
   } else {
     const DeltaParams<__nv_bfloat16> p = {static_cast<const __nv_bfloat16*>(proj), w2, w0, rate_b, norm_w, state, static_cast<__nv_bfloat16*>(out),
                                           heads, dk, dv, rank, ld, log_decay, eps, r};
-    e = scratch != nullptr ? launch_delta_chunks(p, rows, max_rows, scratch, stream) : launch_delta_step(p, stream);
+    e = scratch != nullptr && delta_chunk_supported(p) ? launch_delta_chunks(p, max_rows, scratch, stream) : launch_delta_step(p, stream);
   }
   eredu_count_launches(1);
   return static_cast<int>(e);

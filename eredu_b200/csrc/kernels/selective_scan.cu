@@ -6,6 +6,10 @@
 // step sizes and inputs of some tokens at a time in shared memory. Because a step is affine in S and its factors over a tile
 // multiply to exp(A sum dt), long portions are cut into tiles that run in parallel: one launch leaves what every tile adds to a zero
 // state and its summed step size, a second one chains the tiles in front of its own and replays it.
+//
+// Prompts in bf16 with at most 32 states a channel take a form of their own, bound by the exponentials: a thread owns a whole channel, B and
+// C come as broadcasts from shared memory, states are updated in pairs (two-wide fp32 instructions), and a part of the exponentials is
+// a polynomial on the FMA pipe, which the special-function unit would otherwise hold up.
 #include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
@@ -173,7 +177,166 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(ScanParams
   }
 }
 
+// ---------------------------------------------------------------- prompts in bf16, NP pairs of states
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+// 2^x for a pair, x <= 0, on the FMA pipe: n = round(x) by the 1.5 * 2^23 trick, the Taylor series of 2^f = e^(f ln 2) on f = x - n in
+// [-1/2, 1/2] up to f^6 (relative error below 2e-7; exact at 0, so slow decays keep their accuracy), n added into the exponent.
+__device__ __forceinline__ uint64_t ex2_pair_poly(uint64_t x) {
+  float x0, x1;
+  unpack_f32x2(x, x0, x1);
+  x = pack_f32x2(fmaxf(x0, -126.f), fmaxf(x1, -126.f));
+  const uint64_t magic = pack_f32x2(12582912.f, 12582912.f), back = pack_f32x2(-12582912.f, -12582912.f), minus = pack_f32x2(-1.f, -1.f);
+  const uint64_t t = add_f32x2(x, magic);
+  const uint64_t f = fma_f32x2(add_f32x2(t, back), minus, x);
+  auto two = [](float c) { return pack_f32x2(c, c); };
+  uint64_t y = fma_f32x2(f, two(1.5403530e-4f), two(1.3333558e-3f));      // ln(2)^k / k!
+  y = fma_f32x2(y, f, two(9.6181291e-3f));
+  y = fma_f32x2(y, f, two(5.5504109e-2f));
+  y = fma_f32x2(y, f, two(2.4022651e-1f));
+  y = fma_f32x2(y, f, two(6.9314718e-1f));
+  y = fma_f32x2(y, f, two(1.f));
+  float y0, y1, t0, t1;
+  unpack_f32x2(y, y0, y1);
+  unpack_f32x2(t, t0, t1);
+  return pack_f32x2(__int_as_float(__float_as_int(y0) + (__float_as_int(t0) << 23)), __int_as_float(__float_as_int(y1) + (__float_as_int(t1) << 23)));
+}
+__device__ __forceinline__ uint64_t ex2_pair(uint64_t x, bool poly) {
+  if (poly) return ex2_pair_poly(x);
+  float a, b;
+  unpack_f32x2(x, a, b);
+  return pack_f32x2(ex2_approx(a), ex2_approx(b));
+}
+// softplus with 32-bit accuracy from the fast logarithm: log(1 + t) keeps its relative accuracy for small t by the correction
+// t / ((1 + t) - 1) (Goldberg, "What every computer scientist should know about floating-point arithmetic").
+__device__ __forceinline__ float softplus_fast(float x) {
+  const float t = ex2_approx(-fabsf(x) * kLog2e), u = 1.f + t;
+  return fmaxf(x, 0.f) + (u == 1.f ? t : __logf(u) * __fdividef(t, u - 1.f));
+}
+
+constexpr int kWideStage = 32;       // tokens of B and C staged at a time
+constexpr int kWideAhead = 4;        // tokens whose channel values are in flight
+
+template <int NP, bool MAPS>
+__global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv_bfloat16> p) {
+  using T = __nv_bfloat16;
+  __shared__ __align__(16) float bc[2][kWideStage][2][2 * NP];             // buffer, token, B or C
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = blockIdx.z, tile = blockIdx.y;
+  const RaggedSeq s = ragged_seq(p.seqs, b);
+  const int t_begin = tile * p.tile_len, t_end = min(s.rows, t_begin + p.tile_len);
+  if (t_begin >= t_end) return;                                            // uniform
+  if (MAPS && t_end >= s.rows) return;                                     // nothing follows the last tile
+  const int c = blockIdx.x * kScanThreads + threadIdx.x;
+  const bool in = c < p.C;
+  const int cc = in ? c : 0;
+  uint64_t a[NP], S[NP];
+  auto state_pair = [&](const float* src, int i) {
+    return pack_f32x2(2 * i < p.N ? src[2 * i] : 0.f, 2 * i + 1 < p.N ? src[2 * i + 1] : 0.f);
+  };
+  const size_t cell = static_cast<size_t>(cc) * p.N;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    a[i] = mul_f32x2(state_pair(p.A + cell, i), pack_f32x2(kLog2e, kLog2e));
+    S[i] = 0ull;
+  }
+  float* st = p.state + static_cast<size_t>(s.slot) * p.state_elems + cell;
+  float* maps = p.maps + static_cast<size_t>(b) * p.tiles * p.C * p.N;
+  float* sums = p.maps + static_cast<size_t>(p.seqs.B) * p.tiles * p.C * p.N + static_cast<size_t>(b) * p.tiles * p.C;
+  if (!MAPS) {
+    if (s.live)
+#pragma unroll
+      for (int i = 0; i < NP; ++i) S[i] = state_pair(st, i);
+    for (int j = 0; j < tile; ++j) {                                       // the tiles in front
+      const float dt = sums[static_cast<size_t>(j) * p.C + cc];
+      const uint64_t d2 = pack_f32x2(dt, dt);
+#pragma unroll
+      for (int i = 0; i < NP; ++i) S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), false), S[i], state_pair(maps + static_cast<size_t>(j) * p.C * p.N + cell, i));
+    }
+  }
+  const float bias = p.dt_b[cc], d_skip = MAPS ? 0.f : p.D[cc];
+  const size_t m0 = static_cast<size_t>(s.row0);
+  auto stage = [&](int t0, int buf) {                                      // B and C of some tokens, fp32, silent states zero
+    const int n = min(kWideStage, t_end - t0);
+    for (int i = threadIdx.x; i < n * 4 * NP; i += kScanThreads) {
+      const int t = i / (4 * NP), k = i % (4 * NP), w = k / (2 * NP), j = k % (2 * NP);
+      bc[buf][t][w][j] = j < p.N ? to_f32(p.params[(m0 + t0 + t) * p.ldp + p.rank + w * p.N + j]) : 0.f;
+    }
+  };
+  float dn[kWideAhead];
+  T xn[kWideAhead], zn[kWideAhead];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int u = 0; u < kWideAhead; ++u) {
+      if (t0 + u >= t_end) break;
+      const size_t m = m0 + t0 + u;
+      dn[u] = p.dt[m * p.C + cc];
+      xn[u] = p.x[m * p.C + cc];
+      if (!MAPS) zn[u] = p.z[m * p.ldz + cc];
+    }
+  };
+  float total = 0.f;
+  fetch(t_begin);
+  stage(t_begin, 0);
+  int buf = 0;
+  for (int t0 = t_begin; t0 < t_end; t0 += kWideStage, buf ^= 1) {
+    __syncthreads();                                                       // this buffer is filled, the other one left
+    if (t0 + kWideStage < t_end) stage(t0 + kWideStage, buf ^ 1);
+    const int n = min(kWideStage, t_end - t0);
+    for (int q = 0; q < n; q += kWideAhead) {
+      float dt[kWideAhead], x[kWideAhead], z[kWideAhead];
+#pragma unroll
+      for (int u = 0; u < kWideAhead; ++u) {
+        dt[u] = softplus_fast(dn[u] + bias);
+        x[u] = to_f32(xn[u]);
+        z[u] = MAPS ? 0.f : to_f32(zn[u]);
+      }
+      fetch(t0 + q + kWideAhead);
+#pragma unroll
+      for (int u = 0; u < kWideAhead; ++u) {
+        if (q + u >= n) break;
+        const uint64_t d2 = pack_f32x2(dt[u], dt[u]);
+        const float dx = dt[u] * x[u];
+        const uint64_t dx2 = pack_f32x2(dx, dx);
+        const uint64_t* bp = reinterpret_cast<const uint64_t*>(bc[buf][q + u][0]);
+        const uint64_t* cp = reinterpret_cast<const uint64_t*>(bc[buf][q + u][1]);
+        uint64_t y2 = 0ull;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), i % 8 >= 5), S[i], mul_f32x2(dx2, bp[i]));
+          if (!MAPS) y2 = fma_f32x2(S[i], cp[i], y2);
+        }
+        if (MAPS) {
+          total += dt[u];
+        } else if (in) {
+          float y0, y1;
+          unpack_f32x2(y2, y0, y1);
+          p.out[(m0 + t0 + q + u) * p.C + c] = __float2bfloat16(fmaf(d_skip, x[u], y0 + y1) * silu_fast(z[u]));
+        }
+      }
+    }
+  }
+  if (!in) return;
+  float* dst = MAPS ? maps + static_cast<size_t>(tile) * p.C * p.N + cell : st;
+  if (MAPS) sums[static_cast<size_t>(tile) * p.C + c] = total;
+  if (MAPS || (s.live && t_end >= s.rows)) {
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      float s0, s1;
+      unpack_f32x2(S[i], s0, s1);
+      if (2 * i < p.N) dst[2 * i] = s0;
+      if (2 * i + 1 < p.N) dst[2 * i + 1] = s1;
+    }
+  }
+}
+
 struct ScanShape {
+  bool wide;
   int ns, lanes, stage, tiles, tile_len, channels;
 };
 
@@ -183,8 +346,11 @@ static size_t scan_smem(const ScanShape& s) {
 
 constexpr int kScanMinTile = 64;     // tokens of a tile at least
 
-static ScanShape scan_shape(int C, int N, int batch, int max_rows, int sm_count, bool tiled) {
+constexpr int kWideMinRows = 16;     // portions from here on take the form of a thread per channel
+
+static ScanShape scan_shape(int C, int N, int batch, int max_rows, int sm_count, bool tiled, bool wide_ok) {
   ScanShape s;
+  s.wide = wide_ok && N <= 32 && max_rows >= kWideMinRows;
   s.ns = N <= 128 ? 4 : N <= 256 ? 8 : 16;
   s.lanes = 1;
   while (s.lanes * s.ns < N) s.lanes *= 2;
@@ -193,7 +359,8 @@ static ScanShape scan_shape(int C, int N, int batch, int max_rows, int sm_count,
   while (scan_smem(s) > 48 * 1024) s.stage /= 2;
   if (s.stage > max_rows) s.stage = max_rows;
   // enough CTAs to fill the machine, in tiles of equal length
-  const long long ctas = static_cast<long long>((C + s.channels - 1) / s.channels) * batch;
+  const int per = s.wide ? kScanThreads : s.channels;
+  const long long ctas = static_cast<long long>((C + per - 1) / per) * batch;
   const long long want = tiled ? (8LL * (sm_count > 0 ? sm_count : 148) + ctas - 1) / ctas : 1;
   const int most = max_rows / kScanMinTile;
   s.tiles = static_cast<int>(want < most ? want : most);
@@ -217,12 +384,27 @@ static cudaError_t launch_scan(const ScanParams<T>& p, const ScanShape& s, cudaS
   return launch_pdl(selective_scan_kernel<T, NS, false>, grid, dim3(kScanThreads), smem, stream, p);
 }
 
+template <int NP>
+static cudaError_t launch_scan_wide(const ScanParams<__nv_bfloat16>& p, const ScanShape& s, cudaStream_t stream) {
+  const dim3 grid((p.C + kScanThreads - 1) / kScanThreads, s.tiles, p.seqs.B);
+  if (grid.y > 65535 || grid.z > 65535) return cudaErrorInvalidValue;
+  if (s.tiles > 1) {
+    const cudaError_t e = launch_pdl(scan_wide_kernel<NP, true>, grid, dim3(kScanThreads), 0, stream, p);
+    if (e != cudaSuccess) return e;
+    eredu_count_launches(1);
+  }
+  return launch_pdl(scan_wide_kernel<NP, false>, grid, dim3(kScanThreads), 0, stream, p);
+}
+
 template <typename T>
 static cudaError_t run_scan(const void* x, const void* z, const void* params, const float* dt, const void* dt_w, const float* dt_b, const float* A,
                             const float* D, float* state, void* out, float* scratch, const ScanShape& s, int C, int N, int rank, int ldz, int ldp,
                             int state_elems, const RaggedBatch& r, cudaStream_t stream) {
   const ScanParams<T> p = {static_cast<const T*>(x), static_cast<const T*>(z), static_cast<const T*>(params), dt, static_cast<const T*>(dt_w), dt_b, A, D,
                            state, static_cast<T*>(out), scratch, C, N, rank, ldz, ldp, state_elems, s.lanes, s.stage, s.tiles, s.tile_len, r};
+  if constexpr (sizeof(T) == 2) {
+    if (s.wide) return N <= 8 ? launch_scan_wide<4>(p, s, stream) : N <= 16 ? launch_scan_wide<8>(p, s, stream) : launch_scan_wide<16>(p, s, stream);
+  }
   return s.ns == 4 ? launch_scan<T, 4>(p, s, stream) : s.ns == 8 ? launch_scan<T, 8>(p, s, stream) : launch_scan<T, 16>(p, s, stream);
 }
 
@@ -231,8 +413,8 @@ static cudaError_t run_scan(const void* x, const void* z, const void* params, co
 using namespace eredu;
 
 // fp32 elements of scratch that let a call over `rows` rows of `batch` sequences run its tiles in parallel (0: one tile each).
-extern "C" long long eredu_selective_scan_scratch_elems(int channels, int states, int batch, int max_rows, int sm_count) {
-  const ScanShape s = scan_shape(channels, states, batch, max_rows, sm_count, true);
+extern "C" long long eredu_selective_scan_scratch_elems(int channels, int states, int batch, int max_rows, int sm_count, int fp32) {
+  const ScanShape s = scan_shape(channels, states, batch, max_rows, sm_count, true, fp32 == 0);
   return s.tiles > 1 ? static_cast<long long>(batch) * s.tiles * channels * (states + 1LL) : 0;
 }
 
@@ -246,7 +428,7 @@ extern "C" int eredu_selective_scan(const void* x, const void* z, const void* pa
   if (batch <= 0 || max_rows <= 0) return 0;
   if (channels <= 0 || states <= 0 || states > 512 || rank <= 0) return -1;
   const RaggedBatch r = {block_table, page_to_slot, cu_q, slots, batch, q_per_seq, max_pages};
-  const ScanShape s = scan_shape(channels, states, batch, max_rows, sm_count, scratch != nullptr);
+  const ScanShape s = scan_shape(channels, states, batch, max_rows, sm_count, scratch != nullptr, fp32 == 0 && dt != nullptr);
   const cudaError_t e = fp32 ? run_scan<float>(x, z, params, dt, dt_w, dt_b, A, D, state, out, scratch, s, channels, states, rank, ldz, ldp, state_elems, r, stream)
                              : run_scan<__nv_bfloat16>(x, z, params, dt, dt_w, dt_b, A, D, state, out, scratch, s, channels, states, rank, ldz, ldp,
                                                        state_elems, r, stream);

@@ -433,7 +433,7 @@ def mlstm(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_sl
 
 
 native.register("eredu_selective_scan", I, [P] * 15 + [I] * 12 + [P])
-native.register("eredu_selective_scan_scratch_elems", native.L, [I] * 5)
+native.register("eredu_selective_scan_scratch_elems", native.L, [I] * 6)
 
 # From this many rows a step size is worth a GEMM of its own in front of the scan (below, the scan multiplies it out).
 SCAN_STEP_GEMM_MIN_ROWS = 64
@@ -480,7 +480,7 @@ def selective_scan(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_t
     B = batch.block_table.shape[0]
     rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
     dt = linear(params[:, :dt_rank], dt_w, out_dtype=torch.float32) if M >= SCAN_STEP_GEMM_MIN_ROWS else None
-    elems = int(lib().eredu_selective_scan_scratch_elems(c, n, B, rows, _sm_count(x.device))) if dt is not None else 0
+    elems = int(lib().eredu_selective_scan_scratch_elems(c, n, B, rows, _sm_count(x.device), 1 if x.dtype == torch.float32 else 0)) if dt is not None else 0
     scratch = torch.empty(elems, dtype=torch.float32, device=x.device) if elems else None
     code = lib().eredu_selective_scan(
         ptr(x), ptr(z), ptr(params), ptr(dt), ptr(dt_w), ptr(dt_b), ptr(A), ptr(D), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table),
@@ -491,7 +491,7 @@ def selective_scan(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_t
     return out
 
 
-native.register("eredu_general_delta", I, [P] * 12 + [I] * 12 + [F, F, P])
+native.register("eredu_general_delta", I, [P] * 12 + [I] * 10 + [F, F, P])
 native.register("eredu_general_delta_scratch_bytes", native.L, [I] * 6)
 
 DELTA_UNIT_EPS = 1e-6        # added to the squared length of a key before it is made a unit vector
@@ -551,8 +551,8 @@ def general_delta(proj, w2, w0, rate_b, norm_w, state, heads, dk, dv, log_decay,
             scratch = torch.empty(size, dtype=torch.uint8, device=proj.device)
     code = lib().eredu_general_delta(
         ptr(proj), ptr(w2), ptr(w0), ptr(rate_b), ptr(norm_w), ptr(state), ptr(out), ptr(scratch), ptr(batch.block_table), ptr(page_to_slot),
-        ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv, rank, proj.stride(0), M, B, batch.q_per_seq, rows,
-        batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, _sm_count(proj.device), log_decay, eps,
+        ptr(batch.cu_q) if batch.is_prefill else None, ptr(batch.slots), heads, dk, dv, rank, proj.stride(0), B, batch.q_per_seq, rows,
+        batch.block_table.stride(0), 1 if proj.dtype == torch.float32 else 0, log_decay, eps,
         stream_ptr(proj.device))
     check(code, "eredu_general_delta")
     return out
