@@ -957,12 +957,20 @@ static int launch_decode_all(AttnParams p, int batch, int q_per_seq, int n_q_hea
 #define ER_DECODE(DK_, DV_, EXT_) \
   e = one ? launch_decode<DK_, DV_, 1, EXT_>(p, grid, stream) : launch_decode<DK_, DV_, 2, EXT_>(p, grid, stream)
     if (p.pool > 0) {
-#define ER_POOLED(DK_, DV_) \
-  e = one ? launch_decode<DK_, DV_, 1, true, true>(p, grid, stream) : launch_decode<DK_, DV_, 2, true, true>(p, grid, stream)
-      if (key_dim > 64 && value_dim > 64) ER_POOLED(128, 128);
-      else if (key_dim > 64) ER_POOLED(128, 64);
-      else if (value_dim > 64) ER_POOLED(64, 128);
-      else ER_POOLED(64, 64);
+#define ER_POOLED(DK_, DV_)                                                                                                          \
+  if (key_dim == DK_ && value_dim == DV_)                                                                                             \
+    e = one ? launch_decode<DK_, DV_, 1, false, true>(p, grid, stream) : launch_decode<DK_, DV_, 2, false, true>(p, grid, stream);     \
+  else                                                                                                                                \
+    e = one ? launch_decode<DK_, DV_, 1, true, true>(p, grid, stream) : launch_decode<DK_, DV_, 2, true, true>(p, grid, stream)
+      if (key_dim > 64 && value_dim > 64) {
+        ER_POOLED(128, 128);
+      } else if (key_dim > 64) {
+        ER_POOLED(128, 64);
+      } else if (value_dim > 64) {
+        ER_POOLED(64, 128);
+      } else {
+        ER_POOLED(64, 64);
+      }
 #undef ER_POOLED
     } else if (plain && key_dim == 128) ER_DECODE(128, 128, false);
     else if (plain) ER_DECODE(64, 64, false);

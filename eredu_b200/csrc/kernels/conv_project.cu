@@ -42,9 +42,12 @@ constexpr int kMaxRot = 256;          // rotated dims of a head
 // VEC neighbouring elements; of a pair (VEC = 2) only the first `nv` exist.
 template <typename T, int VEC>
 __device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC], int nv) {
-  if constexpr (VEC == 8) {
-    const float4 a = load4(p), b = load4(p + 4);
-    v[0] = a.x, v[1] = a.y, v[2] = a.z, v[3] = a.w, v[4] = b.x, v[5] = b.y, v[6] = b.z, v[7] = b.w;
+  if constexpr (VEC >= 4) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4) {
+      const float4 a = load4(p + i);
+      v[i] = a.x, v[i + 1] = a.y, v[i + 2] = a.z, v[i + 3] = a.w;
+    }
   } else {
 #pragma unroll
     for (int i = 0; i < VEC; ++i) v[i] = i < nv ? to_f32(p[i]) : 0.f;
@@ -52,9 +55,9 @@ __device__ __forceinline__ void load_vec(const T* p, float (&v)[VEC], int nv) {
 }
 template <typename T, int VEC>
 __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC], int nv) {
-  if constexpr (VEC == 8) {
-    store4(p, make_float4(v[0], v[1], v[2], v[3]));
-    store4(p + 4, make_float4(v[4], v[5], v[6], v[7]));
+  if constexpr (VEC >= 4) {
+#pragma unroll
+    for (int i = 0; i < VEC; i += 4) store4(p + i, make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]));
   } else {
 #pragma unroll
     for (int i = 0; i < VEC; ++i)
@@ -62,66 +65,71 @@ __device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC], int nv) {
   }
 }
 
+// VEC neighbouring elements as they lie in memory.
+template <typename T, int VEC>
+struct alignas(VEC == 4 ? 4 * sizeof(T) : sizeof(T)) RawVec {
+  T v[VEC];
+};
+template <typename T, int VEC>
+__device__ __forceinline__ RawVec<T, VEC> load_raw(const T* p, int nv) {
+  RawVec<T, VEC> r;
+  if constexpr (VEC == 4) {
+    r = *reinterpret_cast<const RawVec<T, VEC>*>(p);
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) r.v[i] = i < nv ? p[i] : from_f32<T>(0.f);
+  }
+  return r;
+}
+// fp32 rows of taps and histories: whole 16-byte pieces when VEC = 4
+template <int VEC>
+__device__ __forceinline__ void load_row(const float* p, float (&v)[VEC], int nv) {
+  load_vec<float, VEC>(p, v, nv);
+}
+
 // Walks one segment of a sequence for VEC neighbouring channels: `emit(t, y)` gets the convolved values of row t. Only the first
 // segment reads the old history and writes the new one, and a segment is at least as long as the history, so no other CTA
-// races it. L taps at compile time keep the window in registers; L = 0: any number, rows are read again.
+// races it. L taps at compile time keep the window in registers and eight rows in flight; L = 0: any number, rows are read again.
 template <typename T, int VEC, int L, typename Emit>
 __device__ __forceinline__ void conv_walk(const T* col, int ld, const float* taps, int taps_ld, int n_taps, float* hist, int nv, int n, int t0, int t1, bool live, Emit emit) {
   auto input = [&](int t, float (&v)[VEC]) {
     if (t >= 0) {
       load_vec<T, VEC>(col + static_cast<size_t>(t) * ld, v, nv);
+    } else if (live) {
+      load_row<VEC>(hist + static_cast<size_t>(n_taps - 1 + t) * taps_ld, v, nv);
     } else {
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v[i] = live && (VEC == 8 || i < nv) ? hist[static_cast<size_t>(n_taps - 1 + t) * taps_ld + i] : 0.f;
+      for (int i = 0; i < VEC; ++i) v[i] = 0.f;
     }
   };
   if constexpr (L > 0) {
-    float w[L][VEC], win[L][VEC];
+    constexpr int U = 8;
+    float w[L][VEC], win[L - 1][VEC];
 #pragma unroll
-    for (int j = 0; j < L; ++j)
+    for (int j = 0; j < L; ++j) load_row<VEC>(taps + static_cast<size_t>(j) * taps_ld, w[j], nv);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) w[j][i] = VEC == 8 || i < nv ? taps[static_cast<size_t>(j) * taps_ld + i] : 0.f;
+    for (int j = 0; j + 1 < L; ++j) input(t0 - (L - 1) + j, win[j]);
+    for (int t = t0; t < t1; t += U) {
+      RawVec<T, VEC> raw[U];
 #pragma unroll
-    for (int j = 0; j + 1 < L; ++j) input(t0 - (L - 1) + j, win[j + 1]);
-    float old[L][VEC];                                      // the history as it was, for portions shorter than it
-    if (t0 == 0) {
+      for (int u = 0; u < U; ++u)
+        if (t + u < t1) raw[u] = load_raw<T, VEC>(col + static_cast<size_t>(t + u) * ld, nv);
 #pragma unroll
-      for (int j = 0; j + 1 < L; ++j)
+      for (int u = 0; u < U; ++u) {
+        if (t + u >= t1) break;
+        float y[VEC];
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) old[j][i] = win[j + 1][i];
-    }
-    for (int t = t0; t < t1; ++t) {
+        for (int i = 0; i < VEC; ++i) {
+          const float now = to_f32(raw[u].v[i]);
+          float a = w[0][i] * win[0][i];
 #pragma unroll
-      for (int j = 0; j + 1 < L; ++j)
+          for (int j = 1; j + 1 < L; ++j) a = fmaf(w[j][i], win[j][i], a);
+          y[i] = fmaf(w[L - 1][i], now, a);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
-      input(t, win[L - 1]);
-      float y[VEC];
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        y[i] = w[0][i] * win[0][i];
-#pragma unroll
-        for (int j = 1; j < L; ++j) y[i] = fmaf(w[j][i], win[j][i], y[i]);
-      }
-      emit(t, y);
-    }
-    if (t0 == 0 && live) {
-#pragma unroll
-      for (int j = 0; j + 1 < L; ++j) {
-        const int t = n - (L - 1) + j;                      // row whose input becomes history row j
-        float v[VEC];
-        if (t >= 0) {
-          input(t, v);
-        } else {
-#pragma unroll
-          for (int k = 0; k + 1 < L; ++k)
-            if (k == L - 1 + t)
-#pragma unroll
-              for (int i = 0; i < VEC; ++i) v[i] = old[k][i];
+          for (int j = 0; j + 2 < L; ++j) win[j][i] = win[j + 1][i];
+          win[L - 2][i] = now;
         }
-#pragma unroll
-        for (int i = 0; i < VEC; ++i)
-          if (VEC == 8 || i < nv) hist[static_cast<size_t>(j) * taps_ld + i] = v[i];
+        emit(t + u, y);
       }
     }
   } else {
@@ -130,22 +138,21 @@ __device__ __forceinline__ void conv_walk(const T* col, int ld, const float* tap
 #pragma unroll
       for (int i = 0; i < VEC; ++i) y[i] = 0.f;
       for (int j = 0; j < n_taps; ++j) {
-        float v[VEC];
+        float v[VEC], w[VEC];
         input(t - (n_taps - 1) + j, v);
+        load_row<VEC>(taps + static_cast<size_t>(j) * taps_ld, w, nv);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) if (VEC == 8 || i < nv) y[i] = fmaf(taps[static_cast<size_t>(j) * taps_ld + i], v[i], y[i]);
+        for (int i = 0; i < VEC; ++i) y[i] = fmaf(w[i], v[i], y[i]);
       }
       emit(t, y);
     }
-    if (t0 == 0 && live)
-      for (int j = 0; j + 1 < n_taps; ++j) {                // in order: row j comes from a later history row or from the portion
-        float v[VEC];
-        input(n - (n_taps - 1) + j, v);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i)
-          if (VEC == 8 || i < nv) hist[static_cast<size_t>(j) * taps_ld + i] = v[i];
-      }
   }
+  if (t0 == 0 && live)
+    for (int j = 0; j + 1 < n_taps; ++j) {                  // in order: row j comes from a later row of the history or from the portion
+      float v[VEC];
+      input(n - (n_taps - 1) + j, v);
+      store_vec<float, VEC>(hist + static_cast<size_t>(j) * taps_ld, v, nv);
+    }
 }
 
 template <typename T, int VEC, typename Emit>
@@ -175,10 +182,10 @@ __device__ __forceinline__ void block_mean(const T* cache, const int* bt, int n_
   for (int i = 0; i < VEC; ++i) m[i] /= n;
 }
 
-// Grid (blocks of channels: heads, then channels; segments; sequences). VEC = 8: head widths, rotated dims and columns are whole
-// groups of eight channels, which a thread owns. VEC = 2: any width; a thread owns a pair of a head (or the last channel of an odd one).
+// Grid (blocks of channels: heads, then channels; segments; sequences). VEC = 4: head widths and columns are whole groups of four
+// channels, which a thread owns. VEC = 2: any width; a thread owns a pair of a head (or the last channel of an odd one).
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kConvThreads) conv_project_kernel(ConvProjectParams p) {
+__global__ void __launch_bounds__(kConvThreads, 4) conv_project_kernel(ConvProjectParams p) {
   __shared__ float cs[kConvSeg * kMaxRot / 2], sn[kConvSeg * kMaxRot / 2];
   pdl_launch_early();
   pdl_wait();
@@ -304,9 +311,9 @@ __global__ void __launch_bounds__(128) pool_blocks_kernel(PoolParams p) {
 
 template <typename T>
 static cudaError_t launch_conv_project(ConvProjectParams& p, int max_rows, cudaStream_t stream) {
-  const bool wide = p.dk % 8 == 0 && p.dv % 8 == 0 && p.rot % 2 == 0 && p.width % 8 == 0 && p.c_start % 8 == 0 && p.ld % 8 == 0 &&
-                    (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0;
-  const int vec = wide ? 8 : 2;
+  const bool wide = p.dk % 4 == 0 && p.dv % 4 == 0 && p.width % 4 == 0 && p.c_start % 4 == 0 && p.ld % 4 == 0 &&
+                    p.h_hist % 4 == 0 && p.c_hist % 4 == 0 && p.state_elems % 4 == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0;
+  const int vec = wide ? 4 : 2;
   const int longest = p.hl > p.cl ? p.hl : p.cl;
   // a segment is never shorter than a history, and its angles fit the table
   p.seg_len = longest - 1 > kConvSeg ? longest - 1 : kConvSeg;
@@ -316,7 +323,7 @@ static cudaError_t launch_conv_project(ConvProjectParams& p, int max_rows, cudaS
   const int per = kConvThreads * vec;
   const dim3 grid(p.h_blocks + (p.width + per - 1) / per, (max_rows + p.seg_len - 1) / p.seg_len, p.seqs.B);
   if (grid.y > 65535 || grid.z > 65535) return cudaErrorInvalidValue;
-  return vec == 8 ? launch_pdl(conv_project_kernel<T, 8>, grid, dim3(kConvThreads), 0, stream, p)
+  return vec == 4 ? launch_pdl(conv_project_kernel<T, 4>, grid, dim3(kConvThreads), 0, stream, p)
                   : launch_pdl(conv_project_kernel<T, 2>, grid, dim3(kConvThreads), 0, stream, p);
 }
 

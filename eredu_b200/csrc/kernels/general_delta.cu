@@ -15,23 +15,39 @@ namespace eredu {
 struct DeltaToken {
   float *r, *k, *w, *u, *au;   // [dk]; w: decay - 1, so that rounding factors just below one does not add up over the tokens
   float *low;                  // [rank] tanh
+  float *red;                  // [8][4] sums of the warps: k . k, r . k, r . a u, o . o
 };
 
-// Fills `d` for row `row` of head h; returns (r . k, r . a u). Every thread of the block takes part.
+__device__ __forceinline__ float delta_sum(const DeltaToken& d, int which) {
+  float t = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) t += d.red[w * 4 + which];
+  return t;
+}
+__device__ __forceinline__ void delta_part(const DeltaToken& d, int which, float v) {
+  v = warp_sum_f32(v);
+  if ((threadIdx.x & 31) == 0) d.red[(threadIdx.x >> 5) * 4 + which] = v;
+}
+
+// Fills `d` for row `row` of head h (256 threads). The sums r . k and r . a u, and the vectors, are there behind the next barrier.
 template <typename T>
-__device__ __forceinline__ float2 delta_token(const DeltaParams<T>& p, const DeltaToken& d, const T* row, int h, float* red) {
-  const int dk = p.dk, qk = p.H * dk, vw = p.H * p.dv, n = blockDim.x;
+__device__ __forceinline__ void delta_token(const DeltaParams<T>& p, const DeltaToken& d, const T* row, int h) {
+  const int dk = p.dk, qk = p.H * dk, vw = p.H * p.dv;
   const T* low = row + 3 * qk + 2 * vw;
-  for (int i = threadIdx.x; i < p.rank; i += n) d.low[i] = tanhf(to_f32(low[i]));
   float ss = 0.f;
-  for (int i = threadIdx.x; i < dk; i += n) {
+  for (int i = threadIdx.x; i < dk; i += 256) {
     const float k = to_f32(row[qk + h * dk + i]);
     d.k[i] = k;
+    d.r[i] = to_f32(row[h * dk + i]);
+    d.au[i] = sigmoid_f32(to_f32(row[2 * qk + 2 * vw + h * dk + i]) + p.rate_b[h * dk + i]);
     ss += k * k;
   }
-  const float inv = 1.f / sqrtf(block_sum_f32(ss, red) + kUnitEps);        // its barriers also publish low
+  for (int i = threadIdx.x; i < p.rank; i += 256) d.low[i] = tanhf(to_f32(low[i]));
+  delta_part(d, 0, ss);
+  __syncthreads();
+  const float inv = 1.f / sqrtf(delta_sum(d, 0) + kUnitEps);
   float rk = 0.f, ra = 0.f;
-  for (int i = threadIdx.x; i < dk; i += n) {
+  for (int i = threadIdx.x; i < dk; i += 256) {
     const int c = h * dk + i;
     const float* w2 = p.w2 + static_cast<size_t>(c) * p.rank;
     float z = p.w0[c];
@@ -44,83 +60,119 @@ __device__ __forceinline__ float2 delta_token(const DeltaParams<T>& p, const Del
     } else {
       for (int j = 0; j < p.rank; ++j) z = fmaf(w2[j], d.low[j], z);
     }
-    const float r = to_f32(row[c]), k = d.k[i], u = k * inv;
-    const float au = sigmoid_f32(to_f32(row[2 * qk + 2 * vw + c]) + p.rate_b[c]) * u;
+    const float u = d.k[i] * inv, au = d.au[i] * u;
     d.w[i] = expm1f(-p.log_decay * sigmoid_f32(z));
-    d.r[i] = r;
     d.u[i] = u;
     d.au[i] = au;
-    rk = fmaf(r, k, rk);
-    ra = fmaf(r, au, ra);
+    rk = fmaf(d.r[i], d.k[i], rk);
+    ra = fmaf(d.r[i], au, ra);
   }
-  rk = block_sum_f32(rk, red);
-  ra = block_sum_f32(ra, red);                                             // and the vectors are visible
-  return make_float2(rk, ra);
+  delta_part(d, 1, rk);
+  delta_part(d, 2, ra);
+  __syncthreads();
 }
 
-// Norm over the head, output gate, store: os holds o of the head.
+// Norm over the head, output gate, store. A thread brings o of column j = threadIdx.x (and 256 on) in os; ends behind a barrier.
 template <typename T>
-__device__ __forceinline__ void delta_store(const DeltaParams<T>& p, const float* os, const T* row, size_t m, int h, float* red) {
+__device__ __forceinline__ void delta_store(const DeltaParams<T>& p, const DeltaToken& d, const float* os, const T* row, size_t m, int h) {
   const int qk = p.H * p.dk, vw = p.H * p.dv;
   float ss = 0.f;
-  for (int j = threadIdx.x; j < p.dv; j += blockDim.x) ss += os[j] * os[j];
-  const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / static_cast<float>(p.dv) + p.eps);
-  for (int j = threadIdx.x; j < p.dv; j += blockDim.x) {
+  for (int j = threadIdx.x; j < p.dv; j += 256) ss += os[j] * os[j];
+  delta_part(d, 3, ss);
+  __syncthreads();
+  const float inv = 1.f / sqrtf(delta_sum(d, 3) / static_cast<float>(p.dv) + p.eps);
+  for (int j = threadIdx.x; j < p.dv; j += 256) {
     const float g = to_f32(row[2 * qk + vw + h * p.dv + j]);
     p.out[m * vw + h * p.dv + j] = from_f32<T>(os[j] * inv * p.norm_w[h * p.dv + j] * sigmoid_f32(g));
   }
 }
 
+constexpr int kStepRank = 16;        // inputs of a channel's decay a thread keeps in registers
+
 // Decode steps and short portions, head sizes up to 128 in multiples of four: one CTA per (head, sequence), the state in registers for the
 // whole portion - a thread holds NR rows of four columns. Each token takes one pass for u^T S and (r w)^T S, since
-// o = (r w)^T S - (r . a u) u^T S + (r . k) v, and one for the update.
-template <typename T, int NR>
-__global__ void __launch_bounds__(256) delta_step_kernel(DeltaParams<T> p) {
+// o = (r w)^T S - (r . a u) u^T S + (r . k) v, and one for the update. TPC neighbouring threads share the decay of a key channel; what a
+// token needs is on its way at once, and the weights are fetched before the dependency wait.
+// DV > 0: value columns, and the rows of all threads together are the key channels; 0: any sizes.
+template <typename T, int NR, int TPC, int DV>
+__global__ void __launch_bounds__(256, NR <= 4 ? 4 : 2) delta_step_kernel(DeltaParams<T> p) {
   extern __shared__ float sm[];
-  __shared__ float red[8];
+  __shared__ float red[32];
   pdl_launch_early();
-  const int dk = p.dk, dv = p.dv, h = blockIdx.x;
+  const int dv = DV > 0 ? DV : p.dv, dk = DV > 0 ? NR * (1024 / (DV > 0 ? DV : 1)) : p.dk, h = blockIdx.x, tid = threadIdx.x;
   DeltaToken d;
+  d.red = red;
   d.r = sm;
   d.k = d.r + dk;
   d.w = d.k + dk;
   d.u = d.w + dk;
   d.au = d.u + dk;
-  float* os = d.au + dk;                                                   // [dv]
-  float* part = os + dv;                                                   // [groups][2][dv]
+  float* part = d.au + dk;                                                 // [parts][2][dv]
   const int per_row = dv / 4, groups = 256 / per_row;
-  d.low = part + 2 * groups * dv;
-  const int grp = threadIdx.x / per_row, c = (threadIdx.x % per_row) * 4;
-  const bool mine = grp < groups;
-  float4 S[NR];
+  // neighbouring row groups of a warp are summed with a shuffle where they fill it evenly
+  const bool paired = per_row == 16, lone = per_row == 16 || per_row == 32;
+  const int parts = paired ? 8 : groups;
+  d.low = part + 2 * parts * dv;
+  const int grp = tid / per_row, c = (tid % per_row) * 4;
+  const bool mine = lone || grp < groups;
+  const int ch = tid / TPC, sub = tid % TPC, qk = p.H * dk, vw = p.H * dv, ci = h * dk + min(ch, dk - 1);
+  const bool has = ch < dk;
+  // weights: nothing in the stream writes them
+  const int share = (p.rank + TPC - 1) / TPC, k0 = sub * share, kn = max(0, min(share, p.rank - k0));
+  const float* w2 = p.w2 + static_cast<size_t>(ci) * p.rank + k0;
+  float w2r[kStepRank / TPC];
 #pragma unroll
-  for (int i = 0; i < NR; ++i) S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-  auto load_state = [&](const float* st) {
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int r = grp + i * groups;
-      if (mine && r < dk) S[i] = load4(st + static_cast<size_t>(r) * dv + c);
-    }
-  };
-  // decode: nothing in front of this launch in the step writes the state, so it is fetched before the wait (an idle row fetches slot 0's)
+  for (int j = 0; j < kStepRank / TPC; ++j) w2r[j] = j < kn ? w2[j] : 0.f;
+  const float w0 = p.w0[ci], rate_b = p.rate_b[ci], norm_w = tid < dv ? p.norm_w[h * dv + tid] : 0.f;
+  // decode: nothing in front of this launch in the step writes the state or the tables, so it is fetched before the wait (an idle row fetches slot 0's)
   const bool early = p.seqs.cu_q == nullptr;
+  int slot = 0;
   if (early) {
-    const int slot = p.seqs.page_to_slot[p.seqs.block_table[static_cast<size_t>(blockIdx.y) * p.seqs.max_pages]];
+    slot = p.seqs.page_to_slot[p.seqs.block_table[static_cast<size_t>(blockIdx.y) * p.seqs.max_pages]];
     const char* base = reinterpret_cast<const char*>(p.state + (static_cast<size_t>(slot) * p.H + h) * dk * dv);
     const size_t bytes = static_cast<size_t>(dk) * dv * sizeof(float);
-    for (size_t o = threadIdx.x * 1024; o < bytes; o += 256 * 1024) bulk_prefetch_l2(base + o, static_cast<uint32_t>(bytes - o < 1024 ? bytes - o : 1024));
+    for (size_t o = tid * 1024; o < bytes; o += 256 * 1024) bulk_prefetch_l2(base + o, static_cast<uint32_t>(bytes - o < 1024 ? bytes - o : 1024));
   }
   pdl_wait();
   pdl_launch_dependents();
   const RaggedSeq s = ragged_seq(p.seqs, blockIdx.y);
   if (s.rows <= 0) return;                                                 // uniform
-  float* st = p.state + (static_cast<size_t>(s.slot) * p.H + h) * dk * dv;
-  if (s.live) load_state(st);
-  const int qk = p.H * dk;
+  if (!early) slot = s.slot;
+  float* st = p.state + (static_cast<size_t>(slot) * p.H + h) * dk * dv;
+  float4 S[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int r = grp + i * groups;
+    S[i] = mine && r < dk ? load4(st + static_cast<size_t>(r) * dv + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
   for (int t = 0; t < s.rows; ++t) {
     const size_t m = static_cast<size_t>(s.row0 + t);
     const T* row = p.proj + m * p.ld;
-    const float2 dots = delta_token(p, d, row, h, red);
+    const T* vr = row + 2 * qk + h * dv + c;
+    const float4 v = mine ? make_float4(to_f32(vr[0]), to_f32(vr[1]), to_f32(vr[2]), to_f32(vr[3])) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const float r0 = has ? to_f32(row[ci]) : 0.f, kv = has ? to_f32(row[qk + ci]) : 0.f;
+    const float rate = has ? to_f32(row[2 * qk + 2 * vw + ci]) : 0.f, gate = tid < dv ? to_f32(row[2 * qk + vw + h * dv + tid]) : 0.f;
+    for (int i = tid; i < p.rank; i += 256) d.low[i] = tanhf(to_f32(row[3 * qk + 2 * vw + i]));
+    delta_part(d, 0, sub == 0 ? kv * kv : 0.f);
+    __syncthreads();
+    float z = 0.f;
+#pragma unroll
+    for (int j = 0; j < kStepRank / TPC; ++j)
+      if (j < kn) z = fmaf(w2r[j], d.low[k0 + j], z);
+    for (int j = kStepRank / TPC; j < kn; ++j) z = fmaf(w2[j], d.low[k0 + j], z);
+#pragma unroll
+    for (int o = TPC >> 1; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+    const float u0 = kv * (1.f / sqrtf(delta_sum(d, 0) + kUnitEps)), au0 = sigmoid_f32(rate + rate_b) * u0;
+    if (has && sub == 0) {
+      d.r[ch] = r0;
+      d.k[ch] = kv;
+      d.w[ch] = expm1f(-p.log_decay * sigmoid_f32(z + w0));
+      d.u[ch] = u0;
+      d.au[ch] = au0;
+    }
+    delta_part(d, 1, sub == 0 ? r0 * kv : 0.f);
+    delta_part(d, 2, sub == 0 ? r0 * au0 : 0.f);
+    __syncthreads();
     if (mine) {
       float4 rec = make_float4(0.f, 0.f, 0.f, 0.f), o = rec;
 #pragma unroll
@@ -131,27 +183,37 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaParams<T> p) {
         rec = make_float4(fmaf(u, S[i].x, rec.x), fmaf(u, S[i].y, rec.y), fmaf(u, S[i].z, rec.z), fmaf(u, S[i].w, rec.w));
         o = make_float4(fmaf(rw, S[i].x, o.x), fmaf(rw, S[i].y, o.y), fmaf(rw, S[i].z, o.z), fmaf(rw, S[i].w, o.w));
       }
-      store4(part + (grp * 2) * dv + c, rec);
-      store4(part + (grp * 2 + 1) * dv + c, o);
+      if (paired) {                                                        // every thread is here
+        rec = make_float4(rec.x + __shfl_xor_sync(0xffffffffu, rec.x, 16), rec.y + __shfl_xor_sync(0xffffffffu, rec.y, 16),
+                          rec.z + __shfl_xor_sync(0xffffffffu, rec.z, 16), rec.w + __shfl_xor_sync(0xffffffffu, rec.w, 16));
+        o = make_float4(o.x + __shfl_xor_sync(0xffffffffu, o.x, 16), o.y + __shfl_xor_sync(0xffffffffu, o.y, 16),
+                        o.z + __shfl_xor_sync(0xffffffffu, o.z, 16), o.w + __shfl_xor_sync(0xffffffffu, o.w, 16));
+      }
+      const int at = paired ? grp >> 1 : grp;
+      if (!paired || (grp & 1) == 0) store4(part + (at * 2) * dv + c, rec);
+      if (!paired || (grp & 1) == 1) store4(part + (at * 2 + 1) * dv + c, o);
     }
     __syncthreads();
+    // o of the column that is this thread's
+    float o = 0.f;
+    if (tid < dv) {
+      float rec = 0.f;
+#pragma unroll 4
+      for (int g = 0; g < parts; ++g) {
+        rec += part[(g * 2) * dv + tid];
+        o += part[(g * 2 + 1) * dv + tid];
+      }
+      o = fmaf(delta_sum(d, 1), to_f32(row[2 * qk + h * dv + tid]), fmaf(-delta_sum(d, 2), rec, o));
+    }
+    delta_part(d, 3, o * o);
     if (mine) {
       float4 rec = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int g = 0; g < groups; ++g) {
+#pragma unroll 4
+      for (int g = 0; g < parts; ++g) {
         const float4 x = load4(part + (g * 2) * dv + c);
         rec = make_float4(rec.x + x.x, rec.y + x.y, rec.z + x.z, rec.w + x.w);
       }
-      const float4 v = make_float4(to_f32(row[2 * qk + h * dv + c]), to_f32(row[2 * qk + h * dv + c + 1]), to_f32(row[2 * qk + h * dv + c + 2]),
-                                   to_f32(row[2 * qk + h * dv + c + 3]));
-      if (grp == 0) {
-        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-        for (int g = 0; g < groups; ++g) {
-          const float4 x = load4(part + (g * 2 + 1) * dv + c);
-          o = make_float4(o.x + x.x, o.y + x.y, o.z + x.z, o.w + x.w);
-        }
-        store4(os + c, make_float4(fmaf(dots.x, v.x, fmaf(-dots.y, rec.x, o.x)), fmaf(dots.x, v.y, fmaf(-dots.y, rec.y, o.y)),
-                                   fmaf(dots.x, v.z, fmaf(-dots.y, rec.z, o.z)), fmaf(dots.x, v.w, fmaf(-dots.y, rec.w, o.w))));
-      }
+      const bool store = t + 1 == s.rows && s.live;
 #pragma unroll
       for (int i = 0; i < NR; ++i) {
         const int r = grp + i * groups;
@@ -159,30 +221,28 @@ __global__ void __launch_bounds__(256) delta_step_kernel(DeltaParams<T> p) {
         const float w = d.w[r], au = d.au[r], k = d.k[r];
         S[i] = make_float4(S[i].x + fmaf(w, S[i].x, fmaf(-au, rec.x, k * v.x)), S[i].y + fmaf(w, S[i].y, fmaf(-au, rec.y, k * v.y)),
                            S[i].z + fmaf(w, S[i].z, fmaf(-au, rec.z, k * v.z)), S[i].w + fmaf(w, S[i].w, fmaf(-au, rec.w, k * v.w)));
+        if (store) store4(st + static_cast<size_t>(r) * dv + c, S[i]);
       }
     }
     __syncthreads();
-    delta_store(p, os, row, m, h, red);
-    __syncthreads();
-  }
-  if (s.live && mine)
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int r = grp + i * groups;
-      if (r < dk) store4(st + static_cast<size_t>(r) * dv + c, S[i]);
+    if (tid < dv) {
+      const float inv = 1.f / sqrtf(delta_sum(d, 3) / static_cast<float>(dv) + p.eps);
+      p.out[m * vw + h * dv + tid] = from_f32<T>(o * inv * norm_w * sigmoid_f32(gate));
     }
+  }
 }
 
 // Any head size: the state stays in memory, a thread owns columns.
 template <typename T>
 __global__ void __launch_bounds__(256) delta_any_kernel(DeltaParams<T> p) {
   extern __shared__ float sm[];
-  __shared__ float red[8];
+  __shared__ float red[32];
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
   const int dk = p.dk, dv = p.dv, h = blockIdx.x;
   DeltaToken d;
+  d.red = red;
   d.r = sm;
   d.k = d.r + dk;
   d.w = d.k + dk;
@@ -197,7 +257,7 @@ __global__ void __launch_bounds__(256) delta_any_kernel(DeltaParams<T> p) {
   for (int t = 0; t < s.rows; ++t) {
     const size_t m = static_cast<size_t>(s.row0 + t);
     const T* row = p.proj + m * p.ld;
-    delta_token(p, d, row, h, red);
+    delta_token(p, d, row, h);
     for (int j = threadIdx.x; j < dv; j += 256) {
       const float v = to_f32(row[2 * qk + h * dv + j]);
       float rec = 0.f, o = 0.f;
@@ -213,7 +273,7 @@ __global__ void __launch_bounds__(256) delta_any_kernel(DeltaParams<T> p) {
       os[j] = o;
     }
     __syncthreads();
-    delta_store(p, os, row, m, h, red);
+    delta_store(p, d, os, row, m, h);
     __syncthreads();
   }
 }
@@ -227,9 +287,13 @@ static cudaError_t launch_delta_step(const DeltaParams<T>& p, cudaStream_t strea
     const int groups = 256 / (p.dv / 4), rows = (p.dk + groups - 1) / groups;
     const size_t smem = base + static_cast<size_t>(2) * groups * p.dv * sizeof(float);
     if (smem <= 48 * 1024) {
-      if (rows <= 4) return launch_pdl(delta_step_kernel<T, 4>, grid, dim3(256), smem, stream, p);
-      if (rows <= 8) return launch_pdl(delta_step_kernel<T, 8>, grid, dim3(256), smem, stream, p);
-      return launch_pdl(delta_step_kernel<T, 16>, grid, dim3(256), smem, stream, p);
+#define ER_STEP(NR_, TPC_, DV_) return launch_pdl(delta_step_kernel<T, NR_, TPC_, DV_>, grid, dim3(256), smem, stream, p)
+      if (p.dk == 64 && p.dv == 64) ER_STEP(4, 4, 64);
+      if (p.dk == 128 && p.dv == 128) ER_STEP(16, 2, 128);
+      if (rows <= 4) ER_STEP(4, 2, 0);
+      if (rows <= 8) ER_STEP(8, 2, 0);
+      ER_STEP(16, 2, 0);
+#undef ER_STEP
     }
   }
   if (base > 48 * 1024) return cudaErrorInvalidValue;

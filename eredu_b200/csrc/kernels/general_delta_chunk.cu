@@ -511,17 +511,26 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
   };
 #pragma unroll
   for (int c = 0; c + 1 < C::kStages; ++c) fetch(c);
-  for (int c = 0; c < chunks; ++c) {
-    DeltaCell<D>& now = cell[static_cast<size_t>(c) * p.H];
-    bf16 *sh = ss + (c & 1) * 2 * C::kSide, *sl = sh + C::kSide;
-    float2 nn[4][2], hh[4];
+  float2 nn[4][2], hh[4];                                                 // what the chunk adds and h^2, in flight a chunk ahead
+  auto ahead = [&](int c) {
+    const DeltaCell<D>& src = cell[static_cast<size_t>(min(c, chunks - 1)) * p.H];
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt) {
       const int i = i0 + nt * 8 + tig * 2;
-      hh[nt] = *reinterpret_cast<const float2*>(now.h2 + i);
+      hh[nt] = *reinterpret_cast<const float2*>(src.h2 + i);
+#pragma unroll
+      for (int r = 0; r < 2; ++r) nn[nt][r] = *reinterpret_cast<const float2*>(src.n + (j0 + g + r * 8) * D + i);
+    }
+  };
+  ahead(0);
+  for (int c = 0; c < chunks; ++c) {
+    DeltaCell<D>& now = cell[static_cast<size_t>(c) * p.H];
+    bf16 *sh = ss + (c & 1) * 2 * C::kSide, *sl = sh + C::kSide;
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt) {
+      const int i = i0 + nt * 8 + tig * 2;
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        nn[nt][r] = *reinterpret_cast<const float2*>(now.n + (j0 + g + r * 8) * D + i);
         uint32_t hi, lo;
         split2(x[nt][2 * r], x[nt][2 * r + 1], hi, lo);
         const int at = (tile * 16 + g + r * 8) * S + i, out = (j0 + g + r * 8) * D + i;
@@ -539,6 +548,7 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) x[nt][e] = fmaf((e & 1) ? hh[nt].y : hh[nt].x, x[nt][e], (e & 1) ? nn[nt][e >> 1].y : nn[nt][e >> 1].x);
+    ahead(c + 1);
 #pragma unroll
     for (int ks = 0; ks < D; ks += 16) {
       uint32_t ah[4], al[4];

@@ -232,24 +232,31 @@ struct BranchNormParams {
   float gain, eps;
 };
 
-// Sums of two values over the block.
-__device__ __forceinline__ float2 block_sum2_f32(float a, float b, float2* red) {
-  a = warp_sum_f32(a);
-  b = warp_sum_f32(b);
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
+// Sums over a block of 256 threads with one barrier; `red` is not used again.
+__device__ __forceinline__ float block_sum_once(float v, float* red) {
+  v = warp_sum_f32(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
   __syncthreads();
-  float2 t = make_float2(0.f, 0.f);
-  for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) t.x += red[w].x, t.y += red[w].y;
+  const float4 a = load4(red), b = load4(red + 4);
+  return ((a.x + a.y) + (a.z + a.w)) + ((b.x + b.y) + (b.z + b.w));
+}
+__device__ __forceinline__ float2 block_sum2_once(float u, float v, float* red) {
+  u = warp_sum_f32(u);
+  v = warp_sum_f32(v);
+  if ((threadIdx.x & 31) == 0) {
+    red[threadIdx.x >> 5] = u;
+    red[8 + (threadIdx.x >> 5)] = v;
+  }
   __syncthreads();
-  return t;
+  const float4 a = load4(red), b = load4(red + 4), c = load4(red + 8), d = load4(red + 12);
+  return make_float2(((a.x + a.y) + (a.z + a.w)) + ((b.x + b.y) + (b.z + b.w)), ((c.x + c.y) + (c.z + c.w)) + ((d.x + d.y) + (d.z + d.w)));
 }
 
 // x' = x + rms(gain (y0 + y1)) weight (each branch RMS-normed by itself first where it has a weight), act = rms(x') next. One CTA per row;
 // NV groups of four columns per thread stay in registers; NV = 0: any width, rows are read again.
 template <typename T, int NV>
 __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
-  __shared__ float2 red2[8];
-  __shared__ float red[8];
+  __shared__ __align__(16) float red2[16], red_y[8], red_x[8];
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
@@ -278,7 +285,7 @@ __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
         s1 += u[i].x * u[i].x + u[i].y * u[i].y + u[i].z * u[i].z + u[i].w * u[i].w;
       }
       if (p.w0 != nullptr) {
-        const float2 t = block_sum2_f32(s0, s1, red2);
+        const float2 t = block_sum2_once(s0, s1, red2);
         i0 = 1.f / sqrtf(t.x / n + p.eps);
         i1 = 1.f / sqrtf(t.y / n + p.eps);
       }
@@ -302,7 +309,7 @@ __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
-    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    const float inv = 1.f / sqrtf(block_sum_once(ss, red_y) / n + p.eps);
     ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -314,7 +321,7 @@ __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
       ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
     }
     if (p.next == nullptr) return;
-    const float out = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    const float out = 1.f / sqrtf(block_sum_once(ss, red_x) / n + p.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
       const int c = (threadIdx.x + i * 256) * 4;
@@ -330,7 +337,7 @@ __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
         s0 += a * a;
         s1 += b * b;
       }
-      const float2 t = block_sum2_f32(s0, s1, red2);
+      const float2 t = block_sum2_once(s0, s1, red2);
       i0 = 1.f / sqrtf(t.x / n + p.eps);
       i1 = 1.f / sqrtf(t.y / n + p.eps);
     }
@@ -344,7 +351,7 @@ __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
       const float m = mixed(c);
       ss += m * m;
     }
-    const float inv = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    const float inv = 1.f / sqrtf(block_sum_once(ss, red_y) / n + p.eps);
     ss = 0.f;
     for (int c = threadIdx.x; c < W; c += 256) {
       const float o = fmaf(mixed(c) * inv, p.weight[c], p.x[base + c]);
@@ -352,7 +359,7 @@ __global__ void __launch_bounds__(256) branch_norm_kernel(BranchNormParams p) {
       ss += o * o;
     }
     if (p.next == nullptr) return;
-    const float out = 1.f / sqrtf(block_sum_f32(ss, red) / n + p.eps);
+    const float out = 1.f / sqrtf(block_sum_once(ss, red_x) / n + p.eps);
     for (int c = threadIdx.x; c < W; c += 256) act[base + c] = from_f32<T>(p.x_out[base + c] * out * p.next[c]);
   }
 }

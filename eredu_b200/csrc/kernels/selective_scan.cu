@@ -13,6 +13,7 @@
 #include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
+#include "../common/mma.cuh"
 #include "../common/ptx.cuh"
 #include "../common/ragged.cuh"
 
@@ -23,14 +24,14 @@ struct ScanParams {
   const T* x;              // [M, C]
   const T* z;              // [M, ldz]
   const T* params;         // [M, ldp]
-  const float* dt;         // [M, C] W_dt low, or null: formed here
+  float* dt;               // [M, C] W_dt low, or null: formed here; the form below leaves finished step sizes in the tiles of its first launch
   const T* dt_w;           // [C, rank]
   const float* dt_b;       // [C]
   const float* A;          // [C, N]
   const float* D;          // [C]
   float* state;
   T* out;                  // [M, C]
-  float* maps;             // [B, tiles, C, N] what a tile adds, then [B, tiles, C] summed step sizes
+  float* maps;             // [B, tiles, N, C] what a tile adds, then [B, tiles, C] summed step sizes
   int C, N, rank, ldz, ldp, state_elems;
   int lanes, stage, tiles, tile_len;   // lanes of a channel; tokens staged at a time; tiles of the longest portion and their length
   RaggedBatch seqs;
@@ -89,7 +90,7 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(ScanParams
       const float dt = sums[static_cast<size_t>(j) * p.C + c];
 #pragma unroll
       for (int i = 0; i < NS; ++i)
-        if (n0 + i < p.N) S[i] = scan_step<T>(dt, a[i], S[i], maps[static_cast<size_t>(j) * p.C * p.N + cell + i]);
+        if (n0 + i < p.N) S[i] = scan_step<T>(dt, a[i], S[i], maps[(static_cast<size_t>(j) * p.N + n0 + i) * p.C + c]);
     }
   }
   float total = 0.f;
@@ -165,10 +166,9 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(ScanParams
   }
   if (!in) return;
   if (MAPS) {
-    float* map = maps + static_cast<size_t>(tile) * p.C * p.N + cell;
 #pragma unroll
     for (int i = 0; i < NS; ++i)
-      if (n0 + i < p.N) map[i] = S[i];
+      if (n0 + i < p.N) maps[(static_cast<size_t>(tile) * p.N + n0 + i) * p.C + c] = S[i];
     if (part == 0) sums[static_cast<size_t>(tile) * p.C + c] = total;
   } else if (s.live && t_end >= s.rows) {
 #pragma unroll
@@ -218,6 +218,10 @@ __device__ __forceinline__ float softplus_fast(float x) {
 }
 
 constexpr int kWideStage = 32;       // tokens of B and C staged at a time
+#ifndef EREDU_SCAN_POLY
+#define EREDU_SCAN_POLY 1
+#endif
+constexpr bool kWidePoly = EREDU_SCAN_POLY != 0;   // every eighth pair of exponentials on the FMA pipe
 constexpr int kWideAhead = 4;        // tokens whose channel values are in flight
 
 template <int NP, bool MAPS>
@@ -231,7 +235,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv
   const RaggedSeq s = ragged_seq(p.seqs, b);
   const int t_begin = tile * p.tile_len, t_end = min(s.rows, t_begin + p.tile_len);
   if (t_begin >= t_end) return;                                            // uniform
-  if (MAPS && t_end >= s.rows) return;                                     // nothing follows the last tile
+  const bool last = t_end >= s.rows, split = p.tiles > 1;                  // nothing follows the last tile: its first launch only forms step sizes
   const int c = blockIdx.x * kScanThreads + threadIdx.x;
   const bool in = c < p.C;
   const int cc = in ? c : 0;
@@ -256,7 +260,10 @@ __global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv
       const float dt = sums[static_cast<size_t>(j) * p.C + cc];
       const uint64_t d2 = pack_f32x2(dt, dt);
 #pragma unroll
-      for (int i = 0; i < NP; ++i) S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), false), S[i], state_pair(maps + static_cast<size_t>(j) * p.C * p.N + cell, i));
+      for (int i = 0; i < NP; ++i) {
+        const float* add = maps + (static_cast<size_t>(j) * p.N + 2 * i) * p.C + cc;
+        S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), false), S[i], pack_f32x2(2 * i < p.N ? add[0] : 0.f, 2 * i + 1 < p.N ? add[p.C] : 0.f));
+      }
     }
   }
   const float bias = p.dt_b[cc], d_skip = MAPS ? 0.f : p.D[cc];
@@ -281,6 +288,11 @@ __global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv
     }
   };
   float total = 0.f;
+  if (MAPS && last) {
+    if (in)
+      for (size_t m = m0 + t_begin; m < m0 + t_end; ++m) p.dt[m * p.C + c] = softplus_fast(p.dt[m * p.C + c] + bias);
+    return;
+  }
   fetch(t_begin);
   stage(t_begin, 0);
   int buf = 0;
@@ -292,7 +304,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv
       float dt[kWideAhead], x[kWideAhead], z[kWideAhead];
 #pragma unroll
       for (int u = 0; u < kWideAhead; ++u) {
-        dt[u] = softplus_fast(dn[u] + bias);
+        dt[u] = !MAPS && split ? dn[u] : softplus_fast(dn[u] + bias);
         x[u] = to_f32(xn[u]);
         z[u] = MAPS ? 0.f : to_f32(zn[u]);
       }
@@ -303,36 +315,123 @@ __global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv
         const uint64_t d2 = pack_f32x2(dt[u], dt[u]);
         const float dx = dt[u] * x[u];
         const uint64_t dx2 = pack_f32x2(dx, dx);
-        const uint64_t* bp = reinterpret_cast<const uint64_t*>(bc[buf][q + u][0]);
-        const uint64_t* cp = reinterpret_cast<const uint64_t*>(bc[buf][q + u][1]);
-        uint64_t y2 = 0ull;
+        const ulonglong2* bp = reinterpret_cast<const ulonglong2*>(bc[buf][q + u][0]);
+        const ulonglong2* cp = reinterpret_cast<const ulonglong2*>(bc[buf][q + u][1]);
+        uint64_t y2 = 0ull, y3 = 0ull;
 #pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), i % 8 >= 5), S[i], mul_f32x2(dx2, bp[i]));
-          if (!MAPS) y2 = fma_f32x2(S[i], cp[i], y2);
+        for (int i = 0; i < NP; i += 2) {
+          const ulonglong2 bb = bp[i / 2];
+          S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), false), S[i], mul_f32x2(dx2, bb.x));
+          S[i + 1] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i + 1]), kWidePoly && i % 8 == 6), S[i + 1], mul_f32x2(dx2, bb.y));
+          if (!MAPS) {
+            const ulonglong2 cv = cp[i / 2];
+            y2 = fma_f32x2(S[i], cv.x, y2);
+            y3 = fma_f32x2(S[i + 1], cv.y, y3);
+          }
         }
         if (MAPS) {
           total += dt[u];
+          if (in) p.dt[(m0 + t0 + q + u) * p.C + c] = dt[u];
         } else if (in) {
           float y0, y1;
-          unpack_f32x2(y2, y0, y1);
+          unpack_f32x2(add_f32x2(y2, y3), y0, y1);
           p.out[(m0 + t0 + q + u) * p.C + c] = __float2bfloat16(fmaf(d_skip, x[u], y0 + y1) * silu_fast(z[u]));
         }
       }
     }
   }
   if (!in) return;
-  float* dst = MAPS ? maps + static_cast<size_t>(tile) * p.C * p.N + cell : st;
   if (MAPS) sums[static_cast<size_t>(tile) * p.C + c] = total;
-  if (MAPS || (s.live && t_end >= s.rows)) {
+  if (MAPS || (s.live && last)) {
+    float* dst = MAPS ? maps + static_cast<size_t>(tile) * p.N * p.C + c : st;
+    const size_t step = MAPS ? p.C : 1;
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
       float s0, s1;
       unpack_f32x2(S[i], s0, s1);
-      if (2 * i < p.N) dst[2 * i] = s0;
-      if (2 * i + 1 < p.N) dst[2 * i + 1] = s1;
+      if (2 * i < p.N) dst[2 * i * step] = s0;
+      if (2 * i + 1 < p.N) dst[(2 * i + 1) * step] = s1;
     }
   }
+}
+
+// ---------------------------------------------------------------- decode steps in bf16
+// One token per sequence. A CTA takes 512 / N channels of up to eight sequences: the step sizes of all of them are one small product on the
+// tensor cores, so W_dt is read once for them, and a thread then updates four states of one channel for every sequence, all its states in flight.
+constexpr int kDecodeSeqs = 8;
+
+__global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(ScanParams<__nv_bfloat16> p) {
+  using T = __nv_bfloat16;
+  __shared__ float ds[kDecodeSeqs][64], xs[kDecodeSeqs][64], zs[kDecodeSeqs][64];
+  __shared__ __align__(16) float bc[kDecodeSeqs][128];                     // B, then C
+  __shared__ int slot_of[kDecodeSeqs];
+  pdl_launch_early();
+  const int quads = p.N / 4, per = kScanThreads / quads;                   // lanes of a channel, channels of the CTA
+  const int c0 = blockIdx.x * per, b0 = blockIdx.y * kDecodeSeqs, nb = min(kDecodeSeqs, p.seqs.B - b0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3;
+  const int ch = threadIdx.x / quads, quad = threadIdx.x % quads, c = c0 + ch;
+  const float4 a = load4(p.A + static_cast<size_t>(c) * p.N + quad * 4);   // weights: nothing in the stream writes them
+  const float bias = p.dt_b[c], d_skip = p.D[c];
+  pdl_wait();
+  pdl_launch_dependents();
+  if (threadIdx.x < kDecodeSeqs) {
+    int slot = -1;
+    if (threadIdx.x < nb) {
+      const RaggedSeq s = ragged_seq(p.seqs, b0 + threadIdx.x);
+      slot = s.live ? s.slot : -1;
+    }
+    slot_of[threadIdx.x] = slot;
+  }
+  for (int i = threadIdx.x; i < nb * per; i += kScanThreads) {
+    const int q = i / per, k = i - q * per;
+    const size_t m = b0 + q;
+    xs[q][k] = to_f32(p.x[m * p.C + c0 + k]);
+    zs[q][k] = to_f32(p.z[m * p.ldz + c0 + k]);
+  }
+  for (int i = threadIdx.x; i < nb * 2 * p.N; i += kScanThreads) {
+    const int q = i / (2 * p.N), k = i - q * 2 * p.N;
+    bc[q][k] = to_f32(p.params[static_cast<size_t>(b0 + q) * p.ldp + p.rank + k]);
+  }
+  // step sizes: rows are sequences (the upper eight of the product stay empty), a tile of eight channels per turn
+  for (int nt = warp; nt < per / 8; nt += kScanThreads / 32) {
+    const T* w = p.dt_w + static_cast<size_t>(c0 + nt * 8 + g) * p.rank + tig * 2;
+    const T* low = p.params + static_cast<size_t>(b0 + min(g, nb - 1)) * p.ldp + tig * 2;
+    float acc[2][4] = {};
+    auto ld = [](const T* q, bool in) { return in ? *reinterpret_cast<const uint32_t*>(q) : 0u; };
+#pragma unroll 8
+    for (int k = 0; k < p.rank; k += 16) {
+      const bool full = k + 8 < p.rank;                                    // rank is a multiple of eight
+      mma16816(acc[(k >> 4) & 1], ld(low + k, true), 0u, ld(low + k + 8, full), 0u, ld(w + k, true), ld(w + k + 8, full));
+    }
+    ds[g][nt * 8 + tig * 2] = acc[0][0] + acc[1][0];
+    ds[g][nt * 8 + tig * 2 + 1] = acc[0][1] + acc[1][1];
+  }
+  __syncthreads();
+  float4 S[kDecodeSeqs];
+  float* st = p.state + static_cast<size_t>(c) * p.N + quad * 4;
+#pragma unroll
+  for (int i = 0; i < kDecodeSeqs; ++i)
+    if (i < nb && slot_of[i] >= 0) S[i] = load4(st + static_cast<size_t>(slot_of[i]) * p.state_elems);
+#pragma unroll
+  for (int i = 0; i < kDecodeSeqs; ++i) {
+    const int slot = i < nb ? slot_of[i] : -1;
+    if (slot >= 0) {                                                       // uniform
+      const float dt = softplus_fast(ds[i][ch] + bias), x = xs[i][ch], dx = dt * x, d2 = dt * kLog2e;
+      const float4 bv = load4(&bc[i][quad * 4]), cv = load4(&bc[i][p.N + quad * 4]);
+      S[i] = make_float4(fmaf(ex2_approx(d2 * a.x), S[i].x, dx * bv.x), fmaf(ex2_approx(d2 * a.y), S[i].y, dx * bv.y),
+                         fmaf(ex2_approx(d2 * a.z), S[i].z, dx * bv.z), fmaf(ex2_approx(d2 * a.w), S[i].w, dx * bv.w));
+      store4(st + static_cast<size_t>(slot) * p.state_elems, S[i]);
+      float y = fmaf(S[i].x, cv.x, fmaf(S[i].y, cv.y, fmaf(S[i].z, cv.z, S[i].w * cv.w)));
+      for (int o = quads >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+      if (quad == 0) p.out[static_cast<size_t>(b0 + i) * p.C + c] = __float2bfloat16(fmaf(d_skip, x, y) * silu_fast(zs[i][ch]));
+    }
+  }
+}
+
+static bool scan_decode_ok(const ScanParams<__nv_bfloat16>& p) {
+  const int quads = p.N / 4;
+  return p.seqs.cu_q == nullptr && p.seqs.q_per_seq == 1 && p.dt == nullptr && p.N >= 8 && p.N <= 64 && (p.N & (p.N - 1)) == 0 &&
+         p.C % (kScanThreads / quads) == 0 && p.rank % 8 == 0 && p.ldp % 2 == 0 && p.state_elems % 4 == 0;
 }
 
 struct ScanShape {
@@ -361,7 +460,7 @@ static ScanShape scan_shape(int C, int N, int batch, int max_rows, int sm_count,
   // enough CTAs to fill the machine, in tiles of equal length
   const int per = s.wide ? kScanThreads : s.channels;
   const long long ctas = static_cast<long long>((C + per - 1) / per) * batch;
-  const long long want = tiled ? (8LL * (sm_count > 0 ? sm_count : 148) + ctas - 1) / ctas : 1;
+  const long long want = tiled ? (4LL * (sm_count > 0 ? sm_count : 148)) / ctas : 1;
   const int most = max_rows / kScanMinTile;
   s.tiles = static_cast<int>(want < most ? want : most);
   if (s.tiles < 1) s.tiles = 1;
@@ -397,12 +496,16 @@ static cudaError_t launch_scan_wide(const ScanParams<__nv_bfloat16>& p, const Sc
 }
 
 template <typename T>
-static cudaError_t run_scan(const void* x, const void* z, const void* params, const float* dt, const void* dt_w, const float* dt_b, const float* A,
+static cudaError_t run_scan(const void* x, const void* z, const void* params, float* dt, const void* dt_w, const float* dt_b, const float* A,
                             const float* D, float* state, void* out, float* scratch, const ScanShape& s, int C, int N, int rank, int ldz, int ldp,
                             int state_elems, const RaggedBatch& r, cudaStream_t stream) {
   const ScanParams<T> p = {static_cast<const T*>(x), static_cast<const T*>(z), static_cast<const T*>(params), dt, static_cast<const T*>(dt_w), dt_b, A, D,
                            state, static_cast<T*>(out), scratch, C, N, rank, ldz, ldp, state_elems, s.lanes, s.stage, s.tiles, s.tile_len, r};
   if constexpr (sizeof(T) == 2) {
+    if (scan_decode_ok(p)) {
+      const int per = kScanThreads / (N / 4);
+      return launch_pdl(scan_decode_kernel, dim3(C / per, (r.B + kDecodeSeqs - 1) / kDecodeSeqs), dim3(kScanThreads), 0, stream, p);
+    }
     if (s.wide) return N <= 8 ? launch_scan_wide<4>(p, s, stream) : N <= 16 ? launch_scan_wide<8>(p, s, stream) : launch_scan_wide<16>(p, s, stream);
   }
   return s.ns == 4 ? launch_scan<T, 4>(p, s, stream) : s.ns == 8 ? launch_scan<T, 8>(p, s, stream) : launch_scan<T, 16>(p, s, stream);
@@ -418,9 +521,9 @@ extern "C" long long eredu_selective_scan_scratch_elems(int channels, int states
   return s.tiles > 1 ? static_cast<long long>(batch) * s.tiles * channels * (states + 1LL) : 0;
 }
 
-// dt: fp32 [M, channels] = dt_w low, or null (formed in the kernel); scratch: fp32 [eredu_selective_scan_scratch_elems(...)] or null.
+// dt: fp32 [M, channels] = dt_w low (overwritten), or null (formed in the kernel); scratch: fp32 [eredu_selective_scan_scratch_elems(...)] or null.
 // At most 512 states a channel.
-extern "C" int eredu_selective_scan(const void* x, const void* z, const void* params, const float* dt, const void* dt_w, const float* dt_b,
+extern "C" int eredu_selective_scan(const void* x, const void* z, const void* params, float* dt, const void* dt_w, const float* dt_b,
                                     const float* A, const float* D, float* state, void* out, float* scratch, const int* block_table,
                                     const int* page_to_slot, const int* cu_q, const long long* slots, int channels, int states, int rank, int ldz,
                                     int ldp, int state_elems, int batch, int q_per_seq, int max_rows, int max_pages, int fp32, int sm_count,

@@ -435,7 +435,7 @@ def mlstm(proj, gates, norm_w, state, heads, dk, dv, cap, eps, batch, page_to_sl
 native.register("eredu_selective_scan", I, [P] * 15 + [I] * 12 + [P])
 native.register("eredu_selective_scan_scratch_elems", native.L, [I] * 6)
 
-# From this many rows a step size is worth a GEMM of its own in front of the scan (below, the scan multiplies it out).
+# Prompts of this many rows form their step sizes by a GEMM of its own in front of the scan (shorter ones and decode steps: in the scan).
 SCAN_STEP_GEMM_MIN_ROWS = 64
 
 
@@ -479,7 +479,7 @@ def selective_scan(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_t
         return out
     B = batch.block_table.shape[0]
     rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
-    dt = linear(params[:, :dt_rank], dt_w, out_dtype=torch.float32) if M >= SCAN_STEP_GEMM_MIN_ROWS else None
+    dt = linear(params[:, :dt_rank], dt_w, out_dtype=torch.float32) if M >= SCAN_STEP_GEMM_MIN_ROWS and (batch.is_prefill or x.dtype == torch.float32) else None
     elems = int(lib().eredu_selective_scan_scratch_elems(c, n, B, rows, _sm_count(x.device), 1 if x.dtype == torch.float32 else 0)) if dt is not None else 0
     scratch = torch.empty(elems, dtype=torch.float32, device=x.device) if elems else None
     code = lib().eredu_selective_scan(

@@ -182,12 +182,13 @@ def test_convolved_projections(dev, dt, H, G, dk, dv, rot, width, taps, ctaps, p
     for sizes in ([T], [1], [40, 1, 1, 2, 3, 64, 5, 34], [2, 1, 7, 90, 17, 33]):
         kc, vc = (torch.zeros(12, G, 16, d, device=dev, dtype=dt) for d in (dk, dv))
         pooled = tuple(torch.zeros(12, G, -(-16 // pool), d, device=dev, dtype=dt) for d in (dk, dv))
-        state = torch.zeros(3, 5 + hist + (ctaps - 1) * width, device=dev)
+        first = 4 if dk % 8 == 0 and taps != 4 else 5                             # histories at whole 16-byte pieces and elsewhere
+        state = torch.zeros(3, first + hist + (ctaps - 1) * width + (-(first + hist + (ctaps - 1) * width) % 4 if first == 4 else 0), device=dev)
         state[0] = 9.0
         p2s = torch.zeros(12, dtype=torch.int32, device=dev)
         p2s[table[0]] = 2
-        heads = ops.ConvHeads(f(ht), H, G, dk, dv, inv.to(dev), kc, vc, f(temp), pool, pooled, 5)
-        chans = ops.ConvChannels(f(ct), f(bias), start, 5 + hist)
+        heads = ops.ConvHeads(f(ht), H, G, dk, dv, inv.to(dev), kc, vc, f(temp), pool, pooled, first)
+        chans = ops.ConvChannels(f(ct), f(bias), start, first + hist)
         at, i, qs, cs = 0, 0, [], []
         while at < T:
             m = min(sizes[min(i, len(sizes) - 1)], T - at)
@@ -207,8 +208,8 @@ def test_convolved_projections(dev, dt, H, G, dk, dv, rot, width, taps, ctaps, p
         close(mk.transpose(0, 1), R.pooled(k, pool), dt, scale=float(k.abs().max()), limit=limit)
         close(mv.transpose(0, 1), R.pooled(v, pool), dt, scale=float(v.abs().max()))
         st = state[2].double().cpu()
-        close(st[5:5 + hist].view(taps - 1, n), x[T - taps + 1:, :n], torch.float32, scale=1.0)
-        close(st[5 + hist:].view(ctaps - 1, width), x[T - ctaps + 1:, start:start + width], torch.float32, scale=1.0)
+        close(st[first:first + hist].view(taps - 1, n), x[T - taps + 1:, :n], torch.float32, scale=1.0)
+        close(st[first + hist:first + hist + (ctaps - 1) * width].view(ctaps - 1, width), x[T - ctaps + 1:, start:start + width], torch.float32, scale=1.0)
         assert bool((state[0] == 9.0).all()) and not state[1].any()
         outside = [p for p in range(12) if p not in table]
         assert not kc[outside].any() and not pooled[0][outside].any()
@@ -330,7 +331,8 @@ PORTIONS = [[300], [1] * 12 + [40, 2, 2, 100, 64, 65, 15], [64, 128, 16, 8, 9, 7
 
 @both
 @pytest.mark.parametrize("portions", PORTIONS)
-@pytest.mark.parametrize("C,N,rank,kind", [(72, 20, 8, "plain"), (104, 16, 24, "keep"), (40, 130, 16, "swing"), (33, 5, 3, "swing"), (10, 1, 1, "plain"), (520, 32, 40, "keep")])
+@pytest.mark.parametrize("C,N,rank,kind", [(72, 20, 8, "plain"), (104, 16, 24, "keep"), (40, 130, 16, "swing"), (33, 5, 3, "swing"), (10, 1, 1, "plain"), (520, 32, 40, "keep"), (128, 16, 40, "swing"),
+                                           (48, 32, 8, "plain"), (192, 8, 16, "keep"), (40, 64, 72, "plain")])
 def test_selective_scan(dev, dt, C, N, rank, kind, portions):
     T = 300
     x, z, p, w, b, A, D = scan_inputs(T, C, N, rank, 7, kind)
@@ -345,7 +347,7 @@ def test_selective_scan(dev, dt, C, N, rank, kind, portions):
     while at < T:
         k = min(portions[min(i, len(portions) - 1)], T - at)
         g = lambda t: t[at:at + k].contiguous().to(dev, dt)                             # noqa: E731
-        bt = batch_of([(0, k)], [[1] * 20], dev)
+        bt = batch_of([(0, k)], [[1] * 20], dev, prefill=k > 1)
         outs.append(ops.selective_scan(g(x), g(zz)[:, 8:], g(p), rank, w.to(dev, dt).contiguous(), f(b), f(A), f(D), state, bt, p2s))
         at, i = at + k, i + 1
     close(torch.cat(outs), want, dt, limit=1e-4 if dt == torch.float32 else None)
@@ -355,7 +357,7 @@ def test_selective_scan(dev, dt, C, N, rank, kind, portions):
 
 @both
 def test_selective_scan_of_a_ragged_batch_and_idle_rows(dev, dt):
-    C, N, rank = 48, 12, 8
+    C, N, rank = 64, 16, 24
     rows, pages = [200, 1, 130, 2, 64, 17], [3, 1, 5, 2, 4, 6]
     x, z, p, w, b, A, D = scan_inputs(sum(rows), C, N, rank, 3, "plain")
     f = lambda t: t.float().contiguous().to(dev)                                        # noqa: E731
@@ -378,6 +380,33 @@ def test_selective_scan_of_a_ragged_batch_and_idle_rows(dev, dt):
     for i in range(6):
         slot = int(p2s[pages[i]])
         assert torch.equal(st[slot], st0[slot]) == (i in (1, 3))
+
+
+@both
+@pytest.mark.parametrize("C,N,rank", [(64, 16, 24), (96, 8, 8), (24, 64, 16), (40, 12, 5)])
+def test_scan_steps_of_many_sequences(dev, dt, C, N, rank):
+    """Decode steps of more sequences than a CTA takes, idle rows among them."""
+    n = 37
+    x, z, p, w, b, A, D = scan_inputs(n, C, N, rank, 3, "plain")
+    S0 = rand(n, C, N, seed=5)
+    st = torch.zeros(n + 1, C * N + 8, device=dev)
+    st[1:, :C * N] = S0.flip(0).reshape(n, -1).float().to(dev)                        # sequence i has slot n - i
+    p2s = torch.tensor([0] + [n - i for i in range(n)], dtype=torch.int32, device=dev)
+    bt = batch_of([(3, 1)] * n, [[i + 1] for i in range(n)], dev, prefill=False)
+    idle = [5, 16, 30]
+    bt.slots[idle] = -1
+    f = lambda t: t.float().contiguous().to(dev)                                        # noqa: E731
+    p = torch.cat((p, torch.zeros(n, -p.shape[1] % 8, dtype=torch.float64)), 1)
+    before = st.clone()
+    got = ops.selective_scan(x.to(dev, dt), z.to(dev, dt), p.to(dev, dt), rank, w.to(dev, dt).contiguous(), f(b), f(A), f(D), st, bt, p2s)
+    for i in range(n):
+        if i in idle:
+            assert torch.equal(st[n - i], before[n - i])
+            continue
+        y, S = R.selective_scan(x[i:i + 1], R.softplus(p[i:i + 1, :rank] @ w.t() + b), p[i:i + 1, rank:rank + N], p[i:i + 1, rank + N:rank + 2 * N], A, D, S0[i])
+        close(got[i:i + 1], y * R.silu(z[i:i + 1]), dt)
+        close(st[n - i, :C * N].view(C, N), S, torch.float32)
+    assert not st[0].any() and not st[:, C * N:].any()
 
 
 def delta_inputs(T, H, dk, dv, rank, seed, kind):
@@ -424,8 +453,8 @@ def test_generalised_delta_rule(dev, dt, H, dk, dv, rank, kind, c, portions):
     outs, at, i = [], 0, 0
     while at < T:
         k = min(portions[min(i, len(portions) - 1)], T - at)
-        outs.append(ops.general_delta(x[at:at + k].contiguous().to(dev, dt), *map(f, args[1:]), state, H, dk, dv, c, 1e-5, batch_of([(0, k)], [[1] * 20], dev),
-                                      p2s))
+        outs.append(ops.general_delta(x[at:at + k].contiguous().to(dev, dt), *map(f, args[1:]), state, H, dk, dv, c, 1e-5,
+                                      batch_of([(0, k)], [[1] * 20], dev, prefill=k > 1), p2s))
         at, i = at + k, i + 1
     close(torch.cat(outs), want, dt, limit=1e-4 if dt == torch.float32 else None)
     close(state[1], S, torch.float32, limit=1e-4)                       # the state is fp32 in both
