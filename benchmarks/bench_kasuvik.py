@@ -194,9 +194,7 @@ def kernel_numbers(size: str, T: int = 8192, Bn: int = 32, context: int = 2048, 
             x, s = rnd(M, 3 * C), torch.zeros(n, C, device=DEV)
             return lambda: ops.mingru_scan(x, s, C, bt, p2s)
 
-        io = M * (C * 10 + (R + 2 * N) * 2) + C * R * 2 + n * C * N * 8
-        if not prefill:
-            io -= M * C * 4
+        io = M * (C * 6 + (R + 2 * N) * 2) + C * R * 2 + n * C * N * 8
         mio = M * (C * 4 + 16 * 64 * 2 + MH * 4) + n * MH * 64 * 64 * 8
         add(f"{phase} selective_scan (step sizes, scan, gate)", io, 2.0 * M * C * R, scan, "mamba2_scan (closest model)", mamba2, mio, 4.0 * M * MH * 64 * 64)
         add(f"{phase} selective_scan (step sizes, scan, gate)", io, 2.0 * M * C * R, scan, "mingru_scan, equal channels", mingru, M * C * 8 + n * C * 8, 0)

@@ -49,6 +49,7 @@ struct PGemmParams {
   float norm_eps;
   float norm_inv_dim;
   float* ssq_out;
+  int out_fp32;  // plain tiles without residual and sums of squares: y is fp32
   int act;  // plain tiles: 2 = squared ReLU before the residual; dual tiles: 0 = silu(g) * u, 3 = relu(g) * u
   int n_tiles, m_tiles;
   // grouped form: m_tiles work items, used ones first (the rest have no rows); the expert's weights start at row expert * w_rows_per_expert
@@ -292,6 +293,14 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
               v[j] *= v[j];
             }
           }
+          if (!DUAL && p.out_fp32) {
+            if (item_ok[i]) {
+              float4* dst = reinterpret_cast<float4*>(static_cast<float*>(p.y) + static_cast<size_t>(m) * p.ldy + gn);
+              dst[0] = make_float4(v[0], v[1], v[2], v[3]);
+              dst[1] = make_float4(v[4], v[5], v[6], v[7]);
+            }
+            continue;
+          }
           const uint32_t r[4] = {rv[i].x, rv[i].y, rv[i].z, rv[i].w};
           uint4 o;
           o.x = pack_bf16x2(v[0] + bf16_lo(r[0]), v[1] + bf16_hi(r[0]));
@@ -330,8 +339,9 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
 int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* residual, const void* bias, int M, int N,
                            int K, int ldx, int ldw, int ldy, int ldr, int w_rows, int dual, int dual_row_offset,
                            int sm_count, int* status, const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim,
-                           float* ssq_out, int act, cudaStream_t stream) {
+                           float* ssq_out, int act, int out_fp32, cudaStream_t stream) {
   if (N % 8 != 0 || ldy % 8 != 0 || (reinterpret_cast<uintptr_t>(Y) & 15) != 0) return kPersistentUnsupported;
+  if (out_fp32 && (dual || residual != nullptr || ssq_out != nullptr)) return kPersistentUnsupported;
   if (dual && (ssq_out != nullptr || N % 64 != 0 || dual_row_offset % 8 != 0)) return kPersistentUnsupported;
   if (residual != nullptr && (ldr % 8 != 0 || (reinterpret_cast<uintptr_t>(residual) & 15) != 0)) return kPersistentUnsupported;
   CUtensorMap tmW, tmX;
@@ -356,6 +366,7 @@ int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* re
   p.norm_inv_dim = norm_dim > 0 ? 1.0f / static_cast<float>(norm_dim) : 0.f;
   p.ssq_out = ssq_out;
   p.act = act;
+  p.out_fp32 = out_fp32;
   p.n_tiles = dual ? (N + 63) / 64 : (N + 127) / 128;
   p.m_tiles = (M + kTN - 1) / kTN;
   const int total = p.n_tiles * p.m_tiles;

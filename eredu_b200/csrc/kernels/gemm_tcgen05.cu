@@ -799,12 +799,10 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   int tn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
   // a narrow output over many tokens (a router) fills the machine with small token tiles instead
   if (tn == 256 && out_fp32 && ((N + 127) / 128) * ((M + 255) / 256) * 2 <= sm_count) tn = 64;
-  // and so does an fp32 output of a short inner dimension, which is bound by its epilogue
-  if (tn == 256 && out_fp32 && K <= 512) tn = 64;
-  if (tn == 256 && !out_fp32 && force_split <= 1 && persistent_enabled()) {
+  if (tn == 256 && force_split <= 1 && persistent_enabled()) {
     // prefill-sized: persistent kernel with double-buffered accumulators
     const int pr = launch_gemm_persistent(X, W, Y, residual, bias, M, N, K, ldx, ldw, ldy, ldr, w_rows, dual, dual_row_offset,
-                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : 0,
+                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : 0, out_fp32,
                                          stream);
     if (pr != kPersistentUnsupported) return pr;
   }

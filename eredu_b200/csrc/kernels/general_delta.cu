@@ -305,8 +305,8 @@ static cudaError_t launch_delta_step(const DeltaParams<T>& p, cudaStream_t strea
 using namespace eredu;
 
 // Bytes of scratch a bf16 call over `rows` rows of `batch` sequences can use (0: the token-by-token kernel serves it).
-extern "C" long long eredu_general_delta_scratch_bytes(int heads, int dk, int dv, int rows, int batch, int max_rows) {
-  return delta_chunk_bytes(heads, dk, dv, rows, batch, max_rows);
+extern "C" long long eredu_general_delta_scratch_bytes(int heads, int dk, int dv, int rank, int rows, int batch, int max_rows) {
+  return delta_chunk_bytes(heads, dk, dv, rank, rows, batch, max_rows);
 }
 
 // scratch: [eredu_general_delta_scratch_bytes(...)] of a bf16 call whose rows are whole 16-byte pieces, or null (token by token).

@@ -24,7 +24,7 @@ struct DeltaParams {
 constexpr float kUnitEps = 1e-6f;    // added to a key's squared length
 
 // Chunk-parallel form for long bf16 portions (general_delta_chunk.cu): bytes of scratch it needs (0: not taken).
-long long delta_chunk_bytes(int H, int dk, int dv, int rows, int batch, int max_rows);
+long long delta_chunk_bytes(int H, int dk, int dv, int rank, int rows, int batch, int max_rows);
 bool delta_chunk_supported(const DeltaParams<__nv_bfloat16>& p);
 cudaError_t launch_delta_chunks(const DeltaParams<__nv_bfloat16>& p, int max_rows, void* scratch, cudaStream_t stream);
 

@@ -11,8 +11,8 @@
 //   O = Y S_in + Z,  S_out = h^2 S_in + M S_in + N,
 //   Y = (r~ - A_rb W) h,  Z = A_rk V - A_rb X,  M = -h (b~^T W) h,  N = h (k~^T V - b~^T X)
 // so three launches do it, and only the second walks a sequence:
-//   1. delta_chunk_kernel:  Y, Z, M, N, h^2 of every chunk. Scores by all warps, the inverses of the four diagonal blocks by one each;
-//      then a warp owns 16 columns of W or X from the substitution to what is stored, in registers.
+//   1. delta_chunk_kernel:  Y, Z, M, N, h^2 of every chunk. Scores by all warps (of u, later of r in their place), the inverses of the four
+//      diagonal blocks by one each; a warp owns 16 columns of W or X from the substitution to what is stored, in registers.
 //   2. delta_scan_kernel:   the state that enters every chunk, transposed; a few warps share 16 of its columns, the state stays in fp32
 //      registers and meets the others of its group in shared memory once per chunk.
 //   3. delta_out_kernel:    O, per-head norm, output gate.
@@ -33,9 +33,7 @@ namespace eredu {
 using bf16 = __nv_bfloat16;
 
 constexpr int kC = 64;               // tokens of a chunk
-constexpr int kCS = kC + 8;          // row stride of score tiles
 constexpr int kChunkMinRows = 16;    // from this portion length on the chunk-parallel form takes over
-constexpr int kDeltaMaxRank = 128;
 constexpr float kMaxLogDecay = 2.f;  // 32 c log2(e) stays below 2^93
 
 // What launch 1 leaves of one chunk and head, and launch 2 adds (`s`), head sizes padded to D.
@@ -54,11 +52,23 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   hi = pack_bf16x2(a, b);
   lo = pack_bf16x2(a - bf16_lo(hi), b - bf16_hi(hi));
 }
-// c += a b with both factors split
-__device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
-  mma16816(c, ah[0], ah[1], ah[2], ah[3], bh0, bh1);
-  mma16816(c, ah[0], ah[1], ah[2], ah[3], bl0, bl1);
-  mma16816(c, al[0], al[1], al[2], al[3], bh0, bh1);
+// c += a b with both factors split, for N n-tiles
+template <int N>
+__device__ __forceinline__ void mma_split(float (&c)[N][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[N][2], const uint32_t (&bl)[N][2]) {
+#pragma unroll
+  for (int n = 0; n < N; ++n) mma16816(c[n], ah[0], ah[1], ah[2], ah[3], bh[n][0], bh[n][1]);
+#pragma unroll
+  for (int n = 0; n < N; ++n) mma16816(c[n], ah[0], ah[1], ah[2], ah[3], bl[n][0], bl[n][1]);
+#pragma unroll
+  for (int n = 0; n < N; ++n) mma16816(c[n], al[0], al[1], al[2], al[3], bh[n][0], bh[n][1]);
+}
+// the same with a left factor that is exact in bf16
+template <int N>
+__device__ __forceinline__ void mma_left(float (&c)[N][4], const uint32_t (&f)[4], const uint32_t (&bh)[N][2], const uint32_t (&bl)[N][2]) {
+#pragma unroll
+  for (int n = 0; n < N; ++n) mma16816(c[n], f[0], f[1], f[2], f[3], bh[n][0], bh[n][1]);
+#pragma unroll
+  for (int n = 0; n < N; ++n) mma16816(c[n], f[0], f[1], f[2], f[3], bl[n][0], bl[n][1]);
 }
 __device__ __forceinline__ uint32_t ld32(const bf16* p) { return *reinterpret_cast<const uint32_t*>(p); }
 __device__ __forceinline__ void st32(bf16* p, uint32_t v) { *reinterpret_cast<uint32_t*>(p) = v; }
@@ -70,31 +80,67 @@ __device__ __forceinline__ void frag_a(const bf16* tile, int stride, int lane, u
 __device__ __forceinline__ void frag_at(const bf16* tile, int stride, int lane, uint32_t (&f)[4]) {
   ldsm_x4_t(smem_u32(tile + ((lane & 7) + (lane >> 4) * 8) * stride + ((lane >> 3) & 1) * 8), f[0], f[1], f[2], f[3]);
 }
-// B fragments (16 k x 16 columns, two n-tiles) of a row-major [k][n] tile: f[0], f[1] of the first eight columns, f[2], f[3] of the others
-__device__ __forceinline__ void frag_b(const bf16* tile, int stride, int lane, uint32_t (&f)[4]) {
-  ldsm_x4_t(smem_u32(tile + ((lane & 7) + ((lane >> 3) & 1) * 8) * stride + (lane >> 4) * 8), f[0], f[1], f[2], f[3]);
+// B fragments (16 k x 16 columns, two n-tiles) of a row-major [k][n] tile
+__device__ __forceinline__ void frag_b(const bf16* tile, int stride, int lane, uint32_t (&f)[2][2]) {
+  ldsm_x4_t(smem_u32(tile + ((lane & 7) + ((lane >> 3) & 1) * 8) * stride + (lane >> 4) * 8), f[0][0], f[0][1], f[1][0], f[1][1]);
+}
+// the same of a row-major [n][k] tile
+__device__ __forceinline__ void frag_bt(const bf16* tile, int stride, int lane, uint32_t (&f)[2][2]) {
+  ldsm_x4(smem_u32(tile + ((lane & 7) + (lane >> 4) * 8) * stride + ((lane >> 3) & 1) * 8), f[0][0], f[0][1], f[1][0], f[1][1]);
 }
 __device__ __forceinline__ int delta_chunk_id(const RaggedSeq& s, int b, int c) { return s.row0 / kC + b + c; }   // unique over the batch
+
+constexpr int kBS = 24, kBlock = 16 * kBS;   // row stride and size of a 16 x 16 block of scores
+__host__ __device__ constexpr int score_block(int I, int J) { return (I * (I + 1) / 2 + J) * kBlock; }
 
 template <int D>
 struct ChunkSmem {
   static constexpr int S = D + 8;    // row stride
-  bf16 rh[kC * S], rl[kC * S], kh[kC * S], kl[kC * S], bh[kC * S], bl[kC * S], uh[kC * S], ul[kC * S], v[kC * S];
+  bf16 rh[kC * S], rl[kC * S], kh[kC * S], kl[kC * S], bh[kC * S], bl[kC * S], v[kC * S];
+  bf16 uh[kC * S], ul[kC * S];       // first the decays' inputs, tanh hi and lo
   union {
-    struct {
-      bf16 ubh[kC * kCS], ubl[kC * kCS], ukh[kC * kCS], ukl[kC * kCS], rbh[kC * kCS], rbl[kC * kCS], rkh[kC * kCS], rkl[kC * kCS];
-    } a;                             // scores
-    struct {
-      float dec[kC * S];             // log2 decay since the start of the token's block of 16, inclusive
-      bf16 low[2 * kC * (kDeltaMaxRank + 8)];
-    } d;
+    float dec[kC * S];               // log2 decay since the start of the token's block of 16, inclusive
+    bf16 sc[4][10 * kBlock];         // scores up to the diagonal: against b hi, lo, against k hi, lo; of u first, then of r
   };
   float R[4 * D];                    // log2 decay at the starts of blocks 1, 2, 3 and at the end; later h in its first D
 };
 
+// Scores of one kind of row against b and k, in 16 x 16 blocks: below the diagonal (STRICT) or up to it.
+template <int D, bool STRICT>
+__device__ __forceinline__ void delta_scores(ChunkSmem<D>& s, const bf16* qh, const bf16* ql, int warp, int lane) {
+  constexpr int S = ChunkSmem<D>::S;
+  const int g = lane >> 2, tig = lane & 3;
+  for (int i = warp; i < 20; i += 8) {
+    const int blk = i >> 1, I = blk >= 6 ? 3 : blk >= 3 ? 2 : blk >= 1 ? 1 : 0, J = blk - I * (I + 1) / 2;
+    const bool is_k = i & 1;
+    const bf16 *xh = (is_k ? s.kh : s.bh) + J * 16 * S, *xl = (is_k ? s.kl : s.bl) + J * 16 * S;
+    float acc[2][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < D; ks += 16) {
+      uint32_t ah[4], al[4], bh[2][2], bl[2][2];
+      frag_a(qh + I * 16 * S + ks, S, lane, ah);
+      frag_a(ql + I * 16 * S + ks, S, lane, al);
+      frag_bt(xh + ks, S, lane, bh);
+      frag_bt(xl + ks, S, lane, bl);
+      mma_split(acc, ah, al, bh, bl);
+    }
+    bf16 *oh = s.sc[is_k ? 2 : 0] + blk * kBlock, *ol = s.sc[is_k ? 3 : 1] + blk * kBlock;
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int t = g + r * 8, c = h * 8 + tig * 2, last = I == J ? (STRICT ? t - 1 : t) : 16;   // last column that counts
+        uint32_t hi, lo;
+        split2(c <= last ? acc[h][2 * r] : 0.f, c + 1 <= last ? acc[h][2 * r + 1] : 0.f, hi, lo);
+        st32(oh + t * kBS + c, hi);
+        st32(ol + t * kBS + c, lo);
+      }
+  }
+}
+
 // ---------------------------------------------------------------- 1. chunks
 template <int D>
-__global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p, DeltaCell<D>* __restrict__ cells) {
+__global__ void __launch_bounds__(256, D == 64 ? 2 : 1) delta_chunk_kernel(DeltaParams<bf16> p, DeltaCell<D>* __restrict__ cells) {
   using Sm = ChunkSmem<D>;
   constexpr int S = Sm::S;
   extern __shared__ __align__(16) uint8_t raw[];
@@ -110,7 +156,7 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
   const bf16* rows = p.proj + static_cast<size_t>(seq.row0 + t0) * p.ld;
   DeltaCell<D>& cell = cells[static_cast<size_t>(delta_chunk_id(seq, b, blockIdx.x)) * p.H + hd];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3;
-  bf16 *low_h = s.d.low, *low_l = s.d.low + kC * rs;
+  bf16 *low_h = s.uh, *low_l = s.ul;
 
   // ---- rows of the chunk; rows behind the portion and channels behind the head size are zero
   constexpr int P = D / 8;
@@ -144,11 +190,11 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
   // ---- decays: a tile = one block of 16 tokens x 8 channels, summed along its tokens with shuffles
   for (int i = warp; i < 4 * (D / 8); i += 8) {
     const int blk = i & 3, c0 = (i >> 2) * 8;
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    float acc[1][4] = {};
     const int ch = c0 + g;
     const float* w2 = p.w2 + static_cast<size_t>(hd * dk + min(ch, dk - 1)) * rank;
     for (int ks = 0; ks < rs - 8; ks += 16) {
-      uint32_t ah[4], al[4], bh[2], bl[2];
+      uint32_t ah[4], al[4], bh[1][2], bl[1][2];
       frag_a(low_h + blk * 16 * rs + ks, rs, lane, ah);
       frag_a(low_l + blk * 16 * rs + ks, rs, lane, al);
 #pragma unroll
@@ -156,16 +202,16 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
         const int k = ks + tig * 2 + e * 8;
         const bool in = k < rank && ch < dk;                              // rank is a multiple of eight
         const float2 w = in ? *reinterpret_cast<const float2*>(w2 + k) : make_float2(0.f, 0.f);
-        split2(w.x, w.y, bh[e], bl[e]);
+        split2(w.x, w.y, bh[0][e], bl[0][e]);
       }
-      mma_split(acc, ah, al, bh[0], bh[1], bl[0], bl[1]);
+      mma_split(acc, ah, al, bh, bl);
     }
     const int c = c0 + tig * 2;
     float d[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int cc = c + (e & 1), t = blk * 16 + g + (e >> 1) * 8;
-      d[e] = cc < dk && t < n ? -p.log_decay * 1.4426950408889634f * sigmoid_fast(acc[e] + p.w0[hd * dk + cc]) : 0.f;
+      d[e] = cc < dk && t < n ? -p.log_decay * 1.4426950408889634f * sigmoid_fast(acc[0][e] + p.w0[hd * dk + cc]) : 0.f;
     }
 #pragma unroll
     for (int o = 4; o < 32; o <<= 1)
@@ -176,14 +222,14 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
       }
     d[2] += __shfl_sync(0xffffffffu, d[0], 28 + tig);
     d[3] += __shfl_sync(0xffffffffu, d[1], 28 + tig);
-    *reinterpret_cast<float2*>(s.d.dec + (blk * 16 + g) * S + c) = make_float2(d[0], d[1]);
-    *reinterpret_cast<float2*>(s.d.dec + (blk * 16 + g + 8) * S + c) = make_float2(d[2], d[3]);
+    *reinterpret_cast<float2*>(s.dec + (blk * 16 + g) * S + c) = make_float2(d[0], d[1]);
+    *reinterpret_cast<float2*>(s.dec + (blk * 16 + g + 8) * S + c) = make_float2(d[2], d[3]);
   }
   __syncthreads();
   for (int c = threadIdx.x; c < D; c += 256) {
     float acc = 0.f;
     for (int blk = 0; blk < 4; ++blk) {
-      acc += s.d.dec[(blk * 16 + 15) * S + c];
+      acc += s.dec[(blk * 16 + 15) * S + c];
       s.R[blk * D + c] = acc;
     }
     cell.h2[c] = ex2_approx(acc);
@@ -215,9 +261,9 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
       for (int q = 0; q < Q; ++q) {
         const int c = lane * 2 + q * 64, at = t * S + c;
         const uint32_t rr = ld32(s.rh + at), aa = ld32(s.bh + at);
-        const float2 dec = *reinterpret_cast<const float2*>(s.d.dec + at);
+        const float2 dec = *reinterpret_cast<const float2*>(s.dec + at);
         const float2 start = t < 16 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(s.R + ((t >> 4) - 1) * D + c);
-        const float2 before = (t & 15) == 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(s.d.dec + at - S);
+        const float2 before = (t & 15) == 0 ? make_float2(0.f, 0.f) : *reinterpret_cast<const float2*>(s.dec + at - S);
         const float l0 = start.x + dec.x - mid[2 * q], l1 = start.y + dec.y - mid[2 * q + 1];
         const float x0 = ex2_approx(start.x + before.x - mid[2 * q]), x1 = ex2_approx(start.y + before.y - mid[2 * q + 1]);
         const float e0 = ex2_approx(l0), e1 = ex2_approx(l1), i0 = ex2_approx(-l0), i1 = ex2_approx(-l1);
@@ -241,47 +287,17 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
   }
   __syncthreads();
   for (int c = threadIdx.x; c < D; c += 256) s.R[c] = ex2_approx(0.5f * s.R[3 * D + c]);      // h
-  // ---- scores: 16 x 16 blocks up to the diagonal of u and r against b and k
-  for (int i = warp; i < 40; i += 8) {
-    const int blk = i >> 2, I = blk >= 6 ? 3 : blk >= 3 ? 2 : blk >= 1 ? 1 : 0, J = blk - I * (I + 1) / 2;
-    const bool is_r = i & 1, is_k = i & 2;
-    const bf16 *qh = (is_r ? s.rh : s.uh) + I * 16 * S, *ql = (is_r ? s.rl : s.ul) + I * 16 * S;
-    const bf16 *xh = (is_k ? s.kh : s.bh) + J * 16 * S, *xl = (is_k ? s.kl : s.bl) + J * 16 * S;
-    float acc[2][4] = {};
-#pragma unroll
-    for (int ks = 0; ks < D; ks += 16) {
-      uint32_t ah[4], al[4];
-      frag_a(qh + ks, S, lane, ah);
-      frag_a(ql + ks, S, lane, al);
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int at = (h * 8 + g) * S + ks + tig * 2;
-        mma_split(acc[h], ah, al, ld32(xh + at), ld32(xh + at + 8), ld32(xl + at), ld32(xl + at + 8));
-      }
-    }
-    bf16* oh = (is_r ? (is_k ? s.a.rkh : s.a.rbh) : (is_k ? s.a.ukh : s.a.ubh)) + I * 16 * kCS + J * 16;
-    bf16* ol = (is_r ? (is_k ? s.a.rkl : s.a.rbl) : (is_k ? s.a.ukl : s.a.ubl)) + I * 16 * kCS + J * 16;
-#pragma unroll
-    for (int h = 0; h < 2; ++h)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int t = g + r * 8, c = h * 8 + tig * 2, last = I == J ? (is_r ? t : t - 1) : 16;   // last column that counts
-        uint32_t hi, lo;
-        split2(c <= last ? acc[h][2 * r] : 0.f, c + 1 <= last ? acc[h][2 * r + 1] : 0.f, hi, lo);
-        st32(oh + t * kCS + c, hi);
-        st32(ol + t * kCS + c, lo);
-      }
-  }
+  delta_scores<D, true>(s, s.uh, s.ul, warp, lane);
   __syncthreads();
   // ---- inverses of the unit lower-triangular diagonal blocks, in their place: a lane forms one column by substitution
   if (warp < 4) {
-    bf16 *lh = s.a.ubh + warp * 16 * (kCS + 1), *ll = s.a.ubl + warp * 16 * (kCS + 1);
+    bf16 *lh = s.sc[0] + score_block(warp, warp), *ll = s.sc[1] + score_block(warp, warp);
     float x[16];
 #pragma unroll
     for (int i = 0; i < 16; ++i) {
       float v = i == (lane & 15) ? 1.f : 0.f;
 #pragma unroll
-      for (int k = 0; k < i; ++k) v = fmaf(-(to_f32(lh[i * kCS + k]) + to_f32(ll[i * kCS + k])), x[k], v);
+      for (int k = 0; k < i; ++k) v = fmaf(-(to_f32(lh[i * kBS + k]) + to_f32(ll[i * kBS + k])), x[k], v);
       x[i] = v;
     }
     __syncwarp();
@@ -289,24 +305,23 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         const bf16 hi = __float2bfloat16(x[i]);
-        lh[i * kCS + lane] = hi;
-        ll[i * kCS + lane] = __float2bfloat16(x[i] - to_f32(hi));
+        lh[i * kBS + lane] = hi;
+        ll[i * kBS + lane] = __float2bfloat16(x[i] - to_f32(hi));
       }
   }
   __syncthreads();
   // ---- 16 columns of W (from u~) or of X (from A_uk V), transposed: rows are columns, block I covers the tokens 16 I ..
-  for (int grp = warp; grp < 2 * (D / 16); grp += 8) {
-    const bool is_w = grp < D / 16;
-    const int c0 = (is_w ? grp : grp - D / 16) * 16;
-    uint32_t nh[4][4], nl[4][4];                                          // -W^T or -X^T as A fragments, hi and lo
-    uint32_t vf[4][4];                                                    // V^T, X groups
-    if (!is_w) {
+  constexpr int G = D / 64;                                               // groups of columns a warp owns
+  auto group_is_w = [&](int gi) { return G == 1 ? warp < 4 : gi == 0; };
+  auto group_col = [&]() { return (G == 1 ? warp & 3 : warp) * 16; };
+  const int c0 = group_col();
+  uint32_t nh[G][4][4], nl[G][4][4];                                      // -W^T or -X^T as A fragments, hi and lo
 #pragma unroll
-      for (int J = 0; J < 4; ++J) frag_at(s.v + J * 16 * S + c0, S, lane, vf[J]);
-    }
+  for (int gi = 0; gi < G; ++gi) {
+    const bool is_w = group_is_w(gi);
 #pragma unroll
     for (int I = 0; I < 4; ++I) {
-      float acc[2][4];
+      float acc[2][4] = {};
       if (is_w) {
 #pragma unroll
         for (int h = 0; h < 2; ++h)
@@ -317,41 +332,44 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
           }
       } else {
 #pragma unroll
-        for (int h = 0; h < 2; ++h) acc[h][0] = acc[h][1] = acc[h][2] = acc[h][3] = 0.f;
-#pragma unroll
-        for (int J = 0; J <= I; ++J)
-#pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            const int at = (I * 16 + h * 8 + g) * kCS + J * 16 + tig * 2;
-            mma16816(acc[h], vf[J][0], vf[J][1], vf[J][2], vf[J][3], ld32(s.a.ukh + at), ld32(s.a.ukh + at + 8));
-            mma16816(acc[h], vf[J][0], vf[J][1], vf[J][2], vf[J][3], ld32(s.a.ukl + at), ld32(s.a.ukl + at + 8));
-          }
+        for (int J = 0; J <= I; ++J) {
+          uint32_t vf[4], bh[2][2], bl[2][2];
+          frag_at(s.v + J * 16 * S + c0, S, lane, vf);
+          frag_bt(s.sc[2] + score_block(I, J), kBS, lane, bh);
+          frag_bt(s.sc[3] + score_block(I, J), kBS, lane, bl);
+          mma_left(acc, vf, bh, bl);
+        }
       }
 #pragma unroll
-      for (int J = 0; J < I; ++J)
-#pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int at = (I * 16 + h * 8 + g) * kCS + J * 16 + tig * 2;
-          mma_split(acc[h], nh[J], nl[J], ld32(s.a.ubh + at), ld32(s.a.ubh + at + 8), ld32(s.a.ubl + at), ld32(s.a.ubl + at + 8));
-        }
-      uint32_t ah[4], al[4];
+      for (int J = 0; J < I; ++J) {
+        uint32_t bh[2][2], bl[2][2];
+        frag_bt(s.sc[0] + score_block(I, J), kBS, lane, bh);
+        frag_bt(s.sc[1] + score_block(I, J), kBS, lane, bl);
+        mma_split(acc, nh[gi][J], nl[gi][J], bh, bl);
+      }
+      uint32_t ah[4], al[4], ih[2][2], il[2][2];
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
         split2(acc[h][0], acc[h][1], ah[2 * h], al[2 * h]);
         split2(acc[h][2], acc[h][3], ah[2 * h + 1], al[2 * h + 1]);
       }
       float x[2][4] = {};
+      frag_bt(s.sc[0] + score_block(I, I), kBS, lane, ih);
+      frag_bt(s.sc[1] + score_block(I, I), kBS, lane, il);
+      mma_split(x, ah, al, ih, il);
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
-        const int at = (I * 16 + h * 8 + g) * kCS + I * 16 + tig * 2;
-        mma_split(x[h], ah, al, ld32(s.a.ubh + at), ld32(s.a.ubh + at + 8), ld32(s.a.ubl + at), ld32(s.a.ubl + at + 8));
-      }
-#pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        split2(-x[h][0], -x[h][1], nh[I][2 * h], nl[I][2 * h]);
-        split2(-x[h][2], -x[h][3], nh[I][2 * h + 1], nl[I][2 * h + 1]);
+        split2(-x[h][0], -x[h][1], nh[gi][I][2 * h], nl[gi][I][2 * h]);
+        split2(-x[h][2], -x[h][3], nh[gi][I][2 * h + 1], nl[gi][I][2 * h + 1]);
       }
     }
+  }
+  __syncthreads();                                                        // the scores of u are done with
+  delta_scores<D, false>(s, s.rh, s.rl, warp, lane);
+  __syncthreads();
+#pragma unroll
+  for (int gi = 0; gi < G; ++gi) {
+    const bool is_w = group_is_w(gi);
     // as B fragments (k: tokens, n: the 16 columns) block J is {n[J][0], n[J][2]} and {n[J][1], n[J][3]}
     // ---- Y or Z: rows are tokens
 #pragma unroll
@@ -374,20 +392,20 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
 #pragma unroll
       for (int J = 0; J <= I; ++J) {
         uint32_t ah[4], al[4];
-        frag_a(s.a.rbh + I * 16 * kCS + J * 16, kCS, lane, ah);
-        frag_a(s.a.rbl + I * 16 * kCS + J * 16, kCS, lane, al);
-        mma_split(acc[0], ah, al, nh[J][0], nh[J][2], nl[J][0], nl[J][2]);
-        mma_split(acc[1], ah, al, nh[J][1], nh[J][3], nl[J][1], nl[J][3]);
+        frag_a(s.sc[0] + score_block(I, J), kBS, lane, ah);
+        frag_a(s.sc[1] + score_block(I, J), kBS, lane, al);
+        const uint32_t bh[2][2] = {{nh[gi][J][0], nh[gi][J][2]}, {nh[gi][J][1], nh[gi][J][3]}};
+        const uint32_t bl[2][2] = {{nl[gi][J][0], nl[gi][J][2]}, {nl[gi][J][1], nl[gi][J][3]}};
+        mma_split(acc, ah, al, bh, bl);
         if (!is_w) {
-          uint32_t vb[4];
+          uint32_t vb[2][2];
           frag_b(s.v + J * 16 * S + c0, S, lane, vb);
-          frag_a(s.a.rkh + I * 16 * kCS + J * 16, kCS, lane, ah);
-          frag_a(s.a.rkl + I * 16 * kCS + J * 16, kCS, lane, al);
+          frag_a(s.sc[2] + score_block(I, J), kBS, lane, ah);
+          frag_a(s.sc[3] + score_block(I, J), kBS, lane, al);
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            mma16816(acc[h], ah[0], ah[1], ah[2], ah[3], vb[2 * h], vb[2 * h + 1]);
-            mma16816(acc[h], al[0], al[1], al[2], al[3], vb[2 * h], vb[2 * h + 1]);
-          }
+          for (int h = 0; h < 2; ++h) mma16816(acc[h], ah[0], ah[1], ah[2], ah[3], vb[h][0], vb[h][1]);
+#pragma unroll
+          for (int h = 0; h < 2; ++h) mma16816(acc[h], al[0], al[1], al[2], al[3], vb[h][0], vb[h][1]);
         }
       }
 #pragma unroll
@@ -405,67 +423,55 @@ __global__ void __launch_bounds__(256, 1) delta_chunk_kernel(DeltaParams<bf16> p
           }
         }
     }
-    if (is_w) {
-      // ---- M: rows are key channels
+    // ---- M (rows are key channels) or N transposed (rows are this warp's value columns)
+#pragma unroll 2
+    for (int it = 0; it < D / 16; ++it) {
+      float acc[2][4] = {};
 #pragma unroll
-      for (int it = 0; it < D / 16; ++it) {
-        float acc[2][4] = {};
-#pragma unroll
-        for (int J = 0; J < 4; ++J) {
+      for (int J = 0; J < 4; ++J) {
+        if (is_w) {
           uint32_t ah[4], al[4];
           frag_at(s.bh + J * 16 * S + it * 16, S, lane, ah);
           frag_at(s.bl + J * 16 * S + it * 16, S, lane, al);
-          mma_split(acc[0], ah, al, nh[J][0], nh[J][2], nl[J][0], nl[J][2]);
-          mma_split(acc[1], ah, al, nh[J][1], nh[J][3], nl[J][1], nl[J][3]);
+          const uint32_t bh[2][2] = {{nh[gi][J][0], nh[gi][J][2]}, {nh[gi][J][1], nh[gi][J][3]}};
+          const uint32_t bl[2][2] = {{nl[gi][J][0], nl[gi][J][2]}, {nl[gi][J][1], nl[gi][J][3]}};
+          mma_split(acc, ah, al, bh, bl);
+        } else {
+          uint32_t vf[4], bh[2][2], bl[2][2];
+          frag_b(s.bh + J * 16 * S + it * 16, S, lane, bh);
+          frag_b(s.bl + J * 16 * S + it * 16, S, lane, bl);
+          mma_split(acc, nh[gi][J], nl[gi][J], bh, bl);
+          frag_at(s.v + J * 16 * S + c0, S, lane, vf);
+          frag_b(s.kh + J * 16 * S + it * 16, S, lane, bh);
+          frag_b(s.kl + J * 16 * S + it * 16, S, lane, bl);
+          mma_left(acc, vf, bh, bl);
         }
+      }
 #pragma unroll
-        for (int h = 0; h < 2; ++h)
+      for (int h = 0; h < 2; ++h)
 #pragma unroll
-          for (int r = 0; r < 2; ++r) {
+        for (int r = 0; r < 2; ++r) {
+          if (is_w) {
             const int row = it * 16 + g + r * 8, c = c0 + h * 8 + tig * 2;
             uint32_t hi, lo;
             split2(acc[h][2 * r] * s.R[row] * s.R[c], acc[h][2 * r + 1] * s.R[row] * s.R[c + 1], hi, lo);
             st32(cell.mh + row * D + c, hi);
             st32(cell.ml + row * D + c, lo);
-          }
-      }
-    } else {
-      // ---- N transposed: rows are this warp's value columns
-#pragma unroll
-      for (int it = 0; it < D / 16; ++it) {
-        float acc[2][4] = {};
-#pragma unroll
-        for (int J = 0; J < 4; ++J) {
-          uint32_t bh[4], bl[4];
-          frag_b(s.bh + J * 16 * S + it * 16, S, lane, bh);
-          frag_b(s.bl + J * 16 * S + it * 16, S, lane, bl);
-#pragma unroll
-          for (int h = 0; h < 2; ++h) mma_split(acc[h], nh[J], nl[J], bh[2 * h], bh[2 * h + 1], bl[2 * h], bl[2 * h + 1]);
-          frag_b(s.kh + J * 16 * S + it * 16, S, lane, bh);
-          frag_b(s.kl + J * 16 * S + it * 16, S, lane, bl);
-#pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            mma16816(acc[h], vf[J][0], vf[J][1], vf[J][2], vf[J][3], bh[2 * h], bh[2 * h + 1]);
-            mma16816(acc[h], vf[J][0], vf[J][1], vf[J][2], vf[J][3], bl[2 * h], bl[2 * h + 1]);
-          }
-        }
-#pragma unroll
-        for (int h = 0; h < 2; ++h)
-#pragma unroll
-          for (int r = 0; r < 2; ++r) {
+          } else {
             const int c = it * 16 + h * 8 + tig * 2;
             *reinterpret_cast<float2*>(cell.n + (c0 + g + r * 8) * D + c) = make_float2(acc[h][2 * r] * s.R[c], acc[h][2 * r + 1] * s.R[c + 1]);
           }
-      }
+        }
     }
   }
 }
 
 // ---------------------------------------------------------------- 2. entering states
-// A CTA takes JT tiles of 16 value columns of one head; D / 32 warps share a tile, each with 32 key channels of the transposed state.
+// A CTA takes kTiles tiles of 16 value columns of one head; D / 16 warps share a tile, each with 16 key channels of the transposed state: a
+// step of the walk is bound by the instructions of one warp.
 template <int D>
 struct ScanCfg {
-  static constexpr int kParts = D / 32, kTiles = D == 64 ? 2 : 2, kWarps = kParts * kTiles, kThreads = 32 * kWarps;
+  static constexpr int kParts = D / 16, kTiles = D == 64 ? 1 : 2, kWarps = kParts * kTiles, kThreads = 32 * kWarps;
   static constexpr int kStages = D == 64 ? 3 : 2, S = D + 8;
   static constexpr int kStage = 2 * D * S;                                // M hi, lo (elements)
   static constexpr int kSide = kTiles * 16 * S;                           // state hi or lo of the CTA's tiles
@@ -487,12 +493,12 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
   if (!seq.live) return;                                                  // uniform
   const int chunks = (seq.rows + kC - 1) / kC;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3;
-  const int tile = warp / C::kParts, i0 = (warp % C::kParts) * 32, j0 = (blockIdx.x * C::kTiles + tile) * 16;
+  const int tile = warp / C::kParts, i0 = (warp % C::kParts) * 16, j0 = (blockIdx.x * C::kTiles + tile) * 16;
   DeltaCell<D>* cell = cells + static_cast<size_t>(delta_chunk_id(seq, b, 0)) * p.H + hd;
   float* st = p.state + (static_cast<size_t>(seq.slot) * p.H + hd) * p.dk * p.dv;
-  float x[4][4];                                                          // S^T: rows j0 + g (+ 8), columns i0 + nt * 8 + tig * 2 (+ 1)
+  float x[2][4];                                                          // S^T: rows j0 + g (+ 8), columns i0 + nt * 8 + tig * 2 (+ 1)
 #pragma unroll
-  for (int nt = 0; nt < 4; ++nt)
+  for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int j = j0 + g + (e >> 1) * 8, i = i0 + nt * 8 + tig * 2 + (e & 1);
@@ -511,11 +517,11 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
   };
 #pragma unroll
   for (int c = 0; c + 1 < C::kStages; ++c) fetch(c);
-  float2 nn[4][2], hh[4];                                                 // what the chunk adds and h^2, in flight a chunk ahead
+  float2 nn[2][2], hh[2];                                                 // what the chunk adds and h^2, in flight a chunk ahead
   auto ahead = [&](int c) {
     const DeltaCell<D>& src = cell[static_cast<size_t>(min(c, chunks - 1)) * p.H];
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
+    for (int nt = 0; nt < 2; ++nt) {
       const int i = i0 + nt * 8 + tig * 2;
       hh[nt] = *reinterpret_cast<const float2*>(src.h2 + i);
 #pragma unroll
@@ -527,7 +533,7 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
     DeltaCell<D>& now = cell[static_cast<size_t>(c) * p.H];
     bf16 *sh = ss + (c & 1) * 2 * C::kSide, *sl = sh + C::kSide;
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt) {
+    for (int nt = 0; nt < 2; ++nt) {
       const int i = i0 + nt * 8 + tig * 2;
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
@@ -543,26 +549,24 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
     cp_async_wait<C::kStages - 2>();
     __syncthreads();                                                      // M of this chunk has landed, the state is in shared memory
     fetch(c + C::kStages - 1);                                            // into the stage of the chunk before, which everyone has left
-    const bf16 *mh = ms + (c % C::kStages) * C::kStage + (i0 + g) * S + tig * 2, *ml = mh + D * S;
+    const bf16 *mh = ms + (c % C::kStages) * C::kStage + i0 * S, *ml = mh + D * S;
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
+    for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) x[nt][e] = fmaf((e & 1) ? hh[nt].y : hh[nt].x, x[nt][e], (e & 1) ? nn[nt][e >> 1].y : nn[nt][e >> 1].x);
     ahead(c + 1);
 #pragma unroll
     for (int ks = 0; ks < D; ks += 16) {
-      uint32_t ah[4], al[4];
+      uint32_t ah[4], al[4], bh[2][2], bl[2][2];
       frag_a(sh + tile * 16 * S + ks, S, lane, ah);
       frag_a(sl + tile * 16 * S + ks, S, lane, al);
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {
-        const int at = nt * 8 * S + ks;
-        mma_split(x[nt], ah, al, ld32(mh + at), ld32(mh + at + 8), ld32(ml + at), ld32(ml + at + 8));
-      }
+      frag_bt(mh + ks, S, lane, bh);
+      frag_bt(ml + ks, S, lane, bl);
+      mma_split(x, ah, al, bh, bl);
     }
   }
 #pragma unroll
-  for (int nt = 0; nt < 4; ++nt)
+  for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int j = j0 + g + (e >> 1) * 8, i = i0 + nt * 8 + tig * 2 + (e & 1);
@@ -620,9 +624,11 @@ __global__ void __launch_bounds__(256) delta_out_kernel(DeltaParams<bf16> p, con
     frag_a(yh + I * 16 * S + ks, S, lane, ah);
     frag_a(yl + I * 16 * S + ks, S, lane, al);
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      const int at = (j0 + nt * 8 + g) * S + ks + tig * 2;
-      mma_split(acc[nt], ah, al, ld32(sh + at), ld32(sh + at + 8), ld32(sl + at), ld32(sl + at + 8));
+    for (int n2 = 0; n2 < NT; n2 += 2) {
+      uint32_t bh[2][2], bl[2][2];
+      frag_bt(sh + (j0 + n2 * 8) * S + ks, S, lane, bh);
+      frag_bt(sl + (j0 + n2 * 8) * S + ks, S, lane, bl);
+      mma_split(*reinterpret_cast<float(*)[2][4]>(&acc[n2]), ah, al, bh, bl);
     }
   }
 #pragma unroll
@@ -654,9 +660,12 @@ __global__ void __launch_bounds__(256) delta_out_kernel(DeltaParams<bf16> p, con
 static bool chunk_sizes(int dk, int dv) { return dk % 8 == 0 && dv % 8 == 0 && dk > 0 && dv > 0 && dk <= 128 && dv <= 128; }
 static long long chunk_count(int rows, int batch) { return (rows + kC - 1) / kC + batch; }
 
-long long delta_chunk_bytes(int H, int dk, int dv, int rows, int batch, int max_rows) {
+// sizes padded to 64 or 128; the decays' inputs take the place of a tile
+static int chunk_width(int dk, int dv, int rank) { return dk <= 64 && dv <= 64 && rank <= 64 ? 64 : 128; }
+
+long long delta_chunk_bytes(int H, int dk, int dv, int rank, int rows, int batch, int max_rows) {
   if (max_rows < kChunkMinRows || !chunk_sizes(dk, dv)) return 0;
-  const long long cell = dk <= 64 && dv <= 64 ? sizeof(DeltaCell<64>) : sizeof(DeltaCell<128>);
+  const long long cell = chunk_width(dk, dv, rank) == 64 ? sizeof(DeltaCell<64>) : sizeof(DeltaCell<128>);
   return chunk_count(rows, batch) * H * cell;
 }
 
@@ -688,12 +697,12 @@ static cudaError_t launch_chunks(const DeltaParams<bf16>& p, int max_rows, void*
 }
 
 bool delta_chunk_supported(const DeltaParams<bf16>& p) {
-  return chunk_sizes(p.dk, p.dv) && p.rank % 8 == 0 && p.rank <= kDeltaMaxRank && p.log_decay <= kMaxLogDecay && p.ld % 8 == 0 &&
+  return chunk_sizes(p.dk, p.dv) && p.rank % 8 == 0 && p.rank <= 128 && p.log_decay <= kMaxLogDecay && p.ld % 8 == 0 &&
          (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0;
 }
 
 cudaError_t launch_delta_chunks(const DeltaParams<bf16>& p, int max_rows, void* scratch, cudaStream_t stream) {
-  return p.dk <= 64 && p.dv <= 64 ? launch_chunks<64>(p, max_rows, scratch, stream) : launch_chunks<128>(p, max_rows, scratch, stream);
+  return chunk_width(p.dk, p.dv, p.rank) == 64 ? launch_chunks<64>(p, max_rows, scratch, stream) : launch_chunks<128>(p, max_rows, scratch, stream);
 }
 
 }  // namespace eredu

@@ -492,7 +492,7 @@ def selective_scan(x, z, params, dt_rank, dt_w, dt_b, A, D, state, batch, page_t
 
 
 native.register("eredu_general_delta", I, [P] * 12 + [I] * 10 + [F, F, P])
-native.register("eredu_general_delta_scratch_bytes", native.L, [I] * 6)
+native.register("eredu_general_delta_scratch_bytes", native.L, [I] * 7)
 
 DELTA_UNIT_EPS = 1e-6        # added to the squared length of a key before it is made a unit vector
 
@@ -546,7 +546,7 @@ def general_delta(proj, w2, w0, rate_b, norm_w, state, heads, dk, dv, log_decay,
     rows = batch.max_q_len if batch.is_prefill else batch.q_per_seq
     scratch = None
     if proj.dtype == torch.bfloat16 and proj.data_ptr() % 16 == 0 and proj.stride(0) % 8 == 0 and rank % 8 == 0:
-        size = int(lib().eredu_general_delta_scratch_bytes(heads, dk, dv, M, B, rows))
+        size = int(lib().eredu_general_delta_scratch_bytes(heads, dk, dv, rank, M, B, rows))
         if size:
             scratch = torch.empty(size, dtype=torch.uint8, device=proj.device)
     code = lib().eredu_general_delta(

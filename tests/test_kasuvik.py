@@ -440,7 +440,7 @@ def delta_reference(x, w2, w0, rb, nw, H, dk, dv, c, eps, state):
 @pytest.mark.parametrize("portions", PORTIONS)
 @pytest.mark.parametrize("H,dk,dv,rank,kind,c", [(3, 40, 40, 16, "plain", 0.6), (2, 64, 64, 8, "keep", math.exp(-0.5)), (2, 64, 64, 24, "wipe", math.exp(-0.5)),
                                                  (1, 128, 128, 64, "plain", 0.3), (2, 128, 64, 16, "same", 0.6), (1, 24, 96, 40, "keep", 1.0), (3, 7, 5, 3, "plain", 0.6),
-                                                 (1, 132, 140, 8, "keep", 0.6), (2, 16, 16, 8, "same", 0.6)])
+                                                 (1, 132, 140, 8, "keep", 0.6), (2, 16, 16, 8, "same", 0.6), (1, 64, 48, 104, "plain", 0.6), (2, 128, 128, 24, "wipe", 0.6)])
 def test_generalised_delta_rule(dev, dt, H, dk, dv, rank, kind, c, portions):
     T = 300
     args = delta_inputs(T, H, dk, dv, rank, 7, kind)
