@@ -528,8 +528,21 @@ __global__ void __launch_bounds__(ScanCfg<D>::kThreads) delta_scan_kernel(DeltaP
       for (int r = 0; r < 2; ++r) nn[nt][r] = *reinterpret_cast<const float2*>(src.n + (j0 + g + r * 8) * D + i);
     }
   };
+  // what launch 1 left has gone to memory by now: it comes back to L2 some chunks ahead, M by shares of the CTAs of the head
+  constexpr int kAhead = 6;
+  auto warm = [&](int c) {
+    if (c >= chunks) return;
+    const DeltaCell<D>& src = cell[static_cast<size_t>(c) * p.H];
+    const uint32_t share = 4 * D * D / gridDim.x;
+    bulk_prefetch_l2(reinterpret_cast<const char*>(src.mh) + blockIdx.x * share, share);
+    bulk_prefetch_l2(src.n + blockIdx.x * C::kTiles * 16 * D, C::kTiles * 16 * D * sizeof(float));
+    if (blockIdx.x == 0) bulk_prefetch_l2(src.h2, D * sizeof(float));
+  };
+  if (threadIdx.x == 0)
+    for (int c = C::kStages - 1; c < kAhead; ++c) warm(c);
   ahead(0);
   for (int c = 0; c < chunks; ++c) {
+    if (threadIdx.x == 0) warm(c + kAhead);
     DeltaCell<D>& now = cell[static_cast<size_t>(c) * p.H];
     bf16 *sh = ss + (c & 1) * 2 * C::kSide, *sl = sh + C::kSide;
 #pragma unroll

@@ -218,14 +218,11 @@ __device__ __forceinline__ float softplus_fast(float x) {
 }
 
 constexpr int kWideStage = 32;       // tokens of B and C staged at a time
-#ifndef EREDU_SCAN_POLY
-#define EREDU_SCAN_POLY 1
-#endif
-constexpr bool kWidePoly = EREDU_SCAN_POLY != 0;   // every eighth pair of exponentials on the FMA pipe
+constexpr bool kWidePoly = true;     // one of every eight pairs of exponentials on the FMA pipe (none, two and three measured slower)
 constexpr int kWideAhead = 4;        // tokens whose channel values are in flight
 
 template <int NP, bool MAPS>
-__global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv_bfloat16> p) {
+__global__ void __launch_bounds__(kScanThreads, NP <= 8 ? 6 : 3) scan_wide_kernel(ScanParams<__nv_bfloat16> p) {
   using T = __nv_bfloat16;
   __shared__ __align__(16) float bc[2][kWideStage][2][2 * NP];             // buffer, token, B or C
   pdl_launch_early();
@@ -322,7 +319,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_wide_kernel(ScanParams<__nv
         for (int i = 0; i < NP; i += 2) {
           const ulonglong2 bb = bp[i / 2];
           S[i] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i]), false), S[i], mul_f32x2(dx2, bb.x));
-          S[i + 1] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i + 1]), kWidePoly && i % 8 == 6), S[i + 1], mul_f32x2(dx2, bb.y));
+          S[i + 1] = fma_f32x2(ex2_pair(mul_f32x2(d2, a[i + 1]), i % 8 == 0 && kWidePoly), S[i + 1], mul_f32x2(dx2, bb.y));
           if (!MAPS) {
             const ulonglong2 cv = cp[i / 2];
             y2 = fma_f32x2(S[i], cv.x, y2);
@@ -460,7 +457,7 @@ static ScanShape scan_shape(int C, int N, int batch, int max_rows, int sm_count,
   // enough CTAs to fill the machine, in tiles of equal length
   const int per = s.wide ? kScanThreads : s.channels;
   const long long ctas = static_cast<long long>((C + per - 1) / per) * batch;
-  const long long want = tiled ? (4LL * (sm_count > 0 ? sm_count : 148)) / ctas : 1;
+  const long long want = tiled ? (12LL * (sm_count > 0 ? sm_count : 148)) / ctas : 1;
   const int most = max_rows / kScanMinTile;
   s.tiles = static_cast<int>(want < most ? want : most);
   if (s.tiles < 1) s.tiles = 1;
