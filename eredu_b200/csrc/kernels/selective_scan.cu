@@ -361,24 +361,22 @@ __global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(ScanParams<__
   using T = __nv_bfloat16;
   __shared__ float ds[kDecodeSeqs][64], xs[kDecodeSeqs][64], zs[kDecodeSeqs][64];
   __shared__ __align__(16) float bc[kDecodeSeqs][128];                     // B, then C
-  __shared__ int slot_of[kDecodeSeqs];
+  __shared__ int slot_of[kDecodeSeqs], live[kDecodeSeqs];
   pdl_launch_early();
   const int quads = p.N / 4, per = kScanThreads / quads;                   // lanes of a channel, channels of the CTA
   const int c0 = blockIdx.x * per, b0 = blockIdx.y * kDecodeSeqs, nb = min(kDecodeSeqs, p.seqs.B - b0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tig = lane & 3;
   const int ch = threadIdx.x / quads, quad = threadIdx.x % quads, c = c0 + ch;
-  const float4 a = load4(p.A + static_cast<size_t>(c) * p.N + quad * 4);   // weights: nothing in the stream writes them
+  const float4 a = load4(p.A + static_cast<size_t>(c) * p.N + quad * 4);   // weights and tables: nothing in front of this launch writes them
   const float bias = p.dt_b[c], d_skip = p.D[c];
+  if (threadIdx.x < kDecodeSeqs)
+    slot_of[threadIdx.x] = threadIdx.x < nb ? p.seqs.page_to_slot[p.seqs.block_table[static_cast<size_t>(b0 + threadIdx.x) * p.seqs.max_pages]] : 0;
+  __syncthreads();
+  if (threadIdx.x < nb)                                                    // the states of these channels start towards L2
+    bulk_prefetch_l2(p.state + static_cast<size_t>(slot_of[threadIdx.x]) * p.state_elems + static_cast<size_t>(c0) * p.N, per * p.N * sizeof(float));
   pdl_wait();
   pdl_launch_dependents();
-  if (threadIdx.x < kDecodeSeqs) {
-    int slot = -1;
-    if (threadIdx.x < nb) {
-      const RaggedSeq s = ragged_seq(p.seqs, b0 + threadIdx.x);
-      slot = s.live ? s.slot : -1;
-    }
-    slot_of[threadIdx.x] = slot;
-  }
+  if (threadIdx.x < kDecodeSeqs) live[threadIdx.x] = threadIdx.x < nb && p.seqs.slots[b0 + threadIdx.x] >= 0;
   for (int i = threadIdx.x; i < nb * per; i += kScanThreads) {
     const int q = i / per, k = i - q * per;
     const size_t m = b0 + q;
@@ -408,16 +406,15 @@ __global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(ScanParams<__
   float* st = p.state + static_cast<size_t>(c) * p.N + quad * 4;
 #pragma unroll
   for (int i = 0; i < kDecodeSeqs; ++i)
-    if (i < nb && slot_of[i] >= 0) S[i] = load4(st + static_cast<size_t>(slot_of[i]) * p.state_elems);
+    if (i < nb) S[i] = load4(st + static_cast<size_t>(slot_of[i]) * p.state_elems);
 #pragma unroll
   for (int i = 0; i < kDecodeSeqs; ++i) {
-    const int slot = i < nb ? slot_of[i] : -1;
-    if (slot >= 0) {                                                       // uniform
+    if (i < nb && live[i]) {                                               // uniform
       const float dt = softplus_fast(ds[i][ch] + bias), x = xs[i][ch], dx = dt * x, d2 = dt * kLog2e;
       const float4 bv = load4(&bc[i][quad * 4]), cv = load4(&bc[i][p.N + quad * 4]);
       S[i] = make_float4(fmaf(ex2_approx(d2 * a.x), S[i].x, dx * bv.x), fmaf(ex2_approx(d2 * a.y), S[i].y, dx * bv.y),
                          fmaf(ex2_approx(d2 * a.z), S[i].z, dx * bv.z), fmaf(ex2_approx(d2 * a.w), S[i].w, dx * bv.w));
-      store4(st + static_cast<size_t>(slot) * p.state_elems, S[i]);
+      store4(st + static_cast<size_t>(slot_of[i]) * p.state_elems, S[i]);
       float y = fmaf(S[i].x, cv.x, fmaf(S[i].y, cv.y, fmaf(S[i].z, cv.z, S[i].w * cv.w)));
       for (int o = quads >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
       if (quad == 0) p.out[static_cast<size_t>(b0 + i) * p.C + c] = __float2bfloat16(fmaf(d_skip, x, y) * silu_fast(zs[i][ch]));
