@@ -89,7 +89,7 @@ __device__ __forceinline__ void load_row(const float* p, float (&v)[VEC], int nv
 
 // Walks one segment of a sequence for VEC neighbouring channels: `emit(t, y)` gets the convolved values of row t. Only the first
 // segment reads the old history and writes the new one, and a segment is at least as long as the history, so no other CTA
-// races it. L taps at compile time keep the window in registers and eight rows in flight; L = 0: any number, rows are read again.
+// races it. L taps at compile time keep the window in registers and four rows in flight; L = 0: any number, rows are read again.
 template <typename T, int VEC, int L, typename Emit>
 __device__ __forceinline__ void conv_walk(const T* col, int ld, const float* taps, int taps_ld, int n_taps, float* hist, int nv, int n, int t0, int t1, bool live, Emit emit) {
   auto input = [&](int t, float (&v)[VEC]) {
@@ -103,7 +103,7 @@ __device__ __forceinline__ void conv_walk(const T* col, int ld, const float* tap
     }
   };
   if constexpr (L > 0) {
-    constexpr int U = 8;
+    constexpr int U = 4;
     float w[L][VEC], win[L - 1][VEC];
 #pragma unroll
     for (int j = 0; j < L; ++j) load_row<VEC>(taps + static_cast<size_t>(j) * taps_ld, w[j], nv);
@@ -185,7 +185,7 @@ __device__ __forceinline__ void block_mean(const T* cache, const int* bt, int n_
 // Grid (blocks of channels: heads, then channels; segments; sequences). VEC = 4: head widths and columns are whole groups of four
 // channels, which a thread owns. VEC = 2: any width; a thread owns a pair of a head (or the last channel of an odd one).
 template <typename T, int VEC>
-__global__ void __launch_bounds__(kConvThreads, 4) conv_project_kernel(ConvProjectParams p) {
+__global__ void __launch_bounds__(kConvThreads, 7) conv_project_kernel(ConvProjectParams p) {
   __shared__ float cs[kConvSeg * kMaxRot / 2], sn[kConvSeg * kMaxRot / 2];
   pdl_launch_early();
   pdl_wait();
