@@ -82,6 +82,7 @@ FAMILY_SOURCES = {
                 "moe", "residual_stream", "simt_fp32"),
     "kasuvik": ("attention", "attention_tc", "conv_project", "gemm_persistent", "gemm_tcgen05", "general_delta", "general_delta_chunk",
                 "launch_count", "residual_stream", "selective_scan", "simt_fp32"),
+    "gulazen": ("gemm_persistent", "gemm_tcgen05", "launch_count", "moe", "residual_stream", "simt_fp32", "talking_attention"),
 }
 
 

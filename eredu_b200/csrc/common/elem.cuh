@@ -39,6 +39,16 @@ __device__ __forceinline__ float silu_fast(float x) { return x * sigmoid_fast(x)
 // log(sigmoid(x)) without overflow for either sign
 __device__ __forceinline__ float log_sigmoid_f32(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
 
+// xIELU: above z^2 + z / 2 for z > 0, below (e^z - 1 - z) + z / 2 elsewhere. Near zero e^z - 1 - z comes from its power series, where the
+// difference would cancel. FAST: the approximate exponential, for bf16 results.
+template <bool FAST>
+__device__ __forceinline__ float xielu(float z, float above, float below) {
+  const float n = fminf(z, 0.f);
+  const float series = n * n * fmaf(n, fmaf(n, fmaf(n, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
+  const float tail = n > -0.0625f ? series : (FAST ? __expf(n) : expf(n)) - 1.f - n;
+  return fmaf(0.5f, z, z > 0.f ? above * z * z : below * tail);
+}
+
 __device__ __forceinline__ float warp_sum_f32(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -17,6 +17,7 @@
 // (eredu-architectures/src/llama.rs:270-286,418-431; safemlx/src/ops/arithmetic.rs matmul).
 #include "gemm_persistent.h"
 
+#include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
 #include "../common/ptx.cuh"
@@ -50,7 +51,8 @@ struct PGemmParams {
   float norm_inv_dim;
   float* ssq_out;
   int out_fp32;  // plain tiles without residual and sums of squares: y is fp32
-  int act;  // plain tiles: 2 = squared ReLU before the residual; dual tiles: 0 = silu(g) * u, 3 = relu(g) * u
+  float act_a, act_b;  // xIELU
+  int act;  // plain tiles: 2 = squared ReLU before the residual, 4 = xIELU; dual tiles: 0 = silu(g) * u, 3 = relu(g) * u
   int n_tiles, m_tiles;
   // grouped form: m_tiles work items, used ones first (the rest have no rows); the expert's weights start at row expert * w_rows_per_expert
   const int4* work;
@@ -293,6 +295,10 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
               v[j] *= v[j];
             }
           }
+          if (!DUAL && p.act == 4) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = xielu<true>(v[j], p.act_a, p.act_b);
+          }
           if (!DUAL && p.out_fp32) {
             if (item_ok[i]) {
               float4* dst = reinterpret_cast<float4*>(static_cast<float*>(p.y) + static_cast<size_t>(m) * p.ldy + gn);
@@ -339,7 +345,7 @@ gemm_persistent_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_con
 int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* residual, const void* bias, int M, int N,
                            int K, int ldx, int ldw, int ldy, int ldr, int w_rows, int dual, int dual_row_offset,
                            int sm_count, int* status, const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim,
-                           float* ssq_out, int act, int out_fp32, cudaStream_t stream) {
+                           float* ssq_out, int act, float act_a, float act_b, int out_fp32, cudaStream_t stream) {
   if (N % 8 != 0 || ldy % 8 != 0 || (reinterpret_cast<uintptr_t>(Y) & 15) != 0) return kPersistentUnsupported;
   if (out_fp32 && (dual || residual != nullptr || ssq_out != nullptr)) return kPersistentUnsupported;
   if (dual && (ssq_out != nullptr || N % 64 != 0 || dual_row_offset % 8 != 0)) return kPersistentUnsupported;
@@ -366,6 +372,8 @@ int launch_gemm_persistent(const void* X, const void* W, void* Y, const void* re
   p.norm_inv_dim = norm_dim > 0 ? 1.0f / static_cast<float>(norm_dim) : 0.f;
   p.ssq_out = ssq_out;
   p.act = act;
+  p.act_a = act_a;
+  p.act_b = act_b;
   p.out_fp32 = out_fp32;
   p.n_tiles = dual ? (N + 63) / 64 : (N + 127) / 128;
   p.m_tiles = (M + kTN - 1) / kTN;

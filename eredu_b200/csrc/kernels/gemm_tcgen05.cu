@@ -20,6 +20,7 @@
 // (eredu/src/backend/mlx/nn/layers.rs:21-24).
 #include <cooperative_groups.h>
 
+#include "../common/elem.cuh"
 #include "../common/launch.h"
 #include "../common/launch_count.h"
 #include "../common/peer.cuh"
@@ -58,10 +59,11 @@ struct GemmParams {
   // Large token tiles: the epilogue goes through shared memory so that the output (and the residual) move as
   // 16-byte row chunks instead of one 2-byte element per thread. Needs 16-byte aligned rows (host-checked).
   int staged;
-  // Plain tiles: 2 = squared ReLU of the output (after bias, before the residual). Gated activation of DUAL tiles: 0 = silu(g) * u (SwiGLU); 1 = g * sigmoid(1.702 g) * (u + 1) (GPT-OSS); 3 = relu(g) * u. With
+  // Plain tiles: 2 = squared ReLU of the output (after bias, before the residual), 4 = xIELU with factors act_a and act_b. Gated activation of DUAL tiles: 0 = silu(g) * u (SwiGLU); 1 = g * sigmoid(1.702 g) * (u + 1) (GPT-OSS); 3 = relu(g) * u. With
   // act_limit > 0 the gate is clamped from above and the linear branch to [-limit, limit] first
   // (eredu/src/backend/mlx/architectures/gpt_oss/model.rs:748-753; nn/moe.rs swiglu_limit).
   int act;
+  float act_a, act_b;
   float act_limit;
   int bias_expert_stride;  // grouped mode: elements between two experts' bias vectors (0 = one shared vector)
   // Weights that no kernel of the stream rewrites (every model weight): their first tiles are fetched, and the
@@ -115,6 +117,8 @@ __device__ __forceinline__ float plain_act(const GemmParams& p, float g) {
   if (p.act == 2) {
     g = fmaxf(g, 0.f);
     g *= g;
+  } else if (p.act == 4) {
+    g = xielu<true>(g, p.act_a, p.act_b);
   }
   return g;
 }
@@ -794,7 +798,8 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
                                int N, int K, int ldx, int ldw, int ldy, int ldr, int w_rows, int dual,
                                int dual_row_offset, int out_fp32, int force_split, int sm_count, int* status,
                                const float* ssq_in, int ssq_parts, float norm_eps, int norm_dim, float* ssq_out,
-                               int flags, cudaStream_t stream) {
+                               int flags, float act_a, float act_b, cudaStream_t stream) {
+  const int act = dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : (flags & 8) ? 4 : 0;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   int tn = M <= 16 ? 16 : M <= 32 ? 32 : M <= 64 ? 64 : M <= 128 ? 128 : 256;
   // a narrow output over many tokens (a router) fills the machine with small token tiles instead
@@ -802,8 +807,8 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   if (tn == 256 && force_split <= 1 && persistent_enabled()) {
     // prefill-sized: persistent kernel with double-buffered accumulators
     const int pr = launch_gemm_persistent(X, W, Y, residual, bias, M, N, K, ldx, ldw, ldy, ldr, w_rows, dual, dual_row_offset,
-                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : 0, out_fp32,
-                                         stream);
+                                          sm_count, status, ssq_in, ssq_parts, norm_eps, norm_dim, ssq_out, act, act_a, act_b, out_fp32,
+                                          stream);
     if (pr != kPersistentUnsupported) return pr;
   }
   CUtensorMap tmW, tmX;
@@ -832,10 +837,12 @@ extern "C" int eredu_gemm_bf16(const void* X, const void* W, void* Y, const void
   p.work = nullptr;
   p.w_rows_per_expert = 0;
   p.staged = 0;
-  p.act = dual ? ((flags & 4) ? 3 : 0) : (flags & 2) ? 2 : 0;
+  p.act = act;
+  p.act_a = act_a;
+  p.act_b = act_b;
   p.act_limit = 0.f;
   p.bias_expert_stride = 0;
-  // flag bit 1: squared ReLU of the output (plain tiles). Flag bit 2: ReLU instead of SiLU of the gate (dual tiles). Flag bit 0: W was produced by a preceding kernel of the stream (no early fetch at all). Otherwise the ring's
+  // flag bit 1: squared ReLU of the output (plain tiles), bit 3: xIELU with factors act_a and act_b. Flag bit 2: ReLU instead of SiLU of the gate (dual tiles). Flag bit 0: W was produced by a preceding kernel of the stream (no early fetch at all). Otherwise the ring's
   // first stages are fetched before the dependency wait (level 1), and for matrices that fit L2 many times over
   // the remaining tiles are prefetched into L2 as well (level 2). EREDU_GEMM_PREFETCH overrides the level.
   p.w_static = (flags & 1) ? 0 : prefetch_level(static_cast<long long>(w_rows) * K * 2);
@@ -916,6 +923,7 @@ extern "C" int eredu_gemm_bf16_comm(const void* X, const void* W, void* Y, const
   p.w_rows_per_expert = 0;
   p.staged = 0;
   p.act = 0;
+  p.act_a = p.act_b = 0.f;
   p.act_limit = 0.f;
   p.bias_expert_stride = 0;
   p.w_static = prefetch_level(static_cast<long long>(w_rows) * K * 2);
@@ -980,6 +988,7 @@ extern "C" int eredu_gemm_bf16_grouped(const void* X, const void* W, void* Y, co
   p.bias = bias;  // per expert: [w_rows_per_expert] (dual: gate part then up part), bias_expert_stride apart
   p.bias_expert_stride = bias_expert_stride;
   p.act = act;
+  p.act_a = p.act_b = 0.f;
   p.act_limit = act_limit;
   const int n_tiles = (N + 127) / 128;
   const int kblocks = (K + 63) / 64;

@@ -4,7 +4,9 @@
 //     projections read (one number or one vector as w; without a residual: a plain norm, as in front of the head)
 //   * branch_norm (norms in front of and behind a sublayer): x' = x + w rms(gain (y0 + y1)), the branches normed by themselves first
 //     where they have weights, and the norm of x' in front of the next sublayer
-//   * embedding_stream: the first rows of the stream and their copy
+//   * rms_routed_residual: rms_residual of a sublayer's output plus weighted expert rows; the copy may be x + conv(x) in decode steps
+//   * stream_conv: x + conv(x), a causal convolution over the stream with the last inputs as state
+//   * embedding_stream: the first rows of the stream and their copy, with sinusoidal position vectors where a model adds them
 //   * qkv_prepare: RMSNorm over the WHOLE query and key projections, rotation of the leading dims of every head, RMSNorm of
 //     every value head, and the append to the paged cache, whose key and value widths may differ
 // All of them for bf16 and for fp32 activations.
@@ -12,6 +14,7 @@
 #include "../common/launch.h"
 #include "../common/launch_count.h"
 #include "../common/ptx.cuh"
+#include "../common/ragged.cuh"
 
 namespace eredu {
 
@@ -382,9 +385,257 @@ static cudaError_t launch_branch_norm(const BranchNormParams& p, int M, bool qua
 #undef ER_BN
 }
 
+struct RoutedResidualParams {
+  const void* y;            // [M, W] a sublayer's output, or null
+  const void* rows;         // expert outputs, or null
+  const int* route_pos;     // [M * k] row of a route, negative: none
+  const float* route_w;     // [M * k]
+  const float* weight;      // [W]
+  const float* residual;    // [M, W]
+  float* x_out;             // [M, W]
+  void* act;                // [M, W] or null
+  // decode steps of one row per sequence: act = x' + conv(x')
+  const float* taps;        // [taps, W] or null
+  float* state;             // [slots, state_elems] of which the first (taps - 1) W are the last inputs, oldest first; null: one tap
+  RaggedBatch seqs;
+  int n_taps, state_elems;
+  int W, k;
+  float eps;
+};
+
+// One CTA per row: x' = residual + weight rms(y + sum_k w_k rows_k). NV groups of four columns per thread stay in registers; NV = 0: any
+// width, the sum is formed twice.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidualParams p) {
+  __shared__ __align__(16) float red[8];
+  __shared__ int pos[kMaxRoutes];
+  __shared__ float rw[kMaxRoutes];
+  pdl_launch_early();
+  const int W = p.W;
+  pdl_wait();
+  pdl_launch_dependents();
+  const size_t base = static_cast<size_t>(blockIdx.x) * W;
+  const T* y = p.y != nullptr ? static_cast<const T*>(p.y) + base : nullptr;
+  const T* rows = static_cast<const T*>(p.rows);
+  T* act = p.act != nullptr ? static_cast<T*>(p.act) + base : nullptr;
+  if (p.k > 0) {
+    if (threadIdx.x < p.k) {
+      pos[threadIdx.x] = p.route_pos[static_cast<size_t>(blockIdx.x) * p.k + threadIdx.x];
+      rw[threadIdx.x] = p.route_w[static_cast<size_t>(blockIdx.x) * p.k + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float* hist = nullptr;
+  if (p.state != nullptr) {
+    const RaggedSeq s = ragged_seq(p.seqs, blockIdx.x);
+    if (s.live) hist = p.state + static_cast<size_t>(s.slot) * p.state_elems;
+  }
+  const float n = static_cast<float>(W);
+  if constexpr (NV > 0) {
+    float4 v[NV], rv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      v[i] = rv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < W) {
+        if (y != nullptr) v[i] = load4(y + c);
+        rv[i] = load4(p.residual + base + c);
+      }
+    }
+#pragma unroll 4
+    for (int s = 0; s < p.k; ++s) {
+      if (pos[s] < 0) continue;
+      const T* r = rows + static_cast<size_t>(pos[s]) * W;
+      const float w = rw[s];
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * 256) * 4;
+        if (c >= W) continue;
+        const float4 a = load4(r + c);
+        v[i] = make_float4(fmaf(w, a.x, v[i].x), fmaf(w, a.y, v[i].y), fmaf(w, a.z, v[i].z), fmaf(w, a.w, v[i].w));
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    const float inv = 1.f / sqrtf(block_sum_once(ss, red) / n + p.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (threadIdx.x + i * 256) * 4;
+      if (c >= W) continue;
+      const float4 g = load4(p.weight + c);
+      const float4 o = make_float4(fmaf(v[i].x * inv, g.x, rv[i].x), fmaf(v[i].y * inv, g.y, rv[i].y), fmaf(v[i].z * inv, g.z, rv[i].z),
+                                   fmaf(v[i].w * inv, g.w, rv[i].w));
+      store4(p.x_out + base + c, o);
+      if (act == nullptr) continue;
+      float4 h = o;
+      if (p.taps != nullptr) {
+        for (int j = 0; j < p.n_taps; ++j) {
+          const float4 t = load4(p.taps + static_cast<size_t>(j) * W + c);
+          const bool own = j == p.n_taps - 1;
+          if (!own && hist == nullptr) continue;
+          const float4 u = own ? o : load4(hist + static_cast<size_t>(j) * W + c);
+          if (j > 0 && hist != nullptr) store4(hist + static_cast<size_t>(j - 1) * W + c, u);
+          h = make_float4(fmaf(t.x, u.x, h.x), fmaf(t.y, u.y, h.y), fmaf(t.z, u.z, h.z), fmaf(t.w, u.w, h.w));
+        }
+      }
+      store4(act + c, h);
+    }
+  } else {
+    auto summed = [&](int c) {
+      float t = y != nullptr ? to_f32(y[c]) : 0.f;
+      for (int s = 0; s < p.k; ++s)
+        if (pos[s] >= 0) t = fmaf(rw[s], to_f32(rows[static_cast<size_t>(pos[s]) * W + c]), t);
+      return t;
+    };
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float t = summed(c);
+      ss += t * t;
+    }
+    const float inv = 1.f / sqrtf(block_sum_once(ss, red) / n + p.eps);
+    for (int c = threadIdx.x; c < W; c += 256) {
+      const float o = fmaf(summed(c) * inv, p.weight[c], p.residual[base + c]);
+      p.x_out[base + c] = o;
+      if (act == nullptr) continue;
+      float h = o;
+      if (p.taps != nullptr) {
+        for (int j = 0; j < p.n_taps; ++j) {
+          const bool own = j == p.n_taps - 1;
+          if (!own && hist == nullptr) continue;
+          const float u = own ? o : hist[static_cast<size_t>(j) * W + c];
+          if (j > 0 && hist != nullptr) hist[static_cast<size_t>(j - 1) * W + c] = u;
+          h = fmaf(p.taps[static_cast<size_t>(j) * W + c], u, h);
+        }
+      }
+      act[c] = from_f32<T>(h);
+    }
+  }
+}
+
+template <typename T>
+static cudaError_t launch_rms_routed_residual(const RoutedResidualParams& p, int M, bool quads_ok, cudaStream_t stream) {
+  const int quads = quads_ok ? (p.W / 4 + 255) / 256 : 0;
+#define ER_RR(NV_) launch_pdl(rms_routed_residual_kernel<T, NV_>, dim3(M), dim3(256), 0, stream, p)
+  switch (quads) {
+    case 1: return ER_RR(1);
+    case 2: return ER_RR(2);
+    case 3:
+    case 4: return ER_RR(4);
+    case 5:
+    case 6:
+    case 7:
+    case 8: return ER_RR(8);
+    default: return ER_RR(0);
+  }
+#undef ER_RR
+}
+
+struct StreamConvParams {
+  const float* x;       // [M, W]
+  void* act;            // [M, W]
+  const float* taps;    // [taps, W]
+  float* state;         // as RoutedResidualParams
+  RaggedBatch seqs;
+  int W, n_taps, state_elems, tile;   // tile: rows of a CTA, at least taps - 1
+};
+
+template <int VEC>
+__device__ __forceinline__ void load_vec(float (&v)[VEC], const float* p) {
+  if constexpr (VEC == 4) {
+    const float4 f = load4(p);
+    v[0] = f.x;
+    v[1] = f.y;
+    v[2] = f.z;
+    v[3] = f.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int VEC, typename T>
+__device__ __forceinline__ void store_vec(T* p, const float (&v)[VEC]) {
+  if constexpr (VEC == 4) store4(p, make_float4(v[0], v[1], v[2], v[3]));
+  else *p = from_f32<T>(v[0]);
+}
+
+// A thread owns VEC channels of one tile of a sequence's rows. L > 0: that many taps, the last inputs in registers; L = 0: any number,
+// inputs are read again. The thread that has the sequence's first rows also moves the history on, after it has read it.
+template <typename T, int VEC, int L>
+__global__ void __launch_bounds__(256) stream_conv_kernel(StreamConvParams p) {
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int W = p.W, c = (blockIdx.x * 256 + threadIdx.x) * VEC;
+  const RaggedSeq s = ragged_seq(p.seqs, blockIdx.z);
+  const int t0 = blockIdx.y * p.tile, t1 = min(t0 + p.tile, s.rows), n_taps = L > 0 ? L : p.n_taps;
+  if (t0 >= s.rows || c >= W) return;
+  const float* x = p.x + static_cast<size_t>(s.row0) * W + c;
+  T* act = static_cast<T*>(p.act) + static_cast<size_t>(s.row0) * W + c;
+  float* hist = p.state != nullptr && s.live ? p.state + static_cast<size_t>(s.slot) * p.state_elems + c : nullptr;
+  // input of position t of this portion, t >= -(taps - 1)
+  auto input = [&](float (&v)[VEC], int t) {
+    if (t >= 0) load_vec<VEC>(v, x + static_cast<size_t>(t) * W);
+    else if (hist != nullptr) load_vec<VEC>(v, hist + static_cast<size_t>(t + n_taps - 1) * W);
+    else
+      for (int e = 0; e < VEC; ++e) v[e] = 0.f;
+  };
+  if constexpr (L > 0) {
+    float w[L][VEC], in[L][VEC];
+#pragma unroll
+    for (int j = 0; j < L; ++j) load_vec<VEC>(w[j], p.taps + static_cast<size_t>(j) * W + c);
+#pragma unroll
+    for (int j = 0; j + 1 < L; ++j) input(in[j + 1], t0 - (L - 1) + j);
+#pragma unroll 4
+    for (int t = t0; t < t1; ++t) {
+#pragma unroll
+      for (int j = 0; j + 1 < L; ++j)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) in[j][e] = in[j + 1][e];
+      load_vec<VEC>(in[L - 1], x + static_cast<size_t>(t) * W);
+      float h[VEC];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        h[e] = in[L - 1][e];
+#pragma unroll
+        for (int j = 0; j < L; ++j) h[e] = fmaf(w[j][e], in[j][e], h[e]);
+      }
+      store_vec<VEC>(act + static_cast<size_t>(t) * W, h);
+    }
+  } else {
+    for (int t = t0; t < t1; ++t) {
+      float h[VEC], u[VEC], w[VEC];
+      load_vec<VEC>(h, x + static_cast<size_t>(t) * W);
+      for (int j = 0; j < n_taps; ++j) {
+        input(u, t - (n_taps - 1) + j);
+        load_vec<VEC>(w, p.taps + static_cast<size_t>(j) * W + c);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) h[e] = fmaf(w[e], u[e], h[e]);
+      }
+      store_vec<VEC>(act + static_cast<size_t>(t) * W, h);
+    }
+  }
+  if (t0 > 0 || hist == nullptr) return;
+  for (int j = 0; j + 1 < n_taps; ++j) {      // what row j takes lies behind it: upwards, in place
+    float v[VEC];
+    input(v, s.rows - (n_taps - 1) + j);
+    store_vec<VEC>(hist + static_cast<size_t>(j) * W, v);
+  }
+}
+
+template <typename T, int VEC>
+static cudaError_t launch_stream_conv(const StreamConvParams& p, dim3 grid, cudaStream_t stream) {
+  switch (p.n_taps) {
+    case 2: return launch_pdl(stream_conv_kernel<T, VEC, 2>, grid, dim3(256), 0, stream, p);
+    case 3: return launch_pdl(stream_conv_kernel<T, VEC, 3>, grid, dim3(256), 0, stream, p);
+    case 4: return launch_pdl(stream_conv_kernel<T, VEC, 4>, grid, dim3(256), 0, stream, p);
+    default: return launch_pdl(stream_conv_kernel<T, VEC, 0>, grid, dim3(256), 0, stream, p);
+  }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table,
-                                                                float* __restrict__ x, T* __restrict__ act, int W, int rows, float scale) {
+                                                                float* __restrict__ x, T* __restrict__ act, const int* __restrict__ positions,
+                                                                const float* __restrict__ inv_freq, int W, int rows, float scale) {
   pdl_launch_early();
   pdl_wait();
   pdl_launch_dependents();
@@ -392,11 +643,22 @@ __global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __rest
   const bool ok = id >= 0 && id < rows;
   const T* src = table + static_cast<size_t>(ok ? id : 0) * W;
   const size_t base = static_cast<size_t>(blockIdx.x) * W;
-  for (int c = threadIdx.x; c < W; c += 256) {
-    const float v = ok ? to_f32(src[c]) * scale : 0.f;
+  auto put = [&](int c, float add) {
+    const float v = (ok ? to_f32(src[c]) * scale : 0.f) + add;
     x[base + c] = v;
     if (act != nullptr) act[base + c] = from_f32<T>(v);
+  };
+  if (inv_freq != nullptr) {
+    const float pos = static_cast<float>(positions[blockIdx.x]);
+    for (int i = threadIdx.x; 2 * i < W; i += 256) {
+      float sn, cs;
+      sincosf(pos * inv_freq[i], &sn, &cs);
+      put(2 * i, sn);
+      if (2 * i + 1 < W) put(2 * i + 1, cs);
+    }
+    return;
   }
+  for (int c = threadIdx.x; c < W; c += 256) put(c, 0.f);
 }
 
 struct QkvPrepParams {
@@ -530,15 +792,54 @@ extern "C" int eredu_branch_norm(const float* x, const void* y0, const void* y1,
   return static_cast<int>(e);
 }
 
+// weight, residual, x_out, taps, state fp32; y (or null), rows, act (or null) bf16 (fp32 = 0) or fp32; k <= 32 routes per row. taps: row m is
+// the only row of sequence m; state may be null for one tap.
+extern "C" int eredu_rms_routed_residual(const void* y, const void* rows, const int* route_pos, const float* route_w, const float* weight,
+                                         const float* residual, float* x_out, void* act, const float* taps, float* state,
+                                         const int* block_table, const int* page_to_slot, const long long* slots, int M, int W, int k,
+                                         int n_taps, int state_elems, int max_pages, int fp32, int quads, float eps, cudaStream_t stream) {
+  if (M <= 0 || W <= 0) return 0;
+  if (k < 0 || k > kMaxRoutes || (k > 0 && (rows == nullptr || route_pos == nullptr || route_w == nullptr)) || (y == nullptr && k == 0) ||
+      (taps != nullptr && (n_taps < 1 || act == nullptr || (n_taps > 1 && state == nullptr))) ||
+      (state != nullptr && state_elems < (n_taps - 1) * W))
+    return -1;
+  const RaggedBatch seqs = {block_table, page_to_slot, nullptr, slots, M, 1, max_pages};
+  const RoutedResidualParams p = {y, rows, route_pos, route_w, weight, residual, x_out, act, taps, state, seqs, n_taps, state_elems, W, k, eps};
+  const bool q4 = quads != 0 && state_elems % 4 == 0;
+  const cudaError_t e = fp32 ? launch_rms_routed_residual<float>(p, M, q4, stream) : launch_rms_routed_residual<__nv_bfloat16>(p, M, q4, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// x fp32 [M, W]; act bf16 (fp32 = 0) or fp32; state may be null for one tap. max_rows: the most rows of a sequence.
+extern "C" int eredu_stream_conv(const float* x, void* act, const float* taps, float* state, const int* block_table, const int* page_to_slot,
+                                 const int* cu_q, const long long* slots, int batch, int q_per_seq, int max_rows, int max_pages, int W,
+                                 int n_taps, int state_elems, int fp32, cudaStream_t stream) {
+  if (batch <= 0 || max_rows <= 0 || W <= 0) return 0;
+  if (n_taps < 1 || (n_taps > 1 && (state == nullptr || state_elems < (n_taps - 1) * W)) || batch > 65535) return -1;
+  int tile = 16;
+  while (tile < n_taps - 1 || (max_rows + tile - 1) / tile > 65535) tile *= 2;
+  const RaggedBatch seqs = {block_table, page_to_slot, cu_q, slots, batch, q_per_seq, max_pages};
+  const StreamConvParams p = {x, act, taps, state, seqs, W, n_taps, state_elems, tile};
+  const int vec = W % 4 == 0 && state_elems % 4 == 0 ? 4 : 1;
+  const dim3 grid((W + 256 * vec - 1) / (256 * vec), (max_rows + tile - 1) / tile, batch);
+  cudaError_t e;
+  if (vec == 4) e = fp32 ? launch_stream_conv<float, 4>(p, grid, stream) : launch_stream_conv<__nv_bfloat16, 4>(p, grid, stream);
+  else e = fp32 ? launch_stream_conv<float, 1>(p, grid, stream) : launch_stream_conv<__nv_bfloat16, 1>(p, grid, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
 // table [rows, W] bf16 or fp32, times scale; x fp32 [M, W]; act [M, W] in the table's dtype or null.
-extern "C" int eredu_embedding_stream(const int* ids, const void* table, float* x, void* act, int M, int W, int rows, int fp32,
-                                      float scale, cudaStream_t stream) {
+// inv_freq [(W + 1) / 2] or null: columns 2 i and 2 i + 1 get sin and cos of positions[m] * inv_freq[i] added.
+extern "C" int eredu_embedding_stream(const int* ids, const void* table, float* x, void* act, const int* positions, const float* inv_freq,
+                                      int M, int W, int rows, int fp32, float scale, cudaStream_t stream) {
   if (M <= 0 || W <= 0) return 0;
   cudaError_t e;
   if (fp32) e = launch_pdl(embedding_stream_kernel<float>, dim3(M), dim3(256), 0, stream, ids, static_cast<const float*>(table), x,
-                           static_cast<float*>(act), W, rows, scale);
+                           static_cast<float*>(act), positions, inv_freq, W, rows, scale);
   else e = launch_pdl(embedding_stream_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, stream, ids,
-                      static_cast<const __nv_bfloat16*>(table), x, static_cast<__nv_bfloat16*>(act), W, rows, scale);
+                      static_cast<const __nv_bfloat16*>(table), x, static_cast<__nv_bfloat16*>(act), positions, inv_freq, W, rows, scale);
   eredu_count_launches(1);
   return static_cast<int>(e);
 }

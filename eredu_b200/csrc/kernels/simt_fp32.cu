@@ -16,7 +16,7 @@ constexpr int kTile = 64, kTileK = 16;
 template <typename T, typename TO, bool GATED>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, TO* __restrict__ y,
                                                          const T* __restrict__ bias, int M, int N, int K, int ldx, int ldw, int ldy,
-                                                         int act) {
+                                                         int act, float act_a, float act_b) {
   constexpr int PARTS = GATED ? 2 : 1;
   __shared__ float xs[kTileK][kTile + 4], ws[PARTS][kTileK][kTile + 4];
   pdl_launch_early();
@@ -65,6 +65,8 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ x,
       } else if (act == 1) {
         v = fmaxf(v, 0.f);
         v *= v;
+      } else if (act == 4) {
+        v = xielu<false>(v, act_a, act_b);
       }
       y[static_cast<size_t>(m) * ldy + n] = from_f32<TO>(v);
     }
@@ -247,21 +249,22 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(AttnSimtParams p) {
 
 using namespace eredu;
 
-// X [M, K], W [N, K], bias [N] (or null) fp32 (in_fp32 = 1) or bf16; Y [M, N] fp32 or bf16. act 1: squared ReLU; act 2, 3: W is [2 N, K],
-// Y = silu(gate) * up or relu(gate) * up (bias [2 N]).
+// X [M, K], W [N, K], bias [N] (or null) fp32 (in_fp32 = 1) or bf16; Y [M, N] fp32 or bf16. act 1: squared ReLU; act 4: xIELU
+// with factors act_a and act_b; act 2, 3: W is [2 N, K], Y = silu(gate) * up or relu(gate) * up (bias [2 N]).
 extern "C" int eredu_gemm_simt(const void* x, const void* w, void* y, const void* bias, int M, int N, int K, int ldx, int ldw, int ldy,
-                               int in_fp32, int out_fp32, int act, cudaStream_t stream) {
+                               int in_fp32, int out_fp32, int act, float act_a, float act_b, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
+  const bool gated = act == 2 || act == 3;
   const dim3 grid((N + kTile - 1) / kTile, (M + kTile - 1) / kTile);
   if (grid.y > 65535 || (in_fp32 && !out_fp32)) return -1;
   cudaError_t e;
   using B = __nv_bfloat16;
 #define ER_SIMT(T_, TO_, G_)                                                                                                     \
   launch_pdl(gemm_simt_kernel<T_, TO_, G_>, grid, dim3(256), 0, stream, static_cast<const T_*>(x), static_cast<const T_*>(w),      \
-             static_cast<TO_*>(y), static_cast<const T_*>(bias), M, N, K, ldx, ldw, ldy, act)
-  if (in_fp32) e = act >= 2 ? ER_SIMT(float, float, true) : ER_SIMT(float, float, false);
-  else if (out_fp32) e = act >= 2 ? ER_SIMT(B, float, true) : ER_SIMT(B, float, false);
-  else e = act >= 2 ? ER_SIMT(B, B, true) : ER_SIMT(B, B, false);
+             static_cast<TO_*>(y), static_cast<const T_*>(bias), M, N, K, ldx, ldw, ldy, act, act_a, act_b)
+  if (in_fp32) e = gated ? ER_SIMT(float, float, true) : ER_SIMT(float, float, false);
+  else if (out_fp32) e = gated ? ER_SIMT(B, float, true) : ER_SIMT(B, float, false);
+  else e = gated ? ER_SIMT(B, B, true) : ER_SIMT(B, B, false);
 #undef ER_SIMT
   eredu_count_launches(1);
   return static_cast<int>(e);

@@ -1,0 +1,726 @@
+// Paged attention whose heads exchange their scores before the softmax: the score of head h is sum_g talk[h, g] cap(scale q_g . k_g),
+// cap(s) = softcap tanh(s / softcap), over a sliding window and the first tokens of the sequence, with a sink per head.
+//
+// A query's heads cannot be computed apart, so a group of warps owns ALL heads of a few queries and walks the visible pages of 16 keys:
+//   score    S^T[key, column] = K Q^T per key / value head on the tensor cores, a column being one (query, head of the group); the cap in
+//            fp32; S goes to shared memory with the heads of a (query, key) pair side by side
+//   mix      S'[head, pair] = talk S on the tensor cores: S as three bf16 pieces (exact), talk is bf16 itself, fp32 accumulation
+//   combine  online softmax per column and O^T[value dim, column] += V^T P^T, O in registers
+// The score step of page i + 1 and the combine step of page i lie between the same two barriers; keys and values arrive by cp.async two
+// stages deep. Prompts: one group of up to 16 warps and as many queries as fit its registers. Decode steps: several groups per CTA, each
+// with pages of its own, and the CTAs of a cluster share a sequence's keys; partial results meet in (distributed) shared memory.
+//
+// A second kernel on the CUDA cores takes fp32, head sizes the first is not built for, and more than 64 heads.
+#include <algorithm>
+
+#include "../common/elem.cuh"
+#include "../common/launch.h"
+#include "../common/launch_count.h"
+#include "../common/mma.cuh"
+#include "../common/ptx.cuh"
+
+namespace eredu {
+
+constexpr int kPage = 16;
+constexpr float kLog2e = 1.4426950408889634f;
+constexpr int kMaxSplits = 8;          // portable cluster size
+constexpr int kMaxHeadBlocks = 4;      // blocks of 16 heads
+constexpr int kSmemLimit = 227 * 1024;
+
+struct TalkParams {
+  const void* q;           // [rows, H, dk]
+  const void* k_cache;     // [pages, G, 16, dk]
+  const void* v_cache;     // [pages, G, 16, dv]
+  void* out;               // [rows, H, dv]
+  const int* block_table;  // [B, max_pages]
+  const int* seq_lens;     // [B]
+  const int* cu_q;         // [B + 1] or null: q_per_seq rows each
+  const void* talk;        // [H, H]
+  const float* sinks;      // [H] or null
+  int q_per_seq, max_pages, H, G, dk, dv, window, keep;
+  float scale, softcap;
+  // tensor-core kernel
+  int qt;                  // queries of a CTA
+  int octets;              // column octets per key / value head
+  int warps;               // warps of a group
+  int lanes;               // groups of a CTA
+  int splits;              // CTAs of a cluster
+  int group_bytes;         // shared memory of a group
+};
+
+// Visible pages of a run of queries at positions p0 .. p1: those with the first `keep` tokens, then those of the window.
+struct TalkPages {
+  int head, first, count;
+  __device__ __forceinline__ int at(int i) const { return i < head ? i : first + i - head; }
+};
+__device__ __forceinline__ TalkPages talk_pages(int p0, int p1, int window, int keep) {
+  TalkPages t = {0, 0, 0};
+  if (p1 < 0) return t;
+  if (window > 0) {
+    t.head = (min(keep, p1 + 1) + kPage - 1) / kPage;
+    t.first = max(t.head, max(0, p0 - window + 1) / kPage);
+  }
+  t.count = t.head + max(0, p1 / kPage - t.first + 1);
+  return t;
+}
+
+// ---------------------------------------------------------------------------------------------- tensor cores
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// c tanh(x / (2 a)) for a pair: c - 2 c / (1 + 2^(x in)), `in` = log2(e) / a; one reciprocal serves both.
+__device__ __forceinline__ void cap_pair(float& x, float& y, float in, float c) {
+  const float a = 1.f + ex2(fminf(x * in, 60.f)), b = 1.f + ex2(fminf(y * in, 60.f));
+  const float r = rcp(a * b) * (2.f * c);
+  x = fmaf(-r, b, c);
+  y = fmaf(-r, a, c);
+}
+// x = hi + mid + lo, each exact in bf16 (truncation: 8 + 8 + 8 bits); the pieces of two values side by side.
+__device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t& mid, uint32_t& lo) {
+  const uint32_t ux = __float_as_uint(x), uy = __float_as_uint(y);
+  hi = __byte_perm(ux, uy, 0x7632);
+  const float rx = x - __uint_as_float(ux & 0xFFFF0000u), ry = y - __uint_as_float(uy & 0xFFFF0000u);
+  const uint32_t vx = __float_as_uint(rx), vy = __float_as_uint(ry);
+  mid = __byte_perm(vx, vy, 0x7632);
+  lo = __byte_perm(__float_as_uint(rx - __uint_as_float(vx & 0xFFFF0000u)), __float_as_uint(ry - __uint_as_float(vy & 0xFFFF0000u)), 0x7632);
+}
+__device__ __forceinline__ uint32_t pack2(float x, float y) {
+  const __nv_bfloat162 t = __floats2bfloat162_rn(x, y);
+  return *reinterpret_cast<const uint32_t*>(&t);
+}
+__device__ __forceinline__ void group_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+__device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
+  return v;
+}
+
+// Shared memory of a group, in bytes; the same arithmetic on the host and the device. Rows of keys and values are an odd number of
+// 16-byte pieces long and rows of heads 8 or 24 (mod 32) floats, so that fragments load without bank conflicts.
+struct TalkLayout {
+  int hp;                    // heads, in whole blocks of 16
+  int k_pitch, v_pitch;      // bytes of a cached row
+  int k_bytes, v_bytes;      // one stage
+  int s_pair, s_query;       // floats between two keys, two queries
+  int s_bytes, m_bytes;
+  __host__ __device__ __forceinline__ TalkLayout(int H, int G, int dk, int dv, int qt) {
+    hp = (H + 15) / 16 * 16;
+    k_pitch = ((dk + 15) / 16 * 2 + 1) * 16;
+    v_pitch = ((dv + 15) / 16 * 2 + 1) * 16;
+    k_bytes = G * kPage * k_pitch;
+    v_bytes = G * kPage * v_pitch;
+    s_pair = hp + 8;
+    s_query = kPage * s_pair + 4;
+    s_bytes = qt * s_query * 4;
+    m_bytes = qt * hp * kMixPitch * 4;
+  }
+  static constexpr int kMixPitch = 24;   // floats of a (query, head) row of 16 mixed scores
+  __host__ __device__ __forceinline__ int group() const { return 2 * (k_bytes + v_bytes) + s_bytes + m_bytes; }
+  __host__ __device__ __forceinline__ int talk() const { return hp * (hp + 8) * 2; }
+};
+
+// KS, VT: 16-wide steps of the key and value sizes a warp can hold. U: column octets of a warp. The block has lanes * warps warps.
+template <int KS, int VT, int U>
+__global__ void __launch_bounds__(512, 1) talking_attention_kernel(TalkParams p) {
+  using bf16 = __nv_bfloat16;
+  extern __shared__ __align__(16) uint8_t smem[];
+  pdl_launch_early();
+  const TalkLayout lay(p.H, p.G, p.dk, p.dv, p.qt);
+  const int tid = threadIdx.x, lane = tid & 31, quad = lane & 3, oct = lane >> 2;
+  const int gi = (tid >> 5) / p.warps, gw = (tid >> 5) % p.warps;       // group, warp of it
+  const int gthreads = p.warps * 32, gtid = tid - gi * gthreads;
+  const int split = blockIdx.x % p.splits, b = blockIdx.y;
+  const int r = p.H / p.G, columns = p.qt * r;
+  uint8_t* talk_s = smem;
+  uint8_t* mine = smem + lay.talk() + gi * p.group_bytes;
+  uint8_t *ks = mine, *vs = ks + 2 * lay.k_bytes;
+  float* sc = reinterpret_cast<float*>(vs + 2 * lay.v_bytes);
+  float* mx = sc + lay.s_bytes / 4;
+
+  // talk, and zeros wherever a fragment reads beyond the sizes
+  for (int i = tid; i < (lay.talk() + p.lanes * p.group_bytes) / 16; i += blockDim.x) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
+  __syncthreads();
+  for (int i = tid; i < p.H * p.H; i += blockDim.x)
+    reinterpret_cast<bf16*>(talk_s)[i / p.H * (lay.hp + 8) + i % p.H] = static_cast<const bf16*>(p.talk)[i];
+
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row0 = p.cu_q != nullptr ? p.cu_q[b] : b * p.q_per_seq;
+  const int q_len = p.cu_q != nullptr ? p.cu_q[b + 1] - row0 : p.q_per_seq;
+  const int qi0 = (blockIdx.x / p.splits) * p.qt;
+  if (qi0 >= q_len) return;                                             // the whole cluster
+  const int nq = min(p.qt, q_len - qi0);
+  const int p0 = p.seq_lens[b] - q_len + qi0, p1 = p0 + nq - 1;
+  const TalkPages pages = talk_pages(p0, p1, p.window, p.keep);
+  const int* bt = p.block_table + static_cast<size_t>(b) * p.max_pages;
+  // page number i of this group: the splits take contiguous shares, their groups every lanes-th page of it
+  const int share = (pages.count + p.splits - 1) / p.splits;
+  const int i0 = split * share + gi, i1 = min(pages.count, (split + 1) * share);
+  const int n = i1 > i0 ? (i1 - i0 + p.lanes - 1) / p.lanes : 0;
+
+  // ---- the warp's columns
+  const bf16* q = static_cast<const bf16*>(p.q) + static_cast<size_t>(row0 + qi0) * p.H * p.dk;
+  const int nks = (p.dk + 15) >> 4, nvt = (p.dv + 15) >> 4;
+  uint32_t qf[U][KS][2];
+  int kvh[U], s_off[U][2], m_off[U], col_q[U], col_h[U];
+  bool on[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    const int unit = gw * U + u;
+    on[u] = unit < p.G * p.octets;
+    kvh[u] = on[u] ? unit / p.octets : 0;
+    const int c0 = on[u] ? (unit % p.octets) * 8 : columns;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {                                       // the two columns of a score fragment
+      const int c = c0 + quad * 2 + e;
+      s_off[u][e] = c < columns ? c / r * lay.s_query + kvh[u] * r + c % r + oct * lay.s_pair : -1;
+    }
+    const int c = c0 + oct;                                             // the column of a probability fragment
+    col_q[u] = c < columns ? c / r : -1;
+    col_h[u] = c < columns ? kvh[u] * r + c % r : 0;
+    m_off[u] = (max(col_q[u], 0) * lay.hp + col_h[u]) * TalkLayout::kMixPitch + quad * 2;
+    const bool real = col_q[u] >= 0 && col_q[u] < nq;
+    const bf16* src = q + (static_cast<size_t>(max(col_q[u], 0)) * p.H + col_h[u]) * p.dk;
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int d = k * 16 + e * 8 + quad * 2;
+        qf[u][k][e] = real && d < p.dk ? *reinterpret_cast<const uint32_t*>(src + d) : 0u;
+      }
+  }
+  const float cap_c = p.softcap * kLog2e, cap_in = p.softcap > 0.f ? 2.f * kLog2e * p.scale / p.softcap : 0.f, plain = p.scale * kLog2e;
+
+  float o[U][VT][4], m[U], l[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    m[u] = -1e30f;
+    l[u] = 0.f;
+#pragma unroll
+    for (int v = 0; v < VT; ++v)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[u][v][e] = 0.f;
+  }
+
+  // ---- asynchronous copies: a page's rows of all key / value heads lie in one piece
+  const int kc = p.dk >> 3, vc = p.dv >> 3;                             // 16-byte pieces of a row
+  const int kl2 = 32 - __clz(kc - 1), vl2 = 32 - __clz(vc - 1);         // threads per row: the next power of two
+  auto load = [&](const void* cache, uint8_t* dst, int pitch, int pieces, int l2, int i) {
+    const size_t page = bt[pages.at(i0 + i * p.lanes)];
+    const uint4* src = static_cast<const uint4*>(cache) + page * (p.G * kPage) * pieces;
+    const int c = gtid & ((1 << l2) - 1);
+    if (c >= pieces) return;
+    for (int row = gtid >> l2; row < p.G * kPage; row += gthreads >> l2)
+      cp_async16(dst + row * pitch + c * 16, src + static_cast<size_t>(row) * pieces + c, 16);
+  };
+  auto load_k = [&](int i) {
+    if (i < n) load(p.k_cache, ks + (i & 1) * lay.k_bytes, lay.k_pitch, kc, kl2, i);
+  };
+  auto load_v = [&](int i) {
+    if (i < n) load(p.v_cache, vs + (i & 1) * lay.v_bytes, lay.v_pitch, vc, vl2, i);
+  };
+
+  auto score = [&](int i) {
+    const uint32_t base = smem_u32(ks + (i & 1) * lay.k_bytes) + (lane & 15) * lay.k_pitch + (lane >> 4) * 16;
+    float s[U][4];
+#pragma unroll
+    for (int u = 0; u < U; ++u) s[u][0] = s[u][1] = s[u][2] = s[u][3] = 0.f;
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+      if (k >= nks) break;
+      uint32_t a0, a1, a2, a3;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (!on[u]) break;
+        if (u == 0 || kvh[u] != kvh[u - 1]) ldsm_x4(base + kvh[u] * (kPage * lay.k_pitch) + k * 32, a0, a1, a2, a3);
+        mma16816(s[u], a0, a1, a2, a3, qf[u][k][0], qf[u][k][1]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (!on[u]) break;
+      if (p.softcap > 0.f) {
+        cap_pair(s[u][0], s[u][1], cap_in, cap_c);
+        cap_pair(s[u][2], s[u][3], cap_in, cap_c);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[u][e] *= plain;
+      }
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (s_off[u][e] >= 0) {
+          sc[s_off[u][e]] = s[u][e];
+          sc[s_off[u][e] + 8 * lay.s_pair] = s[u][2 + e];
+        }
+    }
+  };
+
+  const int blocks = lay.hp >> 4;
+  const uint32_t talk_a = smem_u32(talk_s) + (lane & 15) * (lay.hp + 8) * 2 + (lane >> 4) * 16;
+  auto mix = [&]() {
+    for (int t = gw; t < 2 * p.qt; t += p.warps) {                      // eight keys of a query
+      const int qq = t >> 1, k0 = (t & 1) * 8;
+      const float* src = sc + qq * lay.s_query + (k0 + oct) * lay.s_pair + quad * 2;
+      float acc[kMaxHeadBlocks][4];
+#pragma unroll
+      for (int h = 0; h < kMaxHeadBlocks; ++h) acc[h][0] = acc[h][1] = acc[h][2] = acc[h][3] = 0.f;
+#pragma unroll
+      for (int g = 0; g < kMaxHeadBlocks; ++g) {
+        if (g >= blocks) break;
+        const float2 x = *reinterpret_cast<const float2*>(src + g * 16), y = *reinterpret_cast<const float2*>(src + g * 16 + 8);
+        uint32_t h0, h1, m0, m1, l0, l1;
+        split3(x.x, x.y, h0, m0, l0);
+        split3(y.x, y.y, h1, m1, l1);
+#pragma unroll
+        for (int h = 0; h < kMaxHeadBlocks; ++h) {
+          if (h >= blocks) break;
+          uint32_t a0, a1, a2, a3;
+          ldsm_x4(talk_a + h * 16 * (lay.hp + 8) * 2 + g * 32, a0, a1, a2, a3);
+          mma16816(acc[h], a0, a1, a2, a3, l0, l1);
+          mma16816(acc[h], a0, a1, a2, a3, m0, m1);
+          mma16816(acc[h], a0, a1, a2, a3, h0, h1);
+        }
+      }
+#pragma unroll
+      for (int h = 0; h < kMaxHeadBlocks; ++h) {
+        if (h >= blocks) break;
+        float* dst = mx + (qq * lay.hp + h * 16 + oct) * TalkLayout::kMixPitch + k0 + quad * 2;
+        *reinterpret_cast<float2*>(dst) = make_float2(acc[h][0], acc[h][1]);
+        *reinterpret_cast<float2*>(dst + 8 * TalkLayout::kMixPitch) = make_float2(acc[h][2], acc[h][3]);
+      }
+    }
+  };
+
+  auto combine = [&](int i) {
+    const int key0 = pages.at(i0 + i * p.lanes) * kPage;
+    // every query sees every key of the page
+    const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+    uint32_t pf[U][2];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (!on[u]) break;
+      const float2 x = *reinterpret_cast<const float2*>(mx + m_off[u]), y = *reinterpret_cast<const float2*>(mx + m_off[u] + 8);
+      float s[4] = {x.x, x.y, y.x, y.y};
+      if (!inner) {
+        const int pos = p0 + max(col_q[u], 0);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int key = key0 + quad * 2 + (e & 1) + (e >> 1) * 8;
+          if (key > pos || (p.window > 0 && pos - key >= p.window && key >= p.keep)) s[e] = -INFINITY;
+        }
+      }
+      float top = fmaxf(fmaxf(s[0], s[1]), fmaxf(s[2], s[3]));
+      top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1));
+      top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
+      // the reference point moves only when a score exceeds it by more than 2^8
+      if (__any_sync(0xffffffffu, top > m[u] + 8.f)) {
+        const float next = fmaxf(m[u], top), corr = ex2(m[u] - next);
+        m[u] = next;
+        l[u] *= corr;
+        const float c0 = __shfl_sync(0xffffffffu, corr, quad * 8), c1 = __shfl_sync(0xffffffffu, corr, quad * 8 + 4);
+#pragma unroll
+        for (int v = 0; v < VT; ++v) {
+          o[u][v][0] *= c0;
+          o[u][v][1] *= c1;
+          o[u][v][2] *= c0;
+          o[u][v][3] *= c1;
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[e] = ex2(s[e] - m[u]);
+      l[u] += (s[0] + s[1]) + (s[2] + s[3]);
+      pf[u][0] = pack2(s[0], s[1]);
+      pf[u][1] = pack2(s[2], s[3]);
+    }
+    // matrix j of a quadruple: keys 8 (j >> 1) .., value dims 8 (j & 1) ..
+    const uint32_t base = smem_u32(vs + (i & 1) * lay.v_bytes) + ((lane & 7) + (lane >> 4) * 8) * lay.v_pitch + ((lane >> 3) & 1) * 16;
+#pragma unroll
+    for (int v = 0; v < VT; ++v) {
+      if (v >= nvt) break;
+      uint32_t a0, a1, a2, a3;
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        if (!on[u]) break;
+        if (u == 0 || kvh[u] != kvh[u - 1]) ldsm_x4_t(base + kvh[u] * (kPage * lay.v_pitch) + v * 32, a0, a1, a2, a3);
+        mma16816(o[u][v], a0, a1, a2, a3, pf[u][0], pf[u][1]);
+      }
+    }
+  };
+
+  // ---- pages. Between the barriers of page i: its scores beside the sums of page i - 1, then its mixing. Keys are fetched two pages
+  // ahead, values one: their buffers are free once every warp has passed the barrier behind their last use.
+  const int bar = 1 + gi;
+  load_k(0);
+  load_v(0);
+  cp_async_commit();
+  load_k(1);
+  cp_async_commit();
+  cp_async_wait<1>();
+  __syncthreads();                                                      // talk and the zeros, too
+  if (n > 0) {
+    for (int i = 0; i < n; ++i) {
+      score(i);
+      if (i > 0) combine(i - 1);
+      group_sync(bar, gthreads);
+      load_k(i + 2);
+      load_v(i + 1);
+      cp_async_commit();
+      mix();
+      cp_async_wait<1>();                                               // keys i + 1 (and values i) are there
+      group_sync(bar, gthreads);
+    }
+    cp_async_wait<0>();
+    combine(n - 1);
+  }
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    l[u] += __shfl_xor_sync(0xffffffffu, l[u], 1);
+    l[u] += __shfl_xor_sync(0xffffffffu, l[u], 2);
+  }
+
+  bf16* out = static_cast<bf16*>(p.out) + static_cast<size_t>(row0 + qi0) * p.H * p.dv;
+  if (p.lanes * p.splits == 1) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (!on[u]) break;
+      const float sink = p.sinks != nullptr ? p.sinks[col_h[u]] * kLog2e : -INFINITY;
+      const float top = fmaxf(m[u], sink), e = ex2(m[u] - top), sum = l[u] * e + ex2(sink - top);
+      const float f = sum > 0.f ? e / sum : 0.f;
+      const float f0 = __shfl_sync(0xffffffffu, f, quad * 8), f1 = __shfl_sync(0xffffffffu, f, quad * 8 + 4);
+      const int at = col_q[u] >= 0 && col_q[u] < nq ? (col_q[u] * p.H + col_h[u]) * p.dv : -1;
+      const int at0 = __shfl_sync(0xffffffffu, at, quad * 8), at1 = __shfl_sync(0xffffffffu, at, quad * 8 + 4);
+#pragma unroll
+      for (int v = 0; v < VT; ++v) {
+        if (v >= nvt) break;
+#pragma unroll
+        for (int e2 = 0; e2 < 2; ++e2) {
+          const int d = v * 16 + e2 * 8 + oct;
+          if (d >= p.dv) continue;
+          if (at0 >= 0) out[at0 + d] = __float2bfloat16(o[u][v][e2 * 2] * f0);
+          if (at1 >= 0) out[at1 + d] = __float2bfloat16(o[u][v][e2 * 2 + 1] * f1);
+        }
+      }
+    }
+    return;
+  }
+
+  // ---- partial results of the groups and of the cluster's CTAs: O [lanes][qt H][dv], then (m, l) [lanes][qt H][2], then the weights of
+  // all partials [splits lanes][qt H], over the buffers of the pages
+  const int rows = p.qt * p.H;
+  float* part = reinterpret_cast<float*>(smem + lay.talk());
+  float* ml = part + p.lanes * rows * p.dv;
+  float* weight = ml + p.lanes * rows * 2;
+  __syncthreads();
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+    if (!on[u]) break;
+    const int row = col_q[u] >= 0 ? col_q[u] * p.H + col_h[u] : -1;
+    if (quad == 0 && row >= 0) {
+      ml[(gi * rows + row) * 2] = m[u];
+      ml[(gi * rows + row) * 2 + 1] = l[u];
+    }
+    const int at0 = __shfl_sync(0xffffffffu, row, quad * 8), at1 = __shfl_sync(0xffffffffu, row, quad * 8 + 4);
+#pragma unroll
+    for (int v = 0; v < VT; ++v) {
+      if (v >= nvt) break;
+#pragma unroll
+      for (int e2 = 0; e2 < 2; ++e2) {
+        const int d = v * 16 + e2 * 8 + oct;
+        if (d >= p.dv) continue;
+        if (at0 >= 0) part[(gi * rows + at0) * p.dv + d] = o[u][v][e2 * 2];
+        if (at1 >= 0) part[(gi * rows + at1) * p.dv + d] = o[u][v][e2 * 2 + 1];
+      }
+    }
+  }
+  if (p.splits > 1) {
+    cluster_arrive_release();
+    cluster_wait_acquire();
+  } else {
+    __syncthreads();
+  }
+  const uint32_t ml_a = smem_u32(ml), part_a = smem_u32(part);
+  for (int row = tid; row < nq * p.H; row += blockDim.x) {
+    const float sink = p.sinks != nullptr ? p.sinks[row % p.H] * kLog2e : -INFINITY;
+    float top = sink;
+    for (int s = 0; s < p.splits; ++s)
+      for (int g = 0; g < p.lanes; ++g) top = fmaxf(top, ld_cluster_f32(mapa_shared(ml_a + (g * rows + row) * 8, s)));
+    float sum = ex2(sink - top);
+    for (int s = 0; s < p.splits; ++s)
+      for (int g = 0; g < p.lanes; ++g) {
+        const uint32_t a = mapa_shared(ml_a + (g * rows + row) * 8, s);
+        const float w = ex2(ld_cluster_f32(a) - top);
+        sum += w * ld_cluster_f32(a + 4);
+        weight[(s * p.lanes + g) * rows + row] = w;
+      }
+    const float inv = sum > 0.f ? 1.f / sum : 0.f;
+    for (int s = 0; s < p.splits * p.lanes; ++s) weight[s * rows + row] *= inv;
+  }
+  __syncthreads();
+  for (int i = split * blockDim.x + tid; i < nq * p.H * p.dv; i += p.splits * blockDim.x) {
+    const int row = i / p.dv;
+    float v = 0.f;
+    for (int s = 0; s < p.splits; ++s)
+      for (int g = 0; g < p.lanes; ++g)
+        v = fmaf(weight[(s * p.lanes + g) * rows + row], ld_cluster_f32(mapa_shared(part_a + (g * rows * p.dv + i) * 4, s)), v);
+    out[i] = __float2bfloat16(v);
+  }
+  if (p.splits > 1) {                                                   // nobody reads this CTA's shared memory any more
+    cluster_arrive_release();
+    cluster_wait_acquire();
+  }
+}
+
+// How a step of at most `rows` queries per sequence is cut; qt = 0: this kernel does not take the sizes.
+struct TalkPlan {
+  int qt = 0, octets = 0, units = 0, per_warp = 0, warps = 0, lanes = 1, group_bytes = 0, smem = 0;
+};
+static TalkPlan talk_plan(int H, int G, int dk, int dv, int rows, bool decode) {
+  TalkPlan best;
+  if (G <= 0 || H % G != 0 || H > 16 * kMaxHeadBlocks || dk <= 0 || dv <= 0 || dk > 128 || dv > 128 || dk % 8 != 0 || dv % 8 != 0) return best;
+  const int r = H / G, most = dk <= 64 && dv <= 64 ? 4 : 2;
+  for (int qt = decode ? rows : 32; qt >= 1; qt = decode ? qt - 1 : qt / 2) {
+    if (!decode && qt > 1 && qt / 2 >= rows) continue;
+    TalkPlan t;
+    t.qt = qt;
+    t.octets = (qt * r + 7) / 8;
+    t.units = G * t.octets;
+    t.per_warp = t.units <= 16 ? 1 : t.units <= 32 ? 2 : t.units <= 64 ? 4 : 99;
+    if (t.per_warp > most) continue;
+    t.warps = (t.units + t.per_warp - 1) / t.per_warp;
+    const TalkLayout lay(H, G, dk, dv, qt);
+    t.group_bytes = lay.group();
+    if (decode)
+      while (t.lanes < 8 && (t.lanes + 1) * t.warps <= 16 && lay.talk() + (t.lanes + 1) * t.group_bytes <= kSmemLimit) ++t.lanes;
+    // the partial results of the last phase lie over the buffers
+    const int part = decode ? t.lanes * qt * H * (dv + 2 + kMaxSplits) * 4 : 0;
+    t.smem = lay.talk() + std::max(t.lanes * t.group_bytes, (part + 15) / 16 * 16);
+    if (t.smem > kSmemLimit) continue;
+    return t;
+  }
+  return best;
+}
+
+template <int KS, int VT, int U>
+static cudaError_t launch_talking(const TalkParams& p, dim3 grid, int threads, int smem, cudaStream_t stream) {
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(talking_attention_kernel<KS, VT, U>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit);
+    if (e != cudaSuccess) return e;
+    configured = true;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = dim3(threads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  int n = 0;
+  if (pdl_enabled()) {
+    attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[n++].val.programmaticStreamSerializationAllowed = 1;
+  }
+  if (p.splits > 1) {
+    attr[n].id = cudaLaunchAttributeClusterDimension;
+    attr[n].val.clusterDim.x = p.splits;
+    attr[n].val.clusterDim.y = 1;
+    attr[n++].val.clusterDim.z = 1;
+  }
+  cfg.attrs = attr;
+  cfg.numAttrs = n;
+  return cudaLaunchKernelEx(&cfg, talking_attention_kernel<KS, VT, U>, p);
+}
+
+// ---------------------------------------------------------------------------------------------- CUDA cores
+constexpr int kKeys = 32;
+
+// One CTA per query: groups of 32 visible keys, first the scores of all heads, then their mixture, then a running softmax per head.
+template <typename T>
+__global__ void __launch_bounds__(256) talking_simt_kernel(TalkParams p) {
+  extern __shared__ __align__(16) float fs[];
+  float* q = fs;                            // [H dk]
+  float* o = q + p.H * p.dk;                // [H dv]
+  float* sc = o + p.H * p.dv;               // [32][H + 1]
+  float* mx = sc + kKeys * (p.H + 1);       // [H][33]
+  float* m = mx + p.H * (kKeys + 1);        // [H], then l and the factor of a step
+  float *l = m + p.H, *corr = l + p.H;
+  __shared__ int rows[kKeys];               // page * 16 + offset
+  pdl_launch_early();
+  pdl_wait();
+  pdl_launch_dependents();
+  const int b = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+  const int row0 = p.cu_q != nullptr ? p.cu_q[b] : b * p.q_per_seq;
+  const int q_len = p.cu_q != nullptr ? p.cu_q[b + 1] - row0 : p.q_per_seq;
+  if (static_cast<int>(blockIdx.x) >= q_len) return;
+  const int pos = p.seq_lens[b] - q_len + blockIdx.x, r = p.H / p.G;
+  const int* bt = p.block_table + static_cast<size_t>(b) * p.max_pages;
+  const T* qg = static_cast<const T*>(p.q) + static_cast<size_t>(row0 + blockIdx.x) * p.H * p.dk;
+  const T* talk = static_cast<const T*>(p.talk);
+  for (int i = tid; i < p.H * p.dk; i += 256) q[i] = to_f32(qg[i]);
+  for (int i = tid; i < p.H * p.dv; i += 256) o[i] = 0.f;
+  for (int i = tid; i < p.H; i += 256) {
+    m[i] = p.sinks != nullptr ? p.sinks[i] : -INFINITY;
+    l[i] = p.sinks != nullptr ? 1.f : 0.f;
+  }
+  // visible keys in order: `head` first ones, then from `first` on
+  const int head = p.window > 0 ? min(p.keep, pos + 1) : 0, first = p.window > 0 ? max(head, pos - p.window + 1) : 0;
+  const int total = head + max(0, pos - first + 1);
+  for (int k0 = 0; k0 < total; k0 += kKeys) {
+    const int n = min(kKeys, total - k0);
+    __syncthreads();
+    if (tid < n) {
+      const int i = k0 + tid, key = i < head ? i : first + i - head;
+      rows[tid] = bt[key >> 4] * 16 + (key & 15);
+    }
+    __syncthreads();
+    for (int i = tid; i < p.H * kKeys; i += 256) {
+      const int h = i / kKeys, j = i % kKeys;
+      if (j >= n) continue;
+      const T* k = static_cast<const T*>(p.k_cache) + ((static_cast<size_t>(rows[j] >> 4) * p.G + h / r) * 16 + (rows[j] & 15)) * p.dk;
+      float s = 0.f;
+      for (int d = 0; d < p.dk; ++d) s = fmaf(q[h * p.dk + d], to_f32(k[d]), s);
+      s *= p.scale;
+      sc[j * (p.H + 1) + h] = p.softcap > 0.f ? p.softcap * tanhf(s / p.softcap) : s;
+    }
+    __syncthreads();
+    for (int i = tid; i < p.H * kKeys; i += 256) {
+      const int h = i / kKeys, j = i % kKeys;
+      float s = -INFINITY;
+      if (j < n) {
+        s = 0.f;
+        for (int g = 0; g < p.H; ++g) s = fmaf(to_f32(talk[h * p.H + g]), sc[j * (p.H + 1) + g], s);
+      }
+      mx[h * (kKeys + 1) + j] = s;
+    }
+    __syncthreads();
+    for (int h = tid >> 5; h < p.H; h += 8) {
+      const float s = mx[h * (kKeys + 1) + lane];
+      float top = s;
+#pragma unroll
+      for (int x = 16; x > 0; x >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, x));
+      const float next = fmaxf(m[h], top), e = expf(s - next), sum = warp_sum_f32(e);
+      mx[h * (kKeys + 1) + lane] = e;
+      __syncwarp();
+      if (lane == 0) {
+        corr[h] = expf(m[h] - next);
+        l[h] = l[h] * corr[h] + sum;
+        m[h] = next;
+      }
+    }
+    __syncthreads();
+    for (int i = tid; i < p.H * p.dv; i += 256) {
+      const int h = i / p.dv, d = i - h * p.dv;
+      float v = o[i] * corr[h];
+      for (int j = 0; j < n; ++j)
+        v = fmaf(mx[h * (kKeys + 1) + j],
+                 to_f32(static_cast<const T*>(p.v_cache)[((static_cast<size_t>(rows[j] >> 4) * p.G + h / r) * 16 + (rows[j] & 15)) * p.dv + d]), v);
+      o[i] = v;
+    }
+  }
+  __syncthreads();
+  T* out = static_cast<T*>(p.out) + static_cast<size_t>(row0 + blockIdx.x) * p.H * p.dv;
+  for (int i = tid; i < p.H * p.dv; i += 256) out[i] = from_f32<T>(l[i / p.dv] > 0.f ? o[i] / l[i / p.dv] : 0.f);
+}
+
+static TalkParams talk_params(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table, const int* seq_lens,
+                              const int* cu_q, const void* talk, const float* sinks, int q_per_seq, int max_pages, int H, int G, int dk,
+                              int dv, int window, int keep, float scale, float softcap) {
+  TalkParams p = {};
+  p.q = q;
+  p.k_cache = k_cache;
+  p.v_cache = v_cache;
+  p.out = out;
+  p.block_table = block_table;
+  p.seq_lens = seq_lens;
+  p.cu_q = cu_q;
+  p.talk = talk;
+  p.sinks = sinks;
+  p.q_per_seq = q_per_seq;
+  p.max_pages = max_pages;
+  p.H = H;
+  p.G = G;
+  p.dk = dk;
+  p.dv = dv;
+  p.window = window;
+  p.keep = window > 0 ? keep : 0;
+  p.scale = scale;
+  p.softcap = softcap;
+  return p;
+}
+
+constexpr int kDecodeRows = 8;   // up to this many queries per sequence are cut as decode steps
+
+}  // namespace eredu
+
+using namespace eredu;
+
+// 1 when the tensor-core kernel takes steps of at most `rows` queries per sequence of these sizes.
+extern "C" int eredu_talking_fits(int H, int G, int dk, int dv, int rows) {
+  return talk_plan(H, G, dk, dv, rows, false).qt > 0 && talk_plan(H, G, dk, dv, std::min(rows, kDecodeRows), true).qt > 0;
+}
+
+// bf16. q [rows, H, dk] (rows of sequence b: cu_q[b] .. cu_q[b + 1], or q_per_seq each; at most max_rows), its last positions; caches
+// [pages, G, 16, dk or dv]; talk [H, H] bf16; sinks fp32 [H] or null; window 0: all earlier keys, else the newest `window` and the first
+// `keep`. splits <= 8: CTAs that share a sequence's keys in a decode step (cu_q null).
+extern "C" int eredu_talking_attention(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                                       const int* seq_lens, const int* cu_q, const void* talk, const float* sinks, int batch, int q_per_seq,
+                                       int max_rows, int max_pages, int H, int G, int dk, int dv, int window, int keep, int splits, int qt,
+                                       int lanes, float scale, float softcap, cudaStream_t stream) {
+  if (batch <= 0 || max_rows <= 0) return 0;
+  if (window < 0 || keep < 0 || splits < 1 || splits > kMaxSplits || batch > 65535) return -1;
+  const bool decode = cu_q == nullptr && max_rows <= kDecodeRows;
+  TalkPlan t = talk_plan(H, G, dk, dv, max_rows, decode);
+  if (t.qt == 0) return -1;
+  if (qt > 0 && qt < t.qt) return -1;
+  if (lanes > 0 && lanes < t.lanes) t.lanes = lanes;
+  TalkParams p = talk_params(q, k_cache, v_cache, out, block_table, seq_lens, cu_q, talk, sinks, q_per_seq, max_pages, H, G, dk, dv, window,
+                             keep, scale, softcap);
+  p.qt = t.qt;
+  p.octets = t.octets;
+  p.warps = t.warps;
+  p.lanes = t.lanes;
+  p.splits = decode ? splits : 1;
+  p.group_bytes = t.group_bytes;
+  const dim3 grid((max_rows + t.qt - 1) / t.qt * p.splits, batch);
+  const int threads = t.warps * t.lanes * 32;
+  const bool small = dk <= 64 && dv <= 64;
+  cudaError_t e;
+  if (small && t.per_warp == 4) e = launch_talking<4, 4, 4>(p, grid, threads, t.smem, stream);
+  else if (small && t.per_warp == 2) e = launch_talking<4, 4, 2>(p, grid, threads, t.smem, stream);
+  else if (small) e = launch_talking<4, 4, 1>(p, grid, threads, t.smem, stream);
+  else if (t.per_warp == 2) e = launch_talking<8, 8, 2>(p, grid, threads, t.smem, stream);
+  else e = launch_talking<8, 8, 1>(p, grid, threads, t.smem, stream);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}
+
+// The same for fp32 (fp32 = 1) or bf16 and any sizes whose query and output rows fit shared memory.
+extern "C" int eredu_talking_attention_simt(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
+                                            const int* seq_lens, const int* cu_q, const void* talk, const float* sinks, int batch,
+                                            int q_per_seq, int max_rows, int max_pages, int H, int G, int dk, int dv, int window, int keep,
+                                            int fp32, float scale, float softcap, cudaStream_t stream) {
+  if (batch <= 0 || max_rows <= 0) return 0;
+  if (G <= 0 || H % G != 0 || dk <= 0 || dv <= 0 || window < 0 || keep < 0 || batch > 65535) return -1;
+  const TalkParams p = talk_params(q, k_cache, v_cache, out, block_table, seq_lens, cu_q, talk, sinks, q_per_seq, max_pages, H, G, dk, dv,
+                                   window, keep, scale, softcap);
+  const size_t smem = (static_cast<size_t>(H) * (dk + dv) + kKeys * (H + 1) + H * (kKeys + 1) + 3 * H) * sizeof(float);
+  if (smem > kSmemLimit - 1024) return -1;
+  auto run = [&](auto kernel, bool& configured) -> cudaError_t {
+    if (!configured) {
+      const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 1024);
+      if (e != cudaSuccess) return e;
+      configured = true;
+    }
+    return launch_pdl(kernel, dim3(max_rows, batch), dim3(256), smem, stream, p);
+  };
+  static bool done[2] = {};
+  const cudaError_t e = fp32 ? run(talking_simt_kernel<float>, done[0]) : run(talking_simt_kernel<__nv_bfloat16>, done[1]);
+  eredu_count_launches(1);
+  return static_cast<int>(e);
+}

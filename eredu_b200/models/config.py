@@ -17,7 +17,7 @@ QWEN_HYBRID_TYPES = {"qwen3_next", "qwen3_5", "qwen3_5_moe", "qwen3_5_text", "qw
 
 # Families whose layers each name their mixer and its sizes (``ModelConfig.mixers``). ``models/<model type>.py`` reads the
 # configuration and the tensors, and runs a block.
-MIXER_FAMILIES = ("nidozen", "lenitar", "kasuvik")
+MIXER_FAMILIES = ("nidozen", "lenitar", "kasuvik", "gulazen")
 
 
 def mixer_family(model_type: str):
@@ -39,6 +39,7 @@ class RoutedSpec:
     norm_topk_prob: bool = False
     routed_scaling_factor: float = 1.0
     swiglu_limit: float = 0.0
+    shared_ff: int = 0               # width of an expert that runs for every token (0: none)
 
 
 @dataclass
@@ -68,6 +69,10 @@ class MixerSpec:
     conv: int = 0                    # taps of the causal convolution over q, k and v (attention) or the channels (mamba); 0, 1: no history
     state: int = 0                   # mamba: states of a channel
     dt_rank: int = 0                 # mamba: width of the step size's input
+    keep_first: int = 0              # attention: the first tokens of a sequence stay visible behind the window
+    softcap: float = 0.0             # attention: scores are bounded to +-softcap by a tanh (0: they are not)
+    lead_conv: int = 0               # taps of the causal convolution over what the mixer reads; 0, 1: no history
+    lead_width: int = 0              # channels of that convolution
     left: "MixerSpec | None" = None  # parallel: the attention
     right: "MixerSpec | None" = None  # parallel: the recurrent mixer
 
@@ -103,6 +108,11 @@ class MixerSpec:
         return -(-max(0, self.conv - 1) * self.conv_channels // 4) * 4
 
     @property
+    def lead_elems(self) -> int:
+        """fp32 elements of the history of the convolution in front of the mixer, rounded up to whole 16-byte pieces."""
+        return -(-max(0, self.lead_conv - 1) * self.lead_width // 4) * 4
+
+    @property
     def state_shape(self) -> tuple | None:
         """fp32 recurrent state of one sequence (None: no recurrence)."""
         if self.kind == "general_delta":
@@ -110,8 +120,9 @@ class MixerSpec:
         if self.kind == "mamba":
             # the states of all channels, then the convolution's history [taps - 1, channels]
             return (-(-self.width * self.state // 4) * 4 + self.conv_elems,)
-        if self.kind == "attention" and self.conv > 1:
-            return (self.conv_elems,)
+        if self.kind == "attention" and (self.conv > 1 or self.lead_conv > 1):
+            # the history of the convolution in front of the mixer, then that of the projections
+            return (self.lead_elems + self.conv_elems,)
         if self.kind == "parallel":
             # both, the recurrent one first
             return (self.right.state_shape[0] + (self.left.state_shape or (0,))[0],)

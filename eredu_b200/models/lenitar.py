@@ -143,6 +143,7 @@ def random_tensor(name: str, shape: tuple, generator, std: float = 0.02, device=
 def build(model, cfg, get, has, up) -> None:
     """Fill ``model.layers`` (called by the generic loader after the embedding, final norm and head)."""
     from .llama import LayerWeights
+    from .moe import expert_block
 
     f32 = lambda n: up(get(n), torch.float32)                                          # noqa: E731
 
@@ -174,25 +175,12 @@ def build(model, cfg, get, has, up) -> None:
             e["inv_freq"] = base_inv_freq(s.rot_base, s.rot_dims).to(device=model.device, dtype=torch.float32)
         if s.moe is not None:
             small.append(f"l{li}.mlp.router")
-            lw.moe = _experts(model, li, s.moe, get, up)
+            lw.moe = expert_block(s.moe, li, f"l{li}.mlp.", get, up)
         if small:
             e["small"] = fused(small)
             bias = [get(n + ".b") if has(n + ".b") else torch.zeros(get(n).shape[0]) for n in small]
             e["small_b"] = up(torch.cat([b.to(e["small"].device, torch.float32) for b in bias])) if any(has(n + ".b") for n in small) else None
         model.layers.append(lw)
-
-
-def _experts(model, li, spec, get, up):
-    """Expert banks of one layer; an odd width is padded with zero rows (silu(0) * 0 adds nothing)."""
-    from .moe import MoEBlock
-
-    p, pad = f"l{li}.mlp.", -spec.moe_intermediate_size % 8
-    z = torch.nn.functional.pad
-    gu = torch.stack([torch.cat((z(get(f"{p}e{e}.gate"), (0, 0, 0, pad)), z(get(f"{p}e{e}.up"), (0, 0, 0, pad)))) for e in range(spec.num_experts)])
-    dn = torch.stack([z(get(f"{p}e{e}.down"), (0, pad)) for e in range(spec.num_experts)])
-    block = MoEBlock(spec, up(get(p + "router")), up(gu), up(dn), 0, spec.num_experts)
-    block.layer_index = li
-    return block
 
 
 # ---------------------------------------------------------------------------------------------- forward

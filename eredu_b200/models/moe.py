@@ -50,7 +50,7 @@ class MoEBlock:
             out.extend(self.shared)
         return out
 
-    def _shared_out(self, x):
+    def shared_out(self, x):
         """Dense shared expert (None without one), scaled by its sigmoid gate when the family has it."""
         if self.shared is None:
             return None
@@ -81,7 +81,7 @@ class MoEBlock:
 
     def routed_rows(self, x, logits):
         """Outputs of the routed experts, uncombined (:class:`ops.moe.RoutedRows`), for families that add them to the stream
-        together with the other sublayer. ``logits`` [T, E] fp32: rows of the router projection. Single rank, no shared expert."""
+        together with what else is added. ``logits`` [T, E] fp32: rows of the router projection. Single rank; without the shared expert."""
         self.stats["calls"] += 1
         c = self.cfg
         args = (c.num_experts_per_tok, c.router_scoring, c.norm_topk_prob, c.routed_scaling_factor, self.router_bias)
@@ -104,7 +104,7 @@ class MoEBlock:
         ids, w = moe_ops.route(logits.contiguous(), cfg.num_experts_per_tok, cfg.router_scoring, cfg.norm_topk_prob,
                                cfg.routed_scaling_factor, self.router_bias, cfg.n_group, cfg.topk_group)
         _, raw = moe_ops.route_ref(logits, cfg.num_experts_per_tok, cfg.router_scoring, False, 1.0, self.router_bias)
-        shared = self._shared_out(x)
+        shared = self.shared_out(x)
         cache = getattr(self, "expert_cache", None)
         if cache is not None:
             local = cache.forward(x, ids, w, limit=cfg.swiglu_limit, act=self.act)
@@ -133,7 +133,7 @@ class MoEBlock:
         if cache is not None:
             # experts live in host memory behind a bounded device bank: route, then let the cache run the experts
             ids, w = self.route(x)
-            extra = self._shared_out(x)
+            extra = self.shared_out(x)
             if self.ep_size == 1:
                 return cache.forward(x, ids, w, residual=residual, extra=extra, limit=self.cfg.swiglu_limit, act=self.act)
             partial = cache.forward(x, ids, w, extra=extra if self.e0 == 0 else None, limit=self.cfg.swiglu_limit,
@@ -149,7 +149,7 @@ class MoEBlock:
                                                          self.e0, self.w_gate_up.shape[0], cfg.n_group, cfg.topk_group)
         else:
             ids, w = self.route(x)
-        extra = self._shared_out(x)
+        extra = self.shared_out(x)
         if self.ep_size == 1:
             return moe_ops.experts_forward(x, ids, w, self.w_gate_up, self.w_down, self.e0, residual=residual,
                                            extra=extra, limit=self.cfg.swiglu_limit, plan=plan, xp=xp, gu_bias=self.gu_bias,
@@ -307,3 +307,19 @@ def attach_ep(model, ep_ops) -> None:
     for lw in model.layers:
         if lw.moe is not None:
             lw.moe.ep_ops = ep_ops
+
+
+def expert_block(spec, li: int, prefix: str, get, up) -> MoEBlock:
+    """Experts of one layer from tensors ``<prefix>router``, ``<prefix>e<i>.{gate,up,down}`` and, where ``spec`` (a RoutedSpec) has one,
+    ``<prefix>shared.{gate,up,down}``. An odd width is padded with zero rows (silu(0) * 0 adds nothing)."""
+    z = torch.nn.functional.pad
+
+    def bank(name, pad):
+        return (torch.cat((z(get(f"{name}.gate"), (0, 0, 0, pad)), z(get(f"{name}.up"), (0, 0, 0, pad)))), z(get(f"{name}.down"), (0, pad)))
+
+    banks = [bank(f"{prefix}e{e}", -spec.moe_intermediate_size % 8) for e in range(spec.num_experts)]
+    shared = tuple(up(t) for t in bank(prefix + "shared", -spec.shared_ff % 8)) if spec.shared_ff else None
+    block = MoEBlock(spec, up(get(prefix + "router")), up(torch.stack([b[0] for b in banks])), up(torch.stack([b[1] for b in banks])), 0,
+                     spec.num_experts, shared=shared)
+    block.layer_index = li
+    return block

@@ -198,3 +198,63 @@ def conv_project(proj, state, batch, page_to_slot, heads: Optional[ConvHeads] = 
         1 if fp32 else 0, stream_ptr(proj.device))
     check(code, "eredu_conv_project")
     return q, out
+
+
+native.register("eredu_stream_conv", I, [P] * 8 + [I] * 8 + [P])
+
+
+@dataclass
+class StreamConv:
+    """A causal convolution over the residual stream itself, in front of a sublayer. ``state`` [slots, >= (L - 1) W] starts with the last
+    L - 1 inputs of a sequence, oldest first (None: one tap needs none)."""
+    taps: torch.Tensor                    # fp32 [L, W], the last one multiplies the position itself
+    state: Optional[torch.Tensor]
+    batch: object                         # ForwardBatch
+    page_to_slot: Optional[torch.Tensor]
+
+    def checked(self, width: int):
+        """(taps, state) as the kernels read them."""
+        t, s = self.taps, self.state
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.shape[1] == width
+        if t.shape[0] == 1:
+            return t, None
+        assert s.dtype == torch.float32 and s.is_contiguous() and s[0].numel() >= (t.shape[0] - 1) * width
+        return t, s
+
+
+def stream_conv_ref(x, conv, act_dtype):
+    L, W = conv.taps.shape
+    out = torch.zeros(x.shape, dtype=act_dtype, device=x.device)
+    bounds = _sequences(conv.batch)
+    for b in range(len(bounds) - 1):
+        r0, r1 = bounds[b], bounds[b + 1]
+        if r1 <= r0 or int(conv.batch.slots[r0]) < 0:
+            continue
+        hist = x.new_zeros(0, W)
+        if L > 1:
+            hist = conv.state[int(conv.page_to_slot[int(conv.batch.block_table[b, 0])])].view(-1)[:(L - 1) * W].view(L - 1, W)
+        y, new = _conv_rows(x[r0:r1].float(), conv.taps.float(), hist.clone())
+        hist.copy_(new)
+        out[r0:r1] = (x[r0:r1] + y).to(act_dtype)
+    return out
+
+
+def stream_conv(x, conv: StreamConv, act_dtype):
+    """``x_t + sum_j taps[j] x_(t - L + 1 + j)`` on every channel of the fp32 stream [M, W], in ``act_dtype``; zeros in front of a sequence's
+    first token. The history in ``conv.state`` moves on. Portions may have any length."""
+    if not x.is_cuda:
+        return stream_conv_ref(x, conv, act_dtype)
+    M, W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and act_dtype in (torch.bfloat16, torch.float32)
+    out = torch.empty((M, W), dtype=act_dtype, device=x.device)
+    if M == 0:
+        return out
+    taps, state = conv.checked(W)
+    b = conv.batch
+    code = lib().eredu_stream_conv(
+        ptr(x), ptr(out), ptr(taps), ptr(state), ptr(b.block_table), ptr(conv.page_to_slot) if state is not None else None,
+        ptr(b.cu_q) if b.is_prefill else None, ptr(b.slots), b.block_table.shape[0], b.q_per_seq, b.max_q_len if b.is_prefill else b.q_per_seq,
+        b.block_table.stride(0), W, taps.shape[0], state[0].numel() if state is not None else 0, 1 if act_dtype == torch.float32 else 0,
+        stream_ptr(x.device))
+    check(code, "eredu_stream_conv")
+    return out

@@ -12,6 +12,7 @@ from __future__ import annotations
 from os import environ as _environ
 
 import math
+from dataclasses import dataclass
 
 import torch
 import torch.nn.functional as F
@@ -27,10 +28,30 @@ def _sm_count(device) -> int:
 
 
 # ------------------------------------------------------------------------------------------ linear
+@dataclass(frozen=True)
+class XIELU:
+    """xIELU (Huang, Schlag: "Deriving Activation Functions Using Integration"): ``above z^2 + z / 2`` for z > 0 and
+    ``below (e^z - 1 - z) + z / 2`` elsewhere."""
+    above: float
+    below: float
+
+    @classmethod
+    def from_checkpoint(cls, p: float, q: float) -> "XIELU":
+        """The two learned numbers behind a softplus, the lower one from 1/2 on."""
+        softplus = lambda t: max(t, 0.0) + math.log1p(math.exp(-abs(t)))                # noqa: E731
+        return cls(softplus(p), 0.5 + softplus(q))
+
+    def __call__(self, z):
+        n = z.clamp_max(0)
+        return torch.where(z > 0, self.above * z * z, self.below * (torch.expm1(n) - n)) + z / 2
+
+
 def linear_ref(x, w, bias=None, residual=None, out_dtype=None, activation=None):
     y = F.linear(x.float(), w.float(), None if bias is None else bias.float())
     if activation == "relu2":
         y = torch.relu(y).square()
+    elif activation is not None:
+        y = activation(y)
     if residual is not None:
         y = y + residual.float()
     return y.to(out_dtype or x.dtype)
@@ -63,10 +84,11 @@ def linear(x, w, bias=None, residual=None, out_dtype=None, out=None, force_split
     ``want_ssq``: also return per-128-column-tile sums of squares of the stored output ([M, ceil(N/128)]).
     ``dynamic_weight``: ``w`` was written by a kernel enqueued just before this call (e.g. a dequantised scratch
     matrix); the kernel then does not fetch weight tiles ahead of its stream dependency.
-    ``activation``: None or "relu2" (the square of ReLU), applied in the epilogue before the residual.
+    ``activation``: None, "relu2" (the square of ReLU) or an :class:`XIELU`, applied in the epilogue before the residual.
     fp32 operands are multiplied in true 32-bit; bf16 operands whose rows a TMA descriptor cannot describe (a row pitch or
     start that is not a multiple of 16 bytes) take the same CUDA-core kernel."""
-    if activation not in (None, "relu2"):
+    xielu = activation if isinstance(activation, XIELU) else None
+    if activation not in (None, "relu2") and xielu is None:
         raise ValueError(f"unknown activation {activation!r}")
     if not x.is_cuda:
         if row_ssq is not None:
@@ -91,7 +113,8 @@ def linear(x, w, bias=None, residual=None, out_dtype=None, out=None, force_split
         ptr(x), ptr(w), ptr(out), ptr(residual), ptr(bias), M, N, K, x.stride(0), w.stride(0), out.stride(0),
         residual.stride(0) if residual is not None else 0, w.shape[0], 0, 0, 1 if out_dtype == torch.float32 else 0,
         force_split, _sm_count(x.device), ptr(status_word(x.device)), ptr(ssq_in), parts, eps, dim, ptr(ssq_out),
-        (1 if dynamic_weight else 0) | (2 if activation == "relu2" else 0), stream_ptr(x.device))
+        (1 if dynamic_weight else 0) | (2 if activation == "relu2" else 8 if xielu else 0), xielu.above if xielu else 0.0,
+        xielu.below if xielu else 0.0, stream_ptr(x.device))
     check(code, "eredu_gemm_bf16")
     return (out, ssq_out) if want_ssq else out
 
@@ -100,7 +123,7 @@ def _tma_rows(t) -> bool:
     return t.stride(1) == 1 and (t.stride(0) * t.element_size()) % 16 == 0 and t.data_ptr() % 16 == 0
 
 
-native.register("eredu_gemm_simt", native.I, [native.P] * 4 + [native.I] * 9 + [native.P])
+native.register("eredu_gemm_simt", native.I, [native.P] * 4 + [native.I] * 9 + [native.F, native.F, native.P])
 
 
 def _linear_simt(x, w, bias, out_dtype, activation, out=None):
@@ -108,15 +131,16 @@ def _linear_simt(x, w, bias, out_dtype, activation, out=None):
     assert x.dtype == w.dtype and x.dtype in (torch.float32, torch.bfloat16) and x.stride(1) == 1 and w.stride(1) == 1
     assert bias is None or (bias.dtype == x.dtype and bias.is_contiguous())
     M, K = x.shape
-    act = {None: 0, "relu2": 1, "gated_silu": 2, "gated_relu": 3}[activation]
-    N = w.shape[0] // 2 if act >= 2 else w.shape[0]
+    xielu = isinstance(activation, XIELU)
+    act = 4 if xielu else {None: 0, "relu2": 1, "gated_silu": 2, "gated_relu": 3}[activation]
+    N = w.shape[0] // 2 if act in (2, 3) else w.shape[0]
     if out is None:
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
     if M == 0:
         return out
     code = lib().eredu_gemm_simt(ptr(x), ptr(w), ptr(out), ptr(bias), M, N, K, x.stride(0), w.stride(0), out.stride(0),
                                  1 if x.dtype == torch.float32 else 0, 1 if out.dtype == torch.float32 else 0,
-                                 act, stream_ptr(x.device))
+                                 act, activation.above if xielu else 0.0, activation.below if xielu else 0.0, stream_ptr(x.device))
     check(code, "eredu_gemm_simt")
     return out
 
@@ -143,7 +167,7 @@ def gated_linear(x, w_gate_up, inter, bias=None, out=None, force_split=0, row_ss
     code = lib().eredu_gemm_bf16(
         ptr(x), ptr(w_gate_up), ptr(out), None, ptr(bias), M, inter, K, x.stride(0), w_gate_up.stride(0),
         out.stride(0), 0, w_gate_up.shape[0], 1, inter, 0, force_split, _sm_count(x.device),
-        ptr(status_word(x.device)), ptr(ssq_in), parts, eps, dim, None, 4 if activation == "relu" else 0, stream_ptr(x.device))
+        ptr(status_word(x.device)), ptr(ssq_in), parts, eps, dim, None, 4 if activation == "relu" else 0, 0.0, 0.0, stream_ptr(x.device))
     check(code, "eredu_gemm_bf16(dual)")
     return out
 
@@ -172,50 +196,95 @@ def rmsnorm(x, weight, eps, residual=None, weight_offset=0.0):
 
 
 native.register("eredu_rms_residual", native.I, [native.P] * 5 + [native.I] * 4 + [native.F, native.P])
-native.register("eredu_embedding_stream", native.I, [native.P] * 4 + [native.I] * 4 + [native.F, native.P])
+native.register("eredu_embedding_stream", native.I, [native.P] * 6 + [native.I] * 4 + [native.F, native.P])
+native.register("eredu_rms_routed_residual", native.I, [native.P] * 13 + [native.I] * 8 + [native.F, native.P])
 native.register("eredu_qkv_prepare", native.I, [native.P] * 9 + [native.I] * 10 + [native.F, native.P])
 
 
-def rms_residual_ref(y, weight, eps, residual=None, act_dtype=None):
-    n = y.float()
+MAX_ROUTES = 32         # routes of a token the kernels add up
+
+
+def rms_residual_ref(y, weight, eps, residual=None, act_dtype=None, routed=None, conv=None, want_act=True):
+    n = y.float() if y is not None else 0.0
+    if routed is not None:
+        n = n + routed.summed()
     n = n * torch.rsqrt(n.square().mean(-1, keepdim=True) + eps) * weight.float()
     if residual is not None:
         n = residual + n
+    if not want_act:
+        return n, None
+    if conv is not None:
+        from .conv import stream_conv_ref
+
+        return n, stream_conv_ref(n, conv, act_dtype or y.dtype)
     return n, n.to(act_dtype or y.dtype)
 
 
-def rms_residual(y, weight, eps, residual=None, act_dtype=None):
+def rms_residual(y, weight, eps, residual=None, act_dtype=None, routed=None, conv=None, want_act=True):
     """Norm on a sublayer's output: ``x = residual + weight * y / rms(y)`` in fp32, and its copy in ``act_dtype``.
     ``weight``: fp32, one number for all coordinates ([1]) or one per coordinate. Without a residual only the copy of the
-    normalised rows is made (the first result is then None, or the copy itself when it is fp32). Returns (x, copy)."""
+    normalised rows is made (the first result is then None, or the copy itself when it is fp32). Returns (x, copy).
+    ``routed`` (:class:`ops.moe.RoutedRows`): expert rows whose weighted sum is added to ``y`` (which may be None) first.
+    ``conv`` (:class:`ops.conv.StreamConv`; decode steps of one token per sequence): the copy is ``x + conv(x)``.
+    ``want_act=False``: no copy."""
     act_dtype = act_dtype or y.dtype
-    if not y.is_cuda:
-        return rms_residual_ref(y, weight, eps, residual, act_dtype)
-    assert y.is_contiguous() and weight.dtype == torch.float32 and weight.numel() in (1, y.shape[1])
+    ref = y if y is not None else routed.rows
+    if not ref.is_cuda:
+        return rms_residual_ref(y, weight, eps, residual, act_dtype, routed, conv, want_act)
+    M, W = y.shape if y is not None else (routed.weights.shape[0], routed.rows.shape[1])
+    assert (y is None or y.is_contiguous()) and weight.dtype == torch.float32 and weight.numel() in (1, W)
     assert residual is None or (residual.dtype == torch.float32 and residual.is_contiguous())
-    M, W = y.shape
-    act = torch.empty((M, W), dtype=act_dtype, device=y.device)
-    fp32_act = act_dtype == torch.float32
-    x = act if fp32_act else (torch.empty((M, W), dtype=torch.float32, device=y.device) if residual is not None else None)
-    code = lib().eredu_rms_residual(ptr(y), ptr(weight), ptr(residual), ptr(x), None if fp32_act else ptr(act), M, W,
-                                    1 if y.dtype == torch.float32 else 0, 0 if weight.numel() == 1 else 1, eps,
-                                    stream_ptr(y.device))
-    check(code, "eredu_rms_residual")
+    act = torch.empty((M, W), dtype=act_dtype, device=ref.device) if want_act else None
+    fp32 = ref.dtype == torch.float32
+    if routed is None and conv is None:
+        shared = want_act and act_dtype == torch.float32
+        x = act if shared else (torch.empty((M, W), dtype=torch.float32, device=ref.device) if residual is not None else None)
+        code = lib().eredu_rms_residual(ptr(y), ptr(weight), ptr(residual), ptr(x), None if shared else ptr(act), M, W,
+                                        1 if fp32 else 0, 0 if weight.numel() == 1 else 1, eps, stream_ptr(ref.device))
+        check(code, "eredu_rms_residual")
+        return x, act
+    assert residual is not None and weight.numel() == W and act_dtype == ref.dtype
+    x = torch.empty((M, W), dtype=torch.float32, device=ref.device)
+    rows = pos = w = None
+    k = 0
+    if routed is not None and routed.weights.shape[1] > MAX_ROUTES:
+        y, routed = (routed.summed() if y is None else y.float() + routed.summed()).to(ref.dtype), None
+    if routed is not None:
+        rows, pos, w = routed.rows, routed.route_pos, routed.weights
+        k = w.shape[1]
+        assert rows.is_contiguous() and rows.shape[1] == W and w.shape[0] == M and w.dtype == torch.float32 and (y is None or y.dtype == rows.dtype)
+    taps = state = table = p2s = slots = None
+    if conv is not None:
+        assert want_act and not conv.batch.is_prefill and conv.batch.q_per_seq == 1
+        taps, state = conv.checked(W)
+        if state is not None:
+            table, p2s, slots = conv.batch.block_table, conv.page_to_slot, conv.batch.slots
+    code = lib().eredu_rms_routed_residual(
+        ptr(y), ptr(rows), ptr(pos), ptr(w), ptr(weight), ptr(residual), ptr(x), ptr(act), ptr(taps), ptr(state), ptr(table), ptr(p2s), ptr(slots),
+        M, W, k, taps.shape[0] if taps is not None else 0, state[0].numel() if state is not None else 0,
+        table.stride(0) if table is not None else 0, 1 if fp32 else 0, 1 if W % 4 == 0 else 0, eps, stream_ptr(ref.device))
+    check(code, "eredu_rms_routed_residual")
     return x, act
 
 
-def embedding_stream(ids, table, scale=1.0, want_act=True):
-    """Rows of ``table`` times ``scale`` as the start of an fp32 residual stream: (fp32 rows, rows in the table's dtype or None)."""
+def embedding_stream(ids, table, scale=1.0, want_act=True, positions=None, inv_freq=None):
+    """Rows of ``table`` times ``scale`` as the start of an fp32 residual stream: (fp32 rows, rows in the table's dtype or None).
+    With ``inv_freq`` (fp32, one per pair of columns) sinusoidal position vectors are added: column 2 i gets
+    sin(position * inv_freq[i]), column 2 i + 1 the cosine."""
     if not table.is_cuda:
         x = table[ids.long()].float() * scale
+        if inv_freq is not None:
+            a = positions.float()[:, None] * inv_freq.float()[None]
+            x = x + torch.stack((a.sin(), a.cos()), -1).flatten(1)[:, :x.shape[1]]
         return x, (x.to(table.dtype) if want_act else None)
     assert ids.dtype == torch.int32 and table.is_contiguous()
     M, W = ids.shape[0], table.shape[1]
+    assert inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.numel() == (W + 1) // 2 and positions.dtype == torch.int32)
     x = torch.empty((M, W), dtype=torch.float32, device=table.device)
     fp32 = table.dtype == torch.float32
     act = x if fp32 else (torch.empty((M, W), dtype=table.dtype, device=table.device) if want_act else None)
-    code = lib().eredu_embedding_stream(ptr(ids), ptr(table), ptr(x), None if fp32 else ptr(act), M, W, table.shape[0],
-                                        1 if fp32 else 0, scale, stream_ptr(table.device))
+    code = lib().eredu_embedding_stream(ptr(ids), ptr(table), ptr(x), None if fp32 else ptr(act), ptr(positions) if inv_freq is not None else None,
+                                        ptr(inv_freq), M, W, table.shape[0], 1 if fp32 else 0, scale, stream_ptr(table.device))
     check(code, "eredu_embedding_stream")
     return x, act
 

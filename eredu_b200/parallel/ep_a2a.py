@@ -111,7 +111,7 @@ class CollectiveA2A:
         out_own = (ret.view(n_own, k, H).float() * w[:, :, None]).sum(1)       # slot order
         if residual is not None:
             out_own = out_own + residual[t0:t0 + n_own].float()
-        extra = block._shared_out(x_own) if n_own > 0 else None
+        extra = block.shared_out(x_own) if n_own > 0 else None
         if extra is not None:
             out_own = out_own + extra.float()
         padded = torch.zeros((per, H), dtype=x.dtype, device=x.device)
@@ -200,7 +200,7 @@ class PeerA2A:
                                     act=block.act, rows_only=True)
         native.check(self.lib.eredu_moe_a2a_return(self.pg.comm, view, native.ptr(y), native.ptr(plan.route_pos), native.ptr(st),
                                                    stream), "eredu_moe_a2a_return")
-        extra = block._shared_out(x_own) if n_own > 0 else None
+        extra = block.shared_out(x_own) if n_own > 0 else None
         res_own = residual[t0:t0 + n_own] if (residual is not None and n_own > 0) else None
         native.check(self.lib.eredu_moe_a2a_combine(self.pg.comm, view, native.ptr(w), native.ptr(res_own), native.ptr(extra), n_own,
                                                     t0, native.ptr(st), stream), "eredu_moe_a2a_combine")
