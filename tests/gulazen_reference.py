@@ -121,8 +121,11 @@ def routing(logits, top):
     return idx, e / e.sum(-1, keepdim=True)
 
 
-def experts(p, mlp, w, h):
+def experts(p, mlp, w, h, gaps=None):
     z = h @ w[p + "router"].to(h.dtype).t() + w[p + "router.b"].to(h.dtype)
+    if gaps is not None and mlp["router"]["top"] < mlp["router"]["experts"]:
+        best = torch.sort(z, -1, descending=True).values
+        gaps.append((best[:, mlp["router"]["top"] - 1] - best[:, mlp["router"]["top"]]) / z.std())
     idx, weight = routing(z, mlp["router"]["top"])
     out = gated(p + "shared.", w, h) if mlp.get("shared") else torch.zeros_like(h)
     for e in range(mlp["router"]["experts"]):
@@ -132,24 +135,25 @@ def experts(p, mlp, w, h):
     return out
 
 
-def layer(i, spec, cfg, w, x):
+def layer(i, spec, cfg, w, x, gaps=None):
     p, eps = f"l{i}.", cfg["norm"]["eps"]
     h = x + causal_conv(x, w[p + "canon1"])
     x = x + norm_plus_one(attention(p + "mix.", spec["mixer"], w, h, eps), w[p + "norm1"], eps) * w[p + "ls1"].to(x.dtype)
     mlp = spec.get("mlp")
     if mlp is not None:
-        y = dense(p + "mlp.", w, x) if mlp["kind"] == "dense" else experts(p + "mlp.", mlp, w, x)
+        y = dense(p + "mlp.", w, x) if mlp["kind"] == "dense" else experts(p + "mlp.", mlp, w, x, gaps)
         x = x + norm_plus_one(y, w[p + "norm2"], eps) * w[p + "ls2"].to(x.dtype)
     return x
 
 
-def forward(cfg, w, tokens, dtype=torch.float64, return_layers=False):
-    """Logits [T, vocab] of one sequence (and the stream behind every layer)."""
+def forward(cfg, w, tokens, dtype=torch.float64, return_layers=False, gaps=None):
+    """Logits [T, vocab] of one sequence (and the stream behind every layer). ``gaps`` collects, per routed layer, how far the last chosen
+    expert's logit is ahead of the next one's, over the logits' standard deviation."""
     table = w["embed"].to(dtype)
     x = table[torch.as_tensor(tokens)] + position_vectors(torch.arange(len(tokens)), cfg["width"], dtype)
     layers = []
     for i, spec in enumerate(cfg["layers"]):
-        x = layer(i, spec, cfg, w, x)
+        x = layer(i, spec, cfg, w, x, gaps)
         layers.append(x)
     logits = norm_plus_one(x, w["final.norm"], cfg["norm"]["eps"]) @ table.t()
     return (logits, torch.stack(layers)) if return_layers else logits
@@ -230,3 +234,10 @@ def errors(got, want):
 
 def error(got, want):
     return float(errors(got, want).max())
+
+
+def decided(cfg, w, tokens, gap=0.03):
+    """Rows in which rounding cannot change which experts are chosen."""
+    gaps = []
+    forward(cfg, w, tokens, torch.float32, gaps=gaps)
+    return torch.stack(gaps).min(0).values > gap if gaps else torch.ones(len(tokens), dtype=torch.bool)

@@ -336,8 +336,13 @@ def test_scores_are_mixed_in_32_bit(dev, dt):
 
 
 # ---------------------------------------------------------------------------------------------- whole models
-def agrees(got, want, dt, slack=1.0):
+def agrees(got, want, dt, slack=1.0, of=None):
+    """``of`` (configuration, weights, tokens): in bf16, rows are left out where two experts' logits are so close that rounding chooses."""
     e = R.errors(got, want)
+    if of is not None and dt == torch.bfloat16:
+        keep = R.decided(*of)
+        assert float(keep.float().mean()) > 0.6
+        e = e * keep
     assert float(e.max()) < slack * LIMIT[dt], (float(e.max()), int(e.argmax()))
 
 
@@ -350,7 +355,7 @@ def test_prompt_portions_and_decoding_agree_with_the_restatement(dev, dt, cfg):
     eng = engine_for(cfg, w, dev, dt, max_seq_len=160, num_pages=11, state_slots=1)      # room for one: every run reuses it
     for sizes in ([150], [100, 1], [2, 3, 2, 17, 64], [37, 20, 43, 50], [1]):
         seq = eng.open_sequence()
-        agrees(feed(eng, seq, tokens, sizes), want, dt, 3.0 if cfg is ODD and dt == torch.bfloat16 else 1.0)   # narrow layers amplify rounding
+        agrees(feed(eng, seq, tokens, sizes), want, dt, 3.0 if cfg is ODD and dt == torch.bfloat16 else 1.0, (cfg, w, tokens))   # narrow layers amplify rounding
         eng.release(seq)
 
 
@@ -383,11 +388,11 @@ def test_residual_stream_of_every_layer(dev, dt):
     want, layers = R.forward(MIXED, w, tokens, return_layers=True)
     eng = engine_for(MIXED, w, dev, dt)
     eng.model.observer = watch = Watch()
-    agrees(feed(eng, eng.open_sequence(), tokens, [70]), want, dt)
+    agrees(feed(eng, eng.open_sequence(), tokens, [70]), want, dt, of=(MIXED, w, tokens))
     for i, x in enumerate(layers):
         close(watch.outputs[f"model.layers.{i}.output"], x, dt, limit=1e-4 if dt == torch.float32 else 3e-2)
     seq = eng.open_sequence()
-    agrees(feed(eng, seq, tokens, [60, 1]), want, dt)                     # observed decode steps
+    agrees(feed(eng, seq, tokens, [60, 1]), want, dt, of=(MIXED, w, tokens))                     # observed decode steps
     watch.zero = "model.layers.3.output"                                  # a stream somebody replaced is what the next layer reads
     assert R.error(feed(eng, eng.open_sequence(), tokens, [70]), want) > 0.1
 
@@ -399,7 +404,7 @@ def test_first_tokens_and_one_token_prompts(dev, dt):
     for n in (1, 2, 3, 16, 17):
         tokens = prompt(n, MIXED["vocab"], n)
         seq = eng.open_sequence()
-        agrees(feed(eng, seq, tokens, [n]), R.forward(MIXED, w, tokens), dt)
+        agrees(feed(eng, seq, tokens, [n]), R.forward(MIXED, w, tokens), dt, of=(MIXED, w, tokens))
         eng.release(seq)
 
 
@@ -454,7 +459,7 @@ def test_mixed_batches_and_reused_pages(dev, dt):
             if live[i][1] == len(reqs[i]):
                 eng.release(live.pop(i)[0])
     for i in range(len(reqs)):
-        agrees(torch.cat(got[i]), want[i], dt)
+        agrees(torch.cat(got[i]), want[i], dt, of=(MIXED, w, reqs[i]))
     assert eng.kv.allocator.free_pages() == 19 and len(eng.kv._free_state_slots) == 3
 
 
@@ -463,7 +468,7 @@ def test_long_decoding_across_windows_and_kept_tokens(dev, dt):
     w = R.weights(SMALL, seed=6)
     tokens = prompt(330, SMALL["vocab"], 7)
     eng = engine_for(SMALL, w, dev, dt, max_seq_len=336)
-    agrees(feed(eng, eng.open_sequence(), tokens, [30, 1]), R.forward(SMALL, w, tokens), dt)
+    agrees(feed(eng, eng.open_sequence(), tokens, [30, 1]), R.forward(SMALL, w, tokens), dt, of=(SMALL, w, tokens))
 
 
 @both
@@ -479,7 +484,7 @@ def test_wide_layers(dev, dt):
     first = eng.forward_tokens([(s, r[:n], range(n)) for s, r, n in zip(seqs, reqs, heads)]).split(heads)
     rest = [eng.forward_tokens([(s, [r[n + i]], [0]) for s, r, n in zip(seqs, reqs, heads)]) for i in range(10)]
     for i in range(3):
-        agrees(torch.cat([first[i]] + [x[i:i + 1] for x in rest]), want[i], dt)
+        agrees(torch.cat([first[i]] + [x[i:i + 1] for x in rest]), want[i], dt, of=(cfg, w, reqs[i]))
 
 
 # ---------------------------------------------------------------------------------------------- generation
