@@ -256,7 +256,7 @@ def main() -> int:
                     help="collectives of the tensor / expert ranks: kernels over NVLink peer memory, or torch.distributed (NCCL)")
     ap.add_argument("--router-skew", type=float, default=0.0,
                     help="sparse models: this fraction of the tokens is biased onto 8 hot experts (0 = as routed)")
-    ap.add_argument("--design", default=None, choices=["nidozen", "lenitar", "kasuvik"],
+    ap.add_argument("--design", default=None, choices=["nidozen", "lenitar", "kasuvik", "gulazen"],
                     help="instead of the headline workload: prefill and decode throughput of this design at a few sizes beside the "
                          "closest model at equal size, and its kernels against their rooflines (benchmarks/bench_<design>.py)")
     ap.add_argument("--no-baseline", action="store_true", help="skip the in-process baseline arm that fills vs_baseline")

@@ -335,6 +335,34 @@ def test_scores_are_mixed_in_32_bit(dev, dt):
     close(got, want, dt, limit=1e-3 if dt == torch.float32 else None)
 
 
+@both
+@pytest.mark.parametrize("H,G,d", [(16, 4, 128), (8, 2, 64), (32, 8, 128), (6, 2, 24)])
+@pytest.mark.parametrize("shift", [-400.0, -130.0, 0.0, 130.0, 400.0])
+def test_scores_of_any_size(dev, dt, H, G, d, shift):
+    """Softmaxes of scores far from zero, of some rows and heads only: exponentials of the scores themselves would leave the range of fp32."""
+    T, window, keep = 90, 40, 6
+    q, k, v = rand(T, H, d, seed=1), rand(T, G, d, seed=2) * 0.1, rand(T, G, d, seed=3)
+    q[..., 0], k[..., 0] = 0.0, 1.0
+    q[::3, ::2, 0] = shift                                                   # every third query, every second head
+    q, k = q.to(torch.bfloat16).double(), k.to(torch.bfloat16).double()
+    talk, sink = torch.eye(H, dtype=torch.float64), rand(H, seed=4)
+    talk[0, 1] = 0.5
+    sink[2] = shift
+    table = [4, 2, 7, 1, 3, 6]
+    pos = torch.arange(T)
+    at_page = torch.tensor(table)[pos // 16]
+    kc, vc = (torch.zeros(8, G, 16, d, device=dev, dtype=dt) for _ in range(2))
+    kc[at_page, :, pos % 16], vc[at_page, :, pos % 16] = k.to(dev, dt), v.to(dev, dt)
+    for cap in (0.0, 1000.0):
+        want = R.talking_attention(q, k, v, 1.0, cap or 1e9, talk, sink, window, keep)
+        assert bool(want.isfinite().all())
+        for portions, prefill in (([(0, T)], True), ([(50, 40)], True), ([(33, 1), (60, 1), (89, 1)], False)):
+            rows = [p for a, n in portions for p in range(a, a + n)]
+            got = ops.talking_attention(q[rows].contiguous().to(dev, dt), kc, vc, batch_of(portions, [table] * len(portions), dev, prefill, T), talk.to(dev, dt), 1.0, cap,
+                                        sink.float().to(dev), window, keep)
+            close(got, want[rows], dt, limit=1e-3 if dt == torch.float32 else 1.5e-2)
+
+
 # ---------------------------------------------------------------------------------------------- whole models
 def agrees(got, want, dt, slack=1.0, of=None):
     """``of`` (configuration, weights, tokens): in bf16, rows are left out where two experts' logits are so close that rounding chooses."""
