@@ -10,12 +10,13 @@
 // stages deep. Prompts: one group of up to 16 warps and as many queries as fit its registers. Decode steps: several groups per CTA, each
 // with pages of its own, and the CTAs of a cluster share a sequence's keys; partial results meet in (distributed) shared memory.
 //
-// The kernel for prompts of the usual head sizes knows that exponents of fp32 and bf16 reach far: it forms exp(S' - c) in the mix step with
-// c = 0, keeps the maximum of every row beside, and starts over with c = the maximum in the rare case that one lies beyond 2^+-100. So O is
-// never rescaled, and the three steps of three successive pages share one barrier.
+// The kernel for prompts of the usual head sizes knows that exponents of fp32 and bf16 reach far: its mix step forms exp(S') itself, without
+// a maximum. In the rare case that some row's sum leaves 2^+-100 it finds the maxima in a pass of their own and starts over with
+// exp(S' - maximum). So O is never rescaled, and the three steps of three successive pages share one barrier.
 //
 // A third kernel on the CUDA cores takes fp32, head sizes the first is not built for, and more than 64 heads.
 #include <algorithm>
+#include <type_traits>
 
 #include "../common/elem.cuh"
 #include "../common/launch.h"
@@ -87,6 +88,8 @@ __device__ __forceinline__ void cap_pair(float& x, float& y, float in, float c) 
   x = fmaf(-r, b, c);
   y = fmaf(-r, a, c);
 }
+// The same of one value; for any x, since 2^128 becomes infinity and its reciprocal zero.
+__device__ __forceinline__ float cap_one(float x, float in, float c) { return fmaf(-2.f * c, rcp(1.f + ex2(x * in)), c); }
 // x = hi + mid + lo, each exact in bf16 (truncation: 8 + 8 + 8 bits); the pieces of two values side by side.
 __device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t& mid, uint32_t& lo) {
   const uint32_t ux = __float_as_uint(x), uy = __float_as_uint(y);
@@ -99,6 +102,12 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t&
 __device__ __forceinline__ uint32_t pack2(float x, float y) {
   const __nv_bfloat162 t = __floats2bfloat162_rn(x, y);
   return *reinterpret_cast<const uint32_t*>(&t);
+}
+// The product without an order among other asm statements.
+__device__ __forceinline__ void mma_pure(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void group_sync(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
 __device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
@@ -555,23 +564,25 @@ struct PromptLayout {
   __host__ __device__ __forceinline__ int total() const { return t.talk() + 2 * (t.k_bytes + t.v_bytes + t.s_bytes + p_bytes) + refs(); }
 };
 
-// D: head size. U column octets of one key / value head per warp, HB blocks of 16 heads, NT (query, eight keys) products of the mix step per
-// warp at most, W warps at most.
-template <int D, int U, int HB, int NT, int W>
-__global__ void __launch_bounds__(32 * W, 1) talking_prompt_kernel(TalkParams p) {
+// D: head size; HB blocks of 16 heads; NT (query, eight keys) products of the mix step per warp. A warp holds kUnits column octets of one
+// key / value head.
+constexpr int kUnits = 4, kPromptWarps = 8;
+
+template <int D, int HB, int NT>
+__global__ void __launch_bounds__(32 * kPromptWarps, 1) talking_prompt_kernel(TalkParams p) {
   using bf16 = __nv_bfloat16;
-  constexpr int KS = D / 16, VT = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16;
+  constexpr int U = kUnits, KS = D / 16, VT = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16;
   constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4, PP = PromptLayout::kProbPitch;
   extern __shared__ __align__(16) uint8_t smem[];
   __shared__ int far_row;
   pdl_launch_early();
   const PromptLayout lay(p.H, p.G, D, p.qt);
   const int tid = threadIdx.x, lane = tid & 31, quad = lane & 3, oct = lane >> 2, gw = tid >> 5, threads = blockDim.x, nwarps = threads >> 5;
-  const int b = blockIdx.y, r = p.H / p.G;
+  const int b = blockIdx.y, r = p.H / p.G, columns = p.qt * r;
   uint8_t *ks = smem + lay.t.talk(), *vs = ks + 2 * lay.t.k_bytes;
   float* sc = reinterpret_cast<float*>(vs + 2 * lay.t.v_bytes);
   uint8_t* ps = reinterpret_cast<uint8_t*>(sc) + 2 * lay.t.s_bytes;
-  float* ref = reinterpret_cast<float*>(ps + 2 * lay.p_bytes);          // c of every (query, head)
+  float* ref = reinterpret_cast<float*>(ps + 2 * lay.p_bytes);          // -c of every (query, head)
   const int s_stage = lay.t.s_bytes / 4, p_stage = lay.p_bytes, kv_stage = lay.t.k_bytes;
 
   for (int i = tid; i < lay.total() / 16; i += threads) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
@@ -589,15 +600,19 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_kernel(TalkParams p)
   const TalkPages pages = talk_pages(p0, p1, p.window, p.keep);
   const int* bt = p.block_table + static_cast<size_t>(b) * p.max_pages;
   const int n = pages.count;
+  if (n <= 0) return;
 
-  // ---- the warp's columns: one key / value head, U octets side by side
+  // ---- the warp's columns: one key / value head, U octets side by side; columns beyond the last query are zeros that nobody reads
   const int g = gw * U / p.octets, o0 = gw * U % p.octets;
   uint32_t qf[U][KS][2];
-  int s_off[U];
+  int s_off[U][2];
 #pragma unroll
   for (int u = 0; u < U; ++u) {
-    const int cs = (o0 + u) * 8 + quad * 2;                             // two columns of a score fragment: heads of one query (r is even)
-    s_off[u] = cs / r * SQ + g * r + cs % r + oct * SP;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = (o0 + u) * 8 + quad * 2 + e;
+      s_off[u][e] = c < columns ? c / r * SQ + g * r + c % r + oct * SP : -1;
+    }
     const int c = (o0 + u) * 8 + oct, cq = c / r;
     const bf16* src = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row0 + qi0 + cq) * p.H + g * r + c % r) * D + quad * 2;
 #pragma unroll
@@ -609,106 +624,136 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_kernel(TalkParams p)
   uint32_t p_addr[U / 2];
 #pragma unroll
   for (int u = 0; u < U / 2; ++u) {
-    const int c = (o0 + 2 * u + (lane >> 4)) * 8 + (lane & 7);
+    const int c = min((o0 + 2 * u + (lane >> 4)) * 8 + (lane & 7), columns - 1);
     p_addr[u] = smem_u32(ps) + (c / r * HP + g * r + c % r) * PP + ((lane >> 3) & 1) * 16;
   }
   const uint32_t k_addr = smem_u32(ks) + (g * kPage + (lane & 15)) * PITCH + (lane >> 4) * 16;
   const uint32_t v_addr = smem_u32(vs) + (g * kPage + (lane & 7) + (lane >> 4) * 8) * PITCH + ((lane >> 3) & 1) * 16;
   const uint32_t talk_a = smem_u32(smem) + (lane & 15) * (HP + 8) * 2 + (lane >> 4) * 16;
-  const float cap_c = p.softcap * kLog2e, cap_in = p.softcap > 0.f ? 2.f * kLog2e * p.scale / p.softcap : 0.f, plain = p.scale * kLog2e;
+  const float cap_c = p.softcap * kLog2e, cap_in = 2.f * kLog2e * p.scale / p.softcap;
 
   // ---- asynchronous copies: a page's rows of all key / value heads lie in one piece; a thread's place in it is fixed
-  const int pieces = p.G * kPage * PIECES;
-  const uint32_t copy_dst = (tid / PIECES) * PITCH + (tid % PIECES) * 16;
+  const int pieces = p.G * kPage * PIECES, copies = pieces / threads;
+  const uint32_t copy_dst = (tid / PIECES) * PITCH + (tid % PIECES) * 16, copy_step = threads / PIECES * PITCH;
   auto load = [&](const void* cache, uint32_t dst, int page) {
     const uint4* src = static_cast<const uint4*>(cache) + static_cast<size_t>(page) * pieces + tid;
     dst += copy_dst;
-    for (int i = tid; i < pieces; i += threads) {
+#pragma unroll 4
+    for (int i = 0; i < copies; ++i) {
       asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
       src += threads;
-      dst += threads / PIECES * PITCH;
+      dst += copy_step;
     }
   };
 
-  float o[U][VT][4], l[NT][HB][2], top[NT][HB][2];
+  float o[U][VT][4], l[NT][HB][2];
   auto score = [&](int buf) {
     float s[U][4];
 #pragma unroll
     for (int u = 0; u < U; ++u) s[u][0] = s[u][1] = s[u][2] = s[u][3] = 0.f;
     const uint32_t base = k_addr + buf * kv_stage;
+    uint32_t a[2][4];
+    ldsm_x4(base, a[0][0], a[0][1], a[0][2], a[0][3]);
 #pragma unroll
     for (int k = 0; k < KS; ++k) {
-      uint32_t a0, a1, a2, a3;
-      ldsm_x4(base + k * 32, a0, a1, a2, a3);
+      uint32_t* c = a[k & 1];
+      uint32_t* f = a[(k + 1) & 1];
+      if (k + 1 < KS) ldsm_x4(base + (k + 1) * 32, f[0], f[1], f[2], f[3]);
 #pragma unroll
-      for (int u = 0; u < U; ++u) mma16816(s[u], a0, a1, a2, a3, qf[u][k][0], qf[u][k][1]);
+      for (int u = 0; u < U; ++u) mma_pure(s[u], c[0], c[1], c[2], c[3], qf[u][k][0], qf[u][k][1]);
     }
     float* dst = sc + buf * s_stage;
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      if (p.softcap > 0.f) {
-        cap_pair(s[u][0], s[u][1], cap_in, cap_c);
-        cap_pair(s[u][2], s[u][3], cap_in, cap_c);
-      } else {
+    for (int u = 0; u < U; ++u)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[u][e] *= plain;
-      }
-      *reinterpret_cast<float2*>(dst + s_off[u]) = make_float2(s[u][0], s[u][1]);
-      *reinterpret_cast<float2*>(dst + s_off[u] + 8 * SP) = make_float2(s[u][2], s[u][3]);
+      for (int e = 0; e < 4; ++e) s[u][e] = cap_one(s[u][e], cap_in, cap_c);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (s_off[u][e] >= 0) {
+          dst[s_off[u][e]] = s[u][e];
+          dst[s_off[u][e] + 8 * SP] = s[u][2 + e];
+        }
     }
   };
 
-  auto mix = [&](int buf, int key0) {
-    const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+  // MASK: some key of the page is hidden from some query. MAX: only the maxima, into l.
+  auto mix = [&](int buf, int key0, auto masked, auto maxima) {
+    constexpr bool MASK = decltype(masked)::value, MAX = decltype(maxima)::value;
+    // all products side by side: their steps are long chains
+    float acc[NT][HB][4];
+    int row[NT];                                                        // (query, first head of the thread)
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
-      const int t = gw + j * nwarps, qq = t >> 1, k0 = (t & 1) * 8;
-      if (qq >= p.qt) break;
-      const float* src = sc + buf * s_stage + qq * SQ + (k0 + oct) * SP + quad * 2;
-      float acc[HB][4];
+      const int t = min(gw + j * nwarps, 2 * p.qt - 1);
+      row[j] = (t >> 1) * HP + oct;
 #pragma unroll
       for (int h = 0; h < HB; ++h) {
-        const float c0 = ref[qq * HP + h * 16 + oct], c1 = ref[qq * HP + h * 16 + 8 + oct];     // -c
-        acc[h][0] = acc[h][1] = c0;
-        acc[h][2] = acc[h][3] = c1;
+        acc[j][h][0] = acc[j][h][1] = ref[row[j] + h * 16];
+        acc[j][h][2] = acc[j][h][3] = ref[row[j] + h * 16 + 8];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < HB; ++e) {
+      uint32_t bf[NT][3][2];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int t = min(gw + j * nwarps, 2 * p.qt - 1);
+        const float* src = sc + buf * s_stage + (t >> 1) * SQ + ((t & 1) * 8 + oct) * SP + quad * 2 + e * 16;
+        const float2 x = *reinterpret_cast<const float2*>(src), y = *reinterpret_cast<const float2*>(src + 8);
+        split3(x.x, x.y, bf[j][0][0], bf[j][1][0], bf[j][2][0]);
+        split3(y.x, y.y, bf[j][0][1], bf[j][1][1], bf[j][2][1]);
       }
 #pragma unroll
-      for (int e = 0; e < HB; ++e) {
-        const float2 x = *reinterpret_cast<const float2*>(src + e * 16), y = *reinterpret_cast<const float2*>(src + e * 16 + 8);
-        uint32_t h0, h1, m0, m1, l0, l1;
-        split3(x.x, x.y, h0, m0, l0);
-        split3(y.x, y.y, h1, m1, l1);
+      for (int h = 0; h < HB; ++h) {
+        uint32_t a0, a1, a2, a3;
+        ldsm_x4(talk_a + h * 16 * (HP + 8) * 2 + e * 32, a0, a1, a2, a3);
 #pragma unroll
-        for (int h = 0; h < HB; ++h) {
-          uint32_t a0, a1, a2, a3;
-          ldsm_x4(talk_a + h * 16 * (HP + 8) * 2 + e * 32, a0, a1, a2, a3);
-          mma16816(acc[h], a0, a1, a2, a3, l0, l1);
-          mma16816(acc[h], a0, a1, a2, a3, m0, m1);
-          mma16816(acc[h], a0, a1, a2, a3, h0, h1);
-        }
+        for (int x = 2; x >= 0; --x)
+#pragma unroll
+          for (int j = 0; j < NT; ++j) mma_pure(acc[j][h], a0, a1, a2, a3, bf[j][x][0], bf[j][x][1]);
       }
-      if (!inner) {
-        const int pos = p0 + qq;
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int t = min(gw + j * nwarps, 2 * p.qt - 1), k0 = (t & 1) * 8;
+      if constexpr (MASK) {
+        const int pos = p0 + (t >> 1);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           const int key = key0 + k0 + quad * 2 + e;
-          if (key > pos || (p.window > 0 && pos - key >= p.window && key >= p.keep)) {
+          const bool hide = key > pos || (p.window > 0 && pos - key >= p.window && key >= p.keep);
 #pragma unroll
-            for (int h = 0; h < HB; ++h) acc[h][e] = acc[h][2 + e] = -INFINITY;
+          for (int h = 0; h < HB; ++h) {
+            acc[j][h][e] = hide ? -INFINITY : acc[j][h][e];
+            acc[j][h][2 + e] = hide ? -INFINITY : acc[j][h][2 + e];
           }
         }
       }
-      uint8_t* dst = ps + buf * p_stage + (qq * HP + oct) * PP + (k0 + quad * 2) * 2;
 #pragma unroll
       for (int h = 0; h < HB; ++h) {
-        top[j][h][0] = fmaxf(top[j][h][0], fmaxf(acc[h][0], acc[h][1]));
-        top[j][h][1] = fmaxf(top[j][h][1], fmaxf(acc[h][2], acc[h][3]));
+        if constexpr (MAX) {
+          l[j][h][0] = fmaxf(l[j][h][0], fmaxf(acc[j][h][0], acc[j][h][1]));
+          l[j][h][1] = fmaxf(l[j][h][1], fmaxf(acc[j][h][2], acc[j][h][3]));
+        } else {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) acc[h][e] = ex2(acc[h][e]);
-        l[j][h][0] += acc[h][0] + acc[h][1];
-        l[j][h][1] += acc[h][2] + acc[h][3];
-        *reinterpret_cast<uint32_t*>(dst + h * 16 * PP) = pack2(acc[h][0], acc[h][1]);
-        *reinterpret_cast<uint32_t*>(dst + (h * 16 + 8) * PP) = pack2(acc[h][2], acc[h][3]);
+          for (int e = 0; e < 4; ++e) acc[j][h][e] = ex2(acc[j][h][e]);
+          l[j][h][0] += acc[j][h][0] + acc[j][h][1];
+          l[j][h][1] += acc[j][h][2] + acc[j][h][3];
+        }
+      }
+    }
+    if constexpr (!MAX) {
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int t = min(gw + j * nwarps, 2 * p.qt - 1);
+        uint8_t* dst = ps + buf * p_stage + row[j] * PP + ((t & 1) * 8 + quad * 2) * 2;
+#pragma unroll
+        for (int h = 0; h < HB; ++h) {
+          *reinterpret_cast<uint32_t*>(dst + h * 16 * PP) = pack2(acc[j][h][0], acc[j][h][1]);
+          *reinterpret_cast<uint32_t*>(dst + (h * 16 + 8) * PP) = pack2(acc[j][h][2], acc[j][h][3]);
+        }
       }
     }
   };
@@ -718,87 +763,114 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_kernel(TalkParams p)
 #pragma unroll
     for (int u = 0; u < U; u += 2) ldsm_x4(p_addr[u / 2] + buf * p_stage, pf[u][0], pf[u][1], pf[u + 1][0], pf[u + 1][1]);
     const uint32_t base = v_addr + buf * kv_stage;
+    uint32_t a[2][4];
+    ldsm_x4_t(base, a[0][0], a[0][1], a[0][2], a[0][3]);
 #pragma unroll
     for (int v = 0; v < VT; ++v) {
-      uint32_t a0, a1, a2, a3;
-      ldsm_x4_t(base + v * 32, a0, a1, a2, a3);
+      uint32_t* c = a[v & 1];
+      uint32_t* f = a[(v + 1) & 1];
+      if (v + 1 < VT) ldsm_x4_t(base + (v + 1) * 32, f[0], f[1], f[2], f[3]);
 #pragma unroll
-      for (int u = 0; u < U; ++u) mma16816(o[u][v], a0, a1, a2, a3, pf[u][0], pf[u][1]);
+      for (int u = 0; u < U; ++u) mma_pure(o[u][v], c[0], c[1], c[2], c[3], pf[u][0], pf[u][1]);
     }
   };
 
+  // ---- pages. Iteration i: scores of page i + 1, mixing of page i, sums of page i - 1; keys are fetched two pages ahead, values one. What an
+  // iteration writes was read before the barrier in front of it. The first one's sums are of zeros, the last one's scores are not read.
   const uint32_t ks_a = smem_u32(ks), vs_a = smem_u32(vs);
-  float* sums = nullptr;
-  for (int pass = 0; pass < 2; ++pass) {
-#pragma unroll
-    for (int u = 0; u < U; ++u)
-#pragma unroll
-      for (int v = 0; v < VT; ++v) o[u][v][0] = o[u][v][1] = o[u][v][2] = o[u][v][3] = 0.f;
-#pragma unroll
-    for (int t = 0; t < NT; ++t)
-#pragma unroll
-      for (int h = 0; h < HB; ++h) {
-        l[t][h][0] = l[t][h][1] = 0.f;
-        top[t][h][0] = top[t][h][1] = -INFINITY;
-      }
-    // ---- pages. Iteration i: scores of page i + 1, mixing of page i, sums of page i - 1; keys are fetched two pages ahead, values one.
-    // What an iteration writes was read before its first barrier, by the one in front of it.
-    auto page_at = [&](int i) { return i < n ? bt[pages.at(i)] : 0; };
+  auto page_at = [&](int i) { return bt[pages.at(min(i, n - 1))]; };
+  auto walk = [&](auto maxima) {
+    constexpr bool MAX = decltype(maxima)::value;
     int pg0 = page_at(0), pg1 = page_at(1), pg2 = page_at(2);
     load(p.k_cache, ks_a, pg0);
-    if (n > 1) load(p.k_cache, ks_a + kv_stage, pg1);
+    load(p.k_cache, ks_a + kv_stage, pg1);
     cp_async_commit();
     cp_async_wait<0>();
-    if (tid == 0) far_row = 0;
     __syncthreads();
     score(0);
     __syncthreads();
     for (int i = 0; i < n; ++i) {
-      const int pg3 = page_at(i + 3), cur = i & 1;
-      if (i + 2 < n) load(p.k_cache, ks_a + cur * kv_stage, pg2);
+      const int pg3 = page_at(i + 3), cur = i & 1, key0 = pages.at(i) * kPage;
+      const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+      load(p.k_cache, ks_a + cur * kv_stage, pg2);
       load(p.v_cache, vs_a + cur * kv_stage, pg0);
       cp_async_commit();
-      if (i + 1 < n) score(cur ^ 1);
-      mix(cur, pages.at(i) * kPage);
-      if (i > 0) combine(cur ^ 1);
+      if constexpr (MAX) {
+        score(cur ^ 1);
+        mix(cur, key0, std::true_type(), std::true_type());
+      } else if (gw < kPromptWarps / 2) {
+        score(cur ^ 1);
+        if (inner) mix(cur, key0, std::false_type(), std::false_type());
+        else mix(cur, key0, std::true_type(), std::false_type());
+        combine(cur ^ 1);
+      } else {
+        if (inner) mix(cur, key0, std::false_type(), std::false_type());
+        else mix(cur, key0, std::true_type(), std::false_type());
+        combine(cur ^ 1);
+        score(cur ^ 1);
+      }
       cp_async_wait<0>();
       __syncthreads();
       pg0 = pg1;
       pg1 = pg2;
       pg2 = pg3;
     }
-    combine((n - 1) & 1);
-
-    // ---- maxima and sums of the two halves of the keys, [qt hp][4] over the probabilities of the page before the last
-    sums = reinterpret_cast<float*>(ps + (n & 1) * p_stage);
+  };
+  // The l of all threads, by keys of the two halves of a page: [qt hp][2] over the probabilities of the page before the last.
+  float* sums = reinterpret_cast<float*>(ps + (n & 1) * p_stage);
+  auto spread = [&](auto maxima) {
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
-      const int t = gw + j * nwarps, qq = t >> 1;
-      if (qq >= p.qt) break;
+      const int t = min(gw + j * nwarps, 2 * p.qt - 1), qq = t >> 1;
 #pragma unroll
       for (int h = 0; h < HB; ++h)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          float v = l[j][h][e], m = top[j][h][e];
-          v += __shfl_xor_sync(0xffffffffu, v, 1);
-          v += __shfl_xor_sync(0xffffffffu, v, 2);
-          m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 1));
-          m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, 2));
-          if (quad == 0) *reinterpret_cast<float2*>(sums + ((qq * HP + h * 16 + e * 8 + oct) * 2 + (t & 1)) * 2) = make_float2(v, m);
+          float v = l[j][h][e];
+#pragma unroll
+          for (int x = 1; x <= 2; x *= 2) {
+            const float w = __shfl_xor_sync(0xffffffffu, v, x);
+            v = decltype(maxima)::value ? fmaxf(v, w) : v + w;
+          }
+          if (quad == 0) sums[(qq * HP + h * 16 + e * 8 + oct) * 2 + (t & 1)] = v;
         }
     }
     __syncthreads();
+  };
+  auto reset = [&](float start) {
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int h = 0; h < HB; ++h) l[t][h][0] = l[t][h][1] = start;
+  };
+  for (int pass = 0;; ++pass) {
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int v = 0; v < VT; ++v) o[u][v][0] = o[u][v][1] = o[u][v][2] = o[u][v][3] = 0.f;
+    reset(0.f);
+    if (tid == 0) far_row = 0;
+    walk(std::false_type());
+    combine((n - 1) & 1);
+    spread(std::false_type());
     if (pass > 0) break;
-    for (int i = tid; i < nq * HP; i += threads) {
-      const float m = fmaxf(sums[i * 4 + 1], sums[i * 4 + 3]);
-      if (!(fabsf(m) <= kFar)) {
-        far_row = 1;
-        ref[i] = fabsf(m) < INFINITY ? -m : 0.f;
-      }
+    for (int i = tid; i < nq * p.H; i += threads) {
+      const float2 v = *reinterpret_cast<const float2*>(sums + (i / p.H * HP + i % p.H) * 2);
+      if (!(v.x + v.y >= exp2f(-kFar) && v.x + v.y <= exp2f(kFar))) far_row = 1;
     }
     __syncthreads();
     if (far_row == 0) break;
-    __syncthreads();                                                    // all have read the flag
+    // c = the maximum of every row; probabilities start from zeros again
+    reset(-INFINITY);
+    walk(std::true_type());
+    spread(std::true_type());
+    for (int i = tid; i < p.qt * HP; i += threads) {
+      const float m = fmaxf(sums[i * 2], sums[i * 2 + 1]);
+      ref[i] = fabsf(m) < INFINITY ? -m : 0.f;
+    }
+    __syncthreads();
+    for (int i = tid; i < 2 * p_stage / 16; i += threads) reinterpret_cast<uint4*>(ps)[i] = make_uint4(0, 0, 0, 0);
+    __syncthreads();
   }
 
   bf16* out = static_cast<bf16*>(p.out) + static_cast<size_t>(row0 + qi0) * p.H * D;
@@ -807,11 +879,11 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_kernel(TalkParams p)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int c = (o0 + u) * 8 + quad * 2 + e, cq = c / r, h = g * r + c % r;
-      const float sum = sums[(cq * HP + h) * 4] + sums[(cq * HP + h) * 4 + 2];
+      if (cq >= nq) continue;
+      const float sum = sums[(cq * HP + h) * 2] + sums[(cq * HP + h) * 2 + 1];
       // the sink, in units of the row's own sum
       const float sink = p.sinks != nullptr ? fmaf(p.sinks[h], kLog2e, ref[cq * HP + h]) - __log2f(sum) : -INFINITY;
       const float f = 1.f / (sum * (1.f + ex2(fminf(sink, 120.f))));
-      if (cq >= nq) continue;
       bf16* dst = out + (cq * p.H + h) * D + oct;
 #pragma unroll
       for (int v = 0; v < VT; ++v) {
@@ -826,39 +898,42 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_kernel(TalkParams p)
 struct PromptPlan {
   int qt = 0, octets = 0, warps = 0, smem = 0, blocks = 0, per = 0;   // per: products of the mix step a warp takes
 };
-static PromptPlan prompt_plan(int H, int G, int dk, int dv, int rows) {
+static PromptPlan prompt_plan(int H, int G, int dk, int dv, int rows, float softcap) {
   PromptPlan best;
-  if (G <= 0 || H % G != 0 || (H / G) % 2 != 0 || H > 64 || dk != dv || (dk != 64 && dk != 128)) return best;
-  const int r = H / G, U = dk == 64 ? 4 : 2, blocks = H <= 16 ? 1 : H <= 32 ? 2 : 4;
-  for (int qt = 32; qt >= 4; qt /= 2) {
-    if (qt / 2 >= rows) continue;
+  if (G <= 0 || H % G != 0 || H > 64 || dk != dv || (dk != 64 && dk != 128) || softcap <= 0.f) return best;
+  for (int qt = 32; qt >= 2; qt /= 2) {
+    if (qt / 2 >= rows && qt > 2) continue;
     PromptPlan t;
     t.qt = qt;
-    t.octets = qt * r / 8;
-    if (qt * r % 8 != 0 || t.octets % U != 0) continue;
-    t.warps = G * t.octets / U;
-    t.blocks = blocks;
-    const int pieces = dk / 8;
+    t.octets = ((qt * (H / G) + 7) / 8 + kUnits - 1) / kUnits * kUnits;
+    t.warps = G * t.octets / kUnits;
+    t.blocks = H <= 16 ? 1 : H <= 32 ? 2 : 4;
     t.per = (2 * qt + t.warps - 1) / t.warps;
     const PromptLayout lay(H, G, dk, qt);
     t.smem = lay.total();
-    if (t.warps < 4 || t.warps > 16 || t.warps * 32 % pieces != 0 || t.per > (blocks == 1 ? 2 * U : blocks == 2 ? U : U / 2) ||
-        t.smem > kSmemLimit - 64 || lay.t.hp != 16 * blocks)
+    if (t.warps > kPromptWarps || t.warps * 32 % (dk / 8) != 0 || G * kPage * (dk / 8) % (t.warps * 32) != 0 || t.per > 8 / t.blocks ||
+        t.smem > kSmemLimit - 256 || lay.t.hp != 16 * t.blocks)
       continue;
     return t;
   }
   return best;
 }
 
-template <int D, int U, int HB, int NT, int W>
-static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, int threads, int smem, cudaStream_t stream) {
+template <int D, int HB, int NT>
+static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_kernel<D, U, HB, NT, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 64);
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_kernel<D, HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_kernel<D, U, HB, NT, W>, grid, dim3(threads), smem, stream, p);
+  return launch_pdl(talking_prompt_kernel<D, HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
+}
+template <int D>
+static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
+  if (t.blocks == 1) return t.per <= 4 ? launch_prompt<D, 1, 4>(p, grid, t, stream) : launch_prompt<D, 1, 8>(p, grid, t, stream);
+  if (t.blocks == 2) return t.per <= 2 ? launch_prompt<D, 2, 2>(p, grid, t, stream) : launch_prompt<D, 2, 4>(p, grid, t, stream);
+  return t.per <= 1 ? launch_prompt<D, 4, 1>(p, grid, t, stream) : launch_prompt<D, 4, 2>(p, grid, t, stream);
 }
 
 // ---------------------------------------------------------------------------------------------- CUDA cores
@@ -1001,24 +1076,12 @@ extern "C" int eredu_talking_attention(const void* q, const void* k_cache, const
   const bool decode = cu_q == nullptr && max_rows <= kDecodeRows;
   TalkParams p = talk_params(q, k_cache, v_cache, out, block_table, seq_lens, cu_q, talk, sinks, q_per_seq, max_pages, H, G, dk, dv, window,
                              keep, scale, softcap);
-  const PromptPlan pp = decode ? PromptPlan() : prompt_plan(H, G, dk, dv, max_rows);
+  const PromptPlan pp = decode ? PromptPlan() : prompt_plan(H, G, dk, dv, max_rows, softcap);
   if (pp.qt > 0) {
     p.qt = pp.qt;
     p.octets = pp.octets;
     const dim3 grid((max_rows + pp.qt - 1) / pp.qt, batch);
-    const int threads = pp.warps * 32;
-    cudaError_t e;
-#define ER_PROMPT(D_, U_, HB_, NT_) launch_prompt<D_, U_, HB_, NT_, 16>(p, grid, threads, pp.smem, stream)
-    if (dk == 64) {
-      if (pp.blocks == 1) e = pp.per <= 4 ? ER_PROMPT(64, 4, 1, 4) : ER_PROMPT(64, 4, 1, 8);
-      else if (pp.blocks == 2) e = pp.per <= 2 ? ER_PROMPT(64, 4, 2, 2) : ER_PROMPT(64, 4, 2, 4);
-      else e = ER_PROMPT(64, 4, 4, 2);
-    } else {
-      if (pp.blocks == 1) e = pp.per <= 2 ? ER_PROMPT(128, 2, 1, 2) : ER_PROMPT(128, 2, 1, 4);
-      else if (pp.blocks == 2) e = pp.per <= 1 ? ER_PROMPT(128, 2, 2, 1) : ER_PROMPT(128, 2, 2, 2);
-      else e = ER_PROMPT(128, 2, 4, 1);
-    }
-#undef ER_PROMPT
+    const cudaError_t e = dk == 64 ? launch_prompt<64>(p, grid, pp, stream) : launch_prompt<128>(p, grid, pp, stream);
     eredu_count_launches(1);
     return static_cast<int>(e);
   }
