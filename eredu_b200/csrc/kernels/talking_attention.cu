@@ -45,7 +45,8 @@ struct TalkParams {
   const float* sinks;      // [H] or null
   int q_per_seq, max_pages, H, G, dk, dv, window, keep;
   float scale, softcap;
-  // tensor-core kernel
+  int* status;             // where a wait that runs out is recorded
+  // tensor-core kernels
   int qt;                  // queries of a CTA
   int octets;              // column octets per key / value head
   int warps;               // warps of a group
@@ -900,7 +901,7 @@ struct PromptPlan {
 };
 static PromptPlan prompt_plan(int H, int G, int dk, int dv, int rows, float softcap) {
   PromptPlan best;
-  if (G <= 0 || H % G != 0 || H > 64 || dk != dv || (dk != 64 && dk != 128) || softcap <= 0.f) return best;
+  if (G <= 0 || H % G != 0 || H > 64 || dk != 64 || dv != 64 || softcap <= 0.f) return best;
   for (int qt = 32; qt >= 2; qt /= 2) {
     if (qt / 2 >= rows && qt > 2) continue;
     PromptPlan t;
@@ -919,21 +920,455 @@ static PromptPlan prompt_plan(int H, int G, int dk, int dv, int rows, float soft
   return best;
 }
 
-template <int D, int HB, int NT>
+template <int HB, int NT>
 static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_kernel<D, HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_kernel<64, HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_kernel<D, HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
+  return launch_pdl(talking_prompt_kernel<64, HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
 }
-template <int D>
 static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
-  if (t.blocks == 1) return t.per <= 4 ? launch_prompt<D, 1, 4>(p, grid, t, stream) : launch_prompt<D, 1, 8>(p, grid, t, stream);
-  if (t.blocks == 2) return t.per <= 2 ? launch_prompt<D, 2, 2>(p, grid, t, stream) : launch_prompt<D, 2, 4>(p, grid, t, stream);
-  return t.per <= 1 ? launch_prompt<D, 4, 1>(p, grid, t, stream) : launch_prompt<D, 4, 2>(p, grid, t, stream);
+  if (t.blocks == 1) return t.per <= 4 ? launch_prompt<1, 4>(p, grid, t, stream) : launch_prompt<1, 8>(p, grid, t, stream);
+  if (t.blocks == 2) return t.per <= 2 ? launch_prompt<2, 2>(p, grid, t, stream) : launch_prompt<2, 4>(p, grid, t, stream);
+  return t.per <= 1 ? launch_prompt<4, 1>(p, grid, t, stream) : launch_prompt<4, 2>(p, grid, t, stream);
+}
+
+// ---------------------------------------------------------------------------------------------- prompts, head size 128
+// The same steps with the sums on tcgen05: O^T[value dim, column] of a key / value head lies in tensor memory, one product of 128 value dims x
+// its columns x 16 keys a page, V as it comes (swizzled rows of keys) and P as the mix step leaves it (core matrices of 8 columns x 8 keys).
+constexpr int kTcHead = 128, kTcUnits = 2, kTcWarps = 16;
+
+struct PromptTcLayout {
+  TalkLayout t;
+  int columns;                            // of a key / value head, whole octets
+  int p_head, p_bytes, v_bytes;           // probabilities of a head (64 bytes apart from whole rows of banks), of a page; values of a page
+  int v_off, k_off, s_off, p_off, ref_off, sum_off, total;
+  __host__ __device__ __forceinline__ PromptTcLayout(int H, int G, int qt, int octets) : t(H, G, kTcHead, kTcHead, qt) {
+    columns = octets * 8;
+    p_head = columns * 32 + 64;
+    p_bytes = G * p_head;
+    v_bytes = G * kPage * kTcHead * 2;
+    v_off = 0;                            // 1024-byte aligned
+    k_off = 2 * v_bytes;
+    s_off = k_off + 2 * t.k_bytes;
+    p_off = s_off + 2 * t.s_bytes;
+    ref_off = p_off + 2 * p_bytes;
+    sum_off = ref_off + qt * t.hp * 4;
+    total = sum_off + qt * t.hp * 8 + t.talk();
+  }
+};
+
+// K-major operand in core matrices of 8 rows x 16 bytes: the two halves of K = 16 lie 128 bytes apart, groups of 8 rows 256.
+__device__ __forceinline__ uint64_t umma_desc_k_core(uint32_t smem_addr) {
+  return static_cast<uint64_t>((smem_addr & 0x3FFFF) >> 4) | static_cast<uint64_t>(128 >> 4) << 16 | static_cast<uint64_t>(256 >> 4) << 32 |
+         static_cast<uint64_t>(1) << 46;
+}
+// MN-major operand, rows of 64 elements (128-byte swizzle), 16 rows: the next 64 elements `lbo` bytes on, 8 rows 1024.
+__device__ __forceinline__ uint64_t umma_desc_mn_rows(uint32_t smem_addr, uint32_t lbo) {
+  return static_cast<uint64_t>((smem_addr & 0x3FFFF) >> 4) | static_cast<uint64_t>(lbo >> 4) << 16 | static_cast<uint64_t>(1024 >> 4) << 32 |
+         static_cast<uint64_t>(1) << 46 | static_cast<uint64_t>(2) << 61;
+}
+
+template <int HB, int NT>
+__global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(TalkParams p) {
+  using bf16 = __nv_bfloat16;
+  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16;
+  constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4;
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  __shared__ int far_row;
+  __shared__ uint32_t tmem_slot;
+  __shared__ __align__(8) uint64_t done[2];       // sums of a page of this parity are complete
+  pdl_launch_early();
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const PromptTcLayout lay(p.H, p.G, p.qt, p.octets);
+  const int tid = threadIdx.x, lane = tid & 31, quad = lane & 3, oct = lane >> 2, gw = tid >> 5, threads = blockDim.x, nwarps = threads >> 5;
+  const int b = blockIdx.y, r = p.H / p.G, columns = p.qt * r;
+  float* sc = reinterpret_cast<float*>(smem + lay.s_off);
+  uint8_t* ps = smem + lay.p_off;
+  float* ref = reinterpret_cast<float*>(smem + lay.ref_off);            // -c of every (query, head)
+  float* sums = reinterpret_cast<float*>(smem + lay.sum_off);           // [qt hp][2]
+  bf16* talk_s = reinterpret_cast<bf16*>(smem + lay.total - lay.t.talk());
+  const int s_stage = lay.t.s_bytes / 4, p_stage = lay.p_bytes, k_stage = lay.t.k_bytes, v_stage = lay.v_bytes;
+
+  for (int i = tid; i < lay.total / 16; i += threads) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
+  __syncthreads();
+  for (int i = tid; i < p.H * p.H; i += threads) talk_s[i / p.H * (HP + 8) + i % p.H] = static_cast<const bf16*>(p.talk)[i];
+
+  pdl_wait();
+  pdl_launch_dependents();
+  const int row0 = p.cu_q != nullptr ? p.cu_q[b] : b * p.q_per_seq;
+  const int q_len = p.cu_q != nullptr ? p.cu_q[b + 1] - row0 : p.q_per_seq;
+  const int qi0 = blockIdx.x * p.qt;
+  if (qi0 >= q_len) return;
+  const int nq = min(p.qt, q_len - qi0);
+  const int p0 = p.seq_lens[b] - q_len + qi0, p1 = p0 + nq - 1;
+  const TalkPages pages = talk_pages(p0, p1, p.window, p.keep);
+  const int* bt = p.block_table + static_cast<size_t>(b) * p.max_pages;
+  const int n = pages.count;
+  if (n <= 0) return;
+
+  int tcols = 32;
+  while (tcols < p.G * lay.columns) tcols *= 2;
+  if (gw == 0) {
+    tmem_alloc(&tmem_slot, tcols);
+    tmem_relinquish();
+  }
+  if (tid == 32) {
+    mbar_init(&done[0], 1);
+    mbar_init(&done[1], 1);
+    fence_mbar_init();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem = tmem_slot;
+
+  // ---- the warp's columns: one key / value head, U octets side by side; columns beyond the last query are zeros that nobody reads
+  const int g = gw * U / p.octets, o0 = gw * U % p.octets;
+  uint32_t qf[U][KS][2];
+  int s_off[U][2];
+#pragma unroll
+  for (int u = 0; u < U; ++u) {
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int c = (o0 + u) * 8 + quad * 2 + e;
+      s_off[u][e] = c < columns ? c / r * SQ + g * r + c % r + oct * SP : -1;
+    }
+    const int c = (o0 + u) * 8 + oct, cq = c / r;
+    const bf16* src = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row0 + qi0 + cq) * p.H + g * r + c % r) * D + quad * 2;
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) qf[u][k][e] = cq < nq ? *reinterpret_cast<const uint32_t*>(src + k * 16 + e * 8) : 0u;
+  }
+  // ---- where the warp's products of the mix step read scores and leave probabilities
+  const bool mixes = gw < 2 * p.qt;
+  int mix_src[NT], p_dst[NT][HB][2];
+#pragma unroll
+  for (int j = 0; j < NT; ++j) {
+    const int t = min(gw + j * nwarps, 2 * p.qt - 1), qq = t >> 1;
+    mix_src[j] = qq * SQ + ((t & 1) * 8 + oct) * SP + quad * 2;
+#pragma unroll
+    for (int h = 0; h < HB; ++h)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int head = h * 16 + e * 8 + oct, c = qq * r + head % r;
+        p_dst[j][h][e] = head < p.H ? head / r * lay.p_head + (c >> 3) * 256 + (t & 1) * 128 + (c & 7) * 16 + quad * 4 : -1;
+      }
+  }
+  const uint32_t ks_a = smem_u32(smem + lay.k_off), vs_a = smem_u32(smem + lay.v_off), ps_a = smem_u32(ps);
+  const uint32_t k_addr = ks_a + (g * kPage + (lane & 15)) * PITCH + (lane >> 4) * 16;
+  const uint32_t talk_a = smem_u32(talk_s) + (lane & 15) * (HP + 8) * 2 + (lane >> 4) * 16;
+  const float cap_c = p.softcap * kLog2e, cap_in = 2.f * kLog2e * p.scale / p.softcap;
+
+  // ---- asynchronous copies: a page's rows of all key / value heads lie in one piece; a thread's place in it is fixed
+  const int pieces = p.G * kPage * PIECES, copies = pieces / threads, row = tid / PIECES, chunk = tid % PIECES;
+  const uint32_t k_dst = row * PITCH + chunk * 16, k_step = threads / PIECES * PITCH;
+  const uint32_t v_dst = (row / kPage) * (kPage * D * 2) + (chunk >> 3) * 2048 + (row % kPage) * 128 + (((chunk & 7) ^ (row & 7)) << 4);
+  const uint32_t v_step = threads / PIECES * (D * 2);                   // whole heads: a thread keeps its row of a page
+  auto load = [&](const void* cache, uint32_t dst, uint32_t step, int page) {
+    const uint4* src = static_cast<const uint4*>(cache) + static_cast<size_t>(page) * pieces + tid;
+#pragma unroll 4
+    for (int i = 0; i < copies; ++i) {
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+      src += threads;
+      dst += step;
+    }
+  };
+
+  float l[NT][HB][2];
+  auto score = [&](int buf) {
+    float s[U][4];
+#pragma unroll
+    for (int u = 0; u < U; ++u) s[u][0] = s[u][1] = s[u][2] = s[u][3] = 0.f;
+    const uint32_t base = k_addr + buf * k_stage;
+    uint32_t a[KS][4];
+#pragma unroll
+    for (int k = 0; k < KS; ++k) ldsm_x4(base + k * 32, a[k][0], a[k][1], a[k][2], a[k][3]);
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int u = 0; u < U; ++u) mma_pure(s[u], a[k][0], a[k][1], a[k][2], a[k][3], qf[u][k][0], qf[u][k][1]);
+    float* dst = sc + buf * s_stage;
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) s[u][e] = cap_one(s[u][e], cap_in, cap_c);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (s_off[u][e] >= 0) {
+          dst[s_off[u][e]] = s[u][e];
+          dst[s_off[u][e] + 8 * SP] = s[u][2 + e];
+        }
+    }
+  };
+
+  // MASK: some key of the page is hidden from some query. MAX: only the maxima, into l.
+  auto mix = [&](int buf, int key0, auto masked, auto maxima) {
+    constexpr bool MASK = decltype(masked)::value, MAX = decltype(maxima)::value;
+    float acc[NT][HB][4];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int qq = min(gw + j * nwarps, 2 * p.qt - 1) >> 1;
+#pragma unroll
+      for (int h = 0; h < HB; ++h) {
+        acc[j][h][0] = acc[j][h][1] = ref[qq * HP + h * 16 + oct];
+        acc[j][h][2] = acc[j][h][3] = ref[qq * HP + h * 16 + 8 + oct];
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < HB; ++e) {
+      uint32_t bf[NT][3][2];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const float* src = sc + buf * s_stage + mix_src[j] + e * 16;
+        const float2 x = *reinterpret_cast<const float2*>(src), y = *reinterpret_cast<const float2*>(src + 8);
+        split3(x.x, x.y, bf[j][0][0], bf[j][1][0], bf[j][2][0]);
+        split3(y.x, y.y, bf[j][0][1], bf[j][1][1], bf[j][2][1]);
+      }
+#pragma unroll
+      for (int h = 0; h < HB; ++h) {
+        uint32_t a0, a1, a2, a3;
+        ldsm_x4(talk_a + h * 16 * (HP + 8) * 2 + e * 32, a0, a1, a2, a3);
+#pragma unroll
+        for (int x = 2; x >= 0; --x)
+#pragma unroll
+          for (int j = 0; j < NT; ++j) mma_pure(acc[j][h], a0, a1, a2, a3, bf[j][x][0], bf[j][x][1]);
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int t = min(gw + j * nwarps, 2 * p.qt - 1), k0 = (t & 1) * 8;
+      if constexpr (MASK) {
+        const int pos = p0 + (t >> 1);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int key = key0 + k0 + quad * 2 + e;
+          const bool hide = key > pos || (p.window > 0 && pos - key >= p.window && key >= p.keep);
+#pragma unroll
+          for (int h = 0; h < HB; ++h) {
+            acc[j][h][e] = hide ? -INFINITY : acc[j][h][e];
+            acc[j][h][2 + e] = hide ? -INFINITY : acc[j][h][2 + e];
+          }
+        }
+      }
+#pragma unroll
+      for (int h = 0; h < HB; ++h) {
+        if constexpr (MAX) {
+          l[j][h][0] = fmaxf(l[j][h][0], fmaxf(acc[j][h][0], acc[j][h][1]));
+          l[j][h][1] = fmaxf(l[j][h][1], fmaxf(acc[j][h][2], acc[j][h][3]));
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[j][h][e] = ex2(acc[j][h][e]);
+          l[j][h][0] += acc[j][h][0] + acc[j][h][1];
+          l[j][h][1] += acc[j][h][2] + acc[j][h][3];
+        }
+      }
+    }
+    if constexpr (!MAX) {
+      uint8_t* dst = ps + buf * p_stage;
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int h = 0; h < HB; ++h)
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+            if (p_dst[j][h][e] >= 0) *reinterpret_cast<uint32_t*>(dst + p_dst[j][h][e]) = pack2(acc[j][h][2 * e], acc[j][h][2 * e + 1]);
+    }
+  };
+
+  // ---- pages. Iteration i: scores of page i + 1, mixing of page i, while the tensor cores sum up page i - 1; keys are fetched two pages ahead,
+  // values one. What an iteration writes was read before the barrier in front of it, or by the sums of page i - 2, which it waits for.
+  const uint32_t idesc = umma_idesc_bf16(D, lay.columns) | (1u << 15);  // A is MN-major
+  bool ok = true;
+  uint32_t phase = 0;                                                   // bit s: parity of the next wait on done[s]
+  auto sum_up = [&](int i) {                                            // one thread: O^T += V^T P^T of page i
+    tc_fence_after_sync();
+    for (int h = 0; h < p.G; ++h)
+      umma_f16(tmem + h * lay.columns, umma_desc_mn_rows(vs_a + (i & 1) * v_stage + h * (kPage * D * 2), 2048),
+               umma_desc_k_core(ps_a + (i & 1) * p_stage + h * lay.p_head), idesc, i > 0 ? 1u : 0u);
+    umma_commit(&done[i & 1]);
+  };
+  auto wait_sums = [&](int i) {
+    if (ok) ok = mbar_wait(&done[i & 1], (phase >> (i & 1)) & 1, p.status, 3);
+    phase ^= 1u << (i & 1);
+  };
+  auto page_at = [&](int i) { return bt[pages.at(min(i, n - 1))]; };
+  auto walk = [&](auto maxima) {
+    constexpr bool MAX = decltype(maxima)::value;
+    int pg0 = page_at(0), pg1 = page_at(1), pg2 = page_at(2);
+    load(p.k_cache, ks_a + k_dst, k_step, pg0);
+    load(p.k_cache, ks_a + k_stage + k_dst, k_step, pg1);
+    cp_async_commit();
+    cp_async_wait<0>();
+    __syncthreads();
+    score(0);
+    __syncthreads();
+    for (int i = 0; i < n; ++i) {
+      const int pg3 = page_at(i + 3), cur = i & 1, key0 = pages.at(i) * kPage;
+      const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+      if constexpr (!MAX) {
+        if (i > 0 && tid == 0) sum_up(i - 1);
+        __syncwarp();
+        if (i > 1) wait_sums(i - 2);
+        load(p.v_cache, vs_a + cur * v_stage + v_dst, v_step, pg0);
+      }
+      load(p.k_cache, ks_a + cur * k_stage + k_dst, k_step, pg2);
+      cp_async_commit();
+      if constexpr (MAX) {
+        score(cur ^ 1);
+        mix(cur, key0, std::true_type(), std::true_type());
+      } else if (gw < kTcWarps / 2) {
+        score(cur ^ 1);
+        if (mixes) {
+          if (inner) mix(cur, key0, std::false_type(), std::false_type());
+          else mix(cur, key0, std::true_type(), std::false_type());
+        }
+      } else {
+        if (mixes) {
+          if (inner) mix(cur, key0, std::false_type(), std::false_type());
+          else mix(cur, key0, std::true_type(), std::false_type());
+        }
+        score(cur ^ 1);
+      }
+      cp_async_wait<0>();
+      fence_proxy_async_smem();
+      tc_fence_before_sync();
+      __syncthreads();
+      pg0 = pg1;
+      pg1 = pg2;
+      pg2 = pg3;
+    }
+    if constexpr (!MAX) {
+      if (tid == 0) sum_up(n - 1);
+      __syncwarp();
+      if (n > 1) wait_sums(n - 2);
+      wait_sums(n - 1);
+      tc_fence_after_sync();
+    }
+  };
+  // the l of all threads, by keys of the two halves of a page
+  auto spread = [&](auto maxima) {
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+      const int t = min(gw + j * nwarps, 2 * p.qt - 1), qq = t >> 1;
+#pragma unroll
+      for (int h = 0; h < HB; ++h)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float v = l[j][h][e];
+#pragma unroll
+          for (int x = 1; x <= 2; x *= 2) {
+            const float w = __shfl_xor_sync(0xffffffffu, v, x);
+            v = decltype(maxima)::value ? fmaxf(v, w) : v + w;
+          }
+          if (quad == 0 && mixes) sums[(qq * HP + h * 16 + e * 8 + oct) * 2 + (t & 1)] = v;
+        }
+    }
+    __syncthreads();
+  };
+  auto reset = [&](float start) {
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int h = 0; h < HB; ++h) l[t][h][0] = l[t][h][1] = start;
+  };
+  for (int pass = 0;; ++pass) {
+    reset(0.f);
+    if (tid == 0) far_row = 0;
+    walk(std::false_type());
+    spread(std::false_type());
+    if (pass > 0) break;
+    for (int i = tid; i < nq * p.H; i += threads) {
+      const float2 v = *reinterpret_cast<const float2*>(sums + (i / p.H * HP + i % p.H) * 2);
+      if (!(v.x + v.y >= exp2f(-kFar) && v.x + v.y <= exp2f(kFar))) far_row = 1;
+    }
+    __syncthreads();
+    if (far_row == 0) break;
+    reset(-INFINITY);                                                   // c = the maximum of every row
+    walk(std::true_type());
+    spread(std::true_type());
+    for (int i = tid; i < p.qt * HP; i += threads) {
+      const float m = fmaxf(sums[i * 2], sums[i * 2 + 1]);
+      ref[i] = fabsf(m) < INFINITY ? -m : 0.f;
+    }
+    __syncthreads();
+  }
+
+  // ---- factor and place of every column, over the scores; then O^T, a lane per value dim
+  float* factor = sc;
+  int* place = reinterpret_cast<int*>(sc + p.G * lay.columns);
+  for (int i = tid; i < p.G * lay.columns; i += threads) {
+    const int c = i % lay.columns, cq = c / r, h = i / lay.columns * r + c % r;
+    float f = 0.f;
+    if (cq < nq) {
+      const float sum = sums[(cq * HP + h) * 2] + sums[(cq * HP + h) * 2 + 1];
+      // the sink, in units of the row's own sum
+      const float sink = p.sinks != nullptr ? fmaf(p.sinks[h], kLog2e, ref[cq * HP + h]) - __log2f(sum) : -INFINITY;
+      f = 1.f / (sum * (1.f + ex2(fminf(sink, 120.f))));
+    }
+    factor[i] = f;
+    place[i] = cq < nq ? (cq * p.H + h) * D : -1;
+  }
+  __syncthreads();
+  bf16* out = static_cast<bf16*>(p.out) + static_cast<size_t>(row0 + qi0) * p.H * D + (gw & 3) * 32 + lane;
+  for (int c0 = (gw >> 2) * 16; c0 < p.G * lay.columns; c0 += (nwarps >> 2) * 16) {
+    uint32_t v[16];
+    tmem_ld16(tmem + (static_cast<uint32_t>((gw & 3) * 32) << 16) + c0, v);
+    tmem_wait_ld();
+#pragma unroll
+    for (int c = 0; c < 16; ++c)
+      if (place[c0 + c] >= 0) out[place[c0 + c]] = __float2bfloat16(__uint_as_float(v[c]) * factor[c0 + c]);
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (gw == 0) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem, tcols);
+  }
+}
+
+static PromptPlan prompt_tc_plan(int H, int G, int dk, int dv, int rows, float softcap) {
+  PromptPlan best;
+  if (G <= 0 || H % G != 0 || H > 64 || dk != kTcHead || dv != kTcHead || softcap <= 0.f) return best;
+  for (int qt = 32; qt >= 2; qt /= 2) {
+    if (qt / 2 >= rows && qt > 2) continue;
+    PromptPlan t;
+    t.qt = qt;
+    t.octets = ((qt * (H / G) + 7) / 8 + kTcUnits - 1) / kTcUnits * kTcUnits;
+    t.warps = G * t.octets / kTcUnits;
+    t.blocks = H <= 16 ? 1 : H <= 32 ? 2 : 4;
+    t.per = (2 * qt + t.warps - 1) / t.warps;
+    const PromptTcLayout lay(H, G, qt, t.octets);
+    t.smem = lay.total + 1024;
+    // every thread keeps its row of a page from copy to copy: whole heads at a time; octets * 8 columns are the N of a product
+    if (t.warps > kTcWarps || t.warps % 8 != 0 || G * kPage * 16 % (t.warps * 32) != 0 || t.octets > 32 || t.per > (t.blocks == 4 ? 1 : 4 / t.blocks) ||
+        t.smem > kSmemLimit - 256 || lay.t.hp != 16 * t.blocks)
+      continue;
+    return t;
+  }
+  return best;
+}
+
+template <int HB, int NT>
+static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
+  static bool configured = false;
+  if (!configured) {
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
+    if (e != cudaSuccess) return e;
+    configured = true;
+  }
+  return launch_pdl(talking_prompt_tc_kernel<HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
+}
+static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
+  if (t.blocks == 1) return t.per <= 2 ? launch_prompt_tc<1, 2>(p, grid, t, stream) : launch_prompt_tc<1, 4>(p, grid, t, stream);
+  if (t.blocks == 2) return t.per <= 1 ? launch_prompt_tc<2, 1>(p, grid, t, stream) : launch_prompt_tc<2, 2>(p, grid, t, stream);
+  return launch_prompt_tc<4, 1>(p, grid, t, stream);
 }
 
 // ---------------------------------------------------------------------------------------------- CUDA cores
@@ -1070,20 +1505,24 @@ extern "C" int eredu_talking_fits(int H, int G, int dk, int dv, int rows) {
 extern "C" int eredu_talking_attention(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                                        const int* seq_lens, const int* cu_q, const void* talk, const float* sinks, int batch, int q_per_seq,
                                        int max_rows, int max_pages, int H, int G, int dk, int dv, int window, int keep, int splits,
-                                       float scale, float softcap, cudaStream_t stream) {
+                                       float scale, float softcap, int* status, cudaStream_t stream) {
   if (batch <= 0 || max_rows <= 0) return 0;
   if (window < 0 || keep < 0 || splits < 1 || splits > kMaxSplits || batch > 65535) return -1;
   const bool decode = cu_q == nullptr && max_rows <= kDecodeRows;
   TalkParams p = talk_params(q, k_cache, v_cache, out, block_table, seq_lens, cu_q, talk, sinks, q_per_seq, max_pages, H, G, dk, dv, window,
                              keep, scale, softcap);
-  const PromptPlan pp = decode ? PromptPlan() : prompt_plan(H, G, dk, dv, max_rows, softcap);
-  if (pp.qt > 0) {
-    p.qt = pp.qt;
-    p.octets = pp.octets;
-    const dim3 grid((max_rows + pp.qt - 1) / pp.qt, batch);
-    const cudaError_t e = dk == 64 ? launch_prompt<64>(p, grid, pp, stream) : launch_prompt<128>(p, grid, pp, stream);
-    eredu_count_launches(1);
-    return static_cast<int>(e);
+  p.status = status;
+  if (!decode) {
+    const bool wide = dk == kTcHead;
+    const PromptPlan t = wide ? prompt_tc_plan(H, G, dk, dv, max_rows, softcap) : prompt_plan(H, G, dk, dv, max_rows, softcap);
+    if (t.qt > 0) {
+      p.qt = t.qt;
+      p.octets = t.octets;
+      const dim3 grid((max_rows + t.qt - 1) / t.qt, batch);
+      const cudaError_t e = wide ? launch_prompt_tc(p, grid, t, stream) : launch_prompt(p, grid, t, stream);
+      eredu_count_launches(1);
+      return static_cast<int>(e);
+    }
   }
   const TalkPlan t = talk_plan(H, G, dk, dv, max_rows, decode);
   if (t.qt == 0) return -1;
