@@ -972,38 +972,47 @@ __device__ __forceinline__ uint64_t umma_desc_mn_rows(uint32_t smem_addr, uint32
          static_cast<uint64_t>(1) << 46 | static_cast<uint64_t>(2) << 61;
 }
 
-template <int HB, int NT>
-__global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(TalkParams p) {
+__device__ __forceinline__ void sts_f32(uint32_t addr, float v) { asm volatile("st.shared.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
+__device__ __forceinline__ void sts_u32(uint32_t addr, uint32_t v) { asm volatile("st.shared.u32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
+__device__ __forceinline__ float2 lds_f32x2(uint32_t addr) {
+  float2 v;
+  asm volatile("ld.shared.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(addr));
+  return v;
+}
+// Queries of a CTA: with HB blocks of 16 heads, 256 rows of a (query, head) pair.
+constexpr int tc_queries(int hb) { return 16 / hb; }
+
+// W warps, of which each takes NT products of the mix step; CP copies of 16 bytes per thread make up a page (0: any number).
+template <int HB, int W, int CP>
+__global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams p) {
   using bf16 = __nv_bfloat16;
-  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16;
-  constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4;
+  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16, QT = tc_queries(HB), THREADS = 32 * W;
+  constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4, S_STAGE = QT * SQ * 4, NT = 2 * QT > W ? 2 * QT / W : 1;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ int far_row;
   __shared__ uint32_t tmem_slot;
   __shared__ __align__(8) uint64_t done[2];       // sums of a page of this parity are complete
   pdl_launch_early();
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-  const PromptTcLayout lay(p.H, p.G, p.qt, p.octets);
-  const int tid = threadIdx.x, lane = tid & 31, quad = lane & 3, oct = lane >> 2, gw = tid >> 5, threads = blockDim.x, nwarps = threads >> 5;
-  const int b = blockIdx.y, r = p.H / p.G, columns = p.qt * r;
-  float* sc = reinterpret_cast<float*>(smem + lay.s_off);
-  uint8_t* ps = smem + lay.p_off;
+  uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
+  const PromptTcLayout lay(p.H, p.G, QT, p.octets);
+  const int tid = threadIdx.x, lane = tid & 31, quad = lane & 3, oct = lane >> 2, gw = tid >> 5;
+  const int b = blockIdx.y, r = p.H / p.G, columns = QT * r;
   float* ref = reinterpret_cast<float*>(smem + lay.ref_off);            // -c of every (query, head)
-  float* sums = reinterpret_cast<float*>(smem + lay.sum_off);           // [qt hp][2]
+  float* sums = reinterpret_cast<float*>(smem + lay.sum_off);           // [QT HP][2]
   bf16* talk_s = reinterpret_cast<bf16*>(smem + lay.total - lay.t.talk());
-  const int s_stage = lay.t.s_bytes / 4, p_stage = lay.p_bytes, k_stage = lay.t.k_bytes, v_stage = lay.v_bytes;
+  const int p_stage = lay.p_bytes, k_stage = lay.t.k_bytes, v_stage = lay.v_bytes;
 
-  for (int i = tid; i < lay.total / 16; i += threads) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < lay.total / 16; i += THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
-  for (int i = tid; i < p.H * p.H; i += threads) talk_s[i / p.H * (HP + 8) + i % p.H] = static_cast<const bf16*>(p.talk)[i];
+  for (int i = tid; i < p.H * p.H; i += THREADS) talk_s[i / p.H * (HP + 8) + i % p.H] = static_cast<const bf16*>(p.talk)[i];
 
   pdl_wait();
   pdl_launch_dependents();
   const int row0 = p.cu_q != nullptr ? p.cu_q[b] : b * p.q_per_seq;
   const int q_len = p.cu_q != nullptr ? p.cu_q[b + 1] - row0 : p.q_per_seq;
-  const int qi0 = blockIdx.x * p.qt;
+  const int qi0 = blockIdx.x * QT;
   if (qi0 >= q_len) return;
-  const int nq = min(p.qt, q_len - qi0);
+  const int nq = min(QT, q_len - qi0);
   const int p0 = p.seq_lens[b] - q_len + qi0, p1 = p0 + nq - 1;
   const TalkPages pages = talk_pages(p0, p1, p.window, p.keep);
   const int* bt = p.block_table + static_cast<size_t>(b) * p.max_pages;
@@ -1025,17 +1034,18 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem = tmem_slot;
+  const uint32_t base_a = smem_u32(smem), ks_a = base_a + lay.k_off, vs_a = base_a + lay.v_off, ps_a = base_a + lay.p_off, sc_a = base_a + lay.s_off;
 
-  // ---- the warp's columns: one key / value head, U octets side by side; columns beyond the last query are zeros that nobody reads
+  // ---- the warp's columns: one key / value head, U octets side by side; columns beyond the last query are zeros, their scores go into the
+  // gaps between rows of heads
   const int g = gw * U / p.octets, o0 = gw * U % p.octets;
-  uint32_t qf[U][KS][2];
-  int s_off[U][2];
+  uint32_t qf[U][KS][2], s_dst[U][2];
 #pragma unroll
   for (int u = 0; u < U; ++u) {
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int c = (o0 + u) * 8 + quad * 2 + e;
-      s_off[u][e] = c < columns ? c / r * SQ + g * r + c % r + oct * SP : -1;
+      s_dst[u][e] = sc_a + 4 * (oct * SP + (c < columns ? c / r * SQ + g * r + c % r : HP));
     }
     const int c = (o0 + u) * 8 + oct, cq = c / r;
     const bf16* src = static_cast<const bf16*>(p.q) + (static_cast<size_t>(row0 + qi0 + cq) * p.H + g * r + c % r) * D + quad * 2;
@@ -1044,40 +1054,47 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
 #pragma unroll
       for (int e = 0; e < 2; ++e) qf[u][k][e] = cq < nq ? *reinterpret_cast<const uint32_t*>(src + k * 16 + e * 8) : 0u;
   }
-  // ---- where the warp's products of the mix step read scores and leave probabilities
-  const bool mixes = gw < 2 * p.qt;
-  int mix_src[NT], p_dst[NT][HB][2];
+  // ---- where the warp's products of the mix step (eight keys of a query) read scores and leave probabilities; those of heads that do not
+  // exist go into the gaps between heads
+  const bool mixes = gw < 2 * QT;
+  const int k_half = (gw & 1) * 8;                                      // W is even: all products of a warp are of one half of the keys
+  uint32_t mix_src[NT], p_dst[NT][HB][2];
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
-    const int t = min(gw + j * nwarps, 2 * p.qt - 1), qq = t >> 1;
-    mix_src[j] = qq * SQ + ((t & 1) * 8 + oct) * SP + quad * 2;
+    const int qq = (gw + j * W) >> 1;
+    mix_src[j] = sc_a + 4 * (qq * SQ + (k_half + oct) * SP + quad * 2);
 #pragma unroll
     for (int h = 0; h < HB; ++h)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int head = h * 16 + e * 8 + oct, c = qq * r + head % r;
-        p_dst[j][h][e] = head < p.H ? head / r * lay.p_head + (c >> 3) * 256 + (t & 1) * 128 + (c & 7) * 16 + quad * 4 : -1;
+        p_dst[j][h][e] = ps_a + quad * 4 + (head < p.H ? head / r * lay.p_head + (c >> 3) * 256 + k_half * 16 + (c & 7) * 16 : lay.columns * 32);
       }
   }
-  const uint32_t ks_a = smem_u32(smem + lay.k_off), vs_a = smem_u32(smem + lay.v_off), ps_a = smem_u32(ps);
   const uint32_t k_addr = ks_a + (g * kPage + (lane & 15)) * PITCH + (lane >> 4) * 16;
   const uint32_t talk_a = smem_u32(talk_s) + (lane & 15) * (HP + 8) * 2 + (lane >> 4) * 16;
-  const float cap_c = p.softcap * kLog2e, cap_in = 2.f * kLog2e * p.scale / p.softcap;
+  const float cap_m2c = -2.f * p.softcap * kLog2e, cap_c = p.softcap * kLog2e, cap_in = 2.f * kLog2e * p.scale / p.softcap;
 
   // ---- asynchronous copies: a page's rows of all key / value heads lie in one piece; a thread's place in it is fixed
-  const int pieces = p.G * kPage * PIECES, copies = pieces / threads, row = tid / PIECES, chunk = tid % PIECES;
-  const uint32_t k_dst = row * PITCH + chunk * 16, k_step = threads / PIECES * PITCH;
-  const uint32_t v_dst = (row / kPage) * (kPage * D * 2) + (chunk >> 3) * 2048 + (row % kPage) * 128 + (((chunk & 7) ^ (row & 7)) << 4);
-  const uint32_t v_step = threads / PIECES * (D * 2);                   // whole heads: a thread keeps its row of a page
-  auto load = [&](const void* cache, uint32_t dst, uint32_t step, int page) {
-    const uint4* src = static_cast<const uint4*>(cache) + static_cast<size_t>(page) * pieces + tid;
-#pragma unroll 4
-    for (int i = 0; i < copies; ++i) {
-      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-      src += threads;
-      dst += step;
+  const int pieces = p.G * kPage * PIECES, copies = CP > 0 ? CP : pieces / THREADS, row = tid / PIECES, chunk = tid % PIECES;
+  const uint32_t k_dst = ks_a + row * PITCH + chunk * 16;
+  const uint32_t v_dst = vs_a + (row / kPage) * (kPage * D * 2) + (chunk >> 3) * 2048 + (row % kPage) * 128 + (((chunk & 7) ^ (row & 7)) << 4);
+  const uint4* k_src = static_cast<const uint4*>(p.k_cache) + tid;
+  const uint4* v_src = static_cast<const uint4*>(p.v_cache) + tid;
+  auto load = [&](const uint4* cache, uint32_t dst, auto step, int page) {
+    constexpr uint32_t STEP = decltype(step)::value;
+    const uint4* src = cache + static_cast<size_t>(static_cast<uint32_t>(page)) * static_cast<uint32_t>(pieces);
+    if constexpr (CP > 0) {
+#pragma unroll
+      for (int i = 0; i < CP; ++i)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * STEP), "l"(src + i * THREADS) : "memory");
+    } else {
+      for (int i = 0; i < copies; ++i)
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * STEP), "l"(src + i * THREADS) : "memory");
     }
   };
+  const std::integral_constant<uint32_t, THREADS / PIECES * PITCH> k_step;
+  const std::integral_constant<uint32_t, THREADS / PIECES * D * 2> v_step;   // whole heads: a thread keeps its row of a page
 
   float l[NT][HB][2];
   auto score = [&](int buf) {
@@ -1092,42 +1109,38 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
     for (int k = 0; k < KS; ++k)
 #pragma unroll
       for (int u = 0; u < U; ++u) mma_pure(s[u], a[k][0], a[k][1], a[k][2], a[k][3], qf[u][k][0], qf[u][k][1]);
-    float* dst = sc + buf * s_stage;
 #pragma unroll
     for (int u = 0; u < U; ++u)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[u][e] = cap_one(s[u][e], cap_in, cap_c);
+      for (int e = 0; e < 4; ++e) s[u][e] = fmaf(cap_m2c, rcp(1.f + ex2(s[u][e] * cap_in)), cap_c);
+    const uint32_t stage = buf * S_STAGE;
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
+    for (int u = 0; u < U; ++u)
 #pragma unroll
-      for (int e = 0; e < 2; ++e)
-        if (s_off[u][e] >= 0) {
-          dst[s_off[u][e]] = s[u][e];
-          dst[s_off[u][e] + 8 * SP] = s[u][2 + e];
-        }
-    }
+      for (int e = 0; e < 2; ++e) {
+        sts_f32(s_dst[u][e] + stage, s[u][e]);
+        sts_f32(s_dst[u][e] + stage + 32 * SP, s[u][2 + e]);
+      }
   };
 
-  // MASK: some key of the page is hidden from some query. MAX: only the maxima, into l.
-  auto mix = [&](int buf, int key0, auto masked, auto maxima) {
-    constexpr bool MASK = decltype(masked)::value, MAX = decltype(maxima)::value;
+  // MASK: some key of the page is hidden from some query. MAX: only the maxima, into l. REF: c is not zero.
+  auto mix = [&](int buf, int key0, auto masked, auto maxima, auto refs) {
+    constexpr bool MASK = decltype(masked)::value, MAX = decltype(maxima)::value, REF = decltype(refs)::value;
     float acc[NT][HB][4];
 #pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      const int qq = min(gw + j * nwarps, 2 * p.qt - 1) >> 1;
+    for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int h = 0; h < HB; ++h) {
-        acc[j][h][0] = acc[j][h][1] = ref[qq * HP + h * 16 + oct];
-        acc[j][h][2] = acc[j][h][3] = ref[qq * HP + h * 16 + 8 + oct];
+        acc[j][h][0] = acc[j][h][1] = REF ? ref[((gw + j * W) >> 1) * HP + h * 16 + oct] : 0.f;
+        acc[j][h][2] = acc[j][h][3] = REF ? ref[((gw + j * W) >> 1) * HP + h * 16 + 8 + oct] : 0.f;
       }
-    }
+    const uint32_t s_stage = buf * S_STAGE, stage = buf * p_stage;
 #pragma unroll
     for (int e = 0; e < HB; ++e) {
       uint32_t bf[NT][3][2];
 #pragma unroll
       for (int j = 0; j < NT; ++j) {
-        const float* src = sc + buf * s_stage + mix_src[j] + e * 16;
-        const float2 x = *reinterpret_cast<const float2*>(src), y = *reinterpret_cast<const float2*>(src + 8);
+        const float2 x = lds_f32x2(mix_src[j] + s_stage + e * 64), y = lds_f32x2(mix_src[j] + s_stage + e * 64 + 32);
         split3(x.x, x.y, bf[j][0][0], bf[j][1][0], bf[j][2][0]);
         split3(y.x, y.y, bf[j][0][1], bf[j][1][1], bf[j][2][1]);
       }
@@ -1143,12 +1156,11 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
     }
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
-      const int t = min(gw + j * nwarps, 2 * p.qt - 1), k0 = (t & 1) * 8;
       if constexpr (MASK) {
-        const int pos = p0 + (t >> 1);
+        const int pos = p0 + ((gw + j * W) >> 1);
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int key = key0 + k0 + quad * 2 + e;
+          const int key = key0 + k_half + quad * 2 + e;
           const bool hide = key > pos || (p.window > 0 && pos - key >= p.window && key >= p.keep);
 #pragma unroll
           for (int h = 0; h < HB; ++h) {
@@ -1171,14 +1183,12 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
       }
     }
     if constexpr (!MAX) {
-      uint8_t* dst = ps + buf * p_stage;
 #pragma unroll
       for (int j = 0; j < NT; ++j)
 #pragma unroll
         for (int h = 0; h < HB; ++h)
 #pragma unroll
-          for (int e = 0; e < 2; ++e)
-            if (p_dst[j][h][e] >= 0) *reinterpret_cast<uint32_t*>(dst + p_dst[j][h][e]) = pack2(acc[j][h][2 * e], acc[j][h][2 * e + 1]);
+          for (int e = 0; e < 2; ++e) sts_u32(p_dst[j][h][e] + stage, pack2(acc[j][h][2 * e], acc[j][h][2 * e + 1]));
     }
   };
 
@@ -1199,11 +1209,13 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
     phase ^= 1u << (i & 1);
   };
   auto page_at = [&](int i) { return bt[pages.at(min(i, n - 1))]; };
-  auto walk = [&](auto maxima) {
-    constexpr bool MAX = decltype(maxima)::value;
+  using Yes = std::true_type;
+  using No = std::false_type;
+  auto walk = [&](auto maxima, auto refs) {
+    constexpr bool MAX = decltype(maxima)::value, REF = decltype(refs)::value;
     int pg0 = page_at(0), pg1 = page_at(1), pg2 = page_at(2);
-    load(p.k_cache, ks_a + k_dst, k_step, pg0);
-    load(p.k_cache, ks_a + k_stage + k_dst, k_step, pg1);
+    load(k_src, k_dst, k_step, pg0);
+    load(k_src, k_dst + k_stage, k_step, pg1);
     cp_async_commit();
     cp_async_wait<0>();
     __syncthreads();
@@ -1212,27 +1224,27 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
     for (int i = 0; i < n; ++i) {
       const int pg3 = page_at(i + 3), cur = i & 1, key0 = pages.at(i) * kPage;
       const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+      load(k_src, k_dst + cur * k_stage, k_step, pg2);
       if constexpr (!MAX) {
         if (i > 0 && tid == 0) sum_up(i - 1);
         __syncwarp();
         if (i > 1) wait_sums(i - 2);
-        load(p.v_cache, vs_a + cur * v_stage + v_dst, v_step, pg0);
+        load(v_src, v_dst + cur * v_stage, v_step, pg0);
       }
-      load(p.k_cache, ks_a + cur * k_stage + k_dst, k_step, pg2);
       cp_async_commit();
-      if constexpr (MAX) {
+      if constexpr (MAX || REF) {
         score(cur ^ 1);
-        mix(cur, key0, std::true_type(), std::true_type());
-      } else if (gw < kTcWarps / 2) {
+        if (mixes) mix(cur, key0, Yes(), maxima, refs);
+      } else if (gw < W / 2) {
         score(cur ^ 1);
         if (mixes) {
-          if (inner) mix(cur, key0, std::false_type(), std::false_type());
-          else mix(cur, key0, std::true_type(), std::false_type());
+          if (inner) mix(cur, key0, No(), No(), No());
+          else mix(cur, key0, Yes(), No(), No());
         }
       } else {
         if (mixes) {
-          if (inner) mix(cur, key0, std::false_type(), std::false_type());
-          else mix(cur, key0, std::true_type(), std::false_type());
+          if (inner) mix(cur, key0, No(), No(), No());
+          else mix(cur, key0, Yes(), No(), No());
         }
         score(cur ^ 1);
       }
@@ -1255,8 +1267,7 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
   // the l of all threads, by keys of the two halves of a page
   auto spread = [&](auto maxima) {
 #pragma unroll
-    for (int j = 0; j < NT; ++j) {
-      const int t = min(gw + j * nwarps, 2 * p.qt - 1), qq = t >> 1;
+    for (int j = 0; j < NT; ++j)
 #pragma unroll
       for (int h = 0; h < HB; ++h)
 #pragma unroll
@@ -1267,9 +1278,8 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
             const float w = __shfl_xor_sync(0xffffffffu, v, x);
             v = decltype(maxima)::value ? fmaxf(v, w) : v + w;
           }
-          if (quad == 0 && mixes) sums[(qq * HP + h * 16 + e * 8 + oct) * 2 + (t & 1)] = v;
+          if (quad == 0 && mixes) sums[(((gw + j * W) >> 1) * HP + h * 16 + e * 8 + oct) * 2 + (gw & 1)] = v;
         }
-    }
     __syncthreads();
   };
   auto reset = [&](float start) {
@@ -1278,32 +1288,33 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
 #pragma unroll
       for (int h = 0; h < HB; ++h) l[t][h][0] = l[t][h][1] = start;
   };
-  for (int pass = 0;; ++pass) {
-    reset(0.f);
-    if (tid == 0) far_row = 0;
-    walk(std::false_type());
-    spread(std::false_type());
-    if (pass > 0) break;
-    for (int i = tid; i < nq * p.H; i += threads) {
-      const float2 v = *reinterpret_cast<const float2*>(sums + (i / p.H * HP + i % p.H) * 2);
-      if (!(v.x + v.y >= exp2f(-kFar) && v.x + v.y <= exp2f(kFar))) far_row = 1;
-    }
-    __syncthreads();
-    if (far_row == 0) break;
+  reset(0.f);
+  if (tid == 0) far_row = 0;
+  walk(No(), No());
+  spread(No());
+  for (int i = tid; i < nq * p.H; i += THREADS) {
+    const float2 v = *reinterpret_cast<const float2*>(sums + (i / p.H * HP + i % p.H) * 2);
+    if (!(v.x + v.y >= exp2f(-kFar) && v.x + v.y <= exp2f(kFar))) far_row = 1;
+  }
+  __syncthreads();
+  if (far_row != 0) {
     reset(-INFINITY);                                                   // c = the maximum of every row
-    walk(std::true_type());
-    spread(std::true_type());
-    for (int i = tid; i < p.qt * HP; i += threads) {
+    walk(Yes(), No());
+    spread(Yes());
+    for (int i = tid; i < QT * HP; i += THREADS) {
       const float m = fmaxf(sums[i * 2], sums[i * 2 + 1]);
       ref[i] = fabsf(m) < INFINITY ? -m : 0.f;
     }
     __syncthreads();
+    reset(0.f);
+    walk(No(), Yes());
+    spread(No());
   }
 
   // ---- factor and place of every column, over the scores; then O^T, a lane per value dim
-  float* factor = sc;
-  int* place = reinterpret_cast<int*>(sc + p.G * lay.columns);
-  for (int i = tid; i < p.G * lay.columns; i += threads) {
+  float* factor = reinterpret_cast<float*>(smem + lay.s_off);
+  int* place = reinterpret_cast<int*>(factor + p.G * lay.columns);
+  for (int i = tid; i < p.G * lay.columns; i += THREADS) {
     const int c = i % lay.columns, cq = c / r, h = i / lay.columns * r + c % r;
     float f = 0.f;
     if (cq < nq) {
@@ -1317,7 +1328,7 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
   }
   __syncthreads();
   bf16* out = static_cast<bf16*>(p.out) + static_cast<size_t>(row0 + qi0) * p.H * D + (gw & 3) * 32 + lane;
-  for (int c0 = (gw >> 2) * 16; c0 < p.G * lay.columns; c0 += (nwarps >> 2) * 16) {
+  for (int c0 = (gw >> 2) * 16; c0 < p.G * lay.columns; c0 += (W >> 2) * 16) {
     uint32_t v[16];
     tmem_ld16(tmem + (static_cast<uint32_t>((gw & 3) * 32) << 16) + c0, v);
     tmem_wait_ld();
@@ -1333,42 +1344,41 @@ __global__ void __launch_bounds__(32 * kTcWarps, 1) talking_prompt_tc_kernel(Tal
   }
 }
 
-static PromptPlan prompt_tc_plan(int H, int G, int dk, int dv, int rows, float softcap) {
-  PromptPlan best;
-  if (G <= 0 || H % G != 0 || H > 64 || dk != kTcHead || dv != kTcHead || softcap <= 0.f) return best;
-  for (int qt = 32; qt >= 2; qt /= 2) {
-    if (qt / 2 >= rows && qt > 2) continue;
-    PromptPlan t;
+static PromptPlan prompt_tc_plan(int H, int G, int dk, int dv, float softcap) {
+  PromptPlan t;
+  if (G <= 0 || H % G != 0 || H > 64 || dk != kTcHead || dv != kTcHead || softcap <= 0.f) return t;
+  t.blocks = H <= 16 ? 1 : H <= 32 ? 2 : 4;
+  const int qt = tc_queries(t.blocks);
+  t.octets = ((qt * (H / G) + 7) / 8 + kTcUnits - 1) / kTcUnits * kTcUnits;
+  t.warps = G * t.octets / kTcUnits;
+  const PromptTcLayout lay(H, G, qt, t.octets);
+  t.smem = lay.total + 1024;
+  // every thread keeps its row of a page from copy to copy: whole heads at a time; octets * 8 columns are the N of a product
+  if ((t.warps == 8 || t.warps == 16) && G * kPage * 16 % (t.warps * 32) == 0 && t.octets <= 32 && lay.t.hp == 16 * t.blocks &&
+      t.smem <= kSmemLimit - 256)
     t.qt = qt;
-    t.octets = ((qt * (H / G) + 7) / 8 + kTcUnits - 1) / kTcUnits * kTcUnits;
-    t.warps = G * t.octets / kTcUnits;
-    t.blocks = H <= 16 ? 1 : H <= 32 ? 2 : 4;
-    t.per = (2 * qt + t.warps - 1) / t.warps;
-    const PromptTcLayout lay(H, G, qt, t.octets);
-    t.smem = lay.total + 1024;
-    // every thread keeps its row of a page from copy to copy: whole heads at a time; octets * 8 columns are the N of a product
-    if (t.warps > kTcWarps || t.warps % 8 != 0 || G * kPage * 16 % (t.warps * 32) != 0 || t.octets > 32 || t.per > (t.blocks == 4 ? 1 : 4 / t.blocks) ||
-        t.smem > kSmemLimit - 256 || lay.t.hp != 16 * t.blocks)
-      continue;
-    return t;
-  }
-  return best;
+  return t;
 }
 
-template <int HB, int NT>
+template <int HB, int W, int CP>
 static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, W, CP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_tc_kernel<HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
+  return launch_pdl(talking_prompt_tc_kernel<HB, W, CP>, grid, dim3(W * 32), t.smem, stream, p);
+}
+template <int HB>
+static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
+  const int copies = p.G * 8 / t.warps;
+  if (t.warps == 8) return launch_prompt_tc<HB, 8, 0>(p, grid, t, stream);
+  return copies == 2 ? launch_prompt_tc<HB, 16, 2>(p, grid, t, stream)
+                     : copies == 4 ? launch_prompt_tc<HB, 16, 4>(p, grid, t, stream) : launch_prompt_tc<HB, 16, 0>(p, grid, t, stream);
 }
 static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
-  if (t.blocks == 1) return t.per <= 2 ? launch_prompt_tc<1, 2>(p, grid, t, stream) : launch_prompt_tc<1, 4>(p, grid, t, stream);
-  if (t.blocks == 2) return t.per <= 1 ? launch_prompt_tc<2, 1>(p, grid, t, stream) : launch_prompt_tc<2, 2>(p, grid, t, stream);
-  return launch_prompt_tc<4, 1>(p, grid, t, stream);
+  return t.blocks == 1 ? launch_prompt_tc<1>(p, grid, t, stream) : t.blocks == 2 ? launch_prompt_tc<2>(p, grid, t, stream) : launch_prompt_tc<4>(p, grid, t, stream);
 }
 
 // ---------------------------------------------------------------------------------------------- CUDA cores
@@ -1514,7 +1524,7 @@ extern "C" int eredu_talking_attention(const void* q, const void* k_cache, const
   p.status = status;
   if (!decode) {
     const bool wide = dk == kTcHead;
-    const PromptPlan t = wide ? prompt_tc_plan(H, G, dk, dv, max_rows, softcap) : prompt_plan(H, G, dk, dv, max_rows, softcap);
+    const PromptPlan t = wide ? prompt_tc_plan(H, G, dk, dv, softcap) : prompt_plan(H, G, dk, dv, max_rows, softcap);
     if (t.qt > 0) {
       p.qt = t.qt;
       p.octets = t.octets;
