@@ -23,6 +23,7 @@
 #include "../common/launch_count.h"
 #include "../common/mma.cuh"
 #include "../common/ptx.cuh"
+#include "../common/tma_host.h"
 
 namespace eredu {
 
@@ -939,21 +940,22 @@ static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPla
 // ---------------------------------------------------------------------------------------------- prompts, head size 128
 // The same steps with the sums on tcgen05: O^T[value dim, column] of a key / value head lies in tensor memory, one product of 128 value dims x
 // its columns x 16 keys a page, V as it comes (swizzled rows of keys) and P as the mix step leaves it (core matrices of 8 columns x 8 keys).
-constexpr int kTcHead = 128, kTcUnits = 2, kTcWarps = 16;
+constexpr int kTcHead = 128, kTcUnits = 2;
 
 struct PromptTcLayout {
   TalkLayout t;
   int columns;                            // of a key / value head, whole octets
-  int p_head, p_bytes, v_bytes;           // probabilities of a head (64 bytes apart from whole rows of banks), of a page; values of a page
+  int p_head, p_bytes, kv_bytes, half;    // probabilities of a head (64 bytes apart from whole rows of banks), of a page; keys of a page, 64 dims of them
   int v_off, k_off, s_off, p_off, ref_off, sum_off, total;
   __host__ __device__ __forceinline__ PromptTcLayout(int H, int G, int qt, int octets) : t(H, G, kTcHead, kTcHead, qt) {
     columns = octets * 8;
     p_head = columns * 32 + 64;
     p_bytes = G * p_head;
-    v_bytes = G * kPage * kTcHead * 2;
+    half = G * kPage * 128;
+    kv_bytes = 2 * half;
     v_off = 0;                            // 1024-byte aligned
-    k_off = 2 * v_bytes;
-    s_off = k_off + 2 * t.k_bytes;
+    k_off = 2 * kv_bytes;
+    s_off = k_off + 2 * kv_bytes;
     p_off = s_off + 2 * t.s_bytes;
     ref_off = p_off + 2 * p_bytes;
     sum_off = ref_off + qt * t.hp * 4;
@@ -982,16 +984,17 @@ __device__ __forceinline__ float2 lds_f32x2(uint32_t addr) {
 // Queries of a CTA: with HB blocks of 16 heads, 256 rows of a (query, head) pair.
 constexpr int tc_queries(int hb) { return 16 / hb; }
 
-// W warps, of which each takes NT products of the mix step; CP copies of 16 bytes per thread make up a page (0: any number).
-template <int HB, int W, int CP>
-__global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams p) {
+// W warps, of which each takes NT products of the mix step, and one that starts the copies and the sums. tm_k, tm_v: the caches as rows of 128, boxes of 64 columns and a page's rows.
+template <int HB, int W>
+__global__ void __launch_bounds__(32 * (W + 1), 1)
+talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, TalkParams p) {
   using bf16 = __nv_bfloat16;
-  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16, QT = tc_queries(HB), THREADS = 32 * W;
+  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, QT = tc_queries(HB), THREADS = 32 * (W + 1);
   constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4, S_STAGE = QT * SQ * 4, NT = 2 * QT > W ? 2 * QT / W : 1;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ int far_row;
   __shared__ uint32_t tmem_slot;
-  __shared__ __align__(8) uint64_t done[2];       // sums of a page of this parity are complete
+  __shared__ __align__(8) uint64_t k_full[2], v_full[2], done[2];       // of a page of this parity: keys, values are there, its sums complete
   pdl_launch_early();
   uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
   const PromptTcLayout lay(p.H, p.G, QT, p.octets);
@@ -1000,9 +1003,9 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
   float* ref = reinterpret_cast<float*>(smem + lay.ref_off);            // -c of every (query, head)
   float* sums = reinterpret_cast<float*>(smem + lay.sum_off);           // [QT HP][2]
   bf16* talk_s = reinterpret_cast<bf16*>(smem + lay.total - lay.t.talk());
-  const int p_stage = lay.p_bytes, k_stage = lay.t.k_bytes, v_stage = lay.v_bytes;
+  const int p_stage = lay.p_bytes, kv_stage = lay.kv_bytes;
 
-  for (int i = tid; i < lay.total / 16; i += THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = lay.s_off / 16 + tid; i < lay.total / 16; i += THREADS) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);
   __syncthreads();
   for (int i = tid; i < p.H * p.H; i += THREADS) talk_s[i / p.H * (HP + 8) + i % p.H] = static_cast<const bf16*>(p.talk)[i];
 
@@ -1026,9 +1029,14 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
     tmem_relinquish();
   }
   if (tid == 32) {
-    mbar_init(&done[0], 1);
-    mbar_init(&done[1], 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&v_full[i], 1);
+      mbar_init(&done[i], 1);
+    }
     fence_mbar_init();
+    tma_prefetch_desc(&tm_k);
+    tma_prefetch_desc(&tm_v);
   }
   tc_fence_before_sync();
   __syncthreads();
@@ -1038,7 +1046,8 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
 
   // ---- the warp's columns: one key / value head, U octets side by side; columns beyond the last query are zeros, their scores go into the
   // gaps between rows of heads
-  const int g = gw * U / p.octets, o0 = gw * U % p.octets;
+  const bool works = gw < W;
+  const int g = works ? gw * U / p.octets : 0, o0 = gw * U % p.octets;
   uint32_t qf[U][KS][2], s_dst[U][2];
 #pragma unroll
   for (int u = 0; u < U; ++u) {
@@ -1056,7 +1065,7 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
   }
   // ---- where the warp's products of the mix step (eight keys of a query) read scores and leave probabilities; those of heads that do not
   // exist go into the gaps between heads
-  const bool mixes = gw < 2 * QT;
+  const bool mixes = works && gw < 2 * QT;
   const int k_half = (gw & 1) * 8;                                      // W is even: all products of a warp are of one half of the keys
   uint32_t mix_src[NT], p_dst[NT][HB][2];
 #pragma unroll
@@ -1071,40 +1080,20 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
         p_dst[j][h][e] = ps_a + quad * 4 + (head < p.H ? head / r * lay.p_head + (c >> 3) * 256 + k_half * 16 + (c & 7) * 16 : lay.columns * 32);
       }
   }
-  const uint32_t k_addr = ks_a + (g * kPage + (lane & 15)) * PITCH + (lane >> 4) * 16;
+  // row of a key fragment; the 16-byte piece of a step is found by an exclusive or (128-byte swizzle)
+  const uint32_t k_addr = ks_a + (g * kPage + (lane & 15)) * 128 + (((lane >> 4) ^ (lane & 7)) << 4);
   const uint32_t talk_a = smem_u32(talk_s) + (lane & 15) * (HP + 8) * 2 + (lane >> 4) * 16;
   const float cap_m2c = -2.f * p.softcap * kLog2e, cap_c = p.softcap * kLog2e, cap_in = 2.f * kLog2e * p.scale / p.softcap;
-
-  // ---- asynchronous copies: a page's rows of all key / value heads lie in one piece; a thread's place in it is fixed
-  const int pieces = p.G * kPage * PIECES, copies = CP > 0 ? CP : pieces / THREADS, row = tid / PIECES, chunk = tid % PIECES;
-  const uint32_t k_dst = ks_a + row * PITCH + chunk * 16;
-  const uint32_t v_dst = vs_a + (row / kPage) * (kPage * D * 2) + (chunk >> 3) * 2048 + (row % kPage) * 128 + (((chunk & 7) ^ (row & 7)) << 4);
-  const uint4* k_src = static_cast<const uint4*>(p.k_cache) + tid;
-  const uint4* v_src = static_cast<const uint4*>(p.v_cache) + tid;
-  auto load = [&](const uint4* cache, uint32_t dst, auto step, int page) {
-    constexpr uint32_t STEP = decltype(step)::value;
-    const uint4* src = cache + static_cast<size_t>(static_cast<uint32_t>(page)) * static_cast<uint32_t>(pieces);
-    if constexpr (CP > 0) {
-#pragma unroll
-      for (int i = 0; i < CP; ++i)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * STEP), "l"(src + i * THREADS) : "memory");
-    } else {
-      for (int i = 0; i < copies; ++i)
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i * STEP), "l"(src + i * THREADS) : "memory");
-    }
-  };
-  const std::integral_constant<uint32_t, THREADS / PIECES * PITCH> k_step;
-  const std::integral_constant<uint32_t, THREADS / PIECES * D * 2> v_step;   // whole heads: a thread keeps its row of a page
 
   float l[NT][HB][2];
   auto score = [&](int buf) {
     float s[U][4];
 #pragma unroll
     for (int u = 0; u < U; ++u) s[u][0] = s[u][1] = s[u][2] = s[u][3] = 0.f;
-    const uint32_t base = k_addr + buf * k_stage;
+    const uint32_t base = k_addr + buf * kv_stage;
     uint32_t a[KS][4];
 #pragma unroll
-    for (int k = 0; k < KS; ++k) ldsm_x4(base + k * 32, a[k][0], a[k][1], a[k][2], a[k][3]);
+    for (int k = 0; k < KS; ++k) ldsm_x4((base + (k >> 2) * lay.half) ^ ((k & 3) << 5), a[k][0], a[k][1], a[k][2], a[k][3]);
 #pragma unroll
     for (int k = 0; k < KS; ++k)
 #pragma unroll
@@ -1193,74 +1182,100 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
   };
 
   // ---- pages. Iteration i: scores of page i + 1, mixing of page i, while the tensor cores sum up page i - 1; keys are fetched two pages ahead,
-  // values one. What an iteration writes was read before the barrier in front of it, or by the sums of page i - 2, which it waits for.
+  // values one. What an iteration writes was read before the barrier in front of it, or by the sums of page i - 2, which it waits for. One thread
+  // of the last warp starts the copies and the sums.
   const uint32_t idesc = umma_idesc_bf16(D, lay.columns) | (1u << 15);  // A is MN-major
   bool ok = true;
-  uint32_t phase = 0;                                                   // bit s: parity of the next wait on done[s]
-  auto sum_up = [&](int i) {                                            // one thread: O^T += V^T P^T of page i
+  uint32_t phase = 0;                                                   // parities of the next waits: bits 0, 1 done, 2, 3 k_full, 4, 5 v_full
+  auto wait_for = [&](uint64_t* bar, int bit, int code) {
+    if (ok) ok = mbar_wait(bar, (phase >> bit) & 1, p.status, code);
+    phase ^= 1u << bit;
+  };
+  auto wait_sums = [&](int i) { wait_for(&done[i & 1], i & 1, 3); };
+  auto page_row = [&](int i) { return bt[pages.at(min(i, n - 1))] * (p.G * kPage); };
+  auto load = [&](const CUtensorMap* map, uint64_t* bar, int off, int i, int page_row) {
+    uint8_t* dst = smem + off + (i & 1) * kv_stage;
+    mbar_arrive_expect_tx(&bar[i & 1], kv_stage);
+    tma_load_2d(dst, map, 0, page_row, &bar[i & 1]);
+    tma_load_2d(dst + lay.half, map, 64, page_row, &bar[i & 1]);
+  };
+  auto sum_up = [&](int i) {                                            // O^T += V^T P^T of page i
+    wait_for(&v_full[i & 1], 4 + (i & 1), 1);
     tc_fence_after_sync();
     for (int h = 0; h < p.G; ++h)
-      umma_f16(tmem + h * lay.columns, umma_desc_mn_rows(vs_a + (i & 1) * v_stage + h * (kPage * D * 2), 2048),
+      umma_f16(tmem + h * lay.columns, umma_desc_mn_rows(vs_a + (i & 1) * kv_stage + h * (kPage * 128), lay.half),
                umma_desc_k_core(ps_a + (i & 1) * p_stage + h * lay.p_head), idesc, i > 0 ? 1u : 0u);
     umma_commit(&done[i & 1]);
   };
-  auto wait_sums = [&](int i) {
-    if (ok) ok = mbar_wait(&done[i & 1], (phase >> (i & 1)) & 1, p.status, 3);
-    phase ^= 1u << (i & 1);
-  };
-  auto page_at = [&](int i) { return bt[pages.at(min(i, n - 1))]; };
   using Yes = std::true_type;
   using No = std::false_type;
   auto walk = [&](auto maxima, auto refs) {
     constexpr bool MAX = decltype(maxima)::value, REF = decltype(refs)::value;
-    int pg0 = page_at(0), pg1 = page_at(1), pg2 = page_at(2);
-    load(k_src, k_dst, k_step, pg0);
-    load(k_src, k_dst + k_stage, k_step, pg1);
-    cp_async_commit();
-    cp_async_wait<0>();
-    __syncthreads();
-    score(0);
+    auto score_at = [&](int i) {
+      if (i >= n) return;
+      wait_for(&k_full[i & 1], 2 + (i & 1), 1);
+      score(i & 1);
+    };
+    int at0 = 0, at1 = 0, at2 = 0;                                      // rows of pages i, i + 1, i + 2
+    if (works) {
+      score_at(0);
+    } else if (lane == 0) {
+      at0 = page_row(0);
+      at1 = page_row(1);
+      at2 = page_row(2);
+      load(&tm_k, k_full, lay.k_off, 0, at0);
+      if (n > 1) load(&tm_k, k_full, lay.k_off, 1, at1);
+      if (!MAX) load(&tm_v, v_full, lay.v_off, 0, at0);
+    }
     __syncthreads();
     for (int i = 0; i < n; ++i) {
-      const int pg3 = page_at(i + 3), cur = i & 1, key0 = pages.at(i) * kPage;
-      const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
-      load(k_src, k_dst + cur * k_stage, k_step, pg2);
-      if constexpr (!MAX) {
-        if (i > 0 && tid == 0) sum_up(i - 1);
-        __syncwarp();
-        if (i > 1) wait_sums(i - 2);
-        load(v_src, v_dst + cur * v_stage, v_step, pg0);
-      }
-      cp_async_commit();
-      if constexpr (MAX || REF) {
-        score(cur ^ 1);
-        if (mixes) mix(cur, key0, Yes(), maxima, refs);
-      } else if (gw < W / 2) {
-        score(cur ^ 1);
-        if (mixes) {
-          if (inner) mix(cur, key0, No(), No(), No());
-          else mix(cur, key0, Yes(), No(), No());
+      if (works) {
+        const int cur = i & 1, key0 = pages.at(i) * kPage;
+        const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+        if constexpr (MAX || REF) {
+          score_at(i + 1);
+          if (!MAX && i > 1) wait_sums(i - 2);
+          if (mixes) mix(cur, key0, Yes(), maxima, refs);
+        } else if (gw < W / 2) {
+          score_at(i + 1);
+          if (i > 1) wait_sums(i - 2);
+          if (mixes) {
+            if (inner) mix(cur, key0, No(), No(), No());
+            else mix(cur, key0, Yes(), No(), No());
+          }
+        } else {
+          if (i > 1) wait_sums(i - 2);
+          if (mixes) {
+            if (inner) mix(cur, key0, No(), No(), No());
+            else mix(cur, key0, Yes(), No(), No());
+          }
+          score_at(i + 1);
         }
-      } else {
-        if (mixes) {
-          if (inner) mix(cur, key0, No(), No(), No());
-          else mix(cur, key0, Yes(), No(), No());
+        fence_proxy_async_smem();
+      } else if (lane == 0) {
+        const int at3 = page_row(i + 3);
+        if (i + 2 < n) load(&tm_k, k_full, lay.k_off, i + 2, at2);
+        if (!MAX && i > 0) {
+          sum_up(i - 1);
+          if (i > 1) wait_sums(i - 2);
+          load(&tm_v, v_full, lay.v_off, i, at0);
         }
-        score(cur ^ 1);
+        at0 = at1;
+        at1 = at2;
+        at2 = at3;
       }
-      cp_async_wait<0>();
-      fence_proxy_async_smem();
+      __syncwarp();
       tc_fence_before_sync();
       __syncthreads();
-      pg0 = pg1;
-      pg1 = pg2;
-      pg2 = pg3;
     }
     if constexpr (!MAX) {
-      if (tid == 0) sum_up(n - 1);
+      if (gw == W && lane == 0) sum_up(n - 1);
       __syncwarp();
-      if (n > 1) wait_sums(n - 2);
-      wait_sums(n - 1);
+      if (gw < W || lane == 0) {
+        if (n > 1) wait_sums(n - 2);
+        wait_sums(n - 1);
+      }
+      __syncwarp();
       tc_fence_after_sync();
     }
   };
@@ -1328,7 +1343,7 @@ __global__ void __launch_bounds__(32 * W, 1) talking_prompt_tc_kernel(TalkParams
   }
   __syncthreads();
   bf16* out = static_cast<bf16*>(p.out) + static_cast<size_t>(row0 + qi0) * p.H * D + (gw & 3) * 32 + lane;
-  for (int c0 = (gw >> 2) * 16; c0 < p.G * lay.columns; c0 += (W >> 2) * 16) {
+  for (int c0 = works ? (gw >> 2) * 16 : 1 << 20; c0 < p.G * lay.columns; c0 += (W >> 2) * 16) {
     uint32_t v[16];
     tmem_ld16(tmem + (static_cast<uint32_t>((gw & 3) * 32) << 16) + c0, v);
     tmem_wait_ld();
@@ -1353,32 +1368,36 @@ static PromptPlan prompt_tc_plan(int H, int G, int dk, int dv, float softcap) {
   t.warps = G * t.octets / kTcUnits;
   const PromptTcLayout lay(H, G, qt, t.octets);
   t.smem = lay.total + 1024;
-  // every thread keeps its row of a page from copy to copy: whole heads at a time; octets * 8 columns are the N of a product
-  if ((t.warps == 8 || t.warps == 16) && G * kPage * 16 % (t.warps * 32) == 0 && t.octets <= 32 && lay.t.hp == 16 * t.blocks &&
-      t.smem <= kSmemLimit - 256)
-    t.qt = qt;
+  // octets * 8 columns are the N of a product; a page's rows are one box
+  if ((t.warps == 8 || t.warps == 16) && t.octets <= 32 && G * kPage <= 256 && lay.t.hp == 16 * t.blocks && t.smem <= kSmemLimit - 256) t.qt = qt;
   return t;
 }
 
-template <int HB, int W, int CP>
-static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
+template <int HB, int W>
+static cudaError_t launch_prompt_tc(const CUtensorMap& tm_k, const CUtensorMap& tm_v, const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, W, CP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_tc_kernel<HB, W, CP>, grid, dim3(W * 32), t.smem, stream, p);
+  return launch_pdl(talking_prompt_tc_kernel<HB, W>, grid, dim3((W + 1) * 32), t.smem, stream, tm_k, tm_v, p);
 }
-template <int HB>
-static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
-  const int copies = p.G * 8 / t.warps;
-  if (t.warps == 8) return launch_prompt_tc<HB, 8, 0>(p, grid, t, stream);
-  return copies == 2 ? launch_prompt_tc<HB, 16, 2>(p, grid, t, stream)
-                     : copies == 4 ? launch_prompt_tc<HB, 16, 4>(p, grid, t, stream) : launch_prompt_tc<HB, 16, 0>(p, grid, t, stream);
-}
-static cudaError_t launch_prompt_tc(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
-  return t.blocks == 1 ? launch_prompt_tc<1>(p, grid, t, stream) : t.blocks == 2 ? launch_prompt_tc<2>(p, grid, t, stream) : launch_prompt_tc<4>(p, grid, t, stream);
+// A cudaError_t, or a negative number where a tensor map cannot be made.
+static int launch_prompt_tc(const TalkParams& p, int pages, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
+  CUtensorMap tm_k, tm_v;
+  const uint64_t rows = static_cast<uint64_t>(pages) * p.G * kPage;
+  int r = make_tma_2d(&tm_k, p.k_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, kTcHead, kTcHead, p.G * kPage, 64);
+  if (r != 0) return -100 - r;
+  r = make_tma_2d(&tm_v, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, kTcHead, kTcHead, p.G * kPage, 64);
+  if (r != 0) return -200 - r;
+  cudaError_t e;
+#define ER_TC(HB_) t.warps == 8 ? launch_prompt_tc<HB_, 8>(tm_k, tm_v, p, grid, t, stream) : launch_prompt_tc<HB_, 16>(tm_k, tm_v, p, grid, t, stream)
+  if (t.blocks == 1) e = ER_TC(1);
+  else if (t.blocks == 2) e = ER_TC(2);
+  else e = ER_TC(4);
+#undef ER_TC
+  return static_cast<int>(e);
 }
 
 // ---------------------------------------------------------------------------------------------- CUDA cores
@@ -1514,7 +1533,7 @@ extern "C" int eredu_talking_fits(int H, int G, int dk, int dv, int rows) {
 // `keep`. splits <= 8: CTAs that share a sequence's keys in a decode step (cu_q null).
 extern "C" int eredu_talking_attention(const void* q, const void* k_cache, const void* v_cache, void* out, const int* block_table,
                                        const int* seq_lens, const int* cu_q, const void* talk, const float* sinks, int batch, int q_per_seq,
-                                       int max_rows, int max_pages, int H, int G, int dk, int dv, int window, int keep, int splits,
+                                       int max_rows, int max_pages, int H, int G, int dk, int dv, int window, int keep, int splits, int pages,
                                        float scale, float softcap, int* status, cudaStream_t stream) {
   if (batch <= 0 || max_rows <= 0) return 0;
   if (window < 0 || keep < 0 || splits < 1 || splits > kMaxSplits || batch > 65535) return -1;
@@ -1529,9 +1548,9 @@ extern "C" int eredu_talking_attention(const void* q, const void* k_cache, const
       p.qt = t.qt;
       p.octets = t.octets;
       const dim3 grid((max_rows + t.qt - 1) / t.qt, batch);
-      const cudaError_t e = wide ? launch_prompt_tc(p, grid, t, stream) : launch_prompt(p, grid, t, stream);
+      const int e = wide ? launch_prompt_tc(p, pages, grid, t, stream) : static_cast<int>(launch_prompt(p, grid, t, stream));
       eredu_count_launches(1);
-      return static_cast<int>(e);
+      return e;
     }
   }
   const TalkPlan t = talk_plan(H, G, dk, dv, max_rows, decode);

@@ -8,7 +8,7 @@ from . import native
 from .core import CLUSTER_SPLITS, PAGE, _gather_kv, _sm_count, _tensor_core_dims
 from .native import F, I, P, check, lib, ptr, status_word, stream_ptr
 
-native.register("eredu_talking_attention", I, [P] * 9 + [I] * 11 + [F, F, P, P])
+native.register("eredu_talking_attention", I, [P] * 9 + [I] * 12 + [F, F, P, P])
 native.register("eredu_talking_attention_simt", I, [P] * 9 + [I] * 11 + [F, F, P])
 native.register("eredu_talking_fits", I, [I] * 5)
 
@@ -57,7 +57,7 @@ def talking_attention(q, k_cache, v_cache, batch, talk, scale: float, softcap: f
             ptr(talk), ptr(sinks), B, batch.q_per_seq, rows, batch.block_table.stride(0), H, G, dk, dv, window, keep)
     if _tensor_core_dims(q, k_cache, v_cache) and lib().eredu_talking_fits(H, G, dk, dv, rows):
         splits = 1 if batch.is_prefill else decode_splits(B, batch.max_kv_len, window, keep, _sm_count(q.device))
-        check(lib().eredu_talking_attention(*args, splits, scale, softcap, ptr(status_word(q.device)), stream_ptr(q.device)), "eredu_talking_attention")
+        check(lib().eredu_talking_attention(*args, splits, k_cache.shape[0], scale, softcap, ptr(status_word(q.device)), stream_ptr(q.device)), "eredu_talking_attention")
         return out
     check(lib().eredu_talking_attention_simt(*args, 1 if q.dtype == torch.float32 else 0, scale, softcap, stream_ptr(q.device)),
           "eredu_talking_attention_simt")
