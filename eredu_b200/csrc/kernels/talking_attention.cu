@@ -976,6 +976,9 @@ __device__ __forceinline__ uint64_t umma_desc_mn_rows(uint32_t smem_addr, uint32
 
 __device__ __forceinline__ void sts_f32(uint32_t addr, float v) { asm volatile("st.shared.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
 __device__ __forceinline__ void sts_u32(uint32_t addr, uint32_t v) { asm volatile("st.shared.u32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
+__device__ __forceinline__ void sts_f32x2(uint32_t addr, float x, float y) {
+  asm volatile("st.shared.v2.f32 [%0], {%1, %2};" ::"r"(addr), "f"(x), "f"(y) : "memory");
+}
 __device__ __forceinline__ float2 lds_f32x2(uint32_t addr) {
   float2 v;
   asm volatile("ld.shared.v2.f32 {%0, %1}, [%2];" : "=f"(v.x), "=f"(v.y) : "r"(addr));
@@ -1049,6 +1052,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   const bool works = gw < W;
   const int g = works ? gw * U / p.octets : 0, o0 = gw * U % p.octets;
   uint32_t qf[U][KS][2], s_dst[U][2];
+  const bool pairs = r % 2 == 0;
 #pragma unroll
   for (int u = 0; u < U; ++u) {
 #pragma unroll
@@ -1103,13 +1107,21 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
 #pragma unroll
       for (int e = 0; e < 4; ++e) s[u][e] = fmaf(cap_m2c, rcp(1.f + ex2(s[u][e] * cap_in)), cap_c);
     const uint32_t stage = buf * S_STAGE;
+    if (pairs) {                                                        // two columns are neighbouring heads of one query
 #pragma unroll
-    for (int u = 0; u < U; ++u)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        sts_f32(s_dst[u][e] + stage, s[u][e]);
-        sts_f32(s_dst[u][e] + stage + 32 * SP, s[u][2 + e]);
+      for (int u = 0; u < U; ++u) {
+        sts_f32x2(s_dst[u][0] + stage, s[u][0], s[u][1]);
+        sts_f32x2(s_dst[u][0] + stage + 32 * SP, s[u][2], s[u][3]);
       }
+    } else {
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          sts_f32(s_dst[u][e] + stage, s[u][e]);
+          sts_f32(s_dst[u][e] + stage + 32 * SP, s[u][2 + e]);
+        }
+    }
   };
 
   // MASK: some key of the page is hidden from some query. MAX: only the maxima, into l. REF: c is not zero.

@@ -254,7 +254,8 @@ def test_router_takes_the_largest_logits_and_weighs_those_alone(dev, dt):
 
 
 ATTENTION = [(6, 2, 24, 40, 37, 5), (4, 4, 64, 16, 16, 16), (2, 1, 72, 128, 50, 33), (12, 4, 16, 24, 21, 0), (3, 3, 128, 8, 33, 1), (16, 4, 128, 128, 100, 7),
-             (32, 8, 128, 128, 64, 40), (40, 8, 64, 64, 30, 3), (64, 2, 32, 16, 45, 20), (3, 1, 9, 13, 7, 2), (1, 1, 136, 40, 1, 20), (70, 7, 16, 8, 20, 17), (5, 5, 64, 128, 0, 0)]
+             (32, 8, 128, 128, 64, 40), (40, 8, 64, 64, 30, 3), (64, 2, 32, 16, 45, 20), (3, 1, 9, 13, 7, 2), (1, 1, 136, 40, 1, 20), (70, 7, 16, 8, 20, 17), (5, 5, 64, 128, 0, 0),
+             (64, 8, 128, 128, 33, 18), (24, 8, 128, 128, 17, 3), (8, 2, 128, 128, 90, 32), (24, 8, 64, 64, 40, 1), (64, 8, 64, 64, 16, 0), (16, 4, 64, 64, 70, 48)]
 
 
 def loud_inputs(H, G, dk, dv, edges, T):
