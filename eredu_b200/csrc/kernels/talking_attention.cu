@@ -898,7 +898,7 @@ __global__ void __launch_bounds__(32 * kPromptWarps, 1) talking_prompt_kernel(Ta
 
 // How a run of queries is cut for the kernel above; qt = 0: it does not take the sizes.
 struct PromptPlan {
-  int qt = 0, octets = 0, warps = 0, smem = 0, blocks = 0, per = 0;   // per: products of the mix step a warp takes
+  int qt = 0, octets = 0, warps = 0, smem = 0, blocks = 0, per = 0, stages = 0;   // per: products of the mix step a warp takes
 };
 static PromptPlan prompt_plan(int H, int G, int dk, int dv, int rows, float softcap) {
   PromptPlan best;
@@ -947,15 +947,16 @@ struct PromptTcLayout {
   int columns;                            // of a key / value head, whole octets
   int p_head, p_bytes, kv_bytes, half;    // probabilities of a head (64 bytes apart from whole rows of banks), of a page; keys of a page, 64 dims of them
   int v_off, k_off, s_off, p_off, ref_off, sum_off, total;
-  __host__ __device__ __forceinline__ PromptTcLayout(int H, int G, int qt, int octets) : t(H, G, kTcHead, kTcHead, qt) {
+  // k_stages, v_stages: pages of keys and of values that fit
+  __host__ __device__ __forceinline__ PromptTcLayout(int H, int G, int qt, int octets, int k_stages, int v_stages) : t(H, G, kTcHead, kTcHead, qt) {
     columns = octets * 8;
     p_head = columns * 32 + 64;
     p_bytes = G * p_head;
     half = G * kPage * 128;
     kv_bytes = 2 * half;
     v_off = 0;                            // 1024-byte aligned
-    k_off = 2 * kv_bytes;
-    s_off = k_off + 2 * kv_bytes;
+    k_off = v_stages * kv_bytes;
+    s_off = k_off + k_stages * kv_bytes;
     p_off = s_off + 2 * t.s_bytes;
     ref_off = p_off + 2 * p_bytes;
     sum_off = ref_off + qt * t.hp * 4;
@@ -987,8 +988,8 @@ __device__ __forceinline__ float2 lds_f32x2(uint32_t addr) {
 // Queries of a CTA: with HB blocks of 16 heads, 256 rows of a (query, head) pair.
 constexpr int tc_queries(int hb) { return 16 / hb; }
 
-// W warps, of which each takes NT products of the mix step, and one that starts the copies and the sums. tm_k, tm_v: the caches as rows of 128, boxes of 64 columns and a page's rows.
-template <int HB, int W>
+// W warps, of which each takes NT products of the mix step, and one that starts the copies and the sums. NK, NV: stages of keys and values. tm_k, tm_v: the caches as rows of 128, boxes of 64 columns and a page's rows.
+template <int HB, int W, int NK, int NV>
 __global__ void __launch_bounds__(32 * (W + 1), 1)
 talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, TalkParams p) {
   using bf16 = __nv_bfloat16;
@@ -997,10 +998,10 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ int far_row;
   __shared__ uint32_t tmem_slot;
-  __shared__ __align__(8) uint64_t k_full[2], v_full[2], done[2];       // of a page of this parity: keys, values are there, its sums complete
+  __shared__ __align__(8) uint64_t k_full[NK], v_full[NV], step[2], done[2];
   pdl_launch_early();
   uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
-  const PromptTcLayout lay(p.H, p.G, QT, p.octets);
+  const PromptTcLayout lay(p.H, p.G, QT, p.octets, NK, NV);
   const int tid = threadIdx.x, lane = tid & 31, quad = lane & 3, oct = lane >> 2, gw = tid >> 5;
   const int b = blockIdx.y, r = p.H / p.G, columns = QT * r;
   float* ref = reinterpret_cast<float*>(smem + lay.ref_off);            // -c of every (query, head)
@@ -1032,9 +1033,10 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     tmem_relinquish();
   }
   if (tid == 32) {
+    for (int i = 0; i < NK; ++i) mbar_init(&k_full[i], 1);
+    for (int i = 0; i < NV; ++i) mbar_init(&v_full[i], 1);
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&k_full[i], 1);
-      mbar_init(&v_full[i], 1);
+      mbar_init(&step[i], W);
       mbar_init(&done[i], 1);
     }
     fence_mbar_init();
@@ -1090,11 +1092,11 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   const float cap_m2c = -2.f * p.softcap * kLog2e, cap_c = p.softcap * kLog2e, cap_in = 2.f * kLog2e * p.scale / p.softcap;
 
   float l[NT][HB][2];
-  auto score = [&](int buf) {
+  auto score = [&](int from, int buf) {
     float s[U][4];
 #pragma unroll
     for (int u = 0; u < U; ++u) s[u][0] = s[u][1] = s[u][2] = s[u][3] = 0.f;
-    const uint32_t base = k_addr + buf * kv_stage;
+    const uint32_t base = k_addr + from * kv_stage;
     uint32_t a[KS][4];
 #pragma unroll
     for (int k = 0; k < KS; ++k) ldsm_x4((base + (k >> 2) * lay.half) ^ ((k & 3) << 5), a[k][0], a[k][1], a[k][2], a[k][3]);
@@ -1125,7 +1127,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
   };
 
   // MASK: some key of the page is hidden from some query. MAX: only the maxima, into l. REF: c is not zero.
-  auto mix = [&](int buf, int key0, auto masked, auto maxima, auto refs) {
+  auto mix = [&](int buf, int p_buf, int key0, auto masked, auto maxima, auto refs) {
     constexpr bool MASK = decltype(masked)::value, MAX = decltype(maxima)::value, REF = decltype(refs)::value;
     float acc[NT][HB][4];
 #pragma unroll
@@ -1135,7 +1137,7 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
         acc[j][h][0] = acc[j][h][1] = REF ? ref[((gw + j * W) >> 1) * HP + h * 16 + oct] : 0.f;
         acc[j][h][2] = acc[j][h][3] = REF ? ref[((gw + j * W) >> 1) * HP + h * 16 + 8 + oct] : 0.f;
       }
-    const uint32_t s_stage = buf * S_STAGE, stage = buf * p_stage;
+    const uint32_t s_stage = buf * S_STAGE, stage = p_buf * p_stage;
 #pragma unroll
     for (int e = 0; e < HB; ++e) {
       uint32_t bf[NT][3][2];
@@ -1193,103 +1195,105 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     }
   };
 
-  // ---- pages. Iteration i: scores of page i + 1, mixing of page i, while the tensor cores sum up page i - 1; keys are fetched two pages ahead,
-  // values one. What an iteration writes was read before the barrier in front of it, or by the sums of page i - 2, which it waits for. One thread
-  // of the last warp starts the copies and the sums.
+  // ---- pages. In step i the W warps form the scores of page i + 1 and mix those of page i, in either order; a barrier of theirs ends it. The
+  // last warp's thread sums up page i once all have arrived on `step`, then fetches keys into the stage step i has read (page i + 1) and
+  // values into that of page i - 1. Probabilities of page i take the place of page i - 2 and wait for its sums (`done`). Every pass over the
+  // pages completes each of these barriers once per page of keys (values: only where there are sums), whose running numbers give parities.
   const uint32_t idesc = umma_idesc_bf16(D, lay.columns) | (1u << 15);  // A is MN-major
   bool ok = true;
-  uint32_t phase = 0;                                                   // parities of the next waits: bits 0, 1 done, 2, 3 k_full, 4, 5 v_full
-  auto wait_for = [&](uint64_t* bar, int bit, int code) {
-    if (ok) ok = mbar_wait(bar, (phase >> bit) & 1, p.status, code);
-    phase ^= 1u << bit;
+  int k_base = 0, v_base = 0;
+  auto wait_for = [&](uint64_t* bar, int parity, int code) {
+    if (ok) ok = mbar_wait(bar, parity & 1, p.status, code);
   };
-  auto wait_sums = [&](int i) { wait_for(&done[i & 1], i & 1, 3); };
-  auto page_row = [&](int i) { return bt[pages.at(min(i, n - 1))] * (p.G * kPage); };
-  auto load = [&](const CUtensorMap* map, uint64_t* bar, int off, int i, int page_row) {
-    uint8_t* dst = smem + off + (i & 1) * kv_stage;
-    mbar_arrive_expect_tx(&bar[i & 1], kv_stage);
-    tma_load_2d(dst, map, 0, page_row, &bar[i & 1]);
-    tma_load_2d(dst + lay.half, map, 64, page_row, &bar[i & 1]);
+  auto load = [&](const CUtensorMap* map, uint64_t* bar, uint8_t* dst, int page) {
+    const int page_row = page * (p.G * kPage);
+    mbar_arrive_expect_tx(bar, kv_stage);
+    tma_load_2d(dst, map, 0, page_row, bar);
+    tma_load_2d(dst + lay.half, map, 64, page_row, bar);
   };
-  auto sum_up = [&](int i) {                                            // O^T += V^T P^T of page i
-    wait_for(&v_full[i & 1], 4 + (i & 1), 1);
-    tc_fence_after_sync();
-    for (int h = 0; h < p.G; ++h)
-      umma_f16(tmem + h * lay.columns, umma_desc_mn_rows(vs_a + (i & 1) * kv_stage + h * (kPage * 128), lay.half),
-               umma_desc_k_core(ps_a + (i & 1) * p_stage + h * lay.p_head), idesc, i > 0 ? 1u : 0u);
-    umma_commit(&done[i & 1]);
+  auto load_k = [&](int i) {
+    const int st = (k_base + i) % NK;
+    if (i < n) load(&tm_k, &k_full[st], smem + lay.k_off + st * kv_stage, bt[pages.at(i)]);
   };
+  auto load_v = [&](int i) {
+    const int st = (v_base + i) % NV;
+    if (i < n) load(&tm_v, &v_full[st], smem + lay.v_off + st * kv_stage, bt[pages.at(i)]);
+  };
+  auto wait_sums = [&](int i) { wait_for(&done[(k_base + i) & 1], (k_base + i) >> 1, 3); };
   using Yes = std::true_type;
   using No = std::false_type;
   auto walk = [&](auto maxima, auto refs) {
     constexpr bool MAX = decltype(maxima)::value, REF = decltype(refs)::value;
-    auto score_at = [&](int i) {
-      if (i >= n) return;
-      wait_for(&k_full[i & 1], 2 + (i & 1), 1);
-      score(i & 1);
-    };
-    int at0 = 0, at1 = 0, at2 = 0;                                      // rows of pages i, i + 1, i + 2
     if (works) {
-      score_at(0);
-    } else if (lane == 0) {
-      at0 = page_row(0);
-      at1 = page_row(1);
-      at2 = page_row(2);
-      load(&tm_k, k_full, lay.k_off, 0, at0);
-      if (n > 1) load(&tm_k, k_full, lay.k_off, 1, at1);
-      if (!MAX) load(&tm_v, v_full, lay.v_off, 0, at0);
-    }
-    __syncthreads();
-    for (int i = 0; i < n; ++i) {
-      if (works) {
-        const int cur = i & 1, key0 = pages.at(i) * kPage;
-        const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep);
+      int st = k_base % NK, parity = k_base / NK;
+      auto score_next = [&](int buf) {
+        wait_for(&k_full[st], parity, 1);
+        score(st, buf);
+        if (++st == NK) {
+          st = 0;
+          ++parity;
+        }
+      };
+      score_next(0);
+      group_sync(1, 32 * W);
+      for (int i = 0; i < n; ++i) {
+        const int cur = i & 1, p_buf = (k_base + i) & 1, key0 = pages.at(i) * kPage;
+        const bool inner = key0 + kPage - 1 <= p0 && (p.window <= 0 || p1 - key0 < p.window || key0 + kPage <= p.keep), more = i + 1 < n;
         if constexpr (MAX || REF) {
-          score_at(i + 1);
-          if (!MAX && i > 1) wait_sums(i - 2);
-          if (mixes) mix(cur, key0, Yes(), maxima, refs);
+          if (more) score_next(cur ^ 1);
+          if (i > 1) wait_sums(i - 2);
+          if (mixes) mix(cur, p_buf, key0, Yes(), maxima, refs);
         } else if (gw < W / 2) {
-          score_at(i + 1);
+          if (more) score_next(cur ^ 1);
           if (i > 1) wait_sums(i - 2);
           if (mixes) {
-            if (inner) mix(cur, key0, No(), No(), No());
-            else mix(cur, key0, Yes(), No(), No());
+            if (inner) mix(cur, p_buf, key0, No(), No(), No());
+            else mix(cur, p_buf, key0, Yes(), No(), No());
           }
         } else {
           if (i > 1) wait_sums(i - 2);
           if (mixes) {
-            if (inner) mix(cur, key0, No(), No(), No());
-            else mix(cur, key0, Yes(), No(), No());
+            if (inner) mix(cur, p_buf, key0, No(), No(), No());
+            else mix(cur, p_buf, key0, Yes(), No(), No());
           }
-          score_at(i + 1);
+          if (more) score_next(cur ^ 1);
         }
         fence_proxy_async_smem();
-      } else if (lane == 0) {
-        const int at3 = page_row(i + 3);
-        if (i + 2 < n) load(&tm_k, k_full, lay.k_off, i + 2, at2);
-        if (!MAX && i > 0) {
-          sum_up(i - 1);
-          if (i > 1) wait_sums(i - 2);
-          load(&tm_v, v_full, lay.v_off, i, at0);
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&step[p_buf]);
+        group_sync(1, 32 * W);
+      }
+    } else if (lane == 0) {
+      for (int i = 0; i < NK; ++i) load_k(i);
+      if (!MAX)
+        for (int i = 0; i < NV; ++i) load_v(i);
+      for (int i = 0; i < n; ++i) {
+        const int buf = (k_base + i) & 1, sv = (v_base + i) % NV;
+        wait_for(&step[buf], (k_base + i) >> 1, 2);
+        if constexpr (MAX) {
+          mbar_arrive(&done[buf]);
+        } else {                                                        // O^T += V^T P^T of page i
+          wait_for(&v_full[sv], (v_base + i) / NV, 1);
+          tc_fence_after_sync();
+          for (int h = 0; h < p.G; ++h)
+            umma_f16(tmem + h * lay.columns, umma_desc_mn_rows(vs_a + sv * kv_stage + h * (kPage * 128), lay.half),
+                     umma_desc_k_core(ps_a + buf * p_stage + h * lay.p_head), idesc, i > 0 ? 1u : 0u);
+          umma_commit(&done[buf]);
         }
-        at0 = at1;
-        at1 = at2;
-        at2 = at3;
+        if (i == 0) load_k(NK);
+        load_k(i + 1 + NK);
+        if (!MAX && i > 0) {
+          wait_sums(i - 1);
+          load_v(i - 1 + NV);
+        }
       }
-      __syncwarp();
-      tc_fence_before_sync();
-      __syncthreads();
     }
-    if constexpr (!MAX) {
-      if (gw == W && lane == 0) sum_up(n - 1);
-      __syncwarp();
-      if (gw < W || lane == 0) {
-        if (n > 1) wait_sums(n - 2);
-        wait_sums(n - 1);
-      }
-      __syncwarp();
-      tc_fence_after_sync();
-    }
+    __syncwarp();
+    if (works || lane == 0) wait_sums(n - 1);
+    __syncwarp();
+    tc_fence_after_sync();
+    k_base += n;
+    if (!MAX) v_base += n;
   };
   // the l of all threads, by keys of the two halves of a page
   auto spread = [&](auto maxima) {
@@ -1378,22 +1382,28 @@ static PromptPlan prompt_tc_plan(int H, int G, int dk, int dv, float softcap) {
   const int qt = tc_queries(t.blocks);
   t.octets = ((qt * (H / G) + 7) / 8 + kTcUnits - 1) / kTcUnits * kTcUnits;
   t.warps = G * t.octets / kTcUnits;
-  const PromptTcLayout lay(H, G, qt, t.octets);
-  t.smem = lay.total + 1024;
-  // octets * 8 columns are the N of a product; a page's rows are one box
-  if ((t.warps == 8 || t.warps == 16) && t.octets <= 32 && G * kPage <= 256 && lay.t.hp == 16 * t.blocks && t.smem <= kSmemLimit - 256) t.qt = qt;
+  for (int stages : {4, 3}) {             // of keys; values have as many, or two where the keys have three
+    const PromptTcLayout lay(H, G, qt, t.octets, stages, stages == 4 ? 4 : 2);
+    t.smem = lay.total + 1024;
+    t.stages = stages;
+    // octets * 8 columns are the N of a product; a page's rows are one box
+    if ((t.warps == 8 || t.warps == 16) && t.octets <= 32 && G * kPage <= 256 && lay.t.hp == 16 * t.blocks && t.smem <= kSmemLimit - 256) {
+      t.qt = qt;
+      break;
+    }
+  }
   return t;
 }
 
-template <int HB, int W>
+template <int HB, int W, int NK, int NV>
 static cudaError_t launch_prompt_tc(const CUtensorMap& tm_k, const CUtensorMap& tm_v, const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, W>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_tc_kernel<HB, W, NK, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_tc_kernel<HB, W>, grid, dim3((W + 1) * 32), t.smem, stream, tm_k, tm_v, p);
+  return launch_pdl(talking_prompt_tc_kernel<HB, W, NK, NV>, grid, dim3((W + 1) * 32), t.smem, stream, tm_k, tm_v, p);
 }
 // A cudaError_t, or a negative number where a tensor map cannot be made.
 static int launch_prompt_tc(const TalkParams& p, int pages, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
@@ -1404,10 +1414,11 @@ static int launch_prompt_tc(const TalkParams& p, int pages, dim3 grid, const Pro
   r = make_tma_2d(&tm_v, p.v_cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, kTcHead, kTcHead, p.G * kPage, 64);
   if (r != 0) return -200 - r;
   cudaError_t e;
-#define ER_TC(HB_) t.warps == 8 ? launch_prompt_tc<HB_, 8>(tm_k, tm_v, p, grid, t, stream) : launch_prompt_tc<HB_, 16>(tm_k, tm_v, p, grid, t, stream)
-  if (t.blocks == 1) e = ER_TC(1);
-  else if (t.blocks == 2) e = ER_TC(2);
-  else e = ER_TC(4);
+#define ER_TC(HB_, W_) \
+  (t.stages == 4 ? launch_prompt_tc<HB_, W_, 4, 4>(tm_k, tm_v, p, grid, t, stream) : launch_prompt_tc<HB_, W_, 3, 2>(tm_k, tm_v, p, grid, t, stream))
+  if (t.blocks == 1) e = t.warps == 8 ? ER_TC(1, 8) : ER_TC(1, 16);
+  else if (t.blocks == 2) e = t.warps == 8 ? ER_TC(2, 8) : ER_TC(2, 16);
+  else e = t.warps == 8 ? ER_TC(4, 8) : ER_TC(4, 16);
 #undef ER_TC
   return static_cast<int>(e);
 }
