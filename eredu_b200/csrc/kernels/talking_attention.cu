@@ -988,17 +988,18 @@ __device__ __forceinline__ float2 lds_f32x2(uint32_t addr) {
 // Queries of a CTA: with HB blocks of 16 heads, 256 rows of a (query, head) pair.
 constexpr int tc_queries(int hb) { return 16 / hb; }
 
-// W warps, of which each takes NT products of the mix step, and one that starts the copies and the sums. NK, NV: stages of keys and values. tm_k, tm_v: the caches as rows of 128, boxes of 64 columns and a page's rows.
+// W warps, of which each takes NT products of the mix step, and three that start the copies of keys, those of values, and the sums. NK, NV:
+// stages of keys and values. tm_k, tm_v: the caches as rows of 128, boxes of 64 columns and a page's rows.
 template <int HB, int W, int NK, int NV>
-__global__ void __launch_bounds__(32 * (W + 1), 1)
+__global__ void __launch_bounds__(32 * (W + 3), 1)
 talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, TalkParams p) {
   using bf16 = __nv_bfloat16;
-  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, QT = tc_queries(HB), THREADS = 32 * (W + 1);
+  constexpr int D = kTcHead, U = kTcUnits, KS = D / 16, QT = tc_queries(HB), THREADS = 32 * (W + 3);
   constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4, S_STAGE = QT * SQ * 4, NT = 2 * QT > W ? 2 * QT / W : 1;
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __shared__ int far_row;
   __shared__ uint32_t tmem_slot;
-  __shared__ __align__(8) uint64_t k_full[NK], v_full[NV], step[2], done[2];
+  __shared__ __align__(8) uint64_t k_full[NK], k_free[NK], v_full[NV], v_free[NV], step[2], done[2];
   pdl_launch_early();
   uint8_t* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
   const PromptTcLayout lay(p.H, p.G, QT, p.octets, NK, NV);
@@ -1033,8 +1034,14 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     tmem_relinquish();
   }
   if (tid == 32) {
-    for (int i = 0; i < NK; ++i) mbar_init(&k_full[i], 1);
-    for (int i = 0; i < NV; ++i) mbar_init(&v_full[i], 1);
+    for (int i = 0; i < NK; ++i) {
+      mbar_init(&k_full[i], 1);
+      mbar_init(&k_free[i], W);
+    }
+    for (int i = 0; i < NV; ++i) {
+      mbar_init(&v_full[i], 1);
+      mbar_init(&v_free[i], 1);
+    }
     for (int i = 0; i < 2; ++i) {
       mbar_init(&step[i], W);
       mbar_init(&done[i], 1);
@@ -1195,29 +1202,24 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     }
   };
 
-  // ---- pages. In step i the W warps form the scores of page i + 1 and mix those of page i, in either order; a barrier of theirs ends it. The
-  // last warp's thread sums up page i once all have arrived on `step`, then fetches keys into the stage step i has read (page i + 1) and
-  // values into that of page i - 1. Probabilities of page i take the place of page i - 2 and wait for its sums (`done`). Every pass over the
-  // pages completes each of these barriers once per page of keys (values: only where there are sums), whose running numbers give parities.
+  // ---- pages. In step i the W warps form the scores of page i + 1 and mix those of page i, in either order; a barrier of theirs ends it.
+  // Three threads run beside them: keys are fetched as stages become free of scores, values as they become free of sums, and page i is summed
+  // up once all warps have arrived on `step`. Probabilities of page i take the place of page i - 2 and wait for its sums (`done`). Every pass
+  // over the pages completes each of these barriers once per page (values: only where there are sums); running numbers give parities.
   const uint32_t idesc = umma_idesc_bf16(D, lay.columns) | (1u << 15);  // A is MN-major
   bool ok = true;
   int k_base = 0, v_base = 0;
   auto wait_for = [&](uint64_t* bar, int parity, int code) {
     if (ok) ok = mbar_wait(bar, parity & 1, p.status, code);
   };
-  auto load = [&](const CUtensorMap* map, uint64_t* bar, uint8_t* dst, int page) {
-    const int page_row = page * (p.G * kPage);
-    mbar_arrive_expect_tx(bar, kv_stage);
-    tma_load_2d(dst, map, 0, page_row, bar);
-    tma_load_2d(dst + lay.half, map, 64, page_row, bar);
-  };
-  auto load_k = [&](int i) {
-    const int st = (k_base + i) % NK;
-    if (i < n) load(&tm_k, &k_full[st], smem + lay.k_off + st * kv_stage, bt[pages.at(i)]);
-  };
-  auto load_v = [&](int i) {
-    const int st = (v_base + i) % NV;
-    if (i < n) load(&tm_v, &v_full[st], smem + lay.v_off + st * kv_stage, bt[pages.at(i)]);
+  // page i into its stage, the pages before it counted by `base`
+  auto load = [&](const CUtensorMap* map, uint64_t* full, uint64_t* empty, int off, int stages, int x, int page) {
+    const int st = x % stages, page_row = page * (p.G * kPage);
+    uint8_t* dst = smem + off + st * kv_stage;
+    if (x >= stages) wait_for(&empty[st], x / stages - 1, 2);
+    mbar_arrive_expect_tx(&full[st], kv_stage);
+    tma_load_2d(dst, map, 0, page_row, &full[st]);
+    tma_load_2d(dst + lay.half, map, 64, page_row, &full[st]);
   };
   auto wait_sums = [&](int i) { wait_for(&done[(k_base + i) & 1], (k_base + i) >> 1, 3); };
   using Yes = std::true_type;
@@ -1229,6 +1231,8 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
       auto score_next = [&](int buf) {
         wait_for(&k_full[st], parity, 1);
         score(st, buf);
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&k_free[st]);
         if (++st == NK) {
           st = 0;
           ++parity;
@@ -1263,28 +1267,38 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
         if (lane == 0) mbar_arrive(&step[p_buf]);
         group_sync(1, 32 * W);
       }
+    } else if (lane == 0 && gw == W) {
+      int page = bt[pages.at(0)];
+      for (int i = 0; i < n; ++i) {
+        const int next = i + 1 < n ? bt[pages.at(i + 1)] : 0;
+        load(&tm_k, k_full, k_free, lay.k_off, NK, k_base + i, page);
+        page = next;
+      }
+    } else if (lane == 0 && gw == W + 1) {
+      int page = MAX ? 0 : bt[pages.at(0)];
+      for (int i = 0; !MAX && i < n; ++i) {
+        const int next = i + 1 < n ? bt[pages.at(i + 1)] : 0;
+        load(&tm_v, v_full, v_free, lay.v_off, NV, v_base + i, page);
+        page = next;
+      }
     } else if (lane == 0) {
-      for (int i = 0; i < NK; ++i) load_k(i);
-      if (!MAX)
-        for (int i = 0; i < NV; ++i) load_v(i);
+      const uint64_t a_desc = umma_desc_mn_rows(vs_a, lay.half), b_desc = umma_desc_k_core(ps_a);
       for (int i = 0; i < n; ++i) {
         const int buf = (k_base + i) & 1, sv = (v_base + i) % NV;
+        if constexpr (!MAX) wait_for(&v_full[sv], (v_base + i) / NV, 1);
         wait_for(&step[buf], (k_base + i) >> 1, 2);
         if constexpr (MAX) {
           mbar_arrive(&done[buf]);
         } else {                                                        // O^T += V^T P^T of page i
-          wait_for(&v_full[sv], (v_base + i) / NV, 1);
           tc_fence_after_sync();
-          for (int h = 0; h < p.G; ++h)
-            umma_f16(tmem + h * lay.columns, umma_desc_mn_rows(vs_a + sv * kv_stage + h * (kPage * 128), lay.half),
-                     umma_desc_k_core(ps_a + buf * p_stage + h * lay.p_head), idesc, i > 0 ? 1u : 0u);
+          uint64_t a = a_desc + ((sv * kv_stage) >> 4), b = b_desc + ((buf * p_stage) >> 4);
+          for (int h = 0; h < p.G; ++h) {
+            umma_f16(tmem + h * lay.columns, a, b, idesc, i > 0 ? 1u : 0u);
+            a += (kPage * 128) >> 4;
+            b += lay.p_head >> 4;
+          }
           umma_commit(&done[buf]);
-        }
-        if (i == 0) load_k(NK);
-        load_k(i + 1 + NK);
-        if (!MAX && i > 0) {
-          wait_sums(i - 1);
-          load_v(i - 1 + NV);
+          umma_commit(&v_free[sv]);
         }
       }
     }
@@ -1403,7 +1417,7 @@ static cudaError_t launch_prompt_tc(const CUtensorMap& tm_k, const CUtensorMap& 
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_tc_kernel<HB, W, NK, NV>, grid, dim3((W + 1) * 32), t.smem, stream, tm_k, tm_v, p);
+  return launch_pdl(talking_prompt_tc_kernel<HB, W, NK, NV>, grid, dim3((W + 3) * 32), t.smem, stream, tm_k, tm_v, p);
 }
 // A cudaError_t, or a negative number where a tensor map cannot be made.
 static int launch_prompt_tc(const TalkParams& p, int pages, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
