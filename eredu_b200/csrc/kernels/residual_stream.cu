@@ -455,6 +455,16 @@ __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidual
         v[i] = make_float4(fmaf(w, a.x, v[i].x), fmaf(w, a.y, v[i].y), fmaf(w, a.z, v[i].z), fmaf(w, a.w, v[i].w));
       }
     }
+    // the first rows of the history travel while the sum is formed
+    constexpr int AHEAD = NV <= 4 ? 3 : 0;
+    float4 past[NV][AHEAD > 0 ? AHEAD : 1];
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+#pragma unroll
+      for (int j = 0; j < AHEAD; ++j) {
+        const int c = (threadIdx.x + i * 256) * 4;
+        if (hist != nullptr && c < W && j < p.n_taps - 1) past[i][j] = load4(hist + static_cast<size_t>(j) * W + c);
+      }
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
@@ -470,14 +480,18 @@ __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidual
       if (act == nullptr) continue;
       float4 h = o;
       if (p.taps != nullptr) {
-        for (int j = 0; j < p.n_taps; ++j) {
+        auto tap = [&](int j, const float4& u) {
           const float4 t = load4(p.taps + static_cast<size_t>(j) * W + c);
-          const bool own = j == p.n_taps - 1;
-          if (!own && hist == nullptr) continue;
-          const float4 u = own ? o : load4(hist + static_cast<size_t>(j) * W + c);
           if (j > 0 && hist != nullptr) store4(hist + static_cast<size_t>(j - 1) * W + c, u);
           h = make_float4(fmaf(t.x, u.x, h.x), fmaf(t.y, u.y, h.y), fmaf(t.z, u.z, h.z), fmaf(t.w, u.w, h.w));
+        };
+        if (hist != nullptr) {
+#pragma unroll
+          for (int j = 0; j < AHEAD; ++j)
+            if (j < p.n_taps - 1) tap(j, past[i][j]);
+          for (int j = AHEAD; j < p.n_taps - 1; ++j) tap(j, load4(hist + static_cast<size_t>(j) * W + c));
         }
+        tap(p.n_taps - 1, o);
       }
       store4(act + c, h);
     }
@@ -650,9 +664,14 @@ __global__ void __launch_bounds__(256) embedding_stream_kernel(const int* __rest
   };
   if (inv_freq != nullptr) {
     const float pos = static_cast<float>(positions[blockIdx.x]);
-    for (int i = threadIdx.x; 2 * i < W; i += 256) {
+    for (int i = blockIdx.y * 256 + threadIdx.x; 2 * i < W; i += 256 * gridDim.y) {
       float sn, cs;
       sincosf(pos * inv_freq[i], &sn, &cs);
+      if (W % 2 == 0 && act == nullptr) {
+        const float u = ok ? to_f32(src[2 * i]) * scale : 0.f, v = ok ? to_f32(src[2 * i + 1]) * scale : 0.f;
+        *reinterpret_cast<float2*>(x + base + 2 * i) = make_float2(u + sn, v + cs);
+        continue;
+      }
       put(2 * i, sn);
       if (2 * i + 1 < W) put(2 * i + 1, cs);
     }
@@ -836,9 +855,11 @@ extern "C" int eredu_embedding_stream(const int* ids, const void* table, float* 
                                       int M, int W, int rows, int fp32, float scale, cudaStream_t stream) {
   if (M <= 0 || W <= 0) return 0;
   cudaError_t e;
-  if (fp32) e = launch_pdl(embedding_stream_kernel<float>, dim3(M), dim3(256), 0, stream, ids, static_cast<const float*>(table), x,
+  // few rows: a sine and a cosine per thread
+  const dim3 grid(M, inv_freq != nullptr && M <= 512 ? ((W + 1) / 2 + 255) / 256 : 1);
+  if (fp32) e = launch_pdl(embedding_stream_kernel<float>, grid, dim3(256), 0, stream, ids, static_cast<const float*>(table), x,
                            static_cast<float*>(act), positions, inv_freq, W, rows, scale);
-  else e = launch_pdl(embedding_stream_kernel<__nv_bfloat16>, dim3(M), dim3(256), 0, stream, ids,
+  else e = launch_pdl(embedding_stream_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, ids,
                       static_cast<const __nv_bfloat16*>(table), x, static_cast<__nv_bfloat16*>(act), positions, inv_freq, W, rows, scale);
   eredu_count_launches(1);
   return static_cast<int>(e);

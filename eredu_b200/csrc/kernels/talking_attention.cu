@@ -1106,11 +1106,14 @@ talking_prompt_tc_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_
     const uint32_t base = k_addr + from * kv_stage;
     uint32_t a[KS][4];
 #pragma unroll
-    for (int k = 0; k < KS; ++k) ldsm_x4((base + (k >> 2) * lay.half) ^ ((k & 3) << 5), a[k][0], a[k][1], a[k][2], a[k][3]);
+    for (int k = 0; k < KS / 2; ++k) ldsm_x4(base ^ (k << 5), a[k][0], a[k][1], a[k][2], a[k][3]);
 #pragma unroll
-    for (int k = 0; k < KS; ++k)
+    for (int k = 0; k < KS; ++k) {
+      const int f = k + KS / 2;                                         // fetched while step k is computed
+      if (f < KS) ldsm_x4((base + lay.half) ^ (k << 5), a[f][0], a[f][1], a[f][2], a[f][3]);
 #pragma unroll
       for (int u = 0; u < U; ++u) mma_pure(s[u], a[k][0], a[k][1], a[k][2], a[k][3], qf[u][k][0], qf[u][k][1]);
+    }
 #pragma unroll
     for (int u = 0; u < U; ++u)
 #pragma unroll
