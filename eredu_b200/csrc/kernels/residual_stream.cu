@@ -404,8 +404,8 @@ struct RoutedResidualParams {
 };
 
 // One CTA per row: x' = residual + weight rms(y + sum_k w_k rows_k). NV groups of four columns per thread stay in registers; NV = 0: any
-// width, the sum is formed twice.
-template <typename T, int NV>
+// width, the sum is formed twice. CONV: with the convolution.
+template <typename T, int NV, bool CONV>
 __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidualParams p) {
   __shared__ __align__(16) float red[8];
   __shared__ int pos[kMaxRoutes];
@@ -456,7 +456,7 @@ __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidual
       }
     }
     // the first rows of the history travel while the sum is formed
-    constexpr int AHEAD = NV <= 4 ? 3 : 0;
+    constexpr int AHEAD = CONV && NV <= 4 ? 3 : 0;
     float4 past[NV][AHEAD > 0 ? AHEAD : 1];
 #pragma unroll
     for (int i = 0; i < NV; ++i)
@@ -479,7 +479,7 @@ __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidual
       store4(p.x_out + base + c, o);
       if (act == nullptr) continue;
       float4 h = o;
-      if (p.taps != nullptr) {
+      if constexpr (CONV) {
         auto tap = [&](int j, const float4& u) {
           const float4 t = load4(p.taps + static_cast<size_t>(j) * W + c);
           if (j > 0 && hist != nullptr) store4(hist + static_cast<size_t>(j - 1) * W + c, u);
@@ -513,7 +513,7 @@ __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidual
       p.x_out[base + c] = o;
       if (act == nullptr) continue;
       float h = o;
-      if (p.taps != nullptr) {
+      if constexpr (CONV) {
         for (int j = 0; j < p.n_taps; ++j) {
           const bool own = j == p.n_taps - 1;
           if (!own && hist == nullptr) continue;
@@ -530,7 +530,9 @@ __global__ void __launch_bounds__(256) rms_routed_residual_kernel(RoutedResidual
 template <typename T>
 static cudaError_t launch_rms_routed_residual(const RoutedResidualParams& p, int M, bool quads_ok, cudaStream_t stream) {
   const int quads = quads_ok ? (p.W / 4 + 255) / 256 : 0;
-#define ER_RR(NV_) launch_pdl(rms_routed_residual_kernel<T, NV_>, dim3(M), dim3(256), 0, stream, p)
+#define ER_RR(NV_) \
+  (p.taps != nullptr ? launch_pdl(rms_routed_residual_kernel<T, NV_, true>, dim3(M), dim3(256), 0, stream, p) \
+                     : launch_pdl(rms_routed_residual_kernel<T, NV_, false>, dim3(M), dim3(256), 0, stream, p))
   switch (quads) {
     case 1: return ER_RR(1);
     case 2: return ER_RR(2);
