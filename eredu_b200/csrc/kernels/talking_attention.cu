@@ -10,11 +10,14 @@
 // stages deep. Prompts: one group of up to 16 warps and as many queries as fit its registers. Decode steps: several groups per CTA, each
 // with pages of its own, and the CTAs of a cluster share a sequence's keys; partial results meet in (distributed) shared memory.
 //
-// The kernel for prompts of the usual head sizes knows that exponents of fp32 and bf16 reach far: its mix step forms exp(S') itself, without
-// a maximum. In the rare case that some row's sum leaves 2^+-100 it finds the maxima in a pass of their own and starts over with
-// exp(S' - maximum). So O is never rescaled, and the three steps of three successive pages share one barrier.
+// Prompts of the usual head sizes have kernels of their own. They use that exponents of fp32 and bf16 reach far: the mix step forms exp(S')
+// itself, without a maximum. In the rare case that some row's sum leaves 2^+-100 they find the maxima in a pass of their own and start over
+// with exp(S' - maximum). So O is never rescaled, and the steps of successive pages overlap.
+//   heads of 64    as above, O in registers, four column octets per warp, the three steps of three pages behind one barrier
+//   heads of 128   O in tensor memory: the sums are tcgen05 products of values (by TMA) and probabilities in shared memory, and run beside
+//                  the scores of the next page and the mixing of this one
 //
-// A third kernel on the CUDA cores takes fp32, head sizes the first is not built for, and more than 64 heads.
+// The last kernel, on the CUDA cores, takes fp32, head sizes the others are not built for, and more than 64 heads.
 #include <algorithm>
 #include <type_traits>
 
@@ -566,14 +569,14 @@ struct PromptLayout {
   __host__ __device__ __forceinline__ int total() const { return t.talk() + 2 * (t.k_bytes + t.v_bytes + t.s_bytes + p_bytes) + refs(); }
 };
 
-// D: head size; HB blocks of 16 heads; NT (query, eight keys) products of the mix step per warp. A warp holds kUnits column octets of one
+// Heads of 64; HB blocks of 16 heads; NT (query, eight keys) products of the mix step per warp. A warp holds kUnits column octets of one
 // key / value head.
 constexpr int kUnits = 4, kPromptWarps = 8;
 
-template <int D, int HB, int NT>
+template <int HB, int NT>
 __global__ void __launch_bounds__(32 * kPromptWarps, 1) talking_prompt_kernel(TalkParams p) {
   using bf16 = __nv_bfloat16;
-  constexpr int U = kUnits, KS = D / 16, VT = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16;
+  constexpr int D = 64, U = kUnits, KS = D / 16, VT = D / 16, PIECES = D / 8, PITCH = (PIECES + 1) * 16;
   constexpr int HP = 16 * HB, SP = HP + 8, SQ = kPage * SP + 4, PP = PromptLayout::kProbPitch;
   extern __shared__ __align__(16) uint8_t smem[];
   __shared__ int far_row;
@@ -925,11 +928,11 @@ template <int HB, int NT>
 static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_kernel<64, HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
+    const cudaError_t e = cudaFuncSetAttribute(talking_prompt_kernel<HB, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit - 256);
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  return launch_pdl(talking_prompt_kernel<64, HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
+  return launch_pdl(talking_prompt_kernel<HB, NT>, grid, dim3(t.warps * 32), t.smem, stream, p);
 }
 static cudaError_t launch_prompt(const TalkParams& p, dim3 grid, const PromptPlan& t, cudaStream_t stream) {
   if (t.blocks == 1) return t.per <= 4 ? launch_prompt<1, 4>(p, grid, t, stream) : launch_prompt<1, 8>(p, grid, t, stream);
